@@ -28,6 +28,11 @@ def _load():
         _err = e
 
 
+def built() -> bool:
+    """Whether the shared objects are there (without loading them)."""
+    return any(_ROOT.glob("_C.*.so")) and (_ROOT / "lib" / "libb2kernels.so").exists()
+
+
 def available() -> bool:
     _load()
     return _C is not None

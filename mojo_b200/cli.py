@@ -1,9 +1,10 @@
-"""Command line: `python -m mojo_b200.cli {serve,generate,bench,bench-ops,deviceinfo}`.
+"""Command line: `python -m mojo_b200.cli {serve,generate,bench,bench-ops,replay,deviceinfo}`.
 
   serve       OpenAI-compatible HTTP server
   generate    run prompts (token ids, or text with --tokenizer) to completion and print the outputs
   bench       synthetic serving benchmark (Poisson or fixed-batch trace) with TTFT / ITL / tok/s; JSON (+CSV) out
   bench-ops   fused tensor-parallel op sweep (run under torch.distributed.run)
+  replay      feed a trace of token ids through a model and write logits (options as in mojo_b200/replay.py)
   deviceinfo  capability probe of the visible GPUs
 """
 from __future__ import annotations
@@ -151,6 +152,7 @@ def main(argv=None) -> None:
     b.set_defaults(fn=_cmd_bench)
     o = sub.add_parser("bench-ops", help="run as: python -m torch.distributed.run ... -m mojo_b200.bench_ops")
     o.set_defaults(fn=lambda a: print("launch with: python -m torch.distributed.run --nproc-per-node N -m mojo_b200.bench_ops"))
+    sub.add_parser("replay", help="trace of token ids in, logits out; options as in bin/trace_run --help")
     sub.add_parser("bench-kernels", help="micro-benchmarks of kernels and host runtime; options as in python -m mojo_b200.bench_kernels --help")
     d = sub.add_parser("deviceinfo")
     d.set_defaults(fn=_cmd_deviceinfo)
@@ -162,6 +164,10 @@ def main(argv=None) -> None:
 
         bench_kernels.main(args[1:])
         return
+    if args and args[0] == "replay":
+        from . import replay
+
+        sys.exit(replay.main(args[1:]))
     a = ap.parse_args(args)
     a.fn(a)
 

@@ -71,7 +71,8 @@ void bind_engine(py::module_& m) {
       .def_readonly("evictions", &KVStats::evictions);
 
   py::class_<KVCacheManager>(m, "KVCacheManager")
-      .def(py::init<int64_t, int, bool>(), py::arg("num_pages"), py::arg("page_size"), py::arg("enable_prefix_cache") = false)
+      .def(py::init<int64_t, int, bool, int64_t>(), py::arg("num_pages"), py::arg("page_size"), py::arg("enable_prefix_cache") = false,
+           py::arg("state_slots") = 0)
       .def_property_readonly("page_size", &KVCacheManager::page_size)
       .def_property_readonly("num_pages", &KVCacheManager::num_pages)
       .def("available_pages", &KVCacheManager::available_pages)
@@ -96,6 +97,9 @@ void bind_engine(py::module_& m) {
       .def("block_table", [](const KVCacheManager& k, int64_t id) { return to_array(k.block_table(id)); })
       .def("slot", &KVCacheManager::slot)
       .def("num_tokens_reserved", &KVCacheManager::num_tokens_reserved)
+      .def_property_readonly("state_slots", &KVCacheManager::state_slots)
+      .def("free_state_slots", &KVCacheManager::free_state_slots)
+      .def("advance_state", &KVCacheManager::advance_state)
       .def("stats", &KVCacheManager::stats)
       .def("check_invariants", &KVCacheManager::check_invariants);
 
@@ -121,6 +125,12 @@ void bind_engine(py::module_& m) {
                                a.resize({static_cast<py::ssize_t>(b.seq_ids.size()), static_cast<py::ssize_t>(b.max_blocks)});
                                return a;
                              })
+      .def_property_readonly("seq_state",
+                             [](const Batch& b) {
+                               auto a = to_array(b.seq_state);
+                               a.resize({static_cast<py::ssize_t>(b.seq_state.size() / 2), static_cast<py::ssize_t>(2)});
+                               return a;
+                             })
       .def_property_readonly("sample_rows", [](const Batch& b) { return to_array(b.sample_rows); })
       .def_property_readonly("sample_seq_ids", [](const Batch& b) { return to_array(b.sample_seq_ids); })
       .def_property_readonly("preempted", [](const Batch& b) { return to_array(b.preempted); })
@@ -140,6 +150,7 @@ void bind_engine(py::module_& m) {
            },
            py::arg("id"), py::arg("prompt"), py::arg("max_new_tokens"), py::arg("arrival") = 0.0)
       .def("step", &Scheduler::step)
+      .def("run_tokens", &Scheduler::run_tokens)
       .def("append_token", &Scheduler::append_token)
       .def("finish", &Scheduler::finish)
       .def("abort", &Scheduler::abort)

@@ -1,0 +1,233 @@
+// Bindings of the sequence-mixing kernels (b2/mixers.h): argument checks, then raw pointers on the current stream.
+#include <torch/extension.h>
+#include <c10/cuda/CUDAStream.h>
+#include <c10/cuda/CUDAGuard.h>
+#include "b2/launch.h"
+#include "b2/mixers.h"
+
+namespace py = pybind11;
+
+namespace {
+using OptTensor = c10::optional<at::Tensor>;
+
+cudaStream_t cur_stream() { return c10::cuda::getCurrentCUDAStream().stream(); }
+void check(int rc, const char* what) {
+  if (rc == 0) return;
+  if (b2::is_cuda_rc(rc)) {
+    const cudaError_t e = b2::cuda_error_of(rc);
+    throw std::runtime_error(std::string("mojo_b200: ") + what + " failed: CUDA error " + std::to_string(static_cast<int>(e)) + " (" +
+                             cudaGetErrorName(e) + ": " + cudaGetErrorString(e) + ")");
+  }
+  throw std::runtime_error(std::string("mojo_b200: ") + what + " rejected its arguments: " + b2::status_code_name(-rc));
+}
+void need(bool cond, const char* msg) {
+  if (!cond) throw std::invalid_argument(std::string("mojo_b200: ") + msg);
+}
+b2::Status* status_ptr(const OptTensor& s) { return s.has_value() ? reinterpret_cast<b2::Status*>(s->data_ptr()) : nullptr; }
+bool is_act(const at::Tensor& t) { return t.is_cuda() && (t.scalar_type() == at::kBFloat16 || t.scalar_type() == at::kFloat); }
+bool is_f32(const at::Tensor& t, int64_t n) { return t.is_cuda() && t.scalar_type() == at::kFloat && t.is_contiguous() && t.numel() == n; }
+bool is_i32(const at::Tensor& t) { return t.is_cuda() && t.scalar_type() == at::kInt && t.is_contiguous(); }
+bool is_i64(const at::Tensor& t) { return t.is_cuda() && t.scalar_type() == at::kLong && t.is_contiguous(); }
+template <typename P>
+P* opt(const OptTensor& t) { return t.has_value() ? static_cast<P*>(t->data_ptr()) : nullptr; }
+
+B2SeqRows seq_rows_of(const at::Tensor& row_seq, const at::Tensor& seq_rows, const at::Tensor& seq_state, int64_t banks) {
+  need(is_i32(row_seq) && is_i32(seq_rows) && is_i32(seq_state) && seq_rows.numel() == seq_state.numel() && seq_rows.numel() % 2 == 0,
+       "sequence rows: int32 row_seq [T], seq_rows [S, 2], seq_state [S, 2]");
+  B2SeqRows s{};
+  s.row_seq = row_seq.data_ptr<int32_t>();
+  s.seq_rows = seq_rows.data_ptr<int32_t>();
+  s.seq_state = seq_state.data_ptr<int32_t>();
+  s.rows = static_cast<int32_t>(row_seq.numel());
+  s.seqs = static_cast<int32_t>(seq_rows.numel() / 2);
+  s.banks = static_cast<int32_t>(banks);
+  return s;
+}
+
+void hyper_norm(at::Tensor& x, const OptTensor& y, const OptTensor& mix, const OptTensor& out, const OptTensor& in, const at::Tensor& weight,
+                at::Tensor& h, const OptTensor& ids, const OptTensor& embed, double embed_scale, const OptTensor& rows_index, bool store, double eps,
+                int64_t mean_width, const OptTensor& status) {
+  need(x.dim() == 3 && x.is_cuda() && x.scalar_type() == at::kFloat && x.is_contiguous(), "hyper_norm: x must be contiguous CUDA f32 [rows, streams, width]");
+  const int64_t T = x.size(0), S = x.size(1), W = x.size(2);
+  need(is_act(h) && h.dim() == 2 && h.is_contiguous() && h.size(1) == W && is_f32(weight, W), "hyper_norm: h [n, width], weight f32 [width]");
+  if (y.has_value()) {
+    need(y->scalar_type() == h.scalar_type() && y->is_contiguous() && y->numel() == T * W, "hyper_norm: y [rows, width] like h");
+    need(mix.has_value() && out.has_value() && is_f32(*mix, S * S) && is_f32(*out, S), "hyper_norm: mix [S, S] and out [S] f32");
+  }
+  if (in.has_value()) need(is_f32(*in, S), "hyper_norm: in f32 [S]");
+  if (ids.has_value())
+    need(is_i64(*ids) && ids->numel() == T && embed.has_value() && embed->scalar_type() == h.scalar_type() && embed->is_contiguous() && embed->size(1) == W,
+         "hyper_norm: ids int64 [rows], embed [vocab, width] like h");
+  if (rows_index.has_value()) need(is_i64(*rows_index) && rows_index->numel() == h.size(0), "hyper_norm: rows_index int64 [n]");
+  else need(h.size(0) == T, "hyper_norm: h must have one row per x row");
+  B2HyperArgs a{};
+  a.x = x.data_ptr<float>();
+  a.y = opt<const void>(y);
+  a.mix = opt<const float>(mix);
+  a.out = opt<const float>(out);
+  a.in = opt<const float>(in);
+  a.weight = weight.data_ptr<float>();
+  a.h = h.data_ptr();
+  a.ids = opt<const int64_t>(ids);
+  a.embed = opt<const void>(embed);
+  a.rows_index = opt<const int64_t>(rows_index);
+  a.embed_scale = static_cast<float>(embed_scale);
+  a.eps = static_cast<float>(eps);
+  a.n_out = static_cast<int32_t>(h.size(0));
+  a.rows = static_cast<int32_t>(T);
+  a.width = static_cast<int32_t>(W);
+  a.mean_width = static_cast<int32_t>(mean_width);
+  a.streams = static_cast<int32_t>(S);
+  a.vocab = embed.has_value() ? static_cast<int32_t>(embed->size(0)) : 0;
+  a.store = store ? 1 : 0;
+  c10::cuda::CUDAGuard g(x.device());
+  check(b2_hyper_norm(&a, h.scalar_type() == at::kFloat ? 1 : 0, status_ptr(status), cur_stream()), "hyper_norm");
+}
+
+void conv_qkv(const at::Tensor& proj, const at::Tensor& conv_w, const OptTensor& conv_state, const at::Tensor& cos_sin, const at::Tensor& positions,
+              const at::Tensor& row_seq, const at::Tensor& seq_rows, const at::Tensor& seq_state, int64_t banks, at::Tensor& q_out,
+              const OptTensor& slots, const OptTensor& k_cache, const OptTensor& v_cache, int64_t heads, int64_t kv_heads, int64_t dim, int64_t vdim,
+              double eps, const OptTensor& status) {
+  need(is_act(proj) && proj.dim() == 2 && proj.stride(1) == 1, "conv_qkv: proj must be 2-D with unit inner stride");
+  const int64_t T = proj.size(0), taps = conv_w.size(0), channels = heads * dim + kv_heads * (dim + vdim);
+  need(conv_w.dim() == 2 && is_f32(conv_w, taps * channels) && proj.size(1) >= channels, "conv_qkv: conv_w f32 [taps, channels], proj at least that wide");
+  need(cos_sin.is_cuda() && cos_sin.scalar_type() == at::kFloat && cos_sin.is_contiguous() && cos_sin.dim() == 2, "conv_qkv: cos_sin f32 [max_pos, rot]");
+  need(is_i32(positions) && positions.numel() == T && row_seq.numel() == T, "conv_qkv: positions, row_seq int32 [T]");
+  need(q_out.scalar_type() == proj.scalar_type() && q_out.is_contiguous() && q_out.size(0) == T && q_out.size(1) % heads == 0, "conv_qkv: q_out [T, heads * pad]");
+  const B2SeqRows s = seq_rows_of(row_seq, seq_rows, seq_state, banks);
+  B2ConvQkvArgs a{};
+  if (taps > 1) need(conv_state.has_value() && conv_state->scalar_type() == proj.scalar_type() && conv_state->is_contiguous() &&
+                         conv_state->numel() == banks * (taps - 1) * channels, "conv_qkv: conv_state [banks, taps - 1, channels] like proj");
+  if (kv_heads > 0) {
+    need(k_cache.has_value() && v_cache.has_value() && slots.has_value() && is_i64(*slots) && slots->numel() == T, "conv_qkv: caches and int64 slots [T]");
+    need(k_cache->dim() == 4 && v_cache->dim() == 4 && k_cache->is_contiguous() && v_cache->is_contiguous() && k_cache->scalar_type() == proj.scalar_type() &&
+             v_cache->scalar_type() == proj.scalar_type() && k_cache->size(1) == kv_heads && v_cache->size(1) == kv_heads &&
+             k_cache->size(0) == v_cache->size(0) && k_cache->size(2) == v_cache->size(2),
+         "conv_qkv: caches [pages, kv_heads, page, pad] like proj");
+    a.page_size = static_cast<int32_t>(k_cache->size(2));
+    a.num_slots = k_cache->size(0) * k_cache->size(2);
+    a.pad_vdim = static_cast<int32_t>(v_cache->size(3));
+    need(k_cache->size(3) == q_out.size(1) / heads, "conv_qkv: queries and keys must be padded alike");
+  }
+  a.proj = proj.data_ptr();
+  a.ld = proj.stride(0);
+  a.conv_w = conv_w.data_ptr<float>();
+  a.conv_state = opt<void>(conv_state);
+  a.cos_sin = cos_sin.data_ptr<float>();
+  a.positions = positions.data_ptr<int32_t>();
+  a.slots = opt<const int64_t>(slots);
+  a.q_out = q_out.data_ptr();
+  a.k_cache = opt<void>(k_cache);
+  a.v_cache = opt<void>(v_cache);
+  a.heads = static_cast<int32_t>(heads);
+  a.kv_heads = static_cast<int32_t>(kv_heads);
+  a.dim = static_cast<int32_t>(dim);
+  a.vdim = static_cast<int32_t>(vdim);
+  a.pad_dim = static_cast<int32_t>(q_out.size(1) / heads);
+  a.rot = static_cast<int32_t>(cos_sin.size(1));
+  a.taps = static_cast<int32_t>(taps);
+  a.max_pos = static_cast<int32_t>(cos_sin.size(0));
+  a.eps = static_cast<float>(eps);
+  c10::cuda::CUDAGuard g(proj.device());
+  check(b2_conv_qkv(&a, &s, proj.scalar_type() == at::kFloat ? 1 : 0, status_ptr(status), cur_stream()), "conv_qkv");
+}
+
+// first < 0: decode form over sequences [0, n); otherwise the scan over sequences [first, first + n).
+void delta_rule(const at::Tensor& proj, const at::Tensor& dg, const at::Tensor& conv_w, const OptTensor& conv_state, const at::Tensor& neg_rate,
+                const at::Tensor& dt_bias, const at::Tensor& norm_w, at::Tensor& state, const at::Tensor& row_seq, const at::Tensor& seq_rows,
+                const at::Tensor& seq_state, at::Tensor& out, const OptTensor& o_raw, int64_t b_off, int64_t heads, int64_t kv_heads, int64_t dim,
+                int64_t vdim, double eps, int64_t first, int64_t n, const OptTensor& status) {
+  need(is_act(proj) && proj.dim() == 2 && proj.stride(1) == 1 && dg.scalar_type() == proj.scalar_type() && dg.dim() == 2 && dg.stride(1) == 1 &&
+           out.scalar_type() == proj.scalar_type() && out.dim() == 2 && out.stride(1) == 1, "delta_rule: proj, dg, out of one type with unit inner strides");
+  const int64_t T = proj.size(0), taps = conv_w.size(0), channels = 2 * kv_heads * dim + heads * vdim;
+  need(dg.size(0) == T && dg.size(1) >= heads * (dim + vdim) && out.size(0) == T && out.size(1) >= heads * vdim && proj.size(1) >= channels && b_off >= 0 &&
+           b_off + heads <= proj.size(1) && row_seq.numel() == T, "delta_rule: shape mismatch");
+  need(conv_w.dim() == 2 && is_f32(conv_w, taps * channels) && is_f32(neg_rate, heads) && is_f32(dt_bias, heads * dim) && is_f32(norm_w, vdim),
+       "delta_rule: f32 parameters");
+  need(state.dim() == 4 && state.is_cuda() && state.scalar_type() == at::kFloat && state.is_contiguous() && state.size(1) == heads && state.size(2) == dim &&
+           state.size(3) == vdim, "delta_rule: state f32 [slots, heads, dim, vdim]");
+  const int64_t banks = 2 * state.size(0);
+  if (taps > 1) need(conv_state.has_value() && conv_state->scalar_type() == proj.scalar_type() && conv_state->is_contiguous() &&
+                         conv_state->numel() == banks * (taps - 1) * channels, "delta_rule: conv_state [banks, taps - 1, channels] like proj");
+  const B2SeqRows s = seq_rows_of(row_seq, seq_rows, seq_state, banks);
+  B2DeltaArgs a{};
+  a.proj = proj.data_ptr();
+  a.dg = dg.data_ptr();
+  a.ld = proj.stride(0);
+  a.ld_dg = dg.stride(0);
+  a.conv_w = conv_w.data_ptr<float>();
+  a.conv_state = opt<void>(conv_state);
+  a.neg_rate = neg_rate.data_ptr<float>();
+  a.dt_bias = dt_bias.data_ptr<float>();
+  a.norm_w = norm_w.data_ptr<float>();
+  a.state = state.data_ptr<float>();
+  a.out = out.data_ptr();
+  a.ld_out = out.stride(0);
+  a.b_off = static_cast<int32_t>(b_off);
+  a.heads = static_cast<int32_t>(heads);
+  a.kv_heads = static_cast<int32_t>(kv_heads);
+  a.dim = static_cast<int32_t>(dim);
+  a.vdim = static_cast<int32_t>(vdim);
+  a.taps = static_cast<int32_t>(taps);
+  a.eps = static_cast<float>(eps);
+  const int f32 = proj.scalar_type() == at::kFloat ? 1 : 0;
+  c10::cuda::CUDAGuard g(proj.device());
+  if (first < 0) {
+    check(b2_delta_decode(&a, &s, static_cast<int>(n), f32, status_ptr(status), cur_stream()), "delta_decode");
+  } else {
+    need(o_raw.has_value() && is_f32(*o_raw, T * heads * vdim), "delta_rule: the scan needs an f32 scratch [T, heads * vdim]");
+    a.o_raw = o_raw->data_ptr<float>();
+    check(b2_delta_scan(&a, &s, static_cast<int>(first), static_cast<int>(n), f32, status_ptr(status), cur_stream()), "delta_scan");
+  }
+}
+
+void gemm_f32(const at::Tensor& x, const at::Tensor& w, at::Tensor& y) {
+  for (const at::Tensor* t : {&x, &w, static_cast<const at::Tensor*>(&y)})
+    need(t->is_cuda() && t->scalar_type() == at::kFloat && t->dim() == 2 && t->stride(1) == 1, "gemm_f32: 2-D CUDA f32 with unit inner strides");
+  need(x.size(1) == w.size(1) && y.size(0) == x.size(0) && y.size(1) == w.size(0), "gemm_f32: x [M, K], w [N, K], y [M, N]");
+  c10::cuda::CUDAGuard g(x.device());
+  check(b2_gemm_f32(x.data_ptr<float>(), w.data_ptr<float>(), y.data_ptr<float>(), static_cast<int>(x.size(0)), static_cast<int>(w.size(0)),
+                    static_cast<int>(x.size(1)), x.stride(0), w.stride(0), y.stride(0), cur_stream()), "gemm_f32");
+}
+
+void attn_f32(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out, const at::Tensor& row_seq,
+              const at::Tensor& positions, const at::Tensor& block_tables, double scale, const OptTensor& gate, const OptTensor& status) {
+  need(q.is_cuda() && q.scalar_type() == at::kFloat && q.dim() == 2 && q.is_contiguous() && out.is_contiguous() && out.scalar_type() == at::kFloat,
+       "attn_f32: q, out contiguous CUDA f32");
+  need(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.scalar_type() == at::kFloat &&
+           v_cache.scalar_type() == at::kFloat && k_cache.size(0) == v_cache.size(0) && k_cache.size(1) == v_cache.size(1) && k_cache.size(2) == v_cache.size(2),
+       "attn_f32: f32 caches [pages, n_kv, page, D]");
+  const int64_t T = q.size(0), D = k_cache.size(3), n_q = q.size(1) / D;
+  need(n_q * D == q.size(1) && out.size(0) == T && out.size(1) == n_q * v_cache.size(3), "attn_f32: shape mismatch");
+  need(is_i32(row_seq) && is_i32(positions) && is_i32(block_tables) && row_seq.numel() == T && positions.numel() == T && block_tables.dim() == 2, "attn_f32: int32 metadata");
+  if (gate.has_value()) need(gate->scalar_type() == at::kFloat && gate->dim() == 2 && gate->size(0) == T && gate->size(1) == n_q && gate->stride(1) == 1, "attn_f32: gate f32 [T, n_q]");
+  c10::cuda::CUDAGuard g(q.device());
+  check(b2_attn_f32(q.data_ptr<float>(), k_cache.data_ptr<float>(), v_cache.data_ptr<float>(), out.data_ptr<float>(), row_seq.data_ptr<int32_t>(),
+                    positions.data_ptr<int32_t>(), block_tables.data_ptr<int32_t>(), static_cast<int>(T), static_cast<int>(block_tables.size(0)),
+                    static_cast<int>(block_tables.size(1)), static_cast<int>(n_q), static_cast<int>(k_cache.size(1)), static_cast<int>(D),
+                    static_cast<int>(v_cache.size(3)), static_cast<int>(k_cache.size(2)), static_cast<float>(scale), k_cache.size(0),
+                    gate.has_value() ? gate->data_ptr<float>() : nullptr, gate.has_value() ? gate->stride(0) : 0, status_ptr(status), cur_stream()),
+        "attn_f32");
+}
+}  // namespace
+
+void bind_mixers(py::module_& m) {
+  m.def("hyper_norm", &hyper_norm);
+  m.def("conv_qkv", &conv_qkv);
+  m.def("delta_rule", &delta_rule);
+  m.def("gemm_f32", &gemm_f32);
+  m.def("attn_f32", &attn_f32);
+  m.def("swiglu_f32", [](const at::Tensor& gu, at::Tensor& out) {
+    need(gu.is_cuda() && gu.scalar_type() == at::kFloat && gu.is_contiguous() && out.is_contiguous() && out.scalar_type() == at::kFloat &&
+             gu.size(0) == out.size(0) && gu.size(1) == 2 * out.size(1), "swiglu_f32: gate_up [M, 2F], out [M, F], contiguous CUDA f32");
+    c10::cuda::CUDAGuard g(gu.device());
+    check(b2_swiglu_f32(gu.data_ptr<float>(), out.data_ptr<float>(), static_cast<int>(out.size(0)), static_cast<int>(out.size(1)), cur_stream()), "swiglu_f32");
+  });
+  m.def("gather_rows_f32", [](const at::Tensor& src, const at::Tensor& index, at::Tensor& out, const OptTensor& status) {
+    need(src.is_cuda() && src.scalar_type() == at::kFloat && src.is_contiguous() && src.dim() == 2 && out.is_contiguous() && out.scalar_type() == at::kFloat &&
+             is_i64(index) && out.size(0) == index.numel() && out.size(1) == src.size(1), "gather_rows_f32: f32 [rows, cols], int64 index");
+    c10::cuda::CUDAGuard g(src.device());
+    check(b2_gather_rows_f32(src.data_ptr<float>(), index.data_ptr<int64_t>(), out.data_ptr<float>(), static_cast<int>(index.numel()),
+                             static_cast<int>(src.size(1)), src.size(0), status_ptr(status), cur_stream()), "gather_rows_f32");
+  });
+}

@@ -62,11 +62,14 @@ int b2_sample(const void* logits, int is_bf16, int64_t* ids, const float* temper
 // ---- attention ---------------------------------------------------------------------------------
 // Causal GQA attention over a paged KV cache for a ragged batch of query chunks.
 // q/out: [T, n_q, D]; cache: [num_pages, n_kv, page_size, D]; cu_q: [B+1] query offsets; ctx_lens: [B]
-// total context (cached prefix + this chunk); block_tables: [B, max_blocks]. D == 128 or 64.
+// total context (cached prefix + this chunk); block_tables: [B, max_blocks]. D == 64, 128 or 256.
+// `gate` (may be null), in this and the two kernels below: bf16 [T, n_q] with row stride `gate_stride`; head h of query
+// row t is multiplied by sigmoid(gate[t, h]) before it is rounded.
 int b2_attn_prefill_bf16(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* cu_q,
                          const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                          int n_kv, int head_dim, int page_size, int max_q_len, float scale, int64_t q_stride,
-                         int64_t out_stride, int64_t num_pages, b2::Status* status, cudaStream_t stream);
+                         int64_t out_stride, int64_t num_pages, const void* gate, int64_t gate_stride,
+                         b2::Status* status, cudaStream_t stream);
 // bf16 GEMM on CTA pairs (tcgen05 cta_group::2, 256 x 256 tiles; csrc/kernels/gemm_bf16_pair.cu). Epilogue NONE or SWIGLU.
 int b2_gemm_bf16_pair(const void* x, const void* w, void* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,
                       int epilogue, int bn, b2::Status* status, cudaStream_t stream);
@@ -76,7 +79,7 @@ int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const void* v_ca
                             const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                             int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
                             int64_t num_pages, int variant, const int32_t* work, const int32_t* n_work, int work_items,
-                            b2::Status* status, cudaStream_t stream);
+                            const void* gate, int64_t gate_stride, b2::Status* status, cudaStream_t stream);
 // One query token per sequence, split over the KV length. workspace: f32, size from b2_attn_decode_workspace.
 // `counters` (may be null): u32 [batch * n_kv], zero before the first use and left at zero by every launch; with it
 // (and page sizes that are multiples of 32) the split that finishes last merges the partials itself, otherwise a
@@ -84,7 +87,8 @@ int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const void* v_ca
 int b2_attn_decode_bf16(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* ctx_lens,
                         const int32_t* block_tables, float* workspace, int batch, int max_blocks, int n_q, int n_kv,
                         int head_dim, int page_size, int num_splits, float scale, int64_t q_stride,
-                        int64_t out_stride, int64_t num_pages, uint32_t* counters, b2::Status* status, cudaStream_t stream);
+                        int64_t out_stride, int64_t num_pages, uint32_t* counters, const void* gate, int64_t gate_stride,
+                        b2::Status* status, cudaStream_t stream);
 int64_t b2_attn_decode_counter_bytes(int batch, int n_kv);
 int64_t b2_attn_decode_workspace(int batch, int n_q, int head_dim, int num_splits);
 // MLA decode with absorbed weights: q_lat [B, H, 512], q_rope [B, H, 64]; cache [num_pages, page, 576]

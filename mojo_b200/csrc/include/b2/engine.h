@@ -33,7 +33,9 @@ struct KVStats {
 
 class KVCacheManager {
  public:
-  KVCacheManager(int64_t num_pages, int page_size, bool enable_prefix_cache);
+  // `state_slots` > 0: every sequence also owns one slot of fixed-size recurrent state (models with recurrent layers);
+  // prefix caching is then impossible, because a cached page says nothing about the state at its end.
+  KVCacheManager(int64_t num_pages, int page_size, bool enable_prefix_cache, int64_t state_slots = 0);
 
   int page_size() const { return page_size_; }
   int64_t num_pages() const { return num_pages_; }
@@ -54,6 +56,14 @@ class KVCacheManager {
   // the (src_page, dst_page) pair to copy is appended to `copies`.
   bool fork(int64_t src, int64_t dst, std::vector<std::pair<int64_t, int64_t>>* copies);
 
+  // Recurrent state. A slot holds two banks for what several thread blocks read while others write it (the tail of the
+  // short convolutions): a step reads the bank the previous step wrote and writes the other one. `advance_state` is
+  // called once per step and sequence, in launch order, and returns {bank to read, bank to write} as indices into
+  // 2 * state_slots banks (bank = 2 * slot + parity); reading bank -1 means "no history" (`first_pos` == 0).
+  int64_t state_slots() const { return state_slots_; }
+  int64_t free_state_slots() const { return static_cast<int64_t>(free_state_.size()); }
+  std::pair<int32_t, int32_t> advance_state(int64_t seq_id, int64_t first_pos);
+
   const std::vector<int32_t>& block_table(int64_t seq_id) const;
   int64_t slot(int64_t seq_id, int64_t pos) const;
   int64_t num_tokens_reserved(int64_t seq_id) const;
@@ -67,6 +77,8 @@ class KVCacheManager {
     int64_t reserved_tokens = 0;
     int64_t committed_pages = 0;
     uint64_t last_hash = 0;
+    int32_t state_slot = -1;
+    int32_t state_parity = 0;
   };
   int32_t take_page();
   void release_page(int32_t page);
@@ -74,7 +86,9 @@ class KVCacheManager {
   int64_t num_pages_;
   int page_size_;
   bool prefix_;
+  int64_t state_slots_;
   std::deque<int32_t> free_;
+  std::deque<int32_t> free_state_;
   std::list<int32_t> evictable_;               // cached pages with refcount 0, oldest first
   std::vector<std::list<int32_t>::iterator> evict_pos_;
   std::vector<uint8_t> in_evictable_;
@@ -118,6 +132,7 @@ struct Batch {
   std::vector<int32_t> positions;   // [T]
   std::vector<int64_t> slots;       // [T] physical KV slots
   std::vector<int32_t> block_tables;  // [B, max_blocks], padded with 0
+  std::vector<int32_t> seq_state;   // [B, 2] recurrent-state banks {read, write} per sequence; empty without state slots
   std::vector<int32_t> sample_rows; // indices (into the flat token arrays) whose logits are sampled
   std::vector<int64_t> sample_seq_ids;
   int max_blocks = 0;
@@ -135,6 +150,10 @@ class Scheduler {
   void add_request(int64_t id, const int32_t* prompt, int64_t prompt_len, int64_t max_new_tokens, double arrival);
   // Build the next batch; empty batch when nothing is runnable.
   Batch step();
+  // One externally planned step: every entry appends its tokens to a request (admitted here if it is new) and exactly
+  // these tokens run, from the cache and state that earlier steps left. Nothing is preempted; throws, with no entry
+  // taken up, when pages or state slots run out. Decode rows come first in the batch, as in `step()`.
+  Batch run_tokens(const std::vector<std::pair<int64_t, std::vector<int32_t>>>& entries);
   // Record the token sampled for a sequence after the step. Returns true when the sequence hit
   // max_new_tokens (the caller may also finish it earlier, e.g. on EOS or a stop string).
   bool append_token(int64_t id, int32_t token);
@@ -162,6 +181,7 @@ class Scheduler {
  private:
   bool preempt_one(int64_t keep_id, Batch* b);
   void emit(Request& r, int64_t n_tokens, Batch* b);
+  void flatten(std::vector<std::pair<int64_t, int64_t>>& entries, Batch* b);   // (sequence, tokens to run): decode rows first
   void drop_pending_commit(int64_t id);
 
   SchedulerConfig cfg_;

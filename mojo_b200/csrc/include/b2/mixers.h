@@ -1,0 +1,112 @@
+// C launch API of the sequence-mixing kernels beyond plain attention: residual streams with learned mixing
+// (hyper-connections), short causal convolutions in front of attention, the gated delta rule, and the 32-bit
+// forms of the matrix product and of paged attention. Conventions as in b2/api.h: raw device pointers, a stream, 0 or
+// a negative code back. `f32` selects the element type of activations and caches (0: bf16, 1: f32); parameters that
+// enter 32-bit arithmetic (norm weights, mixing coefficients, convolution taps, decay constants) are always f32.
+#pragma once
+#include <cstdint>
+#include <cuda_runtime.h>
+#include "b2/status.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+// Where the sequences of a step lie in its flat token rows, and which recurrent-state banks they use.
+//   row_seq   [rows]     sequence of each row, -1 for padding
+//   seq_rows  [seqs, 2]  first row and one past the last row (equal: unused entry)
+//   seq_state [seqs, 2]  bank to read (-1: no history) and bank to write (-1: unused entry); bank = 2 * slot + parity
+struct B2SeqRows {
+  const int32_t* row_seq;
+  const int32_t* seq_rows;
+  const int32_t* seq_state;
+  int32_t rows, seqs, banks;
+};
+
+// Residual streams x [rows, streams, width] f32. For every row: x_t <- sum_s mix[s, t] x_s + out[t] y (skipped when y is
+// null), then h = rms_norm(sum_s in[s] x_s) * weight. With `ids` the streams start as embed[id] * embed_scale instead of
+// being read. `store` writes the new streams back. With `rows_index` only those rows are processed and h is compact.
+// Columns from `mean_width` up to `width` are zero padding that the mean leaves out.
+struct B2HyperArgs {
+  float* x;
+  const void* y;
+  const float* mix;
+  const float* out;
+  const float* in;
+  const float* weight;
+  void* h;
+  const int64_t* ids;
+  const void* embed;
+  const int64_t* rows_index;
+  float embed_scale, eps;
+  int32_t n_out, rows, width, mean_width, streams, vocab, store;
+};
+int b2_hyper_norm(const B2HyperArgs* a, int f32, b2::Status* status, cudaStream_t stream);
+
+// Short causal convolution on the q | k | v channels of a projection, rotary embedding on q and k, RMS norm of each q and k
+// head (no weight), and the scatter of k and v into the paged cache; one launch. proj [rows, ld]: the channels start at
+// column 0 in the order q (heads * dim), k (kv_heads * dim), v (kv_heads * vdim); kv_heads == 0: queries only.
+// conv_w f32 [taps, channels]; conv_state [banks, taps - 1, channels] (null when taps == 1).
+// q_out [rows, heads * pad_dim], caches [pages, kv_heads, page_size, pad_dim / pad_vdim]; columns past dim are zero.
+struct B2ConvQkvArgs {
+  const void* proj;
+  int64_t ld;
+  const float* conv_w;
+  void* conv_state;
+  const float* cos_sin;       // [max_pos, rot]
+  const int32_t* positions;   // [rows]
+  const int64_t* slots;       // [rows], -1: nothing is cached
+  void* q_out;
+  void* k_cache;
+  void* v_cache;
+  int64_t num_slots;
+  int32_t heads, kv_heads, dim, vdim, pad_dim, pad_vdim, rot, taps, page_size, max_pos;
+  float eps;
+};
+int b2_conv_qkv(const B2ConvQkvArgs* a, const B2SeqRows* s, int f32, b2::Status* status, cudaStream_t stream);
+
+// Gated delta rule with one decay per key channel. Per head, with S [dim, vdim]:
+//   S <- g * S (rows), u = beta (v - S^T k), S <- S + k u^T, o = S^T q
+// proj [rows, ld]: q (kv_heads * dim) | k | v (heads * vdim) from column 0, the step-size logits at column b_off;
+// dg [rows, ld_dg]: decay inputs (heads * dim) from column 0, output-gate logits (heads * vdim) from column heads * dim.
+// q, k, v pass the short convolution and silu; q, k become unit vectors, q times dim^-0.5; beta = sigmoid(b);
+// g = exp(neg_rate[h] * softplus(decay input + dt_bias)). out = rms_norm(o) * norm_w * sigmoid(gate).
+// state f32 [slots, heads, dim, vdim], updated in place; conv_state as above.
+struct B2DeltaArgs {
+  const void* proj;
+  const void* dg;
+  int64_t ld, ld_dg;
+  const float* conv_w;
+  void* conv_state;
+  const float* neg_rate;      // [heads] = -exp(A_log)
+  const float* dt_bias;       // [heads * dim]
+  const float* norm_w;        // [vdim]
+  float* state;
+  float* o_raw;               // [rows, heads * vdim] scratch of the scan
+  void* out;                  // [rows, ld_out], heads * vdim columns
+  int64_t ld_out;
+  int32_t b_off, heads, kv_heads, dim, vdim, taps;
+  float eps;
+};
+// Sequences [0, n) of the step, one row each: state read and written once, output finished in the same kernel.
+int b2_delta_decode(const B2DeltaArgs* a, const B2SeqRows* s, int n, int f32, b2::Status* status, cudaStream_t stream);
+// Sequences [first, first + n): any number of rows each. Two launches (scan, output norm and gate).
+int b2_delta_scan(const B2DeltaArgs* a, const B2SeqRows* s, int first, int n, int f32, b2::Status* status, cudaStream_t stream);
+
+// Y[M, N] = X[M, K] W[N, K]^T in true f32 (FMA, no reduced-precision matrix mode).
+int b2_gemm_f32(const float* x, const float* w, float* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,
+                cudaStream_t stream);
+// out[r, j] = silu(gate) * up for rows whose gate and up columns alternate in blocks of 16.
+int b2_swiglu_f32(const float* gate_up, float* out, int rows, int ffn, cudaStream_t stream);
+int b2_gather_rows_f32(const float* src, const int64_t* index, float* out, int rows_out, int cols, int64_t rows_src,
+                       b2::Status* status, cudaStream_t stream);
+// Causal GQA attention over the paged cache in f32: any head sizes up to 256, decode rows and prompt chunks alike. Row t
+// of sequence row_seq[t] sees positions 0 .. positions[t]. gate as in b2/api.h, f32.
+int b2_attn_f32(const float* q, const float* k_cache, const float* v_cache, float* out, const int32_t* row_seq,
+                const int32_t* positions, const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv,
+                int dim, int vdim, int page_size, float scale, int64_t num_pages, const float* gate, int64_t gate_stride,
+                b2::Status* status, cudaStream_t stream);
+
+#ifdef __cplusplus
+}
+#endif

@@ -61,6 +61,17 @@ __device__ __forceinline__ uint32_t tile_addr(uint32_t base, int row, int chunk)
   }
 }
 
+// Optional per-head output gate: head h of query row t is multiplied by sigmoid(logits[t * stride + h]) before it is
+// rounded. No gate when `logits` is null.
+struct HeadGate {
+  const __nv_bfloat16* logits;
+  int64_t stride;
+  __device__ __forceinline__ float factor(int64_t row, int head) const {
+    if (logits == nullptr) return 1.0f;
+    return 1.0f / (1.0f + ptx::ex2(-__bfloat162float(logits[row * stride + head]) * ptx::kLog2e));
+  }
+};
+
 struct PagedKV {
   const __nv_bfloat16* k;
   const __nv_bfloat16* v;
@@ -208,7 +219,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, __nv_bfloat16* __restrict__ out, const int32_t* __restrict__ cu_q,
     const int32_t* __restrict__ ctx_lens, const int32_t* __restrict__ block_tables, int max_blocks, int n_q, int n_kv,
-    int page_size, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, Status* status) {
+    int page_size, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate, Status* status) {
   ptx::grid_dep_sync();
   constexpr int BM = 64, BN = 64;
   constexpr int TILE_BYTES = BN * D * 2;
@@ -281,7 +292,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
     const int tok = pr / group, hg = pr % group;
     if (tok >= q_len) continue;
     __nv_bfloat16* dst = out + static_cast<int64_t>(tok0 + tok) * out_stride + static_cast<int64_t>(kvh * group + hg) * D;
-    const float inv = half ? inv_hi : inv_lo;
+    const float inv = (half ? inv_hi : inv_lo) * gate.factor(tok0 + tok, kvh * group + hg);
 #pragma unroll
     for (int d = 0; d < D / 8; ++d) {
       const uint32_t pk = ptx::pack_bf16x2(o[d][half * 2] * inv, o[d][half * 2 + 1] * inv);
@@ -300,7 +311,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     const __nv_bfloat16* __restrict__ v_cache, __nv_bfloat16* __restrict__ out, const int32_t* __restrict__ ctx_lens,
     const int32_t* __restrict__ block_tables, float* __restrict__ workspace, int max_blocks, int n_q, int n_kv,
     int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-    Status* status) {
+    HeadGate gate, Status* status) {
   ptx::grid_dep_sync();
   constexpr int BN = 32;
   constexpr int TILE_BYTES = BN * D * 2;
@@ -399,7 +410,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     }
     const int head = kvh * group + row;
     if (num_splits == 1) {
-      const float inv = ll > 0.0f ? 1.0f / ll : 0.0f;
+      const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D + cs;
 #pragma unroll
       for (int c = 0; c < COLS_PER_THREAD; c += 2)
@@ -428,7 +439,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
     const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, const int32_t* __restrict__ ctx_lens,
     const int32_t* __restrict__ block_tables, float* __restrict__ workspace, int max_blocks, int n_q, int n_kv,
     int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-    uint32_t* __restrict__ split_counters, Status* status) {
+    uint32_t* __restrict__ split_counters, HeadGate gate, Status* status) {
   ptx::grid_dep_sync();
   constexpr int BN = 32;
   constexpr int HALVES = D / 64;
@@ -531,7 +542,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
     if (row >= group) continue;
     const int head = kvh * group + row;
     if (num_splits == 1) {
-      const float inv = l[half] > 0.0f ? 1.0f / l[half] : 0.0f;
+      const float inv = (l[half] > 0.0f ? 1.0f / l[half] : 0.0f) * gate.factor(seq, head);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
       for (int d = 0; d < D / 8; ++d)
@@ -575,7 +586,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
 #pragma unroll
         for (int c = 0; c < D / 32; ++c) acc[c] += __ldcg(base + sp * RS + c * 32 + lane) * f;
       }
-      const float inv = ll > 0.0f ? 1.0f / ll : 0.0f;
+      const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
       for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv);
@@ -586,7 +597,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
 // Merge split partials: one warp per (sequence, head).
 template <int D>
 __global__ void attn_decode_reduce_kernel(const float* __restrict__ workspace, __nv_bfloat16* __restrict__ out,
-                                          int n_q, int num_splits, int64_t out_stride, int total) {
+                                          int n_q, int num_splits, int64_t out_stride, int total, HeadGate gate) {
   ptx::grid_dep_sync();
   constexpr int RS = D + 2;
   const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -607,10 +618,61 @@ __global__ void attn_decode_reduce_kernel(const float* __restrict__ workspace, _
 #pragma unroll
     for (int c = 0; c < D / 32; ++c) acc[c] += base[s * RS + c * 32 + lane] * f;
   }
-  const float inv = ll > 0.0f ? 1.0f / ll : 0.0f;
+  const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head);
   __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
   for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv);
+}
+
+template <int D>
+int launch_prefill(dim3 grid, cudaStream_t stream, const __nv_bfloat16* q, const __nv_bfloat16* k, const __nv_bfloat16* v, __nv_bfloat16* out,
+                   const int32_t* cu_q, const int32_t* ctx_lens, const int32_t* block_tables, int max_blocks, int n_q, int n_kv, int page_size,
+                   float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate, Status* status) {
+  constexpr int SMEM = 4 * 16 * D * 2 + 4 * 64 * D * 2;
+  static DeviceOnce attr_once;
+  if (const int rc = attr_once.max_smem(attn_prefill_kernel<D>, SMEM)) return rc;
+  launch_pdl(attn_prefill_kernel<D>, grid, dim3(128), SMEM, stream, q, k, v, out, cu_q, ctx_lens, block_tables, max_blocks, n_q, n_kv, page_size,
+             scale_log2, q_stride, out_stride, num_pages, gate, status);
+  return last_launch_rc();
+}
+
+template <int D>
+int launch_decode_tma(dim3 grid, cudaStream_t stream, const void* k, const void* v, const __nv_bfloat16* q, __nv_bfloat16* out,
+                      const int32_t* ctx_lens, const int32_t* block_tables, float* workspace, int batch, int max_blocks, int n_q, int n_kv,
+                      int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages,
+                      uint32_t* counters, HeadGate gate, Status* status) {
+  // cache as a 2-D matrix [(page, kv head, token), D], boxes of 32 tokens x 64 columns
+  CUtensorMap tk, tv;
+  const uint64_t rows = static_cast<uint64_t>(num_pages) * n_kv * page_size;
+  if (!make_tmap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, k, rows, D, D * 2, 32, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
+      !make_tmap_2d(&tv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, v, rows, D, D * 2, 32, 64, CU_TENSOR_MAP_SWIZZLE_128B))
+    return -kBadArgument;
+  constexpr int STAGES = 3;
+  constexpr int SMEM = STAGES * 2 * 32 * D * 2 + 16 * D * 2 + 64 + 1024;
+  static DeviceOnce attr_once;
+  if (const int rc = attr_once.max_smem(attn_decode_tma_kernel<D, STAGES>, SMEM)) return rc;
+  launch_pdl(attn_decode_tma_kernel<D, STAGES>, grid, dim3(32), SMEM, stream, tk, tv, q, out, ctx_lens, block_tables, workspace, max_blocks, n_q,
+             n_kv, page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, counters, gate, status);
+  if (num_splits > 1 && counters == nullptr)
+    launch_pdl(attn_decode_reduce_kernel<D>, dim3((batch * n_q + 3) / 4), dim3(128), 0, stream, workspace, out, n_q, num_splits, out_stride,
+               batch * n_q, gate);
+  return last_launch_rc();
+}
+
+template <int D>
+int launch_decode(dim3 grid, cudaStream_t stream, const __nv_bfloat16* k, const __nv_bfloat16* v, const __nv_bfloat16* q, __nv_bfloat16* out,
+                  const int32_t* ctx_lens, const int32_t* block_tables, float* workspace, int batch, int max_blocks, int n_q, int n_kv,
+                  int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate,
+                  Status* status) {
+  constexpr int SMEM = 4 * (16 * D * 2 + 4 * 32 * D * 2);
+  static DeviceOnce attr_once;
+  if (const int rc = attr_once.max_smem(attn_decode_kernel<D>, SMEM)) return rc;
+  launch_pdl(attn_decode_kernel<D>, grid, dim3(128), SMEM, stream, q, k, v, out, ctx_lens, block_tables, workspace, max_blocks, n_q, n_kv,
+             page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, gate, status);
+  if (num_splits > 1)
+    launch_pdl(attn_decode_reduce_kernel<D>, dim3((batch * n_q + 3) / 4), dim3(128), 0, stream, workspace, out, n_q, num_splits, out_stride,
+               batch * n_q, gate);
+  return last_launch_rc();
 }
 
 }  // namespace
@@ -622,33 +684,25 @@ extern "C" int b2_attn_prefill_bf16(const void* q, const void* k_cache, const vo
                                     const int32_t* cu_q, const int32_t* ctx_lens, const int32_t* block_tables,
                                     int batch, int max_blocks, int n_q, int n_kv, int head_dim, int page_size,
                                     int max_q_len, float scale, int64_t q_stride, int64_t out_stride,
-                                    int64_t num_pages, Status* status, cudaStream_t stream) {
+                                    int64_t num_pages, const void* gate, int64_t gate_stride, Status* status,
+                                    cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
-  if (n_kv <= 0 || n_q % n_kv != 0 || (head_dim != 128 && head_dim != 64) || q_stride % 8 != 0 || out_stride % 2 != 0)
-    return -kBadArgument;
+  if (n_kv <= 0 || n_q % n_kv != 0 || q_stride % 8 != 0 || out_stride % 2 != 0) return -kBadArgument;
   const int group = n_q / n_kv;
-  dim3 grid((max_q_len * group + 63) / 64, n_kv, batch);
+  const dim3 grid((max_q_len * group + 63) / 64, n_kv, batch);
   const float scale_log2 = scale * ptx::kLog2e;
-  auto qp = static_cast<const __nv_bfloat16*>(q);
-  auto kp = static_cast<const __nv_bfloat16*>(k_cache);
-  auto vp = static_cast<const __nv_bfloat16*>(v_cache);
-  auto op = static_cast<__nv_bfloat16*>(out);
-  if (head_dim == 128) {
-    constexpr int SMEM = 4 * 16 * 128 * 2 + 4 * 64 * 128 * 2;
-    static DeviceOnce attr_once;
-    if (const int rc = attr_once.run([&] { return cudaFuncSetAttribute(attn_prefill_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); })) return rc;
-    launch_pdl(attn_prefill_kernel<128>, dim3(grid), dim3(128), SMEM, stream, qp, kp, vp, op, cu_q, ctx_lens, block_tables, max_blocks, n_q,
-                                                          n_kv, page_size, scale_log2, q_stride, out_stride, num_pages,
-                                                          status);
-  } else {
-    constexpr int SMEM = 4 * 16 * 64 * 2 + 4 * 64 * 64 * 2;
-    static DeviceOnce attr_once;
-    if (const int rc = attr_once.run([&] { return cudaFuncSetAttribute(attn_prefill_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); })) return rc;
-    launch_pdl(attn_prefill_kernel<64>, dim3(grid), dim3(128), SMEM, stream, qp, kp, vp, op, cu_q, ctx_lens, block_tables, max_blocks, n_q,
-                                                         n_kv, page_size, scale_log2, q_stride, out_stride, num_pages,
-                                                         status);
+  const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride};
+#define B2_PREFILL(D_)                                                                                                          \
+  return launch_prefill<D_>(grid, stream, static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),    \
+                            static_cast<const __nv_bfloat16*>(v_cache), static_cast<__nv_bfloat16*>(out), cu_q, ctx_lens,      \
+                            block_tables, max_blocks, n_q, n_kv, page_size, scale_log2, q_stride, out_stride, num_pages, hg, status)
+  switch (head_dim) {
+    case 64: B2_PREFILL(64);
+    case 128: B2_PREFILL(128);
+    case 256: B2_PREFILL(256);
+    default: return -kBadArgument;
   }
-  return last_launch_rc();
+#undef B2_PREFILL
 }
 
 extern "C" int64_t b2_attn_decode_workspace(int batch, int n_q, int head_dim, int num_splits) {
@@ -663,65 +717,36 @@ extern "C" int b2_attn_decode_bf16(const void* q, const void* k_cache, const voi
                                    const int32_t* ctx_lens, const int32_t* block_tables, float* workspace, int batch,
                                    int max_blocks, int n_q, int n_kv, int head_dim, int page_size, int num_splits,
                                    float scale, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-                                   uint32_t* counters, Status* status, cudaStream_t stream) {
+                                   uint32_t* counters, const void* gate, int64_t gate_stride, Status* status,
+                                   cudaStream_t stream) {
   if (batch <= 0) return 0;
-  if (n_kv <= 0 || n_q % n_kv != 0 || n_q / n_kv > 16 || (head_dim != 128 && head_dim != 64) || q_stride % 8 != 0 ||
-      num_splits < 1 || (num_splits > 1 && workspace == nullptr))
+  if (n_kv <= 0 || n_q % n_kv != 0 || n_q / n_kv > 16 || q_stride % 8 != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr))
     return -kBadArgument;
-  dim3 grid(num_splits, n_kv, batch);
+  const dim3 grid(num_splits, n_kv, batch);
   const float scale_log2 = scale * ptx::kLog2e;
+  const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride};
   auto qp = static_cast<const __nv_bfloat16*>(q);
-  auto kp = static_cast<const __nv_bfloat16*>(k_cache);
-  auto vp = static_cast<const __nv_bfloat16*>(v_cache);
   auto op = static_cast<__nv_bfloat16*>(out);
-  const int total = batch * n_q;
+#define B2_DECODE_TMA(D_)                                                                                                             \
+  return launch_decode_tma<D_>(grid, stream, k_cache, v_cache, qp, op, ctx_lens, block_tables, workspace, batch, max_blocks, n_q, n_kv, \
+                               page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, counters, hg, status)
+#define B2_DECODE(D_)                                                                                                                   \
+  return launch_decode<D_>(grid, stream, static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache), qp, op, \
+                           ctx_lens, block_tables, workspace, batch, max_blocks, n_q, n_kv, page_size, num_splits, scale_log2, q_stride, \
+                           out_stride, num_pages, hg, status)
   if (page_size % 32 == 0) {
-    // TMA path: cache as a 2-D matrix [(page, kv head, token), D], boxes of 32 tokens x 64 columns
-    CUtensorMap tk, tv;
-    const uint64_t rows = static_cast<uint64_t>(num_pages) * n_kv * page_size;
-    if (!make_tmap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, k_cache, rows, head_dim, head_dim * 2, 32, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
-        !make_tmap_2d(&tv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, v_cache, rows, head_dim, head_dim * 2, 32, 64, CU_TENSOR_MAP_SWIZZLE_128B))
-      return -kBadArgument;
-    constexpr int STAGES = 3;
-    if (head_dim == 128) {
-      constexpr int SMEM = STAGES * 2 * 32 * 128 * 2 + 16 * 128 * 2 + 64 + 1024;
-      static DeviceOnce attr_once;
-    if (const int rc = attr_once.run([&] { return cudaFuncSetAttribute(attn_decode_tma_kernel<128, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); })) return rc;
-      launch_pdl(attn_decode_tma_kernel<128, STAGES>, dim3(grid), dim3(32), SMEM, stream, tk, tv, qp, op, ctx_lens, block_tables, workspace, max_blocks,
-                                                                    n_q, n_kv, page_size, num_splits, scale_log2, q_stride,
-                                                                    out_stride, num_pages, counters, status);
-      if (num_splits > 1 && counters == nullptr)
-        launch_pdl(attn_decode_reduce_kernel<128>, dim3((total + 3) / 4), dim3(128), 0, stream, workspace, op, n_q, num_splits, out_stride, total);
-    } else {
-      constexpr int SMEM = STAGES * 2 * 32 * 64 * 2 + 16 * 64 * 2 + 64 + 1024;
-      static DeviceOnce attr_once;
-    if (const int rc = attr_once.run([&] { return cudaFuncSetAttribute(attn_decode_tma_kernel<64, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); })) return rc;
-      launch_pdl(attn_decode_tma_kernel<64, STAGES>, dim3(grid), dim3(32), SMEM, stream, tk, tv, qp, op, ctx_lens, block_tables, workspace, max_blocks,
-                                                                   n_q, n_kv, page_size, num_splits, scale_log2, q_stride,
-                                                                    out_stride, num_pages, counters, status);
-      if (num_splits > 1 && counters == nullptr)
-        launch_pdl(attn_decode_reduce_kernel<64>, dim3((total + 3) / 4), dim3(128), 0, stream, workspace, op, n_q, num_splits, out_stride, total);
+    switch (head_dim) {
+      case 64: B2_DECODE_TMA(64);
+      case 128: B2_DECODE_TMA(128);
+      case 256: B2_DECODE_TMA(256);
+      default: return -kBadArgument;
     }
-    return last_launch_rc();
   }
-  if (head_dim == 128) {
-    constexpr int SMEM = 4 * (16 * 128 * 2 + 4 * 32 * 128 * 2);
-    static DeviceOnce attr_once;
-    if (const int rc = attr_once.run([&] { return cudaFuncSetAttribute(attn_decode_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); })) return rc;
-    launch_pdl(attn_decode_kernel<128>, dim3(grid), dim3(128), SMEM, stream, qp, kp, vp, op, ctx_lens, block_tables, workspace, max_blocks,
-                                                         n_q, n_kv, page_size, num_splits, scale_log2, q_stride,
-                                                         out_stride, num_pages, status);
-    if (num_splits > 1)
-      launch_pdl(attn_decode_reduce_kernel<128>, dim3((total + 3) / 4), dim3(128), 0, stream, workspace, op, n_q, num_splits, out_stride, total);
-  } else {
-    constexpr int SMEM = 4 * (16 * 64 * 2 + 4 * 32 * 64 * 2);
-    static DeviceOnce attr_once;
-    if (const int rc = attr_once.run([&] { return cudaFuncSetAttribute(attn_decode_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM); })) return rc;
-    launch_pdl(attn_decode_kernel<64>, dim3(grid), dim3(128), SMEM, stream, qp, kp, vp, op, ctx_lens, block_tables, workspace, max_blocks,
-                                                        n_q, n_kv, page_size, num_splits, scale_log2, q_stride,
-                                                        out_stride, num_pages, status);
-    if (num_splits > 1)
-      launch_pdl(attn_decode_reduce_kernel<64>, dim3((total + 3) / 4), dim3(128), 0, stream, workspace, op, n_q, num_splits, out_stride, total);
+  switch (head_dim) {
+    case 64: B2_DECODE(64);
+    case 128: B2_DECODE(128);
+    default: return -kBadArgument;    // the cp.async buffers of head_dim 256 exceed an SM's shared memory
   }
-  return last_launch_rc();
+#undef B2_DECODE_TMA
+#undef B2_DECODE
 }

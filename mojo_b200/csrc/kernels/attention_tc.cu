@@ -68,6 +68,9 @@ struct AttnTcParams {
   // every CTA of the grid has an item. Without a list the grid is (query tiles, heads, sequences).
   const int* work;
   const int* n_work;
+  // Optional per-head output gate: head h of row t is multiplied by sigmoid(gate[t * gate_stride + h]). Null: no gate.
+  const __nv_bfloat16* gate;
+  int64_t gate_stride;
 };
 
 // Shared-memory descriptor with explicit leading / stride byte offsets, 128-byte swizzle.
@@ -361,7 +364,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     ptx::named_barrier_sync(5, 256);
     if (ok && *fail == 0 && r < rows) {
       const float l = l_final[r] + l_final[kTile + r];
-      const float inv = l > 0.0f ? 1.0f / l : 0.0f;
+      float inv = l > 0.0f ? 1.0f / l : 0.0f;
+      if (prm.gate != nullptr) {
+        const float z = __bfloat162float(prm.gate[static_cast<int64_t>(q_begin + qt * kTile + r) * prm.gate_stride + head]);
+        inv /= 1.0f + ptx::ex2(-z * ptx::kLog2e);
+      }
       __nv_bfloat16* dst = prm.out + static_cast<int64_t>(q_begin + qt * kTile + r) * prm.ld_out + head * kD + g * 64;
 #pragma unroll
       for (int c = 0; c < 8; ++c) {
@@ -395,7 +402,7 @@ extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const
                                        const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                                        int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
                                        int64_t num_pages, int variant, const int32_t* work, const int32_t* n_work, int work_items,
-                                       Status* status, cudaStream_t stream) {
+                                       const void* gate, int64_t gate_stride, Status* status, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
   if (work != nullptr && work_items <= 0) return 0;
   if (n_q <= 0 || n_kv <= 0 || n_q % n_kv != 0 || q_stride % 8 != 0 || out_stride % 8 != 0 ||
@@ -423,6 +430,8 @@ extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const
   prm.v_sbo = 1024;         // 8 KV rows of 128 bytes
   prm.work = work;
   prm.n_work = work != nullptr ? n_work : nullptr;
+  prm.gate = static_cast<const __nv_bfloat16*>(gate);
+  prm.gate_stride = gate_stride;
   (void)variant;
   static DeviceOnce attr_once;
   if (const int rc = attr_once.run([&] {

@@ -1,0 +1,168 @@
+// True 32-bit forms of the matrix product, SwiGLU, row gather and paged attention, for models that run with f32
+// activations on the GPU. Plain FMA throughout: no TF32 or other reduced-precision matrix mode.
+#include <cstdint>
+#include "b2/api.h"
+#include "b2/elem.cuh"
+#include "b2/launch.h"
+#include "b2/mixers.h"
+#include "b2/ptx.cuh"
+#include "b2/vec.cuh"
+
+namespace b2 {
+namespace {
+
+constexpr int kBM = 64, kBN = 64, kBK = 16;
+
+// 64 x 64 tile, 256 threads of 4 x 4 outputs.
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, float* __restrict__ y, int M, int N,
+                                                       int K, int64_t ldx, int64_t ldw, int64_t ldy) {
+  ptx::grid_dep_sync();
+  __shared__ float xs[kBK][kBM + 4], ws[kBK][kBN + 4];
+  const int m0 = blockIdx.y * kBM, n0 = blockIdx.x * kBN;
+  const int tm = (threadIdx.x >> 4) * 4, tn = (threadIdx.x & 15) * 4;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < K; k0 += kBK) {
+    for (int i = threadIdx.x; i < kBM * kBK; i += 256) {
+      const int r = i / kBK, c = i % kBK;
+      xs[c][r] = m0 + r < M && k0 + c < K ? x[(m0 + r) * ldx + k0 + c] : 0.0f;
+      ws[c][r] = n0 + r < N && k0 + c < K ? w[(n0 + r) * ldw + k0 + c] : 0.0f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < kBK; ++k) {
+      float a[4], b[4];
+      load_f32<4>(&xs[k][tm], a);
+      load_f32<4>(&ws[k][tn], b);
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (m0 + tm + i < M && n0 + tn + j < N) y[(m0 + tm + i) * ldy + n0 + tn + j] = acc[i][j];
+}
+
+__global__ void swiglu_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, int64_t total, int ffn) {
+  ptx::grid_dep_sync();
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
+  if (i >= total) return;
+  const int64_t r = i / ffn;
+  const int c = static_cast<int>(i % ffn);
+  const float* p = gu + r * 2 * ffn + (c / 16) * 32 + c % 16;
+  out[i] = p[0] / (1.0f + expf(-p[0])) * p[16];
+}
+
+__global__ void gather_rows_f32_kernel(const float* __restrict__ src, const int64_t* __restrict__ index, float* __restrict__ out, int cols,
+                                       int64_t rows_src, Status* status) {
+  ptx::grid_dep_sync();
+  const int64_t s = index[blockIdx.x];
+  if (!B2_ASSERT(status, s >= 0 && s < rows_src, kSiteKvIndex, s, rows_src)) return;
+  for (int c = threadIdx.x; c < cols; c += blockDim.x) out[static_cast<int64_t>(blockIdx.x) * cols + c] = src[s * cols + c];
+}
+
+// One warp per (row, head): 32 keys at a time, a key per lane for the scores, a value column per lane for the output.
+constexpr int kAttnMax = 256;
+__global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__ q, const float* __restrict__ kc, const float* __restrict__ vc,
+                                                       float* __restrict__ out, const int32_t* __restrict__ row_seq,
+                                                       const int32_t* __restrict__ positions, const int32_t* __restrict__ tables, int rows, int seqs,
+                                                       int max_blocks, int n_q, int n_kv, int dim, int vdim, int page_size, float scale,
+                                                       int64_t num_pages, const float* __restrict__ gate, int64_t gate_stride, Status* status) {
+  ptx::grid_dep_sync();
+  __shared__ float q_sm[4][kAttnMax];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int64_t idx = static_cast<int64_t>(blockIdx.x) * 4 + warp;
+  if (idx >= static_cast<int64_t>(rows) * n_q) return;
+  const int row = static_cast<int>(idx / n_q), head = static_cast<int>(idx % n_q), kvh = head / (n_q / n_kv);
+  float* dst = out + (static_cast<int64_t>(row) * n_q + head) * vdim;
+  const int seq = row_seq[row];
+  const int ctx = seq >= 0 ? positions[row] + 1 : 0;
+  if (seq < 0 || !B2_ASSERT(status, seq < seqs && ctx >= 1 && (ctx - 1) / page_size < max_blocks, kSiteKvIndex, seq, ctx)) {
+    for (int c = lane; c < vdim; c += 32) dst[c] = 0.0f;
+    return;
+  }
+  for (int i = lane; i < dim; i += 32) q_sm[warp][i] = q[(static_cast<int64_t>(row) * n_q + head) * dim + i];
+  __syncwarp();
+  const int32_t* table = tables + static_cast<int64_t>(seq) * max_blocks;
+  auto slot_of = [&](int pos) -> int64_t {
+    int64_t page = table[pos / page_size];
+    if (!B2_ASSERT(status, page >= 0 && page < num_pages, kSiteKvIndex, page, num_pages)) page = 0;
+    return (page * n_kv + kvh) * page_size + pos % page_size;
+  };
+  float m = -INFINITY, l = 0.0f, o[kAttnMax / 32];
+#pragma unroll
+  for (int j = 0; j < kAttnMax / 32; ++j) o[j] = 0.0f;
+  for (int p0 = 0; p0 < ctx; p0 += 32) {
+    const int pos = p0 + lane;
+    int64_t slot = 0;
+    float s = -INFINITY;
+    if (pos < ctx) {
+      slot = slot_of(pos);
+      const float* k = kc + slot * dim;
+      float dot = 0.0f;
+      for (int i = 0; i < dim; ++i) dot = fmaf(q_sm[warp][i], k[i], dot);
+      s = dot * scale;
+    }
+    const float m_new = fmaxf(m, warp_max(s));
+    const float corr = expf(m - m_new), p = pos < ctx ? expf(s - m_new) : 0.0f;
+    m = m_new;
+    l = l * corr + p;
+#pragma unroll
+    for (int j = 0; j < kAttnMax / 32; ++j) o[j] *= corr;
+    const int n = min(32, ctx - p0);
+    for (int t = 0; t < n; ++t) {
+      const float pt = __shfl_sync(0xffffffffu, p, t);
+      const float* v = vc + __shfl_sync(0xffffffffu, slot, t) * vdim;
+#pragma unroll
+      for (int j = 0; j < kAttnMax / 32; ++j)
+        if (lane + 32 * j < vdim) o[j] = fmaf(pt, v[lane + 32 * j], o[j]);
+    }
+  }
+  float f = 1.0f / warp_sum(l);
+  if (gate != nullptr) f *= sigmoid_f32(gate[row * gate_stride + head]);
+#pragma unroll
+  for (int j = 0; j < kAttnMax / 32; ++j)
+    if (lane + 32 * j < vdim) dst[lane + 32 * j] = o[j] * f;
+}
+
+}  // namespace
+}  // namespace b2
+
+using namespace b2;
+
+extern "C" int b2_gemm_f32(const float* x, const float* w, float* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy, cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if (K <= 0 || (M + kBM - 1) / kBM > 65535) return -kBadArgument;
+  launch_pdl(gemm_f32_kernel, dim3((N + kBN - 1) / kBN, (M + kBM - 1) / kBM), dim3(256), 0, stream, x, w, y, M, N, K, ldx, ldw, ldy);
+  return last_launch_rc();
+}
+
+extern "C" int b2_swiglu_f32(const float* gate_up, float* out, int rows, int ffn, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (ffn <= 0 || ffn % 16 != 0) return -kBadArgument;
+  const int64_t total = static_cast<int64_t>(rows) * ffn;
+  launch_pdl(swiglu_f32_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, stream, gate_up, out, total, ffn);
+  return last_launch_rc();
+}
+
+extern "C" int b2_gather_rows_f32(const float* src, const int64_t* index, float* out, int rows_out, int cols, int64_t rows_src, Status* status,
+                                  cudaStream_t stream) {
+  if (rows_out <= 0) return 0;
+  launch_pdl(gather_rows_f32_kernel, dim3(rows_out), dim3(128), 0, stream, src, index, out, cols, rows_src, status);
+  return last_launch_rc();
+}
+
+extern "C" int b2_attn_f32(const float* q, const float* k_cache, const float* v_cache, float* out, const int32_t* row_seq, const int32_t* positions,
+                           const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv, int dim, int vdim, int page_size,
+                           float scale, int64_t num_pages, const float* gate, int64_t gate_stride, Status* status, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n_kv <= 0 || n_q % n_kv != 0 || dim <= 0 || dim > kAttnMax || vdim <= 0 || vdim > kAttnMax || page_size <= 0) return -kBadArgument;
+  const int64_t warps = static_cast<int64_t>(rows) * n_q;
+  launch_pdl(attn_f32_kernel, dim3(static_cast<unsigned>((warps + 3) / 4)), dim3(128), 0, stream, q, k_cache, v_cache, out, row_seq, positions,
+             block_tables, rows, seqs, max_blocks, n_q, n_kv, dim, vdim, page_size, scale, num_pages, gate, gate_stride, status);
+  return last_launch_rc();
+}

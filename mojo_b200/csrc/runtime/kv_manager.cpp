@@ -26,9 +26,13 @@ uint64_t hash_page(uint64_t parent, const int32_t* tokens, int n) {
   return h == 0 ? 1 : h;  // 0 is reserved for "not cached"
 }
 
-KVCacheManager::KVCacheManager(int64_t num_pages, int page_size, bool enable_prefix_cache)
-    : num_pages_(num_pages), page_size_(page_size), prefix_(enable_prefix_cache) {
+KVCacheManager::KVCacheManager(int64_t num_pages, int page_size, bool enable_prefix_cache, int64_t state_slots)
+    : num_pages_(num_pages), page_size_(page_size), prefix_(enable_prefix_cache), state_slots_(state_slots) {
   if (num_pages <= 0 || page_size <= 0) throw std::invalid_argument("KVCacheManager: num_pages and page_size must be positive");
+  if (state_slots < 0) throw std::invalid_argument("KVCacheManager: state_slots must not be negative");
+  if (state_slots > 0 && enable_prefix_cache)
+    throw std::invalid_argument("KVCacheManager: a prefix cache cannot be combined with recurrent state");
+  for (int64_t s = 0; s < state_slots; ++s) free_state_.push_back(static_cast<int32_t>(s));
   refcount_.assign(num_pages, 0);
   page_hash_.assign(num_pages, 0);
   evict_pos_.resize(num_pages);
@@ -78,6 +82,11 @@ int64_t KVCacheManager::pages_needed(int64_t seq_id, int64_t total_tokens) const
 int64_t KVCacheManager::add_sequence(int64_t seq_id, const int32_t* tokens, int64_t n_tokens) {
   if (seqs_.count(seq_id)) throw std::invalid_argument("KVCacheManager: sequence already exists");
   Seq s;
+  if (state_slots_ > 0) {
+    if (free_state_.empty()) throw std::runtime_error("KVCacheManager: no free state slot");
+    s.state_slot = free_state_.front();
+    free_state_.pop_front();
+  }
   int64_t matched = 0;
   if (prefix_ && tokens != nullptr) {
     // Never match the whole prompt: at least one token must be computed to produce logits.
@@ -140,12 +149,23 @@ void KVCacheManager::free_sequence(int64_t seq_id) {
   if (it == seqs_.end()) return;
   // Leaves first, so that eviction (oldest first) drops the end of a cached prefix before its root.
   for (auto p = it->second.pages.rbegin(); p != it->second.pages.rend(); ++p) release_page(*p);
+  if (it->second.state_slot >= 0) free_state_.push_back(it->second.state_slot);
   seqs_.erase(it);
+}
+
+std::pair<int32_t, int32_t> KVCacheManager::advance_state(int64_t seq_id, int64_t first_pos) {
+  auto it = seqs_.find(seq_id);
+  if (it == seqs_.end() || it->second.state_slot < 0) throw std::invalid_argument("KVCacheManager::advance_state: sequence has no state slot");
+  Seq& s = it->second;
+  const int32_t read = first_pos == 0 ? -1 : 2 * s.state_slot + s.state_parity;
+  s.state_parity ^= 1;
+  return {read, 2 * s.state_slot + s.state_parity};
 }
 
 bool KVCacheManager::fork(int64_t src, int64_t dst, std::vector<std::pair<int64_t, int64_t>>* copies) {
   auto it = seqs_.find(src);
   if (it == seqs_.end() || seqs_.count(dst)) throw std::invalid_argument("KVCacheManager::fork: bad sequence ids");
+  if (state_slots_ > 0) throw std::invalid_argument("KVCacheManager::fork: a sequence with recurrent state cannot be forked");
   const Seq& a = it->second;
   Seq b;
   b.reserved_tokens = a.reserved_tokens;
@@ -211,6 +231,12 @@ std::string KVCacheManager::check_invariants() const {
     if (places != 1) err << "page " << p << ": in " << places << " places; ";
     if (seen[p] && refs[p]) err << "page " << p << ": free and referenced; ";
   }
+  std::vector<int> slot_owners(state_slots_, 0);
+  for (int32_t s : free_state_) slot_owners[s] += 1;
+  for (const auto& kv : seqs_)
+    if (kv.second.state_slot >= 0) slot_owners[kv.second.state_slot] += 1;
+  for (int64_t s = 0; s < state_slots_; ++s)
+    if (slot_owners[s] != 1) err << "state slot " << s << ": in " << slot_owners[s] << " places; ";
   for (const auto& kv : cache_)
     if (page_hash_[kv.second] != kv.first) err << "cache entry for page " << kv.second << " has stale hash; ";
   return err.str();

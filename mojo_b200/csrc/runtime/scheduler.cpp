@@ -57,18 +57,16 @@ bool Scheduler::preempt_one(int64_t keep_id, Batch* b) {
   return victim != keep_id;
 }
 
-namespace {
-struct Entry {
-  int64_t id;
-  int64_t n;
-};
-}  // namespace
-
 void Scheduler::emit(Request& r, int64_t n, Batch* b) {
   const int64_t start = r.computed;
   b->seq_ids.push_back(r.id);
   b->q_lens.push_back(static_cast<int32_t>(n));
   b->ctx_lens.push_back(static_cast<int32_t>(start + n));
+  if (kv_->state_slots() > 0) {
+    const auto banks = kv_->advance_state(r.id, start);
+    b->seq_state.push_back(banks.first);
+    b->seq_state.push_back(banks.second);
+  }
   for (int64_t i = 0; i < n; ++i) {
     b->token_ids.push_back(r.tokens[start + i]);
     b->positions.push_back(static_cast<int32_t>(start + i));
@@ -109,7 +107,7 @@ Batch Scheduler::step() {
   pending_commits_.emplace_back();
   Batch b;
   int64_t budget = cfg_.max_num_batched_tokens;
-  std::vector<Entry> entries;
+  std::vector<std::pair<int64_t, int64_t>> entries;   // (sequence, tokens to run)
 
   // ---- 1. sequences already running ----
   size_t i = 0;
@@ -138,15 +136,18 @@ Batch Scheduler::step() {
     // a sequence preempted in this very step waits for the next one
     if (std::find(b.preempted.begin(), b.preempted.end(), id) != b.preempted.end()) break;
     Request& r = reqs_.at(id);
+    if (!kv_->has_sequence(id) && kv_->state_slots() > 0 && kv_->free_state_slots() == 0) break;   // every state slot is taken
     if (!kv_->has_sequence(id)) r.computed = kv_->add_sequence(id, r.tokens.data(), static_cast<int64_t>(r.tokens.size()));
     const int64_t pending = static_cast<int64_t>(r.tokens.size()) - r.computed;
     int64_t n = std::min(pending, budget);
-    if (!cfg_.enable_chunked_prefill && n < pending && pending <= cfg_.max_num_batched_tokens) break;
+    // a request that stays in the queue gives its state slot back (pages it may have matched in the prefix cache stay)
+    const auto stay = [&] { if (kv_->state_slots() > 0) kv_->free_sequence(id); };
+    if (!cfg_.enable_chunked_prefill && n < pending && pending <= cfg_.max_num_batched_tokens) { stay(); break; }
     // Admission needs the pages of the whole known sequence, not just this chunk: a request that can
     // start but not finish its prompt would only be preempted again.
     const int64_t need_all = kv_->pages_needed(id, static_cast<int64_t>(r.tokens.size()) + 1);
-    if (need_all + cfg_.decode_reserve_pages > kv_->available_pages()) break;
-    if (!kv_->reserve(id, r.computed + n)) break;
+    if (need_all + cfg_.decode_reserve_pages > kv_->available_pages()) { stay(); break; }
+    if (!kv_->reserve(id, r.computed + n)) { stay(); break; }
     waiting_.pop_front();
     running_.push_back(id);
     r.status = SeqStatus::kRunning;
@@ -154,22 +155,74 @@ Batch Scheduler::step() {
     budget -= n;
   }
 
-  // ---- 3. flatten: decode sequences first ----
-  std::stable_partition(entries.begin(), entries.end(), [](const Entry& e) { return e.n == 1; });
-  b.cu_q.push_back(0);
-  for (const Entry& e : entries) {
-    Request& r = reqs_.at(e.id);
-    if (e.n == 1) ++b.num_decode; else ++b.num_prefill;
-    emit(r, e.n, &b);
-  }
-  b.num_tokens = static_cast<int64_t>(b.token_ids.size());
-  for (int64_t id : b.seq_ids) b.max_blocks = std::max<int>(b.max_blocks, static_cast<int>(kv_->block_table(id).size()));
-  b.block_tables.assign(b.seq_ids.size() * static_cast<size_t>(b.max_blocks), 0);
-  for (size_t s = 0; s < b.seq_ids.size(); ++s) {
-    const auto& t = kv_->block_table(b.seq_ids[s]);
-    std::copy(t.begin(), t.end(), b.block_tables.begin() + s * b.max_blocks);
-  }
+  flatten(entries, &b);
   if (b.seq_ids.empty()) pending_commits_.pop_back();   // nothing was scheduled: no batch to confirm later
+  return b;
+}
+
+// Decode sequences first, then prefill chunks; token arrays, block tables and sample rows of the batch.
+void Scheduler::flatten(std::vector<std::pair<int64_t, int64_t>>& entries, Batch* b) {
+  std::stable_partition(entries.begin(), entries.end(), [](const std::pair<int64_t, int64_t>& e) { return e.second == 1; });
+  b->cu_q.push_back(0);
+  for (const auto& e : entries) {
+    if (e.second == 1) ++b->num_decode; else ++b->num_prefill;
+    emit(reqs_.at(e.first), e.second, b);
+  }
+  b->num_tokens = static_cast<int64_t>(b->token_ids.size());
+  for (int64_t id : b->seq_ids) b->max_blocks = std::max<int>(b->max_blocks, static_cast<int>(kv_->block_table(id).size()));
+  b->block_tables.assign(b->seq_ids.size() * static_cast<size_t>(b->max_blocks), 0);
+  for (size_t s = 0; s < b->seq_ids.size(); ++s) {
+    const auto& t = kv_->block_table(b->seq_ids[s]);
+    std::copy(t.begin(), t.end(), b->block_tables.begin() + s * b->max_blocks);
+  }
+}
+
+Batch Scheduler::run_tokens(const std::vector<std::pair<int64_t, std::vector<int32_t>>>& entries) {
+  if (auto_commit_)
+    while (!pending_commits_.empty()) commit_step();
+  // everything that can be refused is checked before the first sequence changes
+  int64_t pages = 0, fresh = 0, total = 0;
+  for (size_t i = 0; i < entries.size(); ++i) {
+    const int64_t id = entries[i].first, n = static_cast<int64_t>(entries[i].second.size());
+    if (n == 0) throw std::invalid_argument("Scheduler::run_tokens: an entry without tokens");
+    for (size_t j = 0; j < i; ++j)
+      if (entries[j].first == id) throw std::invalid_argument("Scheduler::run_tokens: a request appears twice in one step");
+    const Request* r = request(id);
+    if (r != nullptr && (r->status != SeqStatus::kRunning || r->computed != static_cast<int64_t>(r->tokens.size())))
+      throw std::invalid_argument("Scheduler::run_tokens: the request has tokens of its own left to run");
+    const int64_t len = (r != nullptr ? r->computed : 0) + n;
+    if (len > cfg_.max_model_len) throw std::invalid_argument("Scheduler::run_tokens: sequence longer than max_model_len");
+    if (r == nullptr) ++fresh;
+    pages += kv_->pages_needed(id, len);
+    total += n;
+  }
+  if (total > cfg_.max_num_batched_tokens) throw std::invalid_argument("Scheduler::run_tokens: more tokens than max_num_batched_tokens");
+  if (static_cast<int64_t>(running_.size()) + fresh > cfg_.max_num_seqs) throw std::runtime_error("Scheduler::run_tokens: more live requests than max_num_seqs");
+  if (kv_->state_slots() > 0 && fresh > kv_->free_state_slots()) throw std::runtime_error("Scheduler::run_tokens: out of state slots");
+  if (pages > kv_->available_pages()) throw std::runtime_error("Scheduler::run_tokens: out of KV pages");
+  pending_commits_.emplace_back();
+  Batch b;
+  std::vector<std::pair<int64_t, int64_t>> plan;
+  for (const auto& e : entries) {
+    const int64_t id = e.first, n = static_cast<int64_t>(e.second.size());
+    auto it = reqs_.find(id);
+    if (it == reqs_.end()) {
+      Request r;
+      r.id = id;
+      r.prompt_len = n;
+      r.max_new_tokens = cfg_.max_model_len;
+      r.status = SeqStatus::kRunning;
+      it = reqs_.emplace(id, std::move(r)).first;
+      kv_->add_sequence(id, nullptr, 0);
+      running_.push_back(id);
+    }
+    Request& r = it->second;
+    r.tokens.insert(r.tokens.end(), e.second.begin(), e.second.end());
+    kv_->reserve(id, static_cast<int64_t>(r.tokens.size()));
+    plan.emplace_back(id, n);
+  }
+  flatten(plan, &b);
+  if (b.seq_ids.empty()) pending_commits_.pop_back();
   return b;
 }
 

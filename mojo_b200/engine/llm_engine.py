@@ -53,6 +53,7 @@ class EngineConfig:
     num_pages: int | None = None          # None: size from free device memory
     gpu_memory_utilization: float = 0.9
     max_num_seqs: int = 256
+    state_slots: int | None = None        # models with recurrent state: sequences that can hold one (None: max_num_seqs)
     max_num_batched_tokens: int = 8192
     max_model_len: int = 4096
     enable_prefix_cache: bool = False
@@ -108,9 +109,19 @@ class LLMEngine:
         max_pos = int(getattr(self.model.cfg, "max_position_embeddings", 0) or 0)
         if max_pos and cfg.max_model_len > max_pos:
             cfg.max_model_len = max_pos
+        if hasattr(self.model, "reserve_positions"):
+            self.model.reserve_positions(cfg.max_model_len)
+        self.state_slots = 0
+        if getattr(self.model, "recurrent_state", False):
+            if cfg.enable_prefix_cache:
+                raise ValueError("prefix caching is not available for a model with recurrent state: a cached page does not hold the state at its end")
+            self.state_slots = cfg.state_slots or cfg.max_num_seqs
         num_pages = cfg.num_pages or self._auto_num_pages()
-        self.kv_caches = self.model.allocate_kv_cache(num_pages, cfg.page_size)
-        self.kv = self.C.KVCacheManager(num_pages, cfg.page_size, cfg.enable_prefix_cache)
+        if self.state_slots:
+            self.kv_caches = self.model.allocate_kv_cache(num_pages, cfg.page_size, self.state_slots)
+        else:
+            self.kv_caches = self.model.allocate_kv_cache(num_pages, cfg.page_size)
+        self.kv = self.C.KVCacheManager(num_pages, cfg.page_size, cfg.enable_prefix_cache, self.state_slots)
         sc = self.C.SchedulerConfig()
         sc.max_num_seqs = cfg.max_num_seqs
         sc.max_num_batched_tokens = cfg.max_num_batched_tokens
@@ -150,13 +161,15 @@ class LLMEngine:
 
     def _auto_num_pages(self) -> int:
         cfg = self.cfg
-        per_page = self.model.kv_bytes_per_page(cfg.page_size)
+        per_page = max(1, self.model.kv_bytes_per_page(cfg.page_size))     # (a model without attention layers keeps no pages)
         if self.device.type != "cuda":
             return max(64, (cfg.max_num_seqs * cfg.max_model_len) // cfg.page_size // 8)
         free, total = torch.cuda.mem_get_info(self.device)
         budget = int(total * cfg.gpu_memory_utilization) - (total - free)
         # activations of one full token budget + logits, with slack
         budget -= 8 << 30
+        if self.state_slots:
+            budget -= self.state_slots * self.model.state_bytes_per_slot()
         need_max = (cfg.max_num_seqs * cfg.max_model_len + cfg.page_size - 1) // cfg.page_size
         return int(max(16, min(budget // per_page, need_max)))
 
@@ -263,6 +276,32 @@ class LLMEngine:
             self.heartbeat.beat(self.step_count)
         self.step_count += 1
         return self._deliver(sample_ids, tokens, states, self.runner.last_logprobs, None)
+
+    def run_tokens(self, entries, end=()) -> torch.Tensor | None:
+        """One externally planned step: `entries` = [(request id, its next token ids, places among them whose logits are
+        wanted)]. All entries run as one batch from the cache and state that earlier steps left; a request is admitted at
+        its first entry. Nothing is sampled. Returns the logits [wanted, vocab] in the order of the entries and places
+        (None if nothing is wanted) and gives back what the requests in `end` hold."""
+        outs = None
+        if entries:
+            plan = [(int(rid), [int(t) for t in toks]) for rid, toks, _ in entries]
+            vocab = self.model.cfg.vocab_size
+            for (_, toks), (_, _, want) in zip(plan, entries):
+                if any(t < 0 or t >= vocab for t in toks):
+                    raise ValueError("token id outside the vocabulary")
+                if any(w < 0 or w >= len(toks) for w in want):
+                    raise ValueError("a wanted place lies outside its entry's tokens")
+            batch = self.scheduler.run_tokens(plan)
+            start = {int(rid): int(row) for rid, row in zip(batch.seq_ids, batch.cu_q[:-1])}
+            rows = np.array([start[int(rid)] + int(w) for rid, _, want in entries for w in want], dtype=np.int64)
+            self.runner.launch(batch, [], self.step_count, rows=rows)
+            self.step_count += 1
+            if len(rows):
+                outs = self.runner.last_logits
+            self.scheduler.commit_step()
+        for rid in end:
+            self.scheduler.finish(int(rid))
+        return outs
 
     def _deliver(self, sample_ids, tokens, states, step_lp, pending) -> list[RequestOutput]:
         """Book the sampled tokens of one step: append them to their sequences, time them, decide who has finished.

@@ -83,7 +83,9 @@ class ModelRunner:
         self.device = model.device
         self.cuda = self.device.type == "cuda"
         max_blocks = (cfg.max_model_len + cfg.page_size - 1) // cfg.page_size
-        nbytes = cfg.max_num_batched_tokens * 24 + cfg.max_num_seqs * (max_blocks * 4 + 64) + (1 << 16)
+        # models with recurrent state also need the sequence of every row, and rows and state banks of every sequence
+        self.has_state = bool(getattr(model, "recurrent_state", False))
+        nbytes = cfg.max_num_batched_tokens * 28 + cfg.max_num_seqs * (max_blocks * 4 + 96) + (1 << 16)
         self.staging = _Staging(nbytes, self.device)
         self.max_blocks = max_blocks
         self.h2d_bytes = 0
@@ -100,6 +102,7 @@ class ModelRunner:
         self.graph_kernel_launches = 0   # kernels executed inside replayed graphs
         self.step_events = None          # optional (start, end) CUDA events recorded around the device work
         self.last_num_tokens = 0
+        self.last_logits = None          # logits of the rows a caller asked for (`launch(..., rows=...)`)
         self.last_logprobs = None        # per sampled row (logprob of the chosen token, [(id, logprob)] top-k) of the last step, on request
         b, self.buckets = 1, []
         while b < cfg.max_num_seqs:
@@ -271,13 +274,15 @@ class ModelRunner:
         src = np.fromiter((where[int(seq_ids[i])] for i in seq_of_row), dtype=np.int32, count=neg.size)
         return neg.astype(np.int32), src
 
-    def launch(self, batch, states, step: int, prev=None) -> "StepHandle":
-        """Stage and launch one step without waiting for it. `prev` = (handle of the step launched before this one, the
+    def launch(self, batch, states, step: int, prev=None, rows=None) -> "StepHandle":
+        """Stage and launch one step without waiting for it. With `rows` (indices into the batch's token rows) nothing is
+        sampled for the scheduler: the logits of these rows are left in `last_logits`. `prev` = (handle of the step launched before this one, the
         sequence ids of its sampled rows) when the host has not read that step's tokens yet: decode rows whose input is
         such a token carry -1 in the batch and are filled on the device from the previous step's output."""
         self.last_num_tokens = int(batch.num_tokens)
-        self.last_logprobs = None
+        self.last_logprobs = self.last_logits = None
         self.steps_launched += 1
+        want = None if rows is None else np.asarray(rows, dtype=np.int64)
         plan = self._patch_plan(batch, prev)
         prev_ids = prev[0].ids if (plan is not None) else None
         top_lp = max((s.params.logprobs for s in states if s.params.logprobs is not None), default=None)
@@ -287,17 +292,23 @@ class ModelRunner:
             g = self.graphs.get(bb)
             if g is None and self.ep is None and bb not in self.failed_buckets:
                 g = self._capture(bb)          # first use of a bucket that was not captured at start-up
-            if g is not None and g.usable():
-                return self._launch_decode_graph(batch, plan, prev_ids)
+            if g is not None and g.usable() and (want is None or g.logits is not None):
+                h = self._launch_decode_graph(batch, plan, prev_ids)
+                if want is not None:
+                    self.last_logits = g.logits[torch.from_numpy(want).to(self.device)]
+                return h
         if (top_lp is None and self.use_mixed_graphs and batch.num_prefill > 0
                 and all(s.params.temperature <= 0.0 for s in states)):
             key = self.mixed_key(int(batch.num_tokens), int(batch.num_decode), int(batch.num_prefill))
-            if key is not None:
+            if key is not None and (want is None or len(want) <= _MixedGraph.sample_capacity(*key)):
                 g = self.mixed_graphs.get(key)
                 if g is None and key not in self.failed_buckets:
                     g = self._capture_mixed(key)      # first use of a shape that was not captured at start-up
-                if g is not None:
-                    return self._launch_mixed_graph(g, batch, plan, prev_ids)
+                if g is not None and (want is None or g.logits is not None):
+                    h = self._launch_mixed_graph(g, batch, plan, prev_ids, want)
+                    if want is not None:
+                        self.last_logits = g.logits[:len(want)].clone()
+                    return h
         st = self.staging
         st.begin()
         T, B = int(batch.num_tokens), int(batch.num_seqs)
@@ -307,8 +318,14 @@ class ModelRunner:
         seg_cu = st.put(batch.cu_q, np.int32)
         seg_ctx = st.put(batch.ctx_lens, np.int32)
         seg_bt = st.put(batch.block_tables, np.int32)
-        sample_rows = batch.sample_rows
+        sample_rows = batch.sample_rows if want is None else want
         S = len(sample_rows)
+        seg_state = None
+        if self.has_state:
+            cu = batch.cu_q
+            seg_rseq = st.put(np.repeat(np.arange(B, dtype=np.int32), np.diff(cu)), np.int32)
+            seg_srows = st.put(np.stack([cu[:-1], cu[1:]], axis=1), np.int32)
+            seg_state = st.put(batch.seq_state, np.int32)
         seg_rows = st.put(sample_rows.astype(np.int64), np.int64)
         seg_work, n_items = None, 0
         if self.cuda and batch.num_prefill > 0 and getattr(self.model, "supports_static_attention", lambda *_: False)(self.cfg.page_size):
@@ -332,9 +349,13 @@ class ModelRunner:
         slots = st.view(seg_slot, torch.int64)
         positions = st.view(seg_pos, torch.int32)
         ctx_np = batch.ctx_lens
+        seq = None
+        if seg_state is not None:
+            nd = int(batch.num_decode)
+            seq = ops.SeqRows(st.view(seg_rseq, torch.int32), st.view(seg_srows, torch.int32), st.view(seg_state, torch.int32), nd, nd, B - nd)
         meta = ops.AttnMeta(st.view(seg_cu, torch.int32), st.view(seg_ctx, torch.int32), st.view(seg_bt, torch.int32),
                             batch.num_decode, batch.max_q_len, int(ctx_np.max()) if B else 0,
-                            work=st.view(seg_work, torch.int32) if seg_work is not None else None, n_items=n_items)
+                            work=st.view(seg_work, torch.int32) if seg_work is not None else None, n_items=n_items, seq=seq)
         rows = st.view(seg_rows, torch.int64)
         if self.step_events is not None:
             self.step_events[0].record()
@@ -346,6 +367,11 @@ class ModelRunner:
         if S == 0:
             # pure mid-prompt chunks: run the layers for their KV side effect, nothing to sample
             self.model.forward(token_ids, positions, slots, meta, self.kv_caches, rows)
+            if self.step_events is not None:
+                self.step_events[1].record()
+            return self._finish_launch(None, 0)
+        if want is not None:
+            self.last_logits = self.model.forward(token_ids, positions, slots, meta, self.kv_caches, rows)
             if self.step_events is not None:
                 self.step_events[1].record()
             return self._finish_launch(None, 0)
@@ -416,9 +442,11 @@ class ModelRunner:
     def _execute_decode_graph(self, batch) -> list[int]:
         return self.collect(self._launch_decode_graph(batch))
 
-    def _launch_mixed_graph(self, g: "_MixedGraph", batch, plan=None, prev_ids=None) -> "StepHandle":
-        S = int(len(batch.sample_rows))
-        self.h2d_bytes = g.stage(batch, plan)
+    def _launch_mixed_graph(self, g: "_MixedGraph", batch, plan=None, prev_ids=None, rows=None) -> "StepHandle":
+        sampled = rows is None
+        rows = batch.sample_rows if sampled else rows
+        S = int(len(rows)) if sampled else 0      # rows asked for by a caller: their logits are read, not their arg-max
+        self.h2d_bytes = g.stage(batch, rows, plan)
         if plan is not None:
             self._patch(g.tok, g.fix_rows, g.fix_src, prev_ids, len(plan[0]))
         if self.step_events is not None:
@@ -450,12 +478,13 @@ class _DecodeGraph:
         self.runner, self.bb = runner, bb
         mb = runner.max_blocks
         dev = runner.device
-        # host layout: tok i64[bb] | slot i64[bb] | pos i32[bb] | ctx i32[bb] | bt i32[bb * mb]
+        # host layout: tok i64[bb] | slot i64[bb] | pos i32[bb] | ctx i32[bb] | bt i32[bb * mb] | fix i32[2 bb] | state i32[2 bb]
         self.o_tok, self.o_slot = 0, 8 * bb
         self.o_pos, self.o_ctx = 16 * bb, 20 * bb
         self.o_bt = _align(24 * bb)
         self.o_fix = _align(self.o_bt + 4 * bb * mb)      # rows / sources of tokens still on the device (pipelined stepping)
-        nbytes = self.o_fix + 8 * bb
+        self.o_state = _align(self.o_fix + 8 * bb)
+        nbytes = self.o_state + 8 * bb
         self.host = torch.zeros(nbytes, dtype=torch.uint8, pin_memory=True)
         self.np = self.host.numpy()
         self.dev = torch.zeros(nbytes, dtype=torch.uint8, device=dev)
@@ -475,9 +504,17 @@ class _DecodeGraph:
         self.h_pos = self.np[self.o_pos:self.o_pos + 4 * bb].view(np.int32)
         self.h_ctx = self.np[self.o_ctx:self.o_ctx + 4 * bb].view(np.int32)
         self.h_bt = self.np[self.o_bt:self.o_bt + 4 * bb * mb].view(np.int32).reshape(bb, mb)
+        self.h_state = self.np[self.o_state:self.o_state + 8 * bb].view(np.int32).reshape(bb, 2)
         self.h_slot[:] = -1
+        self.h_state[:] = -1
         self.dev.copy_(self.host)
-        self.meta = ops.AttnMeta(self.cu, self.ctx, self.bt, bb, 1, runner.cfg.max_model_len)
+        seq = None
+        if runner.has_state:
+            row = torch.arange(bb, dtype=torch.int32, device=dev)
+            seq = ops.SeqRows(row, torch.stack([row, row + 1], dim=1).contiguous(), d[self.o_state:self.o_state + 8 * bb].view(torch.int32).view(bb, 2),
+                              bb, bb, 0)
+        self.meta = ops.AttnMeta(self.cu, self.ctx, self.bt, bb, 1, runner.cfg.max_model_len, seq=seq)
+        self.logits = None       # the graph's logits, where the forward pass returns them
         model, caches = runner.model, runner.kv_caches
 
         comm = getattr(model, "comm", None)
@@ -489,8 +526,8 @@ class _DecodeGraph:
                 comm.begin_graph()
             if getattr(model, "greedy_in_forward", False):
                 return model.forward(self.tok, self.pos, self.slot, self.meta, caches, None, greedy=True)
-            logits = model.forward(self.tok, self.pos, self.slot, self.meta, caches, None)
-            return ops.argmax(logits)
+            self.logits = model.forward(self.tok, self.pos, self.slot, self.meta, caches, None)
+            return ops.argmax(self.logits)
 
         # one eager pass on a side stream: one-time kernel attribute set-up must not happen under capture
         side = torch.cuda.Stream(device=dev)
@@ -535,6 +572,9 @@ class _DecodeGraph:
             self.h_slot[B:] = -1
             self.h_pos[B:] = 0
             self.h_ctx[B:] = 0
+        if self.runner.has_state:
+            self.h_state[:B] = batch.seq_state
+            self.h_state[B:] = -1
         bt = batch.block_tables
         self.h_bt[:B, :bt.shape[1]] = bt
         self.dev.copy_(self.host, non_blocking=True)
@@ -548,11 +588,17 @@ class _MixedGraph:
     that varies (ids, positions, slots, context lengths, block tables, work items and their count, rows to sample)
     from the device copy of that block."""
 
+    @staticmethod
+    def sample_capacity(tb: int, db: int, pb: int) -> int:
+        """Rows that can be sampled in one step."""
+        return max(1, min(db + pb, tb))
+
     def __init__(self, runner: ModelRunner, tb: int, db: int, pb: int):
         self.runner, self.tb, self.db, self.pb = runner, tb, db, pb
         mb, dev = runner.max_blocks, runner.device
         self.max_items = tb // 128 + pb
-        self.sb = max(1, min(db + pb, tb))          # rows that can be sampled in one step
+        self.sb = self.sample_capacity(tb, db, pb)
+        self.logits = None          # the graph's logits of the sampled rows, where the forward pass returns them
         lay, off = {}, 0
 
         def seg(name, nbytes):
@@ -565,6 +611,8 @@ class _MixedGraph:
         seg("p_cu", 4 * (pb + 1)); seg("p_ctx", 4 * pb); seg("p_bt", 4 * pb * mb)
         seg("work", 8 * self.max_items); seg("n_work", 4); seg("rows", 8 * self.sb)
         seg("fix_rows", 4 * self.sb); seg("fix_src", 4 * self.sb)   # tokens still on the device (pipelined stepping)
+        if runner.has_state:    # decode sequences are entries [0, db), prompt chunks entries [db, db + pb)
+            seg("row_seq", 4 * tb); seg("seq_rows", 8 * (db + pb)); seg("seq_state", 8 * (db + pb))
         self.nbytes = off
         self.host = torch.zeros(off, dtype=torch.uint8, pin_memory=True)
         self.dev = torch.zeros(off, dtype=torch.uint8, device=dev)
@@ -587,16 +635,22 @@ class _MixedGraph:
                   "work": hv("work", np.int32, (self.max_items, 2)), "n_work": hv("n_work", np.int32), "rows": hv("rows", np.int64),
                   "fix_rows": hv("fix_rows", np.int32), "fix_src": hv("fix_src", np.int32)}
         self.h["slot"][:] = -1
+        if runner.has_state:
+            self.h.update(row_seq=hv("row_seq", np.int32), seq_rows=hv("seq_rows", np.int32, (db + pb, 2)), seq_state=hv("seq_state", np.int32, (db + pb, 2)))
+            self.h["row_seq"][:] = -1
+            self.h["seq_state"][:] = -1
         self.dev.copy_(self.host)
         self.tok, self.slot, self.pos = dv("tok", torch.int64), dv("slot", torch.int64), dv("pos", torch.int32)
         self.rows = dv("rows", torch.int64)
         self.fix_rows, self.fix_src = dv("fix_rows", torch.int32), dv("fix_src", torch.int32)
-        n_kv = runner.kv_caches[0][0].shape[1]
         static = ops.StaticAttn(db, dv("d_ctx", torch.int32), dv("d_bt", torch.int32, (max(db, 1), mb)),
-                                ops._decode_splits(db, n_kv, runner.cfg.max_model_len) if db else 1,
+                                runner.cfg.max_model_len,
                                 dv("p_cu", torch.int32), dv("p_ctx", torch.int32), dv("p_bt", torch.int32, (pb, mb)),
                                 dv("work", torch.int32, (self.max_items, 2)), dv("n_work", torch.int32), self.max_items, tb)
-        self.meta = ops.AttnMeta(None, None, None, 0, tb, runner.cfg.max_model_len, static=static)
+        seq = None
+        if runner.has_state:
+            seq = ops.SeqRows(dv("row_seq", torch.int32), dv("seq_rows", torch.int32, (db + pb, 2)), dv("seq_state", torch.int32, (db + pb, 2)), db, db, pb)
+        self.meta = ops.AttnMeta(None, None, None, 0, tb, runner.cfg.max_model_len, static=static, seq=seq)
         model, caches = runner.model, runner.kv_caches
         comm = getattr(model, "comm", None)
 
@@ -605,7 +659,8 @@ class _MixedGraph:
                 comm.begin_graph()
             if getattr(model, "greedy_in_forward", False):
                 return model.forward(self.tok, self.pos, self.slot, self.meta, caches, self.rows, greedy=True)
-            return ops.argmax(model.forward(self.tok, self.pos, self.slot, self.meta, caches, self.rows))
+            self.logits = model.forward(self.tok, self.pos, self.slot, self.meta, caches, self.rows)
+            return ops.argmax(self.logits)
 
         # one eager pass on a side stream (one-time kernel attribute set-up must not happen under capture); the block
         # is all padding at this point: slots -1, no decode context, no work items, so the pass touches no KV page
@@ -624,8 +679,9 @@ class _MixedGraph:
         self.kernel_launches = ops.launch_count - before
         ops.launch_count = before
 
-    def stage(self, batch, plan=None) -> int:
-        """Fill the pinned block from the scheduler's batch and start its copy. Returns the bytes copied."""
+    def stage(self, batch, rows, plan=None) -> int:
+        """Fill the pinned block from the scheduler's batch (`rows`: token rows to sample) and start its copy. Returns the
+        bytes copied."""
         self.copied.synchronize()       # the previous copy out of this block has been consumed
         h = self.h
         if plan is not None:
@@ -659,7 +715,15 @@ class _MixedGraph:
             raise RuntimeError(f"mixed-step graph {self.tb, self.db, self.pb}: {n} attention work items exceed {self.max_items}")
         h["work"][:n] = work
         h["n_work"][0] = n
-        rows = batch.sample_rows
+        if self.runner.has_state:
+            seq_of, db = np.arange(B, dtype=np.int32), self.db
+            seq_of[nd:] += db - nd
+            h["row_seq"][:T] = np.repeat(seq_of, np.diff(cu))
+            h["row_seq"][T:] = -1
+            h["seq_rows"][:] = 0
+            h["seq_state"][:] = -1
+            h["seq_rows"][seq_of, 0], h["seq_rows"][seq_of, 1] = cu[:-1], cu[1:]
+            h["seq_state"][seq_of] = batch.seq_state
         S = len(rows)
         if S > self.sb:
             raise RuntimeError(f"mixed-step graph {self.tb, self.db, self.pb}: {S} rows to sample exceed {self.sb}")

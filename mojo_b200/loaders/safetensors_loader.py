@@ -64,11 +64,14 @@ class _Reader:
 
 
 def load_safetensors_into(model, path: str | Path) -> None:
-    """Fill a model from a Hugging Face checkpoint directory: Llama family, or DeepSeek-V2(-Lite) (MLA + MoE)."""
+    """Fill a model from a checkpoint directory: Llama family or DeepSeek-V2(-Lite) in Hugging Face layout, or Rekudra."""
     rd = _Reader(read_safetensors_index(path))
     cfg = model.cfg
     if getattr(cfg, "architecture", "llama") == "deepseek_v2":
         _load_deepseek_v2(model, rd)
+        return
+    if cfg.architecture == "rekudra":
+        _load_rekudra(model, rd)
         return
     model.layers.clear()
     model.load_tensor("embed", rd.get("model.embed_tokens.weight"))
@@ -140,6 +143,17 @@ def _load_deepseek_v2(model, rd: _Reader) -> None:
     model.final_norm = put(rd.get("model.norm.weight"))
     model.lm_head = put(rd.get("lm_head.weight" if rd.has("lm_head.weight") else "model.embed_tokens.weight"))
     model.finalize()
+
+
+def _load_rekudra(model, rd: _Reader) -> None:
+    """Rekudra names: `embed`, `head`, `final.norm`, and per layer `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`, `l<i>.hc<q>.*`."""
+    model.layers.clear()
+    model.load_tensor("embed", rd.get("embed"))
+    for i, spec in enumerate(model.cfg.layers):
+        names = model.tensor_shapes(spec, model.cfg.hidden_size, model.cfg.residual_streams)
+        model.load_layer(i, {n: rd.get(f"l{i}.{n}") for n in names})
+    model.load_tensor("final.norm", rd.get("final.norm"))
+    model.load_tensor("head", rd.get("head"))
 
 
 def deepseek_v2_state_dict(model) -> dict:

@@ -15,4 +15,8 @@ def build_model(cfg: ModelConfig, device="cpu", dtype=torch.float32, comm=None, 
         from .deepseek_v2 import DeepseekV2Model
 
         return DeepseekV2Model(cfg, device, dtype, comm=comm, ep=ep)
+    if cfg.architecture == "rekudra":
+        from .rekudra import RekudraModel
+
+        return RekudraModel(cfg, device, dtype, comm=comm)
     raise ValueError(f"unsupported architecture {cfg.architecture!r}")

@@ -8,8 +8,34 @@ from pathlib import Path
 
 
 @dataclass
+class RotarySpec:
+    """Rotary embedding of one layer: the first `dims` dimensions of a head turn, the rest pass. `scaling` is the Llama-3.1
+    frequency rescale (factor, low, high, original) or None."""
+    dims: int = 0
+    base: float = 10000.0
+    scaling: dict | None = None
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a decoder whose layers differ: which mixer it has, the mixer's sizes, and its feed-forward width."""
+    mixer: str = "attention"               # "attention" | "channel_delta"
+    heads: int = 0
+    kv_heads: int = 0
+    dim: int = 0                           # query / key size of a head
+    vdim: int = 0                          # value size of a head
+    conv_taps: int = 1                     # short causal convolution (1: none)
+    scale: float = 1.0                     # attention: factor on the scores
+    rot: RotarySpec = field(default_factory=RotarySpec)
+    kv_from: int | None = None             # attention: use the keys and values of this earlier layer
+    ffn: int = 0                           # feed-forward width (0: the layer has no feed-forward)
+    decay_rank: int = 0                    # delta rule: ranks of the decay and gate projections (0: taken from the checkpoint)
+    gate_rank: int = 0
+
+
+@dataclass
 class ModelConfig:
-    architecture: str = "llama"            # "llama" | "deepseek_v2"
+    architecture: str = "llama"            # "llama" | "deepseek_v2" | "rekudra"
     hidden_size: int = 4096
     num_layers: int = 32
     num_heads: int = 32
@@ -38,6 +64,10 @@ class ModelConfig:
     routed_scaling_factor: float = 1.0
     norm_topk_prob: bool = False
     rope_interleaved: bool = False
+    # decoders whose layers differ from one another, and whose residual is several mixed streams
+    layers: list[LayerSpec] | None = None
+    residual_streams: int = 1
+    embedding_scale: float = 1.0
     extra: dict = field(default_factory=dict)
 
     def to_dict(self) -> dict:
@@ -52,6 +82,8 @@ class ModelConfig:
         return self.n_routed_experts > 0
 
     def kv_bytes_per_token(self, dtype_bytes: int = 2, tp: int = 1) -> int:
+        if self.layers is not None:
+            return sum(s.kv_heads * (s.dim + s.vdim) for s in self.layers if s.mixer == "attention" and s.kv_from is None) * dtype_bytes
         if self.is_mla:
             return self.num_layers * (self.kv_lora_rank + self.qk_rope_head_dim) * dtype_bytes
         return self.num_layers * 2 * max(1, self.num_kv_heads // tp) * self.head_dim * dtype_bytes
@@ -59,6 +91,17 @@ class ModelConfig:
     def num_params(self) -> int:
         h = self.hidden_size
         emb = self.vocab_size * h * (1 if self.tie_word_embeddings else 2)
+        if self.layers is not None:
+            n = emb + h
+            for s in self.layers:
+                kv = 0 if s.kv_from is not None else s.kv_heads
+                n += h * (s.heads * s.vdim + 3 * s.ffn)
+                if s.mixer == "attention":
+                    n += h * (s.heads * (s.dim + 1) + kv * (s.dim + s.vdim))
+                else:
+                    n += h * (2 * s.kv_heads * s.dim + s.heads * (s.vdim + 1) + s.decay_rank + s.gate_rank)
+                    n += s.heads * (s.dim * s.decay_rank + s.vdim * s.gate_rank)
+            return n
         if self.architecture == "llama":
             attn = h * (self.num_heads + 2 * self.num_kv_heads) * self.head_dim + self.num_heads * self.head_dim * h
             mlp = 3 * h * self.intermediate_size
@@ -73,6 +116,8 @@ class ModelConfig:
     @staticmethod
     def from_hf(path: str | Path) -> "ModelConfig":
         cfg = json.loads((Path(path) / "config.json").read_text())
+        if cfg.get("architecture") in LAYERED_ARCHITECTURES:
+            return ModelConfig.from_layered(cfg)
         arch = (cfg.get("architectures") or ["LlamaForCausalLM"])[0]
         n_heads = cfg["num_attention_heads"]
         c = ModelConfig(
@@ -97,6 +142,40 @@ class ModelConfig:
             c.routed_scaling_factor = cfg.get("routed_scaling_factor", 1.0); c.norm_topk_prob = cfg.get("norm_topk_prob", False)
             c.rope_interleaved = True
         return c
+
+
+    @staticmethod
+    def from_layered(cfg: dict) -> "ModelConfig":
+        """A config that lists its layers one by one (`layers[i]`: type, mixer sizes, feed-forward)."""
+        layers = []
+        for i, entry in enumerate(cfg["layers"]):
+            m, mlp = entry["mixer"], entry.get("mlp")
+            if entry["type"] not in ("attention", "channel_delta"):
+                raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}")
+            if mlp is not None and mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            rot = m.get("rot") or {}
+            spec = LayerSpec(
+                mixer=entry["type"], heads=m["heads"], kv_heads=m["kv_heads"], dim=m["dim"], vdim=m["vdim"], conv_taps=m.get("conv") or 1,
+                scale=m.get("scale", 1.0), rot=RotarySpec(rot.get("dims", 0), rot.get("base", 10000.0), rot.get("scaling")),
+                kv_from=m.get("kv_from"), ffn=mlp["ff"] if mlp is not None else 0)
+            if spec.kv_from is not None:
+                src = layers[spec.kv_from] if 0 <= spec.kv_from < i else None
+                if src is None or src.mixer != "attention" or src.kv_from is not None:
+                    raise ValueError(f"layer {i}: kv_from must name an earlier attention layer with keys and values of its own")
+                if (src.kv_heads, src.dim, src.vdim) != (spec.kv_heads, spec.dim, spec.vdim):
+                    raise ValueError(f"layer {i}: head sizes differ from those of layer {spec.kv_from}, whose keys and values it uses")
+            layers.append(spec)
+        first = next((s for s in layers if s.mixer == "attention"), layers[0])
+        return ModelConfig(architecture=LAYERED_ARCHITECTURES[cfg["architecture"]], hidden_size=cfg["width"], num_layers=len(layers),
+                           num_heads=first.heads, num_kv_heads=first.kv_heads, head_dim=first.dim,
+                           intermediate_size=max((s.ffn for s in layers), default=0), vocab_size=cfg["vocab"], rms_norm_eps=cfg["norm"]["eps"],
+                           max_position_embeddings=0, layers=layers, residual_streams=cfg.get("streams", 1),
+                           embedding_scale=cfg.get("embedding", {}).get("scale", 1.0))
+
+
+# `architecture` values of configs that list their layers -> model class key
+LAYERED_ARCHITECTURES = {"Rekudra": "rekudra"}
 
 
 def tiny_llama() -> ModelConfig:
@@ -139,12 +218,44 @@ def tiny_deepseek() -> ModelConfig:
                        moe_intermediate_size=128, first_k_dense_replace=1, rope_interleaved=True)
 
 
+def rekudra(width: int, n_layers: int, heads: int, kv_heads: int, dim: int, ffn: int, vocab: int, streams: int = 4, taps: int = 4) -> ModelConfig:
+    """A Rekudra decoder: pairs of a delta-rule layer and an attention layer with feed-forward; the second half of the
+    attention layers shares the keys and values of the last one that has its own."""
+    rot = RotarySpec(dim, 500000.0, {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192})
+    layers, own = [], None
+    for i in range(n_layers // 2):
+        layers.append(LayerSpec("channel_delta", heads, heads, dim, dim, taps, decay_rank=dim, gate_rank=dim))
+        shared = own if i >= (n_layers // 2 + 1) // 2 and own is not None else None
+        layers.append(LayerSpec("attention", heads, kv_heads, dim, dim, taps, scale=dim ** -0.5, rot=rot, kv_from=shared, ffn=ffn))
+        if shared is None:
+            own = len(layers) - 1
+    return ModelConfig(architecture="rekudra", hidden_size=width, num_layers=len(layers), num_heads=heads, num_kv_heads=kv_heads, head_dim=dim,
+                       intermediate_size=ffn, vocab_size=vocab, max_position_embeddings=0, layers=layers, residual_streams=streams,
+                       embedding_scale=float(width) ** 0.5)
+
+
+def rekudra_8b() -> ModelConfig:
+    """Layers of the size of an 8B Llama's (width 4096, 32 heads of 128, FFN 14336)."""
+    return rekudra(4096, 32, 32, 8, 128, 14336, 128256)
+
+
+def rekudra_1b() -> ModelConfig:
+    return rekudra(2048, 16, 16, 4, 128, 8192, 128256)
+
+
+def tiny_rekudra() -> ModelConfig:
+    return rekudra(256, 4, 4, 2, 64, 512, 1024, streams=2)
+
+
 PRESETS = {
     "tiny-llama": tiny_llama,
     "llama-3.1-8b": llama31_8b,
     "llama-3.3-70b-fp8": llama33_70b_fp8,
     "deepseek-v2-lite": deepseek_v2_lite,
     "tiny-deepseek": tiny_deepseek,
+    "rekudra-8b": rekudra_8b,
+    "rekudra-1b": rekudra_1b,
+    "tiny-rekudra": tiny_rekudra,
 }
 
 

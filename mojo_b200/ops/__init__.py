@@ -1,4 +1,5 @@
-"""Op library. Every function takes CUDA bf16 tensors and launches a hand-written sm_100a kernel; given CPU
+"""Op library. Every function takes CUDA bf16 tensors and launches a hand-written sm_100a kernel (the matrix products,
+row gathers, attention and the sequence mixers also take CUDA f32 tensors and then compute in true f32); given CPU
 tensors it evaluates the fp32 reference in `ops.reference` instead (the oracle, and the CPU engine's compute).
 There is no other dispatch: a CUDA tensor without the built extension is an ImportError, never a quiet
 PyTorch fallback.
@@ -132,6 +133,10 @@ def gather_rows(src: torch.Tensor, index: torch.Tensor) -> torch.Tensor:
         return src[index.long()]
     C = _ext.require()
     out = torch.empty(index.numel(), src.shape[1], dtype=src.dtype, device=src.device)
+    if src.dtype == torch.float32:
+        C.gather_rows_f32(src, index, out, _state.get(src.device).status)
+        _count()
+        return out
     C.gather_rows(src, index, out, _state.get(src.device).status)
     _count()
     return out
@@ -171,10 +176,16 @@ def _launch_gemm(C, x, w, out, residual, epi, config, st) -> None:
 
 def linear(x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor | None = None, out: torch.Tensor | None = None,
            config: int = 0) -> torch.Tensor:
-    """y = x @ w.T (+ residual) on the tcgen05 GEMM. x [M, K], w [N, K], both bf16."""
+    """y = x @ w.T (+ residual) on the tcgen05 GEMM. x [M, K], w [N, K], both bf16 (both f32: the FMA kernel)."""
     if not x.is_cuda:
         return reference.linear(x, w, residual).to(x.dtype)
     C = _ext.require()
+    if x.dtype == torch.float32:
+        if out is None:
+            out = torch.empty(x.shape[0], w.shape[0], dtype=x.dtype, device=x.device)
+        C.gemm_f32(x, w, out)
+        _count()
+        return out if residual is None else out.add_(residual)
     st = _state.get(x.device)
     if out is None:
         out = torch.empty(x.shape[0], w.shape[0], dtype=x.dtype, device=x.device)
@@ -197,6 +208,13 @@ def linear_swiglu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor | None 
     if not x.is_cuda:
         return reference.linear_swiglu_interleaved(x, w_gu).to(x.dtype)
     C = _ext.require()
+    if x.dtype == torch.float32:
+        gu = linear(x, w_gu)
+        if out is None:
+            out = torch.empty(x.shape[0], w_gu.shape[0] // 2, dtype=x.dtype, device=x.device)
+        C.swiglu_f32(gu, out)
+        _count()
+        return out
     st = _state.get(x.device)
     if out is None:
         out = torch.empty(x.shape[0], w_gu.shape[0] // 2, dtype=x.dtype, device=x.device)
@@ -270,11 +288,14 @@ class AttnMeta:
                       launches exactly one CTA per item and head
       static          a `StaticAttn`: every shape and grid fixed ahead of the batch, so that the launches can sit in a
                       CUDA graph that serves any batch of its bucket
+      seq             a `SeqRows` for models with recurrent state: sequence of every row, rows and state banks of every
+                      sequence
     """
 
-    __slots__ = ("cu_q", "ctx_lens", "block_tables", "num_decode", "num_seqs", "max_q_len", "num_tokens", "max_ctx", "work", "n_items", "static")
+    __slots__ = ("cu_q", "ctx_lens", "block_tables", "num_decode", "num_seqs", "max_q_len", "num_tokens", "max_ctx", "work", "n_items", "static",
+                 "seq")
 
-    def __init__(self, cu_q, ctx_lens, block_tables, num_decode, max_q_len, max_ctx=0, work=None, n_items=0, static=None):
+    def __init__(self, cu_q, ctx_lens, block_tables, num_decode, max_q_len, max_ctx=0, work=None, n_items=0, static=None, seq=None):
         self.cu_q, self.ctx_lens, self.block_tables = cu_q, ctx_lens, block_tables
         self.num_decode = int(num_decode)
         self.num_seqs = int(ctx_lens.numel()) if ctx_lens is not None else 0
@@ -283,6 +304,7 @@ class AttnMeta:
         self.max_ctx = int(max_ctx)
         self.work, self.n_items = work, int(n_items)
         self.static = static
+        self.seq = seq
 
 
 class StaticAttn:
@@ -292,10 +314,10 @@ class StaticAttn:
     items of which the first `n_work[0]` are valid; `p_cu` / `p_ctx` / `p_bt` describe the prefill sequences only
     (`p_cu` holds absolute token rows; unused entries repeat the last offset)."""
 
-    __slots__ = ("d_rows", "d_ctx", "d_bt", "d_splits", "p_cu", "p_ctx", "p_bt", "work", "n_work", "max_items", "max_q_len")
+    __slots__ = ("d_rows", "d_ctx", "d_bt", "max_ctx", "p_cu", "p_ctx", "p_bt", "work", "n_work", "max_items", "max_q_len")
 
-    def __init__(self, d_rows, d_ctx, d_bt, d_splits, p_cu, p_ctx, p_bt, work, n_work, max_items, max_q_len):
-        self.d_rows, self.d_ctx, self.d_bt, self.d_splits = int(d_rows), d_ctx, d_bt, int(d_splits)
+    def __init__(self, d_rows, d_ctx, d_bt, max_ctx, p_cu, p_ctx, p_bt, work, n_work, max_items, max_q_len):
+        self.d_rows, self.d_ctx, self.d_bt, self.max_ctx = int(d_rows), d_ctx, d_bt, int(max_ctx)
         self.p_cu, self.p_ctx, self.p_bt = p_cu, p_ctx, p_bt
         self.work, self.n_work, self.max_items, self.max_q_len = work, n_work, int(max_items), int(max_q_len)
 
@@ -346,49 +368,72 @@ def prefill_on_tensor_core(head_dim: int, page_size: int) -> bool:
     return bool(prefill_tensor_core and head_dim == 128 and page_size == 128)
 
 
+def _decode_attention(q, k_cache, v_cache, out, ctx_lens, block_tables, head_dim: int, scale: float, max_ctx: int, gate) -> None:
+    """One query row per sequence. More than 16 query heads per KV head (the rows of one MMA tile), or head size 256 in
+    pages the TMA boxes do not fit, take the prefill kernel with chunks of one token."""
+    C, st = _ext.require(), _state.get(q.device)
+    n_kv, page = k_cache.shape[1], k_cache.shape[2]
+    n = q.shape[0]
+    if q.shape[1] // head_dim // n_kv > 16 or (head_dim == 256 and page % 32):
+        cu = torch.arange(n + 1, dtype=torch.int32, device=q.device)
+        C.attn_prefill(q, k_cache, v_cache, out, cu, ctx_lens, block_tables, head_dim, 1, scale, st.status, gate)
+        _count()
+        return
+    splits = _decode_splits(n, n_kv, max_ctx)
+    splits = max(1, min(splits, _state.ATTN_WORKSPACE_BYTES // (n * (q.shape[1] // head_dim) * (head_dim + 2) * 4)))
+    C.attn_decode(q, k_cache, v_cache, out, ctx_lens, block_tables, st.attn_ws, head_dim, splits, scale, st.status, st.attn_counters, gate)
+    _count(_decode_launches(splits, page))
+
+
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, meta: AttnMeta, scale: float,
-                    head_dim: int, out: torch.Tensor | None = None) -> torch.Tensor:
-    """Causal GQA attention over the paged cache. q, out: [T, n_q * D]."""
+                    head_dim: int, out: torch.Tensor | None = None, gate: torch.Tensor | None = None,
+                    positions: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal GQA attention over the paged cache. q, out: [T, n_q * D]. `gate` [T, n_q]: head h of a row is multiplied by
+    sigmoid(gate[row, h]). f32 tensors (any head sizes; key and value sizes may differ) need `meta.seq` and `positions`."""
     if not q.is_cuda:
         T = q.shape[0]
         o = reference.paged_attention(q.reshape(T, -1, head_dim), k_cache, v_cache, meta.cu_q, meta.ctx_lens,
                                       meta.block_tables, scale)
+        if gate is not None:
+            o = o * torch.sigmoid(gate.float()).unsqueeze(-1)
         return o.reshape(T, -1).to(q.dtype)
     C = _ext.require()
     st = _state.get(q.device)
+    if q.dtype == torch.float32:
+        out = torch.empty(q.shape[0], q.shape[1] // head_dim * v_cache.shape[3], dtype=q.dtype, device=q.device)
+        C.attn_f32(q, k_cache, v_cache, out, meta.seq.row_seq, positions, meta.block_tables, scale, gate, st.status)
+        _count()
+        return out
     if out is None:
         out = torch.empty(q.shape[0], q.shape[1], dtype=q.dtype, device=q.device)
     sa = meta.static
     if sa is not None:
         # captured step: fixed grids, everything that varies is read from device memory
         if sa.d_rows > 0:
-            C.attn_decode(q[:sa.d_rows], k_cache, v_cache, out[:sa.d_rows], sa.d_ctx, sa.d_bt, st.attn_ws, head_dim, sa.d_splits,
-                          scale, st.status, st.attn_counters)
-            _count(_decode_launches(sa.d_splits, k_cache.shape[2]))
+            _decode_attention(q[:sa.d_rows], k_cache, v_cache, out[:sa.d_rows], sa.d_ctx, sa.d_bt, head_dim, scale, sa.max_ctx,
+                              gate[:sa.d_rows] if gate is not None else None)
         if sa.max_items > 0:
             C.attn_prefill_tc(q, k_cache, v_cache, out, sa.p_cu, sa.p_ctx, sa.p_bt, sa.max_q_len, scale, 0, st.status,
-                              sa.work, sa.n_work, sa.max_items)
+                              sa.work, sa.n_work, sa.max_items, gate)
             _count()
         return out
     nd, ns = meta.num_decode, meta.num_seqs
     if nd > 0:
-        splits = _decode_splits(nd, k_cache.shape[1], meta.max_ctx)
-        C.attn_decode(q[:nd], k_cache, v_cache, out[:nd], meta.ctx_lens[:nd], meta.block_tables[:nd], st.attn_ws, head_dim,
-                      splits, scale, st.status, st.attn_counters)
-        _count(_decode_launches(splits, k_cache.shape[2]))
+        _decode_attention(q[:nd], k_cache, v_cache, out[:nd], meta.ctx_lens[:nd], meta.block_tables[:nd], head_dim, scale, meta.max_ctx,
+                          gate[:nd] if gate is not None else None)
     if ns > nd:
         # cu_q offsets are absolute token rows, so q/out are passed whole
         if prefill_on_tensor_core(head_dim, k_cache.shape[2]):
             # tcgen05 / TMEM kernel: one KV tile = one 128-token page
             if meta.work is not None and meta.n_items > 0:
                 C.attn_prefill_tc(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:],
-                                  meta.max_q_len, scale, 0, st.status, meta.work, None, meta.n_items)
+                                  meta.max_q_len, scale, 0, st.status, meta.work, None, meta.n_items, gate)
             else:
                 C.attn_prefill_tc(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:],
-                                  meta.max_q_len, scale, 0, st.status)
+                                  meta.max_q_len, scale, 0, st.status, None, None, 0, gate)
         else:
             C.attn_prefill(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:], head_dim,
-                           meta.max_q_len, scale, st.status)
+                           meta.max_q_len, scale, st.status, gate)
         _count()
     return out
 
@@ -466,3 +511,6 @@ def sample(logits: torch.Tensor, temperature: torch.Tensor, top_k: torch.Tensor,
     C.sample(logits, ids, temperature, top_k, top_p, uniforms, seed, step)
     _count()
     return ids
+
+
+from .mixers import DeltaParams, HyperMix, SeqRows, conv_qkv, delta_rule, hyper_norm  # noqa: E402,F401

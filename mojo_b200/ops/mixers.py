@@ -1,0 +1,148 @@
+"""Sequence mixing beyond plain attention: hyper-connections (a residual of several mixed streams), short causal
+convolutions in front of attention, and the gated delta rule. CUDA tensors (bf16, or f32 for the exact mode) go to the
+sm_100a kernels, CPU tensors to `ops.reference`, as in the rest of `ops`."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from .. import _ext
+from . import _state, reference
+
+
+class SeqRows:
+    """Where a step's sequences lie in its flat token rows, and which recurrent-state banks they use.
+
+      row_seq    int32 [T]     sequence of each row (-1: padding)
+      seq_rows   int32 [S, 2]  first row and one past the last row (equal: unused entry)
+      seq_state  int32 [S, 2]  bank to read (-1: no history), bank to write (-1: unused entry); bank = 2 * slot + parity
+    The first `n_decode` entries have one row each; entries [first, first + n_prefill) have any number of rows."""
+
+    __slots__ = ("row_seq", "seq_rows", "seq_state", "n_decode", "first", "n_prefill")
+
+    def __init__(self, row_seq, seq_rows, seq_state, n_decode, first, n_prefill):
+        self.row_seq, self.seq_rows, self.seq_state = row_seq, seq_rows, seq_state
+        self.n_decode, self.first, self.n_prefill = int(n_decode), int(first), int(n_prefill)
+
+
+@dataclass
+class HyperMix:
+    """Mixing coefficients of one sublayer, f32: what it reads from the streams, what it adds to them, stream to stream."""
+    w_in: torch.Tensor
+    w_out: torch.Tensor
+    mix: torch.Tensor
+
+
+def hyper_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, dtype: torch.dtype, read: HyperMix | None, done: HyperMix | None = None,
+               y: torch.Tensor | None = None, ids: torch.Tensor | None = None, embed: torch.Tensor | None = None, embed_scale: float = 1.0,
+               rows: torch.Tensor | None = None, store: bool = True, mean_width: int | None = None) -> torch.Tensor:
+    """Everything between two sublayers in one launch: fold the finished sublayer's output `y` (coefficients `done`) into
+    the streams x [T, streams, width] (f32, in place), read the next sublayer's input (`read`; None: the plain sum) and
+    RMS-normalise it with `weight` (f32). `ids`: x starts from the embedding instead. `rows`: only these rows, x untouched."""
+    from . import _count
+
+    T, S, W = x.shape
+    if not x.is_cuda:
+        if ids is not None:
+            x.copy_((embed.float()[ids.long()] * embed_scale).unsqueeze(1).expand(T, S, W))
+        pick = slice(None) if rows is None else rows.long()
+        h, new = reference.hyper_norm(x[pick], weight, eps, read.w_in if read else None, y[pick] if y is not None else None,
+                                      done.mix if done else None, done.w_out if done else None, mean_width)
+        if store:
+            x.copy_(new)
+        return h.to(dtype)
+    h = torch.empty(T if rows is None else rows.numel(), W, dtype=dtype, device=x.device)
+    _ext.require().hyper_norm(x, y, done.mix if done else None, done.w_out if done else None, read.w_in if read else None, weight, h, ids, embed,
+                              embed_scale, rows, store, eps, mean_width or W, _state.get(x.device).status)
+    _count()
+    return h
+
+
+def conv_qkv(proj: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor | None, cos_sin: torch.Tensor, positions: torch.Tensor, seq: SeqRows,
+             slots: torch.Tensor | None, k_cache: torch.Tensor | None, v_cache: torch.Tensor | None, heads: int, kv_heads: int, dim: int, vdim: int,
+             pad_dim: int, eps: float) -> torch.Tensor:
+    """Short convolution over the q | k | v channels of `proj`, rotary embedding and RMS norm of every q and k head, k and v
+    into the paged cache. kv_heads == 0: queries only. Returns q [T, heads * pad_dim] (zeros past `dim`)."""
+    from . import _count
+
+    T = proj.shape[0]
+    if not proj.is_cuda:
+        u = reference.short_conv(proj, conv_w, conv_state, seq.seq_rows, seq.seq_state)
+
+        def head_norm(z):
+            z = reference.apply_rope(z, positions, cos_sin) if cos_sin.shape[1] else z
+            return z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps)
+
+        q = head_norm(u[:, :heads * dim].reshape(T, heads, dim))
+        if kv_heads:
+            kv = (heads + kv_heads) * dim
+            k, v = head_norm(u[:, heads * dim:kv].reshape(T, kv_heads, dim)), u[:, kv:].reshape(T, kv_heads, vdim)
+            reference.write_kv(k_cache, v_cache, k, v, slots)
+        return q.reshape(T, heads * dim).to(proj.dtype)
+    q = torch.empty(T, heads * pad_dim, dtype=proj.dtype, device=proj.device)
+    banks = conv_state.shape[0] if conv_state is not None else 1 << 30
+    _ext.require().conv_qkv(proj, conv_w, conv_state, cos_sin, positions, seq.row_seq, seq.seq_rows, seq.seq_state, banks, q, slots, k_cache,
+                            v_cache, heads, kv_heads, dim, vdim, eps, _state.get(proj.device).status)
+    _count()
+    return q
+
+
+@dataclass
+class DeltaParams:
+    """f32 parameters of a gated delta-rule layer: convolution taps [taps, channels], -exp(A_log) [heads], dt_bias
+    [heads * dim], output norm [vdim]."""
+    conv_w: torch.Tensor
+    neg_rate: torch.Tensor
+    dt_bias: torch.Tensor
+    norm_w: torch.Tensor
+
+
+def delta_rule(proj: torch.Tensor, dg: torch.Tensor, p: DeltaParams, conv_state: torch.Tensor | None, state: torch.Tensor, seq: SeqRows, b_off: int,
+               heads: int, kv_heads: int, dim: int, vdim: int, out_cols: int, eps: float) -> torch.Tensor:
+    """Gated delta rule over a step's sequences, with everything around it: short convolution + silu and unit norms on
+    q | k | v of `proj`, step sizes from the logits at column `b_off`, decays and output gates from `dg`, output norm and
+    gate. `state` f32 [slots, heads, dim, vdim] and `conv_state` are updated in place. Returns [T, out_cols]."""
+    from . import _count
+
+    T = proj.shape[0]
+    if not proj.is_cuda:
+        u = reference.silu(reference.short_conv(proj, p.conv_w, conv_state, seq.seq_rows, seq.seq_state))
+        ck, per = kv_heads * dim, heads // kv_heads
+
+        def unit(z):
+            z = z.reshape(T, kv_heads, dim)
+            return (z * torch.rsqrt(z.pow(2).sum(-1, keepdim=True) + 1e-6)).repeat_interleave(per, dim=1)
+
+        q, k, v = unit(u[:, :ck]) * dim ** -0.5, unit(u[:, ck:2 * ck]), u[:, 2 * ck:].reshape(T, heads, vdim)
+        z = torch.nn.functional.softplus(dg[:, :heads * dim].float() + p.dt_bias).reshape(T, heads, dim)
+        g = torch.exp(p.neg_rate[None, :, None] * z)
+        beta = torch.sigmoid(proj[:, b_off:b_off + heads].float())
+        out = torch.zeros(T, out_cols, dtype=proj.dtype)
+        for (b, e), (rd, wr) in zip(seq.seq_rows.tolist(), seq.seq_state.tolist()):
+            if wr < 0 or e <= b:
+                continue
+            S = state[wr // 2]
+            if rd < 0:
+                S.zero_()
+            o = reference.delta_rule(q[b:e], k[b:e], v[b:e], g[b:e], beta[b:e], S)
+            o = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * p.norm_w
+            o = o * torch.sigmoid(dg[b:e, heads * dim:heads * (dim + vdim)].float()).reshape(e - b, heads, vdim)
+            out[b:e, :heads * vdim] = o.reshape(e - b, -1).to(out.dtype)
+        return out
+    C = _ext.require()
+    st = _state.get(proj.device)
+    make = torch.empty if out_cols == heads * vdim else torch.zeros
+    out = make(T, out_cols, dtype=proj.dtype, device=proj.device)
+
+    def run(first, n, raw):
+        C.delta_rule(proj, dg, p.conv_w, conv_state, p.neg_rate, p.dt_bias, p.norm_w, state, seq.row_seq, seq.seq_rows, seq.seq_state, out, raw,
+                     b_off, heads, kv_heads, dim, vdim, eps, first, n, st.status)
+
+    if seq.n_decode > 0:
+        run(-1, seq.n_decode, None)
+        _count()
+    if seq.n_prefill > 0:
+        run(seq.first, seq.n_prefill, torch.empty(T, heads * vdim, dtype=torch.float32, device=proj.device))
+        _count(2)
+    return out

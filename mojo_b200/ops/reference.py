@@ -121,10 +121,10 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
     Sequence b owns query rows cu_q[b]:cu_q[b+1]; these are the last q_len positions of a context of ctx_lens[b]
     tokens whose keys/values are all in the cache already.
     """
-    T, n_q, D = q.shape
+    T, n_q, _ = q.shape
     n_kv = k_cache.shape[1]
     group = n_q // n_kv
-    out = torch.zeros(T, n_q, D, dtype=torch.float32, device=q.device)
+    out = torch.zeros(T, n_q, v_cache.shape[3], dtype=torch.float32, device=q.device)
     for b in range(ctx_lens.numel()):
         s, e = int(cu_q[b]), int(cu_q[b + 1])
         ql, ctx = e - s, int(ctx_lens[b])
@@ -275,6 +275,51 @@ def sample(logits: torch.Tensor, temperature: float, top_k: int, top_p: float, u
     target = u * float(cdf[-1])
     idx = int(torch.searchsorted(cdf, torch.tensor(target, dtype=torch.float64), right=True))
     return min(idx, x.numel() - 1)
+
+
+# ------------------------------------------------------------------------------------------------------
+# hyper-connections, short convolutions, gated delta rule
+# ------------------------------------------------------------------------------------------------------
+
+
+def hyper_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, w_in=None, y=None, mix=None, w_out=None, mean_width: int | None = None):
+    """x [rows, streams, width] f32. Returns (normed sublayer input [rows, width], new streams)."""
+    if y is not None:
+        x = torch.einsum("st,nsw->ntw", mix, x) + w_out[None, :, None] * y.float()[:, None]
+    u = x.sum(1) if w_in is None else torch.einsum("s,nsw->nw", w_in, x)
+    ms = u.pow(2).sum(-1, keepdim=True) / (mean_width or u.shape[-1])
+    return u * torch.rsqrt(ms + eps) * weight, x
+
+
+def short_conv(u: torch.Tensor, w: torch.Tensor, conv_state, seq_rows, seq_state) -> torch.Tensor:
+    """Causal convolution over time on the first `channels` columns of u [T, >= channels]; w [taps, channels]. Reads and
+    writes the sequences' state banks [banks, taps - 1, channels]. Rows of unused sequences stay zero."""
+    taps, channels = w.shape
+    y = torch.zeros(u.shape[0], channels, dtype=torch.float32)
+    for (b, e), (rd, wr) in zip(seq_rows.tolist(), seq_state.tolist()):
+        if wr < 0 or e <= b:
+            continue
+        rows = u[b:e, :channels].float()
+        if taps == 1:
+            y[b:e] = rows * w[0]
+            continue
+        past = conv_state[rd].float() if rd >= 0 else torch.zeros(taps - 1, channels)
+        full = torch.cat([past, rows])
+        for j in range(taps):
+            y[b:e] += w[j] * full[j:j + e - b]
+        conv_state[wr] = full[full.shape[0] - (taps - 1):].to(conv_state.dtype)
+    return y
+
+
+def delta_rule(q, k, v, g, beta, S):
+    """One sequence: q, k, g [T, H, d], v [T, H, e], beta [T, H], S [H, d, e] (updated in place). Returns o [T, H, e]."""
+    o = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        S.mul_(g[t].unsqueeze(-1))
+        u = beta[t].unsqueeze(-1) * (v[t] - torch.einsum("hde,hd->he", S, k[t]))
+        S.add_(k[t].unsqueeze(-1) * u.unsqueeze(1))
+        o[t] = torch.einsum("hde,hd->he", S, q[t])
+    return o
 
 
 # ------------------------------------------------------------------------------------------------------

@@ -11,7 +11,7 @@ from dataclasses import asdict, dataclass, fields
 class PipelineConfig:
     model: str = "tiny-llama"             # preset name, HF checkpoint directory, or .gguf file
     random_init: bool = False             # random N(0, 0.02) weights of the named architecture
-    dtype: str = "bfloat16"               # compute dtype on CUDA; CPU always runs fp32
+    dtype: str = "bfloat16"               # compute dtype on CUDA ("float32": true 32-bit, where the model has it); CPU always runs fp32
     quantization: str | None = None       # None | "fp8_block" | "gguf"
     device: str | None = None             # default: cuda if available
     tensor_parallel: int = 1
@@ -19,6 +19,7 @@ class PipelineConfig:
     data_parallel: int = 1                # independent replicas, one per rank, behind one endpoint (`cli serve`)
     page_size: int = 128
     max_num_seqs: int = 256
+    state_slots: int | None = None        # models with recurrent state: live sequences that can hold one (None: max_num_seqs)
     max_num_batched_tokens: int = 4096
     max_model_len: int = 4096
     gpu_memory_utilization: float = 0.9
@@ -45,7 +46,7 @@ class PipelineConfig:
                 ap.add_argument(name, action="store_true" if not f.default else "store_false", dest=f.name, default=f.default)
             elif f.name in ("tensor_parallel", "expert_parallel", "data_parallel", "page_size", "max_num_seqs", "max_num_batched_tokens", "max_model_len", "seed"):
                 ap.add_argument(name, type=int, default=f.default, dest=f.name)
-            elif f.name in ("num_pages", "eos_token_id"):
+            elif f.name in ("num_pages", "eos_token_id", "state_slots"):
                 ap.add_argument(name, type=int, default=None, dest=f.name)
             elif f.name == "gpu_memory_utilization":
                 ap.add_argument(name, type=float, default=f.default, dest=f.name)

@@ -92,6 +92,8 @@ class LLM:
             device = str(self.dist_info.device)
         if degree > 1 and comm is None and ep is None:
             comm, ep, device = self._join_ranks(mcfg, device, degree)
+        if dtype == torch.float32 and device.startswith("cuda") and mcfg.architecture != "rekudra":
+            raise ValueError(f"{mcfg.architecture} runs in bfloat16 on CUDA")
         model = build_model(mcfg, device, dtype, comm=comm, ep=ep)
         if config.random_init or (not is_gguf and not (Path(src) / "config.json").exists()):
             model.init_random(config.seed)
@@ -108,7 +110,7 @@ class LLM:
 
             load_safetensors_into(model, src)
         ecfg = EngineConfig(model=mcfg, device=device, dtype=dtype, page_size=config.page_size, num_pages=config.num_pages,
-                            gpu_memory_utilization=config.gpu_memory_utilization, max_num_seqs=config.max_num_seqs,
+                            gpu_memory_utilization=config.gpu_memory_utilization, max_num_seqs=config.max_num_seqs, state_slots=config.state_slots,
                             max_num_batched_tokens=config.max_num_batched_tokens, max_model_len=config.max_model_len,
                             enable_prefix_cache=config.enable_prefix_cache, enable_chunked_prefill=config.enable_chunked_prefill,
                             eos_token_id=config.eos_token_id, seed=config.seed, use_cuda_graphs=config.use_cuda_graphs,
