@@ -150,7 +150,8 @@ def _load_rekudra(model, rd: _Reader) -> None:
     model.layers.clear()
     model.load_tensor("embed", rd.get("embed"))
     for i, spec in enumerate(model.cfg.layers):
-        names = model.tensor_shapes(spec, model.cfg.hidden_size, model.cfg.residual_streams)
+        names = dict.fromkeys(model.tensor_shapes(spec, model.cfg.hidden_size, model.cfg.residual_streams))
+        names.update(dict.fromkeys(n for n in model.conv_names(spec) if rd.has(f"l{i}.{n}")))
         model.load_layer(i, {n: rd.get(f"l{i}.{n}") for n in names})
     model.load_tensor("final.norm", rd.get("final.norm"))
     model.load_tensor("head", rd.get("head"))

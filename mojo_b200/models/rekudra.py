@@ -142,8 +142,8 @@ class RekudraModel:
 
     @staticmethod
     def tensor_shapes(spec: LayerSpec, width: int, streams: int) -> dict[str, tuple]:
-        """Checkpoint tensors of one layer and their shapes; -1 is a size only the checkpoint tells. Convolution taps of 1
-        stand for layers without a convolution, which have no such tensor."""
+        """Checkpoint tensors of one layer and their shapes; -1 is a size only the checkpoint tells. With one tap the
+        convolution tensors are a factor per channel, and may be missing (`conv_names`)."""
         H, G, d, e, n = spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.conv_taps
         out = {"norm1": (width,)}
         if spec.mixer == "attention":
@@ -154,7 +154,7 @@ class RekudraModel:
             mix = {"q": (G * d, width), "k": (G * d, width), "v": (H * e, width), "b": (H, width), "A_log": (H,), "norm": (e,), "a1": (-1, width),
                    "a2": (H * d, -1), "dt_bias": (H * d,), "g1": (-1, width), "g2": (H * e, -1)}
         if n > 1:
-            mix.update({f"{x}.conv": (mix[x][0], n) for x in ("q", "k", "v") if x in mix})
+            mix.update({c[4:]: (mix[c[4:5]][0], n) for c in RekudraModel.conv_names(spec)})
         mix["o"] = (width, H * e)
         out.update({f"mix.{k}": v for k, v in mix.items()})
         subs = (1, 2) if spec.ffn else (1,)
@@ -163,6 +163,10 @@ class RekudraModel:
         if spec.ffn:
             out.update({"norm2": (width,), "mlp.gate": (spec.ffn, width), "mlp.up": (spec.ffn, width), "mlp.down": (width, spec.ffn)})
         return out
+
+    @staticmethod
+    def conv_names(spec: LayerSpec) -> list[str]:
+        return [f"mix.{x}.conv" for x in ("q", "k", "v") if x == "q" or spec.kv_from is None]
 
     def load_layer(self, idx: int, w: dict[str, torch.Tensor]) -> None:
         """`w`: checkpoint tensors of the layer, named without the layer prefix."""
@@ -180,10 +184,7 @@ class RekudraModel:
 
         qkv = [n for n in ("q", "k", "v") if f"mix.{n}" in w]
         channels = sum(w[f"mix.{n}"].shape[0] for n in qkv)
-        if spec.conv_taps > 1:
-            conv = torch.cat([w[f"mix.{n}.conv"] for n in qkv]).t()
-        else:
-            conv = torch.ones(1, channels)
+        conv = torch.cat([w[f"mix.{n}.conv"] if f"mix.{n}.conv" in w else torch.ones(w[f"mix.{n}"].shape[0], 1) for n in qkv]).t()
         H, d, e = spec.heads, spec.dim, spec.vdim
         parts = [wide(f"mix.{n}") for n in qkv]
         kw: dict = {}
