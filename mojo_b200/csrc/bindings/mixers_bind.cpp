@@ -132,11 +132,10 @@ void conv_qkv(const at::Tensor& proj, const at::Tensor& conv_w, const OptTensor&
   check(b2_conv_qkv(&a, &s, proj.scalar_type() == at::kFloat ? 1 : 0, status_ptr(status), cur_stream()), "conv_qkv");
 }
 
-// first < 0: decode form over sequences [0, n); otherwise the scan over sequences [first, first + n).
 void delta_rule(const at::Tensor& proj, const at::Tensor& dg, const at::Tensor& conv_w, const OptTensor& conv_state, const at::Tensor& neg_rate,
                 const at::Tensor& dt_bias, const at::Tensor& norm_w, at::Tensor& state, const at::Tensor& row_seq, const at::Tensor& seq_rows,
-                const at::Tensor& seq_state, at::Tensor& out, const OptTensor& o_raw, int64_t b_off, int64_t heads, int64_t kv_heads, int64_t dim,
-                int64_t vdim, double eps, int64_t first, int64_t n, const OptTensor& status) {
+                const at::Tensor& seq_state, at::Tensor& out, const at::Tensor& scratch, const OptTensor& o_raw, int64_t b_off, int64_t heads,
+                int64_t kv_heads, int64_t dim, int64_t vdim, double eps, int64_t n_decode, int64_t first, int64_t n_prefill, const OptTensor& status) {
   need(is_act(proj) && proj.dim() == 2 && proj.stride(1) == 1 && dg.scalar_type() == proj.scalar_type() && dg.dim() == 2 && dg.stride(1) == 1 &&
            out.scalar_type() == proj.scalar_type() && out.dim() == 2 && out.stride(1) == 1, "delta_rule: proj, dg, out of one type with unit inner strides");
   const int64_t T = proj.size(0), taps = conv_w.size(0), channels = 2 * kv_heads * dim + heads * vdim;
@@ -172,13 +171,14 @@ void delta_rule(const at::Tensor& proj, const at::Tensor& dg, const at::Tensor& 
   a.eps = static_cast<float>(eps);
   const int f32 = proj.scalar_type() == at::kFloat ? 1 : 0;
   c10::cuda::CUDAGuard g(proj.device());
-  if (first < 0) {
-    check(b2_delta_decode(&a, &s, static_cast<int>(n), f32, status_ptr(status), cur_stream()), "delta_decode");
-  } else {
-    need(o_raw.has_value() && is_f32(*o_raw, T * heads * vdim), "delta_rule: the scan needs an f32 scratch [T, heads * vdim]");
+  need(is_f32(scratch, b2_delta_scratch_floats(a.heads, a.dim, a.vdim, s.rows)), "delta_rule: f32 scratch of delta_scratch_floats elements");
+  a.scratch = scratch.data_ptr<float>();
+  if (o_raw.has_value()) {
+    need(is_f32(*o_raw, T * heads * vdim), "delta_rule: o_raw f32 [T, heads * vdim]");
     a.o_raw = o_raw->data_ptr<float>();
-    check(b2_delta_scan(&a, &s, static_cast<int>(first), static_cast<int>(n), f32, status_ptr(status), cur_stream()), "delta_scan");
   }
+  check(b2_delta_rule(&a, &s, static_cast<int>(n_decode), static_cast<int>(first), static_cast<int>(n_prefill), f32, status_ptr(status), cur_stream()),
+        "delta_rule");
 }
 
 void gemm_f32(const at::Tensor& x, const at::Tensor& w, at::Tensor& y) {
@@ -215,6 +215,9 @@ void bind_mixers(py::module_& m) {
   m.def("hyper_norm", &hyper_norm);
   m.def("conv_qkv", &conv_qkv);
   m.def("delta_rule", &delta_rule);
+  m.def("delta_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows) {
+    return b2_delta_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows));
+  });
   m.def("gemm_f32", &gemm_f32);
   m.def("attn_f32", &attn_f32);
   m.def("swiglu_f32", [](const at::Tensor& gu, at::Tensor& out) {

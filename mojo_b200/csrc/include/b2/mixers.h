@@ -82,16 +82,19 @@ struct B2DeltaArgs {
   const float* dt_bias;       // [heads * dim]
   const float* norm_w;        // [vdim]
   float* state;
-  float* o_raw;               // [rows, heads * vdim] scratch of the scan
+  float* scratch;             // b2_delta_scratch_floats floats: prepared rows
+  float* o_raw;               // [rows, heads * vdim], outputs of the scan before norm and gate
   void* out;                  // [rows, ld_out], heads * vdim columns
   int64_t ld_out;
   int32_t b_off, heads, kv_heads, dim, vdim, taps;
   float eps;
 };
-// Sequences [0, n) of the step, one row each: state read and written once, output finished in the same kernel.
-int b2_delta_decode(const B2DeltaArgs* a, const B2SeqRows* s, int n, int f32, b2::Status* status, cudaStream_t stream);
-// Sequences [first, first + n): any number of rows each. Two launches (scan, output norm and gate).
-int b2_delta_scan(const B2DeltaArgs* a, const B2SeqRows* s, int first, int n, int f32, b2::Status* status, cudaStream_t stream);
+int64_t b2_delta_scratch_floats(int heads, int dim, int vdim, int rows);
+// Sequences [0, n_decode) of the step have one row each (state read and written once, output finished in the same kernel);
+// sequences [first, first + n_prefill) any number of rows (scan, then output norm and gate). The rows of all sequences are
+// prepared by one launch ahead of both.
+int b2_delta_rule(const B2DeltaArgs* a, const B2SeqRows* s, int n_decode, int first, int n_prefill, int f32, b2::Status* status,
+                  cudaStream_t stream);
 
 // Y[M, N] = X[M, K] W[N, K]^T in true f32 (FMA, no reduced-precision matrix mode).
 int b2_gemm_f32(const float* x, const float* w, float* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,

@@ -72,4 +72,79 @@ struct ConvSource {
   }
 };
 
+// VEC raw elements in registers.
+template <typename T, int VEC>
+struct RawVec {
+  float v[VEC];
+  __device__ __forceinline__ void load(const T* p) { load_f32<VEC>(p, v); }
+  __device__ __forceinline__ void store(T* p) const { store_f32<VEC>(p, v); }
+  __device__ __forceinline__ void zero() {
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = 0.0f;
+  }
+  __device__ __forceinline__ float get(int i) const { return v[i]; }
+};
+template <>
+struct RawVec<__nv_bfloat16, 4> {
+  uint2 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint2*>(p); }
+  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint2*>(p) = v; }
+  __device__ __forceinline__ void zero() { v = make_uint2(0, 0); }
+  __device__ __forceinline__ float get(int i) const {
+    const uint32_t w = i < 2 ? v.x : v.y;
+    return i & 1 ? ptx::bf16_hi(w) : ptx::bf16_lo(w);
+  }
+};
+
+// The convolution of `n` (<= TT) consecutive rows of one sequence for VEC channels: the whole window is fetched at once, so
+// that its loads are in flight together, and every row is fetched once. `save` also writes the next step's bank.
+// TAPS == 0: any number of taps, row by row.
+template <typename T, int VEC, int TAPS, int TT>
+__device__ __forceinline__ void conv_rows(const ConvSource<T>& s, const ConvRow& r, int row0, int n, int chan, bool save, float (&y)[TT][VEC]) {
+  if constexpr (TAPS == 0) {
+#pragma unroll
+    for (int t = 0; t < TT; ++t) {
+      if (t < n) {
+        s.template apply<VEC>(r, row0 + t, chan, y[t]);
+        if (save) s.template save<VEC>(r, row0 + t, chan);
+      } else {
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) y[t][v] = 0.0f;
+      }
+    }
+  } else {
+    RawVec<T, VEC> u[TT + TAPS - 1];
+#pragma unroll
+    for (int i = 0; i < TT + TAPS - 1; ++i) {
+      const int src = row0 - (TAPS - 1) + i;
+      const T* p = src >= r.begin ? s.proj + src * s.ld + chan : r.rd >= 0 ? s.bank(r.rd, TAPS - 1 - (r.begin - src), chan) : nullptr;
+      if (i < n + TAPS - 1 && p != nullptr) u[i].load(p);
+      else u[i].zero();
+    }
+    float w[TAPS][VEC];
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load_f32<VEC>(s.w + static_cast<int64_t>(j) * s.channels + chan, w[j]);
+#pragma unroll
+    for (int t = 0; t < TT; ++t)
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) {
+        float a = 0.0f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) a = fmaf(w[j][v], u[t + j].get(v), a);
+        y[t][v] = a;
+      }
+    if (save) {
+#pragma unroll
+      for (int t = 0; t < TT; ++t)
+        if (t < n && r.end - (row0 + t) <= TAPS - 1) u[t + TAPS - 1].store(s.bank(r.wr, TAPS - 1 - (r.end - (row0 + t)), chan));
+      const int total = r.end - r.begin;
+      if (row0 == r.begin && total < TAPS - 1) {       // older part of the history moves over
+#pragma unroll
+        for (int i = 0; i < TAPS - 1; ++i)
+          if (i >= total) u[i].store(s.bank(r.wr, i - total, chan));
+      }
+    }
+  }
+}
+
 }  // namespace b2

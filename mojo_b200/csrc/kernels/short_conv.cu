@@ -16,10 +16,11 @@ namespace {
 constexpr int kMaxHead = 256;
 constexpr int kWarps = 8;
 
-template <typename T, int VEC, int NJ>
-__global__ void __launch_bounds__(kWarps * 32) conv_qkv_kernel(const B2ConvQkvArgs a, const B2SeqRows sq, int rows_per_warp, Status* status) {
+// A warp's rows: runs of rows of one sequence, each convolved at once (`conv_rows`), then rotated and normalised row by row.
+template <typename T, int VEC, int NJ, int TAPS, int TT>
+__global__ void __launch_bounds__(kWarps * 32) conv_qkv_kernel(const B2ConvQkvArgs a, const B2SeqRows sq, Status* status) {
   ptx::grid_dep_sync();
-  __shared__ float head_sm[kWarps][kMaxHead];
+  __shared__ __align__(16) float head_sm[kWarps][kMaxHead];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int head = blockIdx.y * kWarps + warp;
   const int n_heads = a.heads + 2 * a.kv_heads;
@@ -32,96 +33,131 @@ __global__ void __launch_bounds__(kWarps * 32) conv_qkv_kernel(const B2ConvQkvAr
   const int half = a.rot >> 1;
   const ConvSource<T> src{static_cast<const T*>(a.proj), a.ld, a.conv_w, static_cast<T*>(a.conv_state), a.taps, channels, sq.banks};
   float* hs = head_sm[warp];
-  const int row_end = min(sq.rows, static_cast<int>(blockIdx.x + 1) * rows_per_warp);
-  for (int row = blockIdx.x * rows_per_warp; row < row_end; ++row) {
-    const int seq = sq.row_seq[row];
-    T* q_dst = static_cast<T*>(a.q_out) + static_cast<int64_t>(row) * a.heads * a.pad_dim + static_cast<int64_t>(head) * a.pad_dim;
-    if (seq < 0 || !B2_ASSERT(status, seq < sq.seqs, kSiteKvIndex, seq, sq.seqs)) {
+  const int row_end = min(sq.rows, static_cast<int>(blockIdx.x + 1) * TT);
+  int run = 0;
+  for (int row0 = blockIdx.x * TT; row0 < row_end; row0 += run) {
+    run = 1;
+    const int seq = sq.row_seq[row0];
+    ConvRow cr;
+    const bool valid = seq >= 0 && B2_ASSERT(status, seq < sq.seqs, kSiteKvIndex, seq, sq.seqs) && cr.load(sq, seq, row0, sq.banks, status);
+    if (!valid) {      // padding row
       if (is_q)
-        for (int e = lane; e < pad; e += 32) { const float z[1] = {0.0f}; store_f32<1>(q_dst + e, z); }
+        for (int e = lane; e < pad; e += 32) {
+          const float z[1] = {0.0f};
+          store_f32<1>(static_cast<T*>(a.q_out) + (static_cast<int64_t>(row0) * a.heads + head) * a.pad_dim + e, z);
+        }
       continue;
     }
-    ConvRow cr;
-    if (!cr.load(sq, seq, row, sq.banks, status)) continue;
-    float val[NJ][VEC];
+    run = min(row_end, cr.end) - row0;
+    float val[NJ][TT][VEC];
 #pragma unroll
     for (int j = 0; j < NJ; ++j) {
       const int e = (lane + 32 * j) * VEC;
       if (e < dim) {
-        src.template apply<VEC>(cr, row, chan0 + e, val[j]);
-        src.template save<VEC>(cr, row, chan0 + e);
+        conv_rows<T, VEC, TAPS, TT>(src, cr, row0, run, chan0 + e, true, val[j]);
       } else {
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) val[j][v] = 0.0f;
+        for (int t = 0; t < TT; ++t)
+#pragma unroll
+          for (int v = 0; v < VEC; ++v) val[j][t][v] = 0.0f;
       }
     }
-    if (!is_v) {
-      // rotate pairs (i, i + rot / 2), then divide by the root mean square of the head
-      int pos = a.positions[row];
-      if (!B2_ASSERT(status, pos >= 0 && pos < a.max_pos, kSiteKvIndex, pos, a.max_pos)) pos = 0;
-      const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
-      __syncwarp();
+#pragma unroll
+    for (int t = 0; t < TT; ++t) {
+      if (t >= run) break;
+      const int row = row0 + t;
+      if (!is_v) {
+        // rotate pairs (i, i + rot / 2), then divide by the root mean square of the head
+        int pos = a.positions[row];
+        if (!B2_ASSERT(status, pos >= 0 && pos < a.max_pos, kSiteKvIndex, pos, a.max_pos)) pos = 0;
+        const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
+        __syncwarp();
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const int e = (lane + 32 * j) * VEC;
+          if (e < dim) store_f32<VEC>(hs + e, val[j][t]);
+        }
+        __syncwarp();
+        float ss = 0.0f;
+#pragma unroll
+        for (int j = 0; j < NJ; ++j) {
+          const int e0 = (lane + 32 * j) * VEC;
+          if (half % VEC == 0) {      // a vector lies on one side of the rotated span
+            if (e0 < a.rot) {
+              const bool lo = e0 < half;
+              float c[VEC], sn[VEC], other[VEC];
+              load_f32<VEC>(cs + (lo ? e0 : e0 - half), c);
+              load_f32<VEC>(cs + (lo ? half + e0 : e0), sn);
+              load_f32<VEC>(hs + (lo ? e0 + half : e0 - half), other);
+#pragma unroll
+              for (int v = 0; v < VEC; ++v) val[j][t][v] = val[j][t][v] * c[v] + (lo ? -other[v] : other[v]) * sn[v];
+            }
+          } else {
+#pragma unroll
+            for (int v = 0; v < VEC; ++v) {
+              const int e = e0 + v;
+              if (e < half) val[j][t][v] = val[j][t][v] * cs[e] - hs[e + half] * cs[half + e];
+              else if (e < a.rot) val[j][t][v] = val[j][t][v] * cs[e - half] + hs[e - half] * cs[e];
+            }
+          }
+#pragma unroll
+          for (int v = 0; v < VEC; ++v) ss = fmaf(val[j][t][v], val[j][t][v], ss);      // 0 past dim
+        }
+        ss = warp_sum(ss);
+        const float r = 1.0f / sqrtf(ss / static_cast<float>(dim) + a.eps);
+#pragma unroll
+        for (int j = 0; j < NJ; ++j)
+#pragma unroll
+          for (int v = 0; v < VEC; ++v) val[j][t][v] *= r;
+      }
+      T* dst;
+      int lim = pad;          // queries: zeros up to the padded size; cache rows are zero there from the start
+      if (is_q) {
+        dst = static_cast<T*>(a.q_out) + (static_cast<int64_t>(row) * a.heads + head) * a.pad_dim;
+      } else {
+        const int64_t slot = a.slots[row];
+        if (slot < 0 || !B2_ASSERT(status, slot < a.num_slots, kSiteKvIndex, slot, a.num_slots)) continue;
+        T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache);
+        dst = cache + ((slot / a.page_size * a.kv_heads + kvh) * a.page_size + slot % a.page_size) * pad;
+        lim = dim;
+      }
 #pragma unroll
       for (int j = 0; j < NJ; ++j) {
         const int e = (lane + 32 * j) * VEC;
-        if (e < dim) store_f32<VEC>(hs + e, val[j]);
+        if (e < lim) store_f32<VEC>(dst + e, val[j][t]);
       }
-      __syncwarp();
-      float ss = 0.0f;
-#pragma unroll
-      for (int j = 0; j < NJ; ++j) {
-#pragma unroll
-        for (int v = 0; v < VEC; ++v) {
-          const int e = (lane + 32 * j) * VEC + v;
-          if (e < half) val[j][v] = val[j][v] * cs[e] - hs[e + half] * cs[half + e];
-          else if (e < a.rot) val[j][v] = val[j][v] * cs[e - half] + hs[e - half] * cs[e];
-          ss = fmaf(val[j][v], val[j][v], ss);      // 0 past dim
-        }
-      }
-      ss = warp_sum(ss);
-      const float r = 1.0f / sqrtf(ss / static_cast<float>(dim) + a.eps);
-#pragma unroll
-      for (int j = 0; j < NJ; ++j)
-#pragma unroll
-        for (int v = 0; v < VEC; ++v) val[j][v] *= r;
+      if (is_q)
+        for (int e = 32 * NJ * VEC + lane; e < pad; e += 32) { const float z[1] = {0.0f}; store_f32<1>(dst + e, z); }
     }
-    T* dst = q_dst;
-    int lim = pad;          // queries: zeros up to the padded size; cache rows are zero there from the start
-    if (!is_q) {
-      const int64_t slot = a.slots[row];
-      if (slot < 0 || !B2_ASSERT(status, slot < a.num_slots, kSiteKvIndex, slot, a.num_slots)) continue;
-      T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache);
-      dst = cache + ((slot / a.page_size * a.kv_heads + kvh) * a.page_size + slot % a.page_size) * pad;
-      lim = dim;
-    }
-#pragma unroll
-    for (int j = 0; j < NJ; ++j) {
-      const int e = (lane + 32 * j) * VEC;
-      if (e < lim) store_f32<VEC>(dst + e, val[j]);
-    }
-    if (is_q)
-      for (int e = 32 * NJ * VEC + lane; e < pad; e += 32) { const float z[1] = {0.0f}; store_f32<1>(dst + e, z); }
   }
 }
 
-template <typename T, int VEC, int NJ>
+template <typename T, int VEC, int NJ, int TAPS>
 int launch_conv_qkv(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
   const int groups = (a.heads + 2 * a.kv_heads + kWarps - 1) / kWarps;
-  // consecutive rows of one warp share the convolution's history through L1, but a small step wants one warp per row
-  int rpw = 8;
-  while (rpw > 1 && (s.rows + rpw - 1) / rpw * groups < 4 * kNumSMs) rpw >>= 1;
-  launch_pdl(conv_qkv_kernel<T, VEC, NJ>, dim3((s.rows + rpw - 1) / rpw, groups), dim3(kWarps * 32), 0, stream, a, s, rpw, status);
+  // rows of one warp share the convolution's window; a small step wants one warp per row
+  constexpr int kRows = TAPS == 0 ? 2 : VEC * NJ > 4 ? 4 : 8;
+  if ((s.rows + kRows - 1) / kRows * groups < 2 * kNumSMs)
+    launch_pdl(conv_qkv_kernel<T, VEC, NJ, TAPS, 1>, dim3(s.rows, groups), dim3(kWarps * 32), 0, stream, a, s, status);
+  else
+    launch_pdl(conv_qkv_kernel<T, VEC, NJ, TAPS, kRows>, dim3((s.rows + kRows - 1) / kRows, groups), dim3(kWarps * 32), 0, stream, a, s, status);
   return last_launch_rc();
 }
 
 template <typename T>
 int dispatch_conv_qkv(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
-  const int d = a.dim > a.vdim && a.kv_heads > 0 ? a.dim : (a.kv_heads > 0 ? a.vdim : a.dim);
-  const bool even = a.dim % 2 == 0 && (a.kv_heads == 0 || a.vdim % 2 == 0) && a.ld % 2 == 0 && a.pad_dim % 2 == 0 && a.pad_vdim % 2 == 0;
-  if (!even) return launch_conv_qkv<T, 1, 8>(a, s, status, stream);
-  if (d <= 64) return launch_conv_qkv<T, 2, 1>(a, s, status, stream);
-  if (d <= 128) return launch_conv_qkv<T, 2, 2>(a, s, status, stream);
-  return launch_conv_qkv<T, 2, 4>(a, s, status, stream);
+  const bool kv = a.kv_heads > 0;
+  const int d = kv && a.vdim > a.dim ? a.vdim : a.dim;
+  const auto all = [&](int m) { return a.dim % m == 0 && (!kv || (a.vdim % m == 0 && a.pad_vdim % m == 0)) && a.ld % m == 0 && a.pad_dim % m == 0; };
+  if (a.taps == 4 && all(4)) {
+    if (d <= 128) return launch_conv_qkv<T, 4, 1, 4>(a, s, status, stream);
+    return launch_conv_qkv<T, 4, 2, 4>(a, s, status, stream);
+  }
+  if (all(2)) {
+    if (d <= 128) return launch_conv_qkv<T, 2, 2, 0>(a, s, status, stream);
+    return launch_conv_qkv<T, 2, 4, 0>(a, s, status, stream);
+  }
+  return launch_conv_qkv<T, 1, 8, 0>(a, s, status, stream);
 }
 
 }  // namespace
