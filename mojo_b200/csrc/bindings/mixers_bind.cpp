@@ -171,7 +171,7 @@ void delta_rule(const at::Tensor& proj, const at::Tensor& dg, const at::Tensor& 
   a.eps = static_cast<float>(eps);
   const int f32 = proj.scalar_type() == at::kFloat ? 1 : 0;
   c10::cuda::CUDAGuard g(proj.device());
-  need(is_f32(scratch, b2_delta_scratch_floats(a.heads, a.dim, a.vdim, s.rows)), "delta_rule: f32 scratch of delta_scratch_floats elements");
+  need(is_f32(scratch, b2_delta_scratch_floats(a.heads, a.dim, a.vdim, s.rows, s.seqs)), "delta_rule: f32 scratch of delta_scratch_floats elements");
   a.scratch = scratch.data_ptr<float>();
   if (o_raw.has_value()) {
     need(is_f32(*o_raw, T * heads * vdim), "delta_rule: o_raw f32 [T, heads * vdim]");
@@ -215,8 +215,8 @@ void bind_mixers(py::module_& m) {
   m.def("hyper_norm", &hyper_norm);
   m.def("conv_qkv", &conv_qkv);
   m.def("delta_rule", &delta_rule);
-  m.def("delta_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows) {
-    return b2_delta_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows));
+  m.def("delta_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows, int64_t seqs) {
+    return b2_delta_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows), static_cast<int>(seqs));
   });
   m.def("gemm_f32", &gemm_f32);
   m.def("attn_f32", &attn_f32);

@@ -89,7 +89,7 @@ struct B2DeltaArgs {
   int32_t b_off, heads, kv_heads, dim, vdim, taps;
   float eps;
 };
-int64_t b2_delta_scratch_floats(int heads, int dim, int vdim, int rows);
+int64_t b2_delta_scratch_floats(int heads, int dim, int vdim, int rows, int seqs);
 // Sequences [0, n_decode) of the step have one row each (state read and written once, output finished in the same kernel);
 // sequences [first, first + n_prefill) any number of rows (scan, then output norm and gate). The rows of all sequences are
 // prepared by one launch ahead of both.

@@ -7,9 +7,10 @@
 //   scan    any number of rows. CTA = (32 value columns, head, sequence): S stays in the registers of four warps, which walk
 //           over the rows two at a time while bulk copies bring the next rows into shared memory; norm and gate follow in a
 //           kernel of their own
-// S^T k and S^T q are read off the decayed state together, and the new write's share u (k . q) is added to the output, so a
-// row costs one pass over S. Two rows at a time: with A = g1 * S, the second row reads g2 * A, to which the first row's write
-// contributes u1 ((g2 k1) . k2) and u1 ((g2 k1) . q2); both rows' sums come out of one reduction.
+// Rows go in pairs, because a pair costs one reduction over the key rows instead of two. With S the state before the pair,
+//   S^T k of row 1 = S . (g1 k1)                 of row 2 = S . (g1 g2 k2) + u1 ((g2 k1) . k2)      (likewise for q)
+//   S after        = g1 g2 S + (g2 k1) u1^T + k2 u2^T
+// so the prepared vectors g1 k1, g1 q1, g1 g2 k2, g1 g2 q2, g1 g2, g2 k1, k2 and a few scalars are all a pair needs.
 #include <cstdint>
 #include "b2/elem.cuh"
 #include "b2/launch.h"
@@ -23,40 +24,55 @@ namespace {
 
 constexpr int kMaxDim = 256;
 constexpr float kUnitEps = 1e-6f;
-constexpr int kTile = 16;        // rows of one shared-memory stage of the scan
+constexpr int kTile = 8;         // pairs of one shared-memory stage of the scan
 constexpr int kStages = 3;
 constexpr int kCols = 32;        // value columns of a scan CTA
 
-__device__ __forceinline__ float silu_f32(float x) { return x / (1.0f + expf(-x)); }
+// log(1 + e^x): for small t = e^-|x| by the series of log1p, which keeps the relative precision of slow decays.
+__device__ __forceinline__ float softplus(float x) {
+  const float t = ptx::ex2(-fabsf(x) * ptx::kLog2e);
+  float s = fmaf(t, -1.0f / 8, 1.0f / 7);
+  s = fmaf(t, s, -1.0f / 6);
+  s = fmaf(t, s, 1.0f / 5);
+  s = fmaf(t, s, -1.0f / 4);
+  s = fmaf(t, s, 1.0f / 3);
+  s = fmaf(t, s, -1.0f / 2);
+  s = fmaf(t * t, s, t);
+  return fmaxf(x, 0.0f) + (t < 0.125f ? s : ptx::lg2(1.0f + t) * ptx::kLn2);
+}
+__device__ __forceinline__ float sigmoid(float x) { return ptx::rcp(1.0f + ptx::ex2(-x * ptx::kLog2e)); }
 
-// Prepared rows, f32, head-major so that a tile of rows is one contiguous block:
-//   qkg [heads][rows][3][kd]            unit q (times dim^-0.5), unit k, decay; zero / zero / one past dim
-//   v   [heads][col blocks][rows][32]
-//   sc  [heads][rows][4]                beta, k . q, and for every second row of a sequence (g k') . k and (g k') . q, where k'
-//                                       is the row before
+// Prepared pairs, f32, head-major so that a run of pairs is one contiguous block. Sequence number s with first row b starts at
+// pair (b + s) / 2, which leaves every sequence room for a last pair that is half empty.
+//   vec [heads][pairs][7][kd]            the vectors named above; zero (factors of S: one) past dim and for a missing row 2
+//   v   [heads][col blocks][pairs][2][32]
+//   sc  [heads][pairs][8]                beta1, k1 . q1, beta2, k2 . q2, (g2 k1) . k2, (g2 k1) . q2, -, -
+enum PairVec { kGK1 = 0, kGQ1 = 1, kGK2 = 2, kGQ2 = 3, kGG = 4, kW1 = 5, kW2 = 6, kVecs = 7 };
 struct Prepared {
-  float* qkg;
+  float* vec;
   float* v;
   float* sc;
-  int kd, blocks, rows;
-  __device__ __forceinline__ float* qkg_row(int h, int row) const { return qkg + (static_cast<int64_t>(h) * rows + row) * 3 * kd; }
-  __device__ __forceinline__ float* v_row(int h, int blk, int row) const { return v + ((static_cast<int64_t>(h) * blocks + blk) * rows + row) * kCols; }
-  __device__ __forceinline__ float* sc_row(int h, int row) const { return sc + (static_cast<int64_t>(h) * rows + row) * 4; }
+  int kd, blocks, pairs;
+  __device__ __forceinline__ float* vec_at(int h, int pair) const { return vec + (static_cast<int64_t>(h) * pairs + pair) * kVecs * kd; }
+  __device__ __forceinline__ float* v_at(int h, int blk, int pair) const { return v + ((static_cast<int64_t>(h) * blocks + blk) * pairs + pair) * 2 * kCols; }
+  __device__ __forceinline__ float* sc_at(int h, int pair) const { return sc + (static_cast<int64_t>(h) * pairs + pair) * 8; }
 };
+__device__ __forceinline__ int first_pair(int begin, int seq) { return (begin + seq) >> 1; }
 
 int padded_dim(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
-int64_t scratch_floats(int heads, int dim, int vdim, int rows) {
+int pair_count(int rows, int seqs) { return (rows + seqs) / 2 + 1; }
+int64_t scratch_floats(int heads, int dim, int vdim, int rows, int seqs) {
   const int64_t blocks = (vdim + kCols - 1) / kCols;
-  return static_cast<int64_t>(rows) * heads * (3 * padded_dim(dim) + blocks * kCols + 4);
+  return static_cast<int64_t>(pair_count(rows, seqs)) * heads * (kVecs * padded_dim(dim) + blocks * 2 * kCols + 8);
 }
-Prepared prepared_of(const B2DeltaArgs& a, int rows) {
+Prepared prepared_of(const B2DeltaArgs& a, const B2SeqRows& s) {
   Prepared p;
   p.kd = padded_dim(a.dim);
   p.blocks = (a.vdim + kCols - 1) / kCols;
-  p.rows = rows;
-  p.qkg = a.scratch;
-  p.v = p.qkg + static_cast<int64_t>(rows) * a.heads * 3 * p.kd;
-  p.sc = p.v + static_cast<int64_t>(rows) * a.heads * p.blocks * kCols;
+  p.pairs = pair_count(s.rows, s.seqs);
+  p.vec = a.scratch;
+  p.v = p.vec + static_cast<int64_t>(p.pairs) * a.heads * kVecs * p.kd;
+  p.sc = p.v + static_cast<int64_t>(p.pairs) * a.heads * p.blocks * 2 * kCols;
   return p;
 }
 
@@ -66,7 +82,7 @@ Prepared prepared_of(const B2DeltaArgs& a, int rows) {
 // Warp = (TT consecutive rows of one sequence, head); tiles count from each sequence's first row, so a pair of rows never
 // straddles two warps. Lane l holds channels (l + 32 j) * VEC.
 template <typename T, int VEC, int NJ, int TAPS, int TT>
-__global__ void __launch_bounds__(128) delta_prep_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared out, Status* status) {
+__global__ void __launch_bounds__(128, TAPS > 0 && NJ == 1 ? 6 : 1) delta_prep_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared out, Status* status) {
   ptx::grid_dep_sync();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y * 4 + warp;
@@ -101,7 +117,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const B2DeltaArgs a, co
   const bool save_qk = h % per == 0;
 
   float q[NJ][TT][VEC], k[NJ][TT][VEC], g[NJ][TT][VEC];
-  const float neg_rate = a.neg_rate[h];
+  const float rate = a.neg_rate[h] * ptx::kLog2e;
 #pragma unroll
   for (int j = 0; j < NJ; ++j) {
     const int c = (lane + 32 * j) * VEC;
@@ -116,9 +132,10 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const B2DeltaArgs a, co
         if (t < n) load_f32<VEC>(static_cast<const T*>(a.dg) + static_cast<int64_t>(row0 + t) * a.ld_dg + h * d + c, z);
 #pragma unroll
         for (int v = 0; v < VEC; ++v) {
-          q[j][t][v] = silu_f32(q[j][t][v]);
-          k[j][t][v] = silu_f32(k[j][t][v]);
-          g[j][t][v] = expf(neg_rate * softplus_f32(z[v] + bias[v]));
+          // a row that is not there changes nothing
+          q[j][t][v] = t < n ? ptx::silu(q[j][t][v]) : 0.0f;
+          k[j][t][v] = t < n ? ptx::silu(k[j][t][v]) : 0.0f;
+          g[j][t][v] = t < n ? ptx::ex2(rate * softplus(z[v] + bias[v])) : 1.0f;
         }
       }
     } else {
@@ -132,9 +149,9 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const B2DeltaArgs a, co
     }
   }
   const float q_scale = rsqrtf(static_cast<float>(d));
+  float kq[TT];
 #pragma unroll
   for (int t = 0; t < TT; ++t) {
-    if (t >= n) break;
     float qq = 0.0f, kk = 0.0f, qk = 0.0f;
 #pragma unroll
     for (int j = 0; j < NJ; ++j)
@@ -147,36 +164,65 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const B2DeltaArgs a, co
     qq = warp_sum(qq);
     kk = warp_sum(kk);
     qk = warp_sum(qk);
-    const float rq = q_scale / sqrtf(qq + kUnitEps), rk = 1.0f / sqrtf(kk + kUnitEps);
-    float* dst = out.qkg_row(h, row0 + t);
-    float gkk = 0.0f, gkq = 0.0f;
+    const float rq = q_scale * rsqrtf(qq + kUnitEps), rk = rsqrtf(kk + kUnitEps);
+    kq[t] = qk * rq * rk;
 #pragma unroll
-    for (int j = 0; j < NJ; ++j) {
-      const int c = (lane + 32 * j) * VEC;
+    for (int j = 0; j < NJ; ++j)
 #pragma unroll
       for (int v = 0; v < VEC; ++v) {
         q[j][t][v] *= rq;
         k[j][t][v] *= rk;
-        if (t & 1) {
-          const float gk = g[j][t][v] * k[j][t - (t & 1)][v];
-          gkk = fmaf(gk, k[j][t][v], gkk);
-          gkq = fmaf(gk, q[j][t][v], gkq);
+      }
+  }
+  const int pair0 = first_pair(cr.begin, seq) + (row0 - cr.begin) / 2;
+#pragma unroll
+  for (int t = 0; t < TT; t += 2) {
+    if (t >= n) break;
+    constexpr bool kTwo = TT > 1;
+    float* dst = out.vec_at(h, pair0 + t / 2);
+    float wk = 0.0f, wq = 0.0f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int c = (lane + 32 * j) * VEC;
+      float x[kVecs][VEC];
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) {
+        const float g1 = g[j][t][v], k1 = k[j][t][v];
+        x[kGK1][v] = g1 * k1;
+        x[kGQ1][v] = g1 * q[j][t][v];
+        if constexpr (kTwo) {
+          const float g2 = g[j][t + 1][v], k2 = k[j][t + 1][v], q2 = q[j][t + 1][v], gg = g1 * g2, w1 = g2 * k1;
+          x[kGK2][v] = gg * k2;
+          x[kGQ2][v] = gg * q2;
+          x[kGG][v] = gg;
+          x[kW1][v] = w1;
+          x[kW2][v] = k2;
+          wk = fmaf(w1, k2, wk);
+          wq = fmaf(w1, q2, wq);
+        } else {
+          x[kGK2][v] = x[kGQ2][v] = x[kW2][v] = 0.0f;
+          x[kGG][v] = g1;
+          x[kW1][v] = k1;
         }
       }
       if (c < out.kd) {
-        store_f32<VEC>(dst + c, q[j][t]);
-        store_f32<VEC>(dst + out.kd + c, k[j][t]);
-        store_f32<VEC>(dst + 2 * out.kd + c, g[j][t]);
+#pragma unroll
+        for (int i = 0; i < kVecs; ++i) store_f32<VEC>(dst + i * out.kd + c, x[i]);
       }
     }
-    if (t & 1) {
-      gkk = warp_sum(gkk);
-      gkq = warp_sum(gkq);
+    if constexpr (kTwo) {
+      wk = warp_sum(wk);
+      wq = warp_sum(wq);
     }
     if (lane == 0) {
-      float b[1];
-      load_f32<1>(static_cast<const T*>(a.proj) + static_cast<int64_t>(row0 + t) * a.ld + a.b_off + h, b);
-      *reinterpret_cast<float4*>(out.sc_row(h, row0 + t)) = make_float4(sigmoid_f32(b[0]), qk * rq * rk, gkk, gkq);
+      const bool two = kTwo && t + 1 < n;
+      float b1[1], b2v[1] = {0.0f};
+      const T* b = static_cast<const T*>(a.proj) + static_cast<int64_t>(row0 + t) * a.ld + a.b_off + h;
+      load_f32<1>(b, b1);
+      if (two) load_f32<1>(b + a.ld, b2v);
+      float* sc = out.sc_at(h, pair0 + t / 2);
+      *reinterpret_cast<float4*>(sc) = make_float4(sigmoid(b1[0]), kq[t], two ? sigmoid(b2v[0]) : 0.0f, two ? kq[t + (kTwo ? 1 : 0)] : 0.0f);
+      *reinterpret_cast<float4*>(sc + 4) = make_float4(wk, wq, 0.0f, 0.0f);
     }
   }
 #pragma unroll
@@ -187,10 +233,10 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const B2DeltaArgs a, co
     conv_rows<T, VEC, TAPS, TT>(src, cr, row0, n, 2 * ck + h * e + c, true, v);
 #pragma unroll
     for (int t = 0; t < TT; ++t) {
-      if (t >= n) break;
+      if (t >= ((n + 1) & ~1)) break;
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v[t][i] = silu_f32(v[t][i]);
-      store_f32<VEC>(out.v_row(h, c / kCols, row0 + t) + c % kCols, v[t]);
+      for (int i = 0; i < VEC; ++i) v[t][i] = t < n ? ptx::silu(v[t][i]) : 0.0f;
+      store_f32<VEC>(out.v_at(h, c / kCols, pair0 + t / 2) + (t & 1) * kCols + c % kCols, v[t]);
     }
   }
 }
@@ -198,7 +244,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(const B2DeltaArgs a, co
 template <typename T, int VEC, int NJ, int TAPS, int TT>
 int launch_prep(const B2DeltaArgs& a, const B2SeqRows& s, bool one_row_each, Status* status, cudaStream_t stream) {
   const int tiles = one_row_each ? s.seqs : (s.rows + TT - 1) / TT + s.seqs;      // every sequence may end in a partial tile
-  launch_pdl(delta_prep_kernel<T, VEC, NJ, TAPS, TT>, dim3(tiles, (a.heads + 3) / 4), dim3(128), 0, stream, a, s, prepared_of(a, s.rows), status);
+  launch_pdl(delta_prep_kernel<T, VEC, NJ, TAPS, TT>, dim3(tiles, (a.heads + 3) / 4), dim3(128), 0, stream, a, s, prepared_of(a, s), status);
   return last_launch_rc();
 }
 
@@ -216,145 +262,262 @@ int dispatch_prep(const B2DeltaArgs& a, const B2SeqRows& s, bool one_row_each, S
 // ------------------------------------------------------------------------------------------------------------
 // decode
 // ------------------------------------------------------------------------------------------------------------
-// Thread (rg, cg): columns [cg * VEC, + VEC), key rows rg + i * n_rg. RPT > 0: they stay in registers between the two uses;
-// RPT == 0 (states too large, or vdim no multiple of 4): they are read twice.
-template <typename T, int VEC, int RPT, int THREADS>
-__global__ void __launch_bounds__(THREADS, RPT == 16 ? 3 : 1) delta_decode_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared in, int n_cg, int n_rg,
-                                                               Status* status) {
-  ptx::grid_dep_sync();
-  __shared__ __align__(16) float qkg[3 * kMaxDim];
-  __shared__ __align__(16) float red_k[THREADS * VEC], red_q[THREADS * VEC];
-  __shared__ float scratch[33];
-  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
-  const int d = a.dim, e = a.vdim;
-  const int row = sq.seq_rows[2 * seq];
-  ConvRow cr;
-  if (row < 0 || row >= sq.rows || !cr.load(sq, seq, row, sq.banks, status)) return;      // uniform per CTA
-  if (!B2_ASSERT(status, cr.end == row + 1, kSiteKvIndex, row, cr.end)) return;
-  const int cg = tid % n_cg, rg = tid / n_cg;
-  const bool active = rg < n_rg;
-  float* S = a.state + (static_cast<int64_t>(cr.wr >> 1) * a.heads + h) * d * e + cg * VEC;
-  constexpr bool kHeld = RPT > 0;
-  float st[kHeld ? RPT : 1][VEC];
-  const auto fetch = [&](int r, float (&x)[VEC]) {
-#pragma unroll
-    for (int v = 0; v < VEC; ++v) x[v] = 0.0f;
-    if (active && r < d && cr.rd >= 0) load_f32<VEC>(S + static_cast<int64_t>(r) * e, x);
-  };
-  const int passes = kHeld ? RPT : (d + n_rg - 1) / n_rg;
-  if constexpr (kHeld) {
-#pragma unroll
-    for (int i = 0; i < RPT; ++i) fetch(rg + i * n_rg, st[i]);
-  }
-  const float* src = in.qkg_row(h, row);
-  for (int i = tid * 4; i < 3 * in.kd; i += THREADS * 4) *reinterpret_cast<float4*>(qkg + i) = *reinterpret_cast<const float4*>(src + i);
-  const float4 sc = *reinterpret_cast<const float4*>(in.sc_row(h, row));      // beta, k . q
-  float v_in[VEC];
-#pragma unroll
-  for (int v = 0; v < VEC; ++v) v_in[v] = 0.0f;
-  if (active) load_f32<VEC>(in.v_row(h, cg * VEC / kCols, row) + cg * VEC % kCols, v_in);
-  __syncthreads();
-  const float *q_sm = qkg, *k_sm = qkg + in.kd, *g_sm = qkg + 2 * in.kd;
-  if (active) {
-    float ks[VEC], qs[VEC];
-#pragma unroll
-    for (int v = 0; v < VEC; ++v) ks[v] = qs[v] = 0.0f;
-#pragma unroll
-    for (int i = 0; i < passes; ++i) {
-      const int r = rg + i * n_rg;
-      if (r < d) {
-        const float g = g_sm[r], kr = k_sm[r], qr = q_sm[r];
-        float (&x)[VEC] = st[kHeld ? i : 0];
-        if constexpr (!kHeld) fetch(r, x);
-#pragma unroll
-        for (int v = 0; v < VEC; ++v) {
-          x[v] *= g;
-          ks[v] = fmaf(x[v], kr, ks[v]);
-          qs[v] = fmaf(x[v], qr, qs[v]);
-        }
-      }
-    }
-    store_f32<VEC>(red_k + rg * e + cg * VEC, ks);
-    store_f32<VEC>(red_q + rg * e + cg * VEC, qs);
-  }
-  __syncthreads();
-  // every thread sums its own columns, so the write needs no second barrier
-  float u[VEC], o[VEC];
-#pragma unroll
-  for (int v = 0; v < VEC; ++v) u[v] = o[v] = 0.0f;
-  if (active) {
-    for (int i = 0; i < n_rg; ++i) {
-      float x[VEC];
-      load_f32<VEC>(red_k + i * e + cg * VEC, x);
-#pragma unroll
-      for (int v = 0; v < VEC; ++v) u[v] += x[v];
-    }
-#pragma unroll
-    for (int v = 0; v < VEC; ++v) u[v] = sc.x * (v_in[v] - u[v]);
-#pragma unroll
-    for (int i = 0; i < passes; ++i) {
-      const int r = rg + i * n_rg;
-      if (r < d) {
-        const float kr = k_sm[r];
-        float (&x)[VEC] = st[kHeld ? i : 0];
-        if constexpr (!kHeld) {
-          fetch(r, x);
-#pragma unroll
-          for (int v = 0; v < VEC; ++v) x[v] *= g_sm[r];
-        }
-#pragma unroll
-        for (int v = 0; v < VEC; ++v) x[v] = fmaf(kr, u[v], x[v]);
-        store_f32<VEC>(S + static_cast<int64_t>(r) * e, x);
-      }
-    }
-  }
+// Both forms: thread (rg, cg) handles columns [cg * VEC, + VEC) and key rows rg + i * n_rg. `finish` normalises, gates and
+// writes the outputs that the threads with rg == 0 hold.
+template <typename T, int VEC>
+__device__ __forceinline__ void decode_finish(const B2DeltaArgs& a, int row, int h, int cg, bool owner, float (&o)[VEC], float* scratch) {
   float ss = 0.0f;
-  if (rg == 0) {
-    for (int i = 0; i < n_rg; ++i) {
-      float x[VEC];
-      load_f32<VEC>(red_q + i * e + cg * VEC, x);
 #pragma unroll
-      for (int v = 0; v < VEC; ++v) o[v] += x[v];
-    }
-#pragma unroll
-    for (int v = 0; v < VEC; ++v) {
-      o[v] = fmaf(u[v], sc.y, o[v]);
-      ss = fmaf(o[v], o[v], ss);
-    }
-  }
+  for (int v = 0; v < VEC; ++v) ss = fmaf(o[v], o[v], ss);
   ss = block_sum(ss, scratch);
-  if (rg == 0) {
-    const float r_o = 1.0f / sqrtf(ss / static_cast<float>(e) + a.eps);
-    float z[VEC], w[VEC];
-    load_f32<VEC>(static_cast<const T*>(a.dg) + static_cast<int64_t>(row) * a.ld_dg + a.heads * d + h * e + cg * VEC, z);
-    load_f32<VEC>(a.norm_w + cg * VEC, w);
+  if (!owner) return;
+  const float r = rsqrtf(ss / static_cast<float>(a.vdim) + a.eps);
+  float z[VEC], w[VEC];
+  load_f32<VEC>(static_cast<const T*>(a.dg) + static_cast<int64_t>(row) * a.ld_dg + a.heads * a.dim + h * a.vdim + cg * VEC, z);
+  load_f32<VEC>(a.norm_w + cg * VEC, w);
 #pragma unroll
-    for (int v = 0; v < VEC; ++v) o[v] = o[v] * r_o * w[v] * sigmoid_f32(z[v]);
-    store_f32<VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(row) * a.ld_out + static_cast<int64_t>(h) * e + cg * VEC, o);
-  }
+  for (int v = 0; v < VEC; ++v) o[v] = o[v] * r * w[v] * sigmoid(z[v]);
+  store_f32<VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(row) * a.ld_out + static_cast<int64_t>(h) * a.vdim + cg * VEC, o);
 }
 
-template <typename T, int VEC, int RPT>
-int launch_decode(const B2DeltaArgs& a, const B2SeqRows& s, int n, int n_cg, int n_rg, Status* status, cudaStream_t stream) {
-  constexpr int kThreads = 256;
-  launch_pdl(delta_decode_kernel<T, VEC, RPT, kThreads>, dim3(a.heads, n), dim3(kThreads), 0, stream, a, s, prepared_of(a, s.rows), n_cg, n_rg, status);
-  return last_launch_rc();
+// Sequence's decode row if the entry is in use and sound, else -1.
+__device__ __forceinline__ int decode_row(const B2SeqRows& sq, int seq, ConvRow& cr, Status* status) {
+  const int row = sq.seq_rows[2 * seq];
+  if (row < 0 || row >= sq.rows || !cr.load(sq, seq, row, sq.banks, status)) return -1;
+  return B2_ASSERT(status, cr.end == row + 1, kSiteKvIndex, row, cr.end) ? row : -1;
+}
+
+// Plain form for sizes the pipelined one does not take: one CTA per (head, sequence), S read twice.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256) delta_decode_plain_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared in, int n_cg, int n_rg,
+                                                                 Status* status) {
+  ptx::grid_dep_sync();
+  __shared__ __align__(16) float red[2][256 * VEC];
+  __shared__ float scratch[33];
+  const int h = blockIdx.x, seq = blockIdx.y, d = a.dim, e = a.vdim;
+  ConvRow cr;
+  const int row = decode_row(sq, seq, cr, status);
+  if (row < 0) return;      // uniform per CTA
+  const int cg = threadIdx.x % n_cg, rg = threadIdx.x / n_cg, pair = first_pair(cr.begin, seq);
+  const bool active = rg < n_rg, fresh = cr.rd < 0;
+  float* S = a.state + (static_cast<int64_t>(cr.wr >> 1) * a.heads + h) * d * e + cg * VEC;
+  const float *vec = in.vec_at(h, pair), *sc = in.sc_at(h, pair);
+  float ks[VEC] = {}, qs[VEC] = {}, o[VEC] = {};
+  if (active) {
+    for (int r = rg; r < d && !fresh; r += n_rg) {
+      float x[VEC];
+      load_f32<VEC>(S + static_cast<int64_t>(r) * e, x);
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) {
+        ks[v] = fmaf(x[v], vec[kGK1 * in.kd + r], ks[v]);
+        qs[v] = fmaf(x[v], vec[kGQ1 * in.kd + r], qs[v]);
+      }
+    }
+    store_f32<VEC>(red[0] + rg * e + cg * VEC, ks);
+    store_f32<VEC>(red[1] + rg * e + cg * VEC, qs);
+  }
+  __syncthreads();
+  if (active) {
+    float u[VEC], sum[VEC] = {};
+    load_f32<VEC>(in.v_at(h, cg * VEC / kCols, pair) + cg * VEC % kCols, u);
+    for (int i = 0; i < n_rg; ++i) {
+      load_f32<VEC>(red[0] + i * e + cg * VEC, ks);
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) sum[v] += ks[v];
+    }
+#pragma unroll
+    for (int v = 0; v < VEC; ++v) u[v] = sc[0] * (u[v] - sum[v]);
+    for (int r = rg; r < d; r += n_rg) {
+      float x[VEC] = {};
+      if (!fresh) load_f32<VEC>(S + static_cast<int64_t>(r) * e, x);
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) x[v] = fmaf(vec[kW1 * in.kd + r], u[v], x[v] * vec[kGG * in.kd + r]);
+      store_f32<VEC>(S + static_cast<int64_t>(r) * e, x);
+    }
+    if (rg == 0) {
+      for (int i = 0; i < n_rg; ++i) {
+        load_f32<VEC>(red[1] + i * e + cg * VEC, qs);
+#pragma unroll
+        for (int v = 0; v < VEC; ++v) o[v] += qs[v];
+      }
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) o[v] = fmaf(u[v], sc[1], o[v]);
+    }
+  }
+  decode_finish<T, VEC>(a, row, h, cg, rg == 0, o, scratch);
+}
+
+// Pipelined form: persistent CTAs walk over (sequence, head) items. A stage holds one item: S [d][e], then the row's seven
+// vectors, values and scalars. While one item is computed in place, the next one's copies are on their way in and the
+// previous one's state is on its way out.
+constexpr int kDecodeThreads = 512;
+struct DecodeLayout {
+  int state, vec, v, sc, stage, stages, n_cg, n_rg, bytes;      // floats; `bytes`: dynamic shared memory
+};
+template <typename T>
+__global__ void __launch_bounds__(kDecodeThreads, 2) delta_decode_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared in, const DecodeLayout L,
+                                                                        int n_seqs, Status* status) {
+  ptx::grid_dep_sync();
+  extern __shared__ __align__(128) float dec_sm[];
+  __shared__ float scratch[33];
+  const int tid = threadIdx.x, d = a.dim, e = a.vdim, H = a.heads, total = n_seqs * H;
+  float* red_k = dec_sm + L.stages * L.stage;
+  float* red_q = red_k + L.n_rg * e;
+  const uint32_t bars = ptx::smem_u32(red_q + L.n_rg * e);
+  if (tid == 0) {
+    for (int s = 0; s < L.stages; ++s) ptx::mbar_init(bars + 8 * s, 1);
+    ptx::fence_mbar_init();
+  }
+  __syncthreads();
+  const int cg = tid % L.n_cg, rg = tid / L.n_cg;
+  const bool active = rg < L.n_rg;
+  struct Item { int index, row, seq, h; ConvRow cr; };
+  const auto find = [&](int i) {      // the first usable item at or after i of this CTA; the same in every thread
+    Item it{};
+    for (; i < total; i += gridDim.x) {
+      it.seq = i / H;
+      it.h = i % H;
+      it.row = decode_row(sq, it.seq, it.cr, status);
+      if (it.row >= 0) break;
+    }
+    it.index = i;
+    return it;
+  };
+  const auto state_of = [&](const Item& it) { return a.state + (static_cast<int64_t>(it.cr.wr >> 1) * H + it.h) * d * e; };
+  const auto issue = [&](const Item& it, int s) {      // thread 0
+    float* st = dec_sm + s * L.stage;
+    const uint32_t bar = bars + 8 * s;
+    const int pair = first_pair(it.cr.begin, it.seq), state_bytes = it.cr.rd >= 0 ? d * e * 4 : 0;
+    ptx::mbar_arrive_expect_tx(bar, static_cast<uint32_t>(state_bytes + kVecs * in.kd * 4 + in.blocks * kCols * 4 + 32));
+    if (state_bytes) ptx::bulk_load(ptx::smem_u32(st), state_of(it), state_bytes, bar);
+    ptx::bulk_load(ptx::smem_u32(st + L.vec), in.vec_at(it.h, pair), kVecs * in.kd * 4, bar);
+    for (int b = 0; b < in.blocks; ++b) ptx::bulk_load(ptx::smem_u32(st + L.v + b * kCols), in.v_at(it.h, b, pair), kCols * 4, bar);
+    ptx::bulk_load(ptx::smem_u32(st + L.sc), in.sc_at(it.h, pair), 32, bar);
+  };
+  Item cur = find(blockIdx.x);
+  if (tid == 0 && cur.index < total) issue(cur, 0);
+  bool failed = false;
+  int k = 0;
+  for (; cur.index < total; ++k) {
+    const int s = k % L.stages;
+    const Item nxt = find(cur.index + gridDim.x);
+    if (tid == 0 && nxt.index < total) {
+      // the stage's last state must have been read out: with three stages the newest store may still be pending
+      if (L.stages >= 3) ptx::tma_store_wait_read<1>();
+      else ptx::tma_store_wait_read<0>();
+      issue(nxt, (k + 1) % L.stages);
+    }
+    if (!ptx::mbar_wait(bars + 8 * s, (k / L.stages) & 1)) {
+      status_record(status, kTimeout, kSiteAttn, cur.seq, k);
+      failed = true;
+    }
+    if (__syncthreads_or(failed)) break;
+    float* st = dec_sm + s * L.stage + cg * 4;
+    const float* vec = dec_sm + s * L.stage + L.vec;
+    const float* sc = dec_sm + s * L.stage + L.sc;
+    const bool fresh = cur.cr.rd < 0;
+    float o[4] = {};
+    if (active) {
+      float ks[4] = {}, qs[4] = {};
+      if (!fresh) {
+#pragma unroll 4
+        for (int r = rg; r < d; r += L.n_rg) {
+          float x[4];
+          load_f32<4>(st + r * e, x);
+          const float gk = vec[kGK1 * in.kd + r], gq = vec[kGQ1 * in.kd + r];
+#pragma unroll
+          for (int v = 0; v < 4; ++v) {
+            ks[v] = fmaf(x[v], gk, ks[v]);
+            qs[v] = fmaf(x[v], gq, qs[v]);
+          }
+        }
+      }
+      store_f32<4>(red_k + rg * e + cg * 4, ks);
+      store_f32<4>(red_q + rg * e + cg * 4, qs);
+    }
+    __syncthreads();
+    if (active) {
+      float u[4], sum[4] = {};
+      load_f32<4>(dec_sm + s * L.stage + L.v + cg * 4, u);
+      for (int i = 0; i < L.n_rg; ++i) {
+        float x[4];
+        load_f32<4>(red_k + i * e + cg * 4, x);
+#pragma unroll
+        for (int v = 0; v < 4; ++v) sum[v] += x[v];
+      }
+#pragma unroll
+      for (int v = 0; v < 4; ++v) u[v] = sc[0] * (u[v] - sum[v]);
+#pragma unroll 4
+      for (int r = rg; r < d; r += L.n_rg) {
+        float x[4] = {};
+        if (!fresh) load_f32<4>(st + r * e, x);
+        const float gg = vec[kGG * in.kd + r], w = vec[kW1 * in.kd + r];
+#pragma unroll
+        for (int v = 0; v < 4; ++v) x[v] = fmaf(w, u[v], x[v] * gg);
+        store_f32<4>(st + r * e, x);
+      }
+      if (rg == 0) {
+        for (int i = 0; i < L.n_rg; ++i) {
+          float x[4];
+          load_f32<4>(red_q + i * e + cg * 4, x);
+#pragma unroll
+          for (int v = 0; v < 4; ++v) o[v] += x[v];
+        }
+#pragma unroll
+        for (int v = 0; v < 4; ++v) o[v] = fmaf(u[v], sc[1], o[v]);
+      }
+    }
+    ptx::fence_proxy_async_smem();      // the new state, written by ordinary stores, is about to be copied out
+    __syncthreads();
+    if (tid == 0) {
+      ptx::bulk_store(state_of(cur), ptx::smem_u32(dec_sm + s * L.stage), d * e * 4);
+      ptx::tma_store_commit();
+    }
+    decode_finish<T, 4>(a, cur.row, cur.h, cg, rg == 0, o, scratch);
+    cur = nxt;
+  }
+  if (tid == 0) {
+    ptx::tma_store_wait<0>();
+    if (failed)      // let copies in flight land before the CTA's shared memory is released
+      for (int s = 0; s < L.stages; ++s) ptx::mbar_wait(bars + 8 * s, 0, 20000000ull) || ptx::mbar_wait(bars + 8 * s, 1, 20000000ull);
+  }
 }
 
 template <typename T>
 int dispatch_decode(const B2DeltaArgs& a, const B2SeqRows& s, int n, Status* status, cudaStream_t stream) {
   const bool v4 = a.vdim % 4 == 0 && a.ld_dg % 4 == 0 && a.ld_out % 4 == 0 && (a.heads * a.dim) % 4 == 0;
+  const Prepared in = prepared_of(a, s);
+  DecodeLayout L{};
+  if (v4) {
+    L.state = a.dim * a.vdim;
+    L.vec = L.state;
+    L.v = L.vec + kVecs * in.kd;
+    L.sc = L.v + in.blocks * kCols;
+    L.stage = (L.sc + 8 + 31) / 32 * 32;
+    L.n_cg = a.vdim / 4;
+    L.n_rg = kDecodeThreads / L.n_cg;
+    if (L.n_rg > a.dim) L.n_rg = a.dim;
+    for (L.stages = 3; L.stages >= 2; --L.stages) {
+      L.bytes = (L.stages * L.stage + 2 * L.n_rg * a.vdim) * 4 + L.stages * 8;
+      if (L.bytes <= kMaxSmemPerCta - 1024) break;
+    }
+  }
+  if (L.stages >= 2) {
+    static DeviceOnce attr_once;
+    if (const int rc = attr_once.max_smem(delta_decode_kernel<T>, kMaxSmemPerCta - 1024)) return rc;
+    int per_sm = kMaxSmemPerCta / (L.bytes + 1024);
+    if (per_sm > 2) per_sm = 2;
+    const int64_t items = static_cast<int64_t>(n) * a.heads;
+    const int grid = static_cast<int>(items < static_cast<int64_t>(per_sm) * kNumSMs ? items : per_sm * kNumSMs);
+    launch_pdl(delta_decode_kernel<T>, dim3(grid), dim3(kDecodeThreads), L.bytes, stream, a, s, in, L, n, status);
+    return last_launch_rc();
+  }
   const int n_cg = v4 ? a.vdim / 4 : a.vdim;
   int n_rg = 256 / n_cg;
   if (n_rg > a.dim) n_rg = a.dim;
-  if (!v4) return launch_decode<T, 1, 0>(a, s, n, n_cg, n_rg, status, stream);
-  const int rpt = (a.dim + n_rg - 1) / n_rg;
-  if (rpt <= 2) return launch_decode<T, 4, 2>(a, s, n, n_cg, n_rg, status, stream);
-  if (rpt <= 4) return launch_decode<T, 4, 4>(a, s, n, n_cg, n_rg, status, stream);
-  if (rpt <= 8) return launch_decode<T, 4, 8>(a, s, n, n_cg, n_rg, status, stream);
-  if (rpt <= 16) return launch_decode<T, 4, 16>(a, s, n, n_cg, n_rg, status, stream);
-  if (rpt <= 32) return launch_decode<T, 4, 32>(a, s, n, n_cg, n_rg, status, stream);
-  return launch_decode<T, 4, 0>(a, s, n, n_cg, n_rg, status, stream);
+  if (v4) launch_pdl(delta_decode_plain_kernel<T, 4>, dim3(a.heads, n), dim3(256), 0, stream, a, s, in, n_cg, n_rg, status);
+  else launch_pdl(delta_decode_plain_kernel<T, 1>, dim3(a.heads, n), dim3(256), 0, stream, a, s, in, n_cg, n_rg, status);
+  return last_launch_rc();
 }
 
 // ------------------------------------------------------------------------------------------------------------
@@ -386,81 +549,69 @@ __device__ __forceinline__ float half_sum(uint64_t v) {
   return f.x + f.y;
 }
 
-// P pairs of key rows per lane (kd = 32 P). One shared-memory stage: qkg [16][3][kd], v [16][32], sc [16][4].
-template <int P>
+// A lane holds two value columns and Q quads of key rows: quad i of row group rg is rows 32 i + 4 rg + 0..3 (kd = 32 Q).
+template <int Q>
 struct ScanLayout {
-  static constexpr int kD = 32 * P;
-  static constexpr int kQkg = kTile * 3 * kD, kV = kTile * kCols, kSc = kTile * 4;
-  static constexpr int kStage = kQkg + kV + kSc;                 // floats
-  static constexpr int kNeutral = 3 * kD + kCols + 4;            // one row that changes nothing, behind the stages
-  static constexpr int kBytes = (kStages * kStage + kNeutral) * 4 + kStages * 8;
+  static constexpr int kD = 32 * Q;
+  static constexpr int kVec = kVecs * kD, kV = 2 * kCols, kSc = 8;       // floats per pair
+  static constexpr int kOffV = kTile * kVec, kOffSc = kOffV + kTile * kV;
+  static constexpr int kStage = kOffSc + kTile * kSc;
+  static constexpr int kBytes = kStages * kStage * 4 + kStages * 8;
 };
-
-// The pairs of key rows of lane group rg: pair p of P covers rows pair_row(p), pair_row(p) + 1.
-template <int P>
-__device__ __forceinline__ int pair_row(int p, int rg) {
-  if constexpr (P == 1) return 2 * rg;
-  else return (p >> 1) * 64 + rg * 4 + (p & 1) * 2;
-}
-template <int P>
-__device__ __forceinline__ void load_pairs(const float* x, int rg, uint64_t (&v)[P]) {
-  if constexpr (P == 1) {
-    v[0] = *reinterpret_cast<const uint64_t*>(x + 2 * rg);
-  } else {
+template <int Q>
+__device__ __forceinline__ void load_quads(const float* x, int rg, uint64_t (&v)[2 * Q]) {
 #pragma unroll
-    for (int i = 0; i < P / 2; ++i) {
-      const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(x + i * 64 + rg * 4);
-      v[2 * i] = t.x;
-      v[2 * i + 1] = t.y;
-    }
+  for (int i = 0; i < Q; ++i) {
+    const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(x + 32 * i + 4 * rg);
+    v[2 * i] = t.x;
+    v[2 * i + 1] = t.y;
   }
 }
 
-// Lane (rg = lane & 15, half = lane >> 4) of warp w: value columns col0 + (2 w + half) * 4 + 0..3, P pairs of key rows.
-template <int P>
+// Lane (rg = lane & 7, cg = lane >> 3) of warp w: value columns col0 + 8 w + 2 cg + 0, 1.
+template <int Q>
 __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared in, int first, Status* status) {
   ptx::grid_dep_sync();
-  using L = ScanLayout<P>;
+  using L = ScanLayout<Q>;
   extern __shared__ __align__(128) float scan_sm[];
-  const int seq = first + blockIdx.z, h = blockIdx.y, blk = blockIdx.x, col0 = blk * kCols;
+  const int seq = first + blockIdx.z, h = blockIdx.y, blk = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int begin = sq.seq_rows[2 * seq];
   ConvRow cr;
   if (sq.seq_rows[2 * seq + 1] <= begin || !cr.load(sq, seq, begin, sq.banks, status)) return;      // uniform per CTA
   const int d = a.dim, e = a.vdim, n = cr.end - cr.begin;
-  const int n_tiles = (n + kTile - 1) / kTile;
-  float* neutral = scan_sm + kStages * L::kStage;
-  const uint32_t bars = ptx::smem_u32(neutral + L::kNeutral);
+  const int n_pairs = (n + 1) >> 1, n_tiles = (n_pairs + kTile - 1) / kTile, pair0 = first_pair(begin, seq);
+  const uint32_t bars = ptx::smem_u32(scan_sm + kStages * L::kStage);
   if (threadIdx.x == 0) {
     for (int s = 0; s < kStages; ++s) ptx::mbar_init(bars + 8 * s, 1);
     ptx::fence_mbar_init();
   }
-  for (int i = threadIdx.x; i < L::kNeutral; i += 128) neutral[i] = i >= 2 * L::kD && i < 3 * L::kD ? 1.0f : 0.0f;
   __syncthreads();
+  const float *g_vec = in.vec_at(h, pair0), *g_v = in.v_at(h, blk, pair0), *g_sc = in.sc_at(h, pair0);
   const auto issue = [&](int i) {      // thread 0: start the copies of tile i
-    const int rows = min(kTile, n - i * kTile), row = begin + i * kTile;
-    float* st = scan_sm + (i % kStages) * L::kStage;
-    const uint32_t bar = bars + 8 * (i % kStages);
-    ptx::mbar_arrive_expect_tx(bar, static_cast<uint32_t>(rows * (3 * L::kD + kCols + 4) * 4));
-    ptx::bulk_load(ptx::smem_u32(st), in.qkg_row(h, row), rows * 3 * L::kD * 4, bar);
-    ptx::bulk_load(ptx::smem_u32(st + L::kQkg), in.v_row(h, blk, row), rows * kCols * 4, bar);
-    ptx::bulk_load(ptx::smem_u32(st + L::kQkg + L::kV), in.sc_row(h, row), rows * 16, bar);
+    const int m = min(kTile, n_pairs - i * kTile);
+    const uint32_t st = ptx::smem_u32(scan_sm + (i % kStages) * L::kStage), bar = bars + 8 * (i % kStages);
+    ptx::mbar_arrive_expect_tx(bar, static_cast<uint32_t>(m * (L::kVec + L::kV + L::kSc) * 4));
+    ptx::bulk_load(st, g_vec + static_cast<int64_t>(i) * kTile * L::kVec, m * L::kVec * 4, bar);
+    ptx::bulk_load(st + L::kOffV * 4, g_v + static_cast<int64_t>(i) * kTile * L::kV, m * L::kV * 4, bar);
+    ptx::bulk_load(st + L::kOffSc * 4, g_sc + static_cast<int64_t>(i) * kTile * L::kSc, m * L::kSc * 4, bar);
   };
   if (threadIdx.x == 0)
     for (int i = 0; i < kStages - 1 && i < n_tiles; ++i) issue(i);
 
-  const int rg = lane & 15, c4 = (2 * warp + (lane >> 4)) * 4, base_lane = lane & 16;
-  const bool b3 = lane & 8, b2_ = lane & 4, b1 = lane & 2, b0 = lane & 1;
-  const int my_col = lane & 3;      // after the reduction a lane holds one sum: kind (S^T k, S^T q) = bit 3, row = bit 2, column = bits 1, 0
-  float* state = a.state + (static_cast<int64_t>(cr.wr >> 1) * a.heads + h) * d * e + col0 + c4;
-  uint64_t S[P][4];
+  const int rg = lane & 7, c2 = 8 * warp + 2 * (lane >> 3), col = blk * kCols + c2, group = lane & 24;
+  // after the reduction over the 8 row groups a lane holds one sum: kind (S^T k, S^T q) = bit 2, row of the pair = bit 1,
+  // column = bit 0
+  const bool is_q = lane & 4, second = lane & 2, odd = lane & 1;
+  float* state = a.state + (static_cast<int64_t>(cr.wr >> 1) * a.heads + h) * d * e + col;
+  uint64_t S[2 * Q][2];
 #pragma unroll
-  for (int p = 0; p < P; ++p) {
-    const int key = pair_row<P>(p, rg);
+  for (int p = 0; p < 2 * Q; ++p) {
+    const int key = (p >> 1) * 32 + rg * 4 + (p & 1) * 2;
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
+    for (int c = 0; c < 2; ++c) {
       float lo = 0.0f, hi = 0.0f;
-      if (cr.rd >= 0 && col0 + c4 + c < e) {
+      if (cr.rd >= 0 && col + c < e) {
         if (key < d) lo = state[static_cast<int64_t>(key) * e + c];
         if (key + 1 < d) hi = state[static_cast<int64_t>(key + 1) * e + c];
       }
@@ -468,8 +619,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
     }
   }
   const int64_t o_ld = static_cast<int64_t>(a.heads) * e;
-  float* o_dst = a.o_raw + static_cast<int64_t>(begin + (b2_ ? 1 : 0)) * o_ld + static_cast<int64_t>(h) * e + col0 + c4 + my_col;
-  const bool writes = b3 && col0 + c4 + my_col < e;
+  float* o_dst = a.o_raw + static_cast<int64_t>(begin + (second ? 1 : 0)) * o_ld + static_cast<int64_t>(h) * e + col + (odd ? 1 : 0);
+  const bool writes = is_q && col + (odd ? 1 : 0) < e;
   bool failed = false;
   for (int i = 0; i < n_tiles; ++i) {
     // the stage of tile i - 1 was released by the barrier at the end of that tile
@@ -479,72 +630,67 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
       failed = true;
     }
     const float* st = scan_sm + (i % kStages) * L::kStage;
-    const int rows = min(kTile, n - i * kTile);
+    const int m = min(kTile, n_pairs - i * kTile);
 #pragma unroll 1
-    for (int t = 0; t < rows; t += 2) {
-      const bool two = t + 1 < rows;
-      const float* t1 = st + t * 3 * L::kD;
-      const float* t2 = two ? t1 + 3 * L::kD : neutral;
-      const float* v1 = st + L::kQkg + t * kCols + c4;
-      const float* v2 = two ? v1 + kCols : neutral + 3 * L::kD;
-      const float4 sc1 = *reinterpret_cast<const float4*>(st + L::kQkg + L::kV + t * 4);
-      const float4 sc2 = *reinterpret_cast<const float4*>(two ? st + L::kQkg + L::kV + t * 4 + 4 : neutral + 3 * L::kD + kCols);
-      uint64_t q1[P], k1[P], g1[P], q2[P], k2[P], g2[P];
-      load_pairs<P>(t1, rg, q1);
-      load_pairs<P>(t1 + L::kD, rg, k1);
-      load_pairs<P>(t1 + 2 * L::kD, rg, g1);
-      load_pairs<P>(t2, rg, q2);
-      load_pairs<P>(t2 + L::kD, rg, k2);
-      load_pairs<P>(t2 + 2 * L::kD, rg, g2);
-      uint64_t acc[4][4];      // [S1 k1, S1 q1 | S2 k2, S2 q2] per column, even and odd rows apart
+    for (int t = 0; t < m; ++t) {
+      const float* vec = st + t * L::kVec;
+      const float4 sc = *reinterpret_cast<const float4*>(st + L::kOffSc + t * L::kSc);              // beta1, k1.q1, beta2, k2.q2
+      const float2 cross = *reinterpret_cast<const float2*>(st + L::kOffSc + t * L::kSc + 4);      // w1.k2, w1.q2
+      const float* v = st + L::kOffV + t * L::kV + c2 + (odd ? 1 : 0);
+      const float v1 = v[0], v2 = v[kCols];
+      uint64_t acc[4][2];      // S^T of g1 k1, g1 g2 k2, g1 q1, g1 g2 q2; even and odd rows apart
+      const int which[4] = {kGK1, kGK2, kGQ1, kGQ2};
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
+      for (int j = 0; j < 4; ++j) {
+        uint64_t x[2 * Q];
+        load_quads<Q>(vec + which[j] * L::kD, rg, x);
+        acc[j][0] = acc[j][1] = 0;
 #pragma unroll
-        for (int c = 0; c < 4; ++c) acc[j][c] = 0;
-#pragma unroll
-      for (int p = 0; p < P; ++p) {
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          S[p][c] = mul2(S[p][c], g1[p]);
-          acc[0][c] = fma2(S[p][c], k1[p], acc[0][c]);
-          acc[1][c] = fma2(S[p][c], q1[p], acc[1][c]);
-          S[p][c] = mul2(S[p][c], g2[p]);
-          acc[2][c] = fma2(S[p][c], k2[p], acc[2][c]);
-          acc[3][c] = fma2(S[p][c], q2[p], acc[3][c]);
+        for (int p = 0; p < 2 * Q; ++p) {
+          acc[j][0] = fma2(S[p][0], x[p], acc[j][0]);
+          acc[j][1] = fma2(S[p][1], x[p], acc[j][1]);
         }
-        k1[p] = mul2(k1[p], g2[p]);      // the first row's write, decayed by the second row
       }
-      // sum over the 16 lane groups, halving the values per lane: kind, row, then two bits of the column
-      float x8[8], x4[4], x2[2], x;
+      // decay the state while the sums travel
+      {
+        uint64_t gg[2 * Q];
+        load_quads<Q>(vec + kGG * L::kD, rg, gg);
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const float sk1 = half_sum(acc[0][c]), sq1 = half_sum(acc[1][c]), sk2 = half_sum(acc[2][c]), sq2 = half_sum(acc[3][c]);
-        x8[c] = (b3 ? sq1 : sk1) + __shfl_xor_sync(0xffffffffu, b3 ? sk1 : sq1, 8);
-        x8[4 + c] = (b3 ? sq2 : sk2) + __shfl_xor_sync(0xffffffffu, b3 ? sk2 : sq2, 8);
+        for (int p = 0; p < 2 * Q; ++p) {
+          S[p][0] = mul2(S[p][0], gg[p]);
+          S[p][1] = mul2(S[p][1], gg[p]);
+        }
       }
+      float x4[4], x2[2], x;
 #pragma unroll
-      for (int c = 0; c < 4; ++c) x4[c] = (b2_ ? x8[4 + c] : x8[c]) + __shfl_xor_sync(0xffffffffu, b2_ ? x8[c] : x8[4 + c], 4);
-#pragma unroll
-      for (int c = 0; c < 2; ++c) x2[c] = (b1 ? x4[2 + c] : x4[c]) + __shfl_xor_sync(0xffffffffu, b1 ? x4[c] : x4[2 + c], 2);
-      x = (b0 ? x2[1] : x2[0]) + __shfl_xor_sync(0xffffffffu, b0 ? x2[0] : x2[1], 1);
-      const float u1_own = sc1.x * (v1[my_col] - x);                                              // right where bits 3, 2 are clear
-      const float u1s = __shfl_sync(0xffffffffu, u1_own, base_lane + my_col);                     // row 1's u of this lane's column
-      const float u2_own = sc2.x * (v2[my_col] - fmaf(u1s, sc2.z, x));                            // right where bit 3 is clear, bit 2 set
-      float u1[4], u2[4];
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        u1[c] = __shfl_sync(0xffffffffu, u1_own, base_lane + c);
-        u2[c] = __shfl_sync(0xffffffffu, u2_own, base_lane + 4 + c);
+      for (int c = 0; c < 2; ++c) {
+        const float sk1 = half_sum(acc[0][c]), sk2 = half_sum(acc[1][c]), sq1 = half_sum(acc[2][c]), sq2 = half_sum(acc[3][c]);
+        x4[c] = (is_q ? sq1 : sk1) + __shfl_xor_sync(0xffffffffu, is_q ? sk1 : sq1, 4);
+        x4[2 + c] = (is_q ? sq2 : sk2) + __shfl_xor_sync(0xffffffffu, is_q ? sk2 : sq2, 4);
       }
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const uint64_t w1 = pack2(u1[c], u1[c]), w2 = pack2(u2[c], u2[c]);
+      for (int c = 0; c < 2; ++c) x2[c] = (second ? x4[2 + c] : x4[c]) + __shfl_xor_sync(0xffffffffu, second ? x4[c] : x4[2 + c], 2);
+      x = (odd ? x2[1] : x2[0]) + __shfl_xor_sync(0xffffffffu, odd ? x2[0] : x2[1], 1);
+      const float u1_own = sc.x * (v1 - x);                                           // right in lanes 0, 1 of a group
+      const float a0 = __shfl_sync(0xffffffffu, u1_own, group), a1 = __shfl_sync(0xffffffffu, u1_own, group + 1);
+      const float u1s = odd ? a1 : a0;
+      const float u2_own = sc.z * (v2 - fmaf(u1s, cross.x, x));                       // right in lanes 2, 3
+      const float b0 = __shfl_sync(0xffffffffu, u2_own, group + 2), b1 = __shfl_sync(0xffffffffu, u2_own, group + 3);
+      {
+        uint64_t w1[2 * Q], w2[2 * Q];
+        load_quads<Q>(vec + kW1 * L::kD, rg, w1);
+        load_quads<Q>(vec + kW2 * L::kD, rg, w2);
+        const uint64_t ua0 = pack2(a0, a0), ua1 = pack2(a1, a1), ub0 = pack2(b0, b0), ub1 = pack2(b1, b1);
 #pragma unroll
-        for (int p = 0; p < P; ++p) S[p][c] = fma2(k2[p], w2, fma2(k1[p], w1, S[p][c]));
+        for (int p = 0; p < 2 * Q; ++p) {
+          S[p][0] = fma2(w2[p], ub0, fma2(w1[p], ua0, S[p][0]));
+          S[p][1] = fma2(w2[p], ub1, fma2(w1[p], ua1, S[p][1]));
+        }
       }
-      const float u2s = b1 ? (b0 ? u2[3] : u2[2]) : (b0 ? u2[1] : u2[0]);
-      const float o = b2_ ? fmaf(u2s, sc2.y, fmaf(u1s, sc2.w, x)) : fmaf(u1s, sc1.y, x);
-      if (writes && (two || !b2_)) o_dst[static_cast<int64_t>(i * kTile + t) * o_ld] = o;
+      const float u2s = odd ? b1 : b0;
+      const float o = second ? fmaf(u2s, sc.w, fmaf(u1s, cross.y, x)) : fmaf(u1s, sc.y, x);
+      const int row = 2 * (i * kTile + t);
+      if (writes && row + (second ? 1 : 0) < n) o_dst[static_cast<int64_t>(row) * o_ld] = o;
     }
     if (__syncthreads_or(failed)) break;      // also releases the stage
   }
@@ -554,11 +700,11 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
     return;
   }
 #pragma unroll
-  for (int p = 0; p < P; ++p) {
-    const int key = pair_row<P>(p, rg);
+  for (int p = 0; p < 2 * Q; ++p) {
+    const int key = (p >> 1) * 32 + rg * 4 + (p & 1) * 2;
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      if (col0 + c4 + c >= e) continue;
+    for (int c = 0; c < 2; ++c) {
+      if (col + c >= e) continue;
       const float2 f = unpack2(S[p][c]);
       if (key < d) state[static_cast<int64_t>(key) * e + c] = f.x;
       if (key + 1 < d) state[static_cast<int64_t>(key + 1) * e + c] = f.y;
@@ -588,7 +734,7 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const B2DeltaArgs a, con
     for (int i = 0; i < VEC; ++i) ss = fmaf(v[j][i], v[j][i], ss);
   }
   ss = warp_sum(ss);
-  const float r = 1.0f / sqrtf(ss / static_cast<float>(e) + a.eps);
+  const float r = rsqrtf(ss / static_cast<float>(e) + a.eps);
 #pragma unroll
   for (int j = 0; j < NJ; ++j) {
     const int c = (lane + 32 * j) * VEC;
@@ -597,17 +743,17 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const B2DeltaArgs a, con
     load_f32<VEC>(gate + c, z);
     load_f32<VEC>(a.norm_w + c, w);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) v[j][i] = v[j][i] * r * w[i] * sigmoid_f32(z[i]);
+    for (int i = 0; i < VEC; ++i) v[j][i] = v[j][i] * r * w[i] * sigmoid(z[i]);
     store_f32<VEC>(out + c, v[j]);
   }
 }
 
-template <int P>
+template <int Q>
 int launch_scan(const B2DeltaArgs& a, const B2SeqRows& s, int first, int n, Status* status, cudaStream_t stream) {
-  using L = ScanLayout<P>;
+  using L = ScanLayout<Q>;
   static DeviceOnce attr_once;
-  if (const int rc = attr_once.max_smem(delta_scan_kernel<P>, L::kBytes)) return rc;
-  launch_pdl(delta_scan_kernel<P>, dim3((a.vdim + kCols - 1) / kCols, a.heads, n), dim3(128), L::kBytes, stream, a, s, prepared_of(a, s.rows), first, status);
+  if (const int rc = attr_once.max_smem(delta_scan_kernel<Q>, L::kBytes)) return rc;
+  launch_pdl(delta_scan_kernel<Q>, dim3((a.vdim + kCols - 1) / kCols, a.heads, n), dim3(128), L::kBytes, stream, a, s, prepared_of(a, s), first, status);
   return last_launch_rc();
 }
 
@@ -640,7 +786,9 @@ int run_delta(const B2DeltaArgs& a, const B2SeqRows& s, int n_decode, int first,
 
 using namespace b2;
 
-extern "C" int64_t b2_delta_scratch_floats(int heads, int dim, int vdim, int rows) { return scratch_floats(heads, dim, vdim, rows); }
+extern "C" int64_t b2_delta_scratch_floats(int heads, int dim, int vdim, int rows, int seqs) {
+  return scratch_floats(heads, dim, vdim, rows, seqs);
+}
 
 extern "C" int b2_delta_rule(const B2DeltaArgs* a, const B2SeqRows* s, int n_decode, int first, int n_prefill, int f32, Status* status,
                              cudaStream_t stream) {

@@ -18,7 +18,7 @@ constexpr int kWarps = 8;
 
 // A warp's rows: runs of rows of one sequence, each convolved at once (`conv_rows`), then rotated and normalised row by row.
 template <typename T, int VEC, int NJ, int TAPS, int TT>
-__global__ void __launch_bounds__(kWarps * 32) conv_qkv_kernel(const B2ConvQkvArgs a, const B2SeqRows sq, Status* status) {
+__global__ void __launch_bounds__(kWarps * 32, TAPS > 0 && NJ == 1 ? 3 : 1) conv_qkv_kernel(const B2ConvQkvArgs a, const B2SeqRows sq, Status* status) {
   ptx::grid_dep_sync();
   __shared__ __align__(16) float head_sm[kWarps][kMaxHead];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -33,6 +33,7 @@ __global__ void __launch_bounds__(kWarps * 32) conv_qkv_kernel(const B2ConvQkvAr
   const int half = a.rot >> 1;
   const ConvSource<T> src{static_cast<const T*>(a.proj), a.ld, a.conv_w, static_cast<T*>(a.conv_state), a.taps, channels, sq.banks};
   float* hs = head_sm[warp];
+  const float inv_dim = 1.0f / static_cast<float>(dim);
   const int row_end = min(sq.rows, static_cast<int>(blockIdx.x + 1) * TT);
   int run = 0;
   for (int row0 = blockIdx.x * TT; row0 < row_end; row0 += run) {
@@ -104,7 +105,7 @@ __global__ void __launch_bounds__(kWarps * 32) conv_qkv_kernel(const B2ConvQkvAr
           for (int v = 0; v < VEC; ++v) ss = fmaf(val[j][t][v], val[j][t][v], ss);      // 0 past dim
         }
         ss = warp_sum(ss);
-        const float r = 1.0f / sqrtf(ss / static_cast<float>(dim) + a.eps);
+        const float r = rsqrtf(ss * inv_dim + a.eps);
 #pragma unroll
         for (int j = 0; j < NJ; ++j)
 #pragma unroll
@@ -118,7 +119,9 @@ __global__ void __launch_bounds__(kWarps * 32) conv_qkv_kernel(const B2ConvQkvAr
         const int64_t slot = a.slots[row];
         if (slot < 0 || !B2_ASSERT(status, slot < a.num_slots, kSiteKvIndex, slot, a.num_slots)) continue;
         T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache);
-        dst = cache + ((slot / a.page_size * a.kv_heads + kvh) * a.page_size + slot % a.page_size) * pad;
+        const uint32_t page = static_cast<uint32_t>(slot) / static_cast<uint32_t>(a.page_size);      // the host keeps slots below 2^31
+        const uint32_t in_page = static_cast<uint32_t>(slot) - page * a.page_size;
+        dst = cache + ((static_cast<int64_t>(page) * a.kv_heads + kvh) * a.page_size + in_page) * pad;
         lim = dim;
       }
 #pragma unroll
@@ -136,7 +139,7 @@ template <typename T, int VEC, int NJ, int TAPS>
 int launch_conv_qkv(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
   const int groups = (a.heads + 2 * a.kv_heads + kWarps - 1) / kWarps;
   // rows of one warp share the convolution's window; a small step wants one warp per row
-  constexpr int kRows = TAPS == 0 ? 2 : VEC * NJ > 4 ? 4 : 8;
+  constexpr int kRows = TAPS == 0 ? 2 : 4;
   if ((s.rows + kRows - 1) / kRows * groups < 2 * kNumSMs)
     launch_pdl(conv_qkv_kernel<T, VEC, NJ, TAPS, 1>, dim3(s.rows, groups), dim3(kWarps * 32), 0, stream, a, s, status);
   else
@@ -170,7 +173,7 @@ extern "C" int b2_conv_qkv(const B2ConvQkvArgs* a, const B2SeqRows* s, int f32, 
   if (a->heads <= 0 || a->kv_heads < 0 || a->dim <= 0 || a->dim > kMaxHead || a->vdim > kMaxHead || a->pad_dim < a->dim || a->rot % 2 != 0 ||
       a->rot > a->dim || a->taps < 1 || (a->taps > 1 && a->conv_state == nullptr) || a->q_out == nullptr || (a->rot > 0 && a->cos_sin == nullptr))
     return -kBadArgument;
-  if (a->kv_heads > 0 && (a->k_cache == nullptr || a->v_cache == nullptr || a->slots == nullptr || a->pad_vdim < a->vdim || a->page_size <= 0 ||
+  if (a->kv_heads > 0 && (a->k_cache == nullptr || a->v_cache == nullptr || a->slots == nullptr || a->pad_vdim < a->vdim || a->page_size <= 0 || a->num_slots > 0x7fffffff ||
                           a->heads % a->kv_heads != 0))
     return -kBadArgument;
   return f32 ? dispatch_conv_qkv<float>(*a, *s, status, stream) : dispatch_conv_qkv<__nv_bfloat16>(*a, *s, status, stream);

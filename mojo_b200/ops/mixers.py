@@ -135,7 +135,7 @@ def delta_rule(proj: torch.Tensor, dg: torch.Tensor, p: DeltaParams, conv_state:
     make = torch.empty if out_cols == heads * vdim else torch.zeros
     out = make(T, out_cols, dtype=proj.dtype, device=proj.device)
 
-    scratch = torch.empty(C.delta_scratch_floats(heads, dim, vdim, T), dtype=torch.float32, device=proj.device)
+    scratch = torch.empty(C.delta_scratch_floats(heads, dim, vdim, T, seq.seq_rows.shape[0]), dtype=torch.float32, device=proj.device)
     raw = torch.empty(T, heads * vdim, dtype=torch.float32, device=proj.device) if seq.n_prefill else None
     C.delta_rule(proj, dg, p.conv_w, conv_state, p.neg_rate, p.dt_bias, p.norm_w, state, seq.row_seq, seq.seq_rows, seq.seq_state, out, scratch, raw,
                  b_off, heads, kv_heads, dim, vdim, eps, seq.n_decode, seq.first, seq.n_prefill, st.status)
