@@ -114,12 +114,20 @@ __device__ __forceinline__ void conv_rows(const ConvSource<T>& s, const ConvRow&
     }
   } else {
     RawVec<T, VEC> u[TT + TAPS - 1];
+    // inside a sequence, away from its first and last rows of the step, nothing but projection rows is touched
+    const bool interior = n == TT && row0 - (TAPS - 1) >= r.begin && r.end - row0 >= TT + TAPS - 1;
+    if (interior) {
+      const T* p = s.proj + static_cast<int64_t>(row0 - (TAPS - 1)) * s.ld + chan;
 #pragma unroll
-    for (int i = 0; i < TT + TAPS - 1; ++i) {
-      const int src = row0 - (TAPS - 1) + i;
-      const T* p = src >= r.begin ? s.proj + src * s.ld + chan : r.rd >= 0 ? s.bank(r.rd, TAPS - 1 - (r.begin - src), chan) : nullptr;
-      if (i < n + TAPS - 1 && p != nullptr) u[i].load(p);
-      else u[i].zero();
+      for (int i = 0; i < TT + TAPS - 1; ++i, p += s.ld) u[i].load(p);
+    } else {
+#pragma unroll
+      for (int i = 0; i < TT + TAPS - 1; ++i) {
+        const int src = row0 - (TAPS - 1) + i;
+        const T* p = src >= r.begin ? s.proj + src * s.ld + chan : r.rd >= 0 ? s.bank(r.rd, TAPS - 1 - (r.begin - src), chan) : nullptr;
+        if (i < n + TAPS - 1 && p != nullptr) u[i].load(p);
+        else u[i].zero();
+      }
     }
     float w[TAPS][VEC];
 #pragma unroll
@@ -133,7 +141,7 @@ __device__ __forceinline__ void conv_rows(const ConvSource<T>& s, const ConvRow&
         for (int j = 0; j < TAPS; ++j) a = fmaf(w[j][v], u[t + j].get(v), a);
         y[t][v] = a;
       }
-    if (save) {
+    if (save && !interior) {
 #pragma unroll
       for (int t = 0; t < TT; ++t)
         if (t < n && r.end - (row0 + t) <= TAPS - 1) u[t + TAPS - 1].store(s.bank(r.wr, TAPS - 1 - (r.end - (row0 + t)), chan));

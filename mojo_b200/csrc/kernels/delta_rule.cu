@@ -149,23 +149,35 @@ __global__ void __launch_bounds__(128, TAPS > 0 && NJ == 1 ? 6 : 1) delta_prep_k
     }
   }
   const float q_scale = rsqrtf(static_cast<float>(d));
-  float kq[TT];
+  float qq[TT], kk[TT], kq[TT];
 #pragma unroll
   for (int t = 0; t < TT; ++t) {
-    float qq = 0.0f, kk = 0.0f, qk = 0.0f;
+    qq[t] = kk[t] = kq[t] = 0.0f;
 #pragma unroll
     for (int j = 0; j < NJ; ++j)
 #pragma unroll
       for (int v = 0; v < VEC; ++v) {
-        qq = fmaf(q[j][t][v], q[j][t][v], qq);
-        kk = fmaf(k[j][t][v], k[j][t][v], kk);
-        qk = fmaf(q[j][t][v], k[j][t][v], qk);
+        qq[t] = fmaf(q[j][t][v], q[j][t][v], qq[t]);
+        kk[t] = fmaf(k[j][t][v], k[j][t][v], kk[t]);
+        kq[t] = fmaf(q[j][t][v], k[j][t][v], kq[t]);
       }
-    qq = warp_sum(qq);
-    kk = warp_sum(kk);
-    qk = warp_sum(qk);
-    const float rq = q_scale * rsqrtf(qq + kUnitEps), rk = rsqrtf(kk + kUnitEps);
-    kq[t] = qk * rq * rk;
+  }
+  if constexpr (TT == 4) {
+    warp_sum4(qq);
+    warp_sum4(kk);
+    warp_sum4(kq);
+  } else {
+#pragma unroll
+    for (int t = 0; t < TT; ++t) {
+      qq[t] = warp_sum(qq[t]);
+      kk[t] = warp_sum(kk[t]);
+      kq[t] = warp_sum(kq[t]);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < TT; ++t) {
+    const float rq = q_scale * rsqrtf(qq[t] + kUnitEps), rk = rsqrtf(kk[t] + kUnitEps);
+    kq[t] *= rq * rk;
 #pragma unroll
     for (int j = 0; j < NJ; ++j)
 #pragma unroll
@@ -549,30 +561,42 @@ __device__ __forceinline__ float half_sum(uint64_t v) {
   return f.x + f.y;
 }
 
-// A lane holds two value columns and Q quads of key rows: quad i of row group rg is rows 32 i + 4 rg + 0..3 (kd = 32 Q).
-template <int Q>
+// A lane holds four value columns and P pairs of key rows (kd = 32 P). The 16 row groups of a half-warp read 256 different
+// bytes of a vector at once; a mapping with more rows and fewer columns per lane reads the same bytes more often, and
+// shared-memory bandwidth is what two CTAs on one SM run short of first.
+template <int P>
 struct ScanLayout {
-  static constexpr int kD = 32 * Q;
+  static constexpr int kD = 32 * P;
   static constexpr int kVec = kVecs * kD, kV = 2 * kCols, kSc = 8;       // floats per pair
   static constexpr int kOffV = kTile * kVec, kOffSc = kOffV + kTile * kV;
   static constexpr int kStage = kOffSc + kTile * kSc;
   static constexpr int kBytes = kStages * kStage * 4 + kStages * 8;
 };
-template <int Q>
-__device__ __forceinline__ void load_quads(const float* x, int rg, uint64_t (&v)[2 * Q]) {
+// Pair p of row group rg is key rows pair_row(p, rg) and the next one.
+template <int P>
+__device__ __forceinline__ int pair_row(int p, int rg) {
+  if constexpr (P == 1) return 2 * rg;
+  else return (p >> 1) * 64 + rg * 4 + (p & 1) * 2;
+}
+template <int P>
+__device__ __forceinline__ void load_pairs(const float* x, int rg, uint64_t (&v)[P]) {
+  if constexpr (P == 1) {
+    v[0] = *reinterpret_cast<const uint64_t*>(x + 2 * rg);
+  } else {
 #pragma unroll
-  for (int i = 0; i < Q; ++i) {
-    const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(x + 32 * i + 4 * rg);
-    v[2 * i] = t.x;
-    v[2 * i + 1] = t.y;
+    for (int i = 0; i < P / 2; ++i) {
+      const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(x + i * 64 + rg * 4);
+      v[2 * i] = t.x;
+      v[2 * i + 1] = t.y;
+    }
   }
 }
 
-// Lane (rg = lane & 7, cg = lane >> 3) of warp w: value columns col0 + 8 w + 2 cg + 0, 1.
-template <int Q>
+// Lane (rg = lane & 15, half = lane >> 4) of warp w: value columns col0 + 8 w + 4 half + 0..3.
+template <int P>
 __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared in, int first, Status* status) {
   ptx::grid_dep_sync();
-  using L = ScanLayout<Q>;
+  using L = ScanLayout<P>;
   extern __shared__ __align__(128) float scan_sm[];
   const int seq = first + blockIdx.z, h = blockIdx.y, blk = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -599,17 +623,18 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
   if (threadIdx.x == 0)
     for (int i = 0; i < kStages - 1 && i < n_tiles; ++i) issue(i);
 
-  const int rg = lane & 7, c2 = 8 * warp + 2 * (lane >> 3), col = blk * kCols + c2, group = lane & 24;
-  // after the reduction over the 8 row groups a lane holds one sum: kind (S^T k, S^T q) = bit 2, row of the pair = bit 1,
-  // column = bit 0
-  const bool is_q = lane & 4, second = lane & 2, odd = lane & 1;
+  const int rg = lane & 15, c4 = 8 * warp + 4 * (lane >> 4), col = blk * kCols + c4, half = lane & 16;
+  // after the reduction over the 16 row groups a lane holds one sum: kind (S^T k, S^T q) = bit 3, row of the pair = bit 2,
+  // column = bits 1, 0
+  const bool is_q = lane & 8, second = lane & 4, b1 = lane & 2, b0 = lane & 1;
+  const int mine = lane & 3;
   float* state = a.state + (static_cast<int64_t>(cr.wr >> 1) * a.heads + h) * d * e + col;
-  uint64_t S[2 * Q][2];
+  uint64_t S[P][4];
 #pragma unroll
-  for (int p = 0; p < 2 * Q; ++p) {
-    const int key = (p >> 1) * 32 + rg * 4 + (p & 1) * 2;
+  for (int p = 0; p < P; ++p) {
+    const int key = pair_row<P>(p, rg);
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
+    for (int c = 0; c < 4; ++c) {
       float lo = 0.0f, hi = 0.0f;
       if (cr.rd >= 0 && col + c < e) {
         if (key < d) lo = state[static_cast<int64_t>(key) * e + c];
@@ -619,8 +644,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
     }
   }
   const int64_t o_ld = static_cast<int64_t>(a.heads) * e;
-  float* o_dst = a.o_raw + static_cast<int64_t>(begin + (second ? 1 : 0)) * o_ld + static_cast<int64_t>(h) * e + col + (odd ? 1 : 0);
-  const bool writes = is_q && col + (odd ? 1 : 0) < e;
+  float* o_dst = a.o_raw + static_cast<int64_t>(begin + (second ? 1 : 0)) * o_ld + static_cast<int64_t>(h) * e + col + mine;
+  const bool writes = is_q && col + mine < e;
   bool failed = false;
   for (int i = 0; i < n_tiles; ++i) {
     // the stage of tile i - 1 was released by the barrier at the end of that tile
@@ -636,58 +661,62 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
       const float* vec = st + t * L::kVec;
       const float4 sc = *reinterpret_cast<const float4*>(st + L::kOffSc + t * L::kSc);              // beta1, k1.q1, beta2, k2.q2
       const float2 cross = *reinterpret_cast<const float2*>(st + L::kOffSc + t * L::kSc + 4);      // w1.k2, w1.q2
-      const float* v = st + L::kOffV + t * L::kV + c2 + (odd ? 1 : 0);
+      const float* v = st + L::kOffV + t * L::kV + c4 + mine;
       const float v1 = v[0], v2 = v[kCols];
-      uint64_t acc[4][2];      // S^T of g1 k1, g1 g2 k2, g1 q1, g1 g2 q2; even and odd rows apart
+      uint64_t acc[4][4];      // S^T of g1 k1, g1 g2 k2, g1 q1, g1 g2 q2; even and odd rows apart
       const int which[4] = {kGK1, kGK2, kGQ1, kGQ2};
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        uint64_t x[2 * Q];
-        load_quads<Q>(vec + which[j] * L::kD, rg, x);
-        acc[j][0] = acc[j][1] = 0;
+        uint64_t x[P];
+        load_pairs<P>(vec + which[j] * L::kD, rg, x);
 #pragma unroll
-        for (int p = 0; p < 2 * Q; ++p) {
-          acc[j][0] = fma2(S[p][0], x[p], acc[j][0]);
-          acc[j][1] = fma2(S[p][1], x[p], acc[j][1]);
-        }
+        for (int c = 0; c < 4; ++c) acc[j][c] = mul2(S[0][c], x[0]);
+#pragma unroll
+        for (int p = 1; p < P; ++p)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) acc[j][c] = fma2(S[p][c], x[p], acc[j][c]);
       }
       // decay the state while the sums travel
       {
-        uint64_t gg[2 * Q];
-        load_quads<Q>(vec + kGG * L::kD, rg, gg);
+        uint64_t gg[P];
+        load_pairs<P>(vec + kGG * L::kD, rg, gg);
 #pragma unroll
-        for (int p = 0; p < 2 * Q; ++p) {
-          S[p][0] = mul2(S[p][0], gg[p]);
-          S[p][1] = mul2(S[p][1], gg[p]);
-        }
+        for (int p = 0; p < P; ++p)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) S[p][c] = mul2(S[p][c], gg[p]);
       }
-      float x4[4], x2[2], x;
+      float x8[8], x4[4], x2[2], x;
 #pragma unroll
-      for (int c = 0; c < 2; ++c) {
+      for (int c = 0; c < 4; ++c) {
         const float sk1 = half_sum(acc[0][c]), sk2 = half_sum(acc[1][c]), sq1 = half_sum(acc[2][c]), sq2 = half_sum(acc[3][c]);
-        x4[c] = (is_q ? sq1 : sk1) + __shfl_xor_sync(0xffffffffu, is_q ? sk1 : sq1, 4);
-        x4[2 + c] = (is_q ? sq2 : sk2) + __shfl_xor_sync(0xffffffffu, is_q ? sk2 : sq2, 4);
+        x8[c] = (is_q ? sq1 : sk1) + __shfl_xor_sync(0xffffffffu, is_q ? sk1 : sq1, 8);
+        x8[4 + c] = (is_q ? sq2 : sk2) + __shfl_xor_sync(0xffffffffu, is_q ? sk2 : sq2, 8);
       }
 #pragma unroll
-      for (int c = 0; c < 2; ++c) x2[c] = (second ? x4[2 + c] : x4[c]) + __shfl_xor_sync(0xffffffffu, second ? x4[c] : x4[2 + c], 2);
-      x = (odd ? x2[1] : x2[0]) + __shfl_xor_sync(0xffffffffu, odd ? x2[0] : x2[1], 1);
-      const float u1_own = sc.x * (v1 - x);                                           // right in lanes 0, 1 of a group
-      const float a0 = __shfl_sync(0xffffffffu, u1_own, group), a1 = __shfl_sync(0xffffffffu, u1_own, group + 1);
-      const float u1s = odd ? a1 : a0;
-      const float u2_own = sc.z * (v2 - fmaf(u1s, cross.x, x));                       // right in lanes 2, 3
-      const float b0 = __shfl_sync(0xffffffffu, u2_own, group + 2), b1 = __shfl_sync(0xffffffffu, u2_own, group + 3);
-      {
-        uint64_t w1[2 * Q], w2[2 * Q];
-        load_quads<Q>(vec + kW1 * L::kD, rg, w1);
-        load_quads<Q>(vec + kW2 * L::kD, rg, w2);
-        const uint64_t ua0 = pack2(a0, a0), ua1 = pack2(a1, a1), ub0 = pack2(b0, b0), ub1 = pack2(b1, b1);
+      for (int c = 0; c < 4; ++c) x4[c] = (second ? x8[4 + c] : x8[c]) + __shfl_xor_sync(0xffffffffu, second ? x8[c] : x8[4 + c], 4);
 #pragma unroll
-        for (int p = 0; p < 2 * Q; ++p) {
-          S[p][0] = fma2(w2[p], ub0, fma2(w1[p], ua0, S[p][0]));
-          S[p][1] = fma2(w2[p], ub1, fma2(w1[p], ua1, S[p][1]));
+      for (int c = 0; c < 2; ++c) x2[c] = (b1 ? x4[2 + c] : x4[c]) + __shfl_xor_sync(0xffffffffu, b1 ? x4[c] : x4[2 + c], 2);
+      x = (b0 ? x2[1] : x2[0]) + __shfl_xor_sync(0xffffffffu, b0 ? x2[0] : x2[1], 1);
+      const float u1_own = sc.x * (v1 - x);                                           // right in lanes 0-3 of a half
+      const float u1s = __shfl_sync(0xffffffffu, u1_own, half + mine);
+      const float u2_own = sc.z * (v2 - fmaf(u1s, cross.x, x));                       // right in lanes 4-7
+      float u1[4], u2[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) u1[c] = __shfl_sync(0xffffffffu, u1_own, half + c);
+#pragma unroll
+      for (int c = 0; c < 4; ++c) u2[c] = __shfl_sync(0xffffffffu, u2_own, half + 4 + c);
+      {
+        uint64_t w1[P], w2[P];
+        load_pairs<P>(vec + kW1 * L::kD, rg, w1);
+        load_pairs<P>(vec + kW2 * L::kD, rg, w2);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const uint64_t ua = pack2(u1[c], u1[c]), ub = pack2(u2[c], u2[c]);
+#pragma unroll
+          for (int p = 0; p < P; ++p) S[p][c] = fma2(w2[p], ub, fma2(w1[p], ua, S[p][c]));
         }
       }
-      const float u2s = odd ? b1 : b0;
+      const float u2s = b1 ? (b0 ? u2[3] : u2[2]) : (b0 ? u2[1] : u2[0]);
       const float o = second ? fmaf(u2s, sc.w, fmaf(u1s, cross.y, x)) : fmaf(u1s, sc.y, x);
       const int row = 2 * (i * kTile + t);
       if (writes && row + (second ? 1 : 0) < n) o_dst[static_cast<int64_t>(row) * o_ld] = o;
@@ -700,10 +729,10 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
     return;
   }
 #pragma unroll
-  for (int p = 0; p < 2 * Q; ++p) {
-    const int key = (p >> 1) * 32 + rg * 4 + (p & 1) * 2;
+  for (int p = 0; p < P; ++p) {
+    const int key = pair_row<P>(p, rg);
 #pragma unroll
-    for (int c = 0; c < 2; ++c) {
+    for (int c = 0; c < 4; ++c) {
       if (col + c >= e) continue;
       const float2 f = unpack2(S[p][c]);
       if (key < d) state[static_cast<int64_t>(key) * e + c] = f.x;
@@ -748,12 +777,12 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const B2DeltaArgs a, con
   }
 }
 
-template <int Q>
+template <int P>
 int launch_scan(const B2DeltaArgs& a, const B2SeqRows& s, int first, int n, Status* status, cudaStream_t stream) {
-  using L = ScanLayout<Q>;
+  using L = ScanLayout<P>;
   static DeviceOnce attr_once;
-  if (const int rc = attr_once.max_smem(delta_scan_kernel<Q>, L::kBytes)) return rc;
-  launch_pdl(delta_scan_kernel<Q>, dim3((a.vdim + kCols - 1) / kCols, a.heads, n), dim3(128), L::kBytes, stream, a, s, prepared_of(a, s), first, status);
+  if (const int rc = attr_once.max_smem(delta_scan_kernel<P>, L::kBytes)) return rc;
+  launch_pdl(delta_scan_kernel<P>, dim3((a.vdim + kCols - 1) / kCols, a.heads, n), dim3(128), L::kBytes, stream, a, s, prepared_of(a, s), first, status);
   return last_launch_rc();
 }
 

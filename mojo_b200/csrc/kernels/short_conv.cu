@@ -15,6 +15,7 @@ namespace {
 
 constexpr int kMaxHead = 256;
 constexpr int kWarps = 8;
+constexpr int kSplitTarget = 4;      // CTAs per SM a prompt-sized launch aims at
 
 // A warp's rows: runs of rows of one sequence, each convolved at once (`conv_rows`), then rotated and normalised row by row.
 template <typename T, int VEC, int NJ, int TAPS, int TT>
@@ -135,6 +136,130 @@ __global__ void __launch_bounds__(kWarps * 32, TAPS > 0 && NJ == 1 ? 3 : 1) conv
   }
 }
 
+// The common case (4 taps, head sizes up to 128 and multiples of 4): a warp keeps TT rows' rotary factors in registers and
+// walks over heads; rotation partners come from another lane.
+template <typename T, int TT>
+__global__ void __launch_bounds__(kWarps * 32, 3) conv_qkv_rows_kernel(const B2ConvQkvArgs a, const B2SeqRows sq, Status* status) {
+  ptx::grid_dep_sync();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, e0 = lane * 4;
+  const int n_heads = a.heads + 2 * a.kv_heads, half = a.rot >> 1;
+  const int channels = (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim;
+  const ConvSource<T> src{static_cast<const T*>(a.proj), a.ld, a.conv_w, static_cast<T*>(a.conv_state), a.taps, channels, sq.banks};
+  const bool turns = e0 < a.rot, lo = e0 < half;
+  const int partner = turns ? (lo ? lane + half / 4 : lane - half / 4) : lane;
+  const float inv_dim = 1.0f / static_cast<float>(a.dim);
+  const int row_end = min(sq.rows, static_cast<int>(blockIdx.x + 1) * TT);
+  int run = 0;
+  for (int row0 = blockIdx.x * TT; row0 < row_end; row0 += run) {
+    run = 1;
+    const int seq = sq.row_seq[row0];
+    ConvRow cr;
+    const bool valid = seq >= 0 && B2_ASSERT(status, seq < sq.seqs, kSiteKvIndex, seq, sq.seqs) && cr.load(sq, seq, row0, sq.banks, status);
+    if (valid) run = min(row_end, cr.end) - row0;
+    float cs[TT][4], sn[TT][4];
+    int cell[TT];      // cache row of head 0 (heads of a page lie page_size apart); -1: nothing is cached
+#pragma unroll
+    for (int t = 0; t < TT; ++t) {
+      cell[t] = -1;
+#pragma unroll
+      for (int v = 0; v < 4; ++v) {
+        cs[t][v] = 1.0f;
+        sn[t][v] = 0.0f;
+      }
+      if (!valid || t >= run) continue;
+      if (turns) {
+        int pos = a.positions[row0 + t];
+        if (!B2_ASSERT(status, pos >= 0 && pos < a.max_pos, kSiteKvIndex, pos, a.max_pos)) pos = 0;
+        const float* p = a.cos_sin + static_cast<int64_t>(pos) * a.rot + (lo ? e0 : e0 - half);
+        load_f32<4>(p, cs[t]);
+        load_f32<4>(p + half, sn[t]);
+        if (lo) {
+#pragma unroll
+          for (int v = 0; v < 4; ++v) sn[t][v] = -sn[t][v];
+        }
+      }
+      if (a.kv_heads > 0) {
+        const int64_t slot = a.slots[row0 + t];
+        if (slot >= 0 && B2_ASSERT(status, slot < a.num_slots, kSiteKvIndex, slot, a.num_slots)) {
+          // the host keeps num_slots * kv_heads below 2^31
+          const uint32_t page = static_cast<uint32_t>(slot) / static_cast<uint32_t>(a.page_size);
+          cell[t] = static_cast<int>(page * a.kv_heads * a.page_size + (static_cast<uint32_t>(slot) - page * a.page_size));
+        }
+      }
+    }
+    for (int head = blockIdx.y * kWarps + warp; head < n_heads; head += gridDim.y * kWarps) {
+      const bool is_q = head < a.heads, is_v = head >= a.heads + a.kv_heads;
+      const int kvh = is_q ? 0 : head - a.heads - (is_v ? a.kv_heads : 0);
+      const int dim = is_v ? a.vdim : a.dim, pad = is_v ? a.pad_vdim : a.pad_dim;
+      const int chan0 = is_q ? head * a.dim : is_v ? (a.heads + a.kv_heads) * a.dim + kvh * a.vdim : (a.heads + kvh) * a.dim;
+      float y[TT][4];
+#pragma unroll
+      for (int t = 0; t < TT; ++t)
+#pragma unroll
+        for (int v = 0; v < 4; ++v) y[t][v] = 0.0f;
+      if (valid && e0 < dim) conv_rows<T, 4, 4, TT>(src, cr, row0, run, chan0 + e0, true, y);
+      if (!is_v) {
+        float ss[TT];
+#pragma unroll
+        for (int t = 0; t < TT; ++t) {
+          float other[4];
+          ss[t] = 0.0f;
+#pragma unroll
+          for (int v = 0; v < 4; ++v) other[v] = __shfl_sync(0xffffffffu, y[t][v], partner);
+#pragma unroll
+          for (int v = 0; v < 4; ++v) {
+            y[t][v] = fmaf(y[t][v], cs[t][v], other[v] * sn[t][v]);
+            ss[t] = fmaf(y[t][v], y[t][v], ss[t]);      // 0 past dim
+          }
+        }
+        if constexpr (TT == 4) {
+          warp_sum4(ss);
+        } else {
+#pragma unroll
+          for (int t = 0; t < TT; ++t) ss[t] = warp_sum(ss[t]);
+        }
+#pragma unroll
+        for (int t = 0; t < TT; ++t) {
+          const float r = rsqrtf(ss[t] * inv_dim + a.eps);
+#pragma unroll
+          for (int v = 0; v < 4; ++v) y[t][v] *= r;
+        }
+      }
+      if (is_q) {
+        T* dst = static_cast<T*>(a.q_out) + (static_cast<int64_t>(row0) * a.heads + head) * pad + e0;
+#pragma unroll
+        for (int t = 0; t < TT; ++t) {
+          if (t < run) {
+            if (e0 < pad) store_f32<4>(dst, y[t]);
+            for (int e = 128; e + lane < pad; e += 32) { const float z[1] = {0.0f}; store_f32<1>(dst - e0 + e + lane, z); }
+          }
+          dst += static_cast<int64_t>(a.heads) * pad;
+        }
+      } else if (e0 < dim) {
+        T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache) + static_cast<int64_t>(kvh) * a.page_size * pad + e0;
+#pragma unroll
+        for (int t = 0; t < TT; ++t)
+          if (cell[t] >= 0) store_f32<4>(cache + static_cast<int64_t>(cell[t]) * pad, y[t]);
+      }
+    }
+  }
+}
+
+template <typename T>
+int launch_conv_qkv_rows(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
+  const int groups = (a.heads + 2 * a.kv_heads + kWarps - 1) / kWarps;
+  constexpr int kRows = 4;
+  const int tiles = (s.rows + kRows - 1) / kRows;
+  if (tiles * groups < 2 * kNumSMs) {      // a small step: one row per warp, every group of heads a CTA of its own
+    launch_pdl(conv_qkv_rows_kernel<T, 1>, dim3(s.rows, groups), dim3(kWarps * 32), 0, stream, a, s, status);
+  } else {
+    int split = (kSplitTarget * kNumSMs + tiles - 1) / tiles;
+    if (split > groups) split = groups;
+    launch_pdl(conv_qkv_rows_kernel<T, kRows>, dim3(tiles, split), dim3(kWarps * 32), 0, stream, a, s, status);
+  }
+  return last_launch_rc();
+}
+
 template <typename T, int VEC, int NJ, int TAPS>
 int launch_conv_qkv(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
   const int groups = (a.heads + 2 * a.kv_heads + kWarps - 1) / kWarps;
@@ -153,6 +278,7 @@ int dispatch_conv_qkv(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status
   const int d = kv && a.vdim > a.dim ? a.vdim : a.dim;
   const auto all = [&](int m) { return a.dim % m == 0 && (!kv || (a.vdim % m == 0 && a.pad_vdim % m == 0)) && a.ld % m == 0 && a.pad_dim % m == 0; };
   if (a.taps == 4 && all(4)) {
+    if (d <= 128 && a.rot % 8 == 0) return launch_conv_qkv_rows<T>(a, s, status, stream);
     if (d <= 128) return launch_conv_qkv<T, 4, 1, 4>(a, s, status, stream);
     return launch_conv_qkv<T, 4, 2, 4>(a, s, status, stream);
   }
@@ -173,7 +299,7 @@ extern "C" int b2_conv_qkv(const B2ConvQkvArgs* a, const B2SeqRows* s, int f32, 
   if (a->heads <= 0 || a->kv_heads < 0 || a->dim <= 0 || a->dim > kMaxHead || a->vdim > kMaxHead || a->pad_dim < a->dim || a->rot % 2 != 0 ||
       a->rot > a->dim || a->taps < 1 || (a->taps > 1 && a->conv_state == nullptr) || a->q_out == nullptr || (a->rot > 0 && a->cos_sin == nullptr))
     return -kBadArgument;
-  if (a->kv_heads > 0 && (a->k_cache == nullptr || a->v_cache == nullptr || a->slots == nullptr || a->pad_vdim < a->vdim || a->page_size <= 0 || a->num_slots > 0x7fffffff ||
+  if (a->kv_heads > 0 && (a->k_cache == nullptr || a->v_cache == nullptr || a->slots == nullptr || a->pad_vdim < a->vdim || a->page_size <= 0 || a->num_slots * a->kv_heads > 0x7fffffff ||
                           a->heads % a->kv_heads != 0))
     return -kBadArgument;
   return f32 ? dispatch_conv_qkv<float>(*a, *s, status, stream) : dispatch_conv_qkv<__nv_bfloat16>(*a, *s, status, stream);
