@@ -16,6 +16,19 @@ _err: Exception | None = None
 _lib = None
 
 
+class _CoreBuild:
+    """A build without the kernels of every model: what is missing says how to get it."""
+
+    def __init__(self, mod):
+        self._mod = mod
+
+    def __getattr__(self, name):
+        try:
+            return getattr(self._mod, name)
+        except AttributeError:
+            raise ImportError(f"mojo_b200 was built without {name!r} (core build); run `python -m mojo_b200.build` in the source tree") from None
+
+
 def _load():
     global _C, _err
     if _C is not None or _err is not None:
@@ -23,7 +36,8 @@ def _load():
     try:
         import torch  # noqa: F401  (libtorch must be loaded before the extension)
 
-        _C = importlib.import_module("mojo_b200._C")
+        mod = importlib.import_module("mojo_b200._C")
+        _C = mod if hasattr(mod, "gemm_fp8") else _CoreBuild(mod)
     except Exception as e:  # noqa: BLE001
         _err = e
 

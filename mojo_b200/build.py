@@ -27,6 +27,11 @@ CSRC = ROOT / "csrc"
 OBJ = ROOT / "csrc" / "build"
 LIBDIR = ROOT / "lib"
 
+# What a model on one GPU needs in bf16 or f32; the rest (fp8, GGUF, MLA, tensor and expert parallelism, examples) comes with
+# a full build. Both link under the same names; `lib/BUILD` says which one is there.
+CORE_KERNELS = {"attention", "attention_tc", "delta_rule", "elementwise", "f32_ops", "gemm_bf16", "gemm_bf16_pair", "hyper_conn", "sampling", "short_conv"}
+CORE_BINDINGS = {"engine_bind", "io_bind", "mixers_bind", "ops_bind"}
+
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 
 
@@ -64,7 +69,9 @@ def _run(cmd: list[str], verbose: bool) -> str:
     return p.stdout + p.stderr
 
 
-def build(verbose: bool = False, assert_mode: int = 2, ptxas_info: bool = False, jobs: int | None = None) -> None:
+def build(verbose: bool = False, assert_mode: int = 2, ptxas_info: bool = False, jobs: int | None = None,
+          core: bool = False) -> None:
+    """`core`: only the kernels and bindings of CORE_KERNELS / CORE_BINDINGS."""
     t0 = time.time()
     OBJ.mkdir(parents=True, exist_ok=True)
     LIBDIR.mkdir(parents=True, exist_ok=True)
@@ -73,7 +80,9 @@ def build(verbose: bool = False, assert_mode: int = 2, ptxas_info: bool = False,
     cuda_inc = ["-I", str(_cuda_home() / "include")]
     defs = [f"-DB2_ASSERT_MODE={assert_mode}"]
 
-    cu_srcs = sorted((CSRC / "kernels").glob("*.cu"))
+    marker, kind = LIBDIR / "BUILD", "core" if core else "all"
+    relink = not marker.exists() or marker.read_text() != kind
+    cu_srcs = [s for s in sorted((CSRC / "kernels").glob("*.cu")) if not core or s.stem in CORE_KERNELS]
     cpp_srcs = sorted((CSRC / "runtime").glob("*.cpp"))
     tasks = []
     objs = []
@@ -101,7 +110,7 @@ def build(verbose: bool = False, assert_mode: int = 2, ptxas_info: bool = False,
         print("".join(outputs))
 
     lib = LIBDIR / "libb2kernels.so"
-    if tasks or not lib.exists():
+    if tasks or relink or not lib.exists():
         _run([_nvcc(), *NVCC_ARCH, "-shared", "-o", str(lib), *[str(o) for o in objs], "-lcudart", "-ldl", "-lpthread"], verbose)
 
     # ---- PyTorch bindings ----
@@ -110,7 +119,7 @@ def build(verbose: bool = False, assert_mode: int = 2, ptxas_info: bool = False,
 
     ext_suffix = sysconfig.get_config_var("EXT_SUFFIX")
     mod = ROOT / f"_C{ext_suffix}"
-    b_srcs = sorted((CSRC / "bindings").glob("*.cpp"))
+    b_srcs = [s for s in sorted((CSRC / "bindings").glob("*.cpp")) if not core or s.stem in CORE_BINDINGS]
     b_objs = []
     b_tasks = []
     torch_inc = []
@@ -119,20 +128,22 @@ def build(verbose: bool = False, assert_mode: int = 2, ptxas_info: bool = False,
     py_inc = ["-isystem", sysconfig.get_paths()["include"]]
     abi = int(torch._C._GLIBCXX_USE_CXX11_ABI)
     for s in b_srcs:
-        o = OBJ / (s.stem + ".bind.o")
+        core_main = core and s.stem == "ops_bind"       # the module's entry point names the bindings it registers
+        o = OBJ / (s.stem + (".core" if core_main else "") + ".bind.o")
         b_objs.append(o)
         if _needs(o, s, hdr_m):
-            b_tasks.append(["g++", "-O2", "-std=c++17", "-fPIC", "-Wno-unused-variable", *defs, *inc, *cuda_inc, *torch_inc, *py_inc,
+            b_tasks.append(["g++", "-O2", "-std=c++17", "-fPIC", "-Wno-unused-variable", *defs, *(["-DB2_CORE_ONLY"] if core_main else []), *inc, *cuda_inc, *torch_inc, *py_inc,
                             f"-D_GLIBCXX_USE_CXX11_ABI={abi}", "-DTORCH_EXTENSION_NAME=_C", "-DTORCH_API_INCLUDE_EXTENSION_H",
                             "-c", str(s), "-o", str(o)])
     with cf.ThreadPoolExecutor(max_workers=jobs) as ex:
         list(ex.map(lambda c: _run(c, verbose), b_tasks))
-    if b_tasks or tasks or not mod.exists():
+    if b_tasks or tasks or relink or not mod.exists():
         torch_lib = Path(torch.__file__).parent / "lib"
         _run(["g++", "-shared", "-o", str(mod), *[str(o) for o in b_objs], f"-L{LIBDIR}", "-lb2kernels",
               f"-L{torch_lib}", "-lc10", "-ltorch_cpu", "-ltorch", "-ltorch_python", "-lc10_cuda", "-ltorch_cuda",
               f"-L{_cuda_home() / 'lib64'}", "-lcudart",
               "-Wl,-rpath,$ORIGIN/lib", f"-Wl,-rpath,{torch_lib}", f"-Wl,-rpath,{_cuda_home() / 'lib64'}"], verbose)
+    marker.write_text(kind)
     if verbose or tasks or b_tasks:
         print(f"[mojo_b200.build] {len(tasks)} kernel/runtime objects, {len(b_tasks)} binding objects rebuilt in {time.time() - t0:.1f}s")
 
@@ -158,6 +169,7 @@ def main() -> None:
     ap.add_argument("-v", "--verbose", action="store_true")
     ap.add_argument("--assert-mode", type=int, default=2, help="0 none, 1 warn, 2 safe, 3 all")
     ap.add_argument("--ptxas-info", action="store_true", help="print registers / spills / smem per kernel")
+    ap.add_argument("--core", action="store_true", help="only what a model on one GPU needs in bf16 or f32")
     ap.add_argument("--clean", action="store_true")
     ap.add_argument("--selftest", choices=["address", "thread", "plain"], default=None,
                     help="build the host runtime self-test under this sanitizer, run it and exit with its code")
@@ -167,7 +179,7 @@ def main() -> None:
         sys.exit(subprocess.run([str(exe)]).returncode)
     if a.clean and OBJ.exists():
         shutil.rmtree(OBJ)
-    build(verbose=a.verbose, assert_mode=a.assert_mode, ptxas_info=a.ptxas_info)
+    build(verbose=a.verbose, assert_mode=a.assert_mode, ptxas_info=a.ptxas_info, core=a.core)
 
 
 if __name__ == "__main__":

@@ -358,8 +358,10 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("gemm_workspace_bytes", [](int M, int N, int K) { return b2_gemm_workspace_bytes(M, N, K); });
   m.def("attn_decode_workspace_bytes", [](int batch, int n_q, int d, int splits) { return b2_attn_decode_workspace(batch, n_q, d, splits); });
   m.def("device_caps", &device_caps, py::arg("device") = 0);
+#ifndef B2_CORE_ONLY
   bind_ops_extra(m);
   bind_coll(m);
+#endif
   bind_mixers(m);
   bind_io(m);
 }

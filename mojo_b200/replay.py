@@ -24,7 +24,7 @@ TOKEN_UNIT = 64        # a request's share of --max-tokens is counted in units o
 
 
 def ensure_built() -> None:
-    """Build the native extension if this checkout has none (one builder at a time)."""
+    """Build what the models replayed here need if this checkout has no native extension (one builder at a time)."""
     from . import _ext, build
 
     if _ext.built():
@@ -34,7 +34,7 @@ def ensure_built() -> None:
     with open(build.ROOT / ".build.lock", "w") as lock:
         fcntl.flock(lock, fcntl.LOCK_EX)
         if not _ext.built():
-            build.build()
+            build.build(core=True)
 
 
 def open_engine(model: str, dtype: str, max_tokens: int, device: str | None = None):
