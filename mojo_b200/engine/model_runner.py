@@ -85,7 +85,7 @@ class ModelRunner:
         max_blocks = (cfg.max_model_len + cfg.page_size - 1) // cfg.page_size
         # models with recurrent state also need the sequence of every row, and rows and state banks of every sequence
         self.has_state = bool(getattr(model, "recurrent_state", False))
-        nbytes = cfg.max_num_batched_tokens * 28 + cfg.max_num_seqs * (max_blocks * 4 + 96) + (1 << 16)
+        nbytes = cfg.max_num_batched_tokens * 36 + cfg.max_num_seqs * (max_blocks * 4 + 96) + (1 << 16)
         self.staging = _Staging(nbytes, self.device)
         self.max_blocks = max_blocks
         self.h2d_bytes = 0
