@@ -97,7 +97,7 @@ int launch_hyper(const B2HyperArgs& a, Status* status, cudaStream_t stream) {
   if (smem > 40 * 1024)
     if (const int rc = attr_once.max_smem(hyper_norm_kernel<T, S, VEC>, 200 * 1024)) return rc;
   const int vecs = (a.width + VEC - 1) / VEC;
-  const int threads = vecs >= 1024 ? 512 : vecs >= 256 ? 256 : (vecs + 31) / 32 * 32;
+  const int threads = vecs >= 256 ? 256 : (vecs + 31) / 32 * 32;      // more threads per row would leave one row per SM
   launch_pdl(hyper_norm_kernel<T, S, VEC>, dim3(a.n_out), dim3(threads), smem, stream, a, status);
   return last_launch_rc();
 }

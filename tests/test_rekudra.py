@@ -283,7 +283,7 @@ def seq_rows(lengths, banks, device, order=None):
 
 
 @pytest.mark.parametrize("target", TARGETS)
-@pytest.mark.parametrize("streams,width", [(1, 64), (2, 20), (3, 192), (4, 1000), (7, 96), (8, 2048)])
+@pytest.mark.parametrize("streams,width", [(1, 64), (2, 20), (3, 160), (4, 1000), (7, 96), (8, 2048)])
 def test_hyper_connections(target, streams, width):
     g = torch.Generator().manual_seed(streams)
 
