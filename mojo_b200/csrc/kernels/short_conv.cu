@@ -15,7 +15,6 @@ namespace {
 
 constexpr int kMaxHead = 256;
 constexpr int kWarps = 8;
-constexpr int kSplitTarget = 4;      // CTAs per SM a prompt-sized launch aims at
 
 // A warp's rows: runs of rows of one sequence, each convolved at once (`conv_rows`), then rotated and normalised row by row.
 template <typename T, int VEC, int NJ, int TAPS, int TT>
@@ -136,28 +135,18 @@ __global__ void __launch_bounds__(kWarps * 32, TAPS > 0 && NJ == 1 ? 3 : 1) conv
   }
 }
 
-// The common case (4 taps, head sizes up to 128 and multiples of 4): a warp keeps TT rows' rotary factors in registers and
-// walks over heads; rotation partners come from another lane.
-template <typename T, int TT>
-__global__ void __launch_bounds__(kWarps * 32, 3) conv_qkv_rows_kernel(const B2ConvQkvArgs a, const B2SeqRows sq, Status* status) {
-  ptx::grid_dep_sync();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, e0 = lane * 4;
-  const int n_heads = a.heads + 2 * a.kv_heads, half = a.rot >> 1;
-  const int channels = (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim;
-  const ConvSource<T> src{static_cast<const T*>(a.proj), a.ld, a.conv_w, static_cast<T*>(a.conv_state), a.taps, channels, sq.banks};
-  const bool turns = e0 < a.rot, lo = e0 < half;
-  const int partner = turns ? (lo ? lane + half / 4 : lane - half / 4) : lane;
-  const float inv_dim = 1.0f / static_cast<float>(a.dim);
-  const int row_end = min(sq.rows, static_cast<int>(blockIdx.x + 1) * TT);
-  int run = 0;
-  for (int row0 = blockIdx.x * TT; row0 < row_end; row0 += run) {
-    run = 1;
-    const int seq = sq.row_seq[row0];
-    ConvRow cr;
-    const bool valid = seq >= 0 && B2_ASSERT(status, seq < sq.seqs, kSiteKvIndex, seq, sq.seqs) && cr.load(sq, seq, row0, sq.banks, status);
-    if (valid) run = min(row_end, cr.end) - row0;
-    float cs[TT][4], sn[TT][4];
-    int cell[TT];      // cache row of head 0 (heads of a page lie page_size apart); -1: nothing is cached
+// The common case (4 taps, head sizes up to 128 and multiples of 4). Work unit = (tile of TT rows, head); every warp takes
+// the same number of consecutive units, heads first, so that it keeps a tile's rotary factors in registers across heads.
+// Rotation partners come from another lane. Tiles that cross a sequence border go row by row.
+struct RowLane {
+  int lane, e0, half, partner;
+  bool turns, lo;
+};
+template <int TT>
+struct RowFactors {
+  float cs[TT][4], sn[TT][4];
+  int cell[TT];      // cache row of head 0 (heads of a page lie page_size apart); -1: nothing is cached
+  __device__ __forceinline__ void load(const B2ConvQkvArgs& a, const RowLane& l, int row0, int n, bool valid, Status* status) {
 #pragma unroll
     for (int t = 0; t < TT; ++t) {
       cell[t] = -1;
@@ -166,14 +155,14 @@ __global__ void __launch_bounds__(kWarps * 32, 3) conv_qkv_rows_kernel(const B2C
         cs[t][v] = 1.0f;
         sn[t][v] = 0.0f;
       }
-      if (!valid || t >= run) continue;
-      if (turns) {
+      if (!valid || t >= n) continue;
+      if (l.turns) {
         int pos = a.positions[row0 + t];
         if (!B2_ASSERT(status, pos >= 0 && pos < a.max_pos, kSiteKvIndex, pos, a.max_pos)) pos = 0;
-        const float* p = a.cos_sin + static_cast<int64_t>(pos) * a.rot + (lo ? e0 : e0 - half);
+        const float* p = a.cos_sin + static_cast<int64_t>(pos) * a.rot + (l.lo ? l.e0 : l.e0 - l.half);
         load_f32<4>(p, cs[t]);
-        load_f32<4>(p + half, sn[t]);
-        if (lo) {
+        load_f32<4>(p + l.half, sn[t]);
+        if (l.lo) {
 #pragma unroll
           for (int v = 0; v < 4; ++v) sn[t][v] = -sn[t][v];
         }
@@ -187,59 +176,106 @@ __global__ void __launch_bounds__(kWarps * 32, 3) conv_qkv_rows_kernel(const B2C
         }
       }
     }
-    for (int head = blockIdx.y * kWarps + warp; head < n_heads; head += gridDim.y * kWarps) {
-      const bool is_q = head < a.heads, is_v = head >= a.heads + a.kv_heads;
-      const int kvh = is_q ? 0 : head - a.heads - (is_v ? a.kv_heads : 0);
-      const int dim = is_v ? a.vdim : a.dim, pad = is_v ? a.pad_vdim : a.pad_dim;
-      const int chan0 = is_q ? head * a.dim : is_v ? (a.heads + a.kv_heads) * a.dim + kvh * a.vdim : (a.heads + kvh) * a.dim;
-      float y[TT][4];
+  }
+};
+
+// `n` rows from row0 (all of one sequence; valid == false: one padding row) of one head.
+template <typename T, int TT>
+__device__ __forceinline__ void conv_head(const B2ConvQkvArgs& a, const ConvSource<T>& src, const ConvRow& cr, bool valid, int row0, int n, int head,
+                                          const RowLane& l, const RowFactors<TT>& f) {
+  const bool is_q = head < a.heads, is_v = head >= a.heads + a.kv_heads;
+  const int kvh = is_q ? 0 : head - a.heads - (is_v ? a.kv_heads : 0);
+  const int dim = is_v ? a.vdim : a.dim, pad = is_v ? a.pad_vdim : a.pad_dim;
+  const int chan0 = is_q ? head * a.dim : is_v ? (a.heads + a.kv_heads) * a.dim + kvh * a.vdim : (a.heads + kvh) * a.dim;
+  float y[TT][4];
 #pragma unroll
-      for (int t = 0; t < TT; ++t)
+  for (int t = 0; t < TT; ++t)
 #pragma unroll
-        for (int v = 0; v < 4; ++v) y[t][v] = 0.0f;
-      if (valid && e0 < dim) conv_rows<T, 4, 4, TT>(src, cr, row0, run, chan0 + e0, true, y);
-      if (!is_v) {
-        float ss[TT];
+    for (int v = 0; v < 4; ++v) y[t][v] = 0.0f;
+  if (valid && l.e0 < dim) conv_rows<T, 4, 4, TT>(src, cr, row0, n, chan0 + l.e0, true, y);
+  if (!is_v) {
+    float ss[TT];
 #pragma unroll
-        for (int t = 0; t < TT; ++t) {
-          float other[4];
-          ss[t] = 0.0f;
+    for (int t = 0; t < TT; ++t) {
+      float other[4];
+      ss[t] = 0.0f;
 #pragma unroll
-          for (int v = 0; v < 4; ++v) other[v] = __shfl_sync(0xffffffffu, y[t][v], partner);
+      for (int v = 0; v < 4; ++v) other[v] = __shfl_sync(0xffffffffu, y[t][v], l.partner);
 #pragma unroll
-          for (int v = 0; v < 4; ++v) {
-            y[t][v] = fmaf(y[t][v], cs[t][v], other[v] * sn[t][v]);
-            ss[t] = fmaf(y[t][v], y[t][v], ss[t]);      // 0 past dim
-          }
-        }
-        if constexpr (TT == 4) {
-          warp_sum4(ss);
-        } else {
-#pragma unroll
-          for (int t = 0; t < TT; ++t) ss[t] = warp_sum(ss[t]);
-        }
-#pragma unroll
-        for (int t = 0; t < TT; ++t) {
-          const float r = rsqrtf(ss[t] * inv_dim + a.eps);
-#pragma unroll
-          for (int v = 0; v < 4; ++v) y[t][v] *= r;
-        }
+      for (int v = 0; v < 4; ++v) {
+        y[t][v] = fmaf(y[t][v], f.cs[t][v], other[v] * f.sn[t][v]);
+        ss[t] = fmaf(y[t][v], y[t][v], ss[t]);      // 0 past dim
       }
-      if (is_q) {
-        T* dst = static_cast<T*>(a.q_out) + (static_cast<int64_t>(row0) * a.heads + head) * pad + e0;
+    }
+    if constexpr (TT == 4) {
+      warp_sum4(ss);
+    } else {
 #pragma unroll
-        for (int t = 0; t < TT; ++t) {
-          if (t < run) {
-            if (e0 < pad) store_f32<4>(dst, y[t]);
-            for (int e = 128; e + lane < pad; e += 32) { const float z[1] = {0.0f}; store_f32<1>(dst - e0 + e + lane, z); }
-          }
-          dst += static_cast<int64_t>(a.heads) * pad;
-        }
-      } else if (e0 < dim) {
-        T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache) + static_cast<int64_t>(kvh) * a.page_size * pad + e0;
+      for (int t = 0; t < TT; ++t) ss[t] = warp_sum(ss[t]);
+    }
+    const float inv_dim = 1.0f / static_cast<float>(a.dim);
 #pragma unroll
-        for (int t = 0; t < TT; ++t)
-          if (cell[t] >= 0) store_f32<4>(cache + static_cast<int64_t>(cell[t]) * pad, y[t]);
+    for (int t = 0; t < TT; ++t) {
+      const float r = rsqrtf(ss[t] * inv_dim + a.eps);
+#pragma unroll
+      for (int v = 0; v < 4; ++v) y[t][v] *= r;
+    }
+  }
+  if (is_q) {
+    T* dst = static_cast<T*>(a.q_out) + (static_cast<int64_t>(row0) * a.heads + head) * pad + l.e0;
+#pragma unroll
+    for (int t = 0; t < TT; ++t) {
+      if (t < n) {
+        if (l.e0 < pad) store_f32<4>(dst, y[t]);
+        for (int e = 128; e + l.lane < pad; e += 32) { const float z[1] = {0.0f}; store_f32<1>(dst - l.e0 + e + l.lane, z); }
+      }
+      dst += static_cast<int64_t>(a.heads) * pad;
+    }
+  } else if (l.e0 < dim) {
+    T* cache = static_cast<T*>(is_v ? a.v_cache : a.k_cache) + static_cast<int64_t>(kvh) * a.page_size * pad + l.e0;
+#pragma unroll
+    for (int t = 0; t < TT; ++t)
+      if (f.cell[t] >= 0) store_f32<4>(cache + static_cast<int64_t>(f.cell[t]) * pad, y[t]);
+  }
+}
+
+template <typename T, int TT>
+__global__ void __launch_bounds__(kWarps * 32, 3) conv_qkv_rows_kernel(const B2ConvQkvArgs a, const B2SeqRows sq, Status* status) {
+  ptx::grid_dep_sync();
+  const int n_heads = a.heads + 2 * a.kv_heads;
+  const int channels = (a.heads + a.kv_heads) * a.dim + a.kv_heads * a.vdim;
+  const ConvSource<T> src{static_cast<const T*>(a.proj), a.ld, a.conv_w, static_cast<T*>(a.conv_state), a.taps, channels, sq.banks};
+  RowLane l;
+  l.lane = threadIdx.x & 31;
+  l.e0 = l.lane * 4;
+  l.half = a.rot >> 1;
+  l.turns = l.e0 < a.rot;
+  l.lo = l.e0 < l.half;
+  l.partner = l.turns ? (l.lo ? l.lane + l.half / 4 : l.lane - l.half / 4) : l.lane;
+  const int64_t units = static_cast<int64_t>((sq.rows + TT - 1) / TT) * n_heads;
+  const int64_t w = static_cast<int64_t>(blockIdx.x) * kWarps + (threadIdx.x >> 5), n_warps = static_cast<int64_t>(gridDim.x) * kWarps;
+  int64_t left = units * (w + 1) / n_warps - units * w / n_warps;
+  int tile = static_cast<int>(units * w / n_warps / n_heads), head = static_cast<int>(units * w / n_warps % n_heads);
+  const auto place = [&](int row, ConvRow& cr) {
+    const int seq = sq.row_seq[row];
+    return seq >= 0 && B2_ASSERT(status, seq < sq.seqs, kSiteKvIndex, seq, sq.seqs) && cr.load(sq, seq, row, sq.banks, status);
+  };
+  for (; left > 0; ++tile, head = 0) {
+    const int row0 = tile * TT, rows = min(TT, sq.rows - row0);
+    const int stop = head + static_cast<int>(min(left, static_cast<int64_t>(n_heads - head)));      // this warp's heads of the tile
+    left -= stop - head;
+    ConvRow cr;
+    const bool valid = place(row0, cr);
+    if (TT == 1 || (valid && cr.end - row0 >= rows)) {
+      RowFactors<TT> f;
+      f.load(a, l, row0, rows, valid, status);
+      for (; head < stop; ++head) conv_head<T, TT>(a, src, cr, valid, row0, rows, head, l, f);
+    } else {
+      for (int r = row0; r < row0 + rows; ++r) {
+        const bool ok = place(r, cr);
+        RowFactors<1> f;
+        f.load(a, l, r, 1, ok, status);
+        for (int h = head; h < stop; ++h) conv_head<T, 1>(a, src, cr, ok, r, 1, h, l, f);
       }
     }
   }
@@ -247,16 +283,12 @@ __global__ void __launch_bounds__(kWarps * 32, 3) conv_qkv_rows_kernel(const B2C
 
 template <typename T>
 int launch_conv_qkv_rows(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
-  const int groups = (a.heads + 2 * a.kv_heads + kWarps - 1) / kWarps;
-  constexpr int kRows = 4;
-  const int tiles = (s.rows + kRows - 1) / kRows;
-  if (tiles * groups < 2 * kNumSMs) {      // a small step: one row per warp, every group of heads a CTA of its own
-    launch_pdl(conv_qkv_rows_kernel<T, 1>, dim3(s.rows, groups), dim3(kWarps * 32), 0, stream, a, s, status);
-  } else {
-    int split = (kSplitTarget * kNumSMs + tiles - 1) / tiles;
-    if (split > groups) split = groups;
-    launch_pdl(conv_qkv_rows_kernel<T, kRows>, dim3(tiles, split), dim3(kWarps * 32), 0, stream, a, s, status);
-  }
+  const int n_heads = a.heads + 2 * a.kv_heads;
+  const bool small = static_cast<int64_t>((s.rows + 3) / 4) * n_heads < 2 * kNumSMs * kWarps;      // one row at a time then
+  const int64_t units = static_cast<int64_t>(small ? s.rows : (s.rows + 3) / 4) * n_heads, ctas = (units + kWarps - 1) / kWarps;
+  const int grid = static_cast<int>(ctas < 3 * kNumSMs ? ctas : 3 * kNumSMs);
+  if (small) launch_pdl(conv_qkv_rows_kernel<T, 1>, dim3(grid), dim3(kWarps * 32), 0, stream, a, s, status);
+  else launch_pdl(conv_qkv_rows_kernel<T, 4>, dim3(grid), dim3(kWarps * 32), 0, stream, a, s, status);
   return last_launch_rc();
 }
 
