@@ -118,6 +118,7 @@ void bind_engine(py::module_& m) {
       .def_property_readonly("cu_q", [](const Batch& b) { return to_array(b.cu_q); })
       .def_property_readonly("token_ids", [](const Batch& b) { return to_array(b.token_ids); })
       .def_property_readonly("positions", [](const Batch& b) { return to_array(b.positions); })
+      .def_property_readonly("prev_tokens", [](const Batch& b) { return to_array(b.prev_tokens); })
       .def_property_readonly("slots", [](const Batch& b) { return to_array(b.slots); })
       .def_property_readonly("block_tables",
                              [](const Batch& b) {

@@ -181,13 +181,92 @@ void delta_rule(const at::Tensor& proj, const at::Tensor& dg, const at::Tensor& 
         "delta_rule");
 }
 
-void gemm_f32(const at::Tensor& x, const at::Tensor& w, at::Tensor& y) {
+void gemm_f32(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, int64_t batch, int64_t epilogue, double cap, const OptTensor& gate) {
   for (const at::Tensor* t : {&x, &w, static_cast<const at::Tensor*>(&y)})
     need(t->is_cuda() && t->scalar_type() == at::kFloat && t->dim() == 2 && t->stride(1) == 1, "gemm_f32: 2-D CUDA f32 with unit inner strides");
-  need(x.size(1) == w.size(1) && y.size(0) == x.size(0) && y.size(1) == w.size(0), "gemm_f32: x [M, K], w [N, K], y [M, N]");
+  const int64_t K = w.size(1);
+  need(batch >= 1 && w.size(0) % batch == 0 && x.size(1) == batch * K && y.size(0) == x.size(0) && y.size(1) == w.size(0),
+       "gemm_f32: x [M, batch * K], w [batch * N, K], y [M, batch * N]");
+  if (gate.has_value())
+    need(gate->is_cuda() && gate->scalar_type() == at::kFloat && gate->dim() == 2 && gate->stride(1) == 1 && gate->sizes() == y.sizes(), "gemm_f32: gate f32 like y");
+  B2GemmF32Args a{};
+  a.x = x.data_ptr<float>();
+  a.w = w.data_ptr<float>();
+  a.y = y.data_ptr<float>();
+  a.gate = opt<const float>(gate);
+  a.ldx = x.stride(0);
+  a.ldw = w.stride(0);
+  a.ldy = y.stride(0);
+  a.ld_gate = gate.has_value() ? gate->stride(0) : 0;
+  a.cap = static_cast<float>(cap);
+  a.M = static_cast<int32_t>(x.size(0));
+  a.N = static_cast<int32_t>(w.size(0) / batch);
+  a.K = static_cast<int32_t>(K);
+  a.batch = static_cast<int32_t>(batch);
+  a.epilogue = static_cast<int32_t>(epilogue);
   c10::cuda::CUDAGuard g(x.device());
-  check(b2_gemm_f32(x.data_ptr<float>(), w.data_ptr<float>(), y.data_ptr<float>(), static_cast<int>(x.size(0)), static_cast<int>(w.size(0)),
-                    static_cast<int>(x.size(1)), x.stride(0), w.stride(0), y.stride(0), cur_stream()), "gemm_f32");
+  check(b2_gemm_f32(&a, cur_stream()), "gemm_f32");
+}
+
+void residual_norm(at::Tensor& x, const OptTensor& y, const OptTensor& experts, const OptTensor& slot, const OptTensor& expert_w, const OptTensor& y_scale,
+                   const OptTensor& weight, at::Tensor& h, const OptTensor& ids, const OptTensor& embed, double embed_scale, const OptTensor& prev,
+                   const OptTensor& bigram, int64_t mul_prev, int64_t mul_cur, const OptTensor& x0, const OptTensor& rows_index, bool store, double eps,
+                   int64_t mean_width, const OptTensor& status) {
+  need(x.dim() == 2 && x.is_cuda() && x.scalar_type() == at::kFloat && x.is_contiguous(), "residual_norm: x must be contiguous CUDA f32 [rows, width]");
+  const int64_t T = x.size(0), W = x.size(1);
+  need(is_act(h) && h.dim() == 2 && h.stride(1) == 1 && h.size(1) == W, "residual_norm: h [n, width]");
+  B2ResidualArgs a{};
+  if (y.has_value()) need(y->scalar_type() == h.scalar_type() && y->is_contiguous() && y->numel() == T * W, "residual_norm: y [rows, width] like h");
+  if (y.has_value() || experts.has_value()) need(y_scale.has_value() && is_f32(*y_scale, W), "residual_norm: y_scale f32 [width]");
+  if (weight.has_value()) need(is_f32(*weight, W), "residual_norm: weight f32 [width]");
+  if (experts.has_value()) {
+    need(experts->scalar_type() == h.scalar_type() && experts->dim() == 2 && experts->is_contiguous() && experts->size(1) == W && slot.has_value() &&
+             is_i32(*slot) && slot->dim() == 2 && slot->size(0) == T && expert_w.has_value() && is_f32(*expert_w, slot->numel()),
+         "residual_norm: expert rows [n, width] like h, slots int32 and weights f32 [rows, top]");
+    a.top = static_cast<int32_t>(slot->size(1));
+    a.expert_rows = static_cast<int32_t>(experts->size(0));
+  }
+  if (ids.has_value())
+    need(is_i64(*ids) && ids->numel() == T && embed.has_value() && embed->scalar_type() == h.scalar_type() && embed->is_contiguous() && embed->size(1) == W,
+         "residual_norm: ids int64 [rows], embed [vocab, width] like h");
+  if (bigram.has_value()) {
+    need(ids.has_value() && prev.has_value() && is_i32(*prev) && prev->numel() == T && bigram->scalar_type() == h.scalar_type() && bigram->is_contiguous() &&
+             bigram->dim() == 2 && bigram->size(1) == W && bigram->size(0) >= 2, "residual_norm: prev int32 [rows], bigram [buckets + 1, width] like h");
+    a.buckets = bigram->size(0) - 1;
+  }
+  if (x0.has_value()) {
+    need(x0->scalar_type() == h.scalar_type() && x0->dim() == 2 && x0->stride(1) == 1 && x0->size(0) == T && x0->size(1) == W, "residual_norm: x0 [rows, width] like h");
+    a.ld_x0 = x0->stride(0);
+  }
+  if (rows_index.has_value()) need(is_i64(*rows_index) && rows_index->numel() == h.size(0), "residual_norm: rows_index int64 [n]");
+  else need(h.size(0) == T, "residual_norm: h must have one row per x row");
+  a.x = x.data_ptr<float>();
+  a.y = opt<const void>(y);
+  a.experts = opt<const void>(experts);
+  a.expert_slot = opt<const int32_t>(slot);
+  a.expert_w = opt<const float>(expert_w);
+  a.y_scale = opt<const float>(y_scale);
+  a.weight = opt<const float>(weight);
+  a.h = h.data_ptr();
+  a.ids = opt<const int64_t>(ids);
+  a.embed = opt<const void>(embed);
+  a.prev = opt<const int32_t>(prev);
+  a.bigram = opt<const void>(bigram);
+  a.x0 = opt<void>(x0);
+  a.rows_index = opt<const int64_t>(rows_index);
+  a.ld_h = h.stride(0);
+  a.mul_prev = mul_prev;
+  a.mul_cur = mul_cur;
+  a.embed_scale = static_cast<float>(embed_scale);
+  a.eps = static_cast<float>(eps);
+  a.n_out = static_cast<int32_t>(h.size(0));
+  a.rows = static_cast<int32_t>(T);
+  a.width = static_cast<int32_t>(W);
+  a.mean_width = static_cast<int32_t>(mean_width);
+  a.vocab = embed.has_value() ? static_cast<int32_t>(embed->size(0)) : 0;
+  a.store = store ? 1 : 0;
+  c10::cuda::CUDAGuard g(x.device());
+  check(b2_residual_norm(&a, h.scalar_type() == at::kFloat ? 1 : 0, status_ptr(status), cur_stream()), "residual_norm");
 }
 
 void attn_f32(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out, const at::Tensor& row_seq,
@@ -218,13 +297,16 @@ void bind_mixers(py::module_& m) {
   m.def("delta_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows, int64_t seqs) {
     return b2_delta_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows), static_cast<int>(seqs));
   });
-  m.def("gemm_f32", &gemm_f32);
+  m.def("residual_norm", &residual_norm);
+  m.def("gemm_f32", &gemm_f32, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("batch") = 1, py::arg("epilogue") = 0, py::arg("cap") = 0.0,
+        py::arg("gate") = py::none());
   m.def("attn_f32", &attn_f32);
-  m.def("swiglu_f32", [](const at::Tensor& gu, at::Tensor& out) {
+  m.def("glu_f32", [](const at::Tensor& gu, at::Tensor& out, double limit, double alpha, double up_bias) {
     need(gu.is_cuda() && gu.scalar_type() == at::kFloat && gu.is_contiguous() && out.is_contiguous() && out.scalar_type() == at::kFloat &&
-             gu.size(0) == out.size(0) && gu.size(1) == 2 * out.size(1), "swiglu_f32: gate_up [M, 2F], out [M, F], contiguous CUDA f32");
+             gu.size(0) == out.size(0) && gu.size(1) == 2 * out.size(1), "glu_f32: gate_up [M, 2F], out [M, F], contiguous CUDA f32");
+    const B2EpiAct act{static_cast<float>(limit), static_cast<float>(alpha), static_cast<float>(up_bias), 0.0f};
     c10::cuda::CUDAGuard g(gu.device());
-    check(b2_swiglu_f32(gu.data_ptr<float>(), out.data_ptr<float>(), static_cast<int>(out.size(0)), static_cast<int>(out.size(1)), cur_stream()), "swiglu_f32");
+    check(b2_glu_f32(gu.data_ptr<float>(), out.data_ptr<float>(), out.size(0), static_cast<int>(out.size(1)), &act, cur_stream()), "glu_f32");
   });
   m.def("gather_rows_f32", [](const at::Tensor& src, const at::Tensor& index, at::Tensor& out, const OptTensor& status) {
     need(src.is_cuda() && src.scalar_type() == at::kFloat && src.is_contiguous() && src.dim() == 2 && out.is_contiguous() && out.scalar_type() == at::kFloat &&

@@ -1,5 +1,7 @@
 // PyTorch bindings: thin argument checking around the C launch API (b2/api.h). Tensors are passed through as
 // raw pointers on the current CUDA stream; nothing here allocates.
+#include <array>
+#include <cmath>
 #include <torch/extension.h>
 #include <c10/cuda/CUDAStream.h>
 #include <c10/cuda/CUDAGuard.h>
@@ -184,7 +186,7 @@ void check_cache(const at::Tensor& q, const at::Tensor& k_cache, const at::Tenso
   need(k_cache.size(3) == head_dim && v_cache.sizes() == k_cache.sizes(), "attention: cache geometry mismatch");
 }
 
-// Optional per-head output gate: bf16 [T, n_q] logits with unit inner stride.
+// Optional output gate: bf16 [T, n_q] logits with unit inner stride (n_q: heads, or output elements).
 const void* gate_ptr(const c10::optional<at::Tensor>& gate, const at::Tensor& q, int64_t n_q) {
   if (!gate.has_value()) return nullptr;
   need(gate->is_cuda() && is_bf16(*gate) && gate->dim() == 2 && gate->size(0) == q.size(0) && gate->size(1) == n_q && gate->stride(1) == 1,
@@ -212,22 +214,38 @@ void attn_prefill(const at::Tensor& q, const at::Tensor& k_cache, const at::Tens
         "attn_prefill");
 }
 
-void gemm_bf16_pair(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, int64_t epilogue, int64_t bn, c10::optional<at::Tensor> status) {
+using OptAct = c10::optional<std::array<double, 4>>;     // limit, alpha, up_bias, cap (B2EpiAct)
+B2EpiAct epi_act(const OptAct& a) {
+  if (!a.has_value()) return B2EpiAct{INFINITY, 1.0f, 0.0f, 0.0f};
+  return B2EpiAct{static_cast<float>((*a)[0]), static_cast<float>((*a)[1]), static_cast<float>((*a)[2]), static_cast<float>((*a)[3])};
+}
+
+void gemm_bf16_pair(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, int64_t epilogue, int64_t bn, c10::optional<at::Tensor> status,
+                    OptAct act) {
   need(x.is_cuda() && is_bf16(x) && is_bf16(w) && is_bf16(y) && x.dim() == 2 && w.dim() == 2 && y.dim() == 2, "gemm_bf16_pair: 2-D CUDA bf16 tensors");
   need(x.stride(1) == 1 && w.stride(1) == 1 && y.stride(1) == 1 && x.size(1) == w.size(1) && y.size(0) == x.size(0) &&
            y.size(1) == (epilogue == B2_EPI_SWIGLU ? w.size(0) / 2 : w.size(0)),
        "gemm_bf16_pair: x [M, K], w [N, K], y [M, N] (or [M, N / 2] with the SwiGLU epilogue), unit inner strides");
   c10::cuda::CUDAGuard g(x.device());
+  const B2EpiAct ea = epi_act(act);
   check(b2_gemm_bf16_pair(x.data_ptr(), w.data_ptr(), y.data_ptr(), static_cast<int>(x.size(0)), static_cast<int>(w.size(0)),
-                          static_cast<int>(x.size(1)), x.stride(0), w.stride(0), y.stride(0), static_cast<int>(epilogue), static_cast<int>(bn), status_ptr(status), cur_stream()),
+                          static_cast<int>(x.size(1)), x.stride(0), w.stride(0), y.stride(0), static_cast<int>(epilogue), &ea, static_cast<int>(bn), status_ptr(status), cur_stream()),
         "gemm_bf16_pair");
 }
 
 void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out,
                      const at::Tensor& cu_q, const at::Tensor& ctx_lens, const at::Tensor& block_tables, int64_t max_q_len,
-                     double scale, int64_t variant, c10::optional<at::Tensor> status, c10::optional<at::Tensor> work,
+                     double scale, c10::optional<at::Tensor> status, c10::optional<at::Tensor> work,
                      c10::optional<at::Tensor> n_work, int64_t work_items, c10::optional<at::Tensor> gate) {
-  check_cache(q, k_cache, v_cache, 128);
+  // contiguous paged caches, or a [pages, n_kv, 128, 128] view of matrices with one row per token and all heads in it
+  const int64_t token_stride = k_cache.is_contiguous() ? 0 : k_cache.stride(2);
+  if (token_stride == 0) check_cache(q, k_cache, v_cache, 128);
+  else
+    need(q.is_cuda() && is_bf16(q) && q.dim() == 2 && q.stride(1) == 1 && is_bf16(k_cache) && is_bf16(v_cache) && k_cache.dim() == 4 &&
+             v_cache.sizes() == k_cache.sizes() && v_cache.strides() == k_cache.strides() && k_cache.stride(3) == 1 && k_cache.stride(1) == 128 &&
+             k_cache.stride(0) == 128 * token_stride && token_stride >= 128 * k_cache.size(1),
+         "attn_prefill_tc: strided keys and values must have one row per token with the heads side by side");
+  const bool gate_elems = gate.has_value() && gate->dim() == 2 && gate->size(1) == q.size(1);
   if (work.has_value()) {
     need(work->is_cuda() && work->scalar_type() == at::kInt && work->is_contiguous() && work->numel() >= 2 * work_items, "attn_prefill_tc: work must be CUDA int32 [items, 2]");
     if (n_work.has_value()) need(n_work->is_cuda() && n_work->scalar_type() == at::kInt && n_work->numel() >= 1, "attn_prefill_tc: n_work must be a CUDA int32 scalar");
@@ -243,10 +261,11 @@ void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::T
                                 ctx_lens.data_ptr<int32_t>(), block_tables.data_ptr<int32_t>(), batch,
                                 static_cast<int>(block_tables.size(1)), static_cast<int>(q.size(1) / 128),
                                 static_cast<int>(k_cache.size(1)), static_cast<int>(max_q_len), static_cast<float>(scale), q.size(0),
-                                q.stride(0), out.stride(0), k_cache.size(0), static_cast<int>(variant),
+                                q.stride(0), out.stride(0), k_cache.size(0), token_stride,
                                 work.has_value() ? work->data_ptr<int32_t>() : nullptr,
                                 work.has_value() && n_work.has_value() ? n_work->data_ptr<int32_t>() : nullptr,
-                                static_cast<int>(work_items), gate_ptr(gate, q, q.size(1) / 128), gate_ld(gate), status_ptr(status), cur_stream()),
+                                static_cast<int>(work_items), gate_ptr(gate, q, gate_elems ? q.size(1) : q.size(1) / 128), gate_ld(gate), gate_elems ? 1 : 0,
+                                status_ptr(status), cur_stream()),
         "attn_prefill_tc");
 }
 
@@ -282,8 +301,8 @@ void attn_decode(const at::Tensor& q, const at::Tensor& k_cache, const at::Tenso
 }
 
 void gemm_bf16(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, c10::optional<at::Tensor> residual,
-               int64_t epilogue, int64_t config, c10::optional<at::Tensor> workspace, c10::optional<at::Tensor> status) {
-  need(x.is_cuda() && is_bf16(x) && is_bf16(w) && is_bf16(y) && x.dim() == 2 && w.dim() == 2 && y.dim() == 2, "gemm: 2-D CUDA bf16 x [M,K], w [N,K], y [M,N]");
+               int64_t epilogue, int64_t config, c10::optional<at::Tensor> workspace, c10::optional<at::Tensor> status, OptAct act) {
+  need(x.is_cuda() && is_bf16(x) && is_bf16(w) && y.scalar_type() == (epilogue == B2_EPI_F32 ? at::kFloat : at::kBFloat16) && x.dim() == 2 && w.dim() == 2 && y.dim() == 2, "gemm: 2-D CUDA bf16 x [M,K], w [N,K], y [M,N]");
   need(x.stride(1) == 1 && w.stride(1) == 1 && y.stride(1) == 1, "gemm: unit inner strides required");
   const int M = static_cast<int>(x.size(0)), K = static_cast<int>(x.size(1)), N = static_cast<int>(w.size(0));
   need(w.size(1) == K, "gemm: K mismatch");
@@ -291,8 +310,9 @@ void gemm_bf16(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, c10::opt
   need(y.size(0) == M && y.size(1) == out_cols, "gemm: output shape mismatch");
   if (residual.has_value()) need(is_bf16(*residual) && residual->sizes() == y.sizes() && residual->stride(1) == 1 && residual->stride(0) == y.stride(0), "gemm: residual must match y");
   c10::cuda::CUDAGuard g(x.device());
+  const B2EpiAct ea = epi_act(act);
   check(b2_gemm_bf16(x.data_ptr(), w.data_ptr(), y.data_ptr(), opt_ptr(residual), M, N, K, x.stride(0), w.stride(0),
-                     y.stride(0), static_cast<int>(epilogue), static_cast<int>(config), opt_ptr(workspace),
+                     y.stride(0), static_cast<int>(epilogue), &ea, static_cast<int>(config), opt_ptr(workspace),
                      workspace.has_value() ? workspace->numel() * workspace->element_size() : 0, status_ptr(status),
                      cur_stream()),
         "gemm_bf16");
@@ -322,6 +342,7 @@ py::dict device_caps(int device) {
 void bind_ops_extra(py::module_& m);
 void bind_coll(py::module_& m);
 void bind_mixers(py::module_& m);
+void bind_latent(py::module_& m);
 void bind_io(py::module_& m);
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
@@ -345,16 +366,16 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("attn_prefill", &attn_prefill, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("cu_q"),
         py::arg("ctx_lens"), py::arg("block_tables"), py::arg("head_dim"), py::arg("max_q_len"), py::arg("scale"),
         py::arg("status") = py::none(), py::arg("gate") = py::none());
-  m.def("gemm_bf16_pair", &gemm_bf16_pair, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("epilogue") = 0, py::arg("bn") = 256, py::arg("status") = py::none());
+  m.def("gemm_bf16_pair", &gemm_bf16_pair, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("epilogue") = 0, py::arg("bn") = 256, py::arg("status") = py::none(), py::arg("act") = py::none());
   m.def("attn_prefill_tc", &attn_prefill_tc, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("cu_q"),
-        py::arg("ctx_lens"), py::arg("block_tables"), py::arg("max_q_len"), py::arg("scale"), py::arg("variant") = 0,
+        py::arg("ctx_lens"), py::arg("block_tables"), py::arg("max_q_len"), py::arg("scale"),
         py::arg("status") = py::none(), py::arg("work") = py::none(), py::arg("n_work") = py::none(), py::arg("work_items") = 0,
         py::arg("gate") = py::none());
   m.def("attn_decode", &attn_decode, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("ctx_lens"),
         py::arg("block_tables"), py::arg("workspace"), py::arg("head_dim"), py::arg("num_splits"), py::arg("scale"),
         py::arg("status") = py::none(), py::arg("counters") = py::none(), py::arg("gate") = py::none());
   m.def("gemm_bf16", &gemm_bf16, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("residual") = py::none(),
-        py::arg("epilogue") = 0, py::arg("config") = 0, py::arg("workspace") = py::none(), py::arg("status") = py::none());
+        py::arg("epilogue") = 0, py::arg("config") = 0, py::arg("workspace") = py::none(), py::arg("status") = py::none(), py::arg("act") = py::none());
   m.def("gemm_workspace_bytes", [](int M, int N, int K) { return b2_gemm_workspace_bytes(M, N, K); });
   m.def("attn_decode_workspace_bytes", [](int batch, int n_q, int d, int splits) { return b2_attn_decode_workspace(batch, n_q, d, splits); });
   m.def("device_caps", &device_caps, py::arg("device") = 0);
@@ -363,5 +384,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   bind_coll(m);
 #endif
   bind_mixers(m);
+  bind_latent(m);
   bind_io(m);
 }

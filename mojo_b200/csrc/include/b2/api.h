@@ -70,16 +70,19 @@ int b2_attn_prefill_bf16(const void* q, const void* k_cache, const void* v_cache
                          int n_kv, int head_dim, int page_size, int max_q_len, float scale, int64_t q_stride,
                          int64_t out_stride, int64_t num_pages, const void* gate, int64_t gate_stride,
                          b2::Status* status, cudaStream_t stream);
-// bf16 GEMM on CTA pairs (tcgen05 cta_group::2, 256 x 256 tiles; csrc/kernels/gemm_bf16_pair.cu). Epilogue NONE or SWIGLU.
+// bf16 GEMM on CTA pairs (tcgen05 cta_group::2, 256 x 256 tiles; csrc/kernels/gemm_bf16_pair.cu). Epilogue NONE, SWIGLU
+// or RELU2.
 int b2_gemm_bf16_pair(const void* x, const void* w, void* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,
-                      int epilogue, int bn, b2::Status* status, cudaStream_t stream);
+                      int epilogue, const struct B2EpiAct* act, int bn, b2::Status* status, cudaStream_t stream);
 // The same attention on tcgen05 / TMEM (csrc/kernels/attention_tc.cu): head_dim 128 and page_size 128 only.
-// q_rows = rows of the q matrix (for the tensor map); variant = descriptor variant of the V operand (0 = default).
+// q_rows = rows of the q matrix (for the tensor map). token_stride 0: paged caches; otherwise keys and values lie in
+// matrices with one row per token (elements between rows), all heads side by side, and a page is 128 such rows.
+// gate_elems: the gate has one logit per output element, [T, n_q * 128].
 int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* cu_q,
                             const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                             int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
-                            int64_t num_pages, int variant, const int32_t* work, const int32_t* n_work, int work_items,
-                            const void* gate, int64_t gate_stride, b2::Status* status, cudaStream_t stream);
+                            int64_t num_pages, int64_t token_stride, const int32_t* work, const int32_t* n_work, int work_items,
+                            const void* gate, int64_t gate_stride, int gate_elems, b2::Status* status, cudaStream_t stream);
 // One query token per sequence, split over the KV length. workspace: f32, size from b2_attn_decode_workspace.
 // `counters` (may be null): u32 [batch * n_kv], zero before the first use and left at zero by every launch; with it
 // (and page sizes that are multiples of 32) the split that finishes last merges the partials itself, otherwise a
@@ -105,6 +108,12 @@ int b2_mla_attend_bf16(const void* q_lat, const void* q_rope, const void* kv_cac
                        const int32_t* block_tables, const int32_t* row_seq, float* workspace, int rows, int max_blocks,
                        int n_heads, int page_size, int num_splits, float scale, int64_t num_pages, int64_t q_lat_stride,
                        int64_t q_rope_stride, b2::Status* status, cudaStream_t stream);
+// The same attention without a rotated part, for latents of 64, 128, 256, 512 or 1024 columns (cache [num_pages, page, latent],
+// page a multiple of 8; out_lat [rows, H, latent]).
+int b2_latent_attend_bf16(const void* q_lat, const void* cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
+                          const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int latent, int page_size,
+                          int num_splits, float scale, int64_t num_pages, int64_t q_lat_stride, b2::Status* status, cudaStream_t stream);
+int64_t b2_latent_attend_workspace(int rows, int n_heads, int latent, int num_splits);
 // row_ctx[t] / row_seq[t] for every token t of a batch described by cu_q [num_seqs + 1] and ctx_lens [num_seqs]:
 // token i of a sequence's chunk sees ctx - q_len + i + 1 positions (causal mask of chunked prefill; decode rows: ctx).
 int b2_mla_rows_meta(const int32_t* cu_q, const int32_t* ctx_lens, int num_seqs, int32_t* row_ctx, int32_t* row_seq,
@@ -112,13 +121,19 @@ int b2_mla_rows_meta(const int32_t* cu_q, const int32_t* ctx_lens, int num_seqs,
 
 // ---- GEMM (tcgen05 / TMEM / TMA) ---------------------------------------------------------------
 // Epilogue selector for the tcgen05 GEMMs.
-enum B2Epilogue { B2_EPI_NONE = 0, B2_EPI_ADD_RESIDUAL = 1, B2_EPI_SWIGLU = 2 };
+//   RELU2    y = max(v, 0)^2            SOFTCAP  y = cap * tanh(v / cap)          F32  y is float, not bf16
+enum B2Epilogue { B2_EPI_NONE = 0, B2_EPI_ADD_RESIDUAL = 1, B2_EPI_SWIGLU = 2, B2_EPI_RELU2 = 3, B2_EPI_SOFTCAP = 4, B2_EPI_F32 = 5 };
+// Constants of an epilogue's activation. Gated linear units compute g * sigmoid(alpha * g) * (u + up_bias) after
+// g = min(g, limit), u = clamp(u, -limit, limit); {infinity, 1, 0} is SwiGLU. `cap` belongs to SOFTCAP.
+struct B2EpiAct {
+  float limit, alpha, up_bias, cap;
+};
 // Y[M, N] = X[M, K] * W[N, K]^T (+ residual), bf16 in, f32 accumulate, bf16 out.
 // ldx/ldw/ldy are row strides in elements. `workspace`/`counters` are split-K scratch (may be null when
-// the chosen configuration does not split); sizes from b2_gemm_workspace_bytes.
+// the chosen configuration does not split); sizes from b2_gemm_workspace_bytes. `act` null: SwiGLU's constants.
 int b2_gemm_bf16(const void* x, const void* w, void* y, const void* residual, int M, int N, int K, int64_t ldx,
-                 int64_t ldw, int64_t ldy, int epilogue, int config, void* workspace, int64_t workspace_bytes,
-                 b2::Status* status, cudaStream_t stream);
+                 int64_t ldw, int64_t ldy, int epilogue, const struct B2EpiAct* act, int config, void* workspace,
+                 int64_t workspace_bytes, b2::Status* status, cudaStream_t stream);
 int64_t b2_gemm_workspace_bytes(int M, int N, int K);
 // fp8 block-scaled: X e4m3 [M, K] with f32 scales [M, K/128]; W e4m3 [N, K] with f32 scales [N/128, K/128].
 int b2_gemm_fp8_block(const void* xq, const float* xs, const void* wq, const float* ws, void* y, int M, int N, int K,

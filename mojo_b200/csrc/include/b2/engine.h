@@ -130,6 +130,7 @@ struct Batch {
   std::vector<int32_t> cu_q;        // [B + 1] offsets into the flat token arrays
   std::vector<int64_t> token_ids;   // [T]
   std::vector<int32_t> positions;   // [T]
+  std::vector<int32_t> prev_tokens; // [T] the token before each row's in its sequence; -1: there is none; -2: not read back yet
   std::vector<int64_t> slots;       // [T] physical KV slots
   std::vector<int32_t> block_tables;  // [B, max_blocks], padded with 0
   std::vector<int32_t> seq_state;   // [B, 2] recurrent-state banks {read, write} per sequence; empty without state slots

@@ -22,6 +22,8 @@
 // (stdlib/src/sys/info.mojo:423-434) and it contains no MMA code at all.
 #pragma once
 #include <cstdint>
+#include <type_traits>
+#include <utility>
 #include <cuda.h>
 #include "b2/ptx.cuh"
 #include "b2/status.h"
@@ -83,6 +85,17 @@ constexpr int kThreadsWithFill = kThreads + 128;
 struct NoSide {
   static constexpr int kWarps = 0;
   __device__ __forceinline__ void operator()(int, int) const {}
+};
+
+// First K column of a unit's P operand. Schedulers whose units read different column ranges of one P matrix (heads side
+// by side in a row) define `int p_kx(const WorkUnit&) const` (a multiple of 8 elements); for all others it is 0.
+template <class Sched, class = void>
+struct PColumn {
+  static __device__ __forceinline__ int of(const Sched&, const WorkUnit&) { return 0; }
+};
+template <class Sched>
+struct PColumn<Sched, std::void_t<decltype(std::declval<const Sched&>().p_kx(std::declval<const WorkUnit&>()))>> {
+  static __device__ __forceinline__ int of(const Sched& s, const WorkUnit& u) { return s.p_kx(u); }
 };
 
 // Byte offset of 16-byte chunk `c` (0..7) of row `r` (0..127) inside a 128 x 64 bf16 tile stored with the
@@ -163,7 +176,7 @@ __device__ __forceinline__ void run(const CUtensorMap* tmap_p, const CUtensorMap
           const uint32_t sp = smem_base + stage * L::kStageBytes;
           ptx::mbar_arrive_expect_tx(full_bar(stage), PFill::kActive ? L::kQBytes : L::kStageBytes);
           const int kx = kb * (128 / ELEM_BYTES);
-          if (!PFill::kActive) ptx::tma_load_2d(sp, tmap_p, full_bar(stage), kx, u.p_coord, policy_p);
+          if (!PFill::kActive) ptx::tma_load_2d(sp, tmap_p, full_bar(stage), kx + PColumn<Sched>::of(sched, u), u.p_coord, policy_p);
           ptx::tma_load_2d(sp + L::kPBytes, tmap_q, full_bar(stage), kx, u.q_coord, policy_q);
           ++issued;
           if (++stage == STAGES) { stage = 0; phase ^= 1u; }

@@ -6,6 +6,7 @@
 #pragma once
 #include <cstdint>
 #include <cuda_runtime.h>
+#include "b2/api.h"
 #include "b2/status.h"
 
 #ifdef __cplusplus
@@ -42,6 +43,33 @@ struct B2HyperArgs {
   int32_t n_out, rows, width, mean_width, streams, vocab, store;
 };
 int b2_hyper_norm(const B2HyperArgs* a, int f32, b2::Status* status, cudaStream_t stream);
+
+// One f32 residual stream x [rows, width] with a scale per channel. For every row: x += y_scale * (y + sum_j w[j] e[slot[j]]),
+// where y (a sublayer's output) and the expert rows e (`top` of them per row, w and slot [rows, top]) may each be null;
+// then h = rms_norm(x) * weight, or x itself rounded where weight is null. With `ids` x starts as
+// embed[id] * embed_scale (+ bigram[(prev * mul_prev + id * mul_cur) mod buckets], or its last row, number `buckets`, where
+// prev is -1) instead of being read, and x0 (may be null) receives a rounded copy of that. `store` writes x back. With
+// `rows_index` only those rows are processed and h is compact. Columns from `mean_width` up to `width` are zero padding.
+struct B2ResidualArgs {
+  float* x;
+  const void* y;
+  const void* experts;
+  const int32_t* expert_slot;
+  const float* expert_w;
+  const float* y_scale;
+  const float* weight;
+  void* h;
+  const int64_t* ids;
+  const void* embed;
+  const int32_t* prev;
+  const void* bigram;
+  void* x0;
+  const int64_t* rows_index;
+  int64_t ld_h, ld_x0, mul_prev, mul_cur, buckets;
+  float embed_scale, eps;
+  int32_t top, expert_rows, n_out, rows, width, mean_width, vocab, store;
+};
+int b2_residual_norm(const B2ResidualArgs* a, int f32, b2::Status* status, cudaStream_t stream);
 
 // Short causal convolution on the q | k | v channels of a projection, rotary embedding on q and k, RMS norm of each q and k
 // head (no weight), and the scatter of k and v into the paged cache; one launch. proj [rows, ld]: the channels start at
@@ -96,14 +124,24 @@ int64_t b2_delta_scratch_floats(int heads, int dim, int vdim, int rows, int seqs
 int b2_delta_rule(const B2DeltaArgs* a, const B2SeqRows* s, int n_decode, int first, int n_prefill, int f32, b2::Status* status,
                   cudaStream_t stream);
 
-// Y[M, N] = X[M, K] W[N, K]^T in true f32 (FMA, no reduced-precision matrix mode).
-int b2_gemm_f32(const float* x, const float* w, float* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,
-                cudaStream_t stream);
-// out[r, j] = silu(gate) * up for rows whose gate and up columns alternate in blocks of 16.
-int b2_swiglu_f32(const float* gate_up, float* out, int rows, int ffn, cudaStream_t stream);
+// Y[M, N] = X[M, K] W[N, K]^T in true f32 (FMA, no reduced-precision matrix mode), `batch` such products side by side: product
+// b reads x columns b * K ..., weight rows b * N ... and writes y columns b * N .... Epilogue NONE, RELU2 or SOFTCAP
+// (B2Epilogue); then y is multiplied by sigmoid(gate) element by element where a gate [M, batch * N] is given.
+struct B2GemmF32Args {
+  const float* x;
+  const float* w;
+  float* y;
+  const float* gate;
+  int64_t ldx, ldw, ldy, ld_gate;
+  float cap;
+  int32_t M, N, K, batch, epilogue;
+};
+int b2_gemm_f32(const B2GemmF32Args* a, cudaStream_t stream);
+// Gated linear unit (B2EpiAct) of rows whose gate and up columns alternate in blocks of 16.
+int b2_glu_f32(const float* gate_up, float* out, int64_t rows, int ffn, const struct B2EpiAct* act, cudaStream_t stream);
 int b2_gather_rows_f32(const float* src, const int64_t* index, float* out, int rows_out, int cols, int64_t rows_src,
                        b2::Status* status, cudaStream_t stream);
-// Causal GQA attention over the paged cache in f32: any head sizes up to 256, decode rows and prompt chunks alike. Row t
+// Causal GQA attention over the paged cache in f32: any head sizes up to 1024, decode rows and prompt chunks alike. Row t
 // of sequence row_seq[t] sees positions 0 .. positions[t]. gate as in b2/api.h, f32.
 int b2_attn_f32(const float* q, const float* k_cache, const float* v_cache, float* out, const int32_t* row_seq,
                 const int32_t* positions, const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv,

@@ -30,6 +30,7 @@
 #include "b2/ptx.cuh"
 #include "b2/status.h"
 #include "b2/tma.h"
+#include "b2/vec.cuh"
 
 namespace b2 {
 namespace {
@@ -68,9 +69,14 @@ struct AttnTcParams {
   // every CTA of the grid has an item. Without a list the grid is (query tiles, heads, sequences).
   const int* work;
   const int* n_work;
-  // Optional per-head output gate: head h of row t is multiplied by sigmoid(gate[t * gate_stride + h]). Null: no gate.
+  // Optional output gate, null: none. One factor sigmoid(gate[t * gate_stride + h]) for head h of row t, or with
+  // `gate_elems` one per output element, sigmoid(gate[t * gate_stride + h * 128 + c]).
   const __nv_bfloat16* gate;
   int64_t gate_stride;
+  int gate_elems;
+  // Where the tile of (page, KV head) lies in the K and V matrices: row page * page_rows + head * head_rows, column
+  // head * head_cols. Paged cache: {n_kv * 128, 128, 0}; rows of one token with its heads side by side: {128, 0, 128}.
+  int page_rows, head_rows, head_cols;
 };
 
 // Shared-memory descriptor with explicit leading / stride byte offsets, 128-byte swizzle.
@@ -176,16 +182,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
           status_record(status, kOutOfBounds, kSiteKvIndex, seq, page);
           page = 0;
         }
-        const int row = (page * prm.n_kv + kvh) * kTile;
+        const int row = page * prm.page_rows + kvh * prm.head_rows, col = kvh * prm.head_cols;
         if (!ptx::mbar_wait(k_empty(s), ph ^ 1u)) { give_up(1, j); ok = false; break; }
         ptx::mbar_arrive_expect_tx(k_full(s), kTileBytes);
-        ptx::tma_load_2d(base + kOffK + s * kTileBytes, &tmap_k, k_full(s), 0, row, ptx::kEvictLast);
-        ptx::tma_load_2d(base + kOffK + s * kTileBytes + kHalfBytes, &tmap_k, k_full(s), 64, row, ptx::kEvictLast);
+        ptx::tma_load_2d(base + kOffK + s * kTileBytes, &tmap_k, k_full(s), col, row, ptx::kEvictLast);
+        ptx::tma_load_2d(base + kOffK + s * kTileBytes + kHalfBytes, &tmap_k, k_full(s), col + 64, row, ptx::kEvictLast);
         ++issued_k;
         if (!ptx::mbar_wait(v_empty(s), ph ^ 1u)) { give_up(2, j); ok = false; break; }
         ptx::mbar_arrive_expect_tx(v_full(s), kTileBytes);
-        ptx::tma_load_2d(base + kOffV + s * kTileBytes, &tmap_v, v_full(s), 0, row, ptx::kEvictLast);
-        ptx::tma_load_2d(base + kOffV + s * kTileBytes + kHalfBytes, &tmap_v, v_full(s), 64, row, ptx::kEvictLast);
+        ptx::tma_load_2d(base + kOffV + s * kTileBytes, &tmap_v, v_full(s), col, row, ptx::kEvictLast);
+        ptx::tma_load_2d(base + kOffV + s * kTileBytes + kHalfBytes, &tmap_v, v_full(s), col + 64, row, ptx::kEvictLast);
         ++issued_v;
       }
       if (!ok) {
@@ -365,7 +371,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     if (ok && *fail == 0 && r < rows) {
       const float l = l_final[r] + l_final[kTile + r];
       float inv = l > 0.0f ? 1.0f / l : 0.0f;
-      if (prm.gate != nullptr) {
+      if (prm.gate != nullptr && prm.gate_elems) {
+        const __nv_bfloat16* z = prm.gate + static_cast<int64_t>(q_begin + qt * kTile + r) * prm.gate_stride + head * kD + g * 64;
+#pragma unroll
+        for (int c = 0; c < 8; ++c) {
+          float f[8];
+          bf16x8_to_f32(ptx::ld_v4(z + c * 8), f);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) o[c * 8 + i] *= ptx::rcp(1.0f + ptx::ex2(-f[i] * ptx::kLog2e));
+        }
+      } else if (prm.gate != nullptr) {
         const float z = __bfloat162float(prm.gate[static_cast<int64_t>(q_begin + qt * kTile + r) * prm.gate_stride + head]);
         inv /= 1.0f + ptx::ex2(-z * ptx::kLog2e);
       }
@@ -395,25 +410,29 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
 using namespace b2;
 
 // Same contract as b2_attn_prefill_bf16 with head_dim = 128 and page_size = 128 fixed; out rows 16-byte aligned.
-// `variant` is reserved (0). With `work` (device memory, `work_items` pairs of (sequence, query tile)) the grid is one
+// `token_stride` 0: paged caches [pages, n_kv, 128, 128]; otherwise the elements between two tokens' rows of keys (and of
+// values) that hold all heads side by side, 128 such rows to a page. With `work` (device memory, `work_items` pairs of (sequence, query tile)) the grid is one
 // CTA per item and head; `n_work` (device memory, may be null) bounds the valid items, for launches whose grid is
 // fixed ahead of the batch (CUDA graphs). The caller orders the items, longest context first for an even finish.
 extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* cu_q,
                                        const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                                        int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
-                                       int64_t num_pages, int variant, const int32_t* work, const int32_t* n_work, int work_items,
-                                       const void* gate, int64_t gate_stride, Status* status, cudaStream_t stream) {
+                                       int64_t num_pages, int64_t token_stride, const int32_t* work, const int32_t* n_work, int work_items,
+                                       const void* gate, int64_t gate_stride, int gate_elems, Status* status, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
   if (work != nullptr && work_items <= 0) return 0;
   if (n_q <= 0 || n_kv <= 0 || n_q % n_kv != 0 || q_stride % 8 != 0 || out_stride % 8 != 0 ||
-      (reinterpret_cast<uintptr_t>(q) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0)
+      (reinterpret_cast<uintptr_t>(q) & 15) != 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0 || token_stride % 8 != 0 ||
+      (gate != nullptr && gate_elems && (gate_stride % 8 != 0 || (reinterpret_cast<uintptr_t>(gate) & 15) != 0)))
     return -kBadArgument;
   CUtensorMap tq, tk, tv;
-  const int64_t kv_rows = num_pages * n_kv * kTile;
+  const bool by_token = token_stride != 0;
+  const int64_t kv_rows = num_pages * (by_token ? 1 : n_kv) * kTile, kv_cols = by_token ? static_cast<int64_t>(n_kv) * kD : kD;
+  const int64_t kv_ld = (by_token ? token_stride : kD) * 2;
   if (!make_tmap_2d(&tq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, q, q_rows, static_cast<int64_t>(n_q) * kD, q_stride * 2, kTile, 64,
                     CU_TENSOR_MAP_SWIZZLE_128B) ||
-      !make_tmap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, k_cache, kv_rows, kD, kD * 2, kTile, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
-      !make_tmap_2d(&tv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, v_cache, kv_rows, kD, kD * 2, kTile, 64, CU_TENSOR_MAP_SWIZZLE_128B))
+      !make_tmap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, k_cache, kv_rows, kv_cols, kv_ld, kTile, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
+      !make_tmap_2d(&tv, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, v_cache, kv_rows, kv_cols, kv_ld, kTile, 64, CU_TENSOR_MAP_SWIZZLE_128B))
     return -kBadArgument;
   AttnTcParams prm{};
   prm.out = static_cast<__nv_bfloat16*>(out);
@@ -432,7 +451,10 @@ extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const
   prm.n_work = work != nullptr ? n_work : nullptr;
   prm.gate = static_cast<const __nv_bfloat16*>(gate);
   prm.gate_stride = gate_stride;
-  (void)variant;
+  prm.gate_elems = gate_elems;
+  prm.page_rows = by_token ? kTile : n_kv * kTile;
+  prm.head_rows = by_token ? 0 : kTile;
+  prm.head_cols = by_token ? kD : 0;
   static DeviceOnce attr_once;
   if (const int rc = attr_once.run([&] {
         cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemAttn);

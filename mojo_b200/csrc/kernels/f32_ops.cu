@@ -1,6 +1,7 @@
-// True 32-bit forms of the matrix product, SwiGLU, row gather and paged attention, for models that run with f32
+// True 32-bit forms of the matrix product, gated linear units, row gather and paged attention, for models that run with f32
 // activations on the GPU. Plain FMA throughout: no TF32 or other reduced-precision matrix mode.
 #include <cstdint>
+#include "b2/act.cuh"
 #include "b2/api.h"
 #include "b2/elem.cuh"
 #include "b2/launch.h"
@@ -14,9 +15,12 @@ namespace {
 constexpr int kBM = 64, kBN = 64, kBK = 16;
 
 // 64 x 64 tile, 256 threads of 4 x 4 outputs.
-__global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, float* __restrict__ y, int M, int N,
-                                                       int K, int64_t ldx, int64_t ldw, int64_t ldy) {
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const B2GemmF32Args a) {
   ptx::grid_dep_sync();
+  const int M = a.M, N = a.N, K = a.K;
+  const int64_t ldx = a.ldx, ldw = a.ldw, col0 = static_cast<int64_t>(blockIdx.z) * N;
+  const float* __restrict__ x = a.x + static_cast<int64_t>(blockIdx.z) * K;
+  const float* __restrict__ w = a.w + col0 * ldw;
   __shared__ float xs[kBK][kBM + 4], ws[kBK][kBN + 4];
   const int m0 = blockIdx.y * kBM, n0 = blockIdx.x * kBN;
   const int tm = (threadIdx.x >> 4) * 4, tn = (threadIdx.x & 15) * 4;
@@ -30,13 +34,13 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     __syncthreads();
 #pragma unroll
     for (int k = 0; k < kBK; ++k) {
-      float a[4], b[4];
-      load_f32<4>(&xs[k][tm], a);
-      load_f32<4>(&ws[k][tn], b);
+      float xv[4], wv[4];
+      load_f32<4>(&xs[k][tm], xv);
+      load_f32<4>(&ws[k][tn], wv);
 #pragma unroll
       for (int i = 0; i < 4; ++i)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(xv[i], wv[j], acc[i][j]);
     }
     __syncthreads();
   }
@@ -44,17 +48,25 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (m0 + tm + i < M && n0 + tn + j < N) y[(m0 + tm + i) * ldy + n0 + tn + j] = acc[i][j];
+      if (m0 + tm + i < M && n0 + tn + j < N) {
+        const int64_t m = m0 + tm + i, n = col0 + n0 + tn + j;
+        float v = acc[i][j];
+        if (a.epilogue == B2_EPI_RELU2) v = relu2(v);
+        if (a.epilogue == B2_EPI_SOFTCAP) v = softcap(v, a.cap);
+        if (a.gate != nullptr) v *= sigmoid_f32(a.gate[m * a.ld_gate + n]);
+        a.y[m * a.ldy + n] = v;
+      }
 }
 
-__global__ void swiglu_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, int64_t total, int ffn) {
+__global__ void glu_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, int64_t total, int ffn, B2EpiAct act) {
   ptx::grid_dep_sync();
   const int64_t i = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= total) return;
   const int64_t r = i / ffn;
   const int c = static_cast<int>(i % ffn);
   const float* p = gu + r * 2 * ffn + (c / 16) * 32 + c % 16;
-  out[i] = p[0] / (1.0f + expf(-p[0])) * p[16];
+  const float g = fminf(p[0], act.limit), u = fminf(fmaxf(p[16], -act.limit), act.limit);
+  out[i] = g / (1.0f + expf(-act.alpha * g)) * (u + act.up_bias);
 }
 
 __global__ void gather_rows_f32_kernel(const float* __restrict__ src, const int64_t* __restrict__ index, float* __restrict__ out, int cols,
@@ -66,7 +78,7 @@ __global__ void gather_rows_f32_kernel(const float* __restrict__ src, const int6
 }
 
 // One warp per (row, head): 32 keys at a time, a key per lane for the scores, a value column per lane for the output.
-constexpr int kAttnMax = 256;
+template <int kAttnMax>
 __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__ q, const float* __restrict__ kc, const float* __restrict__ vc,
                                                        float* __restrict__ out, const int32_t* __restrict__ row_seq,
                                                        const int32_t* __restrict__ positions, const int32_t* __restrict__ tables, int rows, int seqs,
@@ -134,18 +146,20 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
 
 using namespace b2;
 
-extern "C" int b2_gemm_f32(const float* x, const float* w, float* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy, cudaStream_t stream) {
-  if (M <= 0 || N <= 0) return 0;
-  if (K <= 0 || (M + kBM - 1) / kBM > 65535) return -kBadArgument;
-  launch_pdl(gemm_f32_kernel, dim3((N + kBN - 1) / kBN, (M + kBM - 1) / kBM), dim3(256), 0, stream, x, w, y, M, N, K, ldx, ldw, ldy);
+extern "C" int b2_gemm_f32(const B2GemmF32Args* a, cudaStream_t stream) {
+  if (a->M <= 0 || a->N <= 0) return 0;
+  if (a->K <= 0 || (a->M + kBM - 1) / kBM > 65535 || a->batch < 1 || a->batch > 65535 || (a->epilogue == B2_EPI_SOFTCAP && !(a->cap > 0.0f)) ||
+      (a->epilogue != B2_EPI_NONE && a->epilogue != B2_EPI_RELU2 && a->epilogue != B2_EPI_SOFTCAP))
+    return -kBadArgument;
+  launch_pdl(gemm_f32_kernel, dim3((a->N + kBN - 1) / kBN, (a->M + kBM - 1) / kBM, a->batch), dim3(256), 0, stream, *a);
   return last_launch_rc();
 }
 
-extern "C" int b2_swiglu_f32(const float* gate_up, float* out, int rows, int ffn, cudaStream_t stream) {
+extern "C" int b2_glu_f32(const float* gate_up, float* out, int64_t rows, int ffn, const B2EpiAct* act, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (ffn <= 0 || ffn % 16 != 0) return -kBadArgument;
-  const int64_t total = static_cast<int64_t>(rows) * ffn;
-  launch_pdl(swiglu_f32_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, stream, gate_up, out, total, ffn);
+  const int64_t total = rows * ffn;
+  launch_pdl(glu_f32_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, stream, gate_up, out, total, ffn, act != nullptr ? *act : kPlainAct);
   return last_launch_rc();
 }
 
@@ -160,9 +174,10 @@ extern "C" int b2_attn_f32(const float* q, const float* k_cache, const float* v_
                            const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv, int dim, int vdim, int page_size,
                            float scale, int64_t num_pages, const float* gate, int64_t gate_stride, Status* status, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (n_kv <= 0 || n_q % n_kv != 0 || dim <= 0 || dim > kAttnMax || vdim <= 0 || vdim > kAttnMax || page_size <= 0) return -kBadArgument;
+  if (n_kv <= 0 || n_q % n_kv != 0 || dim <= 0 || dim > 1024 || vdim <= 0 || vdim > 1024 || page_size <= 0) return -kBadArgument;
+  auto kern = dim <= 256 && vdim <= 256 ? attn_f32_kernel<256> : attn_f32_kernel<1024>;
   const int64_t warps = static_cast<int64_t>(rows) * n_q;
-  launch_pdl(attn_f32_kernel, dim3(static_cast<unsigned>((warps + 3) / 4)), dim3(128), 0, stream, q, k_cache, v_cache, out, row_seq, positions,
+  launch_pdl(kern, dim3(static_cast<unsigned>((warps + 3) / 4)), dim3(128), 0, stream, q, k_cache, v_cache, out, row_seq, positions,
              block_tables, rows, seqs, max_blocks, n_q, n_kv, dim, vdim, page_size, scale, num_pages, gate, gate_stride, status);
   return last_launch_rc();
 }

@@ -7,10 +7,12 @@
 //                          becomes the UMMA N (16..256). Every byte staged in shared memory is weight data, so
 //                          decode-sized M streams the weights once at HBM rate; K can be split across CTAs
 //                          (f32 partials in a workspace, last CTA of a tile reduces) to fill all 148 SMs.
-// Epilogues: plain store, + residual, SwiGLU on 16-row-interleaved gate/up weights.
+// Epilogues: plain store (bf16 or f32), + residual, squared ReLU, soft cap, gated linear units on 16-row-interleaved
+// gate/up weights.
 #include <cstdint>
 #include <cuda.h>
 #include <cuda_bf16.h>
+#include "b2/act.cuh"
 #include "b2/api.h"
 #include "b2/launch.h"
 #include "b2/gemm_tc.cuh"
@@ -32,6 +34,7 @@ struct EpiParams {
   float* workspace;  // [tiles][splits][BN][128] f32 partials
   uint32_t* counters;  // [tiles], zero on entry and on exit
   int mode;          // B2Epilogue
+  B2EpiAct act;
 };
 
 // Shared by both layouts: either pull a 32-column chunk out of TMEM or, for the reducing CTA of a split-K
@@ -69,6 +72,13 @@ struct Epilogue {
   EpiParams p;
 
   __device__ __forceinline__ void store_chunk(const WorkUnit& u, int c, int p_local, int lane, float (&v)[CH]) const {
+    if (p.mode == B2_EPI_RELU2) {
+#pragma unroll
+      for (int j = 0; j < CH; ++j) v[j] = relu2(v[j]);
+    } else if (p.mode == B2_EPI_SOFTCAP) {
+#pragma unroll
+      for (int j = 0; j < CH; ++j) v[j] = softcap(v[j], p.act.cap);
+    }
     if constexpr (!SWAP) {
       // thread = output row m; chunk = CH consecutive output columns
       const int m = u.pb * 128 + p_local;
@@ -80,7 +90,7 @@ struct Epilogue {
         if (n0 >= p.N) return;
         float o[HALF];
 #pragma unroll
-        for (int j = 0; j < HALF; ++j) o[j] = ptx::silu(v[j]) * v[HALF + j];
+        for (int j = 0; j < HALF; ++j) o[j] = glu(p.act, v[j], v[HALF + j]);
         __nv_bfloat16* dst = p.y + static_cast<int64_t>(m) * p.ldy + n0 / 2;
 #pragma unroll
         for (int g = 0; g < HALF / 8; ++g) {
@@ -91,6 +101,13 @@ struct Epilogue {
           pk.w = ptx::pack_bf16x2(o[g * 8 + 6], o[g * 8 + 7]);
           ptx::st_v4(dst + g * 8, pk);
         }
+        return;
+      }
+      if (p.mode == B2_EPI_F32) {
+        float* dst = reinterpret_cast<float*>(p.y) + static_cast<int64_t>(m) * p.ldy + n0;
+#pragma unroll
+        for (int g = 0; g < CH / 4; ++g)
+          if (n0 + g * 4 < p.N) *reinterpret_cast<float4*>(dst + g * 4) = make_float4(v[g * 4], v[g * 4 + 1], v[g * 4 + 2], v[g * 4 + 3]);
         return;
       }
       __nv_bfloat16* dst = p.y + static_cast<int64_t>(m) * p.ldy + n0;
@@ -126,11 +143,18 @@ struct Epilogue {
         for (int j = 0; j < CH; ++j) {
           const float other = __shfl_xor_sync(0xffffffffu, v[j], 16);
           if (lane < 16 && n < p.N && m0 + j < p.M)
-            p.y[static_cast<int64_t>(m0 + j) * p.ldy + out_col] = __float2bfloat16(ptx::silu(v[j]) * other);
+            p.y[static_cast<int64_t>(m0 + j) * p.ldy + out_col] = __float2bfloat16(glu(p.act, v[j], other));
         }
         return;
       }
       if (n >= p.N) return;
+      if (p.mode == B2_EPI_F32) {
+        float* dst = reinterpret_cast<float*>(p.y);
+#pragma unroll
+        for (int j = 0; j < CH; ++j)
+          if (m0 + j < p.M) dst[static_cast<int64_t>(m0 + j) * p.ldy + n] = v[j];
+        return;
+      }
 #pragma unroll
       for (int j = 0; j < CH; ++j) {
         if (m0 + j >= p.M) break;
@@ -364,9 +388,10 @@ extern "C" int64_t b2_gemm_workspace_bytes(int M, int N, int K) {
 }
 
 extern "C" int b2_gemm_bf16(const void* x, const void* w, void* y, const void* residual, int M, int N, int K,
-                            int64_t ldx, int64_t ldw, int64_t ldy, int epilogue, int config, void* workspace,
+                            int64_t ldx, int64_t ldw, int64_t ldy, int epilogue, const B2EpiAct* act, int config, void* workspace,
                             int64_t workspace_bytes, Status* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
+  if (epilogue < B2_EPI_NONE || epilogue > B2_EPI_F32 || (epilogue == B2_EPI_SOFTCAP && (act == nullptr || !(act->cap > 0.0f)))) return -kBadArgument;
   if (K <= 0 || K % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0) return -kBadArgument;
   Config c = choose_config(M, N, K, epilogue);
   if (config != 0) {
@@ -397,6 +422,7 @@ extern "C" int b2_gemm_bf16(const void* x, const void* w, void* y, const void* r
   ep.M = M;
   ep.N = N;
   ep.mode = epilogue;
+  ep.act = act != nullptr ? *act : kPlainAct;
   if (c.splits > 1) {
     const int64_t counters_bytes = 65536 * 4;
     // P is the 128-row operand: W rows when swapped, X rows otherwise
@@ -527,6 +553,7 @@ extern "C" int b2_gemm_bf16_noalloc(const void* x, const void* w, void* y, int M
   ep.M = M;
   ep.N = N;
   ep.mode = B2_EPI_NONE;
+  ep.act = kPlainAct;
   ep.counters = static_cast<uint32_t*>(scratch);
   ep.workspace = reinterpret_cast<float*>(static_cast<char*>(scratch) + kNoallocCounterBytes);
 #define B2_LAUNCH_NA(BN_, SWAP_) return launch<BN_, SWAP_>(x, w, M, N, K, ldx, ldw, c.splits, false, ep, d->status, stream)

@@ -18,6 +18,7 @@
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 
+#include "b2/act.cuh"
 #include "b2/api.h"
 #include "b2/launch.h"
 #include "b2/config.h"
@@ -47,7 +48,8 @@ struct PairParams {
   int64_t ldy;
   int M, N, num_kb;
   int m_tiles, n_tiles;   // 256-row and 256-column tiles
-  int swiglu;             // 1: W rows alternate 16 gate / 16 up rows; y[M, N / 2] = silu(gate) * up
+  int mode;               // B2Epilogue; SWIGLU: W rows alternate 16 gate / 16 up rows and y is [M, N / 2]
+  B2EpiAct act;
 };
 
 // Tile order: groups of 8 row tiles, column tiles varying slowest inside a group, so that the pairs running at the
@@ -206,7 +208,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
         ptx::tmem_ld_32x32(taddr + c * 32, r);
         ptx::tc_wait_ld();
         const int n0 = nt * kPairBN + c * 32;
-        if (p.swiglu) {
+        if (p.mode == B2_EPI_SWIGLU) {
           // columns [n0, n0 + 16) are gate values, [n0 + 16, n0 + 32) the matching up values: 16 outputs
           if (m < p.M && n0 < p.N) {
             __nv_bfloat16* dst = p.y + static_cast<int64_t>(m) * p.ldy + (n0 >> 1);
@@ -214,7 +216,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
             for (int g = 0; g < 2; ++g) {
               float o[8];
 #pragma unroll
-              for (int i = 0; i < 8; ++i) o[i] = ptx::silu(__uint_as_float(r[g * 8 + i])) * __uint_as_float(r[16 + g * 8 + i]);
+              for (int i = 0; i < 8; ++i) o[i] = glu(p.act, __uint_as_float(r[g * 8 + i]), __uint_as_float(r[16 + g * 8 + i]));
               uint4 pk;
               pk.x = ptx::pack_bf16x2(o[0], o[1]);
               pk.y = ptx::pack_bf16x2(o[2], o[3]);
@@ -224,6 +226,10 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
             }
           }
         } else if (m < p.M) {
+          if (p.mode == B2_EPI_RELU2) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(relu2(__uint_as_float(r[i])));
+          }
           __nv_bfloat16* dst = p.y + static_cast<int64_t>(m) * p.ldy + n0;
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
@@ -256,7 +262,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_c
 
 template <int BN>
 int launch_pair(const void* x, const void* w, void* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy, int epilogue,
-                Status* status, cudaStream_t stream) {
+                const B2EpiAct* act, Status* status, cudaStream_t stream) {
   using Cfg = PairCfg<BN>;
   CUtensorMap tx, tw;
   if (!make_tmap_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, x, M, K, ldx * 2, 128, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
@@ -270,7 +276,8 @@ int launch_pair(const void* x, const void* w, void* y, int M, int N, int K, int6
   p.num_kb = (K + 63) / 64;
   p.m_tiles = (M + 255) / 256;
   p.n_tiles = (N + BN - 1) / BN;
-  p.swiglu = epilogue == B2_EPI_SWIGLU ? 1 : 0;
+  p.mode = epilogue;
+  p.act = act != nullptr ? *act : kPlainAct;
   static DeviceOnce attr_once;
   if (const int rc = attr_once.run([&] {
         cudaError_t e = cudaFuncSetAttribute(gemm_bf16_pair_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::kSmem);
@@ -288,16 +295,16 @@ int launch_pair(const void* x, const void* w, void* y, int M, int N, int K, int6
 
 using namespace b2;
 
-// Y = X W^T on CTA pairs (epilogue B2_EPI_NONE, or B2_EPI_SWIGLU with the 16-row interleaved gate/up weight and
+// Y = X W^T on CTA pairs (epilogue B2_EPI_NONE, B2_EPI_RELU2, or B2_EPI_SWIGLU with the 16-row interleaved gate/up weight and
 // y [M, N / 2]); tiles of 256 rows x `bn` columns, bn = 256 or 128. K a multiple of 8; N a multiple of 8; ldx, ldw,
 // ldy multiples of 8 elements. Any M and N are accepted (edges are zero-filled on load and clipped on store).
 extern "C" int b2_gemm_bf16_pair(const void* x, const void* w, void* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,
-                                 int epilogue, int bn, Status* status, cudaStream_t stream) {
+                                 int epilogue, const B2EpiAct* act, int bn, Status* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8 != 0 || N % 8 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || ldy % 8 != 0) return -kBadArgument;
-  if (epilogue != B2_EPI_NONE && epilogue != B2_EPI_SWIGLU) return -kBadArgument;
+  if (epilogue != B2_EPI_NONE && epilogue != B2_EPI_SWIGLU && epilogue != B2_EPI_RELU2) return -kBadArgument;
   if (epilogue == B2_EPI_SWIGLU && N % 32 != 0) return -kBadArgument;
-  if (bn == 128) return launch_pair<128>(x, w, y, M, N, K, ldx, ldw, ldy, epilogue, status, stream);
-  if (bn == 0 || bn == 256) return launch_pair<256>(x, w, y, M, N, K, ldx, ldw, ldy, epilogue, status, stream);
+  if (bn == 128) return launch_pair<128>(x, w, y, M, N, K, ldx, ldw, ldy, epilogue, act, status, stream);
+  if (bn == 0 || bn == 256) return launch_pair<256>(x, w, y, M, N, K, ldx, ldw, ldy, epilogue, act, status, stream);
   return -kBadArgument;
 }

@@ -6,10 +6,14 @@
 // i.e. one 16-row MMA tile against a 576-wide key that doubles as a 512-wide value: every cache byte is read
 // once and used twice.
 //
-// CTA = 4 warps on one (KV split, head group, sequence). A 32-token tile (36 KB) arrives as nine SWIZZLE_128B
-// TMA boxes through a 3-stage mbarrier ring. The 576-wide dot product is split four ways across the warps and
-// summed through shared memory (one __syncthreads per tile, parity double-buffered); each warp then owns 128
-// of the 512 output columns, so the f32 accumulator is 64 registers per thread.
+// The kernel is a template over the latent and rope widths: 512 + 64 as above, or a latent of 64 ... 1024 columns without a
+// rotated part.
+//
+// CTA = 4 warps on one (KV split, head group, sequence). A 32-token tile (36 KB at 512 + 64) arrives as SWIZZLE_128B
+// TMA boxes of 64 columns through a 2- or 3-stage mbarrier ring (pages below 32 tokens: one set of boxes per page). The
+// dot product is split four ways across the warps and summed through shared memory (one __syncthreads per tile, parity
+// double-buffered); each warp then owns a quarter of the output columns, so the f32 accumulator of a 512-wide latent is
+// 64 registers per thread.
 //
 // A "row group" (grid z) is one query token: its 16 heads, the context length it may see and the block table of
 // its sequence. In decode there is one row group per sequence. A prefill chunk contributes one row group per
@@ -21,6 +25,7 @@
 #include <cuda.h>
 #include <cuda_bf16.h>
 #include "b2/api.h"
+#include "b2/config.h"
 #include "b2/launch.h"
 #include "b2/ptx.cuh"
 #include "b2/tma.h"
@@ -28,10 +33,16 @@
 namespace b2 {
 namespace {
 
-constexpr int kLat = 512, kRope = 64, kRow = kLat + kRope;  // 576
 constexpr int BN = 32;
-constexpr int kSub = kRow / 64;                 // 9 boxes of 64 columns
-constexpr int kTileBytes = kSub * BN * 128;     // 36864
+template <int LAT, int ROPE>
+struct LatentShape {
+  static constexpr int kRow = LAT + ROPE;                 // elements of a cache row
+  static constexpr int kSub = kRow / 64;                  // boxes of 64 columns
+  static constexpr int kTileBytes = kSub * BN * 128;      // 36864 at 512 + 64
+  static constexpr int kSteps = kRow / 64;                // 16-wide steps of one warp's quarter of the dot product
+  static constexpr int kCols = LAT / 4;                   // output columns of one warp
+  static constexpr int smem(int stages) { return stages * kTileBytes + 16 * kRow * 2 + 2 * 4 * 16 * 32 * 4 + 64 + 1024; }
+};
 
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
@@ -53,13 +64,15 @@ __device__ __forceinline__ uint32_t kv_addr(uint32_t base, int row, int chunk) {
 // ldmatrix / mma / barrier latency. Measured against the three-stage ring (146 KB, one CTA per SM, one warp per
 // scheduler, tensor pipe 11 % active): prefill rows 612 -> 408 us for 8 x 512 tokens, decode 45.9 -> 35.7 us for
 // 64 sequences x 768 tokens. Two is therefore the default for both; B2_MLA_STAGES=3 selects the deep ring.
-template <int STAGES>
-__global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
+template <int LAT, int ROPE, int STAGES>
+__global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_decode_kernel(
     const __grid_constant__ CUtensorMap tmap_kv, const __nv_bfloat16* __restrict__ q_lat,
     const __nv_bfloat16* __restrict__ q_rope, __nv_bfloat16* __restrict__ out_lat, const int32_t* __restrict__ ctx_lens,
     const int32_t* __restrict__ block_tables, const int32_t* __restrict__ row_seq, float* __restrict__ workspace,
-    int max_blocks, int n_heads, int page_size, int num_splits, float scale_log2, int64_t num_pages, int64_t q_lat_stride,
+    int max_blocks, int n_heads, int page_size, int box_rows, int num_splits, float scale_log2, int64_t num_pages, int64_t q_lat_stride,
     int64_t q_rope_stride, Status* status) {
+  using S = LatentShape<LAT, ROPE>;
+  constexpr int kLat = LAT, kRope = ROPE, kRow = S::kRow, kSub = S::kSub, kTileBytes = S::kTileBytes, kSteps = S::kSteps, kCols = S::kCols;
   extern __shared__ uint8_t smem_raw[];
   __shared__ int sh_fail;  // set by any thread whose wait ran out; read after the per-tile barrier so all agree
   const uint32_t sbase = (ptx::smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -90,16 +103,18 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
     ptx::fence_mbar_init();
   }
   auto issue = [&](int i) {
-    const int pos = (tile_begin + i) * BN;
-    int64_t page = table[pos / page_size];
-    if (!B2_ASSERT(status, page >= 0 && page < num_pages, kSiteKvIndex, page, num_pages)) page = 0;
-    const int row = static_cast<int>(page * page_size + pos % page_size);
     const int s = i % STAGES;
     const uint32_t bar = bar0 + 8 * s;
     ptx::mbar_arrive_expect_tx(bar, kTileBytes);
+    for (int r0 = 0; r0 < BN; r0 += box_rows) {     // one turn unless a page holds fewer tokens than a tile
+      const int pos = min((tile_begin + i) * BN + r0, (ctx - 1) / box_rows * box_rows);   // past the context: any valid rows
+      int64_t page = table[pos / page_size];
+      if (!B2_ASSERT(status, page >= 0 && page < num_pages, kSiteKvIndex, page, num_pages)) page = 0;
+      const int row = static_cast<int>(page * page_size + pos % page_size);
 #pragma unroll
-    for (int c = 0; c < kSub; ++c)
-      ptx::tma_load_2d(sbase + s * kTileBytes + c * (BN * 128), &tmap_kv, bar, c * 64, row, ptx::kEvictFirst);
+      for (int c = 0; c < kSub; ++c)
+        ptx::tma_load_2d(sbase + s * kTileBytes + c * (BN * 128) + r0 * 128, &tmap_kv, bar, c * 64, row, ptx::kEvictFirst);
+    }
   };
   // stage Q: row r = head head0 + r; columns [0, 512) from q_lat, [512, 576) from q_rope; rows >= `rows` are zero
   for (int i = threadIdx.x; i < 16 * (kRow / 8); i += blockDim.x) {
@@ -107,7 +122,7 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
     uint4 v = make_uint4(0, 0, 0, 0);
     if (r < rows) {
       // row strides in elements: the two query parts may be column slices of one wider projection output
-      v = c < kLat / 8 ? reinterpret_cast<const uint4*>(q_lat + seq * q_lat_stride + static_cast<int64_t>(head0 + r) * kLat)[c]
+      v = ROPE == 0 || c < kLat / 8 ? reinterpret_cast<const uint4*>(q_lat + seq * q_lat_stride + static_cast<int64_t>(head0 + r) * kLat)[c]
                        : reinterpret_cast<const uint4*>(q_rope + seq * q_rope_stride + static_cast<int64_t>(head0 + r) * kRope)[c - kLat / 8];
     }
     // plain row-major with an XOR on the low 3 chunk bits to spread ldmatrix rows over banks
@@ -117,17 +132,17 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
   if (threadIdx.x == 0)
     for (int i = 0; i < STAGES - 1 && i < n_tiles; ++i) issue(i);
 
-  // this warp's slice of the 576-wide dot product: 9 k-steps of 16
-  uint32_t qf[9][4];
+  // this warp's slice of the dot product in k-steps of 16
+  uint32_t qf[kSteps][4];
 #pragma unroll
-  for (int kk = 0; kk < 9; ++kk) {
-    const int row = lane & 15, chunk = (warp * 9 + kk) * 2 + (lane >> 4);
+  for (int kk = 0; kk < kSteps; ++kk) {
+    const int row = lane & 15, chunk = (warp * kSteps + kk) * 2 + (lane >> 4);
     const uint32_t a = q_sm + static_cast<uint32_t>((row * (kRow / 8) + ((chunk & ~7) | ((chunk & 7) ^ (row & 7)))) * 16);
     ldsm_x4(a, qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3]);
   }
-  float o[16][4];
+  float o[kCols / 8][4];
 #pragma unroll
-  for (int d = 0; d < 16; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.0f;
+  for (int d = 0; d < kCols / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.0f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
   const int g = lane >> 2, t4 = lane & 3;
   const int max_lo = g < rows ? ctx - 1 : -1, max_hi = g + 8 < rows ? ctx - 1 : -1;
@@ -141,18 +156,18 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
     }
     const uint32_t kb = sbase + st * kTileBytes;
     const int kv0 = (tile_begin + i) * BN;
-    // ---- partial S over this warp's 144 dims ----
+    // ---- partial S over this warp's quarter of the dims ----
     float s[4][4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
     {
 #pragma unroll
-      for (int kk = 0; kk < 9; ++kk) {
+      for (int kk = 0; kk < kSteps; ++kk) {
 #pragma unroll
         for (int jp = 0; jp < 2; ++jp) {
           uint32_t b0, b1, b2, b3;
           const int row = jp * 16 + (lane & 7) + ((lane >> 4) << 3);
-          const int chunk = (warp * 9 + kk) * 2 + ((lane >> 3) & 1);
+          const int chunk = (warp * kSteps + kk) * 2 + ((lane >> 3) & 1);
           ldsm_x4(kv_addr(kb, row, chunk), b0, b1, b2, b3);
           mma16816(s[2 * jp], qf[kk], b0, b1);
           mma16816(s[2 * jp + 1], qf[kk], b2, b3);
@@ -214,20 +229,20 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
     l[0] = l[0] * corr_lo + sum_lo;
     l[1] = l[1] * corr_hi + sum_hi;
 #pragma unroll
-    for (int d = 0; d < 16; ++d) {
+    for (int d = 0; d < kCols / 8; ++d) {
       o[d][0] *= corr_lo; o[d][1] *= corr_lo;
       o[d][2] *= corr_hi; o[d][3] *= corr_hi;
     }
-    // ---- O[:, 128 w : 128 w + 128] += P . C ----
+    // ---- O[:, this warp's columns] += P . C ----
     const int valid = ctx - kv0;  // rows of the tile inside the context; beyond that the page holds stale data
 #pragma unroll
     for (int kk = 0; kk < 2; ++kk) {
       const uint32_t a[4] = {pf[2 * kk][0], pf[2 * kk][1], pf[2 * kk + 1][0], pf[2 * kk + 1][1]};
 #pragma unroll
-      for (int dp = 0; dp < 8; ++dp) {
+      for (int dp = 0; dp < kCols / 16; ++dp) {
         uint32_t b0, b1, b2, b3;
         const int row = kk * 16 + (lane & 7) + (((lane >> 3) & 1) << 3);
-        const int chunk = warp * 16 + dp * 2 + (lane >> 4);
+        const int chunk = warp * (kCols / 8) + dp * 2 + (lane >> 4);
         ldsm_x4_t(kv_addr(kb, row, chunk), b0, b1, b2, b3);
         if (valid < BN) {
           // P is exactly zero for masked tokens, but 0 * NaN is NaN: blank operand rows past the context.
@@ -257,15 +272,15 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
     const int64_t h = static_cast<int64_t>(seq) * n_heads + head0 + r;
     if (num_splits == 1) {
       const float inv = l[half] > 0.0f ? 1.0f / l[half] : 0.0f;
-      __nv_bfloat16* dst = out_lat + h * kLat + warp * 128;
+      __nv_bfloat16* dst = out_lat + h * kLat + warp * kCols;
 #pragma unroll
-      for (int d = 0; d < 16; ++d)
+      for (int d = 0; d < kCols / 8; ++d)
         *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * t4) = ptx::pack_bf16x2(o[d][half * 2] * inv, o[d][half * 2 + 1] * inv);
     } else {
       float* dst = workspace + (h * num_splits + split) * (kLat + 2);
 #pragma unroll
-      for (int d = 0; d < 16; ++d)
-        *reinterpret_cast<float2*>(dst + warp * 128 + d * 8 + 2 * t4) = make_float2(o[d][half * 2], o[d][half * 2 + 1]);
+      for (int d = 0; d < kCols / 8; ++d)
+        *reinterpret_cast<float2*>(dst + warp * kCols + d * 8 + 2 * t4) = make_float2(o[d][half * 2], o[d][half * 2 + 1]);
       if (warp == 0 && t4 == 0) {
         dst[kLat] = m[half];
         dst[kLat + 1] = l[half];
@@ -274,6 +289,7 @@ __global__ void __launch_bounds__(128, STAGES == 2 ? 2 : 1) mla_decode_kernel(
   }
 }
 
+template <int kLat>
 __global__ void mla_reduce_kernel(const float* __restrict__ workspace, __nv_bfloat16* __restrict__ out, int num_splits, int total) {
   constexpr int RS = kLat + 2;
   const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -309,13 +325,62 @@ __global__ void mla_rows_meta_kernel(const int32_t* __restrict__ cu_q, const int
   }
 }
 
+template <int LAT, int ROPE>
+int launch_latent(const void* q_lat, const void* q_rope, const void* kv_cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
+                  const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int page_size, int num_splits, float scale,
+                  int64_t num_pages, int64_t q_lat_stride, int64_t q_rope_stride, Status* status, cudaStream_t stream) {
+  using S = LatentShape<LAT, ROPE>;
+  if (rows <= 0) return 0;
+  if (n_heads <= 0 || page_size <= 0 || page_size % 8 != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr)) return -kBadArgument;
+  // 16-byte vector loads of the query rows
+  if (q_lat_stride % 8 != 0 || (reinterpret_cast<uintptr_t>(q_lat) & 15) != 0) return -kBadArgument;
+  if (ROPE > 0 && (q_rope_stride % 8 != 0 || (reinterpret_cast<uintptr_t>(q_rope) & 15) != 0)) return -kBadArgument;
+  const int box_rows = page_size % BN == 0 ? BN : page_size % 16 == 0 ? 16 : 8;    // a box lies inside one page
+  CUtensorMap tk;
+  const uint64_t cache_rows = static_cast<uint64_t>(num_pages) * page_size;
+  if (!make_tmap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, kv_cache, cache_rows, S::kRow, S::kRow * 2, box_rows, 64, CU_TENSOR_MAP_SWIZZLE_128B))
+    return -kBadArgument;
+  // two-stage ring (two CTAs per SM) unless B2_MLA_STAGES=3 asks for the deep one
+  static const int forced = [] {
+    const char* e = getenv("B2_MLA_STAGES");
+    return e != nullptr ? atoi(e) : 0;
+  }();
+  constexpr bool kDeep = S::smem(3) <= kMaxSmemPerCta;
+  const int stages = kDeep && forced == 3 ? 3 : 2;
+  auto kern = stages == 2 ? mla_decode_kernel<LAT, ROPE, 2> : mla_decode_kernel<LAT, ROPE, kDeep ? 3 : 2>;
+  static DeviceOnce attr_once[2];
+  if (const int rc = attr_once[stages - 2].max_smem(kern, S::smem(stages))) return rc;
+  // grid z is limited to 65535: larger row counts go out in slices
+  constexpr int kMaxZ = 65535;
+  for (int r0 = 0; r0 < rows; r0 += kMaxZ) {
+    const int n = rows - r0 < kMaxZ ? rows - r0 : kMaxZ;
+    dim3 grid(num_splits, (n_heads + 15) / 16, n);
+    float* ws = workspace == nullptr ? nullptr : workspace + static_cast<int64_t>(r0) * n_heads * num_splits * (LAT + 2);
+    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(out_lat) + static_cast<int64_t>(r0) * n_heads * LAT;
+    kern<<<grid, 128, S::smem(stages), stream>>>(
+        tk, static_cast<const __nv_bfloat16*>(q_lat) + r0 * q_lat_stride, ROPE == 0 ? nullptr : static_cast<const __nv_bfloat16*>(q_rope) + r0 * q_rope_stride,
+        out, row_ctx + r0, row_seq == nullptr ? block_tables + static_cast<int64_t>(r0) * max_blocks : block_tables,
+        row_seq == nullptr ? nullptr : row_seq + r0, ws, max_blocks, n_heads, page_size, box_rows,
+        num_splits, scale * ptx::kLog2e, num_pages, q_lat_stride, q_rope_stride, status);
+    if (num_splits > 1) {
+      const int total = n * n_heads;
+      mla_reduce_kernel<LAT><<<(total + 3) / 4, 128, 0, stream>>>(ws, out, num_splits, total);
+    }
+  }
+  return last_launch_rc();
+}
+
 }  // namespace
 }  // namespace b2
 
 using namespace b2;
 
+extern "C" int64_t b2_latent_attend_workspace(int rows, int n_heads, int latent, int num_splits) {
+  return static_cast<int64_t>(rows) * n_heads * num_splits * (latent + 2) * 4;
+}
+
 extern "C" int64_t b2_mla_decode_workspace(int batch, int n_heads, int num_splits) {
-  return static_cast<int64_t>(batch) * n_heads * num_splits * (kLat + 2) * 4;
+  return b2_latent_attend_workspace(batch, n_heads, 512, num_splits);
 }
 
 extern "C" int b2_mla_rows_meta(const int32_t* cu_q, const int32_t* ctx_lens, int num_seqs, int32_t* row_ctx, int32_t* row_seq,
@@ -330,44 +395,25 @@ extern "C" int b2_mla_attend_bf16(const void* q_lat, const void* q_rope, const v
                                   int rows, int max_blocks, int n_heads, int page_size, int num_splits, float scale,
                                   int64_t num_pages, int64_t q_lat_stride, int64_t q_rope_stride, Status* status,
                                   cudaStream_t stream) {
-  if (rows <= 0) return 0;
-  if (n_heads <= 0 || page_size % BN != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr)) return -kBadArgument;
-  // 16-byte vector loads of the query rows
-  if (q_lat_stride % 8 != 0 || q_rope_stride % 8 != 0 || (reinterpret_cast<uintptr_t>(q_lat) & 15) != 0 ||
-      (reinterpret_cast<uintptr_t>(q_rope) & 15) != 0)
-    return -kBadArgument;
-  CUtensorMap tk;
-  const uint64_t cache_rows = static_cast<uint64_t>(num_pages) * page_size;
-  if (!make_tmap_2d(&tk, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, kv_cache, cache_rows, kRow, kRow * 2, BN, 64, CU_TENSOR_MAP_SWIZZLE_128B))
-    return -kBadArgument;
-  // two-stage ring (two CTAs per SM) unless B2_MLA_STAGES=3 asks for the deep one
-  static const int forced = [] {
-    const char* e = getenv("B2_MLA_STAGES");
-    return e != nullptr ? atoi(e) : 0;
-  }();
-  const int stages = forced == 3 ? 3 : 2;
-  const int SMEM = stages * kTileBytes + 16 * kRow * 2 + 2 * 4 * 16 * 32 * 4 + 64 + 1024;
-  auto kern = stages == 2 ? mla_decode_kernel<2> : mla_decode_kernel<3>;
-  static DeviceOnce attr_once[2];
-  if (const int rc = attr_once[stages - 2].max_smem(kern, SMEM)) return rc;
-  // grid z is limited to 65535: larger row counts go out in slices
-  constexpr int kMaxZ = 65535;
-  for (int r0 = 0; r0 < rows; r0 += kMaxZ) {
-    const int n = rows - r0 < kMaxZ ? rows - r0 : kMaxZ;
-    dim3 grid(num_splits, (n_heads + 15) / 16, n);
-    float* ws = workspace == nullptr ? nullptr : workspace + static_cast<int64_t>(r0) * n_heads * num_splits * (kLat + 2);
-    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(out_lat) + static_cast<int64_t>(r0) * n_heads * kLat;
-    kern<<<grid, 128, SMEM, stream>>>(
-        tk, static_cast<const __nv_bfloat16*>(q_lat) + r0 * q_lat_stride, static_cast<const __nv_bfloat16*>(q_rope) + r0 * q_rope_stride,
-        out, row_ctx + r0, row_seq == nullptr ? block_tables + static_cast<int64_t>(r0) * max_blocks : block_tables,
-        row_seq == nullptr ? nullptr : row_seq + r0, ws, max_blocks, n_heads, page_size,
-        num_splits, scale * ptx::kLog2e, num_pages, q_lat_stride, q_rope_stride, status);
-    if (num_splits > 1) {
-      const int total = n * n_heads;
-      mla_reduce_kernel<<<(total + 3) / 4, 128, 0, stream>>>(ws, out, num_splits, total);
-    }
+  return launch_latent<512, 64>(q_lat, q_rope, kv_cache, out_lat, row_ctx, block_tables, row_seq, workspace, rows, max_blocks, n_heads, page_size,
+                                num_splits, scale, num_pages, q_lat_stride, q_rope_stride, status, stream);
+}
+
+extern "C" int b2_latent_attend_bf16(const void* q_lat, const void* cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
+                                     const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int latent, int page_size,
+                                     int num_splits, float scale, int64_t num_pages, int64_t q_lat_stride, Status* status, cudaStream_t stream) {
+#define B2_LATENT(LAT_)                                                                                                                        \
+  return launch_latent<LAT_, 0>(q_lat, nullptr, cache, out_lat, row_ctx, block_tables, row_seq, workspace, rows, max_blocks, n_heads, page_size, \
+                                num_splits, scale, num_pages, q_lat_stride, 0, status, stream)
+  switch (latent) {
+    case 64: B2_LATENT(64);
+    case 128: B2_LATENT(128);
+    case 256: B2_LATENT(256);
+    case 512: B2_LATENT(512);
+    case 1024: B2_LATENT(1024);
+    default: return -kBadArgument;
   }
-  return last_launch_rc();
+#undef B2_LATENT
 }
 
 extern "C" int b2_mla_decode_bf16(const void* q_lat, const void* q_rope, const void* kv_cache, void* out_lat,
@@ -375,6 +421,6 @@ extern "C" int b2_mla_decode_bf16(const void* q_lat, const void* q_rope, const v
                                   int max_blocks, int n_heads, int page_size, int num_splits, float scale,
                                   int64_t num_pages, Status* status, cudaStream_t stream) {
   return b2_mla_attend_bf16(q_lat, q_rope, kv_cache, out_lat, ctx_lens, block_tables, nullptr, workspace, batch, max_blocks,
-                            n_heads, page_size, num_splits, scale, num_pages, static_cast<int64_t>(n_heads) * kLat,
-                            static_cast<int64_t>(n_heads) * kRope, status, stream);
+                            n_heads, page_size, num_splits, scale, num_pages, static_cast<int64_t>(n_heads) * 512,
+                            static_cast<int64_t>(n_heads) * 64, status, stream);
 }

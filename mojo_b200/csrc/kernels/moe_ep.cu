@@ -20,6 +20,7 @@
 #include "b2/launch.h"
 #include "b2/ep.h"
 #include "b2/gemm_tc.cuh"
+#include "b2/moe_gemm.cuh"
 #include "b2/ptx.cuh"
 #include "b2/tma.h"
 #include "b2/vec.cuh"
@@ -188,59 +189,14 @@ struct GroupedSched {
     // one DeepSeek-V2-Lite layer of 4096 tokens and lost: 951 us against 891 us for the whole layer.
     u.pb = r % p_blocks;          // weight-row tile
     u.qb = r / p_blocks;          // token tile inside the expert
-    u.split = e;                  // carries the expert index to the epilogue
+    u.split = e;
+    u.nsplit = min(bn, min(static_cast<int>(counts[e]), cap) - u.qb * bn);   // rows of the tile that hold tokens
     u.tile = w;
     u.kb0 = 0;
     u.kb1 = num_kb;
     u.p_coord = e * n_rows + u.pb * 128;
     u.q_coord = e * cap + u.qb * bn;
     return u;
-  }
-};
-
-struct GroupedEpiParams {
-  __nv_bfloat16* y;       // [e_local][cap][ldy]
-  int64_t ldy;
-  const uint32_t* counts;
-  int cap, n_rows;
-  int swiglu;
-};
-
-template <int BN>
-struct GroupedEpilogue {
-  static constexpr int CH = BN >= 32 ? 32 : 16;
-  GroupedEpiParams p;
-  __device__ __forceinline__ void operator()(const gemm::WorkUnit& u, uint32_t taddr, int quarter, int lane, uint32_t*,
-                                             Status*) const {
-    const int e = u.split;
-    const int cnt = min(static_cast<int>(p.counts[e]), p.cap);
-    const int p_local = quarter * 32 + lane;
-    const int n = u.pb * 128 + p_local;
-    __nv_bfloat16* base = p.y + static_cast<int64_t>(e) * p.cap * p.ldy;
-#pragma unroll 1
-    for (int c = 0; c < BN / CH; ++c) {
-      uint32_t r[CH];
-      if constexpr (CH == 32) ptx::tmem_ld_32x32(taddr + c * CH, r);
-      else ptx::tmem_ld_32x16(taddr + c * CH, r);
-      ptx::tc_wait_ld();
-      const int m0 = u.qb * BN + c * CH;
-      if (p.swiglu) {
-        const int out_col = (u.pb * 128 + (p_local & ~31)) / 2 + (lane & 15);
-#pragma unroll
-        for (int j = 0; j < CH; ++j) {
-          const float v = __uint_as_float(r[j]);
-          const float other = __shfl_xor_sync(0xffffffffu, v, 16);
-          if (lane < 16 && n < p.n_rows && m0 + j < cnt)
-            base[static_cast<int64_t>(m0 + j) * p.ldy + out_col] = __float2bfloat16(ptx::silu(v) * other);
-        }
-      } else if (n < p.n_rows) {
-#pragma unroll
-        for (int j = 0; j < CH; ++j) {
-          if (m0 + j >= cnt) break;
-          base[static_cast<int64_t>(m0 + j) * p.ldy + n] = __float2bfloat16(__uint_as_float(r[j]));
-        }
-      }
-    }
   }
 };
 
@@ -256,16 +212,10 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_cons
                            static_cast<int>(blockIdx.x), static_cast<int>(gridDim.x));
 }
 
-constexpr int stages_for(int bn) {
-  const int stage = 128 * 64 * 2 + bn * 64 * 2;
-  int s = (200 * 1024) / stage;
-  return s > 10 ? 10 : s;
-}
-
 template <int BN>
 int launch_grouped(const void* x, const void* w, const uint32_t* counts, void* y, int e_local, int cap, int N, int K,
                    int64_t ldy, int swiglu, Status* status, cudaStream_t stream) {
-  constexpr int STAGES = stages_for(BN);
+  constexpr int STAGES = grouped_stages_for(BN);
   using L = gemm::SmemLayout<BN, STAGES>;
   CUtensorMap tw, tx;
   if (!make_tmap_2d(&tw, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, w, static_cast<uint64_t>(e_local) * N, K, static_cast<uint64_t>(K) * 2, 128, 64,
@@ -281,7 +231,7 @@ int launch_grouped(const void* x, const void* w, const uint32_t* counts, void* y
   sched.num_kb = (K + 63) / 64;
   sched.bn = BN;
   sched.p_blocks = (N + 127) / 128;
-  GroupedEpiParams ep{static_cast<__nv_bfloat16*>(y), ldy, counts, cap, N, swiglu};
+  const GroupedEpiParams ep{static_cast<__nv_bfloat16*>(y), ldy, N, swiglu ? B2_EPI_SWIGLU : B2_EPI_NONE, kPlainAct};
   auto kern = moe_grouped_kernel<BN, STAGES>;
   static DeviceOnce attr_once;
   if (const int rc = attr_once.run([&] {

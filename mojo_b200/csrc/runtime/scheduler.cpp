@@ -70,6 +70,8 @@ void Scheduler::emit(Request& r, int64_t n, Batch* b) {
   for (int64_t i = 0; i < n; ++i) {
     b->token_ids.push_back(r.tokens[start + i]);
     b->positions.push_back(static_cast<int32_t>(start + i));
+    const int32_t prev = start + i > 0 ? r.tokens[start + i - 1] : -1;
+    b->prev_tokens.push_back(start + i > 0 && prev < 0 ? -2 : prev);   // a placeholder (-1) must not read as "first token"
     b->slots.push_back(kv_->slot(r.id, start + i));
   }
   b->cu_q.push_back(static_cast<int32_t>(b->token_ids.size()));

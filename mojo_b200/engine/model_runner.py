@@ -85,7 +85,11 @@ class ModelRunner:
         max_blocks = (cfg.max_model_len + cfg.page_size - 1) // cfg.page_size
         # models with recurrent state also need the sequence of every row, and rows and state banks of every sequence
         self.has_state = bool(getattr(model, "recurrent_state", False))
-        nbytes = cfg.max_num_batched_tokens * 36 + cfg.max_num_seqs * (max_blocks * 4 + 96) + (1 << 16)
+        # models whose embedding also looks at the token before each row
+        self.needs_prev = bool(getattr(model, "needs_prev_tokens", False))
+        nbytes = cfg.max_num_batched_tokens * 40 + cfg.max_num_seqs * (max_blocks * 4 + 96) + (1 << 16)
+        if hasattr(model, "plan_latent_prefill"):      # scratch pages of 128 tokens of every context in a step, and their tables
+            nbytes += cfg.max_num_seqs * (cfg.max_model_len // 128 + 1) * 12
         self.staging = _Staging(nbytes, self.device)
         self.max_blocks = max_blocks
         self.h2d_bytes = 0
@@ -258,6 +262,15 @@ class ModelRunner:
         self.ids_events[slot].record()
         return StepHandle(S, ids, slot=slot, event=self.ids_events[slot])
 
+    @staticmethod
+    def prev_tokens(batch) -> np.ndarray:
+        """The token before each row. Under pipelined stepping it is always known by now: only the newest token of a
+        sequence can still be on the device, and nothing follows that one in a step."""
+        prev = batch.prev_tokens
+        if (prev == -2).any():
+            raise RuntimeError("a row follows a token the host has not read back")
+        return prev
+
     def _patch_plan(self, batch, prev):
         """Rows of this batch whose input token is still a placeholder (-1): the token the previous step sampled for that
         sequence, not yet read back by the host. Returns (row indices, indices into the previous step's sampled ids)."""
@@ -315,6 +328,7 @@ class ModelRunner:
         seg_tok = st.put(batch.token_ids, np.int64)
         seg_slot = st.put(batch.slots, np.int64)
         seg_pos = st.put(batch.positions, np.int32)
+        seg_prev = st.put(self.prev_tokens(batch), np.int32) if self.needs_prev else None
         seg_cu = st.put(batch.cu_q, np.int32)
         seg_ctx = st.put(batch.ctx_lens, np.int32)
         seg_bt = st.put(batch.block_tables, np.int32)
@@ -327,8 +341,14 @@ class ModelRunner:
             seg_srows = st.put(np.stack([cu[:-1], cu[1:]], axis=1), np.int32)
             seg_state = st.put(batch.seq_state, np.int32)
         seg_rows = st.put(sample_rows.astype(np.int64), np.int64)
+        expand = None
+        if batch.num_prefill > 0 and hasattr(self.model, "plan_latent_prefill"):
+            expand = self.model.plan_latent_prefill(batch.cu_q, batch.ctx_lens, int(batch.num_decode))
+            if expand is not None:
+                seg_xpages, seg_xtables = st.put(expand[0], np.int32), st.put(expand[1], np.int32)
         seg_work, n_items = None, 0
-        if self.cuda and batch.num_prefill > 0 and getattr(self.model, "supports_static_attention", lambda *_: False)(self.cfg.page_size):
+        if self.cuda and batch.num_prefill > 0 and (
+                expand is not None or getattr(self.model, "supports_static_attention", lambda *_: False)(self.cfg.page_size)):
             # one CTA per (sequence, query tile) of the chunks, longest context first, instead of a padded grid
             work = ops.prefill_work_items(batch.cu_q, batch.ctx_lens, int(batch.num_decode))
             n_items = int(work.shape[0])
@@ -355,7 +375,9 @@ class ModelRunner:
             seq = ops.SeqRows(st.view(seg_rseq, torch.int32), st.view(seg_srows, torch.int32), st.view(seg_state, torch.int32), nd, nd, B - nd)
         meta = ops.AttnMeta(st.view(seg_cu, torch.int32), st.view(seg_ctx, torch.int32), st.view(seg_bt, torch.int32),
                             batch.num_decode, batch.max_q_len, int(ctx_np.max()) if B else 0,
-                            work=st.view(seg_work, torch.int32) if seg_work is not None else None, n_items=n_items, seq=seq)
+                            work=st.view(seg_work, torch.int32) if seg_work is not None else None, n_items=n_items, seq=seq,
+                            prev=st.view(seg_prev, torch.int32) if seg_prev is not None else None,
+                            expand=(st.view(seg_xpages, torch.int32), st.view(seg_xtables, torch.int32)) if expand is not None else None)
         rows = st.view(seg_rows, torch.int64)
         if self.step_events is not None:
             self.step_events[0].record()
@@ -478,13 +500,14 @@ class _DecodeGraph:
         self.runner, self.bb = runner, bb
         mb = runner.max_blocks
         dev = runner.device
-        # host layout: tok i64[bb] | slot i64[bb] | pos i32[bb] | ctx i32[bb] | bt i32[bb * mb] | fix i32[2 bb] | state i32[2 bb]
+        # host layout: tok i64[bb] | slot i64[bb] | pos i32[bb] | ctx i32[bb] | bt i32[bb * mb] | fix i32[2 bb] | state i32[2 bb] | prev i32[bb]
         self.o_tok, self.o_slot = 0, 8 * bb
         self.o_pos, self.o_ctx = 16 * bb, 20 * bb
         self.o_bt = _align(24 * bb)
         self.o_fix = _align(self.o_bt + 4 * bb * mb)      # rows / sources of tokens still on the device (pipelined stepping)
         self.o_state = _align(self.o_fix + 8 * bb)
-        nbytes = self.o_state + 8 * bb
+        self.o_prev = _align(self.o_state + 8 * bb)
+        nbytes = self.o_prev + 4 * bb
         self.host = torch.zeros(nbytes, dtype=torch.uint8, pin_memory=True)
         self.np = self.host.numpy()
         self.dev = torch.zeros(nbytes, dtype=torch.uint8, device=dev)
@@ -505,15 +528,18 @@ class _DecodeGraph:
         self.h_ctx = self.np[self.o_ctx:self.o_ctx + 4 * bb].view(np.int32)
         self.h_bt = self.np[self.o_bt:self.o_bt + 4 * bb * mb].view(np.int32).reshape(bb, mb)
         self.h_state = self.np[self.o_state:self.o_state + 8 * bb].view(np.int32).reshape(bb, 2)
+        self.h_prev = self.np[self.o_prev:self.o_prev + 4 * bb].view(np.int32)
         self.h_slot[:] = -1
         self.h_state[:] = -1
+        self.h_prev[:] = -1
         self.dev.copy_(self.host)
         seq = None
         if runner.has_state:
             row = torch.arange(bb, dtype=torch.int32, device=dev)
             seq = ops.SeqRows(row, torch.stack([row, row + 1], dim=1).contiguous(), d[self.o_state:self.o_state + 8 * bb].view(torch.int32).view(bb, 2),
                               bb, bb, 0)
-        self.meta = ops.AttnMeta(self.cu, self.ctx, self.bt, bb, 1, runner.cfg.max_model_len, seq=seq)
+        prev = d[self.o_prev:self.o_prev + 4 * bb].view(torch.int32) if runner.needs_prev else None
+        self.meta = ops.AttnMeta(self.cu, self.ctx, self.bt, bb, 1, runner.cfg.max_model_len, seq=seq, prev=prev)
         self.logits = None       # the graph's logits, where the forward pass returns them
         model, caches = runner.model, runner.kv_caches
 
@@ -575,6 +601,9 @@ class _DecodeGraph:
         if self.runner.has_state:
             self.h_state[:B] = batch.seq_state
             self.h_state[B:] = -1
+        if self.runner.needs_prev:
+            self.h_prev[:B] = self.runner.prev_tokens(batch)
+            self.h_prev[B:] = -1
         bt = batch.block_tables
         self.h_bt[:B, :bt.shape[1]] = bt
         self.dev.copy_(self.host, non_blocking=True)
@@ -607,6 +636,8 @@ class _MixedGraph:
             off = _align(off + nbytes)
 
         seg("tok", 8 * tb); seg("slot", 8 * tb); seg("pos", 4 * tb)
+        if runner.needs_prev:
+            seg("prev", 4 * tb)
         seg("d_ctx", 4 * max(db, 1)); seg("d_bt", 4 * max(db, 1) * mb)
         seg("p_cu", 4 * (pb + 1)); seg("p_ctx", 4 * pb); seg("p_bt", 4 * pb * mb)
         seg("work", 8 * self.max_items); seg("n_work", 4); seg("rows", 8 * self.sb)
@@ -635,6 +666,9 @@ class _MixedGraph:
                   "work": hv("work", np.int32, (self.max_items, 2)), "n_work": hv("n_work", np.int32), "rows": hv("rows", np.int64),
                   "fix_rows": hv("fix_rows", np.int32), "fix_src": hv("fix_src", np.int32)}
         self.h["slot"][:] = -1
+        if runner.needs_prev:
+            self.h["prev"] = hv("prev", np.int32)
+            self.h["prev"][:] = -1
         if runner.has_state:
             self.h.update(row_seq=hv("row_seq", np.int32), seq_rows=hv("seq_rows", np.int32, (db + pb, 2)), seq_state=hv("seq_state", np.int32, (db + pb, 2)))
             self.h["row_seq"][:] = -1
@@ -650,7 +684,8 @@ class _MixedGraph:
         seq = None
         if runner.has_state:
             seq = ops.SeqRows(dv("row_seq", torch.int32), dv("seq_rows", torch.int32, (db + pb, 2)), dv("seq_state", torch.int32, (db + pb, 2)), db, db, pb)
-        self.meta = ops.AttnMeta(None, None, None, 0, tb, runner.cfg.max_model_len, static=static, seq=seq)
+        self.meta = ops.AttnMeta(None, None, None, 0, tb, runner.cfg.max_model_len, static=static, seq=seq,
+                                 prev=dv("prev", torch.int32) if runner.needs_prev else None)
         model, caches = runner.model, runner.kv_caches
         comm = getattr(model, "comm", None)
 
@@ -698,6 +733,9 @@ class _MixedGraph:
         h["slot"][T:] = -1
         h["pos"][:T] = batch.positions
         h["pos"][T:] = 0
+        if self.runner.needs_prev:
+            h["prev"][:T] = self.runner.prev_tokens(batch)
+            h["prev"][T:] = -1
         ctx, cu, bt = batch.ctx_lens, batch.cu_q, batch.block_tables
         w = bt.shape[1]
         if self.db:

@@ -64,7 +64,7 @@ class _Reader:
 
 
 def load_safetensors_into(model, path: str | Path) -> None:
-    """Fill a model from a checkpoint directory: Llama family or DeepSeek-V2(-Lite) in Hugging Face layout, or Rekudra."""
+    """Fill a model from a checkpoint directory: Llama family or DeepSeek-V2(-Lite) in Hugging Face layout, Rekudra, Rerupel."""
     rd = _Reader(read_safetensors_index(path))
     cfg = model.cfg
     if getattr(cfg, "architecture", "llama") == "deepseek_v2":
@@ -72,6 +72,9 @@ def load_safetensors_into(model, path: str | Path) -> None:
         return
     if cfg.architecture == "rekudra":
         _load_rekudra(model, rd)
+        return
+    if cfg.architecture == "rerupel":
+        _load_rerupel(model, rd)
         return
     model.layers.clear()
     model.load_tensor("embed", rd.get("model.embed_tokens.weight"))
@@ -155,6 +158,15 @@ def _load_rekudra(model, rd: _Reader) -> None:
         model.load_layer(i, {n: rd.get(f"l{i}.{n}") for n in names})
     model.load_tensor("final.norm", rd.get("final.norm"))
     model.load_tensor("head", rd.get("head"))
+
+
+def _load_rerupel(model, rd: _Reader) -> None:
+    """Rerupel names: `embed`, `bigram`, `loop.in`, `final.norm`, and per layer `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`, `l<i>.ls<q>`."""
+    model.layers.clear()
+    for name in model.global_shapes():
+        model.load_tensor(name, rd.get(name))
+    for i, spec in enumerate(model.cfg.layers):
+        model.load_layer(i, {n: rd.get(f"l{i}.{n}") for n in model.tensor_shapes(spec, model.cfg.hidden_size)})
 
 
 def deepseek_v2_state_dict(model) -> dict:

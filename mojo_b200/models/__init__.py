@@ -19,4 +19,8 @@ def build_model(cfg: ModelConfig, device="cpu", dtype=torch.float32, comm=None, 
         from .rekudra import RekudraModel
 
         return RekudraModel(cfg, device, dtype, comm=comm)
+    if cfg.architecture == "rerupel":
+        from .rerupel import RerupelModel
+
+        return RerupelModel(cfg, device, dtype, comm=comm)
     raise ValueError(f"unsupported architecture {cfg.architecture!r}")

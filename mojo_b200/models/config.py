@@ -17,9 +17,42 @@ class RotarySpec:
 
 
 @dataclass
+class ExpertSpec:
+    """Size and constants of one gated feed-forward: min(g, limit), clamp(u, -limit, limit)."""
+    ffn: int = 0
+    limit: float = float("inf")
+
+
+@dataclass
+class MoeSpec:
+    """Mixture of experts of one layer. The shared expert runs for every token."""
+    experts: int = 0
+    top: int = 0
+    scale: float = 1.0                     # on the router's weights
+    expert: ExpertSpec = field(default_factory=ExpertSpec)
+    shared: ExpertSpec | None = None
+
+
+@dataclass
+class LoopSpec:
+    """Layers start .. stop - 1 run `times` times in a row with the same weights."""
+    start: int = 0
+    stop: int = 0
+    times: int = 1
+
+
+@dataclass
+class BigramSpec:
+    """Hashed bigram embedding: row (previous * mul_prev + current * mul_cur) mod buckets."""
+    buckets: int = 0
+    mul_prev: int = 0
+    mul_cur: int = 0
+
+
+@dataclass
 class LayerSpec:
-    """One layer of a decoder whose layers differ: which mixer it has, the mixer's sizes, and its feed-forward width."""
-    mixer: str = "attention"               # "attention" | "channel_delta"
+    """One layer of a decoder whose layers differ: which mixer it has, the mixer's sizes, and its feed-forward."""
+    mixer: str = "attention"               # "attention" | "channel_delta" | "latent_attention"
     heads: int = 0
     kv_heads: int = 0
     dim: int = 0                           # query / key size of a head
@@ -31,11 +64,13 @@ class LayerSpec:
     ffn: int = 0                           # feed-forward width (0: the layer has no feed-forward)
     decay_rank: int = 0                    # delta rule: ranks of the decay and gate projections (0: taken from the checkpoint)
     gate_rank: int = 0
+    kv_rank: int = 0                       # latent attention: size of the cached latent
+    moe: MoeSpec | None = None             # mixture of experts in place of a dense feed-forward
 
 
 @dataclass
 class ModelConfig:
-    architecture: str = "llama"            # "llama" | "deepseek_v2" | "rekudra"
+    architecture: str = "llama"            # "llama" | "deepseek_v2" | "rekudra" | "rerupel"
     hidden_size: int = 4096
     num_layers: int = 32
     num_heads: int = 32
@@ -68,6 +103,10 @@ class ModelConfig:
     layers: list[LayerSpec] | None = None
     residual_streams: int = 1
     embedding_scale: float = 1.0
+    bigram: BigramSpec | None = None
+    loop: LoopSpec | None = None           # layers that run several times
+    residual_mult: float = 1.0             # on everything a sublayer adds to the residual
+    logit_softcap: float | None = None
     extra: dict = field(default_factory=dict)
 
     def to_dict(self) -> dict:
@@ -81,7 +120,17 @@ class ModelConfig:
     def is_moe(self) -> bool:
         return self.n_routed_experts > 0
 
+    def layer_runs(self) -> list[tuple[int, bool]]:
+        """The layers in the order they run, as (layer, whether a pass of the loop begins right before it)."""
+        n, lp = self.num_layers, self.loop
+        if lp is None:
+            return [(i, False) for i in range(n)]
+        body = [(i, i == lp.start) for i in range(lp.start, lp.stop)]
+        return [(i, False) for i in range(lp.start)] + body * lp.times + [(i, False) for i in range(lp.stop, n)]
+
     def kv_bytes_per_token(self, dtype_bytes: int = 2, tp: int = 1) -> int:
+        if self.architecture == "rerupel":
+            return sum(self.layers[i].kv_rank for i, _ in self.layer_runs()) * dtype_bytes
         if self.layers is not None:
             return sum(s.kv_heads * (s.dim + s.vdim) for s in self.layers if s.mixer == "attention" and s.kv_from is None) * dtype_bytes
         if self.is_mla:
@@ -91,6 +140,13 @@ class ModelConfig:
     def num_params(self) -> int:
         h = self.hidden_size
         emb = self.vocab_size * h * (1 if self.tie_word_embeddings else 2)
+        if self.architecture == "rerupel":
+            n = emb + h + (self.bigram.buckets + 1 if self.bigram else 0) * h + (2 * h * h if self.loop else 0)
+            for s in self.layers:
+                n += h * (s.heads * (s.dim + 2 * s.vdim) + s.kv_rank + 4) + s.heads * (s.dim + s.vdim) * s.kv_rank + 2 * h * s.ffn
+                if s.moe is not None:
+                    n += h * (s.moe.experts + 3 * s.moe.experts * s.moe.expert.ffn + 3 * (s.moe.shared.ffn if s.moe.shared else 0))
+            return n
         if self.layers is not None:
             n = emb + h
             for s in self.layers:
@@ -147,6 +203,8 @@ class ModelConfig:
     @staticmethod
     def from_layered(cfg: dict) -> "ModelConfig":
         """A config that lists its layers one by one (`layers[i]`: type, mixer sizes, feed-forward)."""
+        if LAYERED_ARCHITECTURES[cfg["architecture"]] == "rerupel":
+            return ModelConfig._from_latent_layers(cfg)
         layers = []
         for i, entry in enumerate(cfg["layers"]):
             m, mlp = entry["mixer"], entry.get("mlp")
@@ -174,8 +232,41 @@ class ModelConfig:
                            embedding_scale=cfg.get("embedding", {}).get("scale", 1.0))
 
 
+    @staticmethod
+    def _from_latent_layers(cfg: dict) -> "ModelConfig":
+        layers = []
+        for i, entry in enumerate(cfg["layers"]):
+            m, mlp = entry["mixer"], entry.get("mlp")
+            if entry["type"] != "latent_attention":
+                raise ValueError(f"layer {i}: unknown mixer {entry['type']!r}")
+            spec = LayerSpec(mixer="latent_attention", heads=m["heads"], kv_heads=1, dim=m["dim"], vdim=m["vdim"], kv_rank=m["kv_rank"], scale=m["scale"])
+            if mlp is not None and mlp["kind"] == "dense":
+                spec.ffn = mlp["ff"]
+            elif mlp is not None and mlp["kind"] == "moe":
+                r, sh = mlp["router"], mlp.get("shared")
+                spec.moe = MoeSpec(r["experts"], r["top"], r.get("scale", 1.0), ExpertSpec(mlp["expert"]["ff"], mlp["expert"]["limit"]),
+                                   ExpertSpec(sh["ff"], sh["limit"]) if sh else None)
+                if not 1 <= spec.moe.top <= spec.moe.experts:
+                    raise ValueError(f"layer {i}: {spec.moe.top} of {spec.moe.experts} experts")
+            elif mlp is not None:
+                raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+            layers.append(spec)
+        emb, lp = cfg.get("embedding", {}), cfg.get("loop")
+        bg = emb.get("bigram")
+        if lp and not (0 <= lp["start"] < lp["stop"] <= len(layers) and lp["times"] >= 1):
+            raise ValueError(f"loop over layers {lp['start']} .. {lp['stop']}, {lp['times']} times, of {len(layers)}")
+        first = layers[0]
+        return ModelConfig(architecture="rerupel", hidden_size=cfg["width"], num_layers=len(layers), num_heads=first.heads, num_kv_heads=1, head_dim=first.dim,
+                           intermediate_size=max(s.ffn for s in layers), vocab_size=cfg["vocab"], rms_norm_eps=cfg["norm"]["eps"], max_position_embeddings=0,
+                           tie_word_embeddings=True, layers=layers, embedding_scale=emb.get("scale", 1.0), residual_mult=cfg.get("residual_mult", 1.0),
+                           logit_softcap=cfg.get("logit_softcap"), bigram=BigramSpec(bg["buckets"], bg["mul_prev"], bg["mul_cur"]) if bg else None,
+                           loop=LoopSpec(lp["start"], lp["stop"], lp["times"]) if lp else None)
+
+
 # `architecture` values of configs that list their layers -> model class key
-LAYERED_ARCHITECTURES = {"Rekudra": "rekudra"}
+LAYERED_ARCHITECTURES = {"Rekudra": "rekudra", "Rerupel": "rerupel"}
+# model classes that also run in f32 on CUDA (every operation has a true 32-bit kernel)
+F32_ARCHITECTURES = ("rekudra", "rerupel")
 
 
 def tiny_llama() -> ModelConfig:
@@ -247,6 +338,27 @@ def tiny_rekudra() -> ModelConfig:
     return rekudra(256, 4, 4, 2, 64, 512, 1024, streams=2)
 
 
+def rerupel(width: int, n_layers: int, heads: int, dim: int, kv_rank: int, ffn: int, vocab: int, experts: int, top: int, expert_ffn: int,
+            shared_ffn: int, loop: tuple[int, int, int] | None = None) -> ModelConfig:
+    """A Rerupel decoder: one layer with a dense feed-forward, then layers with experts; `loop` = (start, stop, times)."""
+    moe = MoeSpec(experts, top, 1.0, ExpertSpec(expert_ffn, 7.0), ExpertSpec(shared_ffn, 7.0))
+    layers = [LayerSpec("latent_attention", heads, 1, dim, dim, scale=dim ** -0.5, kv_rank=kv_rank, ffn=0 if i else ffn, moe=moe if i else None)
+              for i in range(n_layers)]
+    return ModelConfig(architecture="rerupel", hidden_size=width, num_layers=n_layers, num_heads=heads, num_kv_heads=1, head_dim=dim, intermediate_size=ffn,
+                       vocab_size=vocab, rms_norm_eps=1e-6, max_position_embeddings=0, tie_word_embeddings=True, layers=layers,
+                       embedding_scale=float(width) ** 0.5, logit_softcap=30.0, bigram=BigramSpec(16381, 10007, 31),
+                       loop=LoopSpec(*loop) if loop else None)
+
+
+def rerupel_lite() -> ModelConfig:
+    """Layers of the size of DeepSeek-V2-Lite's; the upper half runs twice."""
+    return rerupel(2048, 14, 16, 128, 512, 10944, 102400, 64, 6, 1408, 2816, (2, 14, 2))
+
+
+def tiny_rerupel() -> ModelConfig:
+    return rerupel(256, 3, 4, 64, 128, 512, 1024, 8, 2, 128, 192, (1, 3, 2))
+
+
 PRESETS = {
     "tiny-llama": tiny_llama,
     "llama-3.1-8b": llama31_8b,
@@ -256,6 +368,8 @@ PRESETS = {
     "rekudra-8b": rekudra_8b,
     "rekudra-1b": rekudra_1b,
     "tiny-rekudra": tiny_rekudra,
+    "rerupel-lite": rerupel_lite,
+    "tiny-rerupel": tiny_rerupel,
 }
 
 

@@ -12,7 +12,9 @@ from .. import _ext
 from . import _state, autotune, reference
 from ._state import KernelError, check_status
 
-EPI_NONE, EPI_ADD_RESIDUAL, EPI_SWIGLU = 0, 1, 2
+from .activation import SWIGLU, Glu
+
+EPI_NONE, EPI_ADD_RESIDUAL, EPI_SWIGLU, EPI_RELU2, EPI_SOFTCAP, EPI_F32 = 0, 1, 2, 3, 4, 5
 
 # Kernel launches issued through this module since the last reset (bench accounting).
 launch_count = 0
@@ -162,16 +164,18 @@ def copy_pages(cache: torch.Tensor, src_pages: torch.Tensor, dst_pages: torch.Te
     _count()
 
 
+PAIR_EPILOGUES = (EPI_NONE, EPI_SWIGLU, EPI_RELU2)
 PAIR_CONFIG = 1 << 28   # configuration word that selects the CTA-pair (cta_group::2) GEMM kernel; low bits = tile width (256 default, 128)
 
 
-def _launch_gemm(C, x, w, out, residual, epi, config, st) -> None:
-    """One bf16 GEMM launch: the CTA-pair kernel when `config` says so (plain and SwiGLU epilogues only), else the
-    single-CTA kernel family with `config` as its tile / split / layout word."""
-    if config & PAIR_CONFIG and residual is None and epi != EPI_ADD_RESIDUAL:
-        C.gemm_bf16_pair(x, w, out, epi, (config & 0xffff) or 256, st.status)
+def _launch_gemm(C, x, w, out, residual, epi, config, st, act=None) -> None:
+    """One bf16 GEMM launch: the CTA-pair kernel when `config` says so (plain, gated and squared-ReLU epilogues only), else
+    the single-CTA kernel family with `config` as its tile / split / layout word. `act`: constants of the epilogue's
+    activation, (limit, alpha, up_bias, cap)."""
+    if config & PAIR_CONFIG and residual is None and epi in PAIR_EPILOGUES:
+        C.gemm_bf16_pair(x, w, out, epi, (config & 0xffff) or 256, st.status, act)
     else:
-        C.gemm_bf16(x, w, out, residual, epi, config & ~PAIR_CONFIG, st.gemm_ws, st.status)
+        C.gemm_bf16(x, w, out, residual, epi, config & ~PAIR_CONFIG, st.gemm_ws, st.status, act)
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, residual: torch.Tensor | None = None, out: torch.Tensor | None = None,
@@ -202,17 +206,46 @@ def linear_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = Non
     return linear(x, w, out=out, config=PAIR_CONFIG)
 
 
-def linear_swiglu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor | None = None, config: int = 0) -> torch.Tensor:
-    """silu(x Wg^T) * (x Wu^T) in one GEMM; `w_gu` is the 16-row interleaved stack from
+def _linear_epi(x: torch.Tensor, w: torch.Tensor, epi: int, cap: float = 0.0) -> torch.Tensor:
+    """x @ w.T with an epilogue that needs nothing but constants."""
+    C = _ext.require()
+    f32 = x.dtype == torch.float32
+    out = torch.empty(x.shape[0], w.shape[0], dtype=torch.float32 if epi == EPI_F32 else x.dtype, device=x.device)
+    if f32:
+        C.gemm_f32(x, w, out, 1, EPI_NONE if epi == EPI_F32 else epi, cap)
+    else:
+        config = autotune.lookup(x.shape[0], w.shape[0], w.shape[1], epi, x.device.index or 0)
+        _launch_gemm(C, x, w, out, None, epi, config, _state.get(x.device), (float("inf"), 1.0, 0.0, cap))
+    _count()
+    return out
+
+
+def linear_f32(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """x @ w.T with the f32 accumulators as the result (routers, projections that become a 32-bit residual)."""
+    return reference.linear(x, w) if not x.is_cuda else _linear_epi(x, w, EPI_F32)
+
+
+def linear_relu2(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """max(x @ w.T, 0)^2."""
+    return reference.linear(x, w).clamp_min(0.0).square().to(x.dtype) if not x.is_cuda else _linear_epi(x, w, EPI_RELU2)
+
+
+def linear_softcap(x: torch.Tensor, w: torch.Tensor, cap: float) -> torch.Tensor:
+    """cap * tanh(x @ w.T / cap)."""
+    return (torch.tanh(reference.linear(x, w) / cap) * cap).to(x.dtype) if not x.is_cuda else _linear_epi(x, w, EPI_SOFTCAP, cap)
+
+
+def linear_swiglu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor | None = None, config: int = 0, glu: Glu = SWIGLU) -> torch.Tensor:
+    """silu(x Wg^T) * (x Wu^T), or another gated linear unit, in one GEMM; `w_gu` is the 16-row interleaved stack from
     `reference.interleave_gate_up`."""
     if not x.is_cuda:
-        return reference.linear_swiglu_interleaved(x, w_gu).to(x.dtype)
+        return reference.linear_swiglu_interleaved(x, w_gu, act=glu).to(x.dtype)
     C = _ext.require()
     if x.dtype == torch.float32:
         gu = linear(x, w_gu)
         if out is None:
             out = torch.empty(x.shape[0], w_gu.shape[0] // 2, dtype=x.dtype, device=x.device)
-        C.swiglu_f32(gu, out)
+        C.glu_f32(gu, out, *glu)
         _count()
         return out
     st = _state.get(x.device)
@@ -220,7 +253,7 @@ def linear_swiglu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor | None 
         out = torch.empty(x.shape[0], w_gu.shape[0] // 2, dtype=x.dtype, device=x.device)
     if config == 0:
         config = autotune.lookup(x.shape[0], w_gu.shape[0], w_gu.shape[1], EPI_SWIGLU, x.device.index or 0)
-    _launch_gemm(C, x, w_gu, out, None, EPI_SWIGLU, config, st)
+    _launch_gemm(C, x, w_gu, out, None, EPI_SWIGLU, config, st, (*glu, 0.0))
     _count()
     return out
 
@@ -290,12 +323,16 @@ class AttnMeta:
                       CUDA graph that serves any batch of its bucket
       seq             a `SeqRows` for models with recurrent state: sequence of every row, rows and state banks of every
                       sequence
+      prev            int32 [T], the token before each row's in its sequence (-1: there is none), for models that look at it
+      expand          (pages int32 [n, 2], tables int32 [prefill sequences, blocks]) when the latents of the prefill
+                      sequences' contexts are to be expanded into keys and values (`latent_prefill`)
     """
 
     __slots__ = ("cu_q", "ctx_lens", "block_tables", "num_decode", "num_seqs", "max_q_len", "num_tokens", "max_ctx", "work", "n_items", "static",
-                 "seq")
+                 "seq", "prev", "expand")
 
-    def __init__(self, cu_q, ctx_lens, block_tables, num_decode, max_q_len, max_ctx=0, work=None, n_items=0, static=None, seq=None):
+    def __init__(self, cu_q, ctx_lens, block_tables, num_decode, max_q_len, max_ctx=0, work=None, n_items=0, static=None, seq=None, prev=None,
+                 expand=None):
         self.cu_q, self.ctx_lens, self.block_tables = cu_q, ctx_lens, block_tables
         self.num_decode = int(num_decode)
         self.num_seqs = int(ctx_lens.numel()) if ctx_lens is not None else 0
@@ -305,6 +342,8 @@ class AttnMeta:
         self.work, self.n_items = work, int(n_items)
         self.static = static
         self.seq = seq
+        self.prev = prev
+        self.expand = expand
 
 
 class StaticAttn:
@@ -413,7 +452,7 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             _decode_attention(q[:sa.d_rows], k_cache, v_cache, out[:sa.d_rows], sa.d_ctx, sa.d_bt, head_dim, scale, sa.max_ctx,
                               gate[:sa.d_rows] if gate is not None else None)
         if sa.max_items > 0:
-            C.attn_prefill_tc(q, k_cache, v_cache, out, sa.p_cu, sa.p_ctx, sa.p_bt, sa.max_q_len, scale, 0, st.status,
+            C.attn_prefill_tc(q, k_cache, v_cache, out, sa.p_cu, sa.p_ctx, sa.p_bt, sa.max_q_len, scale, st.status,
                               sa.work, sa.n_work, sa.max_items, gate)
             _count()
         return out
@@ -427,10 +466,10 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
             # tcgen05 / TMEM kernel: one KV tile = one 128-token page
             if meta.work is not None and meta.n_items > 0:
                 C.attn_prefill_tc(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:],
-                                  meta.max_q_len, scale, 0, st.status, meta.work, None, meta.n_items, gate)
+                                  meta.max_q_len, scale, st.status, meta.work, None, meta.n_items, gate)
             else:
                 C.attn_prefill_tc(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:],
-                                  meta.max_q_len, scale, 0, st.status, None, None, 0, gate)
+                                  meta.max_q_len, scale, st.status, None, None, 0, gate)
         else:
             C.attn_prefill(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:], head_dim,
                            meta.max_q_len, scale, st.status, gate)
@@ -513,4 +552,6 @@ def sample(logits: torch.Tensor, temperature: torch.Tensor, top_k: torch.Tensor,
     return ids
 
 
-from .mixers import DeltaParams, HyperMix, SeqRows, conv_qkv, delta_rule, hyper_norm  # noqa: E402,F401
+from .latent import head_linear, latent_attend, latent_prefill, latent_write, plan_latent_prefill, token_rows  # noqa: E402,F401
+from .mixers import DeltaParams, Finished, HyperMix, SeqRows, StreamStart, conv_qkv, delta_rule, hyper_norm, residual_norm  # noqa: E402,F401
+from .moe import ExpertRows, MoeWeights, moe_experts  # noqa: E402,F401

@@ -35,6 +35,8 @@ class _DeviceState:
         self.attn_ws = torch.empty(ATTN_WORKSPACE_BYTES // 4, dtype=torch.float32, device=device)
         # per (sequence, kv head) arrival counters of the split decode attention (self-resetting; zero between launches)
         self.attn_counters = torch.zeros(1 << 18, dtype=torch.int32, device=device)
+        # rows per expert of the layer being routed, and a ticket word (zero between layers)
+        self.moe_counts = torch.zeros(1025, dtype=torch.int32, device=device)
 
 
 _states: dict[int, _DeviceState] = {}
@@ -64,4 +66,5 @@ def check_status(device: torch.device | None = None, reset: bool = True) -> None
         st.status.zero_()
         st.gemm_ws[: 65536].zero_()  # split-K counters may be left mid-count by an aborted kernel
         st.attn_counters.zero_()
+        st.moe_counts.zero_()
     raise KernelError(code, int(words[1]), int(words[2]), int(words[3]), a, b)

@@ -14,7 +14,7 @@ import bisect
 
 import torch
 
-EPI_NONE, EPI_ADD_RESIDUAL, EPI_SWIGLU = 0, 1, 2
+EPI_NONE, EPI_ADD_RESIDUAL, EPI_SWIGLU, EPI_RELU2, EPI_SOFTCAP, EPI_F32 = 0, 1, 2, 3, 4, 5
 PAIR_CONFIG = 1 << 28
 L2_BYTES = 126 << 20
 
@@ -63,7 +63,7 @@ def candidates(M: int, N: int, K: int, epilogue: int) -> list[int]:
                 if sp > 1 and (num_kb // sp < 4 or not ws_ok(tiles, sp, bn) or tiles * sp > 4 * 148):
                     continue
                 out.append(_encode(False, bn, sp))
-    if M >= 192 and N >= 256 and N % 8 == 0 and epilogue != EPI_ADD_RESIDUAL:
+    if M >= 192 and N >= 256 and N % 8 == 0 and epilogue in (EPI_NONE, EPI_SWIGLU, EPI_RELU2):
         out.append(PAIR_CONFIG | 256)   # 256 x 256 tiles on CTA pairs
         out.append(PAIR_CONFIG | 128)   # 256 x 128
     return out
@@ -100,14 +100,14 @@ def tune(N: int, K: int, epilogue: int, token_counts, device=None, iters: int = 
     bounds, configs = [], []
     for M in sorted(set(int(m) for m in token_counts)):
         x = torch.randn(M, K, device=device, dtype=torch.bfloat16)
-        y = torch.empty(M, n_out, device=device, dtype=torch.bfloat16)
+        y = torch.empty(M, n_out, device=device, dtype=torch.float32 if epilogue == EPI_F32 else torch.bfloat16)
         res = torch.zeros(M, n_out, device=device, dtype=torch.bfloat16) if epilogue == EPI_ADD_RESIDUAL else None
         turn = [0]
 
         def run(cfg):
             w = ws[turn[0] % len(ws)]
             turn[0] += 1
-            _launch(C, x, w, y, res, epilogue, cfg, st)
+            _launch(C, x, w, y, res, epilogue, cfg, st, (float("inf"), 1.0, 0.0, 30.0))
 
         best_cfg, best_t = 0, _time(lambda: run(0), iters)
         t_auto = best_t

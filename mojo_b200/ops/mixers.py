@@ -1,5 +1,5 @@
-"""Sequence mixing beyond plain attention: hyper-connections (a residual of several mixed streams), short causal
-convolutions in front of attention, and the gated delta rule. CUDA tensors (bf16, or f32 for the exact mode) go to the
+"""Sequence mixing beyond plain attention: residuals in 32 bits (hyper-connections, that is several mixed streams, or one
+stream with a scale per channel), short causal convolutions in front of attention, and the gated delta rule. CUDA tensors (bf16, or f32 for the exact mode) go to the
 sm_100a kernels, CPU tensors to `ops.reference`, as in the rest of `ops`."""
 from __future__ import annotations
 
@@ -57,6 +57,72 @@ def hyper_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, dtype: torch.d
                               embed_scale, rows, store, eps, mean_width or W, _state.get(x.device).status)
     _count()
     return h
+
+
+@dataclass
+class StreamStart:
+    """How a residual stream begins: embed[id] * scale, plus (where `bigram` is given, [buckets + 1, width]) the row
+    (previous id * mul_prev + id * mul_cur) mod buckets of a second table, its last row for a sequence's first token.
+    `x0` receives a copy of the result."""
+    ids: torch.Tensor
+    embed: torch.Tensor
+    scale: float = 1.0
+    prev: torch.Tensor | None = None          # int32 [T], -1: none
+    bigram: torch.Tensor | None = None
+    mul_prev: int = 0
+    mul_cur: int = 0
+    x0: torch.Tensor | None = None
+
+
+@dataclass
+class Finished:
+    """A sublayer's result on its way into the residual: rows `y`, or the weighted rows of every token's experts
+    (`ops.ExpertRows`), or both; `scale` f32 [width] is applied to their sum."""
+    scale: torch.Tensor
+    y: torch.Tensor | None = None
+    experts: object | None = None
+
+
+def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, dtype: torch.dtype, done: Finished | None = None,
+                  start: StreamStart | None = None, out: torch.Tensor | None = None, rows: torch.Tensor | None = None, store: bool = True,
+                  mean_width: int | None = None) -> torch.Tensor:
+    """Everything between two sublayers in one launch: add the finished one to the stream x [T, width] (f32, in place) and
+    RMS-normalise the sum with `weight` (f32; None: return x itself, rounded). `start`: x begins from the embedding.
+    `rows`: only these rows, compact. `out`: where the result goes (rows may be strided)."""
+    from . import _count
+
+    T, W = x.shape
+    ex = done.experts if done is not None else None
+    y = done.y if done is not None else None
+    if not x.is_cuda:
+        if start is not None:
+            e = start.embed.float()[start.ids.long()] * start.scale
+            if start.bigram is not None:
+                n, prev = start.bigram.shape[0] - 1, start.prev.long()
+                e = e + start.bigram.float()[torch.where(prev < 0, n, (prev * start.mul_prev + start.ids.long() * start.mul_cur) % n)]
+            x.copy_(e)
+            if start.x0 is not None:
+                start.x0.copy_(e)
+        pick = slice(None) if rows is None else rows.long()
+        add = None
+        if done is not None:
+            add = torch.zeros(T, W) if y is None else y.float()
+            if ex is not None:
+                add = add + torch.einsum("tk,tkw->tw", ex.weights, ex.rows.float()[ex.slot.long()])
+            add = add[pick]
+        h, new = reference.residual_norm(x[pick], weight, eps, add, done.scale if done is not None else None, mean_width)
+        if store:
+            x.copy_(new)
+        return h.to(dtype) if out is None else out.copy_(h)
+    if out is None:
+        out = torch.empty(T if rows is None else rows.numel(), W, dtype=dtype, device=x.device)
+    s = start
+    _ext.require().residual_norm(x, y, ex.rows if ex else None, ex.slot if ex else None, ex.weights if ex else None, done.scale if done else None, weight, out,
+                                 s.ids if s else None, s.embed if s else None, s.scale if s else 1.0, s.prev if s and s.bigram is not None else None,
+                                 s.bigram if s else None, s.mul_prev if s else 0, s.mul_cur if s else 0, s.x0 if s else None, rows, store, eps,
+                                 mean_width or W, _state.get(x.device).status)
+    _count()
+    return out
 
 
 def conv_qkv(proj: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor | None, cos_sin: torch.Tensor, positions: torch.Tensor, seq: SeqRows,

@@ -1,0 +1,80 @@
+"""Mixture of experts with all experts on one GPU: router, permutation of the token rows, grouped products over a packed list
+of tiles. Nothing is read back to the host, so a layer can be captured in a CUDA graph. The weighted sum of the experts'
+rows is left to the kernel that adds them to the residual (`ops.residual_norm`). `parallel.ep` spreads experts over ranks."""
+from __future__ import annotations
+
+from dataclasses import dataclass
+
+import torch
+
+from .. import _ext
+from . import _state, reference
+from .activation import SWIGLU, Glu
+
+SCORING = {"softmax": 0, "sigmoid": 1}
+
+
+@dataclass
+class MoeWeights:
+    """router [>= experts, width] (rows past `experts` are padding), w_gu [experts, 2 ffn, width] (gate and up rows
+    interleaved in blocks of 16), w_down [experts, width, ffn]. A token uses the `top` experts of the largest scores, with
+    their scores (over their sum if `norm_top`) times `scale` as weights."""
+    router: torch.Tensor
+    w_gu: torch.Tensor
+    w_down: torch.Tensor
+    experts: int
+    top: int
+    scoring: str = "softmax"
+    norm_top: bool = False
+    scale: float = 1.0
+    glu: Glu = SWIGLU
+
+
+@dataclass
+class ExpertRows:
+    """Results of a token's experts: rows[slot[t, j]] times weights[t, j], summed over j."""
+    rows: torch.Tensor
+    slot: torch.Tensor          # int32 [T, top]
+    weights: torch.Tensor       # f32 [T, top]
+
+
+def tile_rows(rows_per_expert: float) -> int:
+    """Token rows of one tile of the grouped product: the narrowest that usually holds an expert's rows."""
+    return next((n for n in (16, 32, 64, 128) if rows_per_expert * 1.25 <= n), 256)
+
+
+def moe_experts(h: torch.Tensor, p: MoeWeights) -> ExpertRows:
+    """Run every row of h [T, width] through its experts."""
+    from . import EPI_NONE, EPI_SWIGLU, _count, linear_f32
+
+    T, W = h.shape
+    logits = linear_f32(h, p.router)
+    if not h.is_cuda:
+        weights, ids = reference.moe_route(logits[:, :p.experts], p.top, p.norm_top, p.scale, sigmoid=p.scoring == "sigmoid")
+        rows = torch.empty(T, p.top, W, dtype=h.dtype)
+        for e in range(p.experts):
+            tok, j = torch.where(ids == e)
+            if tok.numel():
+                rows[tok, j] = reference.linear(reference.linear_swiglu_interleaved(h[tok], p.w_gu[e], act=p.glu).to(h.dtype), p.w_down[e]).to(h.dtype)
+        return ExpertRows(rows.view(T * p.top, W), torch.arange(T * p.top, dtype=torch.int32).view(T, p.top), weights.float())
+    C, st = _ext.require(), _state.get(h.device)
+    dev, R, f32 = h.device, T * p.top, h.dtype == torch.float32
+    bn = 64 if f32 else tile_rows(R / p.experts)
+    weights = torch.empty(T, p.top, dtype=torch.float32, device=dev)
+    ids, place, slot = (torch.empty(T, p.top, dtype=torch.int32, device=dev) for _ in range(3))
+    counts = st.moe_counts
+    C.moe_route(logits, weights, ids, place, counts, p.experts, SCORING[p.scoring], p.norm_top, p.scale)
+    xs = torch.empty(R, W, dtype=h.dtype, device=dev)
+    tiles, n_tiles = torch.empty(p.experts + R // bn, 4, dtype=torch.int32, device=dev), torch.empty(1, dtype=torch.int32, device=dev)
+    C.moe_gather(h, ids, place, counts, slot, xs, tiles, n_tiles, p.experts, bn, st.status)
+    f = p.w_down.shape[2]
+    act, y = torch.empty(R, f, dtype=h.dtype, device=dev), torch.empty(R, W, dtype=h.dtype, device=dev)
+    if f32:
+        gu = torch.empty(R, 2 * f, dtype=h.dtype, device=dev)
+        C.moe_tiles_gemm(xs, p.w_gu, tiles, n_tiles, gu, EPI_NONE, bn, None, st.status)
+        C.glu_f32(gu, act, *p.glu)
+    else:
+        C.moe_tiles_gemm(xs, p.w_gu, tiles, n_tiles, act, EPI_SWIGLU, bn, (*p.glu, 0.0), st.status)
+    C.moe_tiles_gemm(act, p.w_down, tiles, n_tiles, y, EPI_NONE, bn, None, st.status)
+    _count(5 if f32 else 4)
+    return ExpertRows(y, slot, weights)

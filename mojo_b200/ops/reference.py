@@ -175,11 +175,18 @@ def deinterleave_gate_up(w_gu: torch.Tensor, block: int = 16):
     return v[:, 0].reshape(two_f // 2, k).contiguous(), v[:, 1].reshape(two_f // 2, k).contiguous()
 
 
-def linear_swiglu_interleaved(x: torch.Tensor, w_gu: torch.Tensor, block: int = 16) -> torch.Tensor:
-    """silu(x @ Wg.T) * (x @ Wu.T) for a weight stored by `interleave_gate_up`."""
+def glu(g: torch.Tensor, u: torch.Tensor, limit: float = float("inf"), alpha: float = 1.0, up_bias: float = 0.0) -> torch.Tensor:
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return g * torch.sigmoid(alpha * g) * (u + up_bias)
+
+
+def linear_swiglu_interleaved(x: torch.Tensor, w_gu: torch.Tensor, block: int = 16, act=None) -> torch.Tensor:
+    """silu(x @ Wg.T) * (x @ Wu.T), or the gated linear unit with constants `act`, for a weight stored by `interleave_gate_up`."""
     y = x.float() @ w_gu.float().t()  # [M, 2F] interleaved
     m = y.shape[0]
     y = y.reshape(m, -1, 2, block)
+    if act is not None:
+        return glu(y[:, :, 0], y[:, :, 1], *act).reshape(m, -1)
     return (silu(y[:, :, 0]) * y[:, :, 1]).reshape(m, -1)
 
 
@@ -291,6 +298,17 @@ def hyper_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, w_in=None, y=N
     return u * torch.rsqrt(ms + eps) * weight, x
 
 
+def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, y=None, y_scale=None, mean_width: int | None = None):
+    """x [rows, width] f32, y what a finished sublayer adds (before its scale). Returns (normed rows, or x itself without a
+    weight; new stream)."""
+    if y is not None:
+        x = x + y_scale * y.float()
+    if weight is None:
+        return x, x
+    ms = x.pow(2).sum(-1, keepdim=True) / (mean_width or x.shape[-1])
+    return x * torch.rsqrt(ms + eps) * weight, x
+
+
 def short_conv(u: torch.Tensor, w: torch.Tensor, conv_state, seq_rows, seq_state) -> torch.Tensor:
     """Causal convolution over time on the first `channels` columns of u [T, >= channels]; w [taps, channels]. Reads and
     writes the sequences' state banks [banks, taps - 1, channels]. Rows of unused sequences stay zero."""
@@ -374,9 +392,10 @@ def mla_attend(q_lat: torch.Tensor, q_rope: torch.Tensor, kv_cache: torch.Tensor
 # ------------------------------------------------------------------------------------------------------
 
 
-def moe_route(router_logits: torch.Tensor, top_k: int, norm_topk: bool = False, scale: float = 1.0):
-    """Softmax over all experts, then top-k (DeepSeek-V2 'greedy' routing). Returns (weights [T, k], ids [T, k])."""
-    p = torch.softmax(router_logits.float(), dim=-1)
+def moe_route(router_logits: torch.Tensor, top_k: int, norm_topk: bool = False, scale: float = 1.0, sigmoid: bool = False):
+    """Softmax over all experts (DeepSeek-V2 'greedy' routing), or the sigmoid of each score alone, then top-k. Returns
+    (weights [T, k], ids [T, k])."""
+    p = torch.sigmoid(router_logits.float()) if sigmoid else torch.softmax(router_logits.float(), dim=-1)
     w, idx = torch.topk(p, top_k, dim=-1)
     if norm_topk:
         w = w / w.sum(dim=-1, keepdim=True)

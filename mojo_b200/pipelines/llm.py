@@ -10,6 +10,7 @@ import torch
 
 from ..engine import EngineConfig, LLMEngine, SamplingParams
 from ..models import build_model, get_config
+from ..models.config import F32_ARCHITECTURES
 from .config import PipelineConfig
 
 
@@ -92,7 +93,7 @@ class LLM:
             device = str(self.dist_info.device)
         if degree > 1 and comm is None and ep is None:
             comm, ep, device = self._join_ranks(mcfg, device, degree)
-        if dtype == torch.float32 and device.startswith("cuda") and mcfg.architecture != "rekudra":
+        if dtype == torch.float32 and device.startswith("cuda") and mcfg.architecture not in F32_ARCHITECTURES:
             raise ValueError(f"{mcfg.architecture} runs in bfloat16 on CUDA")
         model = build_model(mcfg, device, dtype, comm=comm, ep=ep)
         if config.random_init or (not is_gguf and not (Path(src) / "config.json").exists()):
