@@ -87,8 +87,16 @@ def route(h, w_router, top, scale):
     return torch.zeros_like(s).scatter(1, best, s.gather(1, best)) * scale
 
 
-def mixture(h, w, p, mlp):
+def choice_gaps(z, top):
+    """How far the last chosen router logit of every row lies above the first one left out."""
+    best = z.sort(dim=1, descending=True).values
+    return best[:, top - 1] - best[:, top] if top < z.shape[1] else torch.full((z.shape[0],), 9.0, dtype=z.dtype)
+
+
+def mixture(h, w, p, mlp, gaps=None):
     r = mlp["router"]
+    if gaps is not None:
+        gaps.append(choice_gaps(h @ w[p + "router"].T, r["top"]))
     weights = route(h, w[p + "router"], r["top"], r["scale"])
     y = torch.zeros_like(h)
     for e in range(r["experts"]):
@@ -98,16 +106,16 @@ def mixture(h, w, p, mlp):
     return y
 
 
-def feed_forward(h, w, p, mlp):
-    return dense(h, w, p) if mlp["kind"] == "dense" else mixture(h, w, p, mlp)
+def feed_forward(h, w, p, mlp, gaps=None):
+    return dense(h, w, p) if mlp["kind"] == "dense" else mixture(h, w, p, mlp, gaps)
 
 
-def layer(x, w, i, cfg):
+def layer(x, w, i, cfg, gaps=None):
     spec, p, eps, m = cfg["layers"][i], f"l{i}.", cfg["norm"]["eps"], cfg["residual_mult"]
     y = latent_attention(norm(x, w[p + "norm1"], eps), w, p + "mix.", spec["mixer"], eps)
     x = x + m * (y * w[p + "ls1"])
     if spec["mlp"] is not None:
-        x = x + m * (feed_forward(norm(x, w[p + "norm2"], eps), w, p + "mlp.", spec["mlp"]) * w[p + "ls2"])
+        x = x + m * (feed_forward(norm(x, w[p + "norm2"], eps), w, p + "mlp.", spec["mlp"], gaps) * w[p + "ls2"])
     return x
 
 
@@ -124,13 +132,14 @@ def softcap(z, cap):
     return cap * torch.tanh(z / cap)
 
 
-def forward(cfg, w, tokens, layers_out=None):
-    """Logits [T, vocab] of one sequence. `layers_out`, a list, receives the residual stream after every layer run."""
+def forward(cfg, w, tokens, layers_out=None, gaps=None):
+    """Logits [T, vocab] of one sequence. `layers_out`, a list, receives the residual stream after every layer run, `gaps`
+    the margin of every router's choice."""
     x0 = x = embedding(tokens, w, cfg)
     for i, enters in layer_runs(cfg):
         if enters:
             x = torch.cat([x, x0], dim=1) @ w["loop.in"].T
-        x = layer(x, w, i, cfg)
+        x = layer(x, w, i, cfg, gaps)
         if layers_out is not None:
             layers_out.append(x)
     return softcap(norm(x, w["final.norm"], cfg["norm"]["eps"]) @ w["embed"].T, cfg["logit_softcap"])
