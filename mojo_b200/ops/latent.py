@@ -17,6 +17,7 @@ from . import _state, reference
 
 EXPAND_PAGE = 128                  # tokens in a page of expanded keys and values
 EXPAND_BYTES = 2 << 30             # most scratch the expanded form may take
+ABSORBED_RATE, PREFILL_RATE, GEMM_RATE = 90.0, 400.0, 900.0      # TFLOP/s of the kernels the two forms run on
 
 
 def latent_write(c: torch.Tensor, weight: torch.Tensor, eps: float, slots: torch.Tensor, cache: torch.Tensor) -> None:
@@ -99,15 +100,18 @@ def latent_attend(q: torch.Tensor, cache: torch.Tensor, meta, rows, heads: int, 
 
 
 def plan_latent_prefill(cu_q, ctx_lens, num_decode: int, latent: int, heads: int, dim: int, vdim: int):
-    """Whether the prefill sequences of a batch (host arrays) attend in the expanded form: where that takes fewer operations
-    and its scratch stays small. Returns (pages int32 [n, 2] = (prefill sequence, block of 128 positions), tables int32
+    """Whether the prefill sequences of a batch (host arrays) attend in the expanded form: where that is faster by the kernels'
+    rates and its scratch stays small. Returns (pages int32 [n, 2] = (prefill sequence, block of 128 positions), tables int32
     [sequences, blocks]) or None."""
     cu, ctx = np.asarray(cu_q[num_decode:], dtype=np.int64), np.asarray(ctx_lens[num_decode:], dtype=np.int64)
     q_len = cu[1:] - cu[:-1]
-    pairs = int((q_len * ctx).sum())
     blocks = (ctx + EXPAND_PAGE - 1) // EXPAND_PAGE
     n = int(blocks.sum())
-    if n == 0 or n * EXPAND_PAGE * latent * (dim + vdim) >= pairs * (2 * latent - dim - vdim):
+    # operations per head, over rates: the prefill kernel works on tiles of 128 query rows
+    absorbed = float((q_len * ctx).sum()) * 4 * latent / ABSORBED_RATE
+    tiles = float(((q_len + 127) // 128 * 128 * ctx).sum())
+    expanded = tiles * 2 * (dim + vdim) / PREFILL_RATE + n * EXPAND_PAGE * 2 * latent * (dim + vdim) / GEMM_RATE
+    if n == 0 or expanded >= absorbed:
         return None
     if n * EXPAND_PAGE * heads * (dim + vdim) * 2 > EXPAND_BYTES:
         return None

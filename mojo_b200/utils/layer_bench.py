@@ -1,5 +1,6 @@
-"""Rekudra beside Llama at equal layer sizes: prefill and decode throughput of a few layers through the serving engine, and
-each design's own kernels against their rooflines. Random weights, synthetic prompts, one GPU (`bench.py --layer-bench`).
+"""A design beside the closest one at equal layer sizes: prefill and decode throughput of a few layers through the serving
+engine, and each design's own kernels against their rooflines. Random weights, synthetic prompts, one GPU
+(`bench.py --layer-bench`: Rekudra beside Llama; `bench.py --layer-bench rerupel`: Rerupel beside DeepSeek-V2).
 
 Steps are timed with CUDA events around the engine's device work, medians over repeats after warm-up; every step streams
 weights and caches larger than L2. Single kernels are timed with an L2 flush before each launch. Rooflines use the copy
@@ -13,8 +14,13 @@ from pathlib import Path
 
 import torch
 
+DESIGNS = {"rekudra": ("llama", "rekudra"), "rerupel": ("deepseek", "rerupel")}      # (closest model, design)
 SIZES = {"2048x16": dict(width=2048, heads=16, kv=4, dim=128, ffn=8192), "4096x32": dict(width=4096, heads=32, kv=8, dim=128, ffn=14336)}
+# DeepSeek-V2-Lite's layers, and the same at twice the width; latents of 512 columns, 64 experts of which 6 are used
+MOE_SIZES = {"2048x16": dict(width=2048, heads=16, dim=128, rank=512, rope=64, ffn=10944, experts=64, top=6, expert_ffn=1408),
+             "4096x32": dict(width=4096, heads=32, dim=128, rank=512, rope=64, ffn=14336, experts=64, top=6, expert_ffn=1408)}
 VOCAB, LAYERS = 32000, 8
+MOE_RUNS = 9           # one dense layer and eight with experts (the design: four, passed twice)
 PREFILL = [(1, 2048), (2, 2048), (8, 512)]        # (prompts, tokens each), one step
 DECODE = [(16, 1024), (128, 1024)]                # (sequences, context)
 
@@ -27,12 +33,29 @@ def peaks() -> dict:
 
 
 def model_config(design: str, size: dict):
-    from ..models.config import ModelConfig, rekudra
+    from ..models.config import ModelConfig, rekudra, rerupel
 
+    if design == "rerupel":
+        return rerupel(size["width"], 5, size["heads"], size["dim"], size["rank"], size["ffn"], VOCAB, size["experts"], size["top"], size["expert_ffn"],
+                       2 * size["expert_ffn"], (1, 5, 2))
+    if design == "deepseek":
+        return ModelConfig(architecture="deepseek_v2", hidden_size=size["width"], num_layers=MOE_RUNS, num_heads=size["heads"], num_kv_heads=size["heads"],
+                           head_dim=size["dim"] + size["rope"], intermediate_size=size["ffn"], vocab_size=VOCAB, rms_norm_eps=1e-6, rope_theta=10000.0,
+                           max_position_embeddings=4096, kv_lora_rank=size["rank"], qk_rope_head_dim=size["rope"], qk_nope_head_dim=size["dim"],
+                           v_head_dim=size["dim"], n_routed_experts=size["experts"], n_shared_experts=2, num_experts_per_tok=size["top"],
+                           moe_intermediate_size=size["expert_ffn"], first_k_dense_replace=1, rope_interleaved=True)
     if design == "rekudra":
         return rekudra(size["width"], LAYERS, size["heads"], size["kv"], size["dim"], size["ffn"], VOCAB)
     return ModelConfig(hidden_size=size["width"], num_layers=LAYERS, num_heads=size["heads"], num_kv_heads=size["kv"], head_dim=size["dim"],
                        intermediate_size=size["ffn"], vocab_size=VOCAB, max_position_embeddings=4096)
+
+
+def local_experts(size: dict, max_tokens: int):
+    from ..parallel.dist import DistInfo
+    from ..parallel.ep import EPComm
+
+    return EPComm(DistInfo(0, 1, 0, torch.device("cuda:0"), None, None), size["experts"], size["width"], size["expert_ffn"], size["top"], max_tokens=max_tokens,
+                  timeout_s=5.0)
 
 
 class Bench:
@@ -42,7 +65,12 @@ class Bench:
         n_seqs = max(b for b, _ in DECODE)
         cfg = EngineConfig(model=model_config(design, size), device="cuda:0", dtype=torch.bfloat16, page_size=128, num_pages=n_seqs * 12,
                            max_num_seqs=n_seqs, max_num_batched_tokens=4096, max_model_len=2304, autotune=autotune)
-        self.engine, self.cfg = LLMEngine(cfg), cfg
+        model = None
+        if design == "deepseek":      # its experts run through the expert-parallel kernels, here with a world of one
+            from ..models.deepseek_v2 import DeepseekV2Model
+
+            model = DeepseekV2Model(cfg.model, "cuda:0", cfg.dtype, ep=local_experts(size, cfg.max_num_batched_tokens)).init_random(0)
+        self.engine, self.cfg = LLMEngine(cfg, model=model), cfg
         self.gen = torch.Generator().manual_seed(0)
 
     def prompt(self, n: int) -> list[int]:
@@ -122,27 +150,36 @@ def step_rows(n_dec: int, chunks: list[int]):
     return ops.SeqRows(put(np.repeat(np.arange(len(lens), dtype=np.int32), lens)), put(rows), put(banks), n_dec, n_dec, len(chunks))
 
 
+class KernelTable:
+    """Rows of timed kernels: `add` times a call with a cold L2 and sets it against its roofline (bytes moved, f32
+    multiply-adds, bf16 multiply-adds)."""
+
+    def __init__(self):
+        self.pk, self.rows = peaks(), []
+        self.flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+
+    def add(self, name, design, case, fn, nbytes, fma=0.0, mma=0.0):
+        pk = self.pk
+        us = time_kernel(fn, self.flush)
+        floor = max(nbytes / pk["hbm"], fma / pk["fma"], 2 * mma / pk["bf16"]) * 1e6
+        bound = "hbm" if floor == nbytes / pk["hbm"] * 1e6 else "fma" if fma and floor == fma / pk["fma"] * 1e6 else "bf16"
+        self.rows.append({"kernel": name, "design": design, "case": case, "us": round(us, 2), "roofline_us": round(floor, 2), "bound": bound,
+                          "fraction": round(floor / us, 3)})
+
+
+def rnd(*s, dtype=torch.bfloat16, std=1.0):
+    return (torch.randn(*s, device="cuda") * std).to(dtype)
+
+
 def kernel_table(size: dict) -> list[dict]:
     from .. import ops
     from ..ops import reference
 
-    pk = peaks()
     W, H, G, d = size["width"], size["heads"], size["kv"], size["dim"]
     S, taps, page = 4, 4, 128
     dev, bf = torch.device("cuda"), torch.bfloat16
-    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
-    rows = []
-
-    def add(name, design, case, fn, nbytes, fma=0.0, mma=0.0):
-        us = time_kernel(fn, flush)
-        floor = max(nbytes / pk["hbm"], fma / pk["fma"], 2 * mma / pk["bf16"]) * 1e6
-        bound = "hbm" if floor == nbytes / pk["hbm"] * 1e6 else "fma" if fma and floor == fma / pk["fma"] * 1e6 else "bf16"
-        rows.append({"kernel": name, "design": design, "case": case, "us": round(us, 2), "roofline_us": round(floor, 2), "bound": bound,
-                     "fraction": round(floor / us, 3)})
-
-    def rnd(*s, dtype=bf, std=1.0):
-        return (torch.randn(*s, device=dev) * std).to(dtype)
-
+    tab = KernelTable()
+    add = tab.add
     table = reference.rope_table(4096, d, 1e4).to(dev)
     for case, seq, ctx, n_seq, T in (("decode 128 x 1024", step_rows(128, []), 1024, 128, 128), ("prefill 2 x 2048", step_rows(0, [2048, 2048]), 2048, 2, 4096)):
         dec = seq.n_decode > 0
@@ -191,20 +228,141 @@ def kernel_table(size: dict) -> list[dict]:
         hist = n_seq * (taps - 1) * Cd * 2 * (2 if dec else 1)
         add("delta_decode" if dec else "delta_scan + out", "rekudra", case,
             lambda: ops.delta_rule(pd, dg, dp, bd, st, seq, Cd, H, H, d, d, H * d, 1e-5), state_bytes + io + hist, fma=4.0 * T * H * d * d)
-    return rows
+    return tab.rows
+
+
+def latent_kernel_table(size: dict) -> list[dict]:
+    """Rerupel's kernels beside those of DeepSeek-V2."""
+    from .. import ops
+
+    W, H, d, R, E, k, F = size["width"], size["heads"], size["dim"], size["rank"], size["experts"], size["top"], size["expert_ffn"]
+    P, page, dev, bf = size["rope"], 128, torch.device("cuda"), torch.bfloat16
+    tab = KernelTable()
+    add, st, C = tab.add, ops._state.get(torch.device("cuda", 0)), ops._ext.require()
+    ep = local_experts(size, 4096)
+    gu, down = rnd(E, 2 * F, W, std=W ** -0.5), rnd(E, W, F, std=F ** -0.5)
+    router = rnd(E, W, std=W ** -0.5)
+    w_qk, w_kv = rnd(H * R, d, std=d ** -0.5), rnd(2 * H * d, R, std=R ** -0.5)
+    ones, w32 = torch.ones(W, device=dev, dtype=bf), torch.ones(W, device=dev)
+    for case, n_seq, ctx, T in (("decode 128 x 1024", 128, 1024, 128), ("prefill 2 x 2048", 2, 2048, 4096)):
+        dec = n_seq == T
+        per = ctx // page + 1
+        # --- residual and norm
+        x, y, res = rnd(T, W, dtype=torch.float32), rnd(T, W), rnd(T, W)
+        add("residual_norm", "rerupel", case, lambda: ops.residual_norm(x, w32, 1e-6, bf, ops.Finished(w32, y)), T * W * 12)
+        add("rmsnorm + residual", "deepseek", case, lambda: ops.rms_norm(y, ones, 1e-6, res), T * W * 8)
+        # --- attention
+        cache, mla_cache = rnd(n_seq * per, page, R), rnd(n_seq * per, page, R + P)
+        bt = torch.arange(n_seq * per, dtype=torch.int32, device=dev).view(n_seq, per)
+        cl = torch.full((n_seq,), ctx, dtype=torch.int32, device=dev)
+        cu = torch.arange(n_seq + 1, dtype=torch.int32, device=dev) * (T // n_seq)
+        base = torch.arange(n_seq, device=dev) * per * page
+        slots = base + ctx - 1 if dec else (base[:, None] + torch.arange(ctx, device=dev)[None]).flatten()
+        pos = torch.full((T,), ctx - 1, dtype=torch.int32, device=dev) if dec else torch.arange(ctx, dtype=torch.int32, device=dev).repeat(n_seq)
+        meta = ops.AttnMeta(cu, cl, bt, n_seq if dec else 0, T // n_seq, ctx)
+        proj = rnd(T, 2 * H * d + R)
+        norm = torch.ones(R, device=dev)
+        c16 = rnd(T, R)
+        add("latent_write", "rerupel", case, lambda: ops.latent_write(proj[:, H * d:H * d + R], norm, 1e-6, slots, cache), T * R * 4)
+
+        def mla_write():
+            c, _ = ops.rms_norm(c16, ones[:R], 1e-6)
+            ops.scatter_rows(c, slots, cache.view(-1, R))
+
+        add("rmsnorm, scatter", "deepseek", case, mla_write, T * R * 4)
+        rows = ops.token_rows(meta, T, dev)
+        q_lat, q_rope, gate = rnd(T, H * R), rnd(T, H, P), proj[:, H * d + R:]
+        pairs = float(n_seq * ctx) if dec else n_seq * ctx * (ctx + 1) / 2
+        if dec:
+            add("latent_attend", "rerupel", case, lambda: ops.latent_attend(q_lat, cache, meta, rows, H, 0.1, pos), n_seq * ctx * R * 2 + T * H * R * 4,
+                mma=pairs * H * 2 * R)
+            add("mla_attend", "deepseek", case, lambda: ops.mla_attend(q_lat.view(T, H, R), q_rope, mla_cache, meta, 0.1),
+                n_seq * ctx * (R + P) * 2 + T * H * (2 * R + P) * 2, mma=pairs * H * (2 * R + P))
+        else:
+            plan = ops.plan_latent_prefill(cu.cpu().numpy(), cl.cpu().numpy(), 0, R, H, d, d)
+            meta.expand = tuple(torch.from_numpy(a).cuda() for a in plan)
+            work = torch.from_numpy(ops.prefill_work_items(cu.cpu().numpy(), cl.cpu().numpy(), 0)).cuda()
+            meta.work, meta.n_items = work, work.shape[0]
+            out = torch.empty(T, H * d, device=dev, dtype=bf)
+            expand = float(len(plan[0]) * 128) * R * 2 * H * d      # multiply-adds of the expansion
+            add("latent_prefill (gather, expand, attend)", "rerupel", case,
+                lambda: ops.latent_prefill(proj[:, :H * d], cache, w_kv, meta, H, 0.1, gate, out), T * H * d * 8, mma=pairs * H * 2 * d + expand)
+            add("mla_attend", "deepseek", case, lambda: ops.mla_attend(q_lat.view(T, H, R), q_rope, mla_cache, meta, 0.1), T * H * (2 * R + P) * 2,
+                mma=pairs * H * (2 * d + P) + expand)
+        # --- per-head maps beside a plain product of the same operations
+        q = proj[:, :H * d]
+        add("head_gemm (queries)", "rerupel", case, lambda: ops.head_linear(q, w_qk, H), T * H * (d + R) * 2 + H * R * d * 2, mma=float(T) * H * R * d)
+        add("head_gemm (values, gated)", "rerupel", case, lambda: ops.head_linear(q_lat, w_kv[H * d:], H, gate=gate), T * H * (2 * d + R) * 2 + H * R * d * 2,
+            mma=float(T) * H * R * d)
+        xs, ws = rnd(T, H * d), rnd(R, H * d)
+        add("gemm_bf16, same operations", "deepseek", case, lambda: ops.linear(xs, ws), T * (H * d + R) * 2 + H * R * d * 2, mma=float(T) * H * R * d)
+        # --- experts
+        h = rnd(T, W)
+        p = ops.MoeWeights(router, gu, down, E, k, "sigmoid", False, 1.0, ops.Glu(7.0, 1.702, 1.0))
+        used = min(E, T * k)
+        wbytes, flops = used * 3 * W * F * 2, float(T) * k * 3 * W * F
+        add("router, experts", "rerupel", case, lambda: ops.moe_experts(h, p), wbytes + T * k * (3 * W + 2 * F) * 2, mma=flops)
+        l16 = rnd(T, E)
+        add("experts (dispatch, products, combine)", "deepseek", case, lambda: ep.moe(h, l16, gu, down), wbytes + T * k * (5 * W + 2 * F) * 2, mma=flops)
+        ex = ops.moe_experts(h, p)
+        add("residual_norm of expert rows", "rerupel", case, lambda: ops.residual_norm(x, w32, 1e-6, bf, ops.Finished(w32, y, ex)), T * W * (12 + 2 * k))
+        lay, ow = ep.layout, torch.empty(T, W, device=dev, dtype=bf)
+        wts = torch.rand(T, k, device=dev)
+        add("ep_combine", "deepseek", case, lambda: C.ep_combine(ep.y_local, wts, y, ow, 0, ep.peers, lay, k, (ep._calls - 1) & 1, ep.timeout_ns, st.status),
+            T * W * (4 + 6 * k))
+        logits, bn = ops.linear_f32(h, router), ops.moe.tile_rows(T * k / E)
+        ids, place, slot = (torch.empty(T, k, dtype=torch.int32, device=dev) for _ in range(3))
+        xr, tiles, nt = torch.empty(T * k, W, device=dev, dtype=bf), torch.empty(E + T * k // bn, 4, dtype=torch.int32, device=dev), torch.empty(1, dtype=torch.int32, device=dev)
+
+        def route():
+            C.moe_route(logits, wts, ids, place, st.moe_counts, E, 1, False, 1.0)
+            C.moe_gather(h, ids, place, st.moe_counts, slot, xr, tiles, nt, E, bn, st.status)
+
+        def dispatch():
+            slot_ = ep._calls & 1
+            ep._calls += 1
+            C.ep_dispatch(h, l16, wts, ids, 0, ep.peers, lay, k, False, 1.0, slot_, ep.timeout_ns, st.status)
+
+        add("moe_route, moe_gather", "rerupel", case, route, T * W * 2 * (k + 1) + T * E * 4)
+        add("ep_dispatch", "deepseek", case, dispatch, T * W * 2 * (k + 1) + T * E * 2)
+        act, yr = torch.empty(T * k, F, device=dev, dtype=bf), torch.empty(T * k, W, device=dev, dtype=bf)
+        recv, cnt = ep.region.view(lay.off_recv_x, (E * ep.cap, W), bf), ep.region.view(lay.off_recv_count + ((ep._calls - 1) & 1) * E * 4, (E,), torch.int32)
+        ebn = ep._bn(T * k / E)
+        add("expert products, gate / up", "rerupel", case, lambda: C.moe_tiles_gemm(xr, gu, tiles, nt, act, ops.EPI_SWIGLU, bn, (7.0, 1.702, 1.0, 0.0), st.status),
+            used * 2 * W * F * 2 + T * k * (W + F) * 2, mma=flops * 2 / 3)
+        add("expert products, gate / up", "deepseek", case, lambda: C.moe_grouped_gemm(recv, gu, cnt, ep.act, ep.cap, True, ebn, st.status),
+            used * 2 * W * F * 2 + T * k * (W + F) * 2, mma=flops * 2 / 3)
+        add("expert products, down", "rerupel", case, lambda: C.moe_tiles_gemm(act, down, tiles, nt, yr, ops.EPI_NONE, bn, None, st.status),
+            used * W * F * 2 + T * k * (W + F) * 2, mma=flops / 3)
+        add("expert products, down", "deepseek", case, lambda: C.moe_grouped_gemm(ep.act, down, cnt, ep.y_local, ep.cap, False, ebn, st.status),
+            used * W * F * 2 + T * k * (W + F) * 2, mma=flops / 3)
+        # --- dense feed-forward and router
+        ff = size["ffn"]
+        up, gup = rnd(ff, W, std=W ** -0.5), rnd(2 * ff, W, std=W ** -0.5)
+        add("gemm, squared ReLU", "rerupel", case, lambda: ops.linear_relu2(h, up), (ff * W + T * (W + ff)) * 2, mma=float(T) * W * ff)
+        add("gemm, SwiGLU", "deepseek", case, lambda: ops.linear_swiglu(h, gup), (2 * ff * W + T * (W + ff)) * 2, mma=2.0 * T * W * ff)
+        add("router gemm, f32", "rerupel", case, lambda: ops.linear_f32(h, router), (E * W + T * W) * 2 + T * E * 4, mma=float(T) * W * E)
+        add("router gemm", "deepseek", case, lambda: ops.linear(h, router), (E * W + T * W + T * E) * 2, mma=float(T) * W * E)
+        cat, lin = rnd(T, 2 * W), rnd(W, 2 * W, std=W ** -0.5)
+        add("loop entry gemm, f32", "rerupel", case, lambda: ops.linear_f32(cat, lin), (2 * W * W + T * 2 * W) * 2 + T * W * 4, mma=2.0 * T * W * W)
+        add("gemm of the same size", "deepseek", case, lambda: ops.linear(cat, lin), (2 * W * W + T * 3 * W) * 2, mma=2.0 * T * W * W)
+    return tab.rows
 
 
 def run(args) -> dict:
     from .clocks import ClockSampler
 
-    out = {"metric": "layer throughput, Rekudra beside Llama at equal layer sizes", "unit": "tok/s", "n_gpus": 1, "dtype": "bf16", "layers": LAYERS,
-           "data": "synthetic: uniform-random token ids, random weights", "peaks": peaks(), "sizes": {}}
+    base, design = DESIGNS[args.layer_bench]
+    sizes, table = (SIZES, kernel_table) if design == "rekudra" else (MOE_SIZES, latent_kernel_table)
+    out = {"metric": f"layer throughput, {design} beside {base} at equal layer sizes", "unit": "tok/s", "n_gpus": 1, "dtype": "bf16",
+           "layers": LAYERS if design == "rekudra" else MOE_RUNS, "data": "synthetic: uniform-random token ids, random weights", "peaks": peaks(), "sizes": {}}
     with ClockSampler(0) as clocks:
-        for name, size in SIZES.items():
-            rec = {"kernels": kernel_table(size)}
-            for design in ("llama", "rekudra"):
-                b = Bench(design, size, autotune=not args.no_autotune)
-                rec[design] = {"weight_bytes": b.engine.model.weight_bytes(), "prefill": [b.prefill(*c) for c in PREFILL], "decode": [b.decode(*c) for c in DECODE]}
+        for name, size in sizes.items():
+            rec = {"kernels": table(size)}
+            torch.cuda.empty_cache()
+            for d in (base, design):
+                b = Bench(d, size, autotune=not args.no_autotune)
+                rec[d] = {"weight_bytes": b.engine.model.weight_bytes(), "prefill": [b.prefill(*c) for c in PREFILL], "decode": [b.decode(*c) for c in DECODE]}
                 del b
                 torch.cuda.empty_cache()
             out["sizes"][name] = rec

@@ -111,7 +111,7 @@ def check(got, want, target):
         assert err.max() < 1e-4, f"worst {err.max():.2e} at {int(err.argmax())}"
         return
     sure = gaps > 0.05
-    assert err.mean() < 0.04 and (~sure).float().mean() < 0.5, f"mean {err.mean():.2e}, {int((~sure).sum())} close calls of {len(sure)}"
+    assert err.mean() < 0.04 and (len(sure) < 20 or (~sure).float().mean() < 0.6), f"mean {err.mean():.2e}, {int((~sure).sum())} close calls of {len(sure)}"
     if sure.any():
         assert err[sure].max() < 0.12, f"worst {err[sure].max():.2e} at {int((err * sure).argmax())}"
 
@@ -491,12 +491,13 @@ def test_plan_of_the_expanded_form():
     """Long portions expand, short ones do not; the pages cover every context in blocks of 128."""
     plan = lambda cu, ctx, nd, **kw: ops.plan_latent_prefill(cu, ctx, nd, **{"latent": 512, "heads": 16, "dim": 128, "vdim": 128, **kw})  # noqa: E731
     assert plan([0, 1, 2], [50, 60], 2) is None                                           # decode rows only
-    assert plan([0, 64], [1000], 0) is None and plan([0, 2], [2000], 0) is None
+    assert plan([0, 8], [1000], 0) is None and plan([0, 2], [2000], 0) is None
+    assert plan([0, 64], [1000], 0) is not None
     pages, tables = plan([0, 1, 501, 901], [70, 500, 700], 1)
     assert pages.tolist() == [[0, b] for b in range(4)] + [[1, b] for b in range(6)]
     assert tables[0, :4].tolist() == [0, 1, 2, 3] and tables[1].tolist() == [4, 5, 6, 7, 8, 9] and tables.max() < len(pages)
     assert plan([0, 4096], [1 << 20], 0, heads=128) is None                               # scratch would be too large
-    assert plan([0, 200], [200], 0, latent=64, dim=64, vdim=64) is None                   # absorbing never costs more
+    assert plan([0, 24], [2000], 0) is not None and plan([0, 24], [2000], 0, latent=256) is None    # narrow latents are cheap to attend over
 
 
 @pytest.mark.parametrize("target", TARGETS)
