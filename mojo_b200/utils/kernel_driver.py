@@ -4,7 +4,7 @@ Small, self-terminating workloads (inputs larger than the 126 MB L2, a few GB at
 profiler capture of one kernel; with `--time` the case is timed with CUDA events instead and one JSON line is printed.
 Cases: gemm_large, gemm_pair (the same product on CTA pairs), gemm_prefill, gemm_decode, gemm_swiglu, gemm_fp8,
 gemm_fp8_decode, gemm_fp8_decode_nosplit (a narrow tensor-parallel shard at 256 tokens, with and without split-K),
-attn_decode, attn_prefill, mla_decode, mla_prefill, rmsnorm, sampling (arg-max), sample_topk_topp, gemm_gguf_q4k,
+attn_decode, attn_prefill, mla_decode, mla_prefill, latent_decode, latent_prefill, moe_local, residual_norm, rmsnorm, sampling (arg-max), sample_topk_topp, gemm_gguf_q4k,
 gemm_gguf_q6k, rope_kvwrite, all_reduce_norm_single.
 """
 from __future__ import annotations
@@ -106,6 +106,38 @@ def _case(name: str):
         meta = ops.AttnMeta(cu, torch.full((S,), L, dtype=torch.int32, device=DEV), bt, 0, L, L)
         flops = 2.0 * S * H * (576 + 512) * L * (L + 1) / 2
         return (lambda: ops.mla_attend(ql, qr, cache, meta, 1 / math.sqrt(192))), flops, S * L * 576 * 2 + 2 * S * L * H * 576 * 2
+    if name == "latent_decode":
+        B, H, ctx, page, R = 128, 16, 1024, 128, 512
+        bt = torch.arange(B * ctx // page, dtype=torch.int32, device=DEV).view(B, -1)
+        cache, q = rnd(B * ctx // page, page, R, scale=0.5), rnd(B, H * R, scale=0.3)
+        cl = torch.full((B,), ctx, dtype=torch.int32, device=DEV)
+        meta = ops.AttnMeta(torch.arange(B + 1, dtype=torch.int32, device=DEV), cl, bt, B, 1, ctx)
+        return (lambda: ops.latent_attend(q, cache, meta, (cl, None), H, 0.05, cl)), 4.0 * B * H * ctx * R, B * ctx * R * 2 + 4 * B * H * R
+    if name == "latent_prefill":
+        # two prompts of 2048 tokens in the expanded form: gather, expansion product, tensor-core attention
+        S, L, H, page, R = 2, 2048, 16, 128, 512
+        bt = torch.arange(S * L // page, dtype=torch.int32, device=DEV).view(S, -1)
+        cu = torch.arange(0, (S + 1) * L, L, dtype=torch.int32, device=DEV)
+        cache, q, gate, w = rnd(S * L // page, page, R), rnd(S * L, H * 128), rnd(S * L, H * 128), rnd(2 * H * 128, R, scale=0.04)
+        meta = ops.AttnMeta(cu, torch.full((S,), L, dtype=torch.int32, device=DEV), bt, 0, L, L)
+        meta.expand = tuple(torch.from_numpy(a).to(DEV) for a in ops.plan_latent_prefill(cu.tolist(), [L] * S, 0, R, H, 128, 128))
+        out = torch.empty(S * L, H * 128, device=DEV, dtype=torch.bfloat16)
+        flops = 2.0 * S * H * 256 * L * (L + 1) / 2 + 2.0 * S * L * R * 2 * H * 128
+        return (lambda: ops.latent_prefill(q, cache, w, meta, H, 0.09, gate, out)), flops, S * L * H * 128 * 2 * 3
+    if name == "moe_local":
+        # the experts of one DeepSeek-V2-Lite-sized layer, 4096 tokens: router product, routing, permutation, two grouped products
+        T, W, F, E, k = 4096, 2048, 1408, 64, 6
+        x, router = rnd(T, W), rnd(E, W, scale=0.02)
+        p = ops.MoeWeights(router, rnd(E, 2 * F, W, scale=0.02), rnd(E, W, F, scale=0.02), E, k, "sigmoid")
+        return (lambda: ops.moe_experts(x, p)), 6.0 * T * k * W * F, (E * 3 * W * F + T * k * (3 * W + 2 * F)) * 2
+    if name == "residual_norm":
+        # a token's shared-expert row and six expert rows into the f32 residual, then the norm
+        T, W, k = 8192, 2048, 6
+        f32 = lambda *s: torch.randn(*s, generator=g, device=DEV)  # noqa: E731
+        x, ones = f32(T, W), torch.ones(W, device=DEV)
+        ex = ops.ExpertRows(rnd(T * k, W), torch.randperm(T * k, device=DEV).int().view(T, k), torch.rand(T, k, device=DEV))
+        done = ops.Finished(ones, rnd(T, W), ex)
+        return (lambda: ops.residual_norm(x, ones, 1e-6, torch.bfloat16, done)), 0.0, T * W * (8 + 4 + 2 * k)
     if name in ("tp_gemm_rs_single", "tp_ag_gemm_single"):
         # The fused tensor-parallel kernels on ONE rank (a world of one: the only peer is this GPU's own region), so that
         # their tensor-core / epilogue / staging behaviour can be captured under a profiler, which never runs on a
@@ -229,7 +261,7 @@ def _case(name: str):
 
 
 CASES = ("gemm_large", "gemm_pair", "gemm_prefill", "gemm_decode", "gemm_swiglu", "gemm_fp8", "gemm_fp8_decode", "gemm_fp8_decode_nosplit",
-         "attn_decode", "attn_prefill", "mla_decode", "mla_prefill", "rmsnorm", "sampling", "sample_topk_topp", "gemm_gguf_q4k", "gemm_gguf_q6k",
+         "attn_decode", "attn_prefill", "mla_decode", "mla_prefill", "latent_decode", "latent_prefill", "moe_local", "residual_norm", "rmsnorm", "sampling", "sample_topk_topp", "gemm_gguf_q4k", "gemm_gguf_q6k",
          "rope_kvwrite", "all_reduce_norm_single")
 # single-rank forms of the fused tensor-parallel and expert-parallel kernels (profiling only): tp_gemm_rs_single,
 # tp_ag_gemm_single, moe_ep_single
