@@ -10,10 +10,10 @@
 // rotated part.
 //
 // CTA = 4 warps on one (KV split, head group, sequence). A 32-token tile (36 KB at 512 + 64) arrives as SWIZZLE_128B
-// TMA boxes of 64 columns through a 2- or 3-stage mbarrier ring (pages below 32 tokens: one set of boxes per page). The
-// dot product is split four ways across the warps and summed through shared memory (one __syncthreads per tile, parity
-// double-buffered); each warp then owns a quarter of the output columns, so the f32 accumulator of a 512-wide latent is
-// 64 registers per thread.
+// TMA boxes of 64 columns through a 2- or 3-stage mbarrier ring (pages below 32 tokens: one set of boxes per page). Each
+// warp scores eight of the tile's tokens, with the query in registers, and hands the scores to the others through shared
+// memory (one __syncthreads per tile, parity double-buffered); all warps then do the same softmax, and each owns a quarter
+// of the output columns, so the f32 accumulator of a 512-wide latent is 64 registers per thread.
 //
 // A "row group" (grid z) is one query token: its 16 heads, the context length it may see and the block table of
 // its sequence. In decode there is one row group per sequence. A prefill chunk contributes one row group per
@@ -39,9 +39,12 @@ struct LatentShape {
   static constexpr int kRow = LAT + ROPE;                 // elements of a cache row
   static constexpr int kSub = kRow / 64;                  // boxes of 64 columns
   static constexpr int kTileBytes = kSub * BN * 128;      // 36864 at 512 + 64
-  static constexpr int kSteps = kRow / 64;                // 16-wide steps of one warp's quarter of the dot product
+  static constexpr int kSteps = kRow / 16;                // 16-wide steps of a dot product
   static constexpr int kCols = LAT / 4;                   // output columns of one warp
-  static constexpr int smem(int stages) { return stages * kTileBytes + 16 * kRow * 2 + 2 * 4 * 16 * 32 * 4 + 64 + 1024; }
+  static constexpr bool kQueryRegs = kSteps <= 36;        // the query stays in registers; wider ones are read from shared memory
+  static constexpr int kScoreLd = BN + 8;                 // row stride of the scores: 8-byte accesses of a half warp hit all banks
+  static constexpr int kScoreBytes = 2 * 16 * kScoreLd * 4;
+  static constexpr int smem(int stages) { return stages * kTileBytes + 16 * kRow * 2 + kScoreBytes + 64 + 1024; }
 };
 
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
@@ -73,12 +76,13 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
     int64_t q_rope_stride, Status* status) {
   using S = LatentShape<LAT, ROPE>;
   constexpr int kLat = LAT, kRope = ROPE, kRow = S::kRow, kSub = S::kSub, kTileBytes = S::kTileBytes, kSteps = S::kSteps, kCols = S::kCols;
+  constexpr int kScoreLd = S::kScoreLd;
   extern __shared__ uint8_t smem_raw[];
   __shared__ int sh_fail;  // set by any thread whose wait ran out; read after the per-tile barrier so all agree
   const uint32_t sbase = (ptx::smem_u32(smem_raw) + 1023u) & ~1023u;
   const uint32_t q_sm = sbase + STAGES * kTileBytes;        // [16][576] bf16, rows of 1152 bytes (72 chunks)
-  const uint32_t s_sm = q_sm + 16 * kRow * 2;               // [2][4 warps][16][32] f32
-  const uint32_t bar0 = s_sm + 2 * 4 * 16 * 32 * 4;
+  const uint32_t s_sm = q_sm + 16 * kRow * 2;               // [2][16][kScoreLd] f32
+  const uint32_t bar0 = s_sm + S::kScoreBytes;
   uint8_t* gen = smem_raw + (sbase - ptx::smem_u32(smem_raw));
   float* s_red = reinterpret_cast<float*>(gen + STAGES * kTileBytes + 16 * kRow * 2);
   __nv_bfloat16* q_gen = reinterpret_cast<__nv_bfloat16*>(gen + STAGES * kTileBytes);
@@ -102,13 +106,15 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
     for (int s = 0; s < STAGES; ++s) ptx::mbar_init(bar0 + 8 * s, 1);
     ptx::fence_mbar_init();
   }
-  auto issue = [&](int i) {
+  // past the context: any valid rows
+  auto box_pos = [&](int i, int r0) { return min((tile_begin + i) * BN + r0, (ctx - 1) / box_rows * box_rows); };
+  auto issue = [&](int i, int first_page) {
     const int s = i % STAGES;
     const uint32_t bar = bar0 + 8 * s;
     ptx::mbar_arrive_expect_tx(bar, kTileBytes);
     for (int r0 = 0; r0 < BN; r0 += box_rows) {     // one turn unless a page holds fewer tokens than a tile
-      const int pos = min((tile_begin + i) * BN + r0, (ctx - 1) / box_rows * box_rows);   // past the context: any valid rows
-      int64_t page = table[pos / page_size];
+      const int pos = box_pos(i, r0);
+      int64_t page = r0 == 0 ? first_page : table[pos / page_size];
       if (!B2_ASSERT(status, page >= 0 && page < num_pages, kSiteKvIndex, page, num_pages)) page = 0;
       const int row = static_cast<int>(page * page_size + pos % page_size);
 #pragma unroll
@@ -129,16 +135,20 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
     reinterpret_cast<uint4*>(q_gen)[r * (kRow / 8) + ((c & ~7) | ((c & 7) ^ (r & 7)))] = v;
   }
   __syncthreads();
-  if (threadIdx.x == 0)
-    for (int i = 0; i < STAGES - 1 && i < n_tiles; ++i) issue(i);
+  int ahead = 0;      // page of the next tile to be issued, looked up one turn before it is needed
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < STAGES - 1 && i < n_tiles; ++i) issue(i, table[box_pos(i, 0) / page_size]);
+    if (STAGES - 1 < n_tiles) ahead = table[box_pos(STAGES - 1, 0) / page_size];
+  }
 
-  // this warp's slice of the dot product in k-steps of 16
-  uint32_t qf[kSteps][4];
+  auto load_query = [&](int kk, uint32_t (&f)[4]) {
+    const int row = lane & 15, chunk = kk * 2 + (lane >> 4);
+    ldsm_x4(q_sm + static_cast<uint32_t>((row * (kRow / 8) + ((chunk & ~7) | ((chunk & 7) ^ (row & 7)))) * 16), f[0], f[1], f[2], f[3]);
+  };
+  uint32_t qf[S::kQueryRegs ? kSteps : 1][4];
+  if constexpr (S::kQueryRegs) {
 #pragma unroll
-  for (int kk = 0; kk < kSteps; ++kk) {
-    const int row = lane & 15, chunk = (warp * kSteps + kk) * 2 + (lane >> 4);
-    const uint32_t a = q_sm + static_cast<uint32_t>((row * (kRow / 8) + ((chunk & ~7) | ((chunk & 7) ^ (row & 7)))) * 16);
-    ldsm_x4(a, qf[kk][0], qf[kk][1], qf[kk][2], qf[kk][3]);
+    for (int kk = 0; kk < kSteps; ++kk) load_query(kk, qf[kk]);
   }
   float o[kCols / 8][4];
 #pragma unroll
@@ -156,43 +166,46 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
     }
     const uint32_t kb = sbase + st * kTileBytes;
     const int kv0 = (tile_begin + i) * BN;
-    // ---- partial S over this warp's quarter of the dims ----
+    // ---- scores of this warp's eight tokens: four independent chains over the dims ----
     float s[4][4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.0f;
-    {
-#pragma unroll
-      for (int kk = 0; kk < kSteps; ++kk) {
-#pragma unroll
-        for (int jp = 0; jp < 2; ++jp) {
-          uint32_t b0, b1, b2, b3;
-          const int row = jp * 16 + (lane & 7) + ((lane >> 4) << 3);
-          const int chunk = (warp * kSteps + kk) * 2 + ((lane >> 3) & 1);
-          ldsm_x4(kv_addr(kb, row, chunk), b0, b1, b2, b3);
-          mma16816(s[2 * jp], qf[kk], b0, b1);
-          mma16816(s[2 * jp + 1], qf[kk], b2, b3);
-        }
+    auto two_steps = [&](int k2) {
+      uint32_t b0, b1, b2, b3;
+      ldsm_x4(kv_addr(kb, warp * 8 + (lane & 7), k2 * 4 + (lane >> 3)), b0, b1, b2, b3);
+      if constexpr (S::kQueryRegs) {
+        mma16816(s[(2 * k2) & 3], qf[2 * k2], b0, b1);
+        mma16816(s[(2 * k2 + 1) & 3], qf[2 * k2 + 1], b2, b3);
+      } else {
+        uint32_t f0[4], f1[4];
+        load_query(2 * k2, f0);
+        load_query(2 * k2 + 1, f1);
+        mma16816(s[0], f0, b0, b1);
+        mma16816(s[1], f1, b2, b3);
       }
-    }
-    float* mine = s_red + ((i & 1) * 4 + warp) * 512;
+    };
+    if constexpr (S::kQueryRegs) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      *reinterpret_cast<float2*>(mine + g * 32 + j * 8 + 2 * t4) = make_float2(s[j][0], s[j][1]);
-      *reinterpret_cast<float2*>(mine + (g + 8) * 32 + j * 8 + 2 * t4) = make_float2(s[j][2], s[j][3]);
+      for (int k2 = 0; k2 < kSteps / 2; ++k2) two_steps(k2);
+    } else {
+#pragma unroll 4
+      for (int k2 = 0; k2 < kSteps / 2; ++k2) two_steps(k2);
     }
+    float* scores = s_red + (i & 1) * 16 * kScoreLd;
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+      *reinterpret_cast<float2*>(scores + (g + 8 * h) * kScoreLd + warp * 8 + 2 * t4) =
+          make_float2((s[0][2 * h] + s[1][2 * h]) + (s[2][2 * h] + s[3][2 * h]), (s[0][2 * h + 1] + s[1][2 * h + 1]) + (s[2][2 * h + 1] + s[3][2 * h + 1]));
     __syncthreads();  // every warp has finished the previous tile's P.V as well: its stage can be refilled
     if (sh_fail != 0) { ok = false; break; }
-    if (threadIdx.x == 0 && i + STAGES - 1 < n_tiles) issue(i + STAGES - 1);
+    if (threadIdx.x == 0 && i + STAGES - 1 < n_tiles) {
+      issue(i + STAGES - 1, ahead);
+      if (i + STAGES < n_tiles) ahead = table[box_pos(i + STAGES, 0) / page_size];
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      float2 lo = make_float2(0.f, 0.f), hi = make_float2(0.f, 0.f);
-#pragma unroll
-      for (int w = 0; w < 4; ++w) {
-        const float* src = s_red + ((i & 1) * 4 + w) * 512;
-        const float2 a = *reinterpret_cast<const float2*>(src + g * 32 + j * 8 + 2 * t4);
-        const float2 b = *reinterpret_cast<const float2*>(src + (g + 8) * 32 + j * 8 + 2 * t4);
-        lo.x += a.x; lo.y += a.y; hi.x += b.x; hi.y += b.y;
-      }
+      const float2 lo = *reinterpret_cast<const float2*>(scores + g * kScoreLd + j * 8 + 2 * t4);
+      const float2 hi = *reinterpret_cast<const float2*>(scores + (g + 8) * kScoreLd + j * 8 + 2 * t4);
       s[j][0] = lo.x; s[j][1] = lo.y; s[j][2] = hi.x; s[j][3] = hi.y;
     }
     // ---- online softmax (identical in all four warps) ----
