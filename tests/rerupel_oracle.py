@@ -180,7 +180,9 @@ def config(width, vocab, layers, loop=None, bigram=(97, 7, 3), eps=1e-5, scale=2
 
 def random_weights(cfg, seed=0, sharp=1.0):
     """Checkpoint tensors by name, rounded to bfloat16 values (held in float32). `sharp` scales the query projections, so
-    that single scores stand out."""
+    that single scores stand out. Routers mostly look at one channel per expert, where every token's embedding has the same
+    levels in an order of its own and the layers add little: choices vary with the token and are no close calls, which
+    rounding could decide either way."""
     g = torch.Generator().manual_seed(seed)
 
     def rnd(*shape, std):
@@ -192,13 +194,25 @@ def random_weights(cfg, seed=0, sharp=1.0):
         w["bigram"] = rnd(cfg["embedding"]["bigram"]["buckets"] + 1, W, std=0.5)
     if cfg.get("loop"):
         w["loop.in"] = torch.cat([torch.eye(W) * 0.8, torch.eye(W) * 0.3], 1) + rnd(W, 2 * W, std=0.3 * W ** -0.5)
+    C = max([s["mlp"]["router"]["experts"] for s in cfg["layers"] if s["mlp"] and s["mlp"]["kind"] == "moe"], default=0)
+    assert C <= W // 2
+    if C > 1:
+        levels = torch.linspace(-10.0, 10.0, C) / cfg["embedding"]["scale"]
+        w["embed"][:, :C] = torch.stack([levels[torch.randperm(C, generator=g)] for _ in range(cfg["vocab"])])
+        w["final.norm"][:C] = 0.02                    # the logits do not see them
+        if "bigram" in w:
+            w["bigram"][:, :C] = 0
+        if "loop.in" in w:
+            w["loop.in"][:C] = torch.cat([torch.eye(W) * 0.8, torch.eye(W) * 0.3], 1)[:C]
     for i, spec in enumerate(cfg["layers"]):
         p, m = f"l{i}.", spec["mixer"]
         H, d, e, R = m["heads"], m["dim"], m["vdim"], m["kv_rank"]
         for name in ("norm1", "norm2") if spec["mlp"] else ("norm1",):
             w[p + name] = 1 + rnd(W, std=0.2)
+            w[p + name][:C] = 1.0
         for name in ("ls1", "ls2") if spec["mlp"] else ("ls1",):
             w[p + name] = 1 + rnd(W, std=0.3)
+            w[p + name][:C] = 0.02
         for name, rows, cols, std in (("q", H * d, W, sharp), ("dkv", R, W, 1), ("uk", H * d, R, 1), ("uv", H * e, R, 1), ("g", H * e, W, 1), ("o", W, H * e, 1)):
             w[p + "mix." + name] = rnd(rows, cols, std=std * cols ** -0.5)
         w[p + "mix.dkv.norm"] = 1 + rnd(R, std=0.2)
@@ -214,8 +228,10 @@ def random_weights(cfg, seed=0, sharp=1.0):
         if mlp["kind"] == "dense":
             ff(p + "mlp.", mlp["ff"], ("up",))
         else:
-            w[p + "mlp.router"] = rnd(mlp["router"]["experts"], W, std=W ** -0.5)
-            for j in range(mlp["router"]["experts"]):
+            E = mlp["router"]["experts"]
+            w[p + "mlp.router"] = rnd(E, W, std=0.03 * W ** -0.5)
+            w[p + "mlp.router"][:, :E] += 1.5 * torch.eye(E)[torch.randperm(E, generator=g)]
+            for j in range(E):
                 ff(p + f"mlp.e{j}.", mlp["expert"]["ff"], ("gate", "up"))
             if mlp.get("shared"):
                 ff(p + "mlp.shared.", mlp["shared"]["ff"], ("gate", "up"))

@@ -37,7 +37,7 @@ def model_odd():
 def model_wide_heads():
     """Heads that fill the prefill kernel's 128 columns only in part; the loop starts at the first layer."""
     return R.config(256, 200, [
-        R.layer_spec(4, 96, 128, 256, R.moe_spec(8, 2, 64, shared=(96, 2.0))),
+        R.layer_spec(4, 96, 128, 256, R.moe_spec(8, 2, 48, shared=(112, 2.5))),
         R.layer_spec(2, 128, 72, 200, R.dense_spec(160))], loop=(0, 2, 2), bigram=(401, 3, 1))
 
 
@@ -62,12 +62,13 @@ def tokens_of(cfg, n, seed):
 
 
 def expected(name, tokens):
-    """(oracle logits of one sequence in float64, smallest gap of a router's choice per position), once per (model, tokens)."""
+    """Oracle logits of one sequence in float64, once per (model, tokens). Rounding must not decide which experts run."""
     key = (name, tuple(tokens))
     if key not in _cache:
         cfg, w = weights_of(name)
         gaps = []
-        _cache[key] = R.forward(cfg, R.as_double(w), tokens, gaps=gaps), torch.stack(gaps).amin(0) if gaps else torch.full((len(tokens),), 9.0)
+        _cache[key] = R.forward(cfg, R.as_double(w), tokens, gaps=gaps)
+        assert min((float(x.min()) for x in gaps), default=9.0) > 0.2
     return _cache[key]
 
 
@@ -103,17 +104,10 @@ def run_schedule(engine, requests, steps):
 
 
 def check(got, want, target):
-    """bf16: where two experts score almost alike rounding may pick the other one, so such positions only count in the mean."""
-    logits, gaps = want
-    err = R.relative_error(got, logits)
+    err = R.relative_error(got, want)
+    worst, mean = {"float32": (1e-4, 2e-5), "bfloat16": (0.06, 0.02)}[target[1]]
     assert torch.isfinite(got).all()
-    if target[1] == "float32":
-        assert err.max() < 1e-4, f"worst {err.max():.2e} at {int(err.argmax())}"
-        return
-    sure = gaps > 0.05
-    assert err.mean() < 0.04 and (len(sure) < 20 or (~sure).float().mean() < 0.6), f"mean {err.mean():.2e}, {int((~sure).sum())} close calls of {len(sure)}"
-    if sure.any():
-        assert err[sure].max() < 0.12, f"worst {err[sure].max():.2e} at {int((err * sure).argmax())}"
+    assert err.max() < worst and err.mean() < mean, f"worst {err.max():.2e} at {int(err.argmax())}, mean {err.mean():.2e}"
 
 
 # ------------------------------------------------------------------------------------------------------
@@ -211,9 +205,8 @@ def greedy(name, prompt, n):
     w = R.as_double(w)
     toks, margins = list(prompt), []
     for _ in range(n):
-        gaps = []
-        top = R.forward(cfg, w, toks, gaps=gaps)[-1].topk(2)
-        margins.append(min(float(top.values[0] - top.values[1]), float(torch.stack(gaps).min())))
+        top = R.forward(cfg, w, toks)[-1].topk(2)
+        margins.append(float(top.values[0] - top.values[1]))
         toks.append(int(top.indices[0]))
     return toks[len(prompt):], margins
 
@@ -279,9 +272,9 @@ def test_command_line_generate_and_replay(tmp_path, capsys, monkeypatch):
         cli.main(["replay", "--model", str(tmp_path / "m"), "--dtype", "float32", "--device", "cpu", "--out", str(tmp_path / "o"), "--max-tokens", "128"])
     assert done.value.code == 0
     assert [x for x in capsys.readouterr().out.splitlines() if x.startswith("done")] == ["done 0", "done 1", "done 2"]
-    want = expected("looped", prompt)[0]
+    want = expected("looped", prompt)
     got = [torch.from_numpy(np.fromfile(tmp_path / "o" / f"{i}.f32", dtype="<f4")).view(-1, cfg["vocab"]) for i in range(3)]
-    check(torch.cat(got), (torch.stack([want[1], want[4], want[0], want[8]]), None), ("cpu", "float32"))
+    check(torch.cat(got), torch.stack([want[1], want[4], want[0], want[8]]), ("cpu", "float32"))
 
 
 # ------------------------------------------------------------------------------------------------------
@@ -442,7 +435,7 @@ def widened(t, size, dim):
 
 @pytest.mark.parametrize("target", TARGETS)
 @pytest.mark.parametrize("page", [8, 16, 48, 64, 128])
-@pytest.mark.parametrize("heads,dim,vdim,rank", [(1, 16, 24, 64), (4, 32, 32, 128), (16, 64, 64, 512), (20, 40, 24, 96), (3, 64, 128, 1024)])
+@pytest.mark.parametrize("heads,dim,vdim,rank", [(1, 16, 24, 64), (4, 32, 48, 128), (16, 64, 64, 512), (20, 40, 24, 96), (3, 64, 128, 1024)])
 def test_latent_attention_finds_one_key(target, page, heads, dim, vdim, rank):
     """One latent's key matches the last query far better than all others: wherever it lies (first token, page borders, far
     back, the query's own place), decode rows and portions return its value."""
