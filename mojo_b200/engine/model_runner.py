@@ -16,6 +16,9 @@ launch sequence eagerly.
 """
 from __future__ import annotations
 
+import contextlib
+import gc
+
 import numpy as np
 import torch
 
@@ -24,6 +27,19 @@ from .. import ops
 
 def _align(n: int, a: int = 16) -> int:
     return (n + a - 1) // a * a
+
+
+@contextlib.contextmanager
+def _no_gc():
+    """No cyclic garbage collection inside a stream capture: it may free another engine's graphs, events or pinned memory,
+    and such a call invalidates the capture."""
+    on = gc.isenabled()
+    gc.disable()
+    try:
+        yield
+    finally:
+        if on:
+            gc.enable()
 
 
 class _Staging:
@@ -567,7 +583,7 @@ class _DecodeGraph:
         self.ep_parity = (ep._calls & 1) if ep is not None else 0
         before = ops.launch_count
         self.graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(self.graph, pool=runner.graph_pool):
+        with _no_gc(), torch.cuda.graph(self.graph, pool=runner.graph_pool):
             self.ids = run()
         if runner.graph_pool is None:
             runner.graph_pool = self.graph.pool()
@@ -707,7 +723,7 @@ class _MixedGraph:
         torch.cuda.synchronize(dev)
         before = ops.launch_count
         self.graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(self.graph, pool=runner.graph_pool):
+        with _no_gc(), torch.cuda.graph(self.graph, pool=runner.graph_pool):
             self.ids = run()
         if runner.graph_pool is None:
             runner.graph_pool = self.graph.pool()
