@@ -187,9 +187,12 @@ void gemm_f32(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, int64_t b
   const int64_t K = w.size(1);
   need(batch >= 1 && w.size(0) % batch == 0 && x.size(1) == batch * K && y.size(0) == x.size(0) && y.size(1) == w.size(0),
        "gemm_f32: x [M, batch * K], w [batch * N, K], y [M, batch * N]");
-  if (gate.has_value())
-    need(gate->is_cuda() && gate->scalar_type() == at::kFloat && gate->dim() == 2 && gate->stride(1) == 1 && gate->sizes() == y.sizes(), "gemm_f32: gate f32 like y");
   B2GemmF32Args a{};
+  if (gate.has_value()) {
+    need(gate->is_cuda() && gate->scalar_type() == at::kFloat && gate->dim() == 2 && gate->stride(1) == 1 && gate->size(0) == y.size(0) &&
+             (gate->size(1) == y.size(1) || gate->size(1) == batch), "gemm_f32: gate f32 like y, or one column per product");
+    a.gate_heads = gate->size(1) == y.size(1) ? 0 : 1;
+  }
   a.x = x.data_ptr<float>();
   a.w = w.data_ptr<float>();
   a.y = y.data_ptr<float>();
@@ -211,13 +214,21 @@ void gemm_f32(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, int64_t b
 void residual_norm(at::Tensor& x, const OptTensor& y, const OptTensor& experts, const OptTensor& slot, const OptTensor& expert_w, const OptTensor& y_scale,
                    const OptTensor& weight, at::Tensor& h, const OptTensor& ids, const OptTensor& embed, double embed_scale, const OptTensor& prev,
                    const OptTensor& bigram, int64_t mul_prev, int64_t mul_cur, const OptTensor& x0, const OptTensor& rows_index, bool store, double eps,
-                   int64_t mean_width, const OptTensor& status) {
+                   int64_t mean_width, const OptTensor& status, const OptTensor& bias, const OptTensor& own, const OptTensor& gated,
+                   const OptTensor& gate) {
   need(x.dim() == 2 && x.is_cuda() && x.scalar_type() == at::kFloat && x.is_contiguous(), "residual_norm: x must be contiguous CUDA f32 [rows, width]");
   const int64_t T = x.size(0), W = x.size(1);
   need(is_act(h) && h.dim() == 2 && h.stride(1) == 1 && h.size(1) == W, "residual_norm: h [n, width]");
   B2ResidualArgs a{};
   if (y.has_value()) need(y->scalar_type() == h.scalar_type() && y->is_contiguous() && y->numel() == T * W, "residual_norm: y [rows, width] like h");
-  if (y.has_value() || experts.has_value()) need(y_scale.has_value() && is_f32(*y_scale, W), "residual_norm: y_scale f32 [width]");
+  if (y_scale.has_value()) need(is_f32(*y_scale, W), "residual_norm: y_scale f32 [width]");
+  if (bias.has_value()) need(weight.has_value() && is_f32(*bias, W), "residual_norm: bias f32 [width] beside a weight");
+  for (const OptTensor* t : {&own, &gated})
+    if (t->has_value()) need((*t)->scalar_type() == h.scalar_type() && (*t)->is_contiguous() && (*t)->numel() == T * W, "residual_norm: own, gated [rows, width] like h");
+  if (gated.has_value()) {
+    need(gate.has_value() && gate->is_cuda() && gate->scalar_type() == at::kFloat && gate->dim() == 1 && gate->size(0) == T, "residual_norm: gate f32 [rows]");
+    a.ld_gate = gate->stride(0);
+  }
   if (weight.has_value()) need(is_f32(*weight, W), "residual_norm: weight f32 [width]");
   if (experts.has_value()) {
     need(experts->scalar_type() == h.scalar_type() && experts->dim() == 2 && experts->is_contiguous() && experts->size(1) == W && slot.has_value() &&
@@ -254,6 +265,10 @@ void residual_norm(at::Tensor& x, const OptTensor& y, const OptTensor& experts, 
   a.bigram = opt<const void>(bigram);
   a.x0 = opt<void>(x0);
   a.rows_index = opt<const int64_t>(rows_index);
+  a.bias = opt<const float>(bias);
+  a.own = opt<const void>(own);
+  a.gated = opt<const void>(gated);
+  a.gate = gated.has_value() ? opt<const float>(gate) : nullptr;
   a.ld_h = h.stride(0);
   a.mul_prev = mul_prev;
   a.mul_cur = mul_cur;
@@ -270,23 +285,105 @@ void residual_norm(at::Tensor& x, const OptTensor& y, const OptTensor& experts, 
 }
 
 void attn_f32(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out, const at::Tensor& row_seq,
-              const at::Tensor& positions, const at::Tensor& block_tables, double scale, const OptTensor& gate, const OptTensor& status) {
-  need(q.is_cuda() && q.scalar_type() == at::kFloat && q.dim() == 2 && q.is_contiguous() && out.is_contiguous() && out.scalar_type() == at::kFloat,
-       "attn_f32: q, out contiguous CUDA f32");
-  need(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.scalar_type() == at::kFloat &&
-           v_cache.scalar_type() == at::kFloat && k_cache.size(0) == v_cache.size(0) && k_cache.size(1) == v_cache.size(1) && k_cache.size(2) == v_cache.size(2),
+              const at::Tensor& positions, const at::Tensor& block_tables, double scale, const OptTensor& gate, const OptTensor& status, int64_t window,
+              double softcap, double out_scale) {
+  need(q.is_cuda() && q.scalar_type() == at::kFloat && q.dim() == 2 && q.is_contiguous() && out.scalar_type() == at::kFloat && out.dim() == 2 &&
+           out.stride(1) == 1, "attn_f32: q contiguous CUDA f32, out f32 with unit inner stride");
+  // values: a cache like the keys', or the first columns of one
+  need(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && k_cache.scalar_type() == at::kFloat && v_cache.scalar_type() == at::kFloat &&
+           k_cache.size(0) == v_cache.size(0) && k_cache.size(1) == v_cache.size(1) && k_cache.size(2) == v_cache.size(2) && v_cache.stride(3) == 1 &&
+           v_cache.stride(1) == v_cache.size(2) * v_cache.stride(2) && v_cache.stride(0) == v_cache.size(1) * v_cache.stride(1),
        "attn_f32: f32 caches [pages, n_kv, page, D]");
   const int64_t T = q.size(0), D = k_cache.size(3), n_q = q.size(1) / D;
   need(n_q * D == q.size(1) && out.size(0) == T && out.size(1) == n_q * v_cache.size(3), "attn_f32: shape mismatch");
-  need(is_i32(row_seq) && is_i32(positions) && is_i32(block_tables) && row_seq.numel() == T && positions.numel() == T && block_tables.dim() == 2, "attn_f32: int32 metadata");
+  need(is_i32(row_seq) && is_i32(positions) && is_i32(block_tables) && row_seq.numel() >= T && positions.numel() >= T && block_tables.dim() == 2, "attn_f32: int32 metadata");
   if (gate.has_value()) need(gate->scalar_type() == at::kFloat && gate->dim() == 2 && gate->size(0) == T && gate->size(1) == n_q && gate->stride(1) == 1, "attn_f32: gate f32 [T, n_q]");
   c10::cuda::CUDAGuard g(q.device());
   check(b2_attn_f32(q.data_ptr<float>(), k_cache.data_ptr<float>(), v_cache.data_ptr<float>(), out.data_ptr<float>(), row_seq.data_ptr<int32_t>(),
                     positions.data_ptr<int32_t>(), block_tables.data_ptr<int32_t>(), static_cast<int>(T), static_cast<int>(block_tables.size(0)),
                     static_cast<int>(block_tables.size(1)), static_cast<int>(n_q), static_cast<int>(k_cache.size(1)), static_cast<int>(D),
-                    static_cast<int>(v_cache.size(3)), static_cast<int>(k_cache.size(2)), static_cast<float>(scale), k_cache.size(0),
+                    static_cast<int>(v_cache.size(3)), v_cache.stride(2), out.stride(0), static_cast<int>(k_cache.size(2)), static_cast<float>(scale),
+                    static_cast<int>(window), static_cast<float>(softcap), static_cast<float>(out_scale), k_cache.size(0),
                     gate.has_value() ? gate->data_ptr<float>() : nullptr, gate.has_value() ? gate->stride(0) : 0, status_ptr(status), cur_stream()),
         "attn_f32");
+}
+
+void norm_qkv(const at::Tensor& proj, const at::Tensor& bias, const at::Tensor& q_norm, const at::Tensor& k_norm, const at::Tensor& cos_sin,
+              const at::Tensor& positions, const at::Tensor& slots, at::Tensor& k_cache, at::Tensor& v_cache, at::Tensor& q_out, int64_t heads,
+              int64_t kv_heads, int64_t dim, int64_t vdim, double eps, const OptTensor& status) {
+  need(is_act(proj) && proj.dim() == 2 && proj.stride(1) == 1, "norm_qkv: proj must be 2-D with unit inner stride");
+  const int64_t T = proj.size(0), channels = heads * dim + kv_heads * (dim + vdim);
+  need(proj.size(1) >= channels && is_f32(bias, channels) && is_f32(q_norm, heads * dim) && is_f32(k_norm, kv_heads * dim), "norm_qkv: f32 parameters, proj as wide");
+  need(cos_sin.is_cuda() && cos_sin.scalar_type() == at::kFloat && cos_sin.is_contiguous() && cos_sin.dim() == 2, "norm_qkv: cos_sin f32 [max_pos, rot]");
+  need(is_i32(positions) && positions.numel() == T && is_i64(slots) && slots.numel() == T, "norm_qkv: positions int32 [T], slots int64 [T]");
+  need(q_out.scalar_type() == proj.scalar_type() && q_out.is_contiguous() && q_out.size(0) == T && q_out.size(1) % heads == 0, "norm_qkv: q_out [T, heads * pad]");
+  need(k_cache.dim() == 4 && v_cache.dim() == 4 && k_cache.is_contiguous() && v_cache.is_contiguous() && k_cache.scalar_type() == proj.scalar_type() &&
+           v_cache.scalar_type() == proj.scalar_type() && k_cache.size(1) == kv_heads && v_cache.size(1) == kv_heads &&
+           k_cache.size(0) == v_cache.size(0) && k_cache.size(2) == v_cache.size(2) && k_cache.size(3) == q_out.size(1) / heads,
+       "norm_qkv: caches [pages, kv_heads, page, pad] like proj, keys padded like the queries");
+  B2NormQkvArgs a{};
+  a.proj = proj.data_ptr();
+  a.ld = proj.stride(0);
+  a.bias = bias.data_ptr<float>();
+  a.q_norm = q_norm.data_ptr<float>();
+  a.k_norm = k_norm.data_ptr<float>();
+  a.cos_sin = cos_sin.data_ptr<float>();
+  a.positions = positions.data_ptr<int32_t>();
+  a.slots = slots.data_ptr<int64_t>();
+  a.q_out = q_out.data_ptr();
+  a.k_cache = k_cache.data_ptr();
+  a.v_cache = v_cache.data_ptr();
+  a.num_slots = k_cache.size(0) * k_cache.size(2);
+  a.rows = static_cast<int32_t>(T);
+  a.heads = static_cast<int32_t>(heads);
+  a.kv_heads = static_cast<int32_t>(kv_heads);
+  a.dim = static_cast<int32_t>(dim);
+  a.vdim = static_cast<int32_t>(vdim);
+  a.pad_dim = static_cast<int32_t>(k_cache.size(3));
+  a.pad_vdim = static_cast<int32_t>(v_cache.size(3));
+  a.rot = static_cast<int32_t>(cos_sin.size(1));
+  a.page_size = static_cast<int32_t>(k_cache.size(2));
+  a.max_pos = static_cast<int32_t>(cos_sin.size(0));
+  a.eps = static_cast<float>(eps);
+  c10::cuda::CUDAGuard g(proj.device());
+  check(b2_norm_qkv(&a, proj.scalar_type() == at::kFloat ? 1 : 0, status_ptr(status), cur_stream()), "norm_qkv");
+}
+
+void gated_linear(const at::Tensor& proj, const at::Tensor& z, const at::Tensor& decay_bias, const at::Tensor& norm_w, double tau, at::Tensor& state,
+                  const at::Tensor& row_seq, const at::Tensor& seq_rows, const at::Tensor& seq_state, at::Tensor& out, const at::Tensor& scratch, int64_t heads,
+                  int64_t dim, int64_t vdim, double eps, double out_scale, int64_t n_decode, int64_t first, int64_t n_prefill, const OptTensor& status) {
+  need(is_act(proj) && proj.dim() == 2 && proj.stride(1) == 1 && out.scalar_type() == proj.scalar_type() && out.dim() == 2 && out.stride(1) == 1 &&
+           z.is_cuda() && z.scalar_type() == at::kFloat && z.dim() == 2 && z.stride(1) == 1, "gated_linear: proj and out of one type, z f32, unit inner strides");
+  const int64_t T = proj.size(0);
+  need(proj.size(1) == 2 * heads * (dim + vdim) && z.size(0) == T && z.size(1) >= heads * dim && out.size(0) == T && out.size(1) == heads * vdim &&
+           row_seq.numel() == T && tau > 0.0, "gated_linear: shape mismatch");
+  need(is_f32(decay_bias, heads * dim) && is_f32(norm_w, vdim), "gated_linear: f32 parameters");
+  need(state.dim() == 4 && state.is_cuda() && state.scalar_type() == at::kFloat && state.is_contiguous() && state.size(1) == heads && state.size(2) == dim &&
+           state.size(3) == vdim, "gated_linear: state f32 [slots, heads, dim, vdim]");
+  const B2SeqRows s = seq_rows_of(row_seq, seq_rows, seq_state, 2 * state.size(0));
+  B2GatedLinearArgs a{};
+  a.proj = proj.data_ptr();
+  a.z = z.data_ptr<float>();
+  a.ld = proj.stride(0);
+  a.ld_z = z.stride(0);
+  a.decay_bias = decay_bias.data_ptr<float>();
+  a.norm_w = norm_w.data_ptr<float>();
+  a.state = state.data_ptr<float>();
+  a.out = out.data_ptr();
+  a.ld_out = out.stride(0);
+  a.heads = static_cast<int32_t>(heads);
+  a.dim = static_cast<int32_t>(dim);
+  a.vdim = static_cast<int32_t>(vdim);
+  a.inv_tau = static_cast<float>(1.0 / tau);
+  a.eps = static_cast<float>(eps);
+  a.out_scale = static_cast<float>(out_scale);
+  if (n_prefill > 0) {
+    need(is_f32(scratch, b2_gated_linear_scratch_floats(a.heads, a.dim, a.vdim, s.rows)), "gated_linear: f32 scratch of gated_linear_scratch_floats elements");
+    a.scratch = scratch.data_ptr<float>();
+  }
+  c10::cuda::CUDAGuard g(proj.device());
+  check(b2_gated_linear(&a, &s, static_cast<int>(n_decode), static_cast<int>(first), static_cast<int>(n_prefill), proj.scalar_type() == at::kFloat ? 1 : 0,
+                        status_ptr(status), cur_stream()), "gated_linear");
 }
 }  // namespace
 
@@ -297,10 +394,20 @@ void bind_mixers(py::module_& m) {
   m.def("delta_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows, int64_t seqs) {
     return b2_delta_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows), static_cast<int>(seqs));
   });
-  m.def("residual_norm", &residual_norm);
+  m.def("norm_qkv", &norm_qkv);
+  m.def("gated_linear", &gated_linear);
+  m.def("gated_linear_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows) {
+    return b2_gated_linear_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows));
+  });
+  m.def("residual_norm", &residual_norm, py::arg("x"), py::arg("y"), py::arg("experts"), py::arg("slot"), py::arg("expert_w"), py::arg("y_scale"),
+        py::arg("weight"), py::arg("h"), py::arg("ids"), py::arg("embed"), py::arg("embed_scale"), py::arg("prev"), py::arg("bigram"), py::arg("mul_prev"),
+        py::arg("mul_cur"), py::arg("x0"), py::arg("rows_index"), py::arg("store"), py::arg("eps"), py::arg("mean_width"), py::arg("status") = py::none(),
+        py::arg("bias") = py::none(), py::arg("own") = py::none(), py::arg("gated") = py::none(), py::arg("gate") = py::none());
   m.def("gemm_f32", &gemm_f32, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("batch") = 1, py::arg("epilogue") = 0, py::arg("cap") = 0.0,
         py::arg("gate") = py::none());
-  m.def("attn_f32", &attn_f32);
+  m.def("attn_f32", &attn_f32, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("row_seq"), py::arg("positions"),
+        py::arg("block_tables"), py::arg("scale"), py::arg("gate") = py::none(), py::arg("status") = py::none(), py::arg("window") = 0,
+        py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0);
   m.def("glu_f32", [](const at::Tensor& gu, at::Tensor& out, double limit, double alpha, double up_bias) {
     need(gu.is_cuda() && gu.scalar_type() == at::kFloat && gu.is_contiguous() && out.is_contiguous() && out.scalar_type() == at::kFloat &&
              gu.size(0) == out.size(0) && gu.size(1) == 2 * out.size(1), "glu_f32: gate_up [M, 2F], out [M, F], contiguous CUDA f32");

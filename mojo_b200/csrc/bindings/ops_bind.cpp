@@ -197,7 +197,7 @@ int64_t gate_ld(const c10::optional<at::Tensor>& gate) { return gate.has_value()
 
 void attn_prefill(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out,
                   const at::Tensor& cu_q, const at::Tensor& ctx_lens, const at::Tensor& block_tables, int64_t head_dim,
-                  int64_t max_q_len, double scale, c10::optional<at::Tensor> status, c10::optional<at::Tensor> gate) {
+                  int64_t max_q_len, double scale, c10::optional<at::Tensor> status, c10::optional<at::Tensor> gate, int64_t window, double softcap, double out_scale) {
   check_cache(q, k_cache, v_cache, head_dim);
   need(out.dim() == 2 && out.stride(1) == 1 && is_bf16(out) && out.size(0) == q.size(0), "attention: bad out");
   need(cu_q.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt && block_tables.scalar_type() == at::kInt, "attention: metadata must be int32");
@@ -210,7 +210,8 @@ void attn_prefill(const at::Tensor& q, const at::Tensor& k_cache, const at::Tens
                              static_cast<int>(block_tables.size(1)), static_cast<int>(q.size(1) / head_dim),
                              static_cast<int>(k_cache.size(1)), static_cast<int>(head_dim), static_cast<int>(k_cache.size(2)),
                              static_cast<int>(max_q_len), static_cast<float>(scale), q.stride(0), out.stride(0),
-                             k_cache.size(0), gate_ptr(gate, q, q.size(1) / head_dim), gate_ld(gate), status_ptr(status), cur_stream()),
+                             k_cache.size(0), gate_ptr(gate, q, q.size(1) / head_dim), gate_ld(gate), static_cast<int>(window), static_cast<float>(softcap),
+                             static_cast<float>(out_scale), status_ptr(status), cur_stream()),
         "attn_prefill");
 }
 
@@ -236,7 +237,8 @@ void gemm_bf16_pair(const at::Tensor& x, const at::Tensor& w, at::Tensor& y, int
 void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out,
                      const at::Tensor& cu_q, const at::Tensor& ctx_lens, const at::Tensor& block_tables, int64_t max_q_len,
                      double scale, c10::optional<at::Tensor> status, c10::optional<at::Tensor> work,
-                     c10::optional<at::Tensor> n_work, int64_t work_items, c10::optional<at::Tensor> gate) {
+                     c10::optional<at::Tensor> n_work, int64_t work_items, c10::optional<at::Tensor> gate, int64_t window, double softcap,
+                     double out_scale) {
   // contiguous paged caches, or a [pages, n_kv, 128, 128] view of matrices with one row per token and all heads in it
   const int64_t token_stride = k_cache.is_contiguous() ? 0 : k_cache.stride(2);
   if (token_stride == 0) check_cache(q, k_cache, v_cache, 128);
@@ -265,14 +267,14 @@ void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::T
                                 work.has_value() ? work->data_ptr<int32_t>() : nullptr,
                                 work.has_value() && n_work.has_value() ? n_work->data_ptr<int32_t>() : nullptr,
                                 static_cast<int>(work_items), gate_ptr(gate, q, gate_elems ? q.size(1) : q.size(1) / 128), gate_ld(gate), gate_elems ? 1 : 0,
-                                status_ptr(status), cur_stream()),
+                                static_cast<int>(window), static_cast<float>(softcap), static_cast<float>(out_scale), status_ptr(status), cur_stream()),
         "attn_prefill_tc");
 }
 
 void attn_decode(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out,
                  const at::Tensor& ctx_lens, const at::Tensor& block_tables, c10::optional<at::Tensor> workspace,
                  int64_t head_dim, int64_t num_splits, double scale, c10::optional<at::Tensor> status,
-                 c10::optional<at::Tensor> counters, c10::optional<at::Tensor> gate) {
+                 c10::optional<at::Tensor> counters, c10::optional<at::Tensor> gate, int64_t window, double softcap, double out_scale) {
   check_cache(q, k_cache, v_cache, head_dim);
   need(out.dim() == 2 && out.stride(1) == 1 && is_bf16(out) && out.size(0) == q.size(0), "attention: bad out");
   need(ctx_lens.scalar_type() == at::kInt && block_tables.scalar_type() == at::kInt && block_tables.dim() == 2 && block_tables.is_contiguous(), "attention: metadata must be contiguous int32");
@@ -296,7 +298,8 @@ void attn_decode(const at::Tensor& q, const at::Tensor& k_cache, const at::Tenso
                             block_tables.data_ptr<int32_t>(), ws, batch, static_cast<int>(block_tables.size(1)), n_q,
                             static_cast<int>(k_cache.size(1)), static_cast<int>(head_dim), static_cast<int>(k_cache.size(2)),
                             static_cast<int>(num_splits), static_cast<float>(scale), q.stride(0), out.stride(0),
-                            k_cache.size(0), cnt, gate_ptr(gate, q, n_q), gate_ld(gate), status_ptr(status), cur_stream()),
+                            k_cache.size(0), cnt, gate_ptr(gate, q, n_q), gate_ld(gate), static_cast<int>(window), static_cast<float>(softcap),
+                            static_cast<float>(out_scale), status_ptr(status), cur_stream()),
         "attn_decode");
 }
 
@@ -365,15 +368,15 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("top_p") = py::none(), py::arg("uniforms") = py::none(), py::arg("seed") = 0, py::arg("step") = 0);
   m.def("attn_prefill", &attn_prefill, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("cu_q"),
         py::arg("ctx_lens"), py::arg("block_tables"), py::arg("head_dim"), py::arg("max_q_len"), py::arg("scale"),
-        py::arg("status") = py::none(), py::arg("gate") = py::none());
+        py::arg("status") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0);
   m.def("gemm_bf16_pair", &gemm_bf16_pair, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("epilogue") = 0, py::arg("bn") = 256, py::arg("status") = py::none(), py::arg("act") = py::none());
   m.def("attn_prefill_tc", &attn_prefill_tc, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("cu_q"),
         py::arg("ctx_lens"), py::arg("block_tables"), py::arg("max_q_len"), py::arg("scale"),
         py::arg("status") = py::none(), py::arg("work") = py::none(), py::arg("n_work") = py::none(), py::arg("work_items") = 0,
-        py::arg("gate") = py::none());
+        py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0);
   m.def("attn_decode", &attn_decode, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("ctx_lens"),
         py::arg("block_tables"), py::arg("workspace"), py::arg("head_dim"), py::arg("num_splits"), py::arg("scale"),
-        py::arg("status") = py::none(), py::arg("counters") = py::none(), py::arg("gate") = py::none());
+        py::arg("status") = py::none(), py::arg("counters") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0);
   m.def("gemm_bf16", &gemm_bf16, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("residual") = py::none(),
         py::arg("epilogue") = 0, py::arg("config") = 0, py::arg("workspace") = py::none(), py::arg("status") = py::none(), py::arg("act") = py::none());
   m.def("gemm_workspace_bytes", [](int M, int N, int K) { return b2_gemm_workspace_bytes(M, N, K); });

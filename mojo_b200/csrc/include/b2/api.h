@@ -64,12 +64,14 @@ int b2_sample(const void* logits, int is_bf16, int64_t* ids, const float* temper
 // q/out: [T, n_q, D]; cache: [num_pages, n_kv, page_size, D]; cu_q: [B+1] query offsets; ctx_lens: [B]
 // total context (cached prefix + this chunk); block_tables: [B, max_blocks]. D == 64, 128 or 256.
 // `gate` (may be null), in this and the two kernels below: bf16 [T, n_q] with row stride `gate_stride`; head h of query
-// row t is multiplied by sigmoid(gate[t, h]) before it is rounded.
+// row t is multiplied by sigmoid(gate[t, h]) before it is rounded. `window`, in all three: positions a row sees, its own
+// included (<= 0: all of them); `softcap`: scores become softcap * tanh(score / softcap) (<= 0: they do not); `out_scale`:
+// factor of the result.
 int b2_attn_prefill_bf16(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* cu_q,
                          const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                          int n_kv, int head_dim, int page_size, int max_q_len, float scale, int64_t q_stride,
-                         int64_t out_stride, int64_t num_pages, const void* gate, int64_t gate_stride,
-                         b2::Status* status, cudaStream_t stream);
+                         int64_t out_stride, int64_t num_pages, const void* gate, int64_t gate_stride, int window,
+                         float softcap, float out_scale, b2::Status* status, cudaStream_t stream);
 // bf16 GEMM on CTA pairs (tcgen05 cta_group::2, 256 x 256 tiles; csrc/kernels/gemm_bf16_pair.cu). Epilogue NONE, SWIGLU
 // or RELU2.
 int b2_gemm_bf16_pair(const void* x, const void* w, void* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,
@@ -82,7 +84,8 @@ int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const void* v_ca
                             const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                             int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
                             int64_t num_pages, int64_t token_stride, const int32_t* work, const int32_t* n_work, int work_items,
-                            const void* gate, int64_t gate_stride, int gate_elems, b2::Status* status, cudaStream_t stream);
+                            const void* gate, int64_t gate_stride, int gate_elems, int window, float softcap, float out_scale,
+                            b2::Status* status, cudaStream_t stream);
 // One query token per sequence, split over the KV length. workspace: f32, size from b2_attn_decode_workspace.
 // `counters` (may be null): u32 [batch * n_kv], zero before the first use and left at zero by every launch; with it
 // (and page sizes that are multiples of 32) the split that finishes last merges the partials itself, otherwise a
@@ -91,7 +94,7 @@ int b2_attn_decode_bf16(const void* q, const void* k_cache, const void* v_cache,
                         const int32_t* block_tables, float* workspace, int batch, int max_blocks, int n_q, int n_kv,
                         int head_dim, int page_size, int num_splits, float scale, int64_t q_stride,
                         int64_t out_stride, int64_t num_pages, uint32_t* counters, const void* gate, int64_t gate_stride,
-                        b2::Status* status, cudaStream_t stream);
+                        int window, float softcap, float out_scale, b2::Status* status, cudaStream_t stream);
 int64_t b2_attn_decode_counter_bytes(int batch, int n_kv);
 int64_t b2_attn_decode_workspace(int batch, int n_q, int head_dim, int num_splits);
 // MLA decode with absorbed weights: q_lat [B, H, 512], q_rope [B, H, 64]; cache [num_pages, page, 576]
@@ -108,11 +111,12 @@ int b2_mla_attend_bf16(const void* q_lat, const void* q_rope, const void* kv_cac
                        const int32_t* block_tables, const int32_t* row_seq, float* workspace, int rows, int max_blocks,
                        int n_heads, int page_size, int num_splits, float scale, int64_t num_pages, int64_t q_lat_stride,
                        int64_t q_rope_stride, b2::Status* status, cudaStream_t stream);
-// The same attention without a rotated part, for latents of 64, 128, 256, 512 or 1024 columns (cache [num_pages, page, latent],
-// page a multiple of 8; out_lat [rows, H, latent]).
-int b2_latent_attend_bf16(const void* q_lat, const void* cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
-                          const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int latent, int page_size,
-                          int num_splits, float scale, int64_t num_pages, int64_t q_lat_stride, b2::Status* status, cudaStream_t stream);
+// The same attention for latents of 64, 128, 256, 512 or 1024 columns and a rotated part of 0, 64 or 128 (cache [num_pages, page,
+// latent + rot], page a multiple of 8; out_lat [rows, H, latent]); a head's two query parts lie side by side. `window`:
+// positions a row sees, its own included (<= 0: all).
+int b2_latent_attend_bf16(const void* q, const void* cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
+                          const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int latent, int rot, int page_size,
+                          int num_splits, float scale, int window, int64_t num_pages, int64_t q_stride, b2::Status* status, cudaStream_t stream);
 int64_t b2_latent_attend_workspace(int rows, int n_heads, int latent, int num_splits);
 // row_ctx[t] / row_seq[t] for every token t of a batch described by cu_q [num_seqs + 1] and ctx_lens [num_seqs]:
 // token i of a sequence's chunk sees ctx - q_len + i + 1 positions (causal mask of chunked prefill; decode rows: ctx).

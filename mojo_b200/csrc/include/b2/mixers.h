@@ -1,6 +1,6 @@
 // C launch API of the sequence-mixing kernels beyond plain attention: residual streams with learned mixing
-// (hyper-connections), short causal convolutions in front of attention, the gated delta rule, and the 32-bit
-// forms of the matrix product and of paged attention. Conventions as in b2/api.h: raw device pointers, a stream, 0 or
+// (hyper-connections), short causal convolutions or whole-row norms in front of attention, the gated delta rule, gated linear
+// attention, and the 32-bit forms of the matrix product and of paged attention. Conventions as in b2/api.h: raw device pointers, a stream, 0 or
 // a negative code back. `f32` selects the element type of activations and caches (0: bf16, 1: f32); parameters that
 // enter 32-bit arithmetic (norm weights, mixing coefficients, convolution taps, decay constants) are always f32.
 #pragma once
@@ -46,7 +46,9 @@ int b2_hyper_norm(const B2HyperArgs* a, int f32, b2::Status* status, cudaStream_
 
 // One f32 residual stream x [rows, width] with a scale per channel. For every row: x += y_scale * (y + sum_j w[j] e[slot[j]]),
 // where y (a sublayer's output) and the expert rows e (`top` of them per row, w and slot [rows, top]) may each be null;
-// then h = rms_norm(x) * weight, or x itself rounded where weight is null. With `ids` x starts as
+// a row of e with slot -1 is own[row]. `gated` (may be null) is one more addend with a factor sigmoid(gate[row * ld_gate]); y_scale
+// null: one. Then h = rms_norm(x) * weight, layer_norm(x) * weight + bias where a bias is given, or x itself rounded where weight
+// is null. With `ids` x starts as
 // embed[id] * embed_scale (+ bigram[(prev * mul_prev + id * mul_cur) mod buckets], or its last row, number `buckets`, where
 // prev is -1) instead of being read, and x0 (may be null) receives a rounded copy of that. `store` writes x back. With
 // `rows_index` only those rows are processed and h is compact. Columns from `mean_width` up to `width` are zero padding.
@@ -65,7 +67,11 @@ struct B2ResidualArgs {
   const void* bigram;
   void* x0;
   const int64_t* rows_index;
-  int64_t ld_h, ld_x0, mul_prev, mul_cur, buckets;
+  const float* bias;
+  const void* own;
+  const void* gated;
+  const float* gate;
+  int64_t ld_h, ld_x0, mul_prev, mul_cur, buckets, ld_gate;
   float embed_scale, eps;
   int32_t top, expert_rows, n_out, rows, width, mean_width, vocab, store;
 };
@@ -92,6 +98,49 @@ struct B2ConvQkvArgs {
   float eps;
 };
 int b2_conv_qkv(const B2ConvQkvArgs* a, const B2SeqRows* s, int f32, b2::Status* status, cudaStream_t stream);
+
+// Front end of attention with norms over whole rows: biases on the q | k | v columns of a projection, one RMS norm (weights
+// q_norm, k_norm) over all q columns of a row and one over its k columns, rotary embedding of the first `rot` columns of every q
+// and k head (halves pair up), scatter of k and v into the paged cache. Layouts as above; bias f32 [channels].
+struct B2NormQkvArgs {
+  const void* proj;
+  int64_t ld;
+  const float* bias;
+  const float* q_norm;
+  const float* k_norm;
+  const float* cos_sin;       // [max_pos, rot]
+  const int32_t* positions;   // [rows]
+  const int64_t* slots;       // [rows], -1: nothing is cached
+  void* q_out;
+  void* k_cache;
+  void* v_cache;
+  int64_t num_slots;
+  int32_t rows, heads, kv_heads, dim, vdim, pad_dim, pad_vdim, rot, page_size, max_pos;
+  float eps;
+};
+int b2_norm_qkv(const B2NormQkvArgs* a, int f32, b2::Status* status, cudaStream_t stream);
+
+// Gated linear attention. Per head, with S [dim, vdim], all of it in f32:
+//   a = sigmoid(z + decay_bias)^(1 / tau) (one per key channel),  S <- diag(a) S + k v^T,  o = S^T q dim^-0.5
+// out = rms_norm(o) * norm_w * silu(gate) * out_scale. proj [rows, ld]: q | k (heads * dim each) | v | gate (heads * vdim each)
+// from column 0; z f32 [rows, ld_z]; state f32 [slots, heads, dim, vdim], updated in place.
+struct B2GatedLinearArgs {
+  const void* proj;
+  const float* z;
+  int64_t ld, ld_z;
+  const float* decay_bias;    // [heads * dim]
+  const float* norm_w;        // [vdim]
+  float* state;
+  float* scratch;             // b2_gated_linear_scratch_floats floats: prepared rows and raw outputs of the scan
+  void* out;                  // [rows, ld_out], heads * vdim columns
+  int64_t ld_out;
+  int32_t heads, dim, vdim;
+  float inv_tau, eps, out_scale;
+};
+int64_t b2_gated_linear_scratch_floats(int heads, int dim, int vdim, int rows);
+// Sequences as for the delta rule below: [0, n_decode) have one row each, [first, first + n_prefill) any number.
+int b2_gated_linear(const B2GatedLinearArgs* a, const B2SeqRows* s, int n_decode, int first, int n_prefill, int f32, b2::Status* status,
+                    cudaStream_t stream);
 
 // Gated delta rule with one decay per key channel. Per head, with S [dim, vdim]:
 //   S <- g * S (rows), u = beta (v - S^T k), S <- S + k u^T, o = S^T q
@@ -126,7 +175,8 @@ int b2_delta_rule(const B2DeltaArgs* a, const B2SeqRows* s, int n_decode, int fi
 
 // Y[M, N] = X[M, K] W[N, K]^T in true f32 (FMA, no reduced-precision matrix mode), `batch` such products side by side: product
 // b reads x columns b * K ..., weight rows b * N ... and writes y columns b * N .... Epilogue NONE, RELU2 or SOFTCAP
-// (B2Epilogue); then y is multiplied by sigmoid(gate) element by element where a gate [M, batch * N] is given.
+// (B2Epilogue); then y is multiplied by sigmoid(gate) element by element where a gate [M, batch * N] is given, or product by
+// product (`gate_heads`, gate [M, batch]).
 struct B2GemmF32Args {
   const float* x;
   const float* w;
@@ -134,7 +184,7 @@ struct B2GemmF32Args {
   const float* gate;
   int64_t ldx, ldw, ldy, ld_gate;
   float cap;
-  int32_t M, N, K, batch, epilogue;
+  int32_t M, N, K, batch, epilogue, gate_heads;
 };
 int b2_gemm_f32(const B2GemmF32Args* a, cudaStream_t stream);
 // Gated linear unit (B2EpiAct) of rows whose gate and up columns alternate in blocks of 16.
@@ -142,11 +192,12 @@ int b2_glu_f32(const float* gate_up, float* out, int64_t rows, int ffn, const st
 int b2_gather_rows_f32(const float* src, const int64_t* index, float* out, int rows_out, int cols, int64_t rows_src,
                        b2::Status* status, cudaStream_t stream);
 // Causal GQA attention over the paged cache in f32: any head sizes up to 1024, decode rows and prompt chunks alike. Row t
-// of sequence row_seq[t] sees positions 0 .. positions[t]. gate as in b2/api.h, f32.
+// of sequence row_seq[t] sees positions 0 .. positions[t]. Keys are `dim` columns apart, values (the first vdim of) ld_v, rows of
+// out ld_out. gate, window, cap and out_scale as in b2/api.h, the gate f32.
 int b2_attn_f32(const float* q, const float* k_cache, const float* v_cache, float* out, const int32_t* row_seq,
                 const int32_t* positions, const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv,
-                int dim, int vdim, int page_size, float scale, int64_t num_pages, const float* gate, int64_t gate_stride,
-                b2::Status* status, cudaStream_t stream);
+                int dim, int vdim, int64_t ld_v, int64_t ld_out, int page_size, float scale, int window, float cap, float out_scale,
+                int64_t num_pages, const float* gate, int64_t gate_stride, b2::Status* status, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -13,7 +13,7 @@ struct GroupedEpiParams {
   __nv_bfloat16* y;
   int64_t ldy;
   int n_rows;      // rows of one expert's weight
-  int mode;        // B2_EPI_NONE or B2_EPI_SWIGLU
+  int mode;        // B2_EPI_NONE, B2_EPI_RELU2 or B2_EPI_SWIGLU
   B2EpiAct act;
 };
 
@@ -47,7 +47,8 @@ struct GroupedEpilogue {
 #pragma unroll
         for (int j = 0; j < CH; ++j) {
           if (m0 + j >= u.nsplit) break;
-          base[static_cast<int64_t>(m0 + j) * p.ldy + n] = __float2bfloat16(__uint_as_float(r[j]));
+          const float v = __uint_as_float(r[j]);
+          base[static_cast<int64_t>(m0 + j) * p.ldy + n] = __float2bfloat16(p.mode == B2_EPI_RELU2 ? relu2(v) : v);
         }
       }
     }

@@ -14,6 +14,7 @@
 #include "b2/api.h"
 #include "b2/launch.h"
 #include "b2/ptx.cuh"
+#include "b2/score_mods.cuh"
 #include "b2/tma.h"
 #include "b2/vec.cuh"
 
@@ -107,11 +108,12 @@ __device__ __forceinline__ void load_kv_tile(const PagedKV& kv, int kv0, uint32_
 
 // One warp: S = Q K^T on a BN-token tile, online softmax, O += P V.
 //   qf      Q fragments of this warp's 16 rows (D/16 k-steps x 4 regs)
-//   max_lo  highest KV position visible to row g, max_hi to row g + 8 (causal + context limit)
-template <int D, int BN, int TROWS = 0>
+//   max_lo  highest KV position visible to row g, max_hi to row g + 8 (causal + context limit); MODS: also at least
+//           max_lo - window + 1, and the scores may be capped
+template <int D, int BN, int TROWS = 0, bool MODS = false>
 __device__ __forceinline__ void warp_attend(const uint32_t (&qf)[D / 16][4], uint32_t k_sm, uint32_t v_sm, int kv0,
                                             int max_lo, int max_hi, float scale_log2, float (&o)[D / 8][4],
-                                            float (&m)[2], float (&l)[2], int lane) {
+                                            float (&m)[2], float (&l)[2], int lane, const ScoreMods& mods) {
   constexpr int NT_S = BN / 8;
   float s[NT_S][4];
 #pragma unroll
@@ -134,10 +136,18 @@ __device__ __forceinline__ void warp_attend(const uint32_t (&qf)[D / 16][4], uin
 #pragma unroll
   for (int j = 0; j < NT_S; ++j) {
     const int col = kv0 + j * 8 + 2 * t;
-    s[j][0] = col <= max_lo ? s[j][0] * scale_log2 : -INFINITY;
-    s[j][1] = col + 1 <= max_lo ? s[j][1] * scale_log2 : -INFINITY;
-    s[j][2] = col <= max_hi ? s[j][2] * scale_log2 : -INFINITY;
-    s[j][3] = col + 1 <= max_hi ? s[j][3] * scale_log2 : -INFINITY;
+    if constexpr (MODS) {
+      const int lo = max_lo - mods.window, hi = max_hi - mods.window;
+      s[j][0] = col <= max_lo && col > lo ? mods.score(s[j][0], scale_log2) : -INFINITY;
+      s[j][1] = col + 1 <= max_lo && col + 1 > lo ? mods.score(s[j][1], scale_log2) : -INFINITY;
+      s[j][2] = col <= max_hi && col > hi ? mods.score(s[j][2], scale_log2) : -INFINITY;
+      s[j][3] = col + 1 <= max_hi && col + 1 > hi ? mods.score(s[j][3], scale_log2) : -INFINITY;
+    } else {
+      s[j][0] = col <= max_lo ? s[j][0] * scale_log2 : -INFINITY;
+      s[j][1] = col + 1 <= max_lo ? s[j][1] * scale_log2 : -INFINITY;
+      s[j][2] = col <= max_hi ? s[j][2] * scale_log2 : -INFINITY;
+      s[j][3] = col + 1 <= max_hi ? s[j][3] * scale_log2 : -INFINITY;
+    }
     mx_lo = fmaxf(mx_lo, fmaxf(s[j][0], s[j][1]));
     mx_hi = fmaxf(mx_hi, fmaxf(s[j][2], s[j][3]));
   }
@@ -214,12 +224,13 @@ __device__ __forceinline__ void load_q_frags(const __nv_bfloat16* q, int64_t q_s
 // Prefill: CTA = 4 warps x 16 packed rows = 64 rows; KV tiles of 64 tokens, double buffered, shared by
 // the four warps.
 // ------------------------------------------------------------------------------------------------
-template <int D>
+template <int D, bool MODS>
 __global__ void __launch_bounds__(128) attn_prefill_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, __nv_bfloat16* __restrict__ out, const int32_t* __restrict__ cu_q,
     const int32_t* __restrict__ ctx_lens, const int32_t* __restrict__ block_tables, int max_blocks, int n_q, int n_kv,
-    int page_size, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate, Status* status) {
+    int page_size, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate, ScoreMods mods,
+    Status* status) {
   ptx::grid_dep_sync();
   constexpr int BM = 64, BN = 64;
   constexpr int TILE_BYTES = BN * D * 2;
@@ -247,21 +258,23 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
   const int tok_lo = (row0 + g) / group, tok_hi = (row0 + g + 8) / group;
   const int max_lo = tok_lo < q_len ? past + tok_lo : -1;
   const int max_hi = tok_hi < q_len ? past + tok_hi : -1;
-  // the CTA needs KV positions [0, last visible position of its last row]
+  // the CTA needs KV positions from the first visible one of its first row to the last visible one of its last row
   const int last_tok = min(q_len - 1, (row_base + BM - 1) / group);
   const int kv_end = min(ctx, past + last_tok + 1);
   const int n_tiles = (kv_end + BN - 1) / BN;
+  const int first_tile = MODS ? max(0, past + row_base / group - mods.window + 1) / BN : 0;
 
   float o[D / 8][4];
 #pragma unroll
   for (int d = 0; d < D / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.0f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
 
-  if (n_tiles > 0) {
-    load_kv_tile<D, BN, 128>(kv, 0, kv_sm, kv_sm + TILE_BYTES, threadIdx.x, status);
+  if (first_tile < n_tiles) {
+    load_kv_tile<D, BN, 128>(kv, first_tile * BN, kv_sm + (first_tile & 1) * 2 * TILE_BYTES, kv_sm + ((first_tile & 1) * 2 + 1) * TILE_BYTES, threadIdx.x,
+                             status);
     cp_async_commit();
   }
-  for (int t = 0; t < n_tiles; ++t) {
+  for (int t = first_tile; t < n_tiles; ++t) {
     const int stage = t & 1;
     if (t + 1 < n_tiles) {
       const uint32_t nb = kv_sm + (stage ^ 1) * 2 * TILE_BYTES;
@@ -276,7 +289,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
     // a warp whose rows cannot see this tile yet skips the math (causal upper triangle)
     const int warp_max = min(q_len - 1, (row0 + 15) / group) + past;
     if (t * BN <= warp_max && row0 < q_len * group)
-      warp_attend<D, BN>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane);
+      warp_attend<D, BN, 0, MODS>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane, mods);
     __syncthreads();
   }
   // finalise: O / l
@@ -292,7 +305,8 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
     const int tok = pr / group, hg = pr % group;
     if (tok >= q_len) continue;
     __nv_bfloat16* dst = out + static_cast<int64_t>(tok0 + tok) * out_stride + static_cast<int64_t>(kvh * group + hg) * D;
-    const float inv = (half ? inv_hi : inv_lo) * gate.factor(tok0 + tok, kvh * group + hg);
+    float inv = (half ? inv_hi : inv_lo) * gate.factor(tok0 + tok, kvh * group + hg);
+    if constexpr (MODS) inv *= mods.out_scale;
 #pragma unroll
     for (int d = 0; d < D / 8; ++d) {
       const uint32_t pk = ptx::pack_bf16x2(o[d][half * 2] * inv, o[d][half * 2 + 1] * inv);
@@ -305,13 +319,13 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
 // Decode: CTA = (split, kv head, sequence); 4 warps stream disjoint 32-token tiles of the split's KV
 // range through warp-private double buffers; rows = the `group` query heads (<= 16).
 // ------------------------------------------------------------------------------------------------
-template <int D>
+template <int D, bool MODS>
 __global__ void __launch_bounds__(128) attn_decode_kernel(
     const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_cache,
     const __nv_bfloat16* __restrict__ v_cache, __nv_bfloat16* __restrict__ out, const int32_t* __restrict__ ctx_lens,
     const int32_t* __restrict__ block_tables, float* __restrict__ workspace, int max_blocks, int n_q, int n_kv,
     int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-    HeadGate gate, Status* status) {
+    HeadGate gate, ScoreMods mods, Status* status) {
   ptx::grid_dep_sync();
   constexpr int BN = 32;
   constexpr int TILE_BYTES = BN * D * 2;
@@ -327,9 +341,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
   const uint32_t kv_sm = q_sm + 16 * D * 2;
 
   // KV range of this split, in whole tiles
-  const int tiles_total = (ctx + BN - 1) / BN;
-  const int tiles_per_split = (tiles_total + num_splits - 1) / num_splits;
-  const int tile_begin = split * tiles_per_split;
+  const int tiles_total = (ctx + BN - 1) / BN, first_tile = MODS ? max(0, ctx - mods.window) / BN : 0;
+  const int tiles_per_split = (tiles_total - first_tile + num_splits - 1) / num_splits;
+  const int tile_begin = first_tile + split * tiles_per_split;
   const int tile_end = min(tiles_total, tile_begin + tiles_per_split);
 
   PagedKV kv{k_cache, v_cache, block_tables + static_cast<int64_t>(seq) * max_blocks, n_kv, kvh, page_size, ctx, num_pages};
@@ -361,7 +375,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     }
     __syncwarp();
     const uint32_t kb = kv_sm + stage * 2 * TILE_BYTES;
-    warp_attend<D, BN>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane);
+    warp_attend<D, BN, 0, MODS>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane, mods);
     __syncwarp();
     stage ^= 1;
   }
@@ -410,7 +424,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     }
     const int head = kvh * group + row;
     if (num_splits == 1) {
-      const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head);
+      const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head) * (MODS ? mods.out_scale : 1.0f);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D + cs;
 #pragma unroll
       for (int c = 0; c < COLS_PER_THREAD; c += 2)
@@ -433,13 +447,13 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
 // 16 KB tile is four instructions instead of a page-table walk per 16-byte chunk, and several small CTAs per
 // SM keep ~200 KB of loads in flight. The cache is addressed as a 2-D matrix [(page, kv head, token), D].
 // ------------------------------------------------------------------------------------------------
-template <int D, int STAGES>
+template <int D, int STAGES, bool MODS>
 __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
     const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v,
     const __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ out, const int32_t* __restrict__ ctx_lens,
     const int32_t* __restrict__ block_tables, float* __restrict__ workspace, int max_blocks, int n_q, int n_kv,
     int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-    uint32_t* __restrict__ split_counters, HeadGate gate, Status* status) {
+    uint32_t* __restrict__ split_counters, HeadGate gate, ScoreMods mods, Status* status) {
   ptx::grid_dep_sync();
   constexpr int BN = 32;
   constexpr int HALVES = D / 64;
@@ -456,9 +470,9 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
   const int ctx = ctx_lens[seq];
   const int32_t* table = block_tables + static_cast<int64_t>(seq) * max_blocks;
 
-  const int tiles_total = (ctx + BN - 1) / BN;
-  const int tiles_per_split = (tiles_total + num_splits - 1) / num_splits;
-  const int tile_begin = split * tiles_per_split;
+  const int tiles_total = (ctx + BN - 1) / BN, first_tile = MODS ? max(0, ctx - mods.window) / BN : 0;
+  const int tiles_per_split = (tiles_total - first_tile + num_splits - 1) / num_splits;
+  const int tile_begin = first_tile + split * tiles_per_split;
   const int tile_end = min(tiles_total, tile_begin + tiles_per_split);
   const int n_tiles = max(0, tile_end - tile_begin);
 
@@ -523,7 +537,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
         }
       __syncwarp();
     }
-    warp_attend<D, BN, BN>(qf, kb, kb + TILE_BYTES, kv0, max_lo, max_hi, scale_log2, o, m, l, lane);
+    warp_attend<D, BN, BN, MODS>(qf, kb, kb + TILE_BYTES, kv0, max_lo, max_hi, scale_log2, o, m, l, lane, mods);
     __syncwarp();
   }
   if (!ok) {
@@ -542,7 +556,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
     if (row >= group) continue;
     const int head = kvh * group + row;
     if (num_splits == 1) {
-      const float inv = (l[half] > 0.0f ? 1.0f / l[half] : 0.0f) * gate.factor(seq, head);
+      const float inv = (l[half] > 0.0f ? 1.0f / l[half] : 0.0f) * gate.factor(seq, head) * (MODS ? mods.out_scale : 1.0f);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
       for (int d = 0; d < D / 8; ++d)
@@ -586,7 +600,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
 #pragma unroll
         for (int c = 0; c < D / 32; ++c) acc[c] += __ldcg(base + sp * RS + c * 32 + lane) * f;
       }
-      const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head);
+      const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head) * (MODS ? mods.out_scale : 1.0f);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
       for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv);
@@ -597,7 +611,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
 // Merge split partials: one warp per (sequence, head).
 template <int D>
 __global__ void attn_decode_reduce_kernel(const float* __restrict__ workspace, __nv_bfloat16* __restrict__ out,
-                                          int n_q, int num_splits, int64_t out_stride, int total, HeadGate gate) {
+                                          int n_q, int num_splits, int64_t out_stride, int total, HeadGate gate, float out_scale) {
   ptx::grid_dep_sync();
   constexpr int RS = D + 2;
   const int idx = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -618,7 +632,7 @@ __global__ void attn_decode_reduce_kernel(const float* __restrict__ workspace, _
 #pragma unroll
     for (int c = 0; c < D / 32; ++c) acc[c] += base[s * RS + c * 32 + lane] * f;
   }
-  const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head);
+  const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head) * out_scale;
   __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
   for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv);
@@ -627,12 +641,13 @@ __global__ void attn_decode_reduce_kernel(const float* __restrict__ workspace, _
 template <int D>
 int launch_prefill(dim3 grid, cudaStream_t stream, const __nv_bfloat16* q, const __nv_bfloat16* k, const __nv_bfloat16* v, __nv_bfloat16* out,
                    const int32_t* cu_q, const int32_t* ctx_lens, const int32_t* block_tables, int max_blocks, int n_q, int n_kv, int page_size,
-                   float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate, Status* status) {
+                   float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate, const ScoreMods& mods, Status* status) {
   constexpr int SMEM = 4 * 16 * D * 2 + 4 * 64 * D * 2;
-  static DeviceOnce attr_once;
-  if (const int rc = attr_once.max_smem(attn_prefill_kernel<D>, SMEM)) return rc;
-  launch_pdl(attn_prefill_kernel<D>, grid, dim3(128), SMEM, stream, q, k, v, out, cu_q, ctx_lens, block_tables, max_blocks, n_q, n_kv, page_size,
-             scale_log2, q_stride, out_stride, num_pages, gate, status);
+  static DeviceOnce attr_once[2];
+  auto kern = mods.plain() ? attn_prefill_kernel<D, false> : attn_prefill_kernel<D, true>;
+  if (const int rc = attr_once[mods.plain()].max_smem(kern, SMEM)) return rc;
+  launch_pdl(kern, grid, dim3(128), SMEM, stream, q, k, v, out, cu_q, ctx_lens, block_tables, max_blocks, n_q, n_kv, page_size,
+             scale_log2, q_stride, out_stride, num_pages, gate, mods, status);
   return last_launch_rc();
 }
 
@@ -640,7 +655,7 @@ template <int D>
 int launch_decode_tma(dim3 grid, cudaStream_t stream, const void* k, const void* v, const __nv_bfloat16* q, __nv_bfloat16* out,
                       const int32_t* ctx_lens, const int32_t* block_tables, float* workspace, int batch, int max_blocks, int n_q, int n_kv,
                       int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-                      uint32_t* counters, HeadGate gate, Status* status) {
+                      uint32_t* counters, HeadGate gate, const ScoreMods& mods, Status* status) {
   // cache as a 2-D matrix [(page, kv head, token), D], boxes of 32 tokens x 64 columns
   CUtensorMap tk, tv;
   const uint64_t rows = static_cast<uint64_t>(num_pages) * n_kv * page_size;
@@ -649,13 +664,14 @@ int launch_decode_tma(dim3 grid, cudaStream_t stream, const void* k, const void*
     return -kBadArgument;
   constexpr int STAGES = 3;
   constexpr int SMEM = STAGES * 2 * 32 * D * 2 + 16 * D * 2 + 64 + 1024;
-  static DeviceOnce attr_once;
-  if (const int rc = attr_once.max_smem(attn_decode_tma_kernel<D, STAGES>, SMEM)) return rc;
-  launch_pdl(attn_decode_tma_kernel<D, STAGES>, grid, dim3(32), SMEM, stream, tk, tv, q, out, ctx_lens, block_tables, workspace, max_blocks, n_q,
-             n_kv, page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, counters, gate, status);
+  static DeviceOnce attr_once[2];
+  auto kern = mods.plain() ? attn_decode_tma_kernel<D, STAGES, false> : attn_decode_tma_kernel<D, STAGES, true>;
+  if (const int rc = attr_once[mods.plain()].max_smem(kern, SMEM)) return rc;
+  launch_pdl(kern, grid, dim3(32), SMEM, stream, tk, tv, q, out, ctx_lens, block_tables, workspace, max_blocks, n_q,
+             n_kv, page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, counters, gate, mods, status);
   if (num_splits > 1 && counters == nullptr)
     launch_pdl(attn_decode_reduce_kernel<D>, dim3((batch * n_q + 3) / 4), dim3(128), 0, stream, workspace, out, n_q, num_splits, out_stride,
-               batch * n_q, gate);
+               batch * n_q, gate, mods.out_scale);
   return last_launch_rc();
 }
 
@@ -663,15 +679,16 @@ template <int D>
 int launch_decode(dim3 grid, cudaStream_t stream, const __nv_bfloat16* k, const __nv_bfloat16* v, const __nv_bfloat16* q, __nv_bfloat16* out,
                   const int32_t* ctx_lens, const int32_t* block_tables, float* workspace, int batch, int max_blocks, int n_q, int n_kv,
                   int page_size, int num_splits, float scale_log2, int64_t q_stride, int64_t out_stride, int64_t num_pages, HeadGate gate,
-                  Status* status) {
+                  const ScoreMods& mods, Status* status) {
   constexpr int SMEM = 4 * (16 * D * 2 + 4 * 32 * D * 2);
-  static DeviceOnce attr_once;
-  if (const int rc = attr_once.max_smem(attn_decode_kernel<D>, SMEM)) return rc;
-  launch_pdl(attn_decode_kernel<D>, grid, dim3(128), SMEM, stream, q, k, v, out, ctx_lens, block_tables, workspace, max_blocks, n_q, n_kv,
-             page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, gate, status);
+  static DeviceOnce attr_once[2];
+  auto kern = mods.plain() ? attn_decode_kernel<D, false> : attn_decode_kernel<D, true>;
+  if (const int rc = attr_once[mods.plain()].max_smem(kern, SMEM)) return rc;
+  launch_pdl(kern, grid, dim3(128), SMEM, stream, q, k, v, out, ctx_lens, block_tables, workspace, max_blocks, n_q, n_kv,
+             page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, gate, mods, status);
   if (num_splits > 1)
     launch_pdl(attn_decode_reduce_kernel<D>, dim3((batch * n_q + 3) / 4), dim3(128), 0, stream, workspace, out, n_q, num_splits, out_stride,
-               batch * n_q, gate);
+               batch * n_q, gate, mods.out_scale);
   return last_launch_rc();
 }
 
@@ -684,18 +701,19 @@ extern "C" int b2_attn_prefill_bf16(const void* q, const void* k_cache, const vo
                                     const int32_t* cu_q, const int32_t* ctx_lens, const int32_t* block_tables,
                                     int batch, int max_blocks, int n_q, int n_kv, int head_dim, int page_size,
                                     int max_q_len, float scale, int64_t q_stride, int64_t out_stride,
-                                    int64_t num_pages, const void* gate, int64_t gate_stride, Status* status,
-                                    cudaStream_t stream) {
+                                    int64_t num_pages, const void* gate, int64_t gate_stride, int window, float softcap,
+                                    float out_scale, Status* status, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
   if (n_kv <= 0 || n_q % n_kv != 0 || q_stride % 8 != 0 || out_stride % 2 != 0) return -kBadArgument;
   const int group = n_q / n_kv;
   const dim3 grid((max_q_len * group + 63) / 64, n_kv, batch);
   const float scale_log2 = scale * ptx::kLog2e;
   const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride};
+  const ScoreMods mods = make_score_mods(window, softcap, out_scale, scale);
 #define B2_PREFILL(D_)                                                                                                          \
   return launch_prefill<D_>(grid, stream, static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),    \
                             static_cast<const __nv_bfloat16*>(v_cache), static_cast<__nv_bfloat16*>(out), cu_q, ctx_lens,      \
-                            block_tables, max_blocks, n_q, n_kv, page_size, scale_log2, q_stride, out_stride, num_pages, hg, status)
+                            block_tables, max_blocks, n_q, n_kv, page_size, scale_log2, q_stride, out_stride, num_pages, hg, mods, status)
   switch (head_dim) {
     case 64: B2_PREFILL(64);
     case 128: B2_PREFILL(128);
@@ -717,23 +735,24 @@ extern "C" int b2_attn_decode_bf16(const void* q, const void* k_cache, const voi
                                    const int32_t* ctx_lens, const int32_t* block_tables, float* workspace, int batch,
                                    int max_blocks, int n_q, int n_kv, int head_dim, int page_size, int num_splits,
                                    float scale, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-                                   uint32_t* counters, const void* gate, int64_t gate_stride, Status* status,
-                                   cudaStream_t stream) {
+                                   uint32_t* counters, const void* gate, int64_t gate_stride, int window, float softcap,
+                                   float out_scale, Status* status, cudaStream_t stream) {
   if (batch <= 0) return 0;
   if (n_kv <= 0 || n_q % n_kv != 0 || n_q / n_kv > 16 || q_stride % 8 != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr))
     return -kBadArgument;
   const dim3 grid(num_splits, n_kv, batch);
   const float scale_log2 = scale * ptx::kLog2e;
   const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride};
+  const ScoreMods mods = make_score_mods(window, softcap, out_scale, scale);
   auto qp = static_cast<const __nv_bfloat16*>(q);
   auto op = static_cast<__nv_bfloat16*>(out);
 #define B2_DECODE_TMA(D_)                                                                                                             \
   return launch_decode_tma<D_>(grid, stream, k_cache, v_cache, qp, op, ctx_lens, block_tables, workspace, batch, max_blocks, n_q, n_kv, \
-                               page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, counters, hg, status)
+                               page_size, num_splits, scale_log2, q_stride, out_stride, num_pages, counters, hg, mods, status)
 #define B2_DECODE(D_)                                                                                                                   \
   return launch_decode<D_>(grid, stream, static_cast<const __nv_bfloat16*>(k_cache), static_cast<const __nv_bfloat16*>(v_cache), qp, op, \
                            ctx_lens, block_tables, workspace, batch, max_blocks, n_q, n_kv, page_size, num_splits, scale_log2, q_stride, \
-                           out_stride, num_pages, hg, status)
+                           out_stride, num_pages, hg, mods, status)
   if (page_size % 32 == 0) {
     switch (head_dim) {
       case 64: B2_DECODE_TMA(64);

@@ -28,6 +28,7 @@
 #include "b2/config.h"
 #include "b2/gemm_tc.cuh"
 #include "b2/ptx.cuh"
+#include "b2/score_mods.cuh"
 #include "b2/status.h"
 #include "b2/tma.h"
 #include "b2/vec.cuh"
@@ -77,6 +78,7 @@ struct AttnTcParams {
   // Where the tile of (page, KV head) lies in the K and V matrices: row page * page_rows + head * head_rows, column
   // head * head_cols. Paged cache: {n_kv * 128, 128, 0}; rows of one token with its heads side by side: {128, 0, 128}.
   int page_rows, head_rows, head_cols;
+  ScoreMods mods;
 };
 
 // Shared-memory descriptor with explicit leading / stride byte offsets, 128-byte swizzle.
@@ -90,6 +92,9 @@ __device__ __forceinline__ uint64_t smem_desc(uint32_t addr, uint32_t lbo_bytes,
   return d;
 }
 
+// MODS: a window, a soft cap or a factor on the result (AttnTcParams::mods). Tiles before the window of the first row are
+// never visited.
+template <bool MODS>
 __global__ void __launch_bounds__(kThreadsAttn, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                        const __grid_constant__ CUtensorMap tmap_v, AttnTcParams prm, Status* status) {
@@ -106,7 +111,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
   const int ctx = prm.ctx_lens[seq];
   const int pos0 = ctx - q_len + qt * kTile;              // absolute position of this tile's first query row
   const int rows = min(kTile, q_len - qt * kTile);
-  const int n_tiles = min((pos0 + rows + kTile - 1) / kTile, (ctx + kTile - 1) / kTile);  // KV tiles with a visible token
+  const int first_tile = MODS ? max(0, pos0 - prm.mods.window + 1) / kTile : 0;
+  const int n_tiles = min((pos0 + rows + kTile - 1) / kTile, (ctx + kTile - 1) / kTile) - first_tile;  // KV tiles with a visible token
   const int kvh = head / (prm.n_q / prm.n_kv);
 
   extern __shared__ uint8_t smem_raw[];
@@ -177,7 +183,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int s = j % kStages;
         const uint32_t ph = static_cast<uint32_t>((j / kStages) & 1);
-        int page = prm.block_tables[static_cast<int64_t>(seq) * prm.max_blocks + j];
+        int page = prm.block_tables[static_cast<int64_t>(seq) * prm.max_blocks + first_tile + j];
         if (page < 0 || page >= prm.num_pages) {
           status_record(status, kOutOfBounds, kSiteKvIndex, seq, page);
           page = 0;
@@ -265,6 +271,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     const int qpos = pos0 + r;
     const uint32_t lane_bits = static_cast<uint32_t>(quarter * 32) << 16;
     float* pmax = alpha_ring;               // [2 tiles in flight][2 halves][128 rows]
+    const float scale_log2 = MODS ? 1.0f : prm.scale_log2;      // MODS: the scores come scaled
     float m_run = -INFINITY, l_part = 0.0f, alpha_prev = 1.0f;
     float o[64];
 #pragma unroll
@@ -318,7 +325,17 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
 #pragma unroll
         for (int c = 0; c < 64; ++c) s[c] = 0.0f;
       }
-      const int kv0 = j * kTile + g * 64;
+      const int kv0 = (first_tile + j) * kTile + g * 64;
+      if constexpr (MODS) {
+#pragma unroll
+        for (int c = 0; c < 64; ++c) s[c] = prm.mods.score(s[c], prm.scale_log2);
+        if (kv0 <= pos0 + kTile - 1 - prm.mods.window) {   // some row of this tile is past some of these columns
+          const int lo = qpos - prm.mods.window;
+#pragma unroll
+          for (int c = 0; c < 64; ++c)
+            if (kv0 + c <= lo) s[c] = -INFINITY;
+        }
+      }
       if (kv0 + 63 > pos0) {                             // some row of this tile masks some of these columns
 #pragma unroll
         for (int c = 0; c < 64; ++c)
@@ -335,8 +352,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       ptx::named_barrier_sync(5, 256);
       const float m_new = fmaxf(m_run, fmaxf(mloc, pmax[(a * 2 + (g ^ 1)) * kTile + r]));
       const float m_use = m_new == -INFINITY ? 0.0f : m_new;   // a row with nothing visible yet
-      const float alpha = ptx::ex2((m_run - m_use) * prm.scale_log2);
-      const float neg_m = -m_use * prm.scale_log2;
+      const float alpha = ptx::ex2((m_run - m_use) * scale_log2);
+      const float neg_m = -m_use * scale_log2;
       m_run = m_new;
       if (j > 0) ok = wait_all(p_empty, (j - 1) & 1, 10, j);
       if (ok) {
@@ -346,7 +363,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
           float p[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
-            p[i] = ptx::ex2(fmaf(s[ch * 8 + i], prm.scale_log2, neg_m));
+            p[i] = ptx::ex2(fmaf(s[ch * 8 + i], scale_log2, neg_m));
             sum[i & 3] += p[i];
           }
           uint4 pk;
@@ -371,6 +388,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     if (ok && *fail == 0 && r < rows) {
       const float l = l_final[r] + l_final[kTile + r];
       float inv = l > 0.0f ? 1.0f / l : 0.0f;
+      if constexpr (MODS) inv *= prm.mods.out_scale;
       if (prm.gate != nullptr && prm.gate_elems) {
         const __nv_bfloat16* z = prm.gate + static_cast<int64_t>(q_begin + qt * kTile + r) * prm.gate_stride + head * kD + g * 64;
 #pragma unroll
@@ -418,7 +436,8 @@ extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const
                                        const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                                        int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
                                        int64_t num_pages, int64_t token_stride, const int32_t* work, const int32_t* n_work, int work_items,
-                                       const void* gate, int64_t gate_stride, int gate_elems, Status* status, cudaStream_t stream) {
+                                       const void* gate, int64_t gate_stride, int gate_elems, int window, float softcap, float out_scale,
+                                       Status* status, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
   if (work != nullptr && work_items <= 0) return 0;
   if (n_q <= 0 || n_kv <= 0 || n_q % n_kv != 0 || q_stride % 8 != 0 || out_stride % 8 != 0 ||
@@ -455,14 +474,12 @@ extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const
   prm.page_rows = by_token ? kTile : n_kv * kTile;
   prm.head_rows = by_token ? 0 : kTile;
   prm.head_cols = by_token ? kD : 0;
-  static DeviceOnce attr_once;
-  if (const int rc = attr_once.run([&] {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemAttn);
-        return e;
-      }))
-    return rc;
+  prm.mods = make_score_mods(window, softcap, out_scale, scale);
+  static DeviceOnce attr_once[2];
+  auto kern = prm.mods.plain() ? attn_prefill_tc_kernel<false> : attn_prefill_tc_kernel<true>;
+  if (const int rc = attr_once[prm.mods.plain()].max_smem(kern, kSmemAttn)) return rc;
   dim3 grid((max_q_len + kTile - 1) / kTile, n_q, batch);
   if (work != nullptr) grid = dim3(work_items, n_q, 1);
-  launch_pdl(attn_prefill_tc_kernel, dim3(grid), dim3(kThreadsAttn), kSmemAttn, stream, tq, tk, tv, prm, status);
+  launch_pdl(kern, dim3(grid), dim3(kThreadsAttn), kSmemAttn, stream, tq, tk, tv, prm, status);
   return last_launch_rc();
 }

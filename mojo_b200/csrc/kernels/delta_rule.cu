@@ -16,6 +16,7 @@
 #include "b2/launch.h"
 #include "b2/mixers.h"
 #include "b2/ptx.cuh"
+#include "b2/recurrence.cuh"
 #include "b2/short_conv.cuh"
 #include "b2/vec.cuh"
 
@@ -292,13 +293,6 @@ __device__ __forceinline__ void decode_finish(const B2DeltaArgs& a, int row, int
   store_f32<VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(row) * a.ld_out + static_cast<int64_t>(h) * a.vdim + cg * VEC, o);
 }
 
-// Sequence's decode row if the entry is in use and sound, else -1.
-__device__ __forceinline__ int decode_row(const B2SeqRows& sq, int seq, ConvRow& cr, Status* status) {
-  const int row = sq.seq_rows[2 * seq];
-  if (row < 0 || row >= sq.rows || !cr.load(sq, seq, row, sq.banks, status)) return -1;
-  return B2_ASSERT(status, cr.end == row + 1, kSiteKvIndex, row, cr.end) ? row : -1;
-}
-
 // Plain form for sizes the pipelined one does not take: one CTA per (head, sequence), S read twice.
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256) delta_decode_plain_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared in, int n_cg, int n_rg,
@@ -535,35 +529,6 @@ int dispatch_decode(const B2DeltaArgs& a, const B2SeqRows& s, int n, Status* sta
 // ------------------------------------------------------------------------------------------------------------
 // scan
 // ------------------------------------------------------------------------------------------------------------
-// Packed pairs of f32 (two key rows): one instruction per two multiply-adds.
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ float2 unpack2(uint64_t v) {
-  float2 f;
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(f.x), "=f"(f.y) : "l"(v));
-  return f;
-}
-__device__ __forceinline__ float half_sum(uint64_t v) {
-  const float2 f = unpack2(v);
-  return f.x + f.y;
-}
-
-// A lane holds four value columns and P pairs of key rows (kd = 32 P). The 16 row groups of a half-warp read 256 different
-// bytes of a vector at once; a mapping with more rows and fewer columns per lane reads the same bytes more often, and
-// shared-memory bandwidth is what two CTAs on one SM run short of first.
 template <int P>
 struct ScanLayout {
   static constexpr int kD = 32 * P;
@@ -572,26 +537,6 @@ struct ScanLayout {
   static constexpr int kStage = kOffSc + kTile * kSc;
   static constexpr int kBytes = kStages * kStage * 4 + kStages * 8;
 };
-// Pair p of row group rg is key rows pair_row(p, rg) and the next one.
-template <int P>
-__device__ __forceinline__ int pair_row(int p, int rg) {
-  if constexpr (P == 1) return 2 * rg;
-  else return (p >> 1) * 64 + rg * 4 + (p & 1) * 2;
-}
-template <int P>
-__device__ __forceinline__ void load_pairs(const float* x, int rg, uint64_t (&v)[P]) {
-  if constexpr (P == 1) {
-    v[0] = *reinterpret_cast<const uint64_t*>(x + 2 * rg);
-  } else {
-#pragma unroll
-    for (int i = 0; i < P / 2; ++i) {
-      const ulonglong2 t = *reinterpret_cast<const ulonglong2*>(x + i * 64 + rg * 4);
-      v[2 * i] = t.x;
-      v[2 * i + 1] = t.y;
-    }
-  }
-}
-
 // Lane (rg = lane & 15, half = lane >> 4) of warp w: value columns col0 + 8 w + 4 half + 0..3.
 template <int P>
 __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, const B2SeqRows sq, const Prepared in, int first, Status* status) {
@@ -630,19 +575,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
   const int mine = lane & 3;
   float* state = a.state + (static_cast<int64_t>(cr.wr >> 1) * a.heads + h) * d * e + col;
   uint64_t S[P][4];
-#pragma unroll
-  for (int p = 0; p < P; ++p) {
-    const int key = pair_row<P>(p, rg);
-#pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      float lo = 0.0f, hi = 0.0f;
-      if (cr.rd >= 0 && col + c < e) {
-        if (key < d) lo = state[static_cast<int64_t>(key) * e + c];
-        if (key + 1 < d) hi = state[static_cast<int64_t>(key + 1) * e + c];
-      }
-      S[p][c] = pack2(lo, hi);
-    }
-  }
+  load_state<P>(state, cr.rd < 0, d, e, col, rg, S);
   const int64_t o_ld = static_cast<int64_t>(a.heads) * e;
   float* o_dst = a.o_raw + static_cast<int64_t>(begin + (second ? 1 : 0)) * o_ld + static_cast<int64_t>(h) * e + col + mine;
   const bool writes = is_q && col + mine < e;
@@ -728,17 +661,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
     for (int s = 0; s < kStages; ++s) ptx::mbar_wait(bars + 8 * s, 0, 20000000ull) || ptx::mbar_wait(bars + 8 * s, 1, 20000000ull);
     return;
   }
-#pragma unroll
-  for (int p = 0; p < P; ++p) {
-    const int key = pair_row<P>(p, rg);
-#pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      if (col + c >= e) continue;
-      const float2 f = unpack2(S[p][c]);
-      if (key < d) state[static_cast<int64_t>(key) * e + c] = f.x;
-      if (key + 1 < d) state[static_cast<int64_t>(key + 1) * e + c] = f.y;
-    }
-  }
+  store_state<P>(state, d, e, col, rg, S);
 }
 
 // out = rms_norm(o) * w * sigmoid(gate) for the rows of sequences >= first: one warp per (row, head).

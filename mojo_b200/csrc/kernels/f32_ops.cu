@@ -53,7 +53,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const B2GemmF32Args a) {
         float v = acc[i][j];
         if (a.epilogue == B2_EPI_RELU2) v = relu2(v);
         if (a.epilogue == B2_EPI_SOFTCAP) v = softcap(v, a.cap);
-        if (a.gate != nullptr) v *= sigmoid_f32(a.gate[m * a.ld_gate + n]);
+        if (a.gate != nullptr) v *= sigmoid_f32(a.gate[m * a.ld_gate + (a.gate_heads ? static_cast<int64_t>(blockIdx.z) : n)]);
         a.y[m * a.ldy + n] = v;
       }
 }
@@ -82,15 +82,16 @@ template <int kAttnMax>
 __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__ q, const float* __restrict__ kc, const float* __restrict__ vc,
                                                        float* __restrict__ out, const int32_t* __restrict__ row_seq,
                                                        const int32_t* __restrict__ positions, const int32_t* __restrict__ tables, int rows, int seqs,
-                                                       int max_blocks, int n_q, int n_kv, int dim, int vdim, int page_size, float scale,
-                                                       int64_t num_pages, const float* __restrict__ gate, int64_t gate_stride, Status* status) {
+                                                       int max_blocks, int n_q, int n_kv, int dim, int vdim, int64_t ld_v, int64_t ld_out, int page_size,
+                                                       float scale, int window, float cap, float out_scale, int64_t num_pages,
+                                                       const float* __restrict__ gate, int64_t gate_stride, Status* status) {
   ptx::grid_dep_sync();
   __shared__ float q_sm[4][kAttnMax];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int64_t idx = static_cast<int64_t>(blockIdx.x) * 4 + warp;
   if (idx >= static_cast<int64_t>(rows) * n_q) return;
   const int row = static_cast<int>(idx / n_q), head = static_cast<int>(idx % n_q), kvh = head / (n_q / n_kv);
-  float* dst = out + (static_cast<int64_t>(row) * n_q + head) * vdim;
+  float* dst = out + row * ld_out + static_cast<int64_t>(head) * vdim;
   const int seq = row_seq[row];
   const int ctx = seq >= 0 ? positions[row] + 1 : 0;
   if (seq < 0 || !B2_ASSERT(status, seq < seqs && ctx >= 1 && (ctx - 1) / page_size < max_blocks, kSiteKvIndex, seq, ctx)) {
@@ -108,7 +109,7 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
   float m = -INFINITY, l = 0.0f, o[kAttnMax / 32];
 #pragma unroll
   for (int j = 0; j < kAttnMax / 32; ++j) o[j] = 0.0f;
-  for (int p0 = 0; p0 < ctx; p0 += 32) {
+  for (int p0 = max(0, ctx - window); p0 < ctx; p0 += 32) {
     const int pos = p0 + lane;
     int64_t slot = 0;
     float s = -INFINITY;
@@ -118,6 +119,7 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
       float dot = 0.0f;
       for (int i = 0; i < dim; ++i) dot = fmaf(q_sm[warp][i], k[i], dot);
       s = dot * scale;
+      if (cap > 0.0f) s = softcap(s, cap);
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new), p = pos < ctx ? expf(s - m_new) : 0.0f;
@@ -128,13 +130,13 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
     const int n = min(32, ctx - p0);
     for (int t = 0; t < n; ++t) {
       const float pt = __shfl_sync(0xffffffffu, p, t);
-      const float* v = vc + __shfl_sync(0xffffffffu, slot, t) * vdim;
+      const float* v = vc + __shfl_sync(0xffffffffu, slot, t) * ld_v;
 #pragma unroll
       for (int j = 0; j < kAttnMax / 32; ++j)
         if (lane + 32 * j < vdim) o[j] = fmaf(pt, v[lane + 32 * j], o[j]);
     }
   }
-  float f = 1.0f / warp_sum(l);
+  float f = out_scale / warp_sum(l);
   if (gate != nullptr) f *= sigmoid_f32(gate[row * gate_stride + head]);
 #pragma unroll
   for (int j = 0; j < kAttnMax / 32; ++j)
@@ -171,13 +173,17 @@ extern "C" int b2_gather_rows_f32(const float* src, const int64_t* index, float*
 }
 
 extern "C" int b2_attn_f32(const float* q, const float* k_cache, const float* v_cache, float* out, const int32_t* row_seq, const int32_t* positions,
-                           const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv, int dim, int vdim, int page_size,
-                           float scale, int64_t num_pages, const float* gate, int64_t gate_stride, Status* status, cudaStream_t stream) {
+                           const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv, int dim, int vdim, int64_t ld_v, int64_t ld_out,
+                           int page_size, float scale, int window, float cap, float out_scale, int64_t num_pages, const float* gate, int64_t gate_stride,
+                           Status* status, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (n_kv <= 0 || n_q % n_kv != 0 || dim <= 0 || dim > 1024 || vdim <= 0 || vdim > 1024 || page_size <= 0) return -kBadArgument;
-  auto kern = dim <= 256 && vdim <= 256 ? attn_f32_kernel<256> : attn_f32_kernel<1024>;
+  if (n_kv <= 0 || n_q % n_kv != 0 || dim <= 0 || dim > 1152 || vdim <= 0 || vdim > 1152 || ld_v < vdim || ld_out < static_cast<int64_t>(n_q) * vdim ||
+      page_size <= 0)
+    return -kBadArgument;
+  auto kern = dim <= 256 && vdim <= 256 ? attn_f32_kernel<256> : attn_f32_kernel<1152>;
   const int64_t warps = static_cast<int64_t>(rows) * n_q;
   launch_pdl(kern, dim3(static_cast<unsigned>((warps + 3) / 4)), dim3(128), 0, stream, q, k_cache, v_cache, out, row_seq, positions,
-             block_tables, rows, seqs, max_blocks, n_q, n_kv, dim, vdim, page_size, scale, num_pages, gate, gate_stride, status);
+             block_tables, rows, seqs, max_blocks, n_q, n_kv, dim, vdim, ld_v, ld_out, page_size, scale, window > 0 ? window : 1 << 30, cap, out_scale,
+             num_pages, gate, gate_stride, status);
   return last_launch_rc();
 }

@@ -1,6 +1,6 @@
 // One small matrix per head: y[t, h, :] = W_h x[t, h, :] for the heads of a row laid side by side, on the tcgen05 core.
 // The token rows are the P operand, read at the head's columns; a head's weight rows are the Q operand. Optional output
-// gate: every element is multiplied by the sigmoid of its own logit before it is rounded.
+// gate: every element is multiplied by the sigmoid of its own logit, or of its head's, before it is rounded.
 #include <cstdint>
 #include <cuda.h>
 #include <cuda_bf16.h>
@@ -40,10 +40,13 @@ struct HeadEpilogue {
   __nv_bfloat16* y;
   const __nv_bfloat16* gate;
   int64_t ldy, ld_gate;
-  int rows, n;
+  int rows, n, gate_heads;
   __device__ __forceinline__ void operator()(const gemm::WorkUnit& u, uint32_t taddr, int quarter, int lane, uint32_t*, Status*) const {
     const int row = u.pb * gemm::kBlockP + quarter * 32 + lane;
     const int64_t col0 = static_cast<int64_t>(u.split) * n + u.qb * BN;
+    const bool by_head = gate != nullptr && gate_heads;
+    float f_head = 1.0f;
+    if (by_head && row < rows) f_head = ptx::rcp(1.0f + ptx::ex2(-__bfloat162float(gate[row * ld_gate + u.split]) * ptx::kLog2e));
 #pragma unroll 1
     for (int c = 0; c < BN / 32; ++c) {
       uint32_t r[32];
@@ -51,12 +54,12 @@ struct HeadEpilogue {
       ptx::tc_wait_ld();
       if (row >= rows) continue;
       __nv_bfloat16* dst = y + row * ldy + col0 + c * 32;
-      const __nv_bfloat16* z = gate != nullptr ? gate + row * ld_gate + col0 + c * 32 : nullptr;
+      const __nv_bfloat16* z = gate != nullptr && !by_head ? gate + row * ld_gate + col0 + c * 32 : nullptr;
 #pragma unroll
       for (int g = 0; g < 4; ++g) {
         float v[8];
 #pragma unroll
-        for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(r[g * 8 + i]);
+        for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(r[g * 8 + i]) * f_head;
         if (z != nullptr) {
           float f[8];
           bf16x8_to_f32(ptx::ld_v4(z + g * 8), f);
@@ -79,17 +82,17 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_consta
 }
 
 template <int BN>
-int launch_head(const void* x, const void* w, void* y, const void* gate, int rows, int heads, int n, int k_dim, int64_t ldx, int64_t ldy, int64_t ld_gate,
-                Status* status, cudaStream_t stream) {
+int launch_head(const void* x, const void* w, void* y, const void* gate, int rows, int heads, int n, int k_dim, int64_t ldx, int64_t ldw, int64_t ldy, int64_t ld_gate,
+                int gate_heads, Status* status, cudaStream_t stream) {
   constexpr int STAGES = 6;
   using L = gemm::SmemLayout<BN, STAGES>;
   CUtensorMap tx, tw;
   if (!make_tmap_2d(&tx, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, x, rows, static_cast<uint64_t>(heads) * k_dim, ldx * 2, 128, 64, CU_TENSOR_MAP_SWIZZLE_128B) ||
-      !make_tmap_2d(&tw, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, w, static_cast<uint64_t>(heads) * n, k_dim, static_cast<uint64_t>(k_dim) * 2, BN, 64,
+      !make_tmap_2d(&tw, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, w, static_cast<uint64_t>(heads) * n, k_dim, ldw * 2, BN, 64,
                     CU_TENSOR_MAP_SWIZZLE_128B))
     return -kBadArgument;
   const HeadSched sched{(rows + 127) / 128, n / BN, heads, n, k_dim, BN};
-  const HeadEpilogue<BN> epi{static_cast<__nv_bfloat16*>(y), static_cast<const __nv_bfloat16*>(gate), ldy, ld_gate, rows, n};
+  const HeadEpilogue<BN> epi{static_cast<__nv_bfloat16*>(y), static_cast<const __nv_bfloat16*>(gate), ldy, ld_gate, rows, n, gate_heads};
   auto kern = head_gemm_kernel<BN, STAGES>;
   static DeviceOnce attr_once;
   if (const int rc = attr_once.max_smem(kern, L::kTotalBytes)) return rc;
@@ -103,14 +106,14 @@ int launch_head(const void* x, const void* w, void* y, const void* gate, int row
 
 using namespace b2;
 
-extern "C" int b2_head_gemm_bf16(const void* x, const void* w, void* y, const void* gate, int rows, int heads, int n, int k_dim, int64_t ldx, int64_t ldy,
-                                 int64_t ld_gate, Status* status, cudaStream_t stream) {
+extern "C" int b2_head_gemm_bf16(const void* x, const void* w, void* y, const void* gate, int rows, int heads, int n, int k_dim, int64_t ldx, int64_t ldw,
+                                 int64_t ldy, int64_t ld_gate, int gate_heads, Status* status, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (heads <= 0 || n <= 0 || n % 64 != 0 || k_dim <= 0 || k_dim % 64 != 0 || ldx % 8 != 0 || ldy % 8 != 0 || (reinterpret_cast<uintptr_t>(y) & 15) != 0 ||
-      (gate != nullptr && (ld_gate % 8 != 0 || (reinterpret_cast<uintptr_t>(gate) & 15) != 0)))
+  if (heads <= 0 || n <= 0 || n % 64 != 0 || k_dim <= 0 || k_dim % 64 != 0 || ldx % 8 != 0 || ldw % 8 != 0 || ldw < k_dim || ldy % 8 != 0 || (reinterpret_cast<uintptr_t>(y) & 15) != 0 ||
+      (gate != nullptr && !gate_heads && (ld_gate % 8 != 0 || (reinterpret_cast<uintptr_t>(gate) & 15) != 0)))
     return -kBadArgument;
   // wide tiles once they alone fill the machine
   const int64_t wide = static_cast<int64_t>((rows + 127) / 128) * heads * (n / 128);
-  if (n % 128 == 0 && wide >= kNumSMs) return launch_head<128>(x, w, y, gate, rows, heads, n, k_dim, ldx, ldy, ld_gate, status, stream);
-  return launch_head<64>(x, w, y, gate, rows, heads, n, k_dim, ldx, ldy, ld_gate, status, stream);
+  if (n % 128 == 0 && wide >= kNumSMs) return launch_head<128>(x, w, y, gate, rows, heads, n, k_dim, ldx, ldw, ldy, ld_gate, gate_heads, status, stream);
+  return launch_head<64>(x, w, y, gate, rows, heads, n, k_dim, ldx, ldw, ldy, ld_gate, gate_heads, status, stream);
 }

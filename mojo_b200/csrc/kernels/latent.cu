@@ -1,5 +1,5 @@
-// Around latent attention: the normalised latent of every new token into its cache row, and the latents of whole contexts
-// out of their pages (for prompts, whose keys and values are then expanded by one matrix product).
+// Around latent attention: the normalised latent of every new token into its cache row (with the rotated key part that all heads
+// share, while the queries rotate), and the latents of whole contexts out of their pages (for prompts, whose keys and values are then expanded by one matrix product).
 #include <cstdint>
 #include "b2/elem.cuh"
 #include "b2/latent.h"
@@ -10,18 +10,10 @@
 namespace b2 {
 namespace {
 
-// One warp per token; the row, up to 1024 columns, stays in registers.
+// One warp: dst[0 : rank] = rms_norm(src) * weight, zeros up to `pad`. The row, up to 1024 columns, stays in registers.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128) latent_write_kernel(const T* __restrict__ c, int64_t ld, const float* __restrict__ weight, float eps,
-                                                           const int64_t* __restrict__ slots, T* __restrict__ cache, int rows, int rank, int pad,
-                                                           int64_t num_slots, Status* status) {
-  ptx::grid_dep_sync();
+__device__ __forceinline__ void write_latent(const T* src, const float* weight, float eps, T* dst, int rank, int pad, int lane) {
   constexpr int kMaxIt = 32 / VEC;
-  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= rows) return;
-  const int64_t slot = slots[row];
-  if (slot < 0 || !B2_ASSERT(status, slot < num_slots, kSiteKvIndex, slot, num_slots)) return;
-  const T* src = c + row * ld;
   float v[kMaxIt][VEC], ss = 0.0f;
 #pragma unroll
   for (int i = 0; i < kMaxIt; ++i) {
@@ -33,7 +25,6 @@ __global__ void __launch_bounds__(128) latent_write_kernel(const T* __restrict__
     }
   }
   const float r = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(rank) + eps);
-  T* dst = cache + slot * pad;
 #pragma unroll
   for (int i = 0; i < kMaxIt; ++i) {
     const int col = (i * 32 + lane) * VEC;
@@ -46,6 +37,82 @@ __global__ void __launch_bounds__(128) latent_write_kernel(const T* __restrict__
     }
     store_f32<VEC>(dst + col, o);
   }
+}
+
+// One warp per token.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(128) latent_write_kernel(const T* __restrict__ c, int64_t ld, const float* __restrict__ weight, float eps,
+                                                           const int64_t* __restrict__ slots, T* __restrict__ cache, int rows, int rank, int pad,
+                                                           int64_t num_slots, Status* status) {
+  ptx::grid_dep_sync();
+  const int row = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= rows) return;
+  const int64_t slot = slots[row];
+  if (slot < 0 || !B2_ASSERT(status, slot < num_slots, kSiteKvIndex, slot, num_slots)) return;
+  write_latent<T, VEC>(c + row * ld, weight, eps, cache + slot * pad, rank, pad, lane);
+}
+
+// One CTA per token: the first warp writes the cache row, all of them rotate the queries. PAIR: query pairs are aligned.
+template <typename T, int VEC, bool PAIR>
+__global__ void __launch_bounds__(128) latent_rope_kernel(const B2LatentRopeArgs a, Status* status) {
+  ptx::grid_dep_sync();
+  const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = a.rot >> 1;
+  int pos = a.positions[row];
+  if (!B2_ASSERT(status, pos >= 0 && pos < a.max_pos, kSiteKvIndex, pos, a.max_pos)) pos = 0;
+  const float* cs = a.cos_sin + static_cast<int64_t>(pos) * a.rot;
+  const auto turn = [&](int i, float& u, float& v) {
+    const float c = cs[i], s = cs[half + i], x = u;
+    u = x * c - v * s;
+    v = v * c + x * s;
+  };
+  if (warp == 0) {
+    const int64_t slot = a.slots[row];
+    if (slot >= 0 && B2_ASSERT(status, slot < a.num_slots, kSiteKvIndex, slot, a.num_slots)) {
+      T* dst = static_cast<T*>(a.cache) + slot * a.pad;
+      write_latent<T, VEC>(static_cast<const T*>(a.c) + row * a.ld, a.weight, a.eps, dst, a.rank, a.column, lane);
+      const T* k = static_cast<const T*>(a.k) + row * a.ld;
+      for (int i = lane; i < half; i += 32) {
+        float u[1], v[1];
+        load_f32<1>(k + 2 * i, u);
+        load_f32<1>(k + 2 * i + 1, v);
+        turn(i, u[0], v[0]);
+        store_f32<1>(dst + a.column + 2 * i, u);
+        store_f32<1>(dst + a.column + 2 * i + 1, v);
+      }
+      const float zero[1] = {0.0f};
+      for (int i = a.column + a.rot + lane; i < a.pad; i += 32) store_f32<1>(dst + i, zero);
+    }
+  }
+  T* q = static_cast<T*>(a.q) + row * a.ld_q + a.q_off;
+  // the first warp has less of this to do
+  for (int i = threadIdx.x < 32 ? a.heads * half : static_cast<int>(threadIdx.x) - 32; i < a.heads * half; i += 96) {
+    const int h = i / half, p = i - h * half;
+    T* at = q + static_cast<int64_t>(h) * a.q_dim + 2 * p;
+    if constexpr (PAIR) {
+      float uv[2];
+      load_f32<2>(at, uv);
+      turn(p, uv[0], uv[1]);
+      store_f32<2>(at, uv);
+    } else {
+      float u[1], v[1];
+      load_f32<1>(at, u);
+      load_f32<1>(at + 1, v);
+      turn(p, u[0], v[0]);
+      store_f32<1>(at, u);
+      store_f32<1>(at + 1, v);
+    }
+  }
+}
+
+template <typename T>
+int launch_rope(const B2LatentRopeArgs& a, Status* status, cudaStream_t stream) {
+  const uintptr_t addr = reinterpret_cast<uintptr_t>(a.c) | reinterpret_cast<uintptr_t>(a.cache);
+  const bool v4 = a.rank % 4 == 0 && a.column % 4 == 0 && a.pad % 4 == 0 && a.ld % 4 == 0 && addr % 16 == 0;
+  const bool pair = a.q_off % 2 == 0 && a.q_dim % 2 == 0 && a.ld_q % 2 == 0 && reinterpret_cast<uintptr_t>(a.q) % (2 * sizeof(T)) == 0;
+  auto kern = v4 ? (pair ? latent_rope_kernel<T, 4, true> : latent_rope_kernel<T, 4, false>)
+                 : (pair ? latent_rope_kernel<T, 1, true> : latent_rope_kernel<T, 1, false>);
+  launch_pdl(kern, dim3(a.rows), dim3(128), 0, stream, a, status);
+  return last_launch_rc();
 }
 
 template <typename T, int VEC>
@@ -101,6 +168,14 @@ extern "C" int b2_latent_write(const void* c, int64_t ld, const float* weight, f
   if (v4) B2_WRITE(__nv_bfloat16, 4);
   B2_WRITE(__nv_bfloat16, 1);
 #undef B2_WRITE
+}
+
+extern "C" int b2_latent_write_rope(const B2LatentRopeArgs* a, int f32, Status* status, cudaStream_t stream) {
+  if (a->rows <= 0) return 0;
+  if (a->rank <= 0 || a->rot <= 0 || a->rot % 2 != 0 || a->column < a->rank || a->column > 1024 || a->pad < a->column + a->rot || a->heads <= 0 ||
+      a->q_off < 0 || a->q_off + a->rot > a->q_dim || a->ld_q < static_cast<int64_t>(a->heads) * a->q_dim)
+    return -kBadArgument;
+  return f32 ? launch_rope<float>(*a, status, stream) : launch_rope<__nv_bfloat16>(*a, status, stream);
 }
 
 extern "C" int b2_latent_gather_bf16(const void* cache, const int32_t* pages, const int32_t* ctx_lens, const int32_t* block_tables, void* out,

@@ -6,8 +6,8 @@
 // i.e. one 16-row MMA tile against a 576-wide key that doubles as a 512-wide value: every cache byte is read
 // once and used twice.
 //
-// The kernel is a template over the latent and rope widths: 512 + 64 as above, or a latent of 64 ... 1024 columns without a
-// rotated part.
+// The kernel is a template over the latent and rope widths: 512 + 64 as above, or a latent of 64 ... 1024 columns with a rotated
+// part of 0, 64 or 128. A row may see only the last `window` positions of its context; tiles before those are not read.
 //
 // CTA = 4 warps on one (KV split, head group, sequence). A 32-token tile (36 KB at 512 + 64) arrives as SWIZZLE_128B
 // TMA boxes of 64 columns through a 2- or 3-stage mbarrier ring (pages below 32 tokens: one set of boxes per page). Each
@@ -72,8 +72,8 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
     const __grid_constant__ CUtensorMap tmap_kv, const __nv_bfloat16* __restrict__ q_lat,
     const __nv_bfloat16* __restrict__ q_rope, __nv_bfloat16* __restrict__ out_lat, const int32_t* __restrict__ ctx_lens,
     const int32_t* __restrict__ block_tables, const int32_t* __restrict__ row_seq, float* __restrict__ workspace,
-    int max_blocks, int n_heads, int page_size, int box_rows, int num_splits, float scale_log2, int64_t num_pages, int64_t q_lat_stride,
-    int64_t q_rope_stride, Status* status) {
+    int max_blocks, int n_heads, int page_size, int box_rows, int num_splits, float scale_log2, int window, int64_t num_pages, int64_t q_lat_stride,
+    int64_t q_rope_stride, int q_lat_head, int q_rope_head, Status* status) {
   using S = LatentShape<LAT, ROPE>;
   constexpr int kLat = LAT, kRope = ROPE, kRow = S::kRow, kSub = S::kSub, kTileBytes = S::kTileBytes, kSteps = S::kSteps, kCols = S::kCols;
   constexpr int kScoreLd = S::kScoreLd;
@@ -94,9 +94,10 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
   const int head0 = hg * 16;
   const int rows = min(16, n_heads - head0);
 
-  const int tiles_total = (ctx + BN - 1) / BN;
-  const int tiles_per_split = (tiles_total + num_splits - 1) / num_splits;
-  const int tile_begin = split * tiles_per_split;
+  const int first = max(0, ctx - window);      // the first position this row sees
+  const int tiles_total = (ctx + BN - 1) / BN, first_tile = first / BN;
+  const int tiles_per_split = (tiles_total - first_tile + num_splits - 1) / num_splits;
+  const int tile_begin = first_tile + split * tiles_per_split;
   const int tile_end = min(tiles_total, tile_begin + tiles_per_split);
   const int n_tiles = max(0, tile_end - tile_begin);
 
@@ -127,9 +128,9 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
     const int r = i / (kRow / 8), c = i % (kRow / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
     if (r < rows) {
-      // row strides in elements: the two query parts may be column slices of one wider projection output
-      v = ROPE == 0 || c < kLat / 8 ? reinterpret_cast<const uint4*>(q_lat + seq * q_lat_stride + static_cast<int64_t>(head0 + r) * kLat)[c]
-                       : reinterpret_cast<const uint4*>(q_rope + seq * q_rope_stride + static_cast<int64_t>(head0 + r) * kRope)[c - kLat / 8];
+      // row and head strides in elements: the two query parts may be column slices of one wider projection output
+      v = ROPE == 0 || c < kLat / 8 ? reinterpret_cast<const uint4*>(q_lat + seq * q_lat_stride + static_cast<int64_t>(head0 + r) * q_lat_head)[c]
+                       : reinterpret_cast<const uint4*>(q_rope + seq * q_rope_stride + static_cast<int64_t>(head0 + r) * q_rope_head)[c - kLat / 8];
     }
     // plain row-major with an XOR on the low 3 chunk bits to spread ldmatrix rows over banks
     reinterpret_cast<uint4*>(q_gen)[r * (kRow / 8) + ((c & ~7) | ((c & 7) ^ (r & 7)))] = v;
@@ -213,10 +214,10 @@ __global__ void __launch_bounds__(128, STAGES == 2 && LAT <= 512 ? 2 : 1) mla_de
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int col = kv0 + j * 8 + 2 * t4;
-      s[j][0] = col <= max_lo ? s[j][0] * scale_log2 : -INFINITY;
-      s[j][1] = col + 1 <= max_lo ? s[j][1] * scale_log2 : -INFINITY;
-      s[j][2] = col <= max_hi ? s[j][2] * scale_log2 : -INFINITY;
-      s[j][3] = col + 1 <= max_hi ? s[j][3] * scale_log2 : -INFINITY;
+      s[j][0] = col <= max_lo && col >= first ? s[j][0] * scale_log2 : -INFINITY;
+      s[j][1] = col + 1 <= max_lo && col + 1 >= first ? s[j][1] * scale_log2 : -INFINITY;
+      s[j][2] = col <= max_hi && col >= first ? s[j][2] * scale_log2 : -INFINITY;
+      s[j][3] = col + 1 <= max_hi && col + 1 >= first ? s[j][3] * scale_log2 : -INFINITY;
       mx_lo = fmaxf(mx_lo, fmaxf(s[j][0], s[j][1]));
       mx_hi = fmaxf(mx_hi, fmaxf(s[j][2], s[j][3]));
     }
@@ -341,7 +342,8 @@ __global__ void mla_rows_meta_kernel(const int32_t* __restrict__ cu_q, const int
 template <int LAT, int ROPE>
 int launch_latent(const void* q_lat, const void* q_rope, const void* kv_cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
                   const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int page_size, int num_splits, float scale,
-                  int64_t num_pages, int64_t q_lat_stride, int64_t q_rope_stride, Status* status, cudaStream_t stream) {
+                  int window, int64_t num_pages, int64_t q_lat_stride, int64_t q_rope_stride, int q_lat_head, int q_rope_head, Status* status,
+                  cudaStream_t stream) {
   using S = LatentShape<LAT, ROPE>;
   if (rows <= 0) return 0;
   if (n_heads <= 0 || page_size <= 0 || page_size % 8 != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr)) return -kBadArgument;
@@ -374,7 +376,7 @@ int launch_latent(const void* q_lat, const void* q_rope, const void* kv_cache, v
         tk, static_cast<const __nv_bfloat16*>(q_lat) + r0 * q_lat_stride, ROPE == 0 ? nullptr : static_cast<const __nv_bfloat16*>(q_rope) + r0 * q_rope_stride,
         out, row_ctx + r0, row_seq == nullptr ? block_tables + static_cast<int64_t>(r0) * max_blocks : block_tables,
         row_seq == nullptr ? nullptr : row_seq + r0, ws, max_blocks, n_heads, page_size, box_rows,
-        num_splits, scale * ptx::kLog2e, num_pages, q_lat_stride, q_rope_stride, status);
+        num_splits, scale * ptx::kLog2e, window > 0 ? window : 1 << 30, num_pages, q_lat_stride, q_rope_stride, q_lat_head, q_rope_head, status);
     if (num_splits > 1) {
       const int total = n * n_heads;
       mla_reduce_kernel<LAT><<<(total + 3) / 4, 128, 0, stream>>>(ws, out, num_splits, total);
@@ -409,21 +411,35 @@ extern "C" int b2_mla_attend_bf16(const void* q_lat, const void* q_rope, const v
                                   int64_t num_pages, int64_t q_lat_stride, int64_t q_rope_stride, Status* status,
                                   cudaStream_t stream) {
   return launch_latent<512, 64>(q_lat, q_rope, kv_cache, out_lat, row_ctx, block_tables, row_seq, workspace, rows, max_blocks, n_heads, page_size,
-                                num_splits, scale, num_pages, q_lat_stride, q_rope_stride, status, stream);
+                                num_splits, scale, 0, num_pages, q_lat_stride, q_rope_stride, 512, 64, status, stream);
 }
 
-extern "C" int b2_latent_attend_bf16(const void* q_lat, const void* cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
-                                     const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int latent, int page_size,
-                                     int num_splits, float scale, int64_t num_pages, int64_t q_lat_stride, Status* status, cudaStream_t stream) {
-#define B2_LATENT(LAT_)                                                                                                                        \
-  return launch_latent<LAT_, 0>(q_lat, nullptr, cache, out_lat, row_ctx, block_tables, row_seq, workspace, rows, max_blocks, n_heads, page_size, \
-                                num_splits, scale, num_pages, q_lat_stride, 0, status, stream)
-  switch (latent) {
-    case 64: B2_LATENT(64);
-    case 128: B2_LATENT(128);
-    case 256: B2_LATENT(256);
-    case 512: B2_LATENT(512);
-    case 1024: B2_LATENT(1024);
+extern "C" int b2_latent_attend_bf16(const void* q, const void* cache, void* out_lat, const int32_t* row_ctx, const int32_t* block_tables,
+                                     const int32_t* row_seq, float* workspace, int rows, int max_blocks, int n_heads, int latent, int rot, int page_size,
+                                     int num_splits, float scale, int window, int64_t num_pages, int64_t q_stride, Status* status,
+                                     cudaStream_t stream) {
+  const void* q_rot = static_cast<const __nv_bfloat16*>(q) + latent;
+  const int row = latent + rot;
+#define B2_LATENT(LAT_, ROT_)                                                                                                                     \
+  case LAT_ * 1000 + ROT_:                                                                                                                        \
+    return launch_latent<LAT_, ROT_>(q, q_rot, cache, out_lat, row_ctx, block_tables, row_seq, workspace, rows, max_blocks, n_heads, page_size,   \
+                                     num_splits, scale, window, num_pages, q_stride, q_stride, row, row, status, stream)
+  switch (latent * 1000 + rot) {
+    B2_LATENT(64, 0);
+    B2_LATENT(128, 0);
+    B2_LATENT(256, 0);
+    B2_LATENT(512, 0);
+    B2_LATENT(1024, 0);
+    B2_LATENT(64, 64);
+    B2_LATENT(128, 64);
+    B2_LATENT(256, 64);
+    B2_LATENT(512, 64);
+    B2_LATENT(1024, 64);
+    B2_LATENT(64, 128);
+    B2_LATENT(128, 128);
+    B2_LATENT(256, 128);
+    B2_LATENT(512, 128);
+    B2_LATENT(1024, 128);
     default: return -kBadArgument;
   }
 #undef B2_LATENT

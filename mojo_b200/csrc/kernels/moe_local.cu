@@ -19,62 +19,121 @@ namespace {
 constexpr int kMaxTop = 32;
 constexpr int kMaxExperts = 1024;
 
-// One warp per row, NV logits per lane.
+// Index of the largest value over a warp's NV * 32 (lane + 32 i), lowest index on ties; `none` where nothing compares.
 template <int NV>
-__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld, float* __restrict__ weights, int32_t* __restrict__ ids,
-                                                        int32_t* __restrict__ place, int32_t* __restrict__ counts, int rows, int experts, int top,
+__device__ __forceinline__ int warp_argmax(const float (&v)[NV], int lane, int none, float& best) {
+  best = -INFINITY;
+  int at = none;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (v[i] > best) { best = v[i]; at = lane + 32 * i; }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+    const int oe = __shfl_xor_sync(0xffffffffu, at, o);
+    if (ob > best || (ob == best && oe < at)) { best = ob; at = oe; }
+  }
+  return min(at, none);
+}
+
+// One warp per row, NV logits per lane. CHOICE: what chooses is not the score itself (a correction is added, groups are left
+// out); then scores and choice scores are held apart.
+template <int NV, bool CHOICE>
+__global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ correction,
+                                                        float* __restrict__ weights, int32_t* __restrict__ ids, int32_t* __restrict__ place,
+                                                        int32_t* __restrict__ counts, int rows, int experts, int outputs, int top, int groups, int keep,
                                                         int sigmoid, int norm_top, float scale) {
   ptx::grid_dep_sync();
+  __shared__ float pool[CHOICE ? 8 : 1][CHOICE ? NV * 32 : 1];
   const int row = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (row >= rows) return;
   float v[NV], mx = -INFINITY;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int e = lane + 32 * i;
-    v[i] = e < experts ? logits[row * ld + e] : -INFINITY;
+    v[i] = e < outputs ? logits[row * ld + e] : -INFINITY;
     mx = fmaxf(mx, v[i]);
   }
   float inv = 1.0f;
   if (sigmoid) {
 #pragma unroll
-    for (int i = 0; i < NV; ++i) v[i] = lane + 32 * i < experts ? sigmoid_f32(v[i]) : -1.0f;
+    for (int i = 0; i < NV; ++i) v[i] = lane + 32 * i < outputs ? sigmoid_f32(v[i]) : -INFINITY;
   } else {
     mx = warp_max(mx);
     float sum = 0.0f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      v[i] = lane + 32 * i < experts ? expf(v[i] - mx) : -1.0f;
+      v[i] = lane + 32 * i < outputs ? expf(v[i] - mx) : -INFINITY;
       if (v[i] > 0.0f) sum += v[i];
     }
     inv = 1.0f / warp_sum(sum);
   }
+  float score[CHOICE ? NV : 1];
+  if constexpr (CHOICE) {
+    float* mine = pool[threadIdx.x >> 5];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int e = lane + 32 * i;
+      score[i] = v[i] * inv;
+      v[i] = e < outputs ? score[i] + (correction != nullptr ? correction[e] : 0.0f) : -INFINITY;
+      mine[e] = v[i];
+    }
+    inv = 1.0f;
+    if (keep < groups) {
+      const int per = outputs / groups;
+      float gm[NV];
+      uint32_t kept = 0;
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        gm[i] = -INFINITY;
+        if (lane + 32 * i < groups)
+          for (int j = 0; j < per; ++j) gm[i] = fmaxf(gm[i], mine[(lane + 32 * i) * per + j]);
+      }
+      for (int j = 0; j < keep; ++j) {
+        float best;
+        const int g = warp_argmax<NV>(gm, lane, groups - 1, best);
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (g == lane + 32 * i) {
+            gm[i] = -INFINITY;
+            kept |= 1u << i;
+          }
+      }
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (lane + 32 * i < groups) mine[lane + 32 * i] = (kept >> i) & 1u ? 1.0f : 0.0f;
+      __syncwarp();
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (lane + 32 * i < outputs && mine[(lane + 32 * i) / per] == 0.0f) v[i] = -INFINITY;
+    }
+  }
   float sel_w = 0.0f, total = 0.0f;   // lane j keeps the j-th choice
   int sel_e = 0;
   for (int j = 0; j < top; ++j) {
-    float best = -2.0f;
-    int best_e = experts - 1;         // where nothing compares (NaN logits): still a valid expert
+    float best;
+    const int best_e = warp_argmax<NV>(v, lane, outputs - 1, best);    // where nothing compares (NaN logits): still a valid output
+    if constexpr (CHOICE) {
+      float own = 0.0f;
 #pragma unroll
-    for (int i = 0; i < NV; ++i)
-      if (v[i] > best) { best = v[i]; best_e = lane + 32 * i; }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
-      if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
+      for (int i = 0; i < NV; ++i)
+        if (best_e == lane + 32 * i) own = score[i];
+      best = __shfl_sync(0xffffffffu, own, best_e & 31);
     }
-    best_e = min(best_e, experts - 1);
 #pragma unroll
     for (int i = 0; i < NV; ++i)
-      if (best_e == lane + 32 * i) v[i] = -2.0f;   // out of the pool
+      if (best_e == lane + 32 * i) v[i] = -INFINITY;   // out of the pool
     if (lane == j) { sel_w = best * inv; sel_e = best_e; }
     total += best * inv;
   }
   if (lane < top) {
-    if (norm_top) sel_w /= total;
+    if (norm_top) sel_w /= total + 1e-20f;
     const int64_t at = static_cast<int64_t>(row) * top + lane;
     weights[at] = sel_w * scale;
     ids[at] = sel_e;
-    place[at] = atomicAdd(counts + sel_e, 1);
+    place[at] = sel_e < experts ? atomicAdd(counts + sel_e, 1) : 0;
   }
 }
 
@@ -122,8 +181,9 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x
     int mine = 0;
     if (lane < top) {
       const int64_t at = static_cast<int64_t>(t) * top + lane;
-      mine = first[ids[at]] + place[at];
-      if (!B2_ASSERT(status, mine >= 0 && mine < rows * top, kSiteEpCount, mine, rows * top)) mine = 0;
+      const int id = ids[at];
+      mine = id < experts ? first[id] + place[at] : -1;      // what returns its input needs no copy of it
+      if (!B2_ASSERT(status, mine >= -1 && mine < rows * top, kSiteEpCount, mine, rows * top)) mine = 0;
       slot[at] = mine;
     }
     const uint4* src = reinterpret_cast<const uint4*>(x) + static_cast<int64_t>(t) * vecs;
@@ -133,7 +193,9 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x
       for (int u = 0; u < 4; ++u)
         if (c0 + u * 32 + lane < vecs) r[u] = ptx::ld_nc_v4(src + c0 + u * 32 + lane);
       for (int j = 0; j < top; ++j) {
-        uint4* dst = reinterpret_cast<uint4*>(xs) + static_cast<int64_t>(__shfl_sync(0xffffffffu, mine, j)) * vecs;
+        const int to = __shfl_sync(0xffffffffu, mine, j);
+        if (to < 0) continue;
+        uint4* dst = reinterpret_cast<uint4*>(xs) + static_cast<int64_t>(to) * vecs;
 #pragma unroll
         for (int u = 0; u < 4; ++u)
           if (c0 + u * 32 + lane < vecs) dst[c0 + u * 32 + lane] = r[u];
@@ -195,7 +257,7 @@ int launch_tiles(const void* x, const void* w, const int32_t* tiles, const int32
 
 // 64 x 64 tile, 256 threads of 4 x 4 outputs.
 __global__ void __launch_bounds__(256) moe_tiles_f32_kernel(const float* __restrict__ x, const float* __restrict__ w, const int4* __restrict__ tiles,
-                                                            const int32_t* __restrict__ n_tiles, float* __restrict__ y, int n, int k) {
+                                                            const int32_t* __restrict__ n_tiles, float* __restrict__ y, int n, int k, int epilogue) {
   ptx::grid_dep_sync();
   if (static_cast<int>(blockIdx.y) >= *n_tiles) return;
   const int4 tile = tiles[blockIdx.y];
@@ -227,7 +289,7 @@ __global__ void __launch_bounds__(256) moe_tiles_f32_kernel(const float* __restr
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (tm + i < tile.z && n0 + tn + j < n) y[static_cast<int64_t>(tile.y + tm + i) * n + n0 + tn + j] = acc[i][j];
+      if (tm + i < tile.z && n0 + tn + j < n) y[static_cast<int64_t>(tile.y + tm + i) * n + n0 + tn + j] = epilogue == B2_EPI_RELU2 ? relu2(acc[i][j]) : acc[i][j];
 }
 
 }  // namespace
@@ -235,12 +297,19 @@ __global__ void __launch_bounds__(256) moe_tiles_f32_kernel(const float* __restr
 
 using namespace b2;
 
-extern "C" int b2_moe_route(const float* logits, int64_t ld, float* weights, int32_t* ids, int32_t* place, int32_t* counts, int rows, int experts,
-                            int top, int scoring, int norm_top, float scale, cudaStream_t stream) {
+extern "C" int b2_moe_route(const float* logits, int64_t ld, const float* correction, float* weights, int32_t* ids, int32_t* place, int32_t* counts,
+                            int rows, int experts, int identity, int top, int groups, int keep, int scoring, int norm_top, float scale,
+                            cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (experts < 1 || experts > kMaxExperts || top < 1 || top > kMaxTop || top > experts || ld < experts || scoring < 0 || scoring > 1) return -kBadArgument;
-  auto kern = experts <= 256 ? moe_route_kernel<8> : moe_route_kernel<32>;
-  launch_pdl(kern, dim3((rows + 7) / 8), dim3(256), 0, stream, logits, ld, weights, ids, place, counts, rows, experts, top, scoring, norm_top, scale);
+  const int outputs = experts + identity;
+  if (experts < 1 || identity < 0 || outputs > kMaxExperts || groups < 1 || outputs % groups != 0 || keep < 1 || keep > groups || top < 1 || top > kMaxTop ||
+      top > outputs / groups * keep || ld < outputs || scoring < 0 || scoring > 1)
+    return -kBadArgument;
+  const bool choice = correction != nullptr || keep < groups;
+  auto kern = outputs <= 256 ? (choice ? moe_route_kernel<8, true> : moe_route_kernel<8, false>)
+                             : (choice ? moe_route_kernel<32, true> : moe_route_kernel<32, false>);
+  launch_pdl(kern, dim3((rows + 7) / 8), dim3(256), 0, stream, logits, ld, correction, weights, ids, place, counts, rows, experts, outputs, top, groups, keep,
+             scoring, norm_top, scale);
   return last_launch_rc();
 }
 
@@ -264,7 +333,7 @@ extern "C" int b2_moe_gather(const void* x, const int32_t* ids, const int32_t* p
 extern "C" int b2_moe_tiles_gemm_bf16(const void* x, const void* w, const int32_t* tiles, const int32_t* n_tiles, void* y, int rows, int experts, int n,
                                       int k, int epilogue, const B2EpiAct* act, int bn, Status* status, cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (experts < 1 || n <= 0 || k <= 0 || k % 8 != 0 || (epilogue != B2_EPI_NONE && epilogue != B2_EPI_SWIGLU) || (epilogue == B2_EPI_SWIGLU && n % 32 != 0))
+  if (experts < 1 || n <= 0 || k <= 0 || k % 8 != 0 || (epilogue != B2_EPI_NONE && epilogue != B2_EPI_RELU2 && epilogue != B2_EPI_SWIGLU) || (epilogue == B2_EPI_SWIGLU && n % 32 != 0))
     return -kBadArgument;
   switch (bn) {
     case 16: return launch_tiles<16>(x, w, tiles, n_tiles, y, rows, experts, n, k, epilogue, act, status, stream);
@@ -277,9 +346,9 @@ extern "C" int b2_moe_tiles_gemm_bf16(const void* x, const void* w, const int32_
 }
 
 extern "C" int b2_moe_tiles_gemm_f32(const float* x, const float* w, const int32_t* tiles, const int32_t* n_tiles, float* y, int max_tiles, int n, int k,
-                                     cudaStream_t stream) {
+                                     int epilogue, cudaStream_t stream) {
   if (max_tiles <= 0) return 0;
-  if (n <= 0 || k <= 0 || max_tiles > 65535) return -kBadArgument;
-  launch_pdl(moe_tiles_f32_kernel, dim3((n + 63) / 64, max_tiles), dim3(256), 0, stream, x, w, reinterpret_cast<const int4*>(tiles), n_tiles, y, n, k);
+  if (n <= 0 || k <= 0 || max_tiles > 65535 || (epilogue != B2_EPI_NONE && epilogue != B2_EPI_RELU2)) return -kBadArgument;
+  launch_pdl(moe_tiles_f32_kernel, dim3((n + 63) / 64, max_tiles), dim3(256), 0, stream, x, w, reinterpret_cast<const int4*>(tiles), n_tiles, y, n, k, epilogue);
   return last_launch_rc();
 }

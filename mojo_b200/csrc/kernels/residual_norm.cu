@@ -1,5 +1,6 @@
 // A plain residual kept in f32: one kernel between any two sublayers adds the finished one (a matrix product's rows, the
-// weighted rows of a token's experts, or both, scaled per channel) and RMS-normalises what the next one reads. The first
+// weighted rows of a token's experts, a row with a gate, or several of them, scaled per channel) and RMS- or layer-normalises
+// what the next one reads. The first
 // call starts the stream from the embedding tables. One CTA per token row.
 #include <cstdint>
 #include "b2/elem.cuh"
@@ -27,7 +28,7 @@ __global__ void residual_norm_kernel(const B2ResidualArgs a, Status* status) {
   if (a.experts != nullptr) {
     if (threadIdx.x < a.top) {
       const int slot = a.expert_slot[row * a.top + threadIdx.x];
-      const bool ok = B2_ASSERT(status, slot >= 0 && slot < a.expert_rows, kSiteEpCount, slot, a.expert_rows);
+      const bool ok = B2_ASSERT(status, slot >= (a.own != nullptr ? -1 : 0) && slot < a.expert_rows, kSiteEpCount, slot, a.expert_rows);
       e_row[threadIdx.x] = ok ? slot : 0;
       e_w[threadIdx.x] = ok ? a.expert_w[row * a.top + threadIdx.x] : 0.0f;
     }
@@ -48,7 +49,10 @@ __global__ void residual_norm_kernel(const B2ResidualArgs a, Status* status) {
       }
     }
   }
-  const bool fold = y != nullptr || a.experts != nullptr;
+  const T* own = a.own != nullptr ? static_cast<const T*>(a.own) + row * W : nullptr;
+  const T* gated = a.gated != nullptr ? static_cast<const T*>(a.gated) + row * W : nullptr;
+  const float gate = gated != nullptr ? sigmoid_f32(a.gate[row * a.ld_gate]) : 0.0f;
+  const bool fold = y != nullptr || a.experts != nullptr || gated != nullptr;
   float ss = 0.0f;
   for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
     float v[VEC];
@@ -70,7 +74,8 @@ __global__ void residual_norm_kernel(const B2ResidualArgs a, Status* status) {
           float e[4][VEC];
 #pragma unroll
           for (int j = 0; j < 4; ++j)
-            if (j0 + j < a.top) load_f32<VEC>(static_cast<const T*>(a.experts) + static_cast<int64_t>(e_row[j0 + j]) * W + c, e[j]);
+            if (j0 + j < a.top)
+              load_f32<VEC>((e_row[j0 + j] < 0 ? own : static_cast<const T*>(a.experts) + static_cast<int64_t>(e_row[j0 + j]) * W) + c, e[j]);
 #pragma unroll
           for (int j = 0; j < 4; ++j)
             if (j0 + j < a.top)
@@ -78,17 +83,39 @@ __global__ void residual_norm_kernel(const B2ResidualArgs a, Status* status) {
               for (int i = 0; i < VEC; ++i) u[i] = fmaf(e_w[j0 + j], e[j][i], u[i]);
         }
       }
-      load_f32<VEC>(a.y_scale + c, s);
+      if (gated != nullptr) {
+        float g[VEC];
+        load_f32<VEC>(gated + c, g);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v[i] = fmaf(s[i], u[i], v[i]);
+        for (int i = 0; i < VEC; ++i) u[i] = fmaf(gate, g[i], u[i]);
+      }
+      if (a.y_scale != nullptr) {
+        load_f32<VEC>(a.y_scale + c, s);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = fmaf(s[i], u[i], v[i]);
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] += u[i];
+      }
     }
     if (a.store && (fold || a.ids != nullptr)) store_f32<VEC>(x + c, v);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) ss = fmaf(v[i], v[i], ss);
+    for (int i = 0; i < VEC; ++i) ss = a.bias != nullptr ? ss + v[i] : fmaf(v[i], v[i], ss);
     store_f32<VEC>(x_sm + c, v);
   }
   T* h = static_cast<T*>(a.h) + static_cast<int64_t>(blockIdx.x) * a.ld_h;
-  float r = 1.0f;
+  float r = 1.0f, mean = 0.0f;
+  if (a.bias != nullptr) {      // layer norm: squares of the deviations in a second pass
+    mean = block_sum(ss, scratch) / static_cast<float>(a.mean_width);
+    ss = 0.0f;
+    for (int c = threadIdx.x * VEC; c < a.mean_width; c += blockDim.x * VEC) {
+      float v[VEC];
+      load_f32<VEC>(x_sm + c, v);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i)
+        if (c + i < a.mean_width) ss = fmaf(v[i] - mean, v[i] - mean, ss);
+    }
+  }
   if (a.weight != nullptr) r = 1.0f / sqrtf(block_sum(ss, scratch) / static_cast<float>(a.mean_width) + a.eps);
   for (int c = threadIdx.x * VEC; c < W; c += blockDim.x * VEC) {
     float v[VEC], w[VEC];
@@ -96,7 +123,12 @@ __global__ void residual_norm_kernel(const B2ResidualArgs a, Status* status) {
     if (a.weight != nullptr) {
       load_f32<VEC>(a.weight + c, w);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) v[i] = v[i] * r * w[i];
+      for (int i = 0; i < VEC; ++i) v[i] = (v[i] - mean) * r * w[i];
+      if (a.bias != nullptr) {
+        load_f32<VEC>(a.bias + c, w);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] += w[i];
+      }
     }
     store_f32<VEC>(h + c, v);
   }
@@ -121,9 +153,8 @@ using namespace b2;
 
 extern "C" int b2_residual_norm(const B2ResidualArgs* a, int f32, Status* status, cudaStream_t stream) {
   if (a->n_out <= 0) return 0;
-  const bool fold = a->y != nullptr || a->experts != nullptr;
   if (a->width <= 0 || a->width > 50000 || a->mean_width <= 0 || a->mean_width > a->width || a->x == nullptr || a->h == nullptr ||
-      (fold && a->y_scale == nullptr) || (a->experts != nullptr && (a->expert_slot == nullptr || a->expert_w == nullptr || a->top < 1 || a->top > kMaxTop)) ||
+      (a->bias != nullptr && a->weight == nullptr) || (a->gated != nullptr && a->gate == nullptr) || (a->experts != nullptr && (a->expert_slot == nullptr || a->expert_w == nullptr || a->top < 1 || a->top > kMaxTop)) ||
       (a->ids != nullptr && a->embed == nullptr) || (a->bigram != nullptr && (a->prev == nullptr || a->buckets < 1)) ||
       (a->rows_index == nullptr && a->n_out != a->rows))
     return -kBadArgument;

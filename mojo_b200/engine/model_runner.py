@@ -103,6 +103,9 @@ class ModelRunner:
         self.has_state = bool(getattr(model, "recurrent_state", False))
         # models whose embedding also looks at the token before each row
         self.needs_prev = bool(getattr(model, "needs_prev_tokens", False))
+        # models whose prompt chunks attend by a list of work items
+        listed = getattr(model, "lists_prefill_work", None) or getattr(model, "supports_static_attention", None)
+        self.lists_work = bool(listed is not None and listed(cfg.page_size))
         nbytes = cfg.max_num_batched_tokens * 40 + cfg.max_num_seqs * (max_blocks * 4 + 96) + (1 << 16)
         if hasattr(model, "plan_latent_prefill"):      # scratch pages of 128 tokens of every context in a step, and their tables
             nbytes += cfg.max_num_seqs * (cfg.max_model_len // 128 + 1) * 12
@@ -363,8 +366,7 @@ class ModelRunner:
             if expand is not None:
                 seg_xpages, seg_xtables = st.put(expand[0], np.int32), st.put(expand[1], np.int32)
         seg_work, n_items = None, 0
-        if self.cuda and batch.num_prefill > 0 and (
-                expand is not None or getattr(self.model, "supports_static_attention", lambda *_: False)(self.cfg.page_size)):
+        if self.cuda and batch.num_prefill > 0 and (expand is not None or self.lists_work):
             # one CTA per (sequence, query tile) of the chunks, longest context first, instead of a padded grid
             work = ops.prefill_work_items(batch.cu_q, batch.ctx_lens, int(batch.num_decode))
             n_items = int(work.shape[0])

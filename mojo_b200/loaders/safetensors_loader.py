@@ -64,7 +64,7 @@ class _Reader:
 
 
 def load_safetensors_into(model, path: str | Path) -> None:
-    """Fill a model from a checkpoint directory: Llama family or DeepSeek-V2(-Lite) in Hugging Face layout, Rekudra, Rerupel."""
+    """Fill a model from a checkpoint directory: Llama family or DeepSeek-V2(-Lite) in Hugging Face layout, Rekudra, Rerupel, Pilutar."""
     rd = _Reader(read_safetensors_index(path))
     cfg = model.cfg
     if getattr(cfg, "architecture", "llama") == "deepseek_v2":
@@ -73,8 +73,8 @@ def load_safetensors_into(model, path: str | Path) -> None:
     if cfg.architecture == "rekudra":
         _load_rekudra(model, rd)
         return
-    if cfg.architecture == "rerupel":
-        _load_rerupel(model, rd)
+    if cfg.architecture in ("rerupel", "pilutar"):
+        _load_named_layers(model, rd)
         return
     model.layers.clear()
     model.load_tensor("embed", rd.get("model.embed_tokens.weight"))
@@ -160,8 +160,8 @@ def _load_rekudra(model, rd: _Reader) -> None:
     model.load_tensor("head", rd.get("head"))
 
 
-def _load_rerupel(model, rd: _Reader) -> None:
-    """Rerupel names: `embed`, `bigram`, `loop.in`, `final.norm`, and per layer `l<i>.norm1`, `l<i>.mix.*`, `l<i>.mlp.*`, `l<i>.ls<q>`."""
+def _load_named_layers(model, rd: _Reader) -> None:
+    """Rerupel and Pilutar: the names and shapes the model lists, those of layer i behind `l<i>.`."""
     model.layers.clear()
     for name in model.global_shapes():
         model.load_tensor(name, rd.get(name))

@@ -23,4 +23,8 @@ def build_model(cfg: ModelConfig, device="cpu", dtype=torch.float32, comm=None, 
         from .rerupel import RerupelModel
 
         return RerupelModel(cfg, device, dtype, comm=comm)
+    if cfg.architecture == "pilutar":
+        from .pilutar import PilutarModel
+
+        return PilutarModel(cfg, device, dtype, comm=comm)
     raise ValueError(f"unsupported architecture {cfg.architecture!r}")

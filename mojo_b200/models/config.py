@@ -10,10 +10,11 @@ from pathlib import Path
 @dataclass
 class RotarySpec:
     """Rotary embedding of one layer: the first `dims` dimensions of a head turn, the rest pass. `scaling` is the Llama-3.1
-    frequency rescale (factor, low, high, original) or None."""
+    frequency rescale (factor, low, high, original) or None. `interleaved`: neighbours pair up instead of halves."""
     dims: int = 0
     base: float = 10000.0
     scaling: dict | None = None
+    interleaved: bool = False
 
 
 @dataclass
@@ -25,12 +26,16 @@ class ExpertSpec:
 
 @dataclass
 class MoeSpec:
-    """Mixture of experts of one layer. The shared expert runs for every token."""
+    """Mixture of experts of one layer. The shared expert runs for every token. Experts (identity ones included) form `groups`
+    runs of neighbours, of which a token's choice keeps `keep`."""
     experts: int = 0
     top: int = 0
     scale: float = 1.0                     # on the router's weights
     expert: ExpertSpec = field(default_factory=ExpertSpec)
     shared: ExpertSpec | None = None
+    groups: int = 1
+    keep: int = 1
+    identity: int = 0                      # router outputs past the experts whose result is the input itself
 
 
 @dataclass
@@ -52,7 +57,7 @@ class BigramSpec:
 @dataclass
 class LayerSpec:
     """One layer of a decoder whose layers differ: which mixer it has, the mixer's sizes, and its feed-forward."""
-    mixer: str = "attention"               # "attention" | "channel_delta" | "latent_attention"
+    mixer: str = "attention"               # "attention" | "channel_delta" | "latent_attention" | "gated_linear" | "parallel"
     heads: int = 0
     kv_heads: int = 0
     dim: int = 0                           # query / key size of a head
@@ -66,11 +71,16 @@ class LayerSpec:
     gate_rank: int = 0
     kv_rank: int = 0                       # latent attention: size of the cached latent
     moe: MoeSpec | None = None             # mixture of experts in place of a dense feed-forward
+    window: int = 0                        # attention: positions a token sees, itself included (0: all before it)
+    softcap: float = 0.0                   # attention: scores become softcap * tanh(score / softcap) (0: they do not)
+    tau: float = 1.0                       # gated linear attention: decays are sigmoid(z)^(1 / tau)
+    parts: list["LayerSpec"] | None = None # "parallel": the mixers that run side by side ...
+    part_scales: list[float] | None = None # ... and the factors of their results
 
 
 @dataclass
 class ModelConfig:
-    architecture: str = "llama"            # "llama" | "deepseek_v2" | "rekudra" | "rerupel"
+    architecture: str = "llama"            # "llama" | "deepseek_v2" | "rekudra" | "rerupel" | "pilutar"
     hidden_size: int = 4096
     num_layers: int = 32
     num_heads: int = 32
@@ -107,6 +117,7 @@ class ModelConfig:
     loop: LoopSpec | None = None           # layers that run several times
     residual_mult: float = 1.0             # on everything a sublayer adds to the residual
     logit_softcap: float | None = None
+    logit_scale: float = 1.0
     extra: dict = field(default_factory=dict)
 
     def to_dict(self) -> dict:
@@ -128,7 +139,14 @@ class ModelConfig:
         body = [(i, i == lp.start) for i in range(lp.start, lp.stop)]
         return [(i, False) for i in range(lp.start)] + body * lp.times + [(i, False) for i in range(lp.stop, n)]
 
+    def mixers(self) -> list[LayerSpec]:
+        """Every mixer of a config that lists its layers; those that run side by side one by one."""
+        return [m for s in self.layers for m in (s.parts or [s])]
+
     def kv_bytes_per_token(self, dtype_bytes: int = 2, tp: int = 1) -> int:
+        if self.architecture == "pilutar":
+            return sum(s.kv_heads * (s.dim + s.vdim) if s.mixer == "attention" else s.kv_rank + s.rot.dims for s in self.mixers()
+                       if s.mixer != "gated_linear") * dtype_bytes
         if self.architecture == "rerupel":
             return sum(self.layers[i].kv_rank for i, _ in self.layer_runs()) * dtype_bytes
         if self.layers is not None:
@@ -146,6 +164,21 @@ class ModelConfig:
                 n += h * (s.heads * (s.dim + 2 * s.vdim) + s.kv_rank + 4) + s.heads * (s.dim + s.vdim) * s.kv_rank + 2 * h * s.ffn
                 if s.moe is not None:
                     n += h * (s.moe.experts + 3 * s.moe.experts * s.moe.expert.ffn + 3 * (s.moe.shared.ffn if s.moe.shared else 0))
+            return n
+        if self.architecture == "pilutar":
+            n = emb + 2 * h
+            for s in self.mixers():
+                out = s.heads * s.vdim
+                if s.mixer == "attention":
+                    n += h * (s.heads * s.dim + s.kv_heads * (s.dim + s.vdim) + out)
+                elif s.mixer == "latent_attention":
+                    n += h * (s.heads * (s.dim + s.rot.dims + 1) + s.kv_rank + s.rot.dims + out) + s.heads * (s.dim + s.vdim) * s.kv_rank
+                else:
+                    n += h * (2 * s.heads * s.dim + 3 * out + s.decay_rank) + s.heads * s.dim * s.decay_rank
+            for s in self.layers:
+                n += 2 * h + 3 * h * s.ffn
+                if s.moe is not None:
+                    n += h * (s.moe.experts + s.moe.identity + 2 * s.moe.experts * s.moe.expert.ffn + (2 * s.moe.shared.ffn + 1 if s.moe.shared else 0))
             return n
         if self.layers is not None:
             n = emb + h
@@ -205,6 +238,8 @@ class ModelConfig:
         """A config that lists its layers one by one (`layers[i]`: type, mixer sizes, feed-forward)."""
         if LAYERED_ARCHITECTURES[cfg["architecture"]] == "rerupel":
             return ModelConfig._from_latent_layers(cfg)
+        if LAYERED_ARCHITECTURES[cfg["architecture"]] == "pilutar":
+            return ModelConfig._from_parallel_layers(cfg)
         layers = []
         for i, entry in enumerate(cfg["layers"]):
             m, mlp = entry["mixer"], entry.get("mlp")
@@ -262,11 +297,70 @@ class ModelConfig:
                            logit_softcap=cfg.get("logit_softcap"), bigram=BigramSpec(bg["buckets"], bg["mul_prev"], bg["mul_cur"]) if bg else None,
                            loop=LoopSpec(lp["start"], lp["stop"], lp["times"]) if lp else None)
 
+    @staticmethod
+    def _from_parallel_layers(cfg: dict) -> "ModelConfig":
+        def window(m):
+            size = (m.get("mask") or {}).get("size") or 0
+            if size < 0:
+                raise ValueError(f"a window of {size} positions")
+            return size
+
+        def rotary(m, interleaved, dims=None):
+            rot = m.get("rot") or {}
+            spec = RotarySpec(rot.get("dims", 0) if dims is None else dims, rot.get("base", 10000.0), None, interleaved)
+            if spec.dims % 2 or rot.get("dims", spec.dims) != spec.dims or (dims is None and spec.dims > m["dim"]):
+                raise ValueError(f"rotary embedding of {rot.get('dims')} dimensions")
+            return spec
+
+        def mixer(kind, m):
+            if kind == "latent_attention":
+                return LayerSpec("latent_attention", m["heads"], 1, m["dim"], m["vdim"], scale=m["scale"], rot=rotary(m, True, m["rot_dim"]),
+                                 kv_rank=m["kv_rank"], window=window(m))
+            if kind != "parallel":
+                raise ValueError(f"unknown mixer {kind!r}")
+            a, b = m["left"], m["right"]
+            if a["heads"] % a["kv_heads"]:
+                raise ValueError(f"{a['heads']} query heads on {a['kv_heads']} key heads")
+            left = LayerSpec("attention", a["heads"], a["kv_heads"], a["dim"], a["vdim"], scale=a["scale"], rot=rotary(a, False), window=window(a),
+                             softcap=a.get("softcap") or 0.0)
+            right = LayerSpec("gated_linear", b["heads"], 0, b["dim"], b["vdim"], tau=b["tau"])
+            return LayerSpec("parallel", left.heads, left.kv_heads, left.dim, left.vdim, parts=[left, right],
+                             part_scales=[m.get("left_scale", 1.0), m.get("right_scale", 1.0)])
+
+        def feed_forward(spec, mlp):
+            if mlp is None:
+                return
+            if mlp.get("kind", "dense") == "dense":
+                spec.ffn = mlp["ff"]
+                return
+            if mlp["kind"] != "moe":
+                raise ValueError(f"unknown feed-forward {mlp['kind']!r}")
+            r, sh, g = mlp["router"], mlp.get("shared"), mlp["router"].get("groups") or {}
+            moe = spec.moe = MoeSpec(r["experts"], r["top"], 1.0, ExpertSpec(mlp["expert"]["ff"]), ExpertSpec(sh["ff"]) if sh else None,
+                                     g.get("count") or 1, g.get("keep") or 1, r.get("identity") or 0)
+            n = moe.experts + moe.identity
+            if n % moe.groups or not 1 <= moe.keep <= moe.groups or not 1 <= moe.top <= n // moe.groups * moe.keep:
+                raise ValueError(f"{moe.top} of {n} experts in {moe.groups} groups, {moe.keep} kept")
+
+        layers = []
+        for i, entry in enumerate(cfg["layers"]):
+            try:
+                spec = mixer(entry["type"], entry["mixer"])
+                feed_forward(spec, entry.get("mlp"))
+            except ValueError as e:
+                raise ValueError(f"layer {i}: {e}") from None
+            layers.append(spec)
+        first = layers[0]
+        return ModelConfig(architecture="pilutar", hidden_size=cfg["width"], num_layers=len(layers), num_heads=first.heads, num_kv_heads=first.kv_heads,
+                           head_dim=first.dim, intermediate_size=max(s.ffn for s in layers), vocab_size=cfg["vocab"], rms_norm_eps=cfg["norm"]["eps"],
+                           max_position_embeddings=0, layers=layers, embedding_scale=cfg.get("embedding", {}).get("scale", 1.0),
+                           logit_scale=cfg.get("logit_scale", 1.0))
+
 
 # `architecture` values of configs that list their layers -> model class key
-LAYERED_ARCHITECTURES = {"Rekudra": "rekudra", "Rerupel": "rerupel"}
+LAYERED_ARCHITECTURES = {"Rekudra": "rekudra", "Rerupel": "rerupel", "Pilutar": "pilutar"}
 # model classes that also run in f32 on CUDA (every operation has a true 32-bit kernel)
-F32_ARCHITECTURES = ("rekudra", "rerupel")
+F32_ARCHITECTURES = ("rekudra", "rerupel", "pilutar")
 
 
 def tiny_llama() -> ModelConfig:
@@ -359,6 +453,35 @@ def tiny_rerupel() -> ModelConfig:
     return rerupel(256, 3, 4, 64, 128, 512, 1024, 8, 2, 128, 192, (1, 3, 2))
 
 
+def pilutar(width: int, n_layers: int, heads: int, kv_heads: int, dim: int, kv_rank: int, rot_dim: int, ffn: int, vocab: int, experts: int, top: int,
+            expert_ffn: int, shared_ffn: int, window: int, groups: int = 1, keep: int = 1, identity: int = 0, latent_every: int = 4) -> ModelConfig:
+    """A Pilutar decoder: windowed attention beside gated linear attention, every `latent_every`-th layer latent attention
+    instead; one layer with a dense feed-forward, then layers with experts."""
+    moe = MoeSpec(experts, top, 1.0, ExpertSpec(expert_ffn), ExpertSpec(shared_ffn), groups, keep, identity)
+    layers = []
+    for i in range(n_layers):
+        if i % latent_every == latent_every - 1:
+            s = LayerSpec("latent_attention", heads, 1, dim - rot_dim, dim, scale=dim ** -0.5, rot=RotarySpec(rot_dim, 50000.0, None, True), kv_rank=kv_rank,
+                          window=window)
+        else:
+            left = LayerSpec("attention", heads, kv_heads, dim, dim, scale=dim ** -0.5, rot=RotarySpec(dim // 2, 10000.0), window=window, softcap=30.0)
+            right = LayerSpec("gated_linear", heads, 0, dim, dim, tau=16.0, decay_rank=16)
+            s = LayerSpec("parallel", heads, kv_heads, dim, dim, parts=[left, right], part_scales=[0.5, 0.5])
+        s.ffn, s.moe = (ffn, None) if i == 0 else (0, moe)
+        layers.append(s)
+    return ModelConfig(architecture="pilutar", hidden_size=width, num_layers=n_layers, num_heads=heads, num_kv_heads=kv_heads, head_dim=dim,
+                       intermediate_size=ffn, vocab_size=vocab, max_position_embeddings=0, layers=layers, embedding_scale=float(width) ** 0.5)
+
+
+def pilutar_lite() -> ModelConfig:
+    """Layers of the size of DeepSeek-V2-Lite's."""
+    return pilutar(2048, 24, 16, 4, 128, 512, 32, 10944, 102400, 62, 6, 1408, 2816, 1024, groups=8, keep=4, identity=2)
+
+
+def tiny_pilutar() -> ModelConfig:
+    return pilutar(256, 4, 4, 2, 64, 128, 32, 512, 1024, 7, 2, 128, 192, 48, groups=2, identity=1)
+
+
 PRESETS = {
     "tiny-llama": tiny_llama,
     "llama-3.1-8b": llama31_8b,
@@ -370,6 +493,8 @@ PRESETS = {
     "tiny-rekudra": tiny_rekudra,
     "rerupel-lite": rerupel_lite,
     "tiny-rerupel": tiny_rerupel,
+    "pilutar-lite": pilutar_lite,
+    "tiny-pilutar": tiny_pilutar,
 }
 
 

@@ -6,13 +6,15 @@ PyTorch fallback.
 """
 from __future__ import annotations
 
+from typing import NamedTuple
+
 import torch
 
 from .. import _ext
 from . import _state, autotune, reference
 from ._state import KernelError, check_status
 
-from .activation import SWIGLU, Glu
+from .activation import REGLU, SWIGLU, Glu  # noqa: F401
 
 EPI_NONE, EPI_ADD_RESIDUAL, EPI_SWIGLU, EPI_RELU2, EPI_SOFTCAP, EPI_F32 = 0, 1, 2, 3, 4, 5
 
@@ -239,15 +241,17 @@ def linear_swiglu(x: torch.Tensor, w_gu: torch.Tensor, out: torch.Tensor | None 
     """silu(x Wg^T) * (x Wu^T), or another gated linear unit, in one GEMM; `w_gu` is the 16-row interleaved stack from
     `reference.interleave_gate_up`."""
     if not x.is_cuda:
-        return reference.linear_swiglu_interleaved(x, w_gu, act=glu).to(x.dtype)
+        y = reference.linear_swiglu_interleaved(x, w_gu, act=glu).to(x.dtype)
+        return y if out is None else out.copy_(y)
     C = _ext.require()
     if x.dtype == torch.float32:
         gu = linear(x, w_gu)
         if out is None:
             out = torch.empty(x.shape[0], w_gu.shape[0] // 2, dtype=x.dtype, device=x.device)
-        C.glu_f32(gu, out, *glu)
+        to = out if out.is_contiguous() else torch.empty(out.shape, dtype=out.dtype, device=out.device)
+        C.glu_f32(gu, to, *glu)
         _count()
-        return out
+        return out if to is out else out.copy_(to)
     st = _state.get(x.device)
     if out is None:
         out = torch.empty(x.shape[0], w_gu.shape[0] // 2, dtype=x.dtype, device=x.device)
@@ -310,6 +314,14 @@ def gemm_config(swap: bool, bn: int, splits: int = 1, stream_k: bool = False) ->
     """Encode an explicit GEMM configuration (for tuning sweeps): operand swap, UMMA N, split-K factor, or
     stream-K balancing of the ragged last wave (excludes split-K)."""
     return (int(swap) << 30) | (int(stream_k) << 29) | ((1 if stream_k else splits) << 16) | bn
+
+
+class ScoreMods(NamedTuple):
+    """What an attention layer does beyond plain causal softmax. `window`: a row sees that many positions, its own included
+    (0: all); `softcap`: scores become softcap * tanh(score / softcap) (0: they do not); `out_scale`: factor of the result."""
+    window: int = 0
+    softcap: float = 0.0
+    out_scale: float = 1.0
 
 
 class AttnMeta:
@@ -407,7 +419,7 @@ def prefill_on_tensor_core(head_dim: int, page_size: int) -> bool:
     return bool(prefill_tensor_core and head_dim == 128 and page_size == 128)
 
 
-def _decode_attention(q, k_cache, v_cache, out, ctx_lens, block_tables, head_dim: int, scale: float, max_ctx: int, gate) -> None:
+def _decode_attention(q, k_cache, v_cache, out, ctx_lens, block_tables, head_dim: int, scale: float, max_ctx: int, gate, mods: ScoreMods) -> None:
     """One query row per sequence. More than 16 query heads per KV head (the rows of one MMA tile), or head size 256 in
     pages the TMA boxes do not fit, take the prefill kernel with chunks of one token."""
     C, st = _ext.require(), _state.get(q.device)
@@ -415,32 +427,36 @@ def _decode_attention(q, k_cache, v_cache, out, ctx_lens, block_tables, head_dim
     n = q.shape[0]
     if q.shape[1] // head_dim // n_kv > 16 or (head_dim == 256 and page % 32):
         cu = torch.arange(n + 1, dtype=torch.int32, device=q.device)
-        C.attn_prefill(q, k_cache, v_cache, out, cu, ctx_lens, block_tables, head_dim, 1, scale, st.status, gate)
+        C.attn_prefill(q, k_cache, v_cache, out, cu, ctx_lens, block_tables, head_dim, 1, scale, st.status, gate, *mods)
         _count()
         return
-    splits = _decode_splits(n, n_kv, max_ctx)
+    splits = _decode_splits(n, n_kv, min(max_ctx, mods.window) if mods.window else max_ctx)
     splits = max(1, min(splits, _state.ATTN_WORKSPACE_BYTES // (n * (q.shape[1] // head_dim) * (head_dim + 2) * 4)))
-    C.attn_decode(q, k_cache, v_cache, out, ctx_lens, block_tables, st.attn_ws, head_dim, splits, scale, st.status, st.attn_counters, gate)
+    C.attn_decode(q, k_cache, v_cache, out, ctx_lens, block_tables, st.attn_ws, head_dim, splits, scale, st.status, st.attn_counters, gate,
+                  *mods)
     _count(_decode_launches(splits, page))
 
 
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, meta: AttnMeta, scale: float,
                     head_dim: int, out: torch.Tensor | None = None, gate: torch.Tensor | None = None,
-                    positions: torch.Tensor | None = None) -> torch.Tensor:
-    """Causal GQA attention over the paged cache. q, out: [T, n_q * D]. `gate` [T, n_q]: head h of a row is multiplied by
-    sigmoid(gate[row, h]). f32 tensors (any head sizes; key and value sizes may differ) need `meta.seq` and `positions`."""
+                    positions: torch.Tensor | None = None, mods: ScoreMods = ScoreMods()) -> torch.Tensor:
+    """Causal GQA attention over the paged cache. q, out: [T, n_q * D] (rows of out may be strided). `gate` [T, n_q]: head h of a
+    row is multiplied by sigmoid(gate[row, h]). f32 tensors (any head sizes; key and value sizes may differ) need `meta.seq`
+    and `positions`."""
     if not q.is_cuda:
         T = q.shape[0]
         o = reference.paged_attention(q.reshape(T, -1, head_dim), k_cache, v_cache, meta.cu_q, meta.ctx_lens,
-                                      meta.block_tables, scale)
+                                      meta.block_tables, scale, mods.window, mods.softcap) * mods.out_scale
         if gate is not None:
             o = o * torch.sigmoid(gate.float()).unsqueeze(-1)
-        return o.reshape(T, -1).to(q.dtype)
+        o = o.reshape(T, -1).to(q.dtype)
+        return o if out is None else out.copy_(o)
     C = _ext.require()
     st = _state.get(q.device)
     if q.dtype == torch.float32:
-        out = torch.empty(q.shape[0], q.shape[1] // head_dim * v_cache.shape[3], dtype=q.dtype, device=q.device)
-        C.attn_f32(q, k_cache, v_cache, out, meta.seq.row_seq, positions, meta.block_tables, scale, gate, st.status)
+        if out is None:
+            out = torch.empty(q.shape[0], q.shape[1] // head_dim * v_cache.shape[3], dtype=q.dtype, device=q.device)
+        C.attn_f32(q, k_cache, v_cache, out, meta.seq.row_seq, positions, meta.block_tables, scale, gate, st.status, *mods)
         _count()
         return out
     if out is None:
@@ -450,29 +466,29 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         # captured step: fixed grids, everything that varies is read from device memory
         if sa.d_rows > 0:
             _decode_attention(q[:sa.d_rows], k_cache, v_cache, out[:sa.d_rows], sa.d_ctx, sa.d_bt, head_dim, scale, sa.max_ctx,
-                              gate[:sa.d_rows] if gate is not None else None)
+                              gate[:sa.d_rows] if gate is not None else None, mods)
         if sa.max_items > 0:
             C.attn_prefill_tc(q, k_cache, v_cache, out, sa.p_cu, sa.p_ctx, sa.p_bt, sa.max_q_len, scale, st.status,
-                              sa.work, sa.n_work, sa.max_items, gate)
+                              sa.work, sa.n_work, sa.max_items, gate, *mods)
             _count()
         return out
     nd, ns = meta.num_decode, meta.num_seqs
     if nd > 0:
         _decode_attention(q[:nd], k_cache, v_cache, out[:nd], meta.ctx_lens[:nd], meta.block_tables[:nd], head_dim, scale, meta.max_ctx,
-                          gate[:nd] if gate is not None else None)
+                          gate[:nd] if gate is not None else None, mods)
     if ns > nd:
         # cu_q offsets are absolute token rows, so q/out are passed whole
         if prefill_on_tensor_core(head_dim, k_cache.shape[2]):
             # tcgen05 / TMEM kernel: one KV tile = one 128-token page
             if meta.work is not None and meta.n_items > 0:
                 C.attn_prefill_tc(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:],
-                                  meta.max_q_len, scale, st.status, meta.work, None, meta.n_items, gate)
+                                  meta.max_q_len, scale, st.status, meta.work, None, meta.n_items, gate, *mods)
             else:
                 C.attn_prefill_tc(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:],
-                                  meta.max_q_len, scale, st.status, None, None, 0, gate)
+                                  meta.max_q_len, scale, st.status, None, None, 0, gate, *mods)
         else:
             C.attn_prefill(q, k_cache, v_cache, out, meta.cu_q[nd:], meta.ctx_lens[nd:], meta.block_tables[nd:], head_dim,
-                           meta.max_q_len, scale, st.status, gate)
+                           meta.max_q_len, scale, st.status, gate, *mods)
         _count()
     return out
 
@@ -552,6 +568,7 @@ def sample(logits: torch.Tensor, temperature: torch.Tensor, top_k: torch.Tensor,
     return ids
 
 
-from .latent import head_linear, latent_attend, latent_prefill, latent_write, plan_latent_prefill, token_rows  # noqa: E402,F401
-from .mixers import DeltaParams, Finished, HyperMix, SeqRows, StreamStart, conv_qkv, delta_rule, hyper_norm, residual_norm  # noqa: E402,F401
+from .latent import SharedRope, head_linear, latent_attend, latent_prefill, latent_write, plan_latent_prefill, token_rows  # noqa: E402,F401
+from .mixers import (DeltaParams, Finished, GatedLinearParams, HyperMix, QkvNorm, SeqRows, StreamStart, conv_qkv, delta_rule,  # noqa: E402,F401
+                     gated_linear, hyper_norm, norm_qkv, residual_norm)
 from .moe import ExpertRows, MoeWeights, moe_experts  # noqa: E402,F401

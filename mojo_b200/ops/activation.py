@@ -12,3 +12,5 @@ class Glu(NamedTuple):
 
 
 SWIGLU = Glu()
+# max(g, 0) * u: so steep a sigmoid is a step
+REGLU = Glu(alpha=1e30)

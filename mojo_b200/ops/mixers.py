@@ -1,5 +1,6 @@
 """Sequence mixing beyond plain attention: residuals in 32 bits (hyper-connections, that is several mixed streams, or one
-stream with a scale per channel), short causal convolutions in front of attention, and the gated delta rule. CUDA tensors (bf16, or f32 for the exact mode) go to the
+stream with a scale per channel), short causal convolutions or whole-row norms in front of attention, the gated delta rule and
+gated linear attention. CUDA tensors (bf16, or f32 for the exact mode) go to the
 sm_100a kernels, CPU tensors to `ops.reference`, as in the rest of `ops`."""
 from __future__ import annotations
 
@@ -76,18 +77,22 @@ class StreamStart:
 
 @dataclass
 class Finished:
-    """A sublayer's result on its way into the residual: rows `y`, or the weighted rows of every token's experts
-    (`ops.ExpertRows`), or both; `scale` f32 [width] is applied to their sum."""
-    scale: torch.Tensor
+    """Sublayers' results on their way into the residual, any of: rows `y`, the weighted rows of every token's experts
+    (`ops.ExpertRows`), rows `gated` times sigmoid(gate) with one f32 logit per row. `scale` f32 [width] is applied to their sum
+    (None: one)."""
+    scale: torch.Tensor | None
     y: torch.Tensor | None = None
     experts: object | None = None
+    gated: torch.Tensor | None = None
+    gate: torch.Tensor | None = None          # f32 [T], may be a column of a matrix
 
 
 def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, dtype: torch.dtype, done: Finished | None = None,
                   start: StreamStart | None = None, out: torch.Tensor | None = None, rows: torch.Tensor | None = None, store: bool = True,
-                  mean_width: int | None = None) -> torch.Tensor:
+                  mean_width: int | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
     """Everything between two sublayers in one launch: add the finished one to the stream x [T, width] (f32, in place) and
-    RMS-normalise the sum with `weight` (f32; None: return x itself, rounded). `start`: x begins from the embedding.
+    RMS-normalise the sum with `weight` (f32; None: return x itself, rounded), or layer-normalise it where there is a `bias`
+    (f32). `start`: x begins from the embedding.
     `rows`: only these rows, compact. `out`: where the result goes (rows may be strided)."""
     from . import _count
 
@@ -108,9 +113,14 @@ def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, dtyp
         if done is not None:
             add = torch.zeros(T, W) if y is None else y.float()
             if ex is not None:
-                add = add + torch.einsum("tk,tkw->tw", ex.weights, ex.rows.float()[ex.slot.long()])
+                e = ex.rows.float()[ex.slot.clamp_min(0).long()]
+                if ex.own is not None:
+                    e = torch.where((ex.slot < 0).unsqueeze(-1), ex.own.float().unsqueeze(1), e)
+                add = add + torch.einsum("tk,tkw->tw", ex.weights, e)
+            if done.gated is not None:
+                add = add + torch.sigmoid(done.gate.float()).unsqueeze(-1) * done.gated.float()
             add = add[pick]
-        h, new = reference.residual_norm(x[pick], weight, eps, add, done.scale if done is not None else None, mean_width)
+        h, new = reference.residual_norm(x[pick], weight, eps, add, done.scale if done is not None else None, mean_width, bias)
         if store:
             x.copy_(new)
         return h.to(dtype) if out is None else out.copy_(h)
@@ -120,7 +130,8 @@ def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, dtyp
     _ext.require().residual_norm(x, y, ex.rows if ex else None, ex.slot if ex else None, ex.weights if ex else None, done.scale if done else None, weight, out,
                                  s.ids if s else None, s.embed if s else None, s.scale if s else 1.0, s.prev if s and s.bigram is not None else None,
                                  s.bigram if s else None, s.mul_prev if s else 0, s.mul_cur if s else 0, s.x0 if s else None, rows, store, eps,
-                                 mean_width or W, _state.get(x.device).status)
+                                 mean_width or W, _state.get(x.device).status, bias, ex.own if ex else None, done.gated if done else None,
+                                 done.gate if done else None)
     _count()
     return out
 
@@ -152,6 +163,78 @@ def conv_qkv(proj: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor 
                             v_cache, heads, kv_heads, dim, vdim, eps, _state.get(proj.device).status)
     _count()
     return q
+
+
+@dataclass
+class QkvNorm:
+    """f32 parameters in front of attention: biases of the q | k | v columns, weights of the norms over a whole q and k row."""
+    bias: torch.Tensor
+    q_norm: torch.Tensor
+    k_norm: torch.Tensor
+
+
+def norm_qkv(proj: torch.Tensor, p: QkvNorm, cos_sin: torch.Tensor, positions: torch.Tensor, slots: torch.Tensor, k_cache: torch.Tensor,
+             v_cache: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, pad_dim: int, eps: float) -> torch.Tensor:
+    """Biases on the q | k | v columns of `proj`, one RMS norm over all of a row's q columns and one over its k columns, rotary
+    embedding (halves pair up) of the first columns of every head, k and v into the paged cache. Returns q [T, heads * pad_dim]
+    (zeros past `dim`)."""
+    from . import _count
+
+    T, nq, nk = proj.shape[0], heads * dim, kv_heads * dim
+    if not proj.is_cuda:
+        u = proj[:, :nq + nk + kv_heads * vdim].float() + p.bias
+
+        def whole(z, w, n):
+            z = (z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps) * w).reshape(T, n, dim)
+            return reference.apply_rope(z, positions, cos_sin) if cos_sin.shape[1] else z
+
+        reference.write_kv(k_cache, v_cache, whole(u[:, nq:nq + nk], p.k_norm, kv_heads), u[:, nq + nk:].reshape(T, kv_heads, vdim), slots)
+        return whole(u[:, :nq], p.q_norm, heads).reshape(T, nq).to(proj.dtype)
+    q = torch.empty(T, heads * pad_dim, dtype=proj.dtype, device=proj.device)
+    _ext.require().norm_qkv(proj, p.bias, p.q_norm, p.k_norm, cos_sin, positions, slots, k_cache, v_cache, q, heads, kv_heads, dim, vdim, eps,
+                            _state.get(proj.device).status)
+    _count()
+    return q
+
+
+@dataclass
+class GatedLinearParams:
+    """f32 parameters of gated linear attention: bias of the decay logits [heads * dim], output norm [vdim]; decays are
+    sigmoid(z)^(1 / tau)."""
+    decay_bias: torch.Tensor
+    norm_w: torch.Tensor
+    tau: float
+
+
+def gated_linear(proj: torch.Tensor, z: torch.Tensor, p: GatedLinearParams, state: torch.Tensor, seq: SeqRows, heads: int, dim: int, vdim: int, eps: float,
+                 out: torch.Tensor, out_scale: float = 1.0) -> torch.Tensor:
+    """Gated linear attention over a step's sequences: S <- diag(a) S + k v^T, o = S^T q dim^-0.5, o normalised per head, times
+    silu(gate) and `out_scale`. proj [T, q | k | v | gate], z f32 [T, heads * dim] (decay logits without their bias), `state` f32
+    [slots, heads, dim, vdim], updated in place. Writes and returns out [T, heads * vdim] (rows may be strided)."""
+    from . import _count
+
+    T, nk, nv = proj.shape[0], heads * dim, heads * vdim
+    if not proj.is_cuda:
+        q, k = proj[:, :nk].float().reshape(T, heads, dim) * dim ** -0.5, proj[:, nk:2 * nk].float().reshape(T, heads, dim)
+        v, g = proj[:, 2 * nk:2 * nk + nv].float().reshape(T, heads, vdim), proj[:, 2 * nk + nv:2 * (nk + nv)].float()
+        a = torch.exp(torch.nn.functional.logsigmoid(z[:, :nk].float() + p.decay_bias) / p.tau).reshape(T, heads, dim)
+        out.zero_()
+        for (b, e), (rd, wr) in zip(seq.seq_rows.tolist(), seq.seq_state.tolist()):
+            if wr < 0 or e <= b:
+                continue
+            S = state[wr // 2]
+            if rd < 0:
+                S.zero_()
+            o = reference.gated_linear(q[b:e], k[b:e], v[b:e], a[b:e], S)
+            o = (o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * p.norm_w).reshape(e - b, nv)
+            out[b:e] = (o * reference.silu(g[b:e]) * out_scale).to(out.dtype)
+        return out
+    C, st = _ext.require(), _state.get(proj.device)
+    scratch = torch.empty(C.gated_linear_scratch_floats(heads, dim, vdim, T) if seq.n_prefill else 0, dtype=torch.float32, device=proj.device)
+    C.gated_linear(proj, z, p.decay_bias, p.norm_w, p.tau, state, seq.row_seq, seq.seq_rows, seq.seq_state, out, scratch, heads, dim, vdim, eps, out_scale,
+                   seq.n_decode, seq.first, seq.n_prefill, st.status)
+    _count((1 if seq.n_decode else 0) + (3 if seq.n_prefill else 0))
+    return out
 
 
 @dataclass

@@ -16,9 +16,11 @@ SCORING = {"softmax": 0, "sigmoid": 1}
 
 @dataclass
 class MoeWeights:
-    """router [>= experts, width] (rows past `experts` are padding), w_gu [experts, 2 ffn, width] (gate and up rows
-    interleaved in blocks of 16), w_down [experts, width, ffn]. A token uses the `top` experts of the largest scores, with
-    their scores (over their sum if `norm_top`) times `scale` as weights."""
+    """router [>= experts + identity, width] (rows past those are not looked at here), w_gu [experts, 2 ffn, width] (gate and up
+    rows interleaved in blocks of 16; with `glu` None, squared-ReLU experts, [experts, ffn, width]), w_down [experts, width,
+    ffn]. A token uses the `top` experts of the largest scores, with their scores (over their sum if `norm_top`) times `scale`
+    as weights. `correction` f32 [experts + identity] is added to the scores for the choice alone; the choice is among the
+    `keep` of `groups` groups of neighbours with the largest scores in them. The last `identity` experts return their input."""
     router: torch.Tensor
     w_gu: torch.Tensor
     w_down: torch.Tensor
@@ -27,15 +29,21 @@ class MoeWeights:
     scoring: str = "softmax"
     norm_top: bool = False
     scale: float = 1.0
-    glu: Glu = SWIGLU
+    glu: Glu | None = SWIGLU
+    correction: torch.Tensor | None = None
+    groups: int = 1
+    keep: int = 1
+    identity: int = 0
 
 
 @dataclass
 class ExpertRows:
-    """Results of a token's experts: rows[slot[t, j]] times weights[t, j], summed over j."""
+    """Results of a token's experts: rows[slot[t, j]] times weights[t, j], summed over j. A slot of -1 stands for the token's own
+    input row, `own[t]`."""
     rows: torch.Tensor
     slot: torch.Tensor          # int32 [T, top]
     weights: torch.Tensor       # f32 [T, top]
+    own: torch.Tensor | None = None
 
 
 def tile_rows(rows_per_expert: float) -> int:
@@ -43,38 +51,50 @@ def tile_rows(rows_per_expert: float) -> int:
     return next((n for n in (16, 32, 64, 128) if rows_per_expert * 1.25 <= n), 256)
 
 
-def moe_experts(h: torch.Tensor, p: MoeWeights) -> ExpertRows:
-    """Run every row of h [T, width] through its experts."""
-    from . import EPI_NONE, EPI_SWIGLU, _count, linear_f32
+def moe_experts(h: torch.Tensor, p: MoeWeights, logits: torch.Tensor | None = None) -> ExpertRows:
+    """Run every row of h [T, width] through its experts. `logits`: the router's, f32, where the caller has them already."""
+    from . import EPI_NONE, EPI_RELU2, EPI_SWIGLU, _count, linear_f32
 
     T, W = h.shape
-    logits = linear_f32(h, p.router)
+    if logits is None:
+        logits = linear_f32(h, p.router)
+    own = h if p.identity else None
+    n_out = p.experts + p.identity
     if not h.is_cuda:
-        weights, ids = reference.moe_route(logits[:, :p.experts], p.top, p.norm_top, p.scale, sigmoid=p.scoring == "sigmoid")
-        rows = torch.empty(T, p.top, W, dtype=h.dtype)
+        weights, ids = reference.moe_route(logits[:, :n_out], p.top, p.norm_top, p.scale, p.scoring == "sigmoid", p.correction, p.groups, p.keep)
+        rows = torch.zeros(T, p.top, W, dtype=h.dtype)
         for e in range(p.experts):
             tok, j = torch.where(ids == e)
             if tok.numel():
-                rows[tok, j] = reference.linear(reference.linear_swiglu_interleaved(h[tok], p.w_gu[e], act=p.glu).to(h.dtype), p.w_down[e]).to(h.dtype)
-        return ExpertRows(rows.view(T * p.top, W), torch.arange(T * p.top, dtype=torch.int32).view(T, p.top), weights.float())
+                if p.glu is None:
+                    act = reference.linear(h[tok], p.w_gu[e]).clamp_min(0.0).square()
+                else:
+                    act = reference.linear_swiglu_interleaved(h[tok], p.w_gu[e], act=p.glu)
+                rows[tok, j] = reference.linear(act.to(h.dtype), p.w_down[e]).to(h.dtype)
+        slot = torch.where(ids < p.experts, torch.arange(T * p.top).view(T, p.top), -1).int()
+        return ExpertRows(rows.view(T * p.top, W), slot, weights.float(), own)
     C, st = _ext.require(), _state.get(h.device)
     dev, R, f32 = h.device, T * p.top, h.dtype == torch.float32
-    bn = 64 if f32 else tile_rows(R / p.experts)
+    bn = 64 if f32 else tile_rows(R / n_out)
     weights = torch.empty(T, p.top, dtype=torch.float32, device=dev)
     ids, place, slot = (torch.empty(T, p.top, dtype=torch.int32, device=dev) for _ in range(3))
     counts = st.moe_counts
-    C.moe_route(logits, weights, ids, place, counts, p.experts, SCORING[p.scoring], p.norm_top, p.scale)
+    C.moe_route(logits, weights, ids, place, counts, p.experts, SCORING[p.scoring], p.norm_top, p.scale, p.correction, p.groups, p.keep, p.identity)
     xs = torch.empty(R, W, dtype=h.dtype, device=dev)
     tiles, n_tiles = torch.empty(p.experts + R // bn, 4, dtype=torch.int32, device=dev), torch.empty(1, dtype=torch.int32, device=dev)
     C.moe_gather(h, ids, place, counts, slot, xs, tiles, n_tiles, p.experts, bn, st.status)
     f = p.w_down.shape[2]
     act, y = torch.empty(R, f, dtype=h.dtype, device=dev), torch.empty(R, W, dtype=h.dtype, device=dev)
-    if f32:
+    launches = 4
+    if p.glu is None:
+        C.moe_tiles_gemm(xs, p.w_gu, tiles, n_tiles, act, EPI_RELU2, bn, None, st.status)
+    elif f32:
         gu = torch.empty(R, 2 * f, dtype=h.dtype, device=dev)
         C.moe_tiles_gemm(xs, p.w_gu, tiles, n_tiles, gu, EPI_NONE, bn, None, st.status)
         C.glu_f32(gu, act, *p.glu)
+        launches = 5
     else:
         C.moe_tiles_gemm(xs, p.w_gu, tiles, n_tiles, act, EPI_SWIGLU, bn, (*p.glu, 0.0), st.status)
     C.moe_tiles_gemm(act, p.w_down, tiles, n_tiles, y, EPI_NONE, bn, None, st.status)
-    _count(5 if f32 else 4)
-    return ExpertRows(y, slot, weights)
+    _count(launches)
+    return ExpertRows(y, slot, weights, own)

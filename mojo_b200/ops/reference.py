@@ -114,9 +114,16 @@ def gather_kv(cache: torch.Tensor, block_table: torch.Tensor, ctx_len: int) -> t
     return pages.permute(0, 2, 1, 3).reshape(n_pages * page_size, cache.shape[1], cache.shape[3])[:ctx_len]
 
 
+def visible(ctx: int, q_len: int, window: int = 0, device="cpu") -> torch.Tensor:
+    """Which of `ctx` positions the last `q_len` of them see: [q_len, ctx]."""
+    gap = torch.arange(ctx - q_len, ctx, device=device).unsqueeze(1) - torch.arange(ctx, device=device).unsqueeze(0)
+    return (gap >= 0) & (gap < (window or ctx))
+
+
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_q: torch.Tensor, ctx_lens: torch.Tensor,
-                    block_tables: torch.Tensor, scale: float) -> torch.Tensor:
-    """Causal GQA attention for a ragged batch of query chunks. q: [T, n_q, D] -> [T, n_q, D] fp32.
+                    block_tables: torch.Tensor, scale: float, window: int = 0, softcap: float = 0.0) -> torch.Tensor:
+    """Causal GQA attention for a ragged batch of query chunks. q: [T, n_q, D] -> [T, n_q, D] fp32. `window`: a row sees that
+    many positions, its own included (0: all); `softcap`: scores become softcap * tanh(score / softcap) (0: they do not).
 
     Sequence b owns query rows cu_q[b]:cu_q[b+1]; these are the last q_len positions of a context of ctx_lens[b]
     tokens whose keys/values are all in the cache already.
@@ -136,9 +143,9 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         v = v.repeat_interleave(group, dim=1)
         qq = q[s:e].float()  # [ql, n_q, D]
         scores = torch.einsum("qhd,khd->hqk", qq, k) * scale
-        qpos = torch.arange(ctx - ql, ctx, device=q.device).unsqueeze(1)
-        kpos = torch.arange(ctx, device=q.device).unsqueeze(0)
-        scores = scores.masked_fill(~(kpos <= qpos).unsqueeze(0), float("-inf"))
+        if softcap:
+            scores = softcap * torch.tanh(scores / softcap)
+        scores = scores.masked_fill(~visible(ctx, ql, window, q.device).unsqueeze(0), float("-inf"))
         p = torch.softmax(scores, dim=-1)
         out[s:e] = torch.einsum("hqk,khd->qhd", p, v)
     return out
@@ -298,13 +305,17 @@ def hyper_norm(x: torch.Tensor, weight: torch.Tensor, eps: float, w_in=None, y=N
     return u * torch.rsqrt(ms + eps) * weight, x
 
 
-def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, y=None, y_scale=None, mean_width: int | None = None):
+def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, y=None, y_scale=None, mean_width: int | None = None, bias=None):
     """x [rows, width] f32, y what a finished sublayer adds (before its scale). Returns (normed rows, or x itself without a
-    weight; new stream)."""
+    weight; new stream). With `bias` the norm is a layer norm."""
     if y is not None:
-        x = x + y_scale * y.float()
+        x = x + (y.float() if y_scale is None else y_scale * y.float())
     if weight is None:
         return x, x
+    if bias is not None:
+        n = mean_width or x.shape[-1]
+        d = x - x[..., :n].mean(-1, keepdim=True)
+        return d * torch.rsqrt(d[..., :n].pow(2).mean(-1, keepdim=True) + eps) * weight + bias, x
     ms = x.pow(2).sum(-1, keepdim=True) / (mean_width or x.shape[-1])
     return x * torch.rsqrt(ms + eps) * weight, x
 
@@ -340,6 +351,16 @@ def delta_rule(q, k, v, g, beta, S):
     return o
 
 
+def gated_linear(q, k, v, a, S):
+    """One sequence: q, k, a [T, H, d], v [T, H, e], S [H, d, e] (updated in place): S <- a S + k v^T, o = S^T q. Returns o
+    [T, H, e]."""
+    o = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        S.mul_(a[t].unsqueeze(-1)).add_(k[t].unsqueeze(-1) * v[t].unsqueeze(1))
+        o[t] = torch.einsum("hde,hd->he", S, q[t])
+    return o
+
+
 # ------------------------------------------------------------------------------------------------------
 # MLA (multi-head latent attention), absorbed form
 # ------------------------------------------------------------------------------------------------------
@@ -364,10 +385,10 @@ def mla_decode(q_lat: torch.Tensor, q_rope: torch.Tensor, kv_cache: torch.Tensor
 
 
 def mla_attend(q_lat: torch.Tensor, q_rope: torch.Tensor, kv_cache: torch.Tensor, cu_q: torch.Tensor, ctx_lens: torch.Tensor,
-               block_tables: torch.Tensor, scale: float) -> torch.Tensor:
+               block_tables: torch.Tensor, scale: float, window: int = 0) -> torch.Tensor:
     """Absorbed latent attention for a mixed batch: q_lat [T, H, R], q_rope [T, H, P] hold the query tokens of every
     sequence back to back (`cu_q` offsets); token i of a chunk of q_len tokens sees the first ctx - q_len + i + 1 cache
-    positions of its sequence. Returns [T, H, R] in latent space."""
+    positions of its sequence, or the last `window` of those. Returns [T, H, R] in latent space."""
     T, H, R = q_lat.shape
     page_size = kv_cache.shape[1]
     out = torch.zeros(T, H, R, dtype=torch.float32, device=q_lat.device)
@@ -380,9 +401,7 @@ def mla_attend(q_lat: torch.Tensor, q_rope: torch.Tensor, kv_cache: torch.Tensor
         kv = kv_cache[block_tables[b, :n_pages].long()].reshape(n_pages * page_size, -1)[:ctx].float()
         lat, rope = kv[:, :R], kv[:, R:]
         s = (torch.einsum("qhr,kr->hqk", q_lat[s0:e0].float(), lat) + torch.einsum("qhp,kp->hqk", q_rope[s0:e0].float(), rope)) * scale
-        qpos = torch.arange(ctx - (e0 - s0), ctx, device=s.device).unsqueeze(1)
-        kpos = torch.arange(ctx, device=s.device).unsqueeze(0)
-        s = s.masked_fill(~(kpos <= qpos).unsqueeze(0), float("-inf"))
+        s = s.masked_fill(~visible(ctx, e0 - s0, window, s.device).unsqueeze(0), float("-inf"))
         out[s0:e0] = torch.einsum("hqk,kr->qhr", torch.softmax(s, dim=-1), lat)
     return out
 
@@ -392,13 +411,22 @@ def mla_attend(q_lat: torch.Tensor, q_rope: torch.Tensor, kv_cache: torch.Tensor
 # ------------------------------------------------------------------------------------------------------
 
 
-def moe_route(router_logits: torch.Tensor, top_k: int, norm_topk: bool = False, scale: float = 1.0, sigmoid: bool = False):
-    """Softmax over all experts (DeepSeek-V2 'greedy' routing), or the sigmoid of each score alone, then top-k. Returns
-    (weights [T, k], ids [T, k])."""
+def moe_route(router_logits: torch.Tensor, top_k: int, norm_topk: bool = False, scale: float = 1.0, sigmoid: bool = False, correction=None,
+              groups: int = 1, keep: int = 1):
+    """Softmax over all experts (DeepSeek-V2 'greedy' routing), or the sigmoid of each score alone, then top-k. `correction` is
+    added to the scores for the choice only; with `groups` > 1 the choice is among the `keep` groups of neighbours that hold
+    the largest such scores. Returns (weights [T, k], ids [T, k])."""
     p = torch.sigmoid(router_logits.float()) if sigmoid else torch.softmax(router_logits.float(), dim=-1)
-    w, idx = torch.topk(p, top_k, dim=-1)
+    c = p if correction is None else p + correction.float()
+    if keep < groups:
+        per = c.shape[1] // groups
+        best = c.view(-1, groups, per).amax(-1).topk(keep, dim=-1).indices
+        out = torch.ones(c.shape[0], groups, dtype=torch.bool, device=c.device).scatter(1, best, False)
+        c = c.masked_fill(out.repeat_interleave(per, dim=1), float("-inf"))
+    idx = torch.topk(c, top_k, dim=-1).indices
+    w = p.gather(1, idx)
     if norm_topk:
-        w = w / w.sum(dim=-1, keepdim=True)
+        w = w / (w.sum(dim=-1, keepdim=True) + 1e-20)
     return w * scale, idx
 
 
