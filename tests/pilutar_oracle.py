@@ -160,6 +160,13 @@ def choice_scores(s, correction, groups, keep):
     return c.masked_fill(~stays.repeat_interleave(c.shape[1] // groups, dim=1), -math.inf)
 
 
+def margins(choice, s, n):
+    """By how much the n-th best choice leads the next, in units of the two scores (which is what rounding disturbs)."""
+    order = choice.argsort(dim=1, descending=True)
+    a, b = order[:, n - 1:n], order[:, n:n + 1]
+    return ((choice.gather(1, a) - choice.gather(1, b)) / (s.gather(1, a) + s.gather(1, b))).flatten()
+
+
 def route(z, correction, r, gaps=None):
     """Weights [T, E + identity], zero for what a token does not use. `gaps` receives by how much every choice was made."""
     g = r.get("groups") or {"count": 1, "keep": 1}
@@ -167,12 +174,11 @@ def route(z, correction, r, gaps=None):
     s = s / s.sum(1, keepdim=True)
     c = choice_scores(s, correction, g["count"], g["keep"])
     if gaps is not None:
-        best = c.sort(dim=1, descending=True).values
-        if r["top"] < best.shape[1]:
-            gaps.append(best[:, r["top"] - 1] - best[:, r["top"]])
-        per = (s + correction).view(len(s), g["count"], -1).max(-1).values.sort(dim=1, descending=True).values
+        if r["top"] < int(torch.isfinite(c[0]).sum()):
+            gaps.append(margins(c, s, r["top"]))
         if g["keep"] < g["count"]:
-            gaps.append(per[:, g["keep"] - 1] - per[:, g["keep"]])
+            best = (s + correction).view(len(s), g["count"], -1).max(-1)
+            gaps.append(margins(best.values, s.view(len(s), g["count"], -1).gather(2, best.indices[..., None])[..., 0], g["keep"]))
     chosen = c.topk(r["top"], dim=1).indices
     picked = s.gather(1, chosen)
     return torch.zeros_like(s).scatter(1, chosen, picked / (picked.sum(1, keepdim=True) + 1e-20))
@@ -295,8 +301,8 @@ def layer_tensors(spec, width, rank_a):
 def random_weights(cfg, seed=0, sharp=1.0, rank_a=6):
     """Checkpoint tensors by name, rounded to bfloat16 values (held in float32). `sharp` scales the queries, so that single
     scores stand out. Routers mostly look at one channel per expert, where every token's embedding has the same levels in an
-    order of its own and the layers add little: choices vary with the token and are no close calls, which rounding could
-    decide either way."""
+    order of its own and the layers add little, the other channels only differ in sign, and corrections differ by nothing or by more than scores can:
+    choices vary with the token and are no close calls, which rounding could decide either way."""
     g = torch.Generator().manual_seed(seed)
 
     def rnd(*shape, std):
@@ -307,7 +313,8 @@ def random_weights(cfg, seed=0, sharp=1.0, rank_a=6):
     C = max([s["mlp"]["router"]["experts"] + s["mlp"]["router"].get("identity", 0) for s in cfg["layers"] if s["mlp"] and s["mlp"]["kind"] == "moe"], default=0)
     assert C <= W // 2
     if C > 1:
-        levels = torch.linspace(-6.0, 6.0, C) / cfg["embedding"]["scale"]
+        levels = torch.linspace(-3.0, 3.0, C) / cfg["embedding"]["scale"]
+        w["embed"] = w["embed"].sign() * 0.5
         w["embed"][:, :C] = torch.stack([levels[torch.randperm(C, generator=g)] for _ in range(cfg["vocab"])])
     for i, spec in enumerate(cfg["layers"]):
         for name, (shape, kind) in layer_tensors(spec, W, rank_a).items():
@@ -319,11 +326,11 @@ def random_weights(cfg, seed=0, sharp=1.0, rank_a=6):
             elif kind == "decay_bias":
                 w[full] = rnd(*shape, std=2.0)
             elif kind == "correction":
-                w[full] = rnd(*shape, std=0.05) - 0.1
+                w[full] = torch.randint(-1, 2, shape, generator=g) * 1.5 - 0.2
             elif kind == "router":
                 E = shape[0]
                 w[full] = rnd(*shape, std=0.03 * W ** -0.5)
-                w[full][:, :E] += torch.eye(E)[torch.randperm(E, generator=g)] * 1.5
+                w[full][:, :E] += torch.eye(E)[torch.randperm(E, generator=g)] * 0.2 * max(E, 4)
             else:
                 w[full] = rnd(*shape, std=(sharp if kind == "sharp" else 1.0) * shape[-1] ** -0.5)
             if C > 1 and name in ("norm1", "norm1.b"):
