@@ -378,7 +378,7 @@ void gated_linear(const at::Tensor& proj, const at::Tensor& z, const at::Tensor&
   a.eps = static_cast<float>(eps);
   a.out_scale = static_cast<float>(out_scale);
   if (n_prefill > 0) {
-    need(is_f32(scratch, b2_gated_linear_scratch_floats(a.heads, a.dim, a.vdim, s.rows)), "gated_linear: f32 scratch of gated_linear_scratch_floats elements");
+    need(is_f32(scratch, b2_gated_linear_scratch_floats(a.heads, a.dim, a.vdim, s.rows, s.seqs, static_cast<int>(n_prefill))), "gated_linear: f32 scratch of gated_linear_scratch_floats elements");
     a.scratch = scratch.data_ptr<float>();
   }
   c10::cuda::CUDAGuard g(proj.device());
@@ -396,8 +396,12 @@ void bind_mixers(py::module_& m) {
   });
   m.def("norm_qkv", &norm_qkv);
   m.def("gated_linear", &gated_linear);
-  m.def("gated_linear_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows) {
-    return b2_gated_linear_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows));
+  m.def("gated_linear_scratch_floats", [](int64_t heads, int64_t dim, int64_t vdim, int64_t rows, int64_t all_seqs, int64_t seqs) {
+    return b2_gated_linear_scratch_floats(static_cast<int>(heads), static_cast<int>(dim), static_cast<int>(vdim), static_cast<int>(rows),
+                                          static_cast<int>(all_seqs), static_cast<int>(seqs));
+  });
+  m.def("gated_linear_prefill_launches", [](int64_t heads, int64_t vdim, int64_t rows, int64_t seqs) {
+    return b2_gated_linear_prefill_launches(static_cast<int>(heads), static_cast<int>(vdim), static_cast<int>(rows), static_cast<int>(seqs));
   });
   m.def("residual_norm", &residual_norm, py::arg("x"), py::arg("y"), py::arg("experts"), py::arg("slot"), py::arg("expert_w"), py::arg("y_scale"),
         py::arg("weight"), py::arg("h"), py::arg("ids"), py::arg("embed"), py::arg("embed_scale"), py::arg("prev"), py::arg("bigram"), py::arg("mul_prev"),

@@ -44,6 +44,19 @@ __device__ __forceinline__ void store_f32(__nv_bfloat16* p, const float (&v)[N])
 }
 
 __device__ __forceinline__ float sigmoid_f32(float x) { return 1.0f / (1.0f + expf(-x)); }
+// The same by the special-function unit: log(1 + e^x), for small t = e^-|x| by the series of log1p, which keeps the relative
+// precision of slow decays.
+__device__ __forceinline__ float softplus_fast(float x) {
+  const float t = ptx::ex2(-fabsf(x) * ptx::kLog2e);
+  float s = fmaf(t, -1.0f / 8, 1.0f / 7);
+  s = fmaf(t, s, -1.0f / 6);
+  s = fmaf(t, s, 1.0f / 5);
+  s = fmaf(t, s, -1.0f / 4);
+  s = fmaf(t, s, 1.0f / 3);
+  s = fmaf(t, s, -1.0f / 2);
+  s = fmaf(t * t, s, t);
+  return fmaxf(x, 0.0f) + (t < 0.125f ? s : ptx::lg2(1.0f + t) * ptx::kLn2);
+}
 __device__ __forceinline__ float softplus_f32(float x) { return fmaxf(x, 0.0f) + log1pf(expf(-fabsf(x))); }
 
 }  // namespace b2

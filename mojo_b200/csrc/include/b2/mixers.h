@@ -131,13 +131,14 @@ struct B2GatedLinearArgs {
   const float* decay_bias;    // [heads * dim]
   const float* norm_w;        // [vdim]
   float* state;
-  float* scratch;             // b2_gated_linear_scratch_floats floats: prepared rows and raw outputs of the scan
+  float* scratch;             // b2_gated_linear_scratch_floats floats (prompt chunks only)
   void* out;                  // [rows, ld_out], heads * vdim columns
   int64_t ld_out;
   int32_t heads, dim, vdim;
   float inv_tau, eps, out_scale;
 };
-int64_t b2_gated_linear_scratch_floats(int heads, int dim, int vdim, int rows);
+int64_t b2_gated_linear_scratch_floats(int heads, int dim, int vdim, int rows, int all_seqs, int seqs);      // seqs: those with chunks
+int b2_gated_linear_prefill_launches(int heads, int vdim, int rows, int seqs);
 // Sequences as for the delta rule below: [0, n_decode) have one row each, [first, first + n_prefill) any number.
 int b2_gated_linear(const B2GatedLinearArgs* a, const B2SeqRows* s, int n_decode, int first, int n_prefill, int f32, b2::Status* status,
                     cudaStream_t stream);

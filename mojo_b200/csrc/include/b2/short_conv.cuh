@@ -96,6 +96,15 @@ struct RawVec<__nv_bfloat16, 4> {
   }
 };
 
+template <>
+struct RawVec<__nv_bfloat16, 2> {
+  uint32_t v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint32_t*>(p); }
+  __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint32_t*>(p) = v; }
+  __device__ __forceinline__ void zero() { v = 0; }
+  __device__ __forceinline__ float get(int i) const { return i & 1 ? ptx::bf16_hi(v) : ptx::bf16_lo(v); }
+};
+
 // The convolution of `n` (<= TT) consecutive rows of one sequence for VEC channels: the whole window is fetched at once, so
 // that its loads are in flight together, and every row is fetched once. `save` also writes the next step's bank.
 // TAPS == 0: any number of taps, row by row.

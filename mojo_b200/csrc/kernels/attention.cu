@@ -130,6 +130,7 @@ __device__ __forceinline__ void warp_attend(const uint32_t (&qf)[D / 16][4], uin
       mma_bf16(s[2 * jp + 1], qf[kk], b2, b3);
     }
   }
+  if constexpr (MODS) mods.scores<NT_S * 4>(&s[0][0], scale_log2);
   // mask + running max
   const int t = lane & 3;
   float mx_lo = m[0], mx_hi = m[1];
@@ -138,10 +139,10 @@ __device__ __forceinline__ void warp_attend(const uint32_t (&qf)[D / 16][4], uin
     const int col = kv0 + j * 8 + 2 * t;
     if constexpr (MODS) {
       const int lo = max_lo - mods.window, hi = max_hi - mods.window;
-      s[j][0] = col <= max_lo && col > lo ? mods.score(s[j][0], scale_log2) : -INFINITY;
-      s[j][1] = col + 1 <= max_lo && col + 1 > lo ? mods.score(s[j][1], scale_log2) : -INFINITY;
-      s[j][2] = col <= max_hi && col > hi ? mods.score(s[j][2], scale_log2) : -INFINITY;
-      s[j][3] = col + 1 <= max_hi && col + 1 > hi ? mods.score(s[j][3], scale_log2) : -INFINITY;
+      s[j][0] = col <= max_lo && col > lo ? s[j][0] : -INFINITY;
+      s[j][1] = col + 1 <= max_lo && col + 1 > lo ? s[j][1] : -INFINITY;
+      s[j][2] = col <= max_hi && col > hi ? s[j][2] : -INFINITY;
+      s[j][3] = col + 1 <= max_hi && col + 1 > hi ? s[j][3] : -INFINITY;
     } else {
       s[j][0] = col <= max_lo ? s[j][0] * scale_log2 : -INFINITY;
       s[j][1] = col + 1 <= max_lo ? s[j][1] * scale_log2 : -INFINITY;

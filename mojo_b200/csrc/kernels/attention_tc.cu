@@ -327,8 +327,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       }
       const int kv0 = (first_tile + j) * kTile + g * 64;
       if constexpr (MODS) {
-#pragma unroll
-        for (int c = 0; c < 64; ++c) s[c] = prm.mods.score(s[c], prm.scale_log2);
+        prm.mods.scores<64>(s, prm.scale_log2);
         if (kv0 <= pos0 + kTile - 1 - prm.mods.window) {   // some row of this tile is past some of these columns
           const int lo = qpos - prm.mods.window;
 #pragma unroll

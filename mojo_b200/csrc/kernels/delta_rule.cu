@@ -29,18 +29,6 @@ constexpr int kTile = 8;         // pairs of one shared-memory stage of the scan
 constexpr int kStages = 3;
 constexpr int kCols = 32;        // value columns of a scan CTA
 
-// log(1 + e^x): for small t = e^-|x| by the series of log1p, which keeps the relative precision of slow decays.
-__device__ __forceinline__ float softplus(float x) {
-  const float t = ptx::ex2(-fabsf(x) * ptx::kLog2e);
-  float s = fmaf(t, -1.0f / 8, 1.0f / 7);
-  s = fmaf(t, s, -1.0f / 6);
-  s = fmaf(t, s, 1.0f / 5);
-  s = fmaf(t, s, -1.0f / 4);
-  s = fmaf(t, s, 1.0f / 3);
-  s = fmaf(t, s, -1.0f / 2);
-  s = fmaf(t * t, s, t);
-  return fmaxf(x, 0.0f) + (t < 0.125f ? s : ptx::lg2(1.0f + t) * ptx::kLn2);
-}
 __device__ __forceinline__ float sigmoid(float x) { return ptx::rcp(1.0f + ptx::ex2(-x * ptx::kLog2e)); }
 
 // Prepared pairs, f32, head-major so that a run of pairs is one contiguous block. Sequence number s with first row b starts at
@@ -88,26 +76,8 @@ __global__ void __launch_bounds__(128, TAPS > 0 && NJ == 1 ? 6 : 1) delta_prep_k
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int h = blockIdx.y * 4 + warp;
   if (h >= a.heads) return;
-  // which sequence tile number blockIdx.x belongs to: 32 sequences at a time, prefix sum over the lanes
-  int seq = -1, tile = static_cast<int>(blockIdx.x);
-  for (int s0 = 0; s0 < sq.seqs && seq < 0; s0 += 32) {
-    int tiles = 0;
-    if (s0 + lane < sq.seqs) tiles = (max(0, sq.seq_rows[2 * (s0 + lane) + 1] - sq.seq_rows[2 * (s0 + lane)]) + TT - 1) / TT;
-    int sum = tiles;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const int up = __shfl_up_sync(0xffffffffu, sum, o);
-      if (lane >= o) sum += up;
-    }
-    const uint32_t hit = __ballot_sync(0xffffffffu, tile < sum);
-    if (hit != 0) {
-      const int l = __ffs(hit) - 1;
-      seq = s0 + l;
-      tile -= __shfl_sync(0xffffffffu, sum - tiles, l);
-    } else {
-      tile -= __shfl_sync(0xffffffffu, sum, 31);
-    }
-  }
+  int tile = static_cast<int>(blockIdx.x);
+  const int seq = find_tile(sq, 0, sq.seqs, TT, tile);
   if (seq < 0) return;
   const int row0 = sq.seq_rows[2 * seq] + tile * TT;
   ConvRow cr;
@@ -136,7 +106,7 @@ __global__ void __launch_bounds__(128, TAPS > 0 && NJ == 1 ? 6 : 1) delta_prep_k
           // a row that is not there changes nothing
           q[j][t][v] = t < n ? ptx::silu(q[j][t][v]) : 0.0f;
           k[j][t][v] = t < n ? ptx::silu(k[j][t][v]) : 0.0f;
-          g[j][t][v] = t < n ? ptx::ex2(rate * softplus(z[v] + bias[v])) : 1.0f;
+          g[j][t][v] = t < n ? ptx::ex2(rate * softplus_fast(z[v] + bias[v])) : 1.0f;
         }
       }
     } else {
@@ -575,7 +545,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
   const int mine = lane & 3;
   float* state = a.state + (static_cast<int64_t>(cr.wr >> 1) * a.heads + h) * d * e + col;
   uint64_t S[P][4];
-  load_state<P>(state, cr.rd < 0, d, e, col, rg, S);
+  load_state<P, 4>(state, cr.rd < 0, d, e, col, rg, S);
   const int64_t o_ld = static_cast<int64_t>(a.heads) * e;
   float* o_dst = a.o_raw + static_cast<int64_t>(begin + (second ? 1 : 0)) * o_ld + static_cast<int64_t>(h) * e + col + mine;
   const bool writes = is_q && col + mine < e;
@@ -661,7 +631,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
     for (int s = 0; s < kStages; ++s) ptx::mbar_wait(bars + 8 * s, 0, 20000000ull) || ptx::mbar_wait(bars + 8 * s, 1, 20000000ull);
     return;
   }
-  store_state<P>(state, d, e, col, rg, S);
+  store_state<P, 4>(state, d, e, col, rg, S);
 }
 
 // out = rms_norm(o) * w * sigmoid(gate) for the rows of sequences >= first: one warp per (row, head).

@@ -230,10 +230,10 @@ def gated_linear(proj: torch.Tensor, z: torch.Tensor, p: GatedLinearParams, stat
             out[b:e] = (o * reference.silu(g[b:e]) * out_scale).to(out.dtype)
         return out
     C, st = _ext.require(), _state.get(proj.device)
-    scratch = torch.empty(C.gated_linear_scratch_floats(heads, dim, vdim, T) if seq.n_prefill else 0, dtype=torch.float32, device=proj.device)
+    scratch = torch.empty(C.gated_linear_scratch_floats(heads, dim, vdim, T, seq.seq_rows.shape[0], seq.n_prefill) if seq.n_prefill else 0, dtype=torch.float32, device=proj.device)
     C.gated_linear(proj, z, p.decay_bias, p.norm_w, p.tau, state, seq.row_seq, seq.seq_rows, seq.seq_state, out, scratch, heads, dim, vdim, eps, out_scale,
                    seq.n_decode, seq.first, seq.n_prefill, st.status)
-    _count((1 if seq.n_decode else 0) + (3 if seq.n_prefill else 0))
+    _count((1 if seq.n_decode else 0) + (C.gated_linear_prefill_launches(heads, vdim, T, seq.n_prefill) if seq.n_prefill else 0))
     return out
 
 

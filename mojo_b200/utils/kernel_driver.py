@@ -4,7 +4,8 @@ Small, self-terminating workloads (inputs larger than the 126 MB L2, a few GB at
 profiler capture of one kernel; with `--time` the case is timed with CUDA events instead and one JSON line is printed.
 Cases: gemm_large, gemm_pair (the same product on CTA pairs), gemm_prefill, gemm_decode, gemm_swiglu, gemm_fp8,
 gemm_fp8_decode, gemm_fp8_decode_nosplit (a narrow tensor-parallel shard at 256 tokens, with and without split-K),
-attn_decode, attn_prefill, mla_decode, mla_prefill, latent_decode, latent_prefill, moe_local, residual_norm, rmsnorm, sampling (arg-max), sample_topk_topp, gemm_gguf_q4k,
+attn_decode, attn_prefill, mla_decode, mla_prefill, latent_decode, latent_prefill, moe_local, residual_norm, norm_qkv, attn_capped,
+gated_scan, gated_scan_long (one prompt), gated_decode, rmsnorm, sampling (arg-max), sample_topk_topp, gemm_gguf_q4k,
 gemm_gguf_q6k, rope_kvwrite, all_reduce_norm_single.
 """
 from __future__ import annotations
@@ -138,6 +139,34 @@ def _case(name: str):
         ex = ops.ExpertRows(rnd(T * k, W), torch.randperm(T * k, device=DEV).int().view(T, k), torch.rand(T, k, device=DEV))
         done = ops.Finished(ones, rnd(T, W), ex)
         return (lambda: ops.residual_norm(x, ones, 1e-6, torch.bfloat16, done)), 0.0, T * W * (8 + 4 + 2 * k)
+    if name in ("gated_scan", "gated_scan_long", "gated_decode"):
+        # gated linear attention of 16 heads of 128: prompts (prepared rows, scan, output norm and gate), or one row of 256 sequences
+        from .layer_bench import step_rows
+
+        H, d = 16, 128
+        seq = step_rows(256, []) if name == "gated_decode" else step_rows(0, [2048] if name == "gated_scan_long" else [2048, 2048])
+        T, n = seq.row_seq.numel(), seq.seq_rows.shape[0]
+        p = ops.GatedLinearParams(torch.full((H * d,), 2.0, device=DEV), torch.ones(d, device=DEV), 16.0)
+        proj, z, state, out = rnd(T, 4 * H * d), rnd(T, H * d).float(), torch.zeros(n, H, d, d, device=DEV), rnd(T, H * d)
+        run = lambda: ops.gated_linear(proj, z, p, state, seq, H, d, d, 1e-5, out)  # noqa: E731
+        return run, 6.0 * T * H * d * d, n * H * d * d * 4 * (2 if seq.n_decode else 1) + T * H * d * 14
+    if name == "norm_qkv":
+        T, H, G, D, page = 16384, 32, 8, 128, 128
+        proj, table = rnd(T, (H + 2 * G) * D), ref.rope_table(T, D // 2, 10000.0).to(DEV)
+        kc, vc = (torch.zeros(T // page, G, page, D, device=DEV, dtype=torch.bfloat16) for _ in range(2))
+        p = ops.QkvNorm(*(torch.ones(n, device=DEV) for n in ((H + 2 * G) * D, H * D, G * D)))
+        pos, slots = torch.arange(T, dtype=torch.int32, device=DEV), torch.arange(T, dtype=torch.int64, device=DEV)
+        return (lambda: ops.norm_qkv(proj, p, table, pos, slots, kc, vc, H, G, D, D, D, 1e-5)), 0.0, T * (H + 2 * G) * D * 4
+    if name == "attn_capped":
+        # two prompts of 2048 tokens, 32 query heads on 8, a window of 1024 and capped scores
+        S, L, H, G, D, page, win = 2, 2048, 32, 8, 128, 128, 1024
+        kc, vc, q = rnd(S * L // page, G, page, D), rnd(S * L // page, G, page, D), rnd(S * L, H * D)
+        cu = torch.arange(0, (S + 1) * L, L, dtype=torch.int32, device=DEV)
+        cl, bt = torch.full((S,), L, dtype=torch.int32, device=DEV), torch.arange(S * L // page, dtype=torch.int32, device=DEV).view(S, -1)
+        work = torch.from_numpy(ops.prefill_work_items(cu.cpu().numpy(), cl.cpu().numpy(), 0)).to(DEV)
+        meta = ops.AttnMeta(cu, cl, bt, 0, L, L, work=work, n_items=work.shape[0])
+        pairs = S * sum(min(t + 1, win) for t in range(L))
+        return (lambda: ops.paged_attention(q, kc, vc, meta, D ** -0.5, D, mods=ops.ScoreMods(win, 30.0, 0.5))), 4.0 * pairs * H * D, S * L * (2 * H + 2 * G) * D * 2
     if name in ("tp_gemm_rs_single", "tp_ag_gemm_single"):
         # The fused tensor-parallel kernels on ONE rank (a world of one: the only peer is this GPU's own region), so that
         # their tensor-core / epilogue / staging behaviour can be captured under a profiler, which never runs on a
@@ -261,7 +290,8 @@ def _case(name: str):
 
 
 CASES = ("gemm_large", "gemm_pair", "gemm_prefill", "gemm_decode", "gemm_swiglu", "gemm_fp8", "gemm_fp8_decode", "gemm_fp8_decode_nosplit",
-         "attn_decode", "attn_prefill", "mla_decode", "mla_prefill", "latent_decode", "latent_prefill", "moe_local", "residual_norm", "rmsnorm", "sampling", "sample_topk_topp", "gemm_gguf_q4k", "gemm_gguf_q6k",
+         "attn_decode", "attn_prefill", "mla_decode", "mla_prefill", "latent_decode", "latent_prefill", "moe_local", "residual_norm", "norm_qkv", "attn_capped",
+         "gated_scan", "gated_scan_long", "gated_decode", "rmsnorm", "sampling", "sample_topk_topp", "gemm_gguf_q4k", "gemm_gguf_q6k",
          "rope_kvwrite", "all_reduce_norm_single")
 # single-rank forms of the fused tensor-parallel and expert-parallel kernels (profiling only): tp_gemm_rs_single,
 # tp_ag_gemm_single, moe_ep_single

@@ -1,10 +1,11 @@
 """A design beside the closest one at equal layer sizes: prefill and decode throughput of a few layers through the serving
 engine, and each design's own kernels against their rooflines. Random weights, synthetic prompts, one GPU
-(`bench.py --layer-bench`: Rekudra beside Llama; `bench.py --layer-bench rerupel`: Rerupel beside DeepSeek-V2).
+(`bench.py --layer-bench`: Rekudra beside Llama; `bench.py --layer-bench rerupel`: Rerupel beside DeepSeek-V2;
+`bench.py --layer-bench pilutar`: Pilutar beside Rerupel, its single kernels also beside the like ones of Llama and Rekudra).
 
 Steps are timed with CUDA events around the engine's device work, medians over repeats after warm-up; every step streams
 weights and caches larger than L2. Single kernels are timed with an L2 flush before each launch. Rooflines use the copy
-bandwidth and the bf16 rate measured on the machine; the scan of the delta rule works on f32 matrices, so its compute
+bandwidth and the bf16 rate measured on the machine; the scans of recurrent layers work on f32 matrices, so their compute
 bound is the f32 FMA rate (SMs x 128 lanes x maximum clock)."""
 from __future__ import annotations
 
@@ -14,11 +15,12 @@ from pathlib import Path
 
 import torch
 
-DESIGNS = {"rekudra": ("llama", "rekudra"), "rerupel": ("deepseek", "rerupel")}      # (closest model, design)
+DESIGNS = {"rekudra": ("llama", "rekudra"), "rerupel": ("deepseek", "rerupel"), "pilutar": ("rerupel_plain", "pilutar")}      # (closest model, design)
 SIZES = {"2048x16": dict(width=2048, heads=16, kv=4, dim=128, ffn=8192), "4096x32": dict(width=4096, heads=32, kv=8, dim=128, ffn=14336)}
 # DeepSeek-V2-Lite's layers, and the same at twice the width; latents of 512 columns, 64 experts of which 6 are used
 MOE_SIZES = {"2048x16": dict(width=2048, heads=16, dim=128, rank=512, rope=64, ffn=10944, experts=64, top=6, expert_ffn=1408),
              "4096x32": dict(width=4096, heads=32, dim=128, rank=512, rope=64, ffn=14336, experts=64, top=6, expert_ffn=1408)}
+PILUTAR_SIZES = {k: dict(v, kv=4 * (i + 1), rope=32, window=1024, groups=8, keep=4, identity=2) for i, (k, v) in enumerate(MOE_SIZES.items())}
 VOCAB, LAYERS = 32000, 8
 MOE_RUNS = 9           # one dense layer and eight with experts (the design: four, passed twice)
 PREFILL = [(1, 2048), (2, 2048), (8, 512)]        # (prompts, tokens each), one step
@@ -33,8 +35,15 @@ def peaks() -> dict:
 
 
 def model_config(design: str, size: dict):
-    from ..models.config import ModelConfig, rekudra, rerupel
+    from ..models.config import ModelConfig, pilutar, rekudra, rerupel
 
+    if design == "pilutar":
+        return pilutar(size["width"], MOE_RUNS, size["heads"], size["kv"], size["dim"], size["rank"], size["rope"], size["ffn"], VOCAB,
+                       size["experts"] - size["identity"], size["top"], size["expert_ffn"], 2 * size["expert_ffn"], size["window"], size["groups"], size["keep"],
+                       size["identity"])
+    if design == "rerupel_plain":      # every layer run with weights of its own
+        return rerupel(size["width"], MOE_RUNS, size["heads"], size["dim"], size["rank"], size["ffn"], VOCAB, size["experts"], size["top"], size["expert_ffn"],
+                       2 * size["expert_ffn"])
     if design == "rerupel":
         return rerupel(size["width"], 5, size["heads"], size["dim"], size["rank"], size["ffn"], VOCAB, size["experts"], size["top"], size["expert_ffn"],
                        2 * size["expert_ffn"], (1, 5, 2))
@@ -349,11 +358,155 @@ def latent_kernel_table(size: dict) -> list[dict]:
     return tab.rows
 
 
+def pilutar_kernel_table(size: dict) -> list[dict]:
+    """Pilutar's kernels beside those of Rerupel, and of Llama and Rekudra where those have the like one."""
+    from .. import ops
+    from ..ops import reference
+
+    W, H, G, d, R, E, k, F = (size[n] for n in ("width", "heads", "kv", "dim", "rank", "experts", "top", "expert_ffn"))
+    r, win, real, page, dev, bf = size["rope"], size["window"], size["experts"] - size["identity"], 128, torch.device("cuda"), torch.bfloat16
+    tab = KernelTable()
+    add, st, C = tab.add, ops._state.get(torch.device("cuda", 0)), ops._ext.require()
+    f32 = lambda *s, std=1.0: rnd(*s, dtype=torch.float32, std=std)  # noqa: E731
+    ones, table, table_r = torch.ones(max(W, H * d), device=dev), reference.rope_table(4096, d // 2, 1e4).to(dev), reference.rope_table(4096, r, 5e4).to(dev)
+    table_d = reference.rope_table(4096, d, 1e4).to(dev)
+    up, gu, down = rnd(E, F, W, std=W ** -0.5), rnd(E, 2 * F, W, std=W ** -0.5), rnd(E, W, F, std=F ** -0.5)
+    router, corr = rnd(E + 8, W, std=W ** -0.5), f32(E, std=0.02)
+    Q = 64                                             # columns of the rotated part in the cache
+    for case, seq, ctx, n_seq, T in (("decode 128 x 1024", step_rows(128, []), 1024, 128, 128), ("prefill 2 x 2048", step_rows(0, [2048, 2048]), 2048, 2, 4096)):
+        dec = seq.n_decode > 0
+        per = ctx // page + 1
+        bt = torch.arange(n_seq * per, dtype=torch.int32, device=dev).view(n_seq, per)
+        cl = torch.full((n_seq,), ctx, dtype=torch.int32, device=dev)
+        cu = torch.arange(n_seq + 1, dtype=torch.int32, device=dev) * (T // n_seq)
+        host = cu.cpu().numpy(), cl.cpu().numpy()
+        base = torch.arange(n_seq, device=dev) * per * page
+        slots = base + ctx - 1 if dec else (base[:, None] + torch.arange(ctx, device=dev)[None]).flatten()
+        pos = torch.full((T,), ctx - 1, dtype=torch.int32, device=dev) if dec else torch.arange(ctx, dtype=torch.int32, device=dev).repeat(n_seq)
+        work = None if dec else torch.from_numpy(ops.prefill_work_items(*host, 0)).cuda()
+        meta = ops.AttnMeta(cu, cl, bt, n_seq if dec else 0, T // n_seq, ctx, work=work, n_items=0 if dec else work.shape[0])
+        # (query, key) pairs, all and inside the window; keys a sequence's rows see
+        pairs = float(n_seq * ctx) if dec else n_seq * ctx * (ctx + 1) / 2
+        near = float(n_seq * min(ctx, win)) if dec else n_seq * sum(min(t + 1, win) for t in range(ctx))
+        keys = n_seq * min(ctx, win) if dec else n_seq * ctx
+        # --- residual and norm
+        x, y, sh, z = f32(T, W), rnd(T, W), rnd(T, W), f32(T, 8)
+        h = rnd(T, W)
+        p = ops.MoeWeights(router[:E], up[:real], down[:real], real, k, "softmax", True, 1.0, None, corr, size["groups"], size["keep"], size["identity"])
+        pr = ops.MoeWeights(router[:E], gu, down, E, k, "sigmoid", False, 1.0, ops.Glu(7.0, 1.702, 1.0))
+        ex, exr = ops.moe_experts(h, p), ops.moe_experts(h, pr)
+        w1 = ones[:W]
+        add("residual_norm, layer norm", "pilutar", case, lambda: ops.residual_norm(x, w1, 1e-5, bf, ops.Finished(None, y), bias=w1), T * W * 12)
+        add("residual_norm", "rerupel", case, lambda: ops.residual_norm(x, w1, 1e-6, bf, ops.Finished(w1, y)), T * W * 12)
+        add("residual_norm, layer norm, of experts and gated row", "pilutar", case,
+            lambda: ops.residual_norm(x, w1, 1e-5, bf, ops.Finished(None, y, ex, sh, z[:, 0]), bias=w1), T * W * (14 + 2 * k))
+        add("residual_norm of expert rows", "rerupel", case, lambda: ops.residual_norm(x, w1, 1e-6, bf, ops.Finished(w1, y, exr)), T * W * (12 + 2 * k))
+        # --- attention beside the recurrence
+        nq, nk = H * d, G * d
+        kc, vc = (rnd(n_seq * per, G, page, d) for _ in range(2))
+        proj = rnd(T, nq + 2 * nk)
+        qp = ops.QkvNorm(f32(nq + 2 * nk), ones[:nq], ones[:nk])
+        add("norm_qkv", "pilutar", case, lambda: ops.norm_qkv(proj, qp, table, pos, slots, kc, vc, H, G, d, d, d, 1e-5), T * (nq + 2 * nk) * 4)
+        add("rope_kvwrite", "llama", case, lambda: ops.rope_kvwrite(proj[:, :nq], proj[:, nq:nq + nk], proj[:, nq + nk:], table_d, pos, slots, kc, vc, d),
+            T * (2 * nq + 4 * nk) * 2)
+        q, cat = rnd(T, nq), torch.empty(T, 2 * nq, device=dev, dtype=bf)
+        mods = ops.ScoreMods(win, 30.0, 0.5)
+        add("attention, window, capped", "pilutar", case, lambda: ops.paged_attention(q, kc, vc, meta, d ** -0.5, d, out=cat[:, :nq], mods=mods),
+            keys * G * d * 4 + T * nq * 4, mma=0.0 if dec else near * H * d * 2)
+        add("attention", "llama", case, lambda: ops.paged_attention(q, kc, vc, meta, d ** -0.5, d), n_seq * ctx * G * d * 4 + T * nq * 4,
+            mma=0.0 if dec else pairs * H * d * 2)
+        # --- recurrences
+        state = torch.zeros(n_seq, H, d, d, device=dev)
+        pg, zg = rnd(T, 4 * nq), f32(T, nq)
+        gp = ops.GatedLinearParams(torch.full((nq,), 2.0, device=dev), ones[:d], 16.0)
+        state_bytes = n_seq * H * d * d * 4 * (2 if dec else 1)
+        add("gated_linear", "pilutar", case, lambda: ops.gated_linear(pg, zg, gp, state, seq, H, d, d, 1e-5, cat[:, nq:], 0.5), state_bytes + T * nq * 14,
+            fma=0.0 if dec else 3.0 * T * H * d * d)
+        pd, dg, taps = rnd(T, 3 * nq + H), rnd(T, 2 * nq), 4
+        dp = ops.DeltaParams(f32(taps, 3 * nq, std=0.3), -ones[:H], torch.full((nq,), -3.0, device=dev), ones[:d])
+        bank = rnd(2 * n_seq, taps - 1, 3 * nq)
+        add("delta_rule", "rekudra", case, lambda: ops.delta_rule(pd, dg, dp, bank, state, seq, 3 * nq, H, H, d, d, nq, 1e-5),
+            state_bytes + T * (6 * nq + H) * 2 + n_seq * (taps - 1) * 6 * nq * (2 if dec else 1), fma=0.0 if dec else 4.0 * T * H * d * d)
+        # --- latent attention
+        cache, plain = rnd(n_seq * per, page, R + Q), rnd(n_seq * per, page, R)
+        pl = rnd(T, nq + R + r + H)
+        rope = ops.SharedRope(pl[:, nq + R:nq + R + r], pl[:, :nq], H, d - r, R, table_r, pos)
+        add("latent_write, rotated", "pilutar", case, lambda: ops.latent_write(pl[:, nq:nq + R], ones[:R], 1e-5, slots, cache, rope), T * ((R + r) * 4 + H * r * 4))
+        add("latent_write", "rerupel", case, lambda: ops.latent_write(pl[:, nq:nq + R], ones[:R], 1e-6, slots, plain), T * R * 4)
+        w_qk, w_kv = rnd(H * (R + Q), d, std=d ** -0.5), rnd(2 * nq, R + Q, std=R ** -0.5)
+        w_qk_p, w_kv_p = w_qk[:H * R], rnd(2 * nq, R, std=R ** -0.5)
+        gate, gate_e = pl[:, nq + R + r:], rnd(T, nq)
+        rows = ops.token_rows(meta, T, dev)
+        q_lat, q_lat_p = rnd(T, H * (R + Q)), rnd(T, H * R)
+        if dec:
+            add("latent_attend, rotated, window", "pilutar", case, lambda: ops.latent_attend(q_lat, cache, meta, rows, H, 0.1, pos, R, win),
+                keys * (R + r) * 2 + T * H * (2 * R + r) * 2, mma=near * H * (2 * R + r))
+            add("latent_attend", "rerupel", case, lambda: ops.latent_attend(q_lat_p, plain, meta, rows, H, 0.1, pos), n_seq * ctx * R * 2 + T * H * R * 4,
+                mma=pairs * H * 2 * R)
+        else:
+            out = torch.empty(T, nq, device=dev, dtype=bf)
+            plan = ops.plan_latent_prefill(*host, 0, R, H, d, d, win)
+            meta.expand = tuple(torch.from_numpy(a).cuda() for a in plan)
+            expand = float(len(plan[0]) * 128) * R * 2 * nq
+            add("latent_prefill, rotated, window", "pilutar", case, lambda: ops.latent_prefill(pl[:, :nq], cache, w_kv, meta, H, 0.1, gate, out, win), T * nq * 6,
+                mma=near * H * 2 * d + expand)
+            add("latent_prefill", "rerupel", case, lambda: ops.latent_prefill(pl[:, :nq], plain, w_kv_p, meta, H, 0.1, gate_e, out), T * nq * 8,
+                mma=pairs * H * 2 * d + expand)
+        if dec:                                        # prompts take the expanded form
+            add("head_gemm (queries)", "pilutar", case, lambda: ops.head_linear(pl[:, :nq], w_qk, H), T * H * (d + R + r) * 2 + H * R * (d - r) * 2,
+                mma=float(T) * H * R * (d - r))
+            add("head_gemm (queries)", "rerupel", case, lambda: ops.head_linear(pl[:, :nq], w_qk_p, H), T * H * (d + R) * 2 + H * R * d * 2, mma=float(T) * H * R * d)
+            add("head_gemm (values, gate per head)", "pilutar", case, lambda: ops.head_linear(q_lat_p, w_kv[nq:, :R], H, gate=gate), T * H * (d + R) * 2 + H * R * d * 2,
+                mma=float(T) * H * R * d)
+            add("head_gemm (values, gated)", "rerupel", case, lambda: ops.head_linear(q_lat_p, w_kv_p[nq:], H, gate=gate_e), T * H * (2 * d + R) * 2 + H * R * d * 2,
+                mma=float(T) * H * R * d)
+        # --- experts
+        logits = ops.linear_f32(h, router)
+        n_id = float((ex.slot < 0).float().mean()) if size["identity"] else 0.0
+        run_k, used = k * (1.0 - n_id), float(min(real, T * k))
+        add("router, experts", "pilutar", case, lambda: ops.moe_experts(h, p, logits), used * 2 * W * F * 2 + T * run_k * (3 * W + 2 * F) * 2,
+            mma=float(T) * run_k * 2 * W * F)
+        add("router, experts", "rerupel", case, lambda: ops.moe_experts(h, pr, logits), min(E, T * k) * 3 * W * F * 2 + T * k * (3 * W + 2 * F) * 2,
+            mma=float(T) * k * 3 * W * F)
+        wts, bn = torch.empty(T, k, device=dev), ops.moe.tile_rows(T * k / E)
+        ids, place, slot = (torch.empty(T, k, dtype=torch.int32, device=dev) for _ in range(3))
+        xr, tiles, nt = torch.empty(T * k, W, device=dev, dtype=bf), torch.empty(E + T * k // bn, 4, dtype=torch.int32, device=dev), torch.empty(1, dtype=torch.int32, device=dev)
+
+        def route(grouped: bool):
+            n = real if grouped else E
+            if grouped:
+                C.moe_route(logits, wts, ids, place, st.moe_counts, n, 0, True, 1.0, corr, size["groups"], size["keep"], size["identity"])
+            else:
+                C.moe_route(logits, wts, ids, place, st.moe_counts, n, 1, False, 1.0)
+            C.moe_gather(h, ids, place, st.moe_counts, slot, xr, tiles, nt, n, bn, st.status)
+
+        act, yr = torch.empty(T * k, F, device=dev, dtype=bf), torch.empty(T * k, W, device=dev, dtype=bf)
+        add("moe_route, moe_gather, groups", "pilutar", case, lambda: route(True), T * W * 2 * (run_k + 1) + T * E * 4)
+        add("expert products, squared ReLU", "pilutar", case, lambda: C.moe_tiles_gemm(xr, up[:real], tiles, nt, act, ops.EPI_RELU2, bn, None, st.status),
+            used * W * F * 2 + T * run_k * (W + F) * 2, mma=float(T) * run_k * W * F)
+        add("moe_route, moe_gather", "rerupel", case, lambda: route(False), T * W * 2 * (k + 1) + T * E * 4)
+        add("expert products, gate / up", "rerupel", case, lambda: C.moe_tiles_gemm(xr, gu, tiles, nt, act, ops.EPI_SWIGLU, bn, (7.0, 1.702, 1.0, 0.0), st.status),
+            min(E, T * k) * 2 * W * F * 2 + T * k * (W + F) * 2, mma=float(T) * k * 2 * W * F)
+        # --- products that only this design has in this form
+        ff = size["ffn"]
+        w_gu, w_dec, w_out = rnd(2 * ff, W, std=W ** -0.5), rnd(nq, 16), rnd(W, 2 * nq + ff, std=(2 * nq + ff) ** -0.5)
+        wide = rnd(T, 2 * nq + ff)
+        add("gemm, ReLU-gated, into columns", "pilutar", case, lambda: ops.linear_swiglu(h, w_gu, out=wide[:, 2 * nq:], glu=ops.REGLU), (2 * ff * W + T * (W + ff)) * 2,
+            mma=2.0 * T * W * ff)
+        add("gemm, gated unit", "rerupel", case, lambda: ops.linear_swiglu(h, w_gu, glu=ops.Glu(7.0, 1.702, 1.0)), (2 * ff * W + T * (W + ff)) * 2, mma=2.0 * T * W * ff)
+        add("gemm, all output projections", "pilutar", case, lambda: ops.linear(wide, w_out), (w_out.numel() + wide.numel() + T * W) * 2, mma=float(T) * w_out.numel())
+        w_plain, x_plain = w_out[:, :nq].contiguous(), wide[:, :nq].contiguous()
+        add("gemm, output projection", "rerupel", case, lambda: ops.linear(x_plain, w_plain), (w_plain.numel() + x_plain.numel() + T * W) * 2, mma=float(T) * w_plain.numel())
+        low = rnd(T, 4 * nq)[:, :16]
+        add("gemm, decay logits, f32", "pilutar", case, lambda: ops.linear_f32(low, w_dec), (w_dec.numel() + T * 16) * 2 + T * nq * 4, mma=float(T) * w_dec.numel())
+    return tab.rows
+
+
 def run(args) -> dict:
     from .clocks import ClockSampler
 
     base, design = DESIGNS[args.layer_bench]
-    sizes, table = (SIZES, kernel_table) if design == "rekudra" else (MOE_SIZES, latent_kernel_table)
+    sizes, table = {"rekudra": (SIZES, kernel_table), "rerupel": (MOE_SIZES, latent_kernel_table), "pilutar": (PILUTAR_SIZES, pilutar_kernel_table)}[design]
     out = {"metric": f"layer throughput, {design} beside {base} at equal layer sizes", "unit": "tok/s", "n_gpus": 1, "dtype": "bf16",
            "layers": LAYERS if design == "rekudra" else MOE_RUNS, "data": "synthetic: uniform-random token ids, random weights", "peaks": peaks(), "sizes": {}}
     with ClockSampler(0) as clocks:

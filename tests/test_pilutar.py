@@ -367,34 +367,49 @@ def test_residual_and_layer_norm(target, width, pad, top):
 
 
 @pytest.mark.parametrize("target", TARGETS)
-@pytest.mark.parametrize("heads,kv,dim,vdim,rot", [(1, 1, 8, 8, 8), (6, 2, 24, 40, 12), (8, 1, 64, 64, 32), (5, 5, 13, 7, 6), (4, 2, 128, 96, 0), (34, 2, 18, 10, 10)])
-def test_projection_norms_and_rotation(target, heads, kv, dim, vdim, rot):
+@pytest.mark.parametrize("heads,kv,dim,vdim,rot,T", [(1, 1, 8, 8, 8, 5), (6, 2, 24, 40, 12, 5), (8, 1, 64, 64, 32, 5), (5, 5, 13, 7, 6, 5), (4, 2, 128, 96, 0, 5),
+                                                       (34, 2, 18, 10, 10, 5), (3, 1, 128, 128, 64, 700), (2, 1, 256, 256, 256, 650), (9, 3, 32, 32, 16, 1000),
+                                                       (40, 4, 128, 128, 128, 600)])
+def test_projection_norms_and_rotation(target, heads, kv, dim, vdim, rot, T):
     """Biases, one norm over all query (key) columns of a row, rotated halves, keys and values in their cache rows."""
     g = torch.Generator().manual_seed(heads + dim)
-    T, page, n = 5, 4, heads * dim + kv * (dim + vdim)
+    page, n = 4, heads * dim + kv * (dim + vdim)
     pad = next(x for x in (64, 128, 256) if x >= max(dim, vdim)) if target[1] == "bfloat16" else None
     proj = rounded(torch.randn(T, n + 24, generator=g), target)
     proj[2] *= 30.0                                                          # the norm of a row is its own
     bias, qw, kw = (torch.randn(s, generator=g) for s in (n, heads * dim, kv * dim))
     pos, slots = torch.tensor([0, 1, 70, 500, 3]), torch.tensor([7, -1, 0, 19, 12])
+    if T > 5:                                                                # many rows: another kernel, rows in a random order
+        pos, slots = torch.randint(0, 600, (T,), generator=g), torch.randperm(4 * T, generator=g)[:T]
+        slots[3] = -1
     table = reference.rope_table(600, rot, 5000.0)
-    kc, vc = (dev(torch.zeros(5, kv, page, pad or s), target) for s in (dim, vdim))
+    kc, vc = (dev(torch.zeros(5 if T == 5 else T, kv, page, pad or s), target) for s in (dim, vdim))
     q = ops.norm_qkv(dev(proj, target), ops.QkvNorm(*(f32(t, target) for t in (bias, qw, kw))), table.to(target[0]), dev(pos, target, torch.int32),
                      slots.to(target[0]), kc, vc, heads, kv, dim, vdim, pad or dim, 1e-2)
     sync(target)
     u = proj[:, :n] + bias.double()
-    turned = lambda z, m: torch.cat([P.rotate(torch.cat([torch.zeros(int(p), m, dim).double(), z[i:i + 1]]), rot, 5000.0, False)[-1:] if rot else z[i:i + 1]  # noqa: E731
-                                     for i, p in enumerate(pos)])
+
+
+    def turned(z, m):      # row i at position pos[i]
+        if not rot:
+            return z
+        ang, out = P.angles(600, rot, 5000.0, torch.float64)[pos][:, None], z.clone()
+        a, b = z[..., :rot // 2], z[..., rot // 2:rot]
+        out[..., :rot // 2], out[..., rot // 2:rot] = a * torch.cos(ang) - b * torch.sin(ang), b * torch.cos(ang) + a * torch.sin(ang)
+        return out
+
     wq = turned(P.rms_norm(u[:, :heads * dim], qw.double(), 1e-2).view(T, heads, dim), heads)
     wk = turned(P.rms_norm(u[:, heads * dim:(heads + kv) * dim], kw.double(), 1e-2).view(T, kv, dim), kv)
     got = q.view(T, heads, -1)
     close(got[..., :dim], wq, target)
     assert float(got[..., dim:].abs().sum()) == 0
-    for t, s in enumerate(slots.tolist()):
-        if s >= 0:
-            close(kc[s // page, :, s % page, :dim], wk[t], target)
-            close(vc[s // page, :, s % page, :vdim], u[t, (heads + kv) * dim:].view(kv, vdim), target)
-    assert float(kc[..., dim:].abs().sum()) == 0 and float(vc[0, :, 1:].abs().sum()) == 0
+    kept = slots >= 0
+    at = slots[kept].to(target[0])
+    close(kc.transpose(1, 2).flatten(0, 1)[at][..., :dim], wk[kept], target)
+    close(vc.transpose(1, 2).flatten(0, 1)[at][..., :vdim], u[:, (heads + kv) * dim:].view(T, kv, vdim)[kept], target)
+    empty = torch.ones(len(kc) * page, dtype=torch.bool)
+    empty[slots[kept]] = False
+    assert float(kc[..., dim:].abs().sum()) == 0 and float(vc.transpose(1, 2).flatten(0, 1)[empty.to(target[0])].abs().sum()) == 0
 
 
 def edge_batch(target, ctx, page, q_len, heads, kv, dim, vdim, window, cap, seed):
