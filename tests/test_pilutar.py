@@ -573,11 +573,15 @@ def test_latent_attention_with_a_rotated_part(monkeypatch, target, window, heads
 
 @pytest.mark.parametrize("target", TARGETS)
 @pytest.mark.parametrize("heads,dim,vdim,tau", [(1, 8, 8, 1.0), (2, 48, 32, 16.0), (3, 13, 7, 4.0), (4, 128, 128, 16.0), (2, 70, 90, 8.0), (1, 256, 200, 2.0)])
-def test_recurrence(target, heads, dim, vdim, tau):
+@pytest.mark.parametrize("lens", [(1, 1, 1, 37, 2, 5, 130), (1, 1, 1, 700, 16, 531, 2), (1, 1, 1, 1100, 33)], ids=lambda x: f"{sum(x)}rows")
+def test_recurrence(target, heads, dim, vdim, tau, lens):
     """Decode rows beside chunks of several lengths, fresh sequences and ones with history, decays from almost none to almost
-    total; states land in their slots, other slots stay as they are, and a fresh sequence ignores what its slot held."""
+    total; states land in their slots, other slots stay as they are, and a fresh sequence ignores what its slot held. Few long
+    chunks are cut into segments that run side by side."""
+    if sum(lens) > 200 and target[0] == "cpu" and dim != 13:
+        pytest.skip("one size is enough for the plain operations")
     g = torch.Generator().manual_seed(dim + heads)
-    lens, fresh, slots = [1, 1, 1, 37, 2, 5, 130], [False, True, False, True, False, False, False], [5, 0, 7, 2, 3, 8, 1]
+    fresh, slots = [False, True, False, True, False, False, False][:len(lens)], [5, 0, 7, 2, 3, 8, 1][:len(lens)]
     T, nk, nv, n = sum(lens), heads * dim, heads * vdim, len(lens)
     proj = rounded(torch.randn(T, 2 * (nk + nv), generator=g), target)
     z, bias, w = torch.randn(T, nk + 3, generator=g) * 3, torch.randn(nk, generator=g) * 4, 1 + 0.2 * torch.randn(vdim, generator=g)
