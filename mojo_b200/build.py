@@ -30,7 +30,7 @@ LIBDIR = ROOT / "lib"
 # What a model on one GPU needs in bf16 or f32; the rest (fp8, GGUF, tensor and expert parallelism, examples) comes with
 # a full build. Both link under the same names; `lib/BUILD` says which one is there.
 CORE_KERNELS = {"attention", "attention_tc", "delta_rule", "elementwise", "f32_ops", "gated_linear", "gemm_bf16", "gemm_bf16_pair", "head_gemm", "hyper_conn", "latent", "mla_decode",
-                "moe_local", "qkv_norm", "residual_norm", "sampling", "short_conv"}
+                "moe_local", "post_norm", "qkv_norm", "residual_norm", "selective_scan", "sampling", "short_conv"}
 CORE_BINDINGS = {"engine_bind", "io_bind", "latent_bind", "mixers_bind", "ops_bind"}
 
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]

@@ -145,15 +145,16 @@ void moe_route(const at::Tensor& logits, at::Tensor& weights, at::Tensor& ids, a
 }
 
 void moe_gather(const at::Tensor& x, const at::Tensor& ids, const at::Tensor& place, at::Tensor& counts, at::Tensor& slot, at::Tensor& xs, at::Tensor& tiles,
-                at::Tensor& n_tiles, int64_t experts, int64_t bn, const OptTensor& status) {
+                at::Tensor& n_tiles, int64_t experts, int64_t bn, const OptTensor& status, const OptTensor& weights) {
   need(is_act(x) && x.dim() == 2 && x.is_contiguous() && xs.scalar_type() == x.scalar_type() && xs.is_cuda() && xs.is_contiguous(), "moe_gather: x [T, W], xs [T * top, W]");
   const int64_t T = x.size(0), top = ids.size(1);
   need(is_i32(ids) && is_i32(place) && is_i32(slot) && ids.numel() == T * top && place.numel() == T * top && slot.numel() == T * top &&
            xs.numel() == T * top * x.size(1), "moe_gather: ids, place, slot int32 [T, top]");
   need(bn >= 1 && is_i32(counts) && counts.numel() >= experts + 1 && is_i32(tiles) && tiles.numel() >= 4 * (experts + T * top / bn) && is_i32(n_tiles),
        "moe_gather: counts [experts + 1], tiles int32 [experts + T * top / bn, 4], n_tiles int32");
+  if (weights.has_value()) need(is_f32(*weights, T * top), "moe_gather: weights f32 [T, top]");
   c10::cuda::CUDAGuard g(x.device());
-  check(b2_moe_gather(x.data_ptr(), ids.data_ptr<int32_t>(), place.data_ptr<int32_t>(), counts.data_ptr<int32_t>(), slot.data_ptr<int32_t>(), xs.data_ptr(),
+  check(b2_moe_gather(x.data_ptr(), ids.data_ptr<int32_t>(), place.data_ptr<int32_t>(), weights.has_value() ? weights->data_ptr<float>() : nullptr, counts.data_ptr<int32_t>(), slot.data_ptr<int32_t>(), xs.data_ptr(),
                       tiles.data_ptr<int32_t>(), n_tiles.data_ptr<int32_t>(), as_int(T), as_int(experts), as_int(top), as_int(x.size(1)), as_int(bn),
                       x.scalar_type() == at::kFloat ? 1 : 0, status_ptr(status), cur_stream()), "moe_gather");
 }
@@ -192,6 +193,7 @@ void bind_latent(py::module_& m) {
   m.def("moe_route", &moe_route, py::arg("logits"), py::arg("weights"), py::arg("ids"), py::arg("place"), py::arg("counts"), py::arg("experts"),
         py::arg("scoring"), py::arg("norm_top"), py::arg("scale"), py::arg("correction") = py::none(), py::arg("groups") = 1, py::arg("keep") = 1,
         py::arg("identity") = 0);
-  m.def("moe_gather", &moe_gather);
+  m.def("moe_gather", &moe_gather, py::arg("x"), py::arg("ids"), py::arg("place"), py::arg("counts"), py::arg("slot"), py::arg("xs"), py::arg("tiles"),
+        py::arg("n_tiles"), py::arg("experts"), py::arg("bn"), py::arg("status") = py::none(), py::arg("weights") = py::none());
   m.def("moe_tiles_gemm", &moe_tiles_gemm);
 }

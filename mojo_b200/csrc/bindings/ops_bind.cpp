@@ -193,11 +193,21 @@ const void* gate_ptr(const c10::optional<at::Tensor>& gate, const at::Tensor& q,
        "attention: gate must be bf16 [T, n_q] with unit inner stride");
   return gate->data_ptr();
 }
+// The gate has one logit per head, or one per output element.
+bool by_element(const c10::optional<at::Tensor>& gate, const at::Tensor& q) { return gate.has_value() && gate->dim() == 2 && gate->size(1) == q.size(1); }
+B2AttnMods attn_mods(int64_t window, double softcap, double out_scale, int64_t chunk, bool sink, const c10::optional<at::Tensor>& distance, int64_t n_q) {
+  B2AttnMods m{static_cast<int32_t>(window), static_cast<int32_t>(chunk), static_cast<float>(softcap), static_cast<float>(out_scale), nullptr, sink ? 1 : 0};
+  if (distance.has_value()) {
+    need(distance->is_cuda() && distance->scalar_type() == at::kFloat && distance->is_contiguous() && distance->numel() == 2 * n_q, "attention: distance must be f32 [2, n_q]");
+    m.distance = distance->data_ptr<float>();
+  }
+  return m;
+}
 int64_t gate_ld(const c10::optional<at::Tensor>& gate) { return gate.has_value() ? gate->stride(0) : 0; }
 
 void attn_prefill(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out,
                   const at::Tensor& cu_q, const at::Tensor& ctx_lens, const at::Tensor& block_tables, int64_t head_dim,
-                  int64_t max_q_len, double scale, c10::optional<at::Tensor> status, c10::optional<at::Tensor> gate, int64_t window, double softcap, double out_scale) {
+                  int64_t max_q_len, double scale, c10::optional<at::Tensor> status, c10::optional<at::Tensor> gate, int64_t window, double softcap, double out_scale, int64_t chunk, bool sink, c10::optional<at::Tensor> distance) {
   check_cache(q, k_cache, v_cache, head_dim);
   need(out.dim() == 2 && out.stride(1) == 1 && is_bf16(out) && out.size(0) == q.size(0), "attention: bad out");
   need(cu_q.scalar_type() == at::kInt && ctx_lens.scalar_type() == at::kInt && block_tables.scalar_type() == at::kInt, "attention: metadata must be int32");
@@ -205,13 +215,13 @@ void attn_prefill(const at::Tensor& q, const at::Tensor& k_cache, const at::Tens
   const int batch = static_cast<int>(ctx_lens.numel());
   need(cu_q.numel() == batch + 1 && block_tables.size(0) == batch, "attention: metadata batch mismatch");
   c10::cuda::CUDAGuard g(q.device());
+  const B2AttnMods mods = attn_mods(window, softcap, out_scale, chunk, sink, distance, q.size(1) / head_dim);
   check(b2_attn_prefill_bf16(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), cu_q.data_ptr<int32_t>(),
                              ctx_lens.data_ptr<int32_t>(), block_tables.data_ptr<int32_t>(), batch,
                              static_cast<int>(block_tables.size(1)), static_cast<int>(q.size(1) / head_dim),
                              static_cast<int>(k_cache.size(1)), static_cast<int>(head_dim), static_cast<int>(k_cache.size(2)),
                              static_cast<int>(max_q_len), static_cast<float>(scale), q.stride(0), out.stride(0),
-                             k_cache.size(0), gate_ptr(gate, q, q.size(1) / head_dim), gate_ld(gate), static_cast<int>(window), static_cast<float>(softcap),
-                             static_cast<float>(out_scale), status_ptr(status), cur_stream()),
+                             k_cache.size(0), gate_ptr(gate, q, by_element(gate, q) ? q.size(1) : q.size(1) / head_dim), gate_ld(gate), by_element(gate, q) ? 1 : 0, &mods, status_ptr(status), cur_stream()),
         "attn_prefill");
 }
 
@@ -238,7 +248,7 @@ void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::T
                      const at::Tensor& cu_q, const at::Tensor& ctx_lens, const at::Tensor& block_tables, int64_t max_q_len,
                      double scale, c10::optional<at::Tensor> status, c10::optional<at::Tensor> work,
                      c10::optional<at::Tensor> n_work, int64_t work_items, c10::optional<at::Tensor> gate, int64_t window, double softcap,
-                     double out_scale) {
+                     double out_scale, int64_t chunk, bool sink, c10::optional<at::Tensor> distance) {
   // contiguous paged caches, or a [pages, n_kv, 128, 128] view of matrices with one row per token and all heads in it
   const int64_t token_stride = k_cache.is_contiguous() ? 0 : k_cache.stride(2);
   if (token_stride == 0) check_cache(q, k_cache, v_cache, 128);
@@ -247,7 +257,7 @@ void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::T
              v_cache.sizes() == k_cache.sizes() && v_cache.strides() == k_cache.strides() && k_cache.stride(3) == 1 && k_cache.stride(1) == 128 &&
              k_cache.stride(0) == 128 * token_stride && token_stride >= 128 * k_cache.size(1),
          "attn_prefill_tc: strided keys and values must have one row per token with the heads side by side");
-  const bool gate_elems = gate.has_value() && gate->dim() == 2 && gate->size(1) == q.size(1);
+  const bool gate_elems = by_element(gate, q);
   if (work.has_value()) {
     need(work->is_cuda() && work->scalar_type() == at::kInt && work->is_contiguous() && work->numel() >= 2 * work_items, "attn_prefill_tc: work must be CUDA int32 [items, 2]");
     if (n_work.has_value()) need(n_work->is_cuda() && n_work->scalar_type() == at::kInt && n_work->numel() >= 1, "attn_prefill_tc: n_work must be a CUDA int32 scalar");
@@ -259,6 +269,7 @@ void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::T
   const int batch = static_cast<int>(ctx_lens.numel());
   need(cu_q.numel() == batch + 1 && block_tables.size(0) == batch, "attention: metadata batch mismatch");
   c10::cuda::CUDAGuard g(q.device());
+  const B2AttnMods mods = attn_mods(window, softcap, out_scale, chunk, sink, distance, q.size(1) / 128);
   check(b2_attn_prefill_tc_bf16(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), cu_q.data_ptr<int32_t>(),
                                 ctx_lens.data_ptr<int32_t>(), block_tables.data_ptr<int32_t>(), batch,
                                 static_cast<int>(block_tables.size(1)), static_cast<int>(q.size(1) / 128),
@@ -267,14 +278,14 @@ void attn_prefill_tc(const at::Tensor& q, const at::Tensor& k_cache, const at::T
                                 work.has_value() ? work->data_ptr<int32_t>() : nullptr,
                                 work.has_value() && n_work.has_value() ? n_work->data_ptr<int32_t>() : nullptr,
                                 static_cast<int>(work_items), gate_ptr(gate, q, gate_elems ? q.size(1) : q.size(1) / 128), gate_ld(gate), gate_elems ? 1 : 0,
-                                static_cast<int>(window), static_cast<float>(softcap), static_cast<float>(out_scale), status_ptr(status), cur_stream()),
+                                &mods, status_ptr(status), cur_stream()),
         "attn_prefill_tc");
 }
 
 void attn_decode(const at::Tensor& q, const at::Tensor& k_cache, const at::Tensor& v_cache, at::Tensor& out,
                  const at::Tensor& ctx_lens, const at::Tensor& block_tables, c10::optional<at::Tensor> workspace,
                  int64_t head_dim, int64_t num_splits, double scale, c10::optional<at::Tensor> status,
-                 c10::optional<at::Tensor> counters, c10::optional<at::Tensor> gate, int64_t window, double softcap, double out_scale) {
+                 c10::optional<at::Tensor> counters, c10::optional<at::Tensor> gate, int64_t window, double softcap, double out_scale, int64_t chunk, bool sink, c10::optional<at::Tensor> distance) {
   check_cache(q, k_cache, v_cache, head_dim);
   need(out.dim() == 2 && out.stride(1) == 1 && is_bf16(out) && out.size(0) == q.size(0), "attention: bad out");
   need(ctx_lens.scalar_type() == at::kInt && block_tables.scalar_type() == at::kInt && block_tables.dim() == 2 && block_tables.is_contiguous(), "attention: metadata must be contiguous int32");
@@ -294,12 +305,12 @@ void attn_decode(const at::Tensor& q, const at::Tensor& k_cache, const at::Tenso
       cnt = reinterpret_cast<uint32_t*>(counters->data_ptr());
   }
   c10::cuda::CUDAGuard g(q.device());
+  const B2AttnMods mods = attn_mods(window, softcap, out_scale, chunk, sink, distance, n_q);
   check(b2_attn_decode_bf16(q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), ctx_lens.data_ptr<int32_t>(),
                             block_tables.data_ptr<int32_t>(), ws, batch, static_cast<int>(block_tables.size(1)), n_q,
                             static_cast<int>(k_cache.size(1)), static_cast<int>(head_dim), static_cast<int>(k_cache.size(2)),
                             static_cast<int>(num_splits), static_cast<float>(scale), q.stride(0), out.stride(0),
-                            k_cache.size(0), cnt, gate_ptr(gate, q, n_q), gate_ld(gate), static_cast<int>(window), static_cast<float>(softcap),
-                            static_cast<float>(out_scale), status_ptr(status), cur_stream()),
+                            k_cache.size(0), cnt, gate_ptr(gate, q, by_element(gate, q) ? q.size(1) : n_q), gate_ld(gate), by_element(gate, q) ? 1 : 0, &mods, status_ptr(status), cur_stream()),
         "attn_decode");
 }
 
@@ -368,15 +379,15 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("top_p") = py::none(), py::arg("uniforms") = py::none(), py::arg("seed") = 0, py::arg("step") = 0);
   m.def("attn_prefill", &attn_prefill, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("cu_q"),
         py::arg("ctx_lens"), py::arg("block_tables"), py::arg("head_dim"), py::arg("max_q_len"), py::arg("scale"),
-        py::arg("status") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0);
+        py::arg("status") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0, py::arg("chunk") = 0, py::arg("sink") = false, py::arg("distance") = py::none());
   m.def("gemm_bf16_pair", &gemm_bf16_pair, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("epilogue") = 0, py::arg("bn") = 256, py::arg("status") = py::none(), py::arg("act") = py::none());
   m.def("attn_prefill_tc", &attn_prefill_tc, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("cu_q"),
         py::arg("ctx_lens"), py::arg("block_tables"), py::arg("max_q_len"), py::arg("scale"),
         py::arg("status") = py::none(), py::arg("work") = py::none(), py::arg("n_work") = py::none(), py::arg("work_items") = 0,
-        py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0);
+        py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0, py::arg("chunk") = 0, py::arg("sink") = false, py::arg("distance") = py::none());
   m.def("attn_decode", &attn_decode, py::arg("q"), py::arg("k_cache"), py::arg("v_cache"), py::arg("out"), py::arg("ctx_lens"),
         py::arg("block_tables"), py::arg("workspace"), py::arg("head_dim"), py::arg("num_splits"), py::arg("scale"),
-        py::arg("status") = py::none(), py::arg("counters") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0);
+        py::arg("status") = py::none(), py::arg("counters") = py::none(), py::arg("gate") = py::none(), py::arg("window") = 0, py::arg("softcap") = 0.0, py::arg("out_scale") = 1.0, py::arg("chunk") = 0, py::arg("sink") = false, py::arg("distance") = py::none());
   m.def("gemm_bf16", &gemm_bf16, py::arg("x"), py::arg("w"), py::arg("y"), py::arg("residual") = py::none(),
         py::arg("epilogue") = 0, py::arg("config") = 0, py::arg("workspace") = py::none(), py::arg("status") = py::none(), py::arg("act") = py::none());
   m.def("gemm_workspace_bytes", [](int M, int N, int K) { return b2_gemm_workspace_bytes(M, N, K); });

@@ -64,14 +64,25 @@ int b2_sample(const void* logits, int is_bf16, int64_t* ids, const float* temper
 // q/out: [T, n_q, D]; cache: [num_pages, n_kv, page_size, D]; cu_q: [B+1] query offsets; ctx_lens: [B]
 // total context (cached prefix + this chunk); block_tables: [B, max_blocks]. D == 64, 128 or 256.
 // `gate` (may be null), in this and the two kernels below: bf16 [T, n_q] with row stride `gate_stride`; head h of query
-// row t is multiplied by sigmoid(gate[t, h]) before it is rounded. `window`, in all three: positions a row sees, its own
-// included (<= 0: all of them); `softcap`: scores become softcap * tanh(score / softcap) (<= 0: they do not); `out_scale`:
-// factor of the result.
+// row t is multiplied by sigmoid(gate[t, h]) before it is rounded; with gate_elems it is [T, n_q * D], one logit per element.
+// `mods` (may be null), in all three, in this order on a score:
+//   softcap    it becomes softcap * tanh(score / softcap) (<= 0: it does not)
+//   distance   f32 [2, n_q] r1, r2 (may be null): r1_h ln(1 + r2_h d) is taken off, d positions from query to key
+//   window     positions a row sees, its own included (<= 0: all of them)
+//   chunk      a row sees positions j with floor(j / chunk) that of its own only (<= 0: all of them)
+//   sink       one more score, zero, takes part in the softmax and has no value
+//   out_scale  factor of the result
+struct B2AttnMods {
+  int32_t window, chunk;
+  float softcap, out_scale;
+  const float* distance;
+  int32_t sink;
+};
 int b2_attn_prefill_bf16(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* cu_q,
                          const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                          int n_kv, int head_dim, int page_size, int max_q_len, float scale, int64_t q_stride,
-                         int64_t out_stride, int64_t num_pages, const void* gate, int64_t gate_stride, int window,
-                         float softcap, float out_scale, b2::Status* status, cudaStream_t stream);
+                         int64_t out_stride, int64_t num_pages, const void* gate, int64_t gate_stride, int gate_elems,
+                         const struct B2AttnMods* mods, b2::Status* status, cudaStream_t stream);
 // bf16 GEMM on CTA pairs (tcgen05 cta_group::2, 256 x 256 tiles; csrc/kernels/gemm_bf16_pair.cu). Epilogue NONE, SWIGLU
 // or RELU2.
 int b2_gemm_bf16_pair(const void* x, const void* w, void* y, int M, int N, int K, int64_t ldx, int64_t ldw, int64_t ldy,
@@ -79,12 +90,11 @@ int b2_gemm_bf16_pair(const void* x, const void* w, void* y, int M, int N, int K
 // The same attention on tcgen05 / TMEM (csrc/kernels/attention_tc.cu): head_dim 128 and page_size 128 only.
 // q_rows = rows of the q matrix (for the tensor map). token_stride 0: paged caches; otherwise keys and values lie in
 // matrices with one row per token (elements between rows), all heads side by side, and a page is 128 such rows.
-// gate_elems: the gate has one logit per output element, [T, n_q * 128].
 int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const void* v_cache, void* out, const int32_t* cu_q,
                             const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                             int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
                             int64_t num_pages, int64_t token_stride, const int32_t* work, const int32_t* n_work, int work_items,
-                            const void* gate, int64_t gate_stride, int gate_elems, int window, float softcap, float out_scale,
+                            const void* gate, int64_t gate_stride, int gate_elems, const struct B2AttnMods* mods,
                             b2::Status* status, cudaStream_t stream);
 // One query token per sequence, split over the KV length. workspace: f32, size from b2_attn_decode_workspace.
 // `counters` (may be null): u32 [batch * n_kv], zero before the first use and left at zero by every launch; with it
@@ -94,7 +104,7 @@ int b2_attn_decode_bf16(const void* q, const void* k_cache, const void* v_cache,
                         const int32_t* block_tables, float* workspace, int batch, int max_blocks, int n_q, int n_kv,
                         int head_dim, int page_size, int num_splits, float scale, int64_t q_stride,
                         int64_t out_stride, int64_t num_pages, uint32_t* counters, const void* gate, int64_t gate_stride,
-                        int window, float softcap, float out_scale, b2::Status* status, cudaStream_t stream);
+                        int gate_elems, const struct B2AttnMods* mods, b2::Status* status, cudaStream_t stream);
 int64_t b2_attn_decode_counter_bytes(int batch, int n_kv);
 int64_t b2_attn_decode_workspace(int batch, int n_q, int head_dim, int num_splits);
 // MLA decode with absorbed weights: q_lat [B, H, 512], q_rope [B, H, 64]; cache [num_pages, page, 576]

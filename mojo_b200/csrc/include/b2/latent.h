@@ -48,10 +48,10 @@ int b2_head_gemm_bf16(const void* x, const void* w, void* y, const void* gate, i
 // on entry; ids from `experts` on are not counted).
 int b2_moe_route(const float* logits, int64_t ld, const float* correction, float* weights, int32_t* ids, int32_t* place, int32_t* counts, int rows,
                  int experts, int identity, int top, int groups, int keep, int scoring, int norm_top, float scale, cudaStream_t stream);
-// Rows sorted by expert: xs[slot[t, j]] = x[t] (ids from `experts` on get slot -1 and no row). Also lists the tiles of at most `bn` rows of one expert as
+// Rows sorted by expert: xs[slot[t, j]] = x[t], times weights[t, j] where `weights` (may be null) is given (ids from `experts` on get slot -1 and no row). Also lists the tiles of at most `bn` rows of one expert as
 // {expert, first row, rows, 0} in tiles (room for experts + rows * top / bn entries), their number in n_tiles[0], and
 // leaves counts (and the ticket word counts[experts]) at zero.
-int b2_moe_gather(const void* x, const int32_t* ids, const int32_t* place, int32_t* counts, int32_t* slot, void* xs, int32_t* tiles, int32_t* n_tiles,
+int b2_moe_gather(const void* x, const int32_t* ids, const int32_t* place, const float* weights, int32_t* counts, int32_t* slot, void* xs, int32_t* tiles, int32_t* n_tiles,
                   int rows, int experts, int top, int width, int bn, int f32, b2::Status* status, cudaStream_t stream);
 // y[r] = x[r] W[e]^T for the rows of every listed tile; w [experts, n, k]. `epilogue` NONE, RELU2 or SWIGLU (gate and up rows
 // interleaved in blocks of 16, y then has n / 2 columns).

@@ -62,16 +62,50 @@ __device__ __forceinline__ uint32_t tile_addr(uint32_t base, int row, int chunk)
   }
 }
 
-// Optional per-head output gate: head h of query row t is multiplied by sigmoid(logits[t * stride + h]) before it is
-// rounded. No gate when `logits` is null.
+// Optional output gate: head h of query row t is multiplied by sigmoid(logits[t * stride + h]) before it is rounded, or with
+// `elems` its column c by sigmoid(logits[t * stride + h * D + c]). No gate when `logits` is null.
 struct HeadGate {
   const __nv_bfloat16* logits;
   int64_t stride;
+  int elems;
+  __device__ __forceinline__ static float sigmoid(float z) { return 1.0f / (1.0f + ptx::ex2(-z * ptx::kLog2e)); }
   __device__ __forceinline__ float factor(int64_t row, int head) const {
-    if (logits == nullptr) return 1.0f;
-    return 1.0f / (1.0f + ptx::ex2(-__bfloat162float(logits[row * stride + head]) * ptx::kLog2e));
+    if (logits == nullptr || elems) return 1.0f;
+    return sigmoid(__bfloat162float(logits[row * stride + head]));
+  }
+  template <int D>
+  __device__ __forceinline__ float elem(int64_t row, int head, int col) const {
+    if (!elems) return 1.0f;
+    return sigmoid(__bfloat162float(logits[row * stride + static_cast<int64_t>(head) * D + col]));
+  }
+  template <int D>      // two neighbouring columns, the first of them even
+  __device__ __forceinline__ float2 elem2(int64_t row, int head, int col) const {
+    if (!elems) return make_float2(1.0f, 1.0f);
+    const uint32_t z = *reinterpret_cast<const uint32_t*>(logits + row * stride + static_cast<int64_t>(head) * D + col);
+    return make_float2(sigmoid(ptx::bf16_lo(z)), sigmoid(ptx::bf16_hi(z)));
   }
 };
+
+// What a thread needs of a layer's modifications for its two rows of an MMA tile: the first visible positions and the heads'
+// factors of the distance bias.
+struct RowMods {
+  int first[2];
+  float2 bias[2];
+};
+
+__device__ __forceinline__ RowMods row_mods(const ScoreMods& mods, int max_lo, int max_hi, int head_lo, int head_hi) {
+  RowMods r{{max_lo >= 0 ? mods.first(max_lo) : 0, max_hi >= 0 ? mods.first(max_hi) : 0}, {}};
+  if (mods.bias != nullptr) {
+    r.bias[0] = mods.head_bias(head_lo);
+    r.bias[1] = mods.head_bias(head_hi);
+  }
+  return r;
+}
+// A row's softmax that has seen nothing but the sink. The four lanes of a row hold parts of its sum.
+__device__ __forceinline__ void sink_start(float (&m)[2], float (&l)[2], int lane) {
+  m[0] = m[1] = 0.0f;
+  l[0] = l[1] = (lane & 3) == 0 ? 1.0f : 0.0f;
+}
 
 struct PagedKV {
   const __nv_bfloat16* k;
@@ -108,12 +142,12 @@ __device__ __forceinline__ void load_kv_tile(const PagedKV& kv, int kv0, uint32_
 
 // One warp: S = Q K^T on a BN-token tile, online softmax, O += P V.
 //   qf      Q fragments of this warp's 16 rows (D/16 k-steps x 4 regs)
-//   max_lo  highest KV position visible to row g, max_hi to row g + 8 (causal + context limit); MODS: also at least
-//           max_lo - window + 1, and the scores may be capped
+//   max_lo  highest KV position visible to row g, max_hi to row g + 8 (causal + context limit: a row's own position); MODS: also
+//           at least rm.first, and the scores may be capped and biased
 template <int D, int BN, int TROWS = 0, bool MODS = false>
 __device__ __forceinline__ void warp_attend(const uint32_t (&qf)[D / 16][4], uint32_t k_sm, uint32_t v_sm, int kv0,
                                             int max_lo, int max_hi, float scale_log2, float (&o)[D / 8][4],
-                                            float (&m)[2], float (&l)[2], int lane, const ScoreMods& mods) {
+                                            float (&m)[2], float (&l)[2], int lane, const ScoreMods& mods, const RowMods& rm) {
   constexpr int NT_S = BN / 8;
   float s[NT_S][4];
 #pragma unroll
@@ -130,19 +164,31 @@ __device__ __forceinline__ void warp_attend(const uint32_t (&qf)[D / 16][4], uin
       mma_bf16(s[2 * jp + 1], qf[kk], b2, b3);
     }
   }
-  if constexpr (MODS) mods.scores<NT_S * 4>(&s[0][0], scale_log2);
-  // mask + running max
   const int t = lane & 3;
+  if constexpr (MODS) {
+    mods.scores<NT_S * 4>(&s[0][0], scale_log2);
+    if (mods.bias != nullptr) {
+#pragma unroll
+      for (int j = 0; j < NT_S; ++j) {
+        const int lo = max_lo - kv0 - j * 8 - 2 * t, hi = max_hi - kv0 - j * 8 - 2 * t;
+        s[j][0] -= ScoreMods::distance(rm.bias[0], lo);
+        s[j][1] -= ScoreMods::distance(rm.bias[0], lo - 1);
+        s[j][2] -= ScoreMods::distance(rm.bias[1], hi);
+        s[j][3] -= ScoreMods::distance(rm.bias[1], hi - 1);
+      }
+    }
+  }
+  // mask + running max
   float mx_lo = m[0], mx_hi = m[1];
 #pragma unroll
   for (int j = 0; j < NT_S; ++j) {
     const int col = kv0 + j * 8 + 2 * t;
     if constexpr (MODS) {
-      const int lo = max_lo - mods.window, hi = max_hi - mods.window;
-      s[j][0] = col <= max_lo && col > lo ? s[j][0] : -INFINITY;
-      s[j][1] = col + 1 <= max_lo && col + 1 > lo ? s[j][1] : -INFINITY;
-      s[j][2] = col <= max_hi && col > hi ? s[j][2] : -INFINITY;
-      s[j][3] = col + 1 <= max_hi && col + 1 > hi ? s[j][3] : -INFINITY;
+      const int lo = rm.first[0], hi = rm.first[1];
+      s[j][0] = col <= max_lo && col >= lo ? s[j][0] : -INFINITY;
+      s[j][1] = col + 1 <= max_lo && col + 1 >= lo ? s[j][1] : -INFINITY;
+      s[j][2] = col <= max_hi && col >= hi ? s[j][2] : -INFINITY;
+      s[j][3] = col + 1 <= max_hi && col + 1 >= hi ? s[j][3] : -INFINITY;
     } else {
       s[j][0] = col <= max_lo ? s[j][0] * scale_log2 : -INFINITY;
       s[j][1] = col + 1 <= max_lo ? s[j][1] * scale_log2 : -INFINITY;
@@ -263,12 +309,15 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
   const int last_tok = min(q_len - 1, (row_base + BM - 1) / group);
   const int kv_end = min(ctx, past + last_tok + 1);
   const int n_tiles = (kv_end + BN - 1) / BN;
-  const int first_tile = MODS ? max(0, past + row_base / group - mods.window + 1) / BN : 0;
+  const int first_tile = MODS ? mods.first(past + row_base / group) / BN : 0;
 
   float o[D / 8][4];
 #pragma unroll
   for (int d = 0; d < D / 8; ++d) o[d][0] = o[d][1] = o[d][2] = o[d][3] = 0.0f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.0f, 0.0f};
+  RowMods rm{};
+  if constexpr (MODS) rm = row_mods(mods, max_lo, max_hi, kvh * group + (row0 + g) % group, kvh * group + (row0 + g + 8) % group);
+  if (MODS && mods.sink) sink_start(m, l, lane);
 
   if (first_tile < n_tiles) {
     load_kv_tile<D, BN, 128>(kv, first_tile * BN, kv_sm + (first_tile & 1) * 2 * TILE_BYTES, kv_sm + ((first_tile & 1) * 2 + 1) * TILE_BYTES, threadIdx.x,
@@ -290,7 +339,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
     // a warp whose rows cannot see this tile yet skips the math (causal upper triangle)
     const int warp_max = min(q_len - 1, (row0 + 15) / group) + past;
     if (t * BN <= warp_max && row0 < q_len * group)
-      warp_attend<D, BN, 0, MODS>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane, mods);
+      warp_attend<D, BN, 0, MODS>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane, mods, rm);
     __syncthreads();
   }
   // finalise: O / l
@@ -310,7 +359,8 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(
     if constexpr (MODS) inv *= mods.out_scale;
 #pragma unroll
     for (int d = 0; d < D / 8; ++d) {
-      const uint32_t pk = ptx::pack_bf16x2(o[d][half * 2] * inv, o[d][half * 2 + 1] * inv);
+      const float2 f = gate.elem2<D>(tok0 + tok, kvh * group + hg, d * 8 + 2 * t4);
+      const uint32_t pk = ptx::pack_bf16x2(o[d][half * 2] * inv * f.x, o[d][half * 2 + 1] * inv * f.y);
       *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * t4) = pk;
     }
   }
@@ -342,7 +392,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
   const uint32_t kv_sm = q_sm + 16 * D * 2;
 
   // KV range of this split, in whole tiles
-  const int tiles_total = (ctx + BN - 1) / BN, first_tile = MODS ? max(0, ctx - mods.window) / BN : 0;
+  const int tiles_total = (ctx + BN - 1) / BN, first_tile = MODS && ctx > 0 ? mods.first(ctx - 1) / BN : 0;
   const int tiles_per_split = (tiles_total - first_tile + num_splits - 1) / num_splits;
   const int tile_begin = first_tile + split * tiles_per_split;
   const int tile_end = min(tiles_total, tile_begin + tiles_per_split);
@@ -358,6 +408,9 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
   const int g = lane >> 2;
   const int max_lo = g < group ? ctx - 1 : -1;
   const int max_hi = g + 8 < group ? ctx - 1 : -1;
+  RowMods rm{};
+  if constexpr (MODS) rm = row_mods(mods, max_lo, max_hi, kvh * group + min(g, group - 1), kvh * group + min(g + 8, group - 1));
+  if (MODS && mods.sink && split == 0 && warp == 0) sink_start(m, l, lane);
 
   int t = tile_begin + warp;
   if (t < tile_end) {
@@ -376,7 +429,7 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
     }
     __syncwarp();
     const uint32_t kb = kv_sm + stage * 2 * TILE_BYTES;
-    warp_attend<D, BN, 0, MODS>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane, mods);
+    warp_attend<D, BN, 0, MODS>(qf, kb, kb + TILE_BYTES, t * BN, max_lo, max_hi, scale_log2, o, m, l, lane, mods, rm);
     __syncwarp();
     stage ^= 1;
   }
@@ -428,8 +481,10 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(
       const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head) * (MODS ? mods.out_scale : 1.0f);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D + cs;
 #pragma unroll
-      for (int c = 0; c < COLS_PER_THREAD; c += 2)
-        *reinterpret_cast<uint32_t*>(dst + c) = ptx::pack_bf16x2(acc[c] * inv, acc[c + 1] * inv);
+      for (int c = 0; c < COLS_PER_THREAD; c += 2) {
+        const float2 f = gate.elem2<D>(seq, head, cs + c);
+        *reinterpret_cast<uint32_t*>(dst + c) = ptx::pack_bf16x2(acc[c] * inv * f.x, acc[c + 1] * inv * f.y);
+      }
     } else {
       float* dst = workspace + ((static_cast<int64_t>(seq) * n_q + head) * num_splits + split) * RS;
 #pragma unroll
@@ -471,7 +526,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
   const int ctx = ctx_lens[seq];
   const int32_t* table = block_tables + static_cast<int64_t>(seq) * max_blocks;
 
-  const int tiles_total = (ctx + BN - 1) / BN, first_tile = MODS ? max(0, ctx - mods.window) / BN : 0;
+  const int tiles_total = (ctx + BN - 1) / BN, first_tile = MODS && ctx > 0 ? mods.first(ctx - 1) / BN : 0;
   const int tiles_per_split = (tiles_total - first_tile + num_splits - 1) / num_splits;
   const int tile_begin = first_tile + split * tiles_per_split;
   const int tile_end = min(tiles_total, tile_begin + tiles_per_split);
@@ -515,6 +570,9 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
   const int g = lane >> 2;
   const int max_lo = g < group ? ctx - 1 : -1;
   const int max_hi = g + 8 < group ? ctx - 1 : -1;
+  RowMods rm{};
+  if constexpr (MODS) rm = row_mods(mods, max_lo, max_hi, kvh * group + min(g, group - 1), kvh * group + min(g + 8, group - 1));
+  if (MODS && mods.sink && split == 0) sink_start(m, l, lane);
 
   bool ok = true;
   for (int i = 0; i < n_tiles; ++i) {
@@ -538,7 +596,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
         }
       __syncwarp();
     }
-    warp_attend<D, BN, BN, MODS>(qf, kb, kb + TILE_BYTES, kv0, max_lo, max_hi, scale_log2, o, m, l, lane, mods);
+    warp_attend<D, BN, BN, MODS>(qf, kb, kb + TILE_BYTES, kv0, max_lo, max_hi, scale_log2, o, m, l, lane, mods, rm);
     __syncwarp();
   }
   if (!ok) {
@@ -560,8 +618,10 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
       const float inv = (l[half] > 0.0f ? 1.0f / l[half] : 0.0f) * gate.factor(seq, head) * (MODS ? mods.out_scale : 1.0f);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
-      for (int d = 0; d < D / 8; ++d)
-        *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * t4) = ptx::pack_bf16x2(o[d][half * 2] * inv, o[d][half * 2 + 1] * inv);
+      for (int d = 0; d < D / 8; ++d) {
+        const float2 f = gate.elem2<D>(seq, head, d * 8 + 2 * t4);
+        *reinterpret_cast<uint32_t*>(dst + d * 8 + 2 * t4) = ptx::pack_bf16x2(o[d][half * 2] * inv * f.x, o[d][half * 2 + 1] * inv * f.y);
+      }
     } else {
       float* dst = workspace + ((static_cast<int64_t>(seq) * n_q + head) * num_splits + split) * (D + 2);
 #pragma unroll
@@ -604,7 +664,7 @@ __global__ void __launch_bounds__(32) attn_decode_tma_kernel(
       const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head) * (MODS ? mods.out_scale : 1.0f);
       __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
-      for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv);
+      for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv * gate.elem<D>(seq, head, c * 32 + lane));
     }
   }
 }
@@ -636,7 +696,12 @@ __global__ void attn_decode_reduce_kernel(const float* __restrict__ workspace, _
   const float inv = (ll > 0.0f ? 1.0f / ll : 0.0f) * gate.factor(seq, head) * out_scale;
   __nv_bfloat16* dst = out + static_cast<int64_t>(seq) * out_stride + static_cast<int64_t>(head) * D;
 #pragma unroll
-  for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv);
+  for (int c = 0; c < D / 32; ++c) dst[c * 32 + lane] = __float2bfloat16(acc[c] * inv * gate.elem<D>(seq, head, c * 32 + lane));
+}
+
+// Gates by element are read in pairs of columns.
+bool gate_fits(const void* gate, int64_t stride, int elems) {
+  return gate == nullptr || !elems || (stride % 2 == 0 && (reinterpret_cast<uintptr_t>(gate) & 3) == 0);
 }
 
 template <int D>
@@ -702,15 +767,15 @@ extern "C" int b2_attn_prefill_bf16(const void* q, const void* k_cache, const vo
                                     const int32_t* cu_q, const int32_t* ctx_lens, const int32_t* block_tables,
                                     int batch, int max_blocks, int n_q, int n_kv, int head_dim, int page_size,
                                     int max_q_len, float scale, int64_t q_stride, int64_t out_stride,
-                                    int64_t num_pages, const void* gate, int64_t gate_stride, int window, float softcap,
-                                    float out_scale, Status* status, cudaStream_t stream) {
+                                    int64_t num_pages, const void* gate, int64_t gate_stride, int gate_elems,
+                                    const B2AttnMods* am, Status* status, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
-  if (n_kv <= 0 || n_q % n_kv != 0 || q_stride % 8 != 0 || out_stride % 2 != 0) return -kBadArgument;
+  if (n_kv <= 0 || n_q % n_kv != 0 || q_stride % 8 != 0 || out_stride % 2 != 0 || !gate_fits(gate, gate_stride, gate_elems)) return -kBadArgument;
   const int group = n_q / n_kv;
   const dim3 grid((max_q_len * group + 63) / 64, n_kv, batch);
   const float scale_log2 = scale * ptx::kLog2e;
-  const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride};
-  const ScoreMods mods = make_score_mods(window, softcap, out_scale, scale);
+  const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride, gate != nullptr ? gate_elems : 0};
+  const ScoreMods mods = make_score_mods(am, n_q, scale);
 #define B2_PREFILL(D_)                                                                                                          \
   return launch_prefill<D_>(grid, stream, static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_cache),    \
                             static_cast<const __nv_bfloat16*>(v_cache), static_cast<__nv_bfloat16*>(out), cu_q, ctx_lens,      \
@@ -736,15 +801,16 @@ extern "C" int b2_attn_decode_bf16(const void* q, const void* k_cache, const voi
                                    const int32_t* ctx_lens, const int32_t* block_tables, float* workspace, int batch,
                                    int max_blocks, int n_q, int n_kv, int head_dim, int page_size, int num_splits,
                                    float scale, int64_t q_stride, int64_t out_stride, int64_t num_pages,
-                                   uint32_t* counters, const void* gate, int64_t gate_stride, int window, float softcap,
-                                   float out_scale, Status* status, cudaStream_t stream) {
+                                   uint32_t* counters, const void* gate, int64_t gate_stride, int gate_elems,
+                                   const B2AttnMods* am, Status* status, cudaStream_t stream) {
   if (batch <= 0) return 0;
-  if (n_kv <= 0 || n_q % n_kv != 0 || n_q / n_kv > 16 || q_stride % 8 != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr))
+  if (n_kv <= 0 || n_q % n_kv != 0 || n_q / n_kv > 16 || q_stride % 8 != 0 || num_splits < 1 || (num_splits > 1 && workspace == nullptr) ||
+      !gate_fits(gate, gate_stride, gate_elems))
     return -kBadArgument;
   const dim3 grid(num_splits, n_kv, batch);
   const float scale_log2 = scale * ptx::kLog2e;
-  const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride};
-  const ScoreMods mods = make_score_mods(window, softcap, out_scale, scale);
+  const HeadGate hg{static_cast<const __nv_bfloat16*>(gate), gate_stride, gate != nullptr ? gate_elems : 0};
+  const ScoreMods mods = make_score_mods(am, n_q, scale);
   auto qp = static_cast<const __nv_bfloat16*>(q);
   auto op = static_cast<__nv_bfloat16*>(out);
 #define B2_DECODE_TMA(D_)                                                                                                             \

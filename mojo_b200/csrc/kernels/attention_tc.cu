@@ -51,7 +51,8 @@ constexpr int kOffBar = kOffV + kStages * kTileBytes;      // 192 KB
 constexpr int kNumBars = 1 + 4 * kStages + 2 + 2 + 2 + 2 + 1;  // q_full, k/v full+empty, s full/empty, p full/empty, o full/empty, drain
 constexpr int kOffAlpha = kOffBar + 8 * kNumBars + 16;     // float [2][2][128]: partial row maxima
 constexpr int kOffL = kOffAlpha + 4 * kTile * 4;           // float [2][128]
-constexpr int kOffFlags = kOffL + 2 * kTile * 4;           // tmem holder, fail flag
+constexpr int kOffBias = kOffL + 2 * kTile * 4;            // float [2][256]: distance biases of a tile
+constexpr int kOffFlags = kOffBias + 2 * 256 * 4;          // tmem holder, fail flag
 constexpr int kSmemAttn = kOffFlags + 16 + 1024;           // + alignment slack
 
 struct AttnTcParams {
@@ -92,8 +93,8 @@ __device__ __forceinline__ uint64_t smem_desc(uint32_t addr, uint32_t lbo_bytes,
   return d;
 }
 
-// MODS: a window, a soft cap or a factor on the result (AttnTcParams::mods). Tiles before the window of the first row are
-// never visited.
+// MODS: AttnTcParams::mods. Tiles before the first position that the first row sees are never visited. A tile's distance bias
+// depends on 255 distances only: they wait in shared memory, written while the tile before is worked on.
 template <bool MODS>
 __global__ void __launch_bounds__(kThreadsAttn, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
@@ -111,7 +112,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
   const int ctx = prm.ctx_lens[seq];
   const int pos0 = ctx - q_len + qt * kTile;              // absolute position of this tile's first query row
   const int rows = min(kTile, q_len - qt * kTile);
-  const int first_tile = MODS ? max(0, pos0 - prm.mods.window + 1) / kTile : 0;
+  const int first_tile = MODS ? prm.mods.first(pos0) / kTile : 0;
   const int n_tiles = min((pos0 + rows + kTile - 1) / kTile, (ctx + kTile - 1) / kTile) - first_tile;  // KV tiles with a visible token
   const int kvh = head / (prm.n_q / prm.n_kv);
 
@@ -272,7 +273,22 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     const uint32_t lane_bits = static_cast<uint32_t>(quarter * 32) << 16;
     float* pmax = alpha_ring;               // [2 tiles in flight][2 halves][128 rows]
     const float scale_log2 = MODS ? 1.0f : prm.scale_log2;      // MODS: the scores come scaled
-    float m_run = -INFINITY, l_part = 0.0f, alpha_prev = 1.0f;
+    const bool sink = MODS && prm.mods.sink;                    // a score of zero that has been seen already
+    float m_run = sink ? 0.0f : -INFINITY, l_part = sink && g == 0 ? 1.0f : 0.0f, alpha_prev = 1.0f;
+    const int first_seen = MODS ? prm.mods.first(qpos) : 0, first_last = MODS ? prm.mods.first(pos0 + kTile - 1) : 0;
+    const bool biased = MODS && prm.mods.bias != nullptr;
+    float* bias_sm = reinterpret_cast<float*>(smem + kOffBias);
+    float2 head_bias = make_float2(0.0f, 0.0f);
+    // entry i of tile j: distance (row 0's to the tile's last column) + i; a row and column meet at r + 127 - column
+    const auto fill_bias = [&](int j) {
+      const int i = static_cast<int>(threadIdx.x) - 64;
+      bias_sm[(j & 1) * 256 + i] = ScoreMods::distance(head_bias, max(0, pos0 - (first_tile + j) * kTile - (kTile - 1) + i));
+    };
+    if (biased) {
+      head_bias = prm.mods.head_bias(head);
+      fill_bias(0);
+      ptx::named_barrier_sync(5, 256);
+    }
     float o[64];
 #pragma unroll
     for (int i = 0; i < 64; ++i) o[i] = 0.0f;
@@ -328,11 +344,16 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       const int kv0 = (first_tile + j) * kTile + g * 64;
       if constexpr (MODS) {
         prm.mods.scores<64>(s, prm.scale_log2);
-        if (kv0 <= pos0 + kTile - 1 - prm.mods.window) {   // some row of this tile is past some of these columns
-          const int lo = qpos - prm.mods.window;
+        if (biased) {
+          const float* b = bias_sm + (j & 1) * 256 + r + kTile - 1 - g * 64;
+#pragma unroll
+          for (int c = 0; c < 64; ++c) s[c] -= b[-c];
+          if (j + 1 < n_tiles) fill_bias(j + 1);
+        }
+        if (kv0 < first_last) {                            // some row of this tile is past some of these columns
 #pragma unroll
           for (int c = 0; c < 64; ++c)
-            if (kv0 + c <= lo) s[c] = -INFINITY;
+            if (kv0 + c < first_seen) s[c] = -INFINITY;
         }
       }
       if (kv0 + 63 > pos0) {                             // some row of this tile masks some of these columns
@@ -435,7 +456,7 @@ extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const
                                        const int32_t* ctx_lens, const int32_t* block_tables, int batch, int max_blocks, int n_q,
                                        int n_kv, int max_q_len, float scale, int64_t q_rows, int64_t q_stride, int64_t out_stride,
                                        int64_t num_pages, int64_t token_stride, const int32_t* work, const int32_t* n_work, int work_items,
-                                       const void* gate, int64_t gate_stride, int gate_elems, int window, float softcap, float out_scale,
+                                       const void* gate, int64_t gate_stride, int gate_elems, const B2AttnMods* mods,
                                        Status* status, cudaStream_t stream) {
   if (batch <= 0 || max_q_len <= 0) return 0;
   if (work != nullptr && work_items <= 0) return 0;
@@ -473,7 +494,7 @@ extern "C" int b2_attn_prefill_tc_bf16(const void* q, const void* k_cache, const
   prm.page_rows = by_token ? kTile : n_kv * kTile;
   prm.head_rows = by_token ? 0 : kTile;
   prm.head_cols = by_token ? kD : 0;
-  prm.mods = make_score_mods(window, softcap, out_scale, scale);
+  prm.mods = make_score_mods(mods, n_q, scale);
   static DeviceOnce attr_once[2];
   auto kern = prm.mods.plain() ? attn_prefill_tc_kernel<false> : attn_prefill_tc_kernel<true>;
   if (const int rc = attr_once[prm.mods.plain()].max_smem(kern, kSmemAttn)) return rc;

@@ -1,4 +1,4 @@
-// Gated delta rule with one decay per key channel. State S [dim, vdim] per head, all of it in f32:
+// Gated delta rule with one decay per key channel, or one per head. State S [dim, vdim] per head, all of it in f32:
 //   S <- g * S,  u = beta (v - S^T k),  S <- S + k u^T,  o = S^T q
 // Three kernels:
 //   prep    every row and head at once: short convolution and silu of q, k, v, unit norms, decays, step sizes, and the few
@@ -30,6 +30,10 @@ constexpr int kStages = 3;
 constexpr int kCols = 32;        // value columns of a scan CTA
 
 __device__ __forceinline__ float sigmoid(float x) { return ptx::rcp(1.0f + ptx::ex2(-x * ptx::kLog2e)); }
+__device__ __forceinline__ float gate_value(const B2DeltaArgs& a, float z) { return a.gate_silu ? z * sigmoid(z) : sigmoid(z); }
+// The gates of a head in a row.
+template <typename T>
+__device__ __forceinline__ const T* gate_row(const B2DeltaArgs& a, int row, int h) { return static_cast<const T*>(a.gate) + static_cast<int64_t>(row) * a.ld_gate + h * a.vdim; }
 
 // Prepared pairs, f32, head-major so that a run of pairs is one contiguous block. Sequence number s with first row b starts at
 // pair (b + s) / 2, which leaves every sequence room for a last pair that is half empty.
@@ -89,24 +93,34 @@ __global__ void __launch_bounds__(128, TAPS > 0 && NJ == 1 ? 6 : 1) delta_prep_k
 
   float q[NJ][TT][VEC], k[NJ][TT][VEC], g[NJ][TT][VEC];
   const float rate = a.neg_rate[h] * ptx::kLog2e;
+  float head_g[TT];      // one decay for all channels
+  if (a.head_decay) {
+    const float bias = a.dt_bias[h];
+#pragma unroll
+    for (int t = 0; t < TT; ++t) {
+      float z[1] = {0.0f};
+      if (t < n) load_f32<1>(static_cast<const T*>(a.decay) + static_cast<int64_t>(row0 + t) * a.ld_decay + h, z);
+      head_g[t] = ptx::ex2(rate * softplus_fast(z[0] + bias));
+    }
+  }
 #pragma unroll
   for (int j = 0; j < NJ; ++j) {
     const int c = (lane + 32 * j) * VEC;
     if (c < d) {
       conv_rows<T, VEC, TAPS, TT>(src, cr, row0, n, kh * d + c, save_qk, q[j]);
       conv_rows<T, VEC, TAPS, TT>(src, cr, row0, n, ck + kh * d + c, save_qk, k[j]);
-      float bias[VEC];
-      load_f32<VEC>(a.dt_bias + h * d + c, bias);
+      float bias[VEC] = {};
+      if (!a.head_decay) load_f32<VEC>(a.dt_bias + h * d + c, bias);
 #pragma unroll
       for (int t = 0; t < TT; ++t) {
         float z[VEC] = {};
-        if (t < n) load_f32<VEC>(static_cast<const T*>(a.dg) + static_cast<int64_t>(row0 + t) * a.ld_dg + h * d + c, z);
+        if (t < n && !a.head_decay) load_f32<VEC>(static_cast<const T*>(a.decay) + static_cast<int64_t>(row0 + t) * a.ld_decay + h * d + c, z);
 #pragma unroll
         for (int v = 0; v < VEC; ++v) {
           // a row that is not there changes nothing
           q[j][t][v] = t < n ? ptx::silu(q[j][t][v]) : 0.0f;
           k[j][t][v] = t < n ? ptx::silu(k[j][t][v]) : 0.0f;
-          g[j][t][v] = t < n ? ptx::ex2(rate * softplus_fast(z[v] + bias[v])) : 1.0f;
+          g[j][t][v] = t < n ? (a.head_decay ? head_g[t] : ptx::ex2(rate * softplus_fast(z[v] + bias[v]))) : 1.0f;
         }
       }
     } else {
@@ -231,10 +245,14 @@ int launch_prep(const B2DeltaArgs& a, const B2SeqRows& s, bool one_row_each, Sta
   return last_launch_rc();
 }
 
+// Whether rows of four elements can be read at once from every multiple of four on.
+template <typename T>
+bool vec4_rows(const void* p, int64_t ld) { return ld % 4 == 0 && reinterpret_cast<uintptr_t>(p) % (4 * sizeof(T)) == 0; }
+
 template <typename T>
 int dispatch_prep(const B2DeltaArgs& a, const B2SeqRows& s, bool one_row_each, Status* status, cudaStream_t stream) {
   const int m = a.dim > a.vdim ? a.dim : a.vdim;
-  if (a.taps == 4 && a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ld % 4 == 0 && a.ld_dg % 4 == 0) {
+  if (a.taps == 4 && a.dim % 4 == 0 && a.vdim % 4 == 0 && a.ld % 4 == 0 && (a.head_decay || vec4_rows<T>(a.decay, a.ld_decay))) {
     if (m <= 128)
       return one_row_each ? launch_prep<T, 4, 1, 4, 1>(a, s, true, status, stream) : launch_prep<T, 4, 1, 4, 4>(a, s, false, status, stream);
     return launch_prep<T, 4, 2, 4, 2>(a, s, one_row_each, status, stream);
@@ -256,10 +274,10 @@ __device__ __forceinline__ void decode_finish(const B2DeltaArgs& a, int row, int
   if (!owner) return;
   const float r = rsqrtf(ss / static_cast<float>(a.vdim) + a.eps);
   float z[VEC], w[VEC];
-  load_f32<VEC>(static_cast<const T*>(a.dg) + static_cast<int64_t>(row) * a.ld_dg + a.heads * a.dim + h * a.vdim + cg * VEC, z);
+  load_f32<VEC>(gate_row<T>(a, row, h) + cg * VEC, z);
   load_f32<VEC>(a.norm_w + cg * VEC, w);
 #pragma unroll
-  for (int v = 0; v < VEC; ++v) o[v] = o[v] * r * w[v] * sigmoid(z[v]);
+  for (int v = 0; v < VEC; ++v) o[v] = o[v] * r * w[v] * gate_value(a, z[v]);
   store_f32<VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(row) * a.ld_out + static_cast<int64_t>(h) * a.vdim + cg * VEC, o);
 }
 
@@ -461,7 +479,7 @@ __global__ void __launch_bounds__(kDecodeThreads, 2) delta_decode_kernel(const B
 
 template <typename T>
 int dispatch_decode(const B2DeltaArgs& a, const B2SeqRows& s, int n, Status* status, cudaStream_t stream) {
-  const bool v4 = a.vdim % 4 == 0 && a.ld_dg % 4 == 0 && a.ld_out % 4 == 0 && (a.heads * a.dim) % 4 == 0;
+  const bool v4 = a.vdim % 4 == 0 && vec4_rows<T>(a.gate, a.ld_gate) && a.ld_out % 4 == 0;
   const Prepared in = prepared_of(a, s);
   DecodeLayout L{};
   if (v4) {
@@ -634,7 +652,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const B2DeltaArgs a, co
   store_state<P, 4>(state, d, e, col, rg, S);
 }
 
-// out = rms_norm(o) * w * sigmoid(gate) for the rows of sequences >= first: one warp per (row, head).
+// out = rms_norm(o) * w * gate for the rows of sequences >= first: one warp per (row, head).
 template <typename T, int VEC, int NJ>
 __global__ void __launch_bounds__(256) delta_out_kernel(const B2DeltaArgs a, const B2SeqRows sq, int first) {
   ptx::grid_dep_sync();
@@ -643,7 +661,7 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const B2DeltaArgs a, con
   const int row = static_cast<int>(idx / a.heads), h = static_cast<int>(idx % a.heads);
   if (row >= sq.rows || sq.row_seq[row] < first) return;
   const float* o = a.o_raw + (static_cast<int64_t>(row) * a.heads + h) * e;
-  const T* gate = static_cast<const T*>(a.dg) + static_cast<int64_t>(row) * a.ld_dg + a.heads * a.dim + h * e;
+  const T* gate = gate_row<T>(a, row, h);
   T* out = static_cast<T*>(a.out) + static_cast<int64_t>(row) * a.ld_out + static_cast<int64_t>(h) * e;
   float v[NJ][VEC], ss = 0.0f;
 #pragma unroll
@@ -665,7 +683,7 @@ __global__ void __launch_bounds__(256) delta_out_kernel(const B2DeltaArgs a, con
     load_f32<VEC>(gate + c, z);
     load_f32<VEC>(a.norm_w + c, w);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) v[j][i] = v[j][i] * r * w[i] * sigmoid(z[i]);
+    for (int i = 0; i < VEC; ++i) v[j][i] = v[j][i] * r * w[i] * gate_value(a, z[i]);
     store_f32<VEC>(out + c, v[j]);
   }
 }
@@ -696,7 +714,7 @@ int run_delta(const B2DeltaArgs& a, const B2SeqRows& s, int n_decode, int first,
   if (n_prefill == 0) return 0;
   if (const int rc = dispatch_scan(a, s, first, n_prefill, status, stream)) return rc;
   const dim3 grid(static_cast<unsigned>((static_cast<int64_t>(s.rows) * a.heads + 7) / 8));
-  const bool v4 = a.vdim % 4 == 0 && a.ld_dg % 4 == 0 && a.ld_out % 4 == 0 && (a.heads * a.dim) % 4 == 0;
+  const bool v4 = a.vdim % 4 == 0 && vec4_rows<T>(a.gate, a.ld_gate) && a.ld_out % 4 == 0;
   if (v4 && a.vdim <= 128) launch_pdl(delta_out_kernel<T, 4, 1>, grid, dim3(256), 0, stream, a, s, first);
   else if (v4) launch_pdl(delta_out_kernel<T, 4, 2>, grid, dim3(256), 0, stream, a, s, first);
   else launch_pdl(delta_out_kernel<T, 1, 8>, grid, dim3(256), 0, stream, a, s, first);

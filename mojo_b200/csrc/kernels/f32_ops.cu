@@ -83,8 +83,8 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
                                                        float* __restrict__ out, const int32_t* __restrict__ row_seq,
                                                        const int32_t* __restrict__ positions, const int32_t* __restrict__ tables, int rows, int seqs,
                                                        int max_blocks, int n_q, int n_kv, int dim, int vdim, int64_t ld_v, int64_t ld_out, int page_size,
-                                                       float scale, int window, float cap, float out_scale, int64_t num_pages,
-                                                       const float* __restrict__ gate, int64_t gate_stride, Status* status) {
+                                                       float scale, B2AttnMods mods, int64_t num_pages,
+                                                       const float* __restrict__ gate, int64_t gate_stride, int gate_elems, Status* status) {
   ptx::grid_dep_sync();
   __shared__ float q_sm[4][kAttnMax];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -106,10 +106,15 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
     if (!B2_ASSERT(status, page >= 0 && page < num_pages, kSiteKvIndex, page, num_pages)) page = 0;
     return (page * n_kv + kvh) * page_size + pos % page_size;
   };
-  float m = -INFINITY, l = 0.0f, o[kAttnMax / 32];
+  const int own = ctx - 1;
+  int first = mods.window > 0 ? max(0, ctx - mods.window) : 0;
+  if (mods.chunk > 0) first = max(first, own - own % mods.chunk);
+  const float r1 = mods.distance != nullptr ? mods.distance[head] : 0.0f, r2 = mods.distance != nullptr ? mods.distance[n_q + head] : 0.0f;
+  // the sink is a score of zero that has been seen already
+  float m = mods.sink ? 0.0f : -INFINITY, l = mods.sink && lane == 0 ? 1.0f : 0.0f, o[kAttnMax / 32];
 #pragma unroll
   for (int j = 0; j < kAttnMax / 32; ++j) o[j] = 0.0f;
-  for (int p0 = max(0, ctx - window); p0 < ctx; p0 += 32) {
+  for (int p0 = first; p0 < ctx; p0 += 32) {
     const int pos = p0 + lane;
     int64_t slot = 0;
     float s = -INFINITY;
@@ -119,7 +124,8 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
       float dot = 0.0f;
       for (int i = 0; i < dim; ++i) dot = fmaf(q_sm[warp][i], k[i], dot);
       s = dot * scale;
-      if (cap > 0.0f) s = softcap(s, cap);
+      if (mods.softcap > 0.0f) s = softcap(s, mods.softcap);
+      if (mods.distance != nullptr) s -= r1 * log1pf(r2 * static_cast<float>(own - pos));
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new), p = pos < ctx ? expf(s - m_new) : 0.0f;
@@ -136,11 +142,14 @@ __global__ void __launch_bounds__(128) attn_f32_kernel(const float* __restrict__
         if (lane + 32 * j < vdim) o[j] = fmaf(pt, v[lane + 32 * j], o[j]);
     }
   }
-  float f = out_scale / warp_sum(l);
-  if (gate != nullptr) f *= sigmoid_f32(gate[row * gate_stride + head]);
+  float f = mods.out_scale / warp_sum(l);
+  if (gate != nullptr && !gate_elems) f *= sigmoid_f32(gate[row * gate_stride + head]);
 #pragma unroll
   for (int j = 0; j < kAttnMax / 32; ++j)
-    if (lane + 32 * j < vdim) dst[lane + 32 * j] = o[j] * f;
+    if (lane + 32 * j < vdim) {
+      const int c = lane + 32 * j;
+      dst[c] = o[j] * f * (gate_elems ? sigmoid_f32(gate[row * gate_stride + static_cast<int64_t>(head) * vdim + c]) : 1.0f);
+    }
 }
 
 }  // namespace
@@ -174,8 +183,8 @@ extern "C" int b2_gather_rows_f32(const float* src, const int64_t* index, float*
 
 extern "C" int b2_attn_f32(const float* q, const float* k_cache, const float* v_cache, float* out, const int32_t* row_seq, const int32_t* positions,
                            const int32_t* block_tables, int rows, int seqs, int max_blocks, int n_q, int n_kv, int dim, int vdim, int64_t ld_v, int64_t ld_out,
-                           int page_size, float scale, int window, float cap, float out_scale, int64_t num_pages, const float* gate, int64_t gate_stride,
-                           Status* status, cudaStream_t stream) {
+                           int page_size, float scale, const B2AttnMods* mods, int64_t num_pages, const float* gate, int64_t gate_stride,
+                           int gate_elems, Status* status, cudaStream_t stream) {
   if (rows <= 0) return 0;
   if (n_kv <= 0 || n_q % n_kv != 0 || dim <= 0 || dim > 1152 || vdim <= 0 || vdim > 1152 || ld_v < vdim || ld_out < static_cast<int64_t>(n_q) * vdim ||
       page_size <= 0)
@@ -183,7 +192,7 @@ extern "C" int b2_attn_f32(const float* q, const float* k_cache, const float* v_
   auto kern = dim <= 256 && vdim <= 256 ? attn_f32_kernel<256> : attn_f32_kernel<1152>;
   const int64_t warps = static_cast<int64_t>(rows) * n_q;
   launch_pdl(kern, dim3(static_cast<unsigned>((warps + 3) / 4)), dim3(128), 0, stream, q, k_cache, v_cache, out, row_seq, positions,
-             block_tables, rows, seqs, max_blocks, n_q, n_kv, dim, vdim, ld_v, ld_out, page_size, scale, window > 0 ? window : 1 << 30, cap, out_scale,
-             num_pages, gate, gate_stride, status);
+             block_tables, rows, seqs, max_blocks, n_q, n_kv, dim, vdim, ld_v, ld_out, page_size, scale, mods != nullptr ? *mods : B2AttnMods{0, 0, 0.0f, 1.0f, nullptr, 0},
+             num_pages, gate, gate_stride, gate != nullptr ? gate_elems : 0, status);
   return last_launch_rc();
 }

@@ -137,11 +137,27 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
   }
 }
 
+// 16 bytes of a row times f.
+template <typename T>
+__device__ __forceinline__ uint4 scaled(uint4 r, float f) {
+  if constexpr (sizeof(T) == 4) {
+    return make_uint4(__float_as_uint(__uint_as_float(r.x) * f), __float_as_uint(__uint_as_float(r.y) * f), __float_as_uint(__uint_as_float(r.z) * f),
+                      __float_as_uint(__uint_as_float(r.w) * f));
+  } else {
+    float v[8];
+    bf16x8_to_f32(r, v);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= f;
+    return f32_to_bf16x8(v);
+  }
+}
+
 // Every CTA forms the experts' first rows itself (a scan over the counts); CTA 0 also lists the tiles. Then one warp per
-// row copies it to its `top` places. The order inside an expert is the order of the atomics above and does not touch any
+// row copies it to its `top` places, times the choice's weight where `weights` are given. The order inside an expert is the order of the atomics above and does not touch any
 // result: a row's product depends on that row alone.
 template <typename T>
 __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x, const int32_t* __restrict__ ids, const int32_t* __restrict__ place,
+                                                         const float* __restrict__ weights,
                                                          int32_t* __restrict__ counts, int32_t* __restrict__ slot, T* __restrict__ xs,
                                                          int4* __restrict__ tiles, int32_t* __restrict__ n_tiles, int rows, int experts, int top,
                                                          int width, int bn, int max_tiles, Status* status) {
@@ -179,8 +195,10 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x
   const int vecs = width * static_cast<int>(sizeof(T)) / 16, n_warps = gridDim.x * 8;
   for (int t = blockIdx.x * 8 + warp; t < rows; t += n_warps) {
     int mine = 0;
+    float mine_w = 1.0f;
     if (lane < top) {
       const int64_t at = static_cast<int64_t>(t) * top + lane;
+      if (weights != nullptr) mine_w = weights[at];
       const int id = ids[at];
       mine = id < experts ? first[id] + place[at] : -1;      // what returns its input needs no copy of it
       if (!B2_ASSERT(status, mine >= -1 && mine < rows * top, kSiteEpCount, mine, rows * top)) mine = 0;
@@ -194,11 +212,12 @@ __global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x
         if (c0 + u * 32 + lane < vecs) r[u] = ptx::ld_nc_v4(src + c0 + u * 32 + lane);
       for (int j = 0; j < top; ++j) {
         const int to = __shfl_sync(0xffffffffu, mine, j);
+        const float f = __shfl_sync(0xffffffffu, mine_w, j);
         if (to < 0) continue;
         uint4* dst = reinterpret_cast<uint4*>(xs) + static_cast<int64_t>(to) * vecs;
 #pragma unroll
         for (int u = 0; u < 4; ++u)
-          if (c0 + u * 32 + lane < vecs) dst[c0 + u * 32 + lane] = r[u];
+          if (c0 + u * 32 + lane < vecs) dst[c0 + u * 32 + lane] = weights != nullptr ? scaled<T>(r[u], f) : r[u];
       }
     }
   }
@@ -313,7 +332,7 @@ extern "C" int b2_moe_route(const float* logits, int64_t ld, const float* correc
   return last_launch_rc();
 }
 
-extern "C" int b2_moe_gather(const void* x, const int32_t* ids, const int32_t* place, int32_t* counts, int32_t* slot, void* xs, int32_t* tiles,
+extern "C" int b2_moe_gather(const void* x, const int32_t* ids, const int32_t* place, const float* weights, int32_t* counts, int32_t* slot, void* xs, int32_t* tiles,
                              int32_t* n_tiles, int rows, int experts, int top, int width, int bn, int f32, Status* status, cudaStream_t stream) {
   if (rows <= 0) return 0;
   const int esz = f32 ? 4 : 2;
@@ -322,10 +341,10 @@ extern "C" int b2_moe_gather(const void* x, const int32_t* ids, const int32_t* p
     return -kBadArgument;
   const int blocks = (rows + 7) / 8 < 2 * kNumSMs ? (rows + 7) / 8 : 2 * kNumSMs, max_tiles = experts + rows * top / bn;
   if (f32)
-    launch_pdl(moe_gather_kernel<float>, dim3(blocks), dim3(256), 0, stream, static_cast<const float*>(x), ids, place, counts, slot, static_cast<float*>(xs),
+    launch_pdl(moe_gather_kernel<float>, dim3(blocks), dim3(256), 0, stream, static_cast<const float*>(x), ids, place, weights, counts, slot, static_cast<float*>(xs),
                reinterpret_cast<int4*>(tiles), n_tiles, rows, experts, top, width, bn, max_tiles, status);
   else
-    launch_pdl(moe_gather_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(x), ids, place, counts, slot,
+    launch_pdl(moe_gather_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, static_cast<const __nv_bfloat16*>(x), ids, place, weights, counts, slot,
                static_cast<__nv_bfloat16*>(xs), reinterpret_cast<int4*>(tiles), n_tiles, rows, experts, top, width, bn, max_tiles, status);
   return last_launch_rc();
 }

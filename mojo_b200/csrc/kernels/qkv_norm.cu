@@ -1,5 +1,6 @@
-// Attention front end of layers that normalise whole projections: biases, one RMS norm over all q columns of a row and one over
-// its k columns, rotary embedding, scatter of k and v into the paged cache. One CTA per token row.
+// Attention front ends with norms. Over whole projections: biases, one RMS norm over all q columns of a row and one over
+// its k columns, rotary embedding, scatter of k and v into the paged cache. One CTA per token row. Per head: one warp per
+// (row, few heads).
 #include <cstdint>
 #include "b2/elem.cuh"
 #include "b2/launch.h"
@@ -378,10 +379,99 @@ int launch_norm_qkv(const B2NormQkvArgs& a, Status* status, cudaStream_t stream)
   return last_launch_rc();
 }
 
+// Warps take HP neighbouring heads of a row, all of them requested at once; a lane holds columns (lane + 32 j) * VEC.
+template <typename T, int VEC, int NJ, int HP>
+__global__ void __launch_bounds__(256) head_norm_qkv_kernel(const B2HeadNormArgs a, Status* status) {
+  ptx::grid_dep_sync();
+  const int n_heads = a.heads + 2 * a.kv_heads, runs = (n_heads + HP - 1) / HP, lane = threadIdx.x & 31;
+  const int64_t idx = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5), row = idx / runs;
+  if (row >= a.rows) return;
+  const int h0 = static_cast<int>(idx % runs) * HP;
+  const T* src = static_cast<const T*>(a.proj) + row * a.ld;
+  const int64_t slot = a.slots[row];
+  float v[HP][NJ][VEC], ss[HP];
+#pragma unroll
+  for (int i = 0; i < HP; ++i) {
+    const int h = h0 + i, kv = h - a.heads;
+    const bool is_v = kv >= a.kv_heads;
+    const int size = is_v ? a.vdim : a.dim, from = is_v ? a.v_off + (kv - a.kv_heads) * a.vdim : h * a.dim;
+    ss[i] = 0.0f;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int c = (lane + 32 * j) * VEC;
+#pragma unroll
+      for (int x = 0; x < VEC; ++x) v[i][j][x] = 0.0f;
+      if (h < n_heads && c < size) load_f32<VEC>(src + from + c, v[i][j]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < HP; ++i) {
+#pragma unroll
+    for (int j = 0; j < NJ; ++j)
+#pragma unroll
+      for (int x = 0; x < VEC; ++x) ss[i] = fmaf(v[i][j][x], v[i][j][x], ss[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < HP; ++i) ss[i] = warp_sum(ss[i]);
+  const bool cached = slot >= 0 && B2_ASSERT(status, slot < a.num_slots, kSiteKvIndex, slot, a.num_slots);
+  // cache row of head 0; the heads of a page lie page_size rows apart (the host keeps slots below 2^31)
+  const uint32_t page = cached ? static_cast<uint32_t>(slot) / static_cast<uint32_t>(a.page_size) : 0;
+  const int64_t cell = cached ? static_cast<int64_t>(page) * a.kv_heads * a.page_size + (static_cast<uint32_t>(slot) - page * a.page_size) : 0;
+#pragma unroll
+  for (int i = 0; i < HP; ++i) {
+    const int h = h0 + i, kv = h - a.heads;
+    if (h >= n_heads || (kv >= 0 && !cached)) break;      // uniform per warp
+    const bool is_q = kv < 0, is_v = kv >= a.kv_heads;
+    T* dst = is_q ? static_cast<T*>(a.q_out) + (row * a.heads + h) * a.pad_dim
+             : is_v ? static_cast<T*>(a.v_cache) + (cell + static_cast<int64_t>(kv - a.kv_heads) * a.page_size) * a.pad_vdim
+                    : static_cast<T*>(a.k_cache) + (cell + static_cast<int64_t>(kv) * a.page_size) * a.pad_dim;
+    const float* w = is_q ? a.q_norm : a.k_norm;
+    const float r = 1.0f / sqrtf(ss[i] / static_cast<float>(a.dim) + a.eps);
+    const int size = is_v ? a.vdim : a.dim;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) {
+      const int c = (lane + 32 * j) * VEC;
+      if (!is_v && c < size) {
+        float f[VEC];
+        load_f32<VEC>(w + c, f);
+#pragma unroll
+        for (int x = 0; x < VEC; ++x) v[i][j][x] *= r * f[x];
+      }
+      // queries are zero past `dim` (as v is there); cache rows are from the start
+      if (c < (is_q ? a.pad_dim : size)) store_f32<VEC>(dst + c, v[i][j]);
+    }
+  }
+}
+
+template <typename T, int VEC, int NJ, int HP>
+int launch_head_norm(const B2HeadNormArgs& a, Status* status, cudaStream_t stream) {
+  const int64_t warps = static_cast<int64_t>(a.rows) * ((a.heads + 2 * a.kv_heads + HP - 1) / HP);
+  launch_pdl(head_norm_qkv_kernel<T, VEC, NJ, HP>, dim3(static_cast<unsigned>((warps + 7) / 8)), dim3(256), 0, stream, a, status);
+  return last_launch_rc();
+}
+template <typename T>
+int dispatch_head_norm(const B2HeadNormArgs& a, Status* status, cudaStream_t stream) {
+  const int m = a.pad_dim > a.pad_vdim ? a.pad_dim : a.pad_vdim;
+  const bool v4 = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.v_off % 4 == 0 && a.pad_dim % 4 == 0 && a.pad_vdim % 4 == 0 && a.ld % 4 == 0 &&
+                  reinterpret_cast<uintptr_t>(a.proj) % (4 * sizeof(T)) == 0;
+  if (!v4) return launch_head_norm<T, 1, 8, 1>(a, status, stream);
+  if (m > 128) return launch_head_norm<T, 4, 2, 2>(a, status, stream);
+  const bool few = static_cast<int64_t>(a.rows) * (a.heads + 2 * a.kv_heads) < 64 * kNumSMs;
+  return few ? launch_head_norm<T, 4, 1, 1>(a, status, stream) : launch_head_norm<T, 4, 1, 4>(a, status, stream);
+}
+
 }  // namespace
 }  // namespace b2
 
 using namespace b2;
+
+extern "C" int b2_head_norm_qkv(const B2HeadNormArgs* a, int f32, Status* status, cudaStream_t stream) {
+  if (a->rows <= 0) return 0;
+  if (a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads != 0 || a->dim <= 0 || a->vdim <= 0 || a->v_off < 0 || a->pad_dim < a->dim ||
+      a->pad_vdim < a->vdim || a->pad_dim > 256 || a->pad_vdim > 256 || a->page_size <= 0 || a->num_slots > 0x7fffffff || a->q_norm == nullptr || a->k_norm == nullptr)
+    return -kBadArgument;
+  return f32 ? dispatch_head_norm<float>(*a, status, stream) : dispatch_head_norm<__nv_bfloat16>(*a, status, stream);
+}
 
 extern "C" int b2_norm_qkv(const B2NormQkvArgs* a, int f32, Status* status, cudaStream_t stream) {
   if (a->rows <= 0) return 0;

@@ -30,7 +30,7 @@ __global__ void residual_norm_kernel(const B2ResidualArgs a, Status* status) {
       const int slot = a.expert_slot[row * a.top + threadIdx.x];
       const bool ok = B2_ASSERT(status, slot >= (a.own != nullptr ? -1 : 0) && slot < a.expert_rows, kSiteEpCount, slot, a.expert_rows);
       e_row[threadIdx.x] = ok ? slot : 0;
-      e_w[threadIdx.x] = ok ? a.expert_w[row * a.top + threadIdx.x] : 0.0f;
+      e_w[threadIdx.x] = !ok ? 0.0f : a.expert_w != nullptr ? a.expert_w[row * a.top + threadIdx.x] : 1.0f;
     }
     __syncthreads();
   }
@@ -154,7 +154,7 @@ using namespace b2;
 extern "C" int b2_residual_norm(const B2ResidualArgs* a, int f32, Status* status, cudaStream_t stream) {
   if (a->n_out <= 0) return 0;
   if (a->width <= 0 || a->width > 50000 || a->mean_width <= 0 || a->mean_width > a->width || a->x == nullptr || a->h == nullptr ||
-      (a->bias != nullptr && a->weight == nullptr) || (a->gated != nullptr && a->gate == nullptr) || (a->experts != nullptr && (a->expert_slot == nullptr || a->expert_w == nullptr || a->top < 1 || a->top > kMaxTop)) ||
+      (a->bias != nullptr && a->weight == nullptr) || (a->gated != nullptr && a->gate == nullptr) || (a->experts != nullptr && (a->expert_slot == nullptr || a->top < 1 || a->top > kMaxTop)) ||
       (a->ids != nullptr && a->embed == nullptr) || (a->bigram != nullptr && (a->prev == nullptr || a->buckets < 1)) ||
       (a->rows_index == nullptr && a->n_out != a->rows))
     return -kBadArgument;

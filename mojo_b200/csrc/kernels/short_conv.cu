@@ -1,4 +1,4 @@
-// Attention front end of layers with short convolutions: causal convolution over time on every q, k and v channel, rotary
+// Front ends with short causal convolutions over time. For attention: causal convolution over time on every q, k and v channel, rotary
 // embedding, RMS norm of the q and k heads, scatter of k and v into the paged cache. One warp owns one head and a few
 // consecutive rows. What the convolution needs from before the step comes from the sequence's state bank; the step's last
 // taps - 1 projected rows go to its other bank, so no warp reads what another one of the same launch writes.
@@ -7,6 +7,7 @@
 #include "b2/launch.h"
 #include "b2/mixers.h"
 #include "b2/ptx.cuh"
+#include "b2/recurrence.cuh"
 #include "b2/short_conv.cuh"
 #include "b2/vec.cuh"
 
@@ -321,10 +322,64 @@ int dispatch_conv_qkv(const B2ConvQkvArgs& a, const B2SeqRows& s, Status* status
   return launch_conv_qkv<T, 1, 8, 0>(a, s, status, stream);
 }
 
+// A thread's channels over a few rows of one sequence.
+template <typename T, int VEC, int TAPS, int TT>
+__global__ void __launch_bounds__(128) conv_silu_kernel(const B2ConvSiluArgs a, const B2SeqRows sq, Status* status) {
+  ptx::grid_dep_sync();
+  int tile = static_cast<int>(blockIdx.x);
+  const int seq = find_tile(sq, 0, sq.seqs, TT, tile);
+  if (seq < 0) return;
+  const int row0 = sq.seq_rows[2 * seq] + tile * TT, c = static_cast<int>(blockIdx.y * 128 + threadIdx.x) * VEC;
+  ConvRow cr;
+  if (!cr.load(sq, seq, row0, sq.banks, status) || c >= a.channels) return;
+  const ConvSource<T> src{static_cast<const T*>(a.proj), a.ld, a.conv_w, static_cast<T*>(a.conv_state), a.taps, a.channels, sq.banks};
+  const int n = min(TT, cr.end - row0);
+  float y[TT][VEC], b[VEC] = {};
+  conv_rows<T, VEC, TAPS, TT>(src, cr, row0, n, c, true, y);
+  if (a.bias != nullptr) load_f32<VEC>(a.bias + c, b);
+#pragma unroll
+  for (int t = 0; t < TT; ++t) {
+    if (t >= n) break;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) y[t][i] = ptx::silu(y[t][i] + b[i]);
+    store_f32<VEC>(static_cast<T*>(a.out) + static_cast<int64_t>(row0 + t) * a.ld_out + c, y[t]);
+  }
+}
+
+template <typename T, int VEC, int TAPS>
+int launch_conv_silu(const B2ConvSiluArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
+  constexpr int kRows = 8;
+  const unsigned blocks = (a.channels + 128 * VEC - 1) / (128 * VEC);
+  if (s.rows <= s.seqs) launch_pdl(conv_silu_kernel<T, VEC, TAPS, 1>, dim3(s.rows, blocks), dim3(128), 0, stream, a, s, status);
+  else launch_pdl(conv_silu_kernel<T, VEC, TAPS, kRows>, dim3(s.rows / kRows + s.seqs, blocks), dim3(128), 0, stream, a, s, status);
+  return last_launch_rc();
+}
+
+template <typename T>
+int dispatch_conv_silu(const B2ConvSiluArgs& a, const B2SeqRows& s, Status* status, cudaStream_t stream) {
+  if (a.channels % 4 == 0 && a.ld % 4 == 0 && a.ld_out % 4 == 0 && reinterpret_cast<uintptr_t>(a.proj) % (4 * sizeof(T)) == 0 &&
+      reinterpret_cast<uintptr_t>(a.out) % (4 * sizeof(T)) == 0) {
+    switch (a.taps) {
+      case 2: return launch_conv_silu<T, 4, 2>(a, s, status, stream);
+      case 3: return launch_conv_silu<T, 4, 3>(a, s, status, stream);
+      case 4: return launch_conv_silu<T, 4, 4>(a, s, status, stream);
+      default: return launch_conv_silu<T, 4, 0>(a, s, status, stream);
+    }
+  }
+  return launch_conv_silu<T, 1, 0>(a, s, status, stream);
+}
+
 }  // namespace
 }  // namespace b2
 
 using namespace b2;
+
+extern "C" int b2_conv_silu(const B2ConvSiluArgs* a, const B2SeqRows* s, int f32, Status* status, cudaStream_t stream) {
+  if (s->rows <= 0) return 0;
+  if (a->channels <= 0 || a->taps < 1 || (a->taps > 1 && a->conv_state == nullptr) || a->out == nullptr || a->ld < a->channels || a->ld_out < a->channels)
+    return -kBadArgument;
+  return f32 ? dispatch_conv_silu<float>(*a, *s, status, stream) : dispatch_conv_silu<__nv_bfloat16>(*a, *s, status, stream);
+}
 
 extern "C" int b2_conv_qkv(const B2ConvQkvArgs* a, const B2SeqRows* s, int f32, Status* status, cudaStream_t stream) {
   if (s->rows <= 0) return 0;

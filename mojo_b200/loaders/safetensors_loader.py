@@ -64,7 +64,7 @@ class _Reader:
 
 
 def load_safetensors_into(model, path: str | Path) -> None:
-    """Fill a model from a checkpoint directory: Llama family or DeepSeek-V2(-Lite) in Hugging Face layout, Rekudra, Rerupel, Pilutar."""
+    """Fill a model from a checkpoint directory: Llama family or DeepSeek-V2(-Lite) in Hugging Face layout, Rekudra, Rerupel, Pilutar, Noridra."""
     rd = _Reader(read_safetensors_index(path))
     cfg = model.cfg
     if getattr(cfg, "architecture", "llama") == "deepseek_v2":
@@ -73,7 +73,7 @@ def load_safetensors_into(model, path: str | Path) -> None:
     if cfg.architecture == "rekudra":
         _load_rekudra(model, rd)
         return
-    if cfg.architecture in ("rerupel", "pilutar"):
+    if cfg.architecture in ("rerupel", "pilutar", "noridra"):
         _load_named_layers(model, rd)
         return
     model.layers.clear()
@@ -161,7 +161,7 @@ def _load_rekudra(model, rd: _Reader) -> None:
 
 
 def _load_named_layers(model, rd: _Reader) -> None:
-    """Rerupel and Pilutar: the names and shapes the model lists, those of layer i behind `l<i>.`."""
+    """Rerupel, Pilutar, Noridra: the names and shapes the model lists, those of layer i behind `l<i>.`."""
     model.layers.clear()
     for name in model.global_shapes():
         model.load_tensor(name, rd.get(name))

@@ -27,4 +27,8 @@ def build_model(cfg: ModelConfig, device="cpu", dtype=torch.float32, comm=None, 
         from .pilutar import PilutarModel
 
         return PilutarModel(cfg, device, dtype, comm=comm)
+    if cfg.architecture == "noridra":
+        from .noridra import NoridraModel
+
+        return NoridraModel(cfg, device, dtype, comm=comm)
     raise ValueError(f"unsupported architecture {cfg.architecture!r}")

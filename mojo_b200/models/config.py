@@ -57,7 +57,7 @@ class BigramSpec:
 @dataclass
 class LayerSpec:
     """One layer of a decoder whose layers differ: which mixer it has, the mixer's sizes, and its feed-forward."""
-    mixer: str = "attention"               # "attention" | "channel_delta" | "latent_attention" | "gated_linear" | "parallel"
+    mixer: str = "attention"               # "attention" | "channel_delta" | "delta" | "latent_attention" | "gated_linear" | "mamba1" | "parallel"
     heads: int = 0
     kv_heads: int = 0
     dim: int = 0                           # query / key size of a head
@@ -73,6 +73,10 @@ class LayerSpec:
     moe: MoeSpec | None = None             # mixture of experts in place of a dense feed-forward
     window: int = 0                        # attention: positions a token sees, itself included (0: all before it)
     softcap: float = 0.0                   # attention: scores become softcap * tanh(score / softcap) (0: they do not)
+    chunk: int = 0                         # attention: positions see only those of their own run of `chunk` (0: all before them)
+    inner: int = 0                         # selective scan: channels, states of a channel, rank of the step sizes
+    state: int = 0
+    dt_rank: int = 0
     tau: float = 1.0                       # gated linear attention: decays are sigmoid(z)^(1 / tau)
     parts: list["LayerSpec"] | None = None # "parallel": the mixers that run side by side ...
     part_scales: list[float] | None = None # ... and the factors of their results
@@ -80,7 +84,7 @@ class LayerSpec:
 
 @dataclass
 class ModelConfig:
-    architecture: str = "llama"            # "llama" | "deepseek_v2" | "rekudra" | "rerupel" | "pilutar"
+    architecture: str = "llama"            # "llama" | "deepseek_v2" | "rekudra" | "rerupel" | "pilutar" | "noridra"
     hidden_size: int = 4096
     num_layers: int = 32
     num_heads: int = 32
@@ -118,6 +122,10 @@ class ModelConfig:
     residual_mult: float = 1.0             # on everything a sublayer adds to the residual
     logit_softcap: float | None = None
     logit_scale: float = 1.0
+    # decoders that normalise after the sum: x <- norm(residual_alpha * x + sublayer(x + conv(x)))
+    residual_alpha: float = 1.0
+    norm_groups: int = 1                   # runs of columns that the norm treats one by one
+    input_taps: int = 1                    # taps of the convolution over time on what a sublayer reads
     extra: dict = field(default_factory=dict)
 
     def to_dict(self) -> dict:
@@ -180,6 +188,19 @@ class ModelConfig:
                 if s.moe is not None:
                     n += h * (s.moe.experts + s.moe.identity + 2 * s.moe.experts * s.moe.expert.ffn + (2 * s.moe.shared.ffn + 1 if s.moe.shared else 0))
             return n
+        if self.architecture == "noridra":
+            n = emb + h + self.max_position_embeddings * h
+            for s in self.layers:
+                if s.mixer == "mamba1":
+                    n += s.inner * (3 * h + 2 * s.dt_rank + 3 * s.state + s.conv_taps + 3)
+                elif s.mixer == "delta":
+                    n += h * (2 * s.kv_heads * s.dim + 3 * s.heads * s.vdim + 2 * s.heads) + s.conv_taps * (2 * s.kv_heads * s.dim + s.heads * s.vdim)
+                else:
+                    n += h * (3 * s.heads + s.kv_heads) * s.dim
+                n += (2 if s.moe else 1) * h * (2 + self.input_taps)
+                if s.moe is not None:
+                    n += h * (s.moe.experts + 3 * s.moe.experts * s.moe.expert.ffn)
+            return n
         if self.layers is not None:
             n = emb + h
             for s in self.layers:
@@ -240,6 +261,8 @@ class ModelConfig:
             return ModelConfig._from_latent_layers(cfg)
         if LAYERED_ARCHITECTURES[cfg["architecture"]] == "pilutar":
             return ModelConfig._from_parallel_layers(cfg)
+        if LAYERED_ARCHITECTURES[cfg["architecture"]] == "noridra":
+            return ModelConfig._from_postnorm_layers(cfg)
         layers = []
         for i, entry in enumerate(cfg["layers"]):
             m, mlp = entry["mixer"], entry.get("mlp")
@@ -356,11 +379,48 @@ class ModelConfig:
                            max_position_embeddings=0, layers=layers, embedding_scale=cfg.get("embedding", {}).get("scale", 1.0),
                            logit_scale=cfg.get("logit_scale", 1.0))
 
+    @staticmethod
+    def _from_postnorm_layers(cfg: dict) -> "ModelConfig":
+        def mixer(kind, m):
+            if kind == "mamba1":
+                return LayerSpec("mamba1", inner=m["inner"], state=m["state"], dt_rank=m["dt_rank"], conv_taps=m["conv"])
+            if kind not in ("delta", "attention"):
+                raise ValueError(f"unknown mixer {kind!r}")
+            if m["heads"] % m["kv_heads"]:
+                raise ValueError(f"{m['heads']} heads on {m['kv_heads']} key heads")
+            if kind == "delta":
+                return LayerSpec("delta", m["heads"], m["kv_heads"], m["dim"], m["vdim"], m["conv"])
+            chunk = (m.get("mask") or {}).get("size") or 0
+            if m["vdim"] != m["dim"] or chunk < 0:
+                raise ValueError(f"values of size {m['vdim']} that are keys of size {m['dim']}" if chunk >= 0 else f"chunks of {chunk} positions")
+            return LayerSpec("attention", m["heads"], m["kv_heads"], m["dim"], m["vdim"], scale=m["scale"], softcap=m.get("softcap") or 0.0, chunk=chunk)
+
+        layers, norm = [], cfg["norm"]
+        if cfg["width"] % norm["groups"]:
+            raise ValueError(f"{cfg['width']} columns in {norm['groups']} groups")
+        for i, entry in enumerate(cfg["layers"]):
+            try:
+                spec, mlp = mixer(entry["type"], entry["mixer"]), entry.get("mlp")
+                if mlp is not None:
+                    if mlp["kind"] != "moe":
+                        raise ValueError(f"unknown feed-forward {mlp['kind']!r}")
+                    spec.moe = MoeSpec(mlp["router"]["experts"], mlp["router"]["top"], 1.0, ExpertSpec(mlp["expert"]["ff"]))
+                    if not 1 <= spec.moe.top <= spec.moe.experts:
+                        raise ValueError(f"{spec.moe.top} of {spec.moe.experts} experts")
+            except ValueError as e:
+                raise ValueError(f"layer {i}: {e}") from None
+            layers.append(spec)
+        first = next((s for s in layers if s.mixer == "attention"), layers[0])
+        return ModelConfig(architecture="noridra", hidden_size=cfg["width"], num_layers=len(layers), num_heads=first.heads, num_kv_heads=first.kv_heads,
+                           head_dim=first.dim, intermediate_size=0, vocab_size=cfg["vocab"], rms_norm_eps=norm["eps"],
+                           max_position_embeddings=cfg["max_positions"], layers=layers, residual_alpha=cfg["postln_alpha"], norm_groups=norm["groups"],
+                           input_taps=cfg["canon"]["taps"])
+
 
 # `architecture` values of configs that list their layers -> model class key
-LAYERED_ARCHITECTURES = {"Rekudra": "rekudra", "Rerupel": "rerupel", "Pilutar": "pilutar"}
+LAYERED_ARCHITECTURES = {"Rekudra": "rekudra", "Rerupel": "rerupel", "Pilutar": "pilutar", "Noridra": "noridra"}
 # model classes that also run in f32 on CUDA (every operation has a true 32-bit kernel)
-F32_ARCHITECTURES = ("rekudra", "rerupel", "pilutar")
+F32_ARCHITECTURES = ("rekudra", "rerupel", "pilutar", "noridra")
 
 
 def tiny_llama() -> ModelConfig:
@@ -482,6 +542,31 @@ def tiny_pilutar() -> ModelConfig:
     return pilutar(256, 4, 4, 2, 64, 128, 32, 512, 1024, 7, 2, 128, 192, 48, groups=2, identity=1)
 
 
+def noridra(width: int, n_layers: int, heads: int, kv_heads: int, dim: int, vocab: int, experts: int, top: int, expert_ffn: int, chunk: int,
+            state: int = 16, groups: int = 4, taps: int = 4, positions: int = 8192) -> ModelConfig:
+    """A Noridra decoder: in every four layers two with the gated delta rule, one with attention inside chunks, one selective
+    scan over twice the width; experts in all of them."""
+    moe = MoeSpec(experts, top, 1.0, ExpertSpec(expert_ffn))
+    kinds = [lambda: LayerSpec("delta", heads, heads, dim, dim, taps), lambda: LayerSpec("delta", heads, heads, dim, dim, taps),
+             lambda: LayerSpec("attention", heads, kv_heads, dim, dim, scale=dim ** -0.5, softcap=30.0, chunk=chunk),
+             lambda: LayerSpec("mamba1", inner=2 * width, state=state, dt_rank=width // 16, conv_taps=taps)]
+    layers = [kinds[i % 4]() for i in range(n_layers)]
+    for s in layers:
+        s.moe = moe
+    return ModelConfig(architecture="noridra", hidden_size=width, num_layers=n_layers, num_heads=heads, num_kv_heads=kv_heads, head_dim=dim,
+                       intermediate_size=0, vocab_size=vocab, rms_norm_eps=1e-6, max_position_embeddings=positions, layers=layers,
+                       residual_alpha=(2.0 * n_layers) ** 0.25, norm_groups=groups, input_taps=taps)
+
+
+def noridra_lite() -> ModelConfig:
+    """Layers of the size of DeepSeek-V2-Lite's."""
+    return noridra(2048, 24, 16, 4, 128, 102400, 64, 6, 1408, 1024)
+
+
+def tiny_noridra() -> ModelConfig:
+    return noridra(256, 4, 4, 2, 64, 1024, 8, 2, 128, 48, positions=2048)
+
+
 PRESETS = {
     "tiny-llama": tiny_llama,
     "llama-3.1-8b": llama31_8b,
@@ -495,6 +580,8 @@ PRESETS = {
     "tiny-rerupel": tiny_rerupel,
     "pilutar-lite": pilutar_lite,
     "tiny-pilutar": tiny_pilutar,
+    "noridra-lite": noridra_lite,
+    "tiny-noridra": tiny_noridra,
 }
 
 

@@ -317,7 +317,8 @@ class RekudraModel:
         s = lw.spec
         proj = ops.linear(h, lw.w_in)
         dg = ops.linear(proj[:, lw.low_off:lw.b_off], lw.w_dg)
-        o = ops.delta_rule(proj, dg, lw.delta, cache.conv, cache.state, meta.seq, lw.b_off, s.heads, s.kv_heads, s.dim, s.vdim, lw.wo.shape[1],
+        nk = s.heads * s.dim
+        o = ops.delta_rule(proj, dg[:, :nk], dg[:, nk:nk + s.heads * s.vdim], lw.delta, cache.conv, cache.state, meta.seq, lw.b_off, s.heads, s.kv_heads, s.dim, s.vdim, lw.wo.shape[1],
                            self.cfg.rms_norm_eps)
         return ops.linear(o, lw.wo)
 

@@ -318,10 +318,20 @@ def gemm_config(swap: bool, bn: int, splits: int = 1, stream_k: bool = False) ->
 
 class ScoreMods(NamedTuple):
     """What an attention layer does beyond plain causal softmax. `window`: a row sees that many positions, its own included
-    (0: all); `softcap`: scores become softcap * tanh(score / softcap) (0: they do not); `out_scale`: factor of the result."""
+    (0: all); `softcap`: scores become softcap * tanh(score / softcap) (0: they do not); `out_scale`: factor of the result;
+    `chunk`: a row sees positions of its own run of `chunk` only, counted from position 0 (0: of all); `sink`: one more score, zero,
+    takes part in the softmax and has no value; `distance` f32 [2, heads] (r1, r2): r1 ln(1 + r2 d) is taken off a score, behind the
+    cap, d positions from query to key."""
     window: int = 0
     softcap: float = 0.0
     out_scale: float = 1.0
+    chunk: int = 0
+    sink: bool = False
+    distance: torch.Tensor | None = None
+
+    def span(self, ctx: int) -> int:
+        """Most positions that a row of a context sees."""
+        return min(n for n in (ctx, self.window or ctx, self.chunk or ctx))
 
 
 class AttnMeta:
@@ -430,7 +440,7 @@ def _decode_attention(q, k_cache, v_cache, out, ctx_lens, block_tables, head_dim
         C.attn_prefill(q, k_cache, v_cache, out, cu, ctx_lens, block_tables, head_dim, 1, scale, st.status, gate, *mods)
         _count()
         return
-    splits = _decode_splits(n, n_kv, min(max_ctx, mods.window) if mods.window else max_ctx)
+    splits = _decode_splits(n, n_kv, mods.span(max_ctx))
     splits = max(1, min(splits, _state.ATTN_WORKSPACE_BYTES // (n * (q.shape[1] // head_dim) * (head_dim + 2) * 4)))
     C.attn_decode(q, k_cache, v_cache, out, ctx_lens, block_tables, st.attn_ws, head_dim, splits, scale, st.status, st.attn_counters, gate,
                   *mods)
@@ -441,14 +451,15 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
                     head_dim: int, out: torch.Tensor | None = None, gate: torch.Tensor | None = None,
                     positions: torch.Tensor | None = None, mods: ScoreMods = ScoreMods()) -> torch.Tensor:
     """Causal GQA attention over the paged cache. q, out: [T, n_q * D] (rows of out may be strided). `gate` [T, n_q]: head h of a
-    row is multiplied by sigmoid(gate[row, h]). f32 tensors (any head sizes; key and value sizes may differ) need `meta.seq`
+    row is multiplied by sigmoid(gate[row, h]); or like the result, one logit per element. f32 tensors (any head sizes; key and value sizes may differ) need `meta.seq`
     and `positions`."""
     if not q.is_cuda:
         T = q.shape[0]
         o = reference.paged_attention(q.reshape(T, -1, head_dim), k_cache, v_cache, meta.cu_q, meta.ctx_lens,
-                                      meta.block_tables, scale, mods.window, mods.softcap) * mods.out_scale
+                                      meta.block_tables, scale, *mods)
         if gate is not None:
-            o = o * torch.sigmoid(gate.float()).unsqueeze(-1)
+            g = torch.sigmoid(gate.float())
+            o = o * (g.view(o.shape) if g.shape[1] == o[0].numel() else g.unsqueeze(-1))
         o = o.reshape(T, -1).to(q.dtype)
         return o if out is None else out.copy_(o)
     C = _ext.require()
@@ -569,6 +580,6 @@ def sample(logits: torch.Tensor, temperature: torch.Tensor, top_k: torch.Tensor,
 
 
 from .latent import SharedRope, head_linear, latent_attend, latent_prefill, latent_write, plan_latent_prefill, token_rows  # noqa: E402,F401
-from .mixers import (DeltaParams, Finished, GatedLinearParams, HyperMix, QkvNorm, SeqRows, StreamStart, conv_qkv, delta_rule,  # noqa: E402,F401
-                     gated_linear, hyper_norm, norm_qkv, residual_norm)
+from .mixers import (DeltaParams, Finished, GatedLinearParams, GroupNorm, HyperMix, InputConv, QkvNorm, ScanParams, SeqRows, StreamStart,  # noqa: E402,F401
+                     conv_qkv, conv_silu, delta_rule, gated_linear, head_norm_qkv, hyper_norm, norm_qkv, post_norm, residual_norm, selective_scan)
 from .moe import ExpertRows, MoeWeights, moe_experts  # noqa: E402,F401

@@ -20,7 +20,8 @@ class MoeWeights:
     rows interleaved in blocks of 16; with `glu` None, squared-ReLU experts, [experts, ffn, width]), w_down [experts, width,
     ffn]. A token uses the `top` experts of the largest scores, with their scores (over their sum if `norm_top`) times `scale`
     as weights. `correction` f32 [experts + identity] is added to the scores for the choice alone; the choice is among the
-    `keep` of `groups` groups of neighbours with the largest scores in them. The last `identity` experts return their input."""
+    `keep` of `groups` groups of neighbours with the largest scores in them. The last `identity` experts return their input.
+    `on_input`: a weight multiplies what its expert reads, not what it returns."""
     router: torch.Tensor
     w_gu: torch.Tensor
     w_down: torch.Tensor
@@ -34,6 +35,7 @@ class MoeWeights:
     groups: int = 1
     keep: int = 1
     identity: int = 0
+    on_input: bool = False
 
 
 @dataclass
@@ -41,9 +43,16 @@ class ExpertRows:
     """Results of a token's experts: rows[slot[t, j]] times weights[t, j], summed over j. A slot of -1 stands for the token's own
     input row, `own[t]`."""
     rows: torch.Tensor
-    slot: torch.Tensor          # int32 [T, top]
-    weights: torch.Tensor       # f32 [T, top]
+    slot: torch.Tensor                  # int32 [T, top]
+    weights: torch.Tensor | None        # f32 [T, top]; None: one
     own: torch.Tensor | None = None
+
+    def total(self) -> torch.Tensor:
+        """The weighted sums, f32 [T, width], by plain tensor operations."""
+        e = self.rows.float()[self.slot.clamp_min(0).long()]
+        if self.own is not None:
+            e = torch.where((self.slot < 0).unsqueeze(-1), self.own.float().unsqueeze(1), e)
+        return e.sum(1) if self.weights is None else torch.einsum("tk,tkw->tw", self.weights, e)
 
 
 def tile_rows(rows_per_expert: float) -> int:
@@ -66,13 +75,14 @@ def moe_experts(h: torch.Tensor, p: MoeWeights, logits: torch.Tensor | None = No
         for e in range(p.experts):
             tok, j = torch.where(ids == e)
             if tok.numel():
+                x = (h[tok].float() * weights[tok, j].unsqueeze(-1)).to(h.dtype) if p.on_input else h[tok]
                 if p.glu is None:
-                    act = reference.linear(h[tok], p.w_gu[e]).clamp_min(0.0).square()
+                    act = reference.linear(x, p.w_gu[e]).clamp_min(0.0).square()
                 else:
-                    act = reference.linear_swiglu_interleaved(h[tok], p.w_gu[e], act=p.glu)
+                    act = reference.linear_swiglu_interleaved(x, p.w_gu[e], act=p.glu)
                 rows[tok, j] = reference.linear(act.to(h.dtype), p.w_down[e]).to(h.dtype)
         slot = torch.where(ids < p.experts, torch.arange(T * p.top).view(T, p.top), -1).int()
-        return ExpertRows(rows.view(T * p.top, W), slot, weights.float(), own)
+        return ExpertRows(rows.view(T * p.top, W), slot, None if p.on_input else weights.float(), own)
     C, st = _ext.require(), _state.get(h.device)
     dev, R, f32 = h.device, T * p.top, h.dtype == torch.float32
     bn = 64 if f32 else tile_rows(R / n_out)
@@ -82,7 +92,7 @@ def moe_experts(h: torch.Tensor, p: MoeWeights, logits: torch.Tensor | None = No
     C.moe_route(logits, weights, ids, place, counts, p.experts, SCORING[p.scoring], p.norm_top, p.scale, p.correction, p.groups, p.keep, p.identity)
     xs = torch.empty(R, W, dtype=h.dtype, device=dev)
     tiles, n_tiles = torch.empty(p.experts + R // bn, 4, dtype=torch.int32, device=dev), torch.empty(1, dtype=torch.int32, device=dev)
-    C.moe_gather(h, ids, place, counts, slot, xs, tiles, n_tiles, p.experts, bn, st.status)
+    C.moe_gather(h, ids, place, counts, slot, xs, tiles, n_tiles, p.experts, bn, st.status, weights if p.on_input else None)
     f = p.w_down.shape[2]
     act, y = torch.empty(R, f, dtype=h.dtype, device=dev), torch.empty(R, W, dtype=h.dtype, device=dev)
     launches = 4
@@ -97,4 +107,4 @@ def moe_experts(h: torch.Tensor, p: MoeWeights, logits: torch.Tensor | None = No
         C.moe_tiles_gemm(xs, p.w_gu, tiles, n_tiles, act, EPI_SWIGLU, bn, (*p.glu, 0.0), st.status)
     C.moe_tiles_gemm(act, p.w_down, tiles, n_tiles, y, EPI_NONE, bn, None, st.status)
     _count(launches)
-    return ExpertRows(y, slot, weights, own)
+    return ExpertRows(y, slot, None if p.on_input else weights, own)

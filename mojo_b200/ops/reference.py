@@ -114,16 +114,18 @@ def gather_kv(cache: torch.Tensor, block_table: torch.Tensor, ctx_len: int) -> t
     return pages.permute(0, 2, 1, 3).reshape(n_pages * page_size, cache.shape[1], cache.shape[3])[:ctx_len]
 
 
-def visible(ctx: int, q_len: int, window: int = 0, device="cpu") -> torch.Tensor:
+def visible(ctx: int, q_len: int, window: int = 0, device="cpu", chunk: int = 0) -> torch.Tensor:
     """Which of `ctx` positions the last `q_len` of them see: [q_len, ctx]."""
-    gap = torch.arange(ctx - q_len, ctx, device=device).unsqueeze(1) - torch.arange(ctx, device=device).unsqueeze(0)
-    return (gap >= 0) & (gap < (window or ctx))
+    i, j = torch.arange(ctx - q_len, ctx, device=device).unsqueeze(1), torch.arange(ctx, device=device).unsqueeze(0)
+    seen = (j <= i) & (i - j < (window or ctx))
+    return seen & (j >= i // chunk * chunk) if chunk else seen
 
 
 def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_q: torch.Tensor, ctx_lens: torch.Tensor,
-                    block_tables: torch.Tensor, scale: float, window: int = 0, softcap: float = 0.0) -> torch.Tensor:
-    """Causal GQA attention for a ragged batch of query chunks. q: [T, n_q, D] -> [T, n_q, D] fp32. `window`: a row sees that
-    many positions, its own included (0: all); `softcap`: scores become softcap * tanh(score / softcap) (0: they do not).
+                    block_tables: torch.Tensor, scale: float, window: int = 0, softcap: float = 0.0, out_scale: float = 1.0, chunk: int = 0,
+                    sink: bool = False, distance: torch.Tensor | None = None) -> torch.Tensor:
+    """Causal GQA attention for a ragged batch of query chunks. q: [T, n_q, D] -> [T, n_q, D] fp32. The rest as in
+    `ops.ScoreMods`.
 
     Sequence b owns query rows cu_q[b]:cu_q[b+1]; these are the last q_len positions of a context of ctx_lens[b]
     tokens whose keys/values are all in the cache already.
@@ -145,9 +147,15 @@ def paged_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tenso
         scores = torch.einsum("qhd,khd->hqk", qq, k) * scale
         if softcap:
             scores = softcap * torch.tanh(scores / softcap)
-        scores = scores.masked_fill(~visible(ctx, ql, window, q.device).unsqueeze(0), float("-inf"))
-        p = torch.softmax(scores, dim=-1)
-        out[s:e] = torch.einsum("hqk,khd->qhd", p, v)
+        if distance is not None:
+            gap = (torch.arange(ctx - ql, ctx)[:, None] - torch.arange(ctx)[None]).clamp_min(0).float()
+            scores = scores - distance[0][:, None, None] * torch.log1p(distance[1][:, None, None] * gap)
+        scores = scores.masked_fill(~visible(ctx, ql, window, q.device, chunk).unsqueeze(0), float("-inf"))
+        if sink:
+            p = torch.softmax(torch.cat([scores, torch.zeros_like(scores[..., :1])], dim=-1), dim=-1)[..., :-1]
+        else:
+            p = torch.softmax(scores, dim=-1)
+        out[s:e] = torch.einsum("hqk,khd->qhd", p, v) * out_scale
     return out
 
 
@@ -320,6 +328,12 @@ def residual_norm(x: torch.Tensor, weight: torch.Tensor | None, eps: float, y=No
     return x * torch.rsqrt(ms + eps) * weight, x
 
 
+def group_rms(x: torch.Tensor, groups: int, eps: float) -> torch.Tensor:
+    """RMS norm of every one of `groups` equal runs of columns by itself."""
+    z = x.reshape(*x.shape[:-1], groups, -1)
+    return (z * torch.rsqrt(z.pow(2).mean(-1, keepdim=True) + eps)).reshape(x.shape)
+
+
 def short_conv(u: torch.Tensor, w: torch.Tensor, conv_state, seq_rows, seq_state) -> torch.Tensor:
     """Causal convolution over time on the first `channels` columns of u [T, >= channels]; w [taps, channels]. Reads and
     writes the sequences' state banks [banks, taps - 1, channels]. Rows of unused sequences stay zero."""
@@ -349,6 +363,15 @@ def delta_rule(q, k, v, g, beta, S):
         S.add_(k[t].unsqueeze(-1) * u.unsqueeze(1))
         o[t] = torch.einsum("hde,hd->he", S, q[t])
     return o
+
+
+def selective_scan(dt, rate, u, B, C, S):
+    """One sequence: dt, u [T, C], rate [C, N], B, C [T, N], S [C, N] (updated in place); returns S C [T, C]."""
+    y = torch.empty_like(u)
+    for t in range(u.shape[0]):
+        S.mul_(torch.exp2(dt[t].unsqueeze(-1) * rate)).add_((dt[t] * u[t]).unsqueeze(-1) * B[t])
+        y[t] = S @ C[t]
+    return y
 
 
 def gated_linear(q, k, v, a, S):

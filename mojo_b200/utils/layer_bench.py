@@ -236,7 +236,7 @@ def kernel_table(size: dict) -> list[dict]:
         io = T * (Cd + H + 3 * H * d) * 2
         hist = n_seq * (taps - 1) * Cd * 2 * (2 if dec else 1)
         add("delta_decode" if dec else "delta_scan + out", "rekudra", case,
-            lambda: ops.delta_rule(pd, dg, dp, bd, st, seq, Cd, H, H, d, d, H * d, 1e-5), state_bytes + io + hist, fma=4.0 * T * H * d * d)
+            lambda: ops.delta_rule(pd, dg[:, :H * d], dg[:, H * d:2 * H * d], dp, bd, st, seq, Cd, H, H, d, d, H * d, 1e-5), state_bytes + io + hist, fma=4.0 * T * H * d * d)
     return tab.rows
 
 
@@ -425,7 +425,7 @@ def pilutar_kernel_table(size: dict) -> list[dict]:
         pd, dg, taps = rnd(T, 3 * nq + H), rnd(T, 2 * nq), 4
         dp = ops.DeltaParams(f32(taps, 3 * nq, std=0.3), -ones[:H], torch.full((nq,), -3.0, device=dev), ones[:d])
         bank = rnd(2 * n_seq, taps - 1, 3 * nq)
-        add("delta_rule", "rekudra", case, lambda: ops.delta_rule(pd, dg, dp, bank, state, seq, 3 * nq, H, H, d, d, nq, 1e-5),
+        add("delta_rule", "rekudra", case, lambda: ops.delta_rule(pd, dg[:, :nq], dg[:, nq:2 * nq], dp, bank, state, seq, 3 * nq, H, H, d, d, nq, 1e-5),
             state_bytes + T * (6 * nq + H) * 2 + n_seq * (taps - 1) * 6 * nq * (2 if dec else 1), fma=0.0 if dec else 4.0 * T * H * d * d)
         # --- latent attention
         cache, plain = rnd(n_seq * per, page, R + Q), rnd(n_seq * per, page, R)

@@ -421,7 +421,7 @@ def test_gated_delta_rule(target, heads, kv, dim, vdim, taps):
     f32 = lambda t: dev(t, target, torch.float32)  # noqa: E731
     params = ops.DeltaParams(f32(w.T), f32(-torch.exp(a_log)), f32(bias), f32(norm))
     cols = H * vdim + 5
-    out = ops.delta_rule(proj, dg, params, bank, state, seq, b_off, H, kv, dim, vdim, cols, 1e-4)
+    out = ops.delta_rule(proj, dg[:, :H * dim], dg[:, H * dim:H * (dim + vdim)], params, bank, state, seq, b_off, H, kv, dim, vdim, cols, 1e-4)
     if target[0] == "cuda":
         ops.check_status()
     close(out[:, :H * vdim], torch.cat(want_o), target)
