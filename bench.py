@@ -75,9 +75,9 @@ def parse_args():
     ap.add_argument("--secondary", default="auto", choices=["auto", "on", "off"],
                     help="also measure the 70B fp8 and DeepSeek configurations (auto: when the headline model runs on 8 GPUs)")
     ap.add_argument("--whole-batch", action="store_true", help="time one window that runs the whole request set to completion (the mode of the fixed-batch configurations)")
-    ap.add_argument("--layer-bench", nargs="?", const="rekudra", default=None, choices=["rekudra", "rerupel", "pilutar"],
+    ap.add_argument("--layer-bench", nargs="?", const="rekudra", default=None, choices=["rekudra", "rerupel", "pilutar", "noridra"],
                     help="instead of the headline: prefill / decode throughput and kernel rooflines of a design's layers beside those of its closest "
-                         "model at equal size (rekudra: beside Llama; rerupel: beside DeepSeek-V2; pilutar: beside Rerupel)")
+                         "model at equal size (rekudra: beside Llama; rerupel: beside DeepSeek-V2; pilutar: beside Rerupel; noridra: beside Pilutar)")
     ap.add_argument("--layers", type=int, default=None, help="debug only: marks the result invalid")
     ap.add_argument("--profile", default=None, help="debug only: write a per-kernel table of a few steps to this file")
     ap.add_argument("--tune-report", default=None, help="debug only: append the start-up tuning tables (GEMM configurations, all-reduce forms) to this file")

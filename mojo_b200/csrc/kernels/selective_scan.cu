@@ -47,8 +47,25 @@ __device__ __forceinline__ void store_packed(float* p, const uint64_t (&v)[N / 2
     }
   }
 }
+// 2^x for x <= 0. The special-function unit's error has the same sign over wide stretches, which adds up in a state that decays
+// slowly: `EXACT` takes the Taylor series of e^t there.
+template <bool EXACT>
+__device__ __forceinline__ float decay(float x) {
+  if constexpr (EXACT) {
+    const float t = x * ptx::kLn2;
+    if (t > -0.25f) {
+      float p = fmaf(t, 1.0f / 720, 1.0f / 120);
+      p = fmaf(t, p, 1.0f / 24);
+      p = fmaf(t, p, 1.0f / 6);
+      p = fmaf(t, p, 0.5f);
+      p = fmaf(t, p, 1.0f);
+      return fmaf(t, p, 1.0f);
+    }
+  }
+  return ptx::ex2(x);
+}
 // One row: S <- 2^(dt rate) S + dtu B; returns S . C over this thread's states.
-template <int N>
+template <bool EXACT, int N>
 __device__ __forceinline__ float scan_row(uint64_t (&S)[N / 2], const uint64_t (&rate)[N / 2], float dt, float dtu, const uint64_t (&B)[N / 2],
                                           const uint64_t (&C)[N / 2]) {
   const uint64_t dt2 = pack2(dt, dt), u2 = pack2(dtu, dtu);
@@ -56,7 +73,7 @@ __device__ __forceinline__ float scan_row(uint64_t (&S)[N / 2], const uint64_t (
 #pragma unroll
   for (int i = 0; i < N / 2; ++i) {
     const float2 x = unpack2(mul2(dt2, rate[i]));
-    S[i] = fma2(pack2(ptx::ex2(x.x), ptx::ex2(x.y)), S[i], mul2(u2, B[i]));
+    S[i] = fma2(pack2(decay<EXACT>(x.x), decay<EXACT>(x.y)), S[i], mul2(u2, B[i]));
     y = i == 0 ? mul2(S[i], C[i]) : fma2(S[i], C[i], y);
   }
   return half_sum(y);
@@ -110,7 +127,7 @@ __global__ void __launch_bounds__(kThreads) scan_decode_kernel(const B2Selective
     next = request(seq + 1 < seq1 ? seq + 1 : n_seqs);
     if (s.row < 0) continue;      // uniform per CTA
     const float dt = softplus_fast(s.dt + bias);
-    float y = scan_row<NS>(s.S, rate, dt, dt * s.u, s.B, s.C);
+    float y = scan_row<sizeof(T) == 4, NS>(s.S, rate, dt, dt * s.u, s.B, s.C);
 #pragma unroll
     for (int o = L / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
     if (!in) continue;
@@ -230,7 +247,7 @@ __global__ void __launch_bounds__(kThreads) scan_kernel(const B2SelectiveScanArg
         uint64_t B[NS / 2], C[NS / 2];
         load_packed<NS>(b_sm + (r0 + i) * SP + l * NS, B);
         load_packed<NS>(c_sm + (r0 + i) * SP + l * NS, C);
-        y[i] = scan_row<NS>(S, rate, s.x, s.y, B, C);
+        y[i] = scan_row<sizeof(T) == 4, NS>(S, rate, s.x, s.y, B, C);
       }
       // the sums over the lanes of a channel: a lane keeps the half of the rows that its bit names
 #pragma unroll

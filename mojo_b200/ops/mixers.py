@@ -186,7 +186,8 @@ def post_norm(x: torch.Tensor | None, norm: GroupNorm, dtype: torch.dtype, seq: 
             v = normed(v, then)
         if rows is not None:
             return v.to(dtype), None
-        v = torch.where((seq.row_seq >= 0).unsqueeze(-1), v, 0.0)
+        used = (seq.row_seq >= 0) & (seq.seq_state[seq.row_seq.clamp_min(0).long(), 1] >= 0)
+        v = torch.where(used.unsqueeze(-1), v, 0.0)
         h = v if conv is None else v + reference.short_conv(v, conv.w, conv.state, seq.seq_rows, seq.seq_state)
         return h.to(dtype), v
     make = torch.empty if norm.width == W else torch.zeros

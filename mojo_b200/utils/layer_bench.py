@@ -1,12 +1,13 @@
 """A design beside the closest one at equal layer sizes: prefill and decode throughput of a few layers through the serving
 engine, and each design's own kernels against their rooflines. Random weights, synthetic prompts, one GPU
 (`bench.py --layer-bench`: Rekudra beside Llama; `bench.py --layer-bench rerupel`: Rerupel beside DeepSeek-V2;
-`bench.py --layer-bench pilutar`: Pilutar beside Rerupel, its single kernels also beside the like ones of Llama and Rekudra).
+`bench.py --layer-bench pilutar`: Pilutar beside Rerupel, its single kernels also beside the like ones of Llama and Rekudra;
+`bench.py --layer-bench noridra`: Noridra beside Pilutar, its single kernels also beside those of Rekudra).
 
 Steps are timed with CUDA events around the engine's device work, medians over repeats after warm-up; every step streams
 weights and caches larger than L2. Single kernels are timed with an L2 flush before each launch. Rooflines use the copy
 bandwidth and the bf16 rate measured on the machine; the scans of recurrent layers work on f32 matrices, so their compute
-bound is the f32 FMA rate (SMs x 128 lanes x maximum clock)."""
+bound is the f32 FMA rate (SMs x 128 lanes x maximum clock), or for exponentials that of the special-function units (16 lanes)."""
 from __future__ import annotations
 
 import json
@@ -15,12 +16,14 @@ from pathlib import Path
 
 import torch
 
-DESIGNS = {"rekudra": ("llama", "rekudra"), "rerupel": ("deepseek", "rerupel"), "pilutar": ("rerupel_plain", "pilutar")}      # (closest model, design)
+DESIGNS = {"rekudra": ("llama", "rekudra"), "rerupel": ("deepseek", "rerupel"), "pilutar": ("rerupel_plain", "pilutar"),
+           "noridra": ("pilutar_short", "noridra")}      # (closest model, design)
 SIZES = {"2048x16": dict(width=2048, heads=16, kv=4, dim=128, ffn=8192), "4096x32": dict(width=4096, heads=32, kv=8, dim=128, ffn=14336)}
 # DeepSeek-V2-Lite's layers, and the same at twice the width; latents of 512 columns, 64 experts of which 6 are used
 MOE_SIZES = {"2048x16": dict(width=2048, heads=16, dim=128, rank=512, rope=64, ffn=10944, experts=64, top=6, expert_ffn=1408),
              "4096x32": dict(width=4096, heads=32, dim=128, rank=512, rope=64, ffn=14336, experts=64, top=6, expert_ffn=1408)}
 PILUTAR_SIZES = {k: dict(v, kv=4 * (i + 1), rope=32, window=1024, groups=8, keep=4, identity=2) for i, (k, v) in enumerate(MOE_SIZES.items())}
+NORIDRA_SIZES = {k: dict(v, chunk=1024, state=16, norm_groups=4) for k, v in PILUTAR_SIZES.items()}
 VOCAB, LAYERS = 32000, 8
 MOE_RUNS = 9           # one dense layer and eight with experts (the design: four, passed twice)
 PREFILL = [(1, 2048), (2, 2048), (8, 512)]        # (prompts, tokens each), one step
@@ -31,14 +34,18 @@ def peaks() -> dict:
     p = Path(__file__).resolve().parents[2] / "MEASURED_PEAKS.json"
     m = json.loads(p.read_text()) if p.exists() else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0, "sm_max_mhz": 1965.0}
     return {"hbm": m["hbm_gbs"] * 1e9, "bf16": m["bf16_tflops"] * 1e12, "fma": 148 * 128 * m.get("sm_max_mhz", 1965.0) * 1e6,
+            "sfu": 148 * 16 * m.get("sm_max_mhz", 1965.0) * 1e6,
             "source": "measured" if p.exists() else "fallback"}
 
 
 def model_config(design: str, size: dict):
-    from ..models.config import ModelConfig, pilutar, rekudra, rerupel
+    from ..models.config import ModelConfig, noridra, pilutar, rekudra, rerupel
 
-    if design == "pilutar":
-        return pilutar(size["width"], MOE_RUNS, size["heads"], size["kv"], size["dim"], size["rank"], size["rope"], size["ffn"], VOCAB,
+    if design == "noridra":
+        return noridra(size["width"], LAYERS, size["heads"], size["kv"], size["dim"], VOCAB, size["experts"], size["top"], size["expert_ffn"], size["chunk"],
+                       size["state"], size["norm_groups"], positions=4096)
+    if design in ("pilutar", "pilutar_short"):
+        return pilutar(size["width"], LAYERS if design == "pilutar_short" else MOE_RUNS, size["heads"], size["kv"], size["dim"], size["rank"], size["rope"], size["ffn"], VOCAB,
                        size["experts"] - size["identity"], size["top"], size["expert_ffn"], 2 * size["expert_ffn"], size["window"], size["groups"], size["keep"],
                        size["identity"])
     if design == "rerupel_plain":      # every layer run with weights of its own
@@ -167,11 +174,11 @@ class KernelTable:
         self.pk, self.rows = peaks(), []
         self.flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
 
-    def add(self, name, design, case, fn, nbytes, fma=0.0, mma=0.0):
+    def add(self, name, design, case, fn, nbytes, fma=0.0, mma=0.0, sfu=0.0):
         pk = self.pk
         us = time_kernel(fn, self.flush)
-        floor = max(nbytes / pk["hbm"], fma / pk["fma"], 2 * mma / pk["bf16"]) * 1e6
-        bound = "hbm" if floor == nbytes / pk["hbm"] * 1e6 else "fma" if fma and floor == fma / pk["fma"] * 1e6 else "bf16"
+        bound, floor = max((("hbm", nbytes / pk["hbm"]), ("fma", fma / pk["fma"]), ("bf16", 2 * mma / pk["bf16"]), ("sfu", sfu / pk["sfu"])), key=lambda b: b[1])
+        floor *= 1e6
         self.rows.append({"kernel": name, "design": design, "case": case, "us": round(us, 2), "roofline_us": round(floor, 2), "bound": bound,
                           "fraction": round(floor / us, 3)})
 
@@ -502,13 +509,113 @@ def pilutar_kernel_table(size: dict) -> list[dict]:
     return tab.rows
 
 
+def noridra_kernel_table(size: dict) -> list[dict]:
+    """Noridra's kernels beside those of Pilutar, and of Rekudra where that has the like one."""
+    from .. import ops
+    from ..ops import reference
+
+    W, H, G, d, E, k, F, S = (size[n] for n in ("width", "heads", "kv", "dim", "experts", "top", "expert_ffn", "state"))
+    win, chunk, page, dev, bf, taps, I, dr = size["window"], size["chunk"], 128, torch.device("cuda"), torch.bfloat16, 4, 2 * W, W // 16
+    tab = KernelTable()
+    add = tab.add
+    f32 = lambda *s, std=1.0: rnd(*s, dtype=torch.float32, std=std)  # noqa: E731
+    ones = torch.ones(max(W, H * d, I), device=dev)
+    table, table_d = reference.rope_table(4096, d // 2, 1e4).to(dev), reference.rope_table(4096, d, 1e4).to(dev)
+    gu, down, up = rnd(E, 2 * F, W, std=W ** -0.5), rnd(E, W, F, std=F ** -0.5), rnd(E, F, W, std=W ** -0.5)
+    router = rnd(E + 8, W, std=W ** -0.5)
+    for case, seq, ctx, n_seq, T in (("decode 128 x 1024", step_rows(128, []), 1024, 128, 128), ("prefill 2 x 2048", step_rows(0, [2048, 2048]), 2048, 2, 4096)):
+        dec = seq.n_decode > 0
+        per = ctx // page + 1
+        bt = torch.arange(n_seq * per, dtype=torch.int32, device=dev).view(n_seq, per)
+        cl = torch.full((n_seq,), ctx, dtype=torch.int32, device=dev)
+        cu = torch.arange(n_seq + 1, dtype=torch.int32, device=dev) * (T // n_seq)
+        base = torch.arange(n_seq, device=dev) * per * page
+        slots = base + ctx - 1 if dec else (base[:, None] + torch.arange(ctx, device=dev)[None]).flatten()
+        pos = torch.full((T,), ctx - 1, dtype=torch.int32, device=dev) if dec else torch.arange(ctx, dtype=torch.int32, device=dev).repeat(n_seq)
+        work = None if dec else torch.from_numpy(ops.prefill_work_items(cu.cpu().numpy(), cl.cpu().numpy(), 0)).cuda()
+        meta = ops.AttnMeta(cu, cl, bt, n_seq if dec else 0, T // n_seq, ctx, work=work, n_items=0 if dec else work.shape[0])
+        near_c = float(n_seq * min(ctx, chunk)) if dec else n_seq * sum(t % chunk + 1 for t in range(ctx))      # (query, key) pairs
+        near_w = float(n_seq * min(ctx, win)) if dec else n_seq * sum(min(t + 1, win) for t in range(ctx))
+        keys = n_seq * min(ctx, chunk) if dec else n_seq * ctx
+        # --- residual, norm, convolution ahead of a sublayer
+        x, y, h, w1 = f32(T, W), rnd(T, W), rnd(T, W), ones[:W]
+        conv = ops.InputConv(f32(taps, W, std=0.3), f32(2 * n_seq, taps - 1, W))
+        norm = ops.GroupNorm(size["norm_groups"], 1e-6, W)
+        p = ops.MoeWeights(router[:E], gu, down, E, k, "sigmoid", on_input=True)
+        pp = ops.MoeWeights(router[:E], up, down, E, k, "softmax", True, 1.0, None, f32(E, std=0.02), size["groups"], size["keep"])
+        ex, exp = ops.moe_experts(h, p), ops.moe_experts(h, pp)
+        banks = n_seq * (taps - 1) * W * 4 * (2 if dec else 1)
+        add("post_norm, convolution", "noridra", case, lambda: ops.post_norm(x, norm, bf, seq, ops.Finished(w1, y), w1, 2.0, conv=conv), T * W * 12 + banks)
+        add("residual_norm, layer norm", "pilutar", case, lambda: ops.residual_norm(x, w1, 1e-5, bf, ops.Finished(None, y), bias=w1), T * W * 12)
+        add("post_norm, convolution, of experts", "noridra", case, lambda: ops.post_norm(x, norm, bf, seq, ops.Finished(w1, None, ex), w1, 2.0, conv=conv),
+            T * W * (2 * k + 10) + banks)
+        add("residual_norm, layer norm, of experts", "pilutar", case, lambda: ops.residual_norm(x, w1, 1e-5, bf, ops.Finished(None, None, exp), bias=w1),
+            T * W * (2 * k + 10))
+        # --- attention
+        nq, nk = H * d, G * d
+        kc, vc = (rnd(n_seq * per, G, page, d) for _ in range(2))
+        pa, q = rnd(T, 2 * nq + nk), rnd(T, nq)
+        add("head_norm_qkv", "noridra", case, lambda: ops.head_norm_qkv(pa, ones[:d], ones[:d], slots, kc, vc, H, G, d, nq, d, 1e-6), T * (4 * nq + 6 * nk))
+        qn, pn = ops.QkvNorm(ones.new_zeros(nq + 2 * nk), ones[:nq], ones[:nk]), rnd(T, nq + 2 * nk)
+        add("norm_qkv", "pilutar", case, lambda: ops.norm_qkv(pn, qn, table, pos, slots, kc, vc, H, G, d, d, d, 1e-5), T * (nq + 2 * nk) * 4)
+        mods = ops.ScoreMods(softcap=30.0, chunk=chunk, sink=True, distance=torch.full((2, H), 0.5, device=dev))
+        gate = pa[:, nq + nk:]
+        add("attention, chunks, bias, sink, gate", "noridra", case, lambda: ops.paged_attention(q, kc, vc, meta, d ** -0.5, d, gate=gate, mods=mods),
+            keys * G * d * 4 + T * nq * 6, mma=0.0 if dec else near_c * H * d * 2)
+        mw = ops.ScoreMods(win, 30.0, 0.5)
+        add("attention, window, capped", "pilutar", case, lambda: ops.paged_attention(q, kc, vc, meta, d ** -0.5, d, mods=mw),
+            n_seq * (min(ctx, win) if dec else ctx) * G * d * 4 + T * nq * 4, mma=0.0 if dec else near_w * H * d * 2)
+        # --- recurrences
+        state = torch.zeros(n_seq, H, d, d, device=dev)
+        state_bytes = n_seq * H * d * d * 4 * (2 if dec else 1)
+        pd, bank = rnd(T, 4 * nq + 2 * H), rnd(2 * n_seq, taps - 1, 3 * nq)
+        cw = f32(taps, 3 * nq, std=0.3)
+        dn = ops.DeltaParams(cw, -ones[:H], torch.full((H,), -3.0, device=dev), ones[:d], True)
+        hist = n_seq * (taps - 1) * 6 * nq * (2 if dec else 1)
+        add("delta_rule, decay per head", "noridra", case,
+            lambda: ops.delta_rule(pd, pd[:, 3 * nq + H:3 * nq + 2 * H], pd[:, 3 * nq + 2 * H:], dn, bank, state, seq, 3 * nq, H, H, d, d, nq, 1e-6),
+            state_bytes + T * (5 * nq + 2 * H) * 2 + hist, fma=0.0 if dec else 4.0 * T * H * d * d)
+        dg, dk = rnd(T, 2 * nq), ops.DeltaParams(cw, -ones[:H], torch.full((nq,), -3.0, device=dev), ones[:d])
+        add("delta_rule", "rekudra", case, lambda: ops.delta_rule(pd, dg[:, :nq], dg[:, nq:], dk, bank, state, seq, 3 * nq, H, H, d, d, nq, 1e-5),
+            state_bytes + T * (6 * nq + H) * 2 + hist, fma=0.0 if dec else 4.0 * T * H * d * d)
+        xz, f, dt = rnd(T, 2 * I), rnd(T, dr + 2 * S), f32(T, I)
+        cs, cws = rnd(2 * n_seq, taps - 1, I), f32(taps, I, std=0.3)
+        add("conv_silu", "noridra", case, lambda: ops.conv_silu(xz, cws, ones[:I], cs, seq), T * I * 4 + n_seq * (taps - 1) * I * 2 * (2 if dec else 1))
+        kq, vq = rnd(n_seq * per, G, page, d), rnd(n_seq * per, G, page, d)
+        cq, bq = f32(taps, nq + 2 * nk, std=0.3), rnd(2 * n_seq, taps - 1, nq + 2 * nk)
+        add("conv_qkv", "rekudra", case, lambda: ops.conv_qkv(pn, cq, bq, table_d, pos, seq, slots, kq, vq, H, G, d, d, d, 1e-5),
+            T * (nq + 2 * nk) * 4 + n_seq * (taps - 1) * (nq + 2 * nk) * 2 * (2 if dec else 1))
+        sp = ops.ScanParams(-torch.rand(I, S, device=dev) - 0.1, torch.full((I,), -4.0, device=dev), ones[:I])
+        ss = torch.zeros(n_seq, I, S, device=dev)
+        add("selective_scan", "noridra", case, lambda: ops.selective_scan(dt, xz[:, :I], xz[:, I:], f[:, dr:dr + S], f[:, dr + S:], sp, ss, seq),
+            n_seq * I * S * 4 * (2 if dec else 1) + T * I * 10, sfu=0.0 if dec else float(T) * I * S)
+        pg, zg = rnd(T, 4 * nq), f32(T, nq)
+        gp, og = ops.GatedLinearParams(torch.full((nq,), 2.0, device=dev), ones[:d], 16.0), rnd(T, nq)
+        add("gated_linear", "pilutar", case, lambda: ops.gated_linear(pg, zg, gp, state, seq, H, d, d, 1e-5, og), state_bytes + T * nq * 14,
+            fma=0.0 if dec else 3.0 * T * H * d * d)
+        # --- experts
+        logits = ops.linear_f32(h, router)
+        used = float(min(E, T * k))
+        add("router, experts, weighted inputs", "noridra", case, lambda: ops.moe_experts(h, p, logits), used * 3 * W * F * 2 + T * k * (3 * W + 2 * F) * 2,
+            mma=float(T) * k * 3 * W * F)
+        add("router, experts", "pilutar", case, lambda: ops.moe_experts(h, pp, logits), used * 2 * W * F * 2 + T * k * (3 * W + 2 * F) * 2, mma=float(T) * k * 2 * W * F)
+        # --- products of the scan's small matrices
+        w_x, w_dt, low, w_dec = rnd(dr + 2 * S, I, std=I ** -0.5), rnd(I, dr, std=dr ** -0.5), rnd(T, 4 * nq)[:, :16], rnd(nq, 16)
+        u = xz[:, :I].contiguous()
+        add("gemm, step sizes | B | C", "noridra", case, lambda: ops.linear(u, w_x), (w_x.numel() + u.numel() + T * (dr + 2 * S)) * 2, mma=float(T) * w_x.numel())
+        add("gemm, step sizes, f32", "noridra", case, lambda: ops.linear_f32(f[:, :dr], w_dt), (w_dt.numel() + T * dr) * 2 + T * I * 4, mma=float(T) * w_dt.numel())
+        add("gemm, decay logits, f32", "pilutar", case, lambda: ops.linear_f32(low, w_dec), (w_dec.numel() + T * 16) * 2 + T * nq * 4, mma=float(T) * w_dec.numel())
+    return tab.rows
+
+
 def run(args) -> dict:
     from .clocks import ClockSampler
 
     base, design = DESIGNS[args.layer_bench]
-    sizes, table = {"rekudra": (SIZES, kernel_table), "rerupel": (MOE_SIZES, latent_kernel_table), "pilutar": (PILUTAR_SIZES, pilutar_kernel_table)}[design]
+    sizes, table = {"rekudra": (SIZES, kernel_table), "rerupel": (MOE_SIZES, latent_kernel_table), "pilutar": (PILUTAR_SIZES, pilutar_kernel_table),
+                    "noridra": (NORIDRA_SIZES, noridra_kernel_table)}[design]
     out = {"metric": f"layer throughput, {design} beside {base} at equal layer sizes", "unit": "tok/s", "n_gpus": 1, "dtype": "bf16",
-           "layers": LAYERS if design == "rekudra" else MOE_RUNS, "data": "synthetic: uniform-random token ids, random weights", "peaks": peaks(), "sizes": {}}
+           "layers": LAYERS if design in ("rekudra", "noridra") else MOE_RUNS, "data": "synthetic: uniform-random token ids, random weights", "peaks": peaks(), "sizes": {}}
     with ClockSampler(0) as clocks:
         for name, size in sizes.items():
             rec = {"kernels": table(size)}

@@ -232,7 +232,7 @@ def layer_tensors(spec, width, taps):
 def random_weights(cfg, seed=0, sharp=1.0):
     """Checkpoint tensors by name, rounded to bfloat16 values (held in float32). `sharp` scales the queries, so that single
     scores stand out. Routers look at one channel per expert, where every token's embedding has the same levels in an order of
-    its own and the layers add next to nothing: choices vary with the token and are no close calls, which rounding could decide
+    its own and the layers add nothing: choices vary with the token and are no close calls, which rounding could decide
     either way."""
     g = torch.Generator().manual_seed(seed)
 
@@ -270,8 +270,10 @@ def random_weights(cfg, seed=0, sharp=1.0):
                 t = rnd(*shape, std=shape[-1] ** -0.5)
             if E and name in ("norm1", "norm2"):
                 t[:E] = 1.0
-            if E and (name in ("canon1", "canon2", "ls1", "ls2")):
+            if E and name.startswith("canon"):
                 t[:E] *= 0.02
+            if E and name.startswith("ls"):
+                t[:E] = 0.0
             w[f"l{i}.{name}"] = t
     if E:
         w["final.norm"][:E] = 0.02                    # the logits do not see them
