@@ -82,6 +82,7 @@ struct RawVec {
 #pragma unroll
     for (int i = 0; i < VEC; ++i) v[i] = 0.0f;
   }
+  __device__ __forceinline__ void set(T a, T b) { v[0] = a; v[1] = b; }
   __device__ __forceinline__ float get(int i) const { return v[i]; }
 };
 template <>
@@ -102,6 +103,9 @@ struct RawVec<__nv_bfloat16, 2> {
   __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint32_t*>(p); }
   __device__ __forceinline__ void store(__nv_bfloat16* p) const { *reinterpret_cast<uint32_t*>(p) = v; }
   __device__ __forceinline__ void zero() { v = 0; }
+  __device__ __forceinline__ void set(__nv_bfloat16 a, __nv_bfloat16 b) {
+    v = static_cast<uint32_t>(__bfloat16_as_ushort(a)) | static_cast<uint32_t>(__bfloat16_as_ushort(b)) << 16;
+  }
   __device__ __forceinline__ float get(int i) const { return i & 1 ? ptx::bf16_hi(v) : ptx::bf16_lo(v); }
 };
 
