@@ -17,9 +17,6 @@
 namespace b2 {
 namespace {
 
-#ifndef B2_FEW
-#define B2_FEW (4ll * 128 * 1024)
-#endif
 constexpr int kThreads = 128;
 constexpr int kAhead = 4;           // sequences on their way to a decode CTA
 constexpr int kMaxSeqs = 128;       // sequences of one decode CTA
@@ -314,7 +311,8 @@ template <typename T, int L, int NS>
 int launch_decode(const B2SelectiveScanArgs& a, const B2SeqRows& s, int n, Status* status, cudaStream_t stream) {
   constexpr int CH = kThreads / L;
   const int64_t blocks = (a.channels + CH - 1) / CH;
-  int64_t per = (n * blocks + 4 * kNumSMs - 1) / (4 * kNumSMs);      // one wave of CTAs
+  const int64_t runs = blocks < 4 * kNumSMs ? 4 * kNumSMs / blocks : 1;      // of sequences, so that all CTAs fit at once
+  int64_t per = (n + runs - 1) / runs;
   if (per > kMaxSeqs) per = kMaxSeqs;
   launch_pdl(scan_decode_kernel<T, L, NS>, dim3(static_cast<unsigned>(blocks), static_cast<unsigned>((n + per - 1) / per)), dim3(kThreads), 0, stream, a, s, n,
              static_cast<int>(per), status);
@@ -346,7 +344,7 @@ int launch_scan(const B2SelectiveScanArgs& a, const B2SeqRows& s, int first, int
 template <typename T>
 int dispatch_scan(const B2SelectiveScanArgs& a, const B2SeqRows& s, int first, int n, Status* status, cudaStream_t stream) {
   // few channels in all: more lanes for each
-  const bool few = static_cast<int64_t>(a.channels) * n * a.states < B2_FEW;
+  const bool few = static_cast<int64_t>(a.channels) * n * a.states < 4ll * 128 * 1024;
   switch (a.states) {
     case 4: return launch_scan<T, 2, 2>(a, s, first, n, status, stream);
     case 8: return launch_scan<T, 4, 2>(a, s, first, n, status, stream);

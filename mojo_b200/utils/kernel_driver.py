@@ -5,7 +5,7 @@ profiler capture of one kernel; with `--time` the case is timed with CUDA events
 Cases: gemm_large, gemm_pair (the same product on CTA pairs), gemm_prefill, gemm_decode, gemm_swiglu, gemm_fp8,
 gemm_fp8_decode, gemm_fp8_decode_nosplit (a narrow tensor-parallel shard at 256 tokens, with and without split-K),
 attn_decode, attn_prefill, mla_decode, mla_prefill, latent_decode, latent_prefill, moe_local, residual_norm, norm_qkv, attn_capped,
-gated_scan, gated_scan_long (one prompt), gated_decode, rmsnorm, sampling (arg-max), sample_topk_topp, gemm_gguf_q4k,
+gated_scan, gated_scan_long (one prompt), gated_decode, post_norm, attn_chunks, selective_scan, scan_decode, rmsnorm, sampling (arg-max), sample_topk_topp, gemm_gguf_q4k,
 gemm_gguf_q6k, rope_kvwrite, all_reduce_norm_single.
 """
 from __future__ import annotations
@@ -157,8 +157,29 @@ def _case(name: str):
         p = ops.QkvNorm(*(torch.ones(n, device=DEV) for n in ((H + 2 * G) * D, H * D, G * D)))
         pos, slots = torch.arange(T, dtype=torch.int32, device=DEV), torch.arange(T, dtype=torch.int64, device=DEV)
         return (lambda: ops.norm_qkv(proj, p, table, pos, slots, kc, vc, H, G, D, D, D, 1e-5)), 0.0, T * (H + 2 * G) * D * 4
-    if name == "attn_capped":
-        # two prompts of 2048 tokens, 32 query heads on 8, a window of 1024 and capped scores
+    if name == "post_norm":
+        # eight prompts of 2048 rows: sum, norm in four groups, convolution of four taps
+        from .layer_bench import step_rows
+
+        T, W, n = 16384, 4096, 8
+        seq, one = step_rows(0, [T // n] * n), torch.ones(W, device=DEV)
+        x, y, conv = rnd(T, W).float(), rnd(T, W), ops.InputConv(rnd(4, W).float(), torch.zeros(2 * n, 3, W, device=DEV))
+        norm, done = ops.GroupNorm(4, 1e-6, W), ops.Finished(one, y)
+        return (lambda: ops.post_norm(x, norm, torch.bfloat16, seq, done, one, 2.0, conv=conv)), 0.0, T * W * 12
+    if name in ("selective_scan", "scan_decode"):
+        # 4096 channels of 16 states: two prompts of 2048 rows, or 256 decode rows
+        from .layer_bench import step_rows
+
+        I, S, n = 4096, 16, 256 if name == "scan_decode" else 2
+        seq = step_rows(n, []) if name == "scan_decode" else step_rows(0, [2048] * n)
+        T = seq.row_seq.numel()
+        xz, f, dt, state = rnd(T, 2 * I), rnd(T, 128 + 2 * S), rnd(T, I).float(), torch.zeros(n, I, S, device=DEV)
+        p = ops.ScanParams(-rnd(I, S).float().abs() - 0.1, torch.full((I,), -4.0, device=DEV), torch.ones(I, device=DEV))
+        run = lambda: ops.selective_scan(dt, xz[:, :I], xz[:, I:], f[:, 128:128 + S], f[:, 128 + S:], p, state, seq)  # noqa: E731
+        return run, 6.0 * T * I * S, n * I * S * 4 * (2 if seq.n_decode else 1) + T * I * 10
+    if name in ("attn_capped", "attn_chunks"):
+        # two prompts of 2048 tokens, 32 query heads on 8, capped scores: a window of 1024, or chunks of 1024 with distance bias,
+        # sink and a gate by element
         S, L, H, G, D, page, win = 2, 2048, 32, 8, 128, 128, 1024
         kc, vc, q = rnd(S * L // page, G, page, D), rnd(S * L // page, G, page, D), rnd(S * L, H * D)
         cu = torch.arange(0, (S + 1) * L, L, dtype=torch.int32, device=DEV)
@@ -166,6 +187,9 @@ def _case(name: str):
         work = torch.from_numpy(ops.prefill_work_items(cu.cpu().numpy(), cl.cpu().numpy(), 0)).to(DEV)
         meta = ops.AttnMeta(cu, cl, bt, 0, L, L, work=work, n_items=work.shape[0])
         pairs = S * sum(min(t + 1, win) for t in range(L))
+        if name == "attn_chunks":
+            mods, gate, pairs = ops.ScoreMods(softcap=30.0, chunk=win, sink=True, distance=torch.full((2, H), 0.5, device=DEV)), rnd(S * L, H * D), S * L * (win + 1) / 2
+            return (lambda: ops.paged_attention(q, kc, vc, meta, D ** -0.5, D, gate=gate, mods=mods)), 4.0 * pairs * H * D, S * L * (3 * H + 2 * G) * D * 2
         return (lambda: ops.paged_attention(q, kc, vc, meta, D ** -0.5, D, mods=ops.ScoreMods(win, 30.0, 0.5))), 4.0 * pairs * H * D, S * L * (2 * H + 2 * G) * D * 2
     if name in ("tp_gemm_rs_single", "tp_ag_gemm_single"):
         # The fused tensor-parallel kernels on ONE rank (a world of one: the only peer is this GPU's own region), so that
@@ -291,7 +315,7 @@ def _case(name: str):
 
 CASES = ("gemm_large", "gemm_pair", "gemm_prefill", "gemm_decode", "gemm_swiglu", "gemm_fp8", "gemm_fp8_decode", "gemm_fp8_decode_nosplit",
          "attn_decode", "attn_prefill", "mla_decode", "mla_prefill", "latent_decode", "latent_prefill", "moe_local", "residual_norm", "norm_qkv", "attn_capped",
-         "gated_scan", "gated_scan_long", "gated_decode", "rmsnorm", "sampling", "sample_topk_topp", "gemm_gguf_q4k", "gemm_gguf_q6k",
+         "gated_scan", "gated_scan_long", "gated_decode", "post_norm", "attn_chunks", "selective_scan", "scan_decode", "rmsnorm", "sampling", "sample_topk_topp", "gemm_gguf_q4k", "gemm_gguf_q6k",
          "rope_kvwrite", "all_reduce_norm_single")
 # single-rank forms of the fused tensor-parallel and expert-parallel kernels (profiling only): tp_gemm_rs_single,
 # tp_ag_gemm_single, moe_ep_single
