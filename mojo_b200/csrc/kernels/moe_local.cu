@@ -36,8 +36,9 @@ __device__ __forceinline__ int warp_argmax(const float (&v)[NV], int lane, int n
   return min(at, none);
 }
 
-// One warp per row, NV logits per lane. CHOICE: what chooses is not the score itself (a correction is added, groups are left
-// out); then scores and choice scores are held apart.
+// One warp per row, NV logits per lane. The largest logits have the largest scores, and differ where scores are as good as one.
+// CHOICE: what chooses is not the score itself (a correction is added, groups are left out); then scores and choice scores are held
+// apart.
 template <int NV, bool CHOICE>
 __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ correction,
                                                         float* __restrict__ weights, int32_t* __restrict__ ids, int32_t* __restrict__ place,
@@ -55,18 +56,17 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
     mx = fmaxf(mx, v[i]);
   }
   float inv = 1.0f;
-  if (sigmoid) {
-#pragma unroll
-    for (int i = 0; i < NV; ++i) v[i] = lane + 32 * i < outputs ? sigmoid_f32(v[i]) : -INFINITY;
-  } else {
-    mx = warp_max(mx);
+  const auto score_of = [&](float logit) { return sigmoid ? sigmoid_f32(logit) : expf(logit - mx); };
+  if (!sigmoid) mx = warp_max(mx);
+  if (CHOICE || !sigmoid) {
     float sum = 0.0f;
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
-      v[i] = lane + 32 * i < outputs ? expf(v[i] - mx) : -INFINITY;
-      if (v[i] > 0.0f) sum += v[i];
+      const float p = lane + 32 * i < outputs ? score_of(v[i]) : -INFINITY;
+      if (p > 0.0f) sum += p;
+      if constexpr (CHOICE) v[i] = p;
     }
-    inv = 1.0f / warp_sum(sum);
+    if (!sigmoid) inv = 1.0f / warp_sum(sum);
   }
   float score[CHOICE ? NV : 1];
   if constexpr (CHOICE) {
@@ -121,6 +121,8 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const float* __restrict_
       for (int i = 0; i < NV; ++i)
         if (best_e == lane + 32 * i) own = score[i];
       best = __shfl_sync(0xffffffffu, own, best_e & 31);
+    } else {
+      best = score_of(best);
     }
 #pragma unroll
     for (int i = 0; i < NV; ++i)

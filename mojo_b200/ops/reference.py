@@ -440,7 +440,7 @@ def moe_route(router_logits: torch.Tensor, top_k: int, norm_topk: bool = False, 
     added to the scores for the choice only; with `groups` > 1 the choice is among the `keep` groups of neighbours that hold
     the largest such scores. Returns (weights [T, k], ids [T, k])."""
     p = torch.sigmoid(router_logits.float()) if sigmoid else torch.softmax(router_logits.float(), dim=-1)
-    c = p if correction is None else p + correction.float()
+    c = router_logits.float() if correction is None and keep >= groups else p if correction is None else p + correction.float()
     if keep < groups:
         per = c.shape[1] // groups
         best = c.view(-1, groups, per).amax(-1).topk(keep, dim=-1).indices

@@ -674,6 +674,24 @@ def test_weights_on_the_experts_input(target, experts, top, rows):
     sync(target)
 
 
+@pytest.mark.parametrize("target", TARGETS)
+@pytest.mark.parametrize("scoring", ["sigmoid", "softmax"])
+def test_choice_among_scores_that_round_to_the_same(target, scoring):
+    """Where scores are one (or zero) in 32 bits, the larger logit still goes first."""
+    E, top, rows, W = 24, 3, 50, 16
+    g = torch.Generator().manual_seed(2)
+    logits = torch.stack([torch.randperm(E, generator=g) * (0.25 if scoring == "sigmoid" else 8.0) + (20.0 if scoring == "sigmoid" else -100.0) for _ in range(rows)])
+    h = torch.zeros(rows, W) + 1.0
+    gu, down = torch.zeros(E, 32, W), torch.zeros(E, W, 16)
+    for e in range(E):                                                       # an expert's result names it
+        gu[e, :, 0], down[e, :, 0] = 1.0, e + 1.0
+    p = ops.MoeWeights(dev(torch.zeros(E, W), target), dev(gu, target), dev(down, target), E, top, scoring)
+    ex = ops.moe_experts(dev(h, target), p, f32(logits, target))
+    sync(target)
+    name = ex.rows.float().cpu()[ex.slot.long().cpu()][..., 0] / (1.0 / (1.0 + math.exp(-1.0)))
+    assert torch.equal(name.round().long() - 1, logits.topk(top, dim=1).indices)
+
+
 # ------------------------------------------------------------------------------------------------------
 # configuration and bookkeeping
 # ------------------------------------------------------------------------------------------------------
