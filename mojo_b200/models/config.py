@@ -547,10 +547,10 @@ def noridra(width: int, n_layers: int, heads: int, kv_heads: int, dim: int, voca
     """A Noridra decoder: in every four layers two with the gated delta rule, one with attention inside chunks, one selective
     scan over twice the width; experts in all of them."""
     moe = MoeSpec(experts, top, 1.0, ExpertSpec(expert_ffn))
-    kinds = [lambda: LayerSpec("delta", heads, heads, dim, dim, taps), lambda: LayerSpec("delta", heads, heads, dim, dim, taps),
-             lambda: LayerSpec("attention", heads, kv_heads, dim, dim, scale=dim ** -0.5, softcap=30.0, chunk=chunk),
-             lambda: LayerSpec("mamba1", inner=2 * width, state=state, dt_rank=width // 16, conv_taps=taps)]
-    layers = [kinds[i % 4]() for i in range(n_layers)]
+    kinds = {"delta": lambda: LayerSpec("delta", heads, heads, dim, dim, taps),
+             "mamba1": lambda: LayerSpec("mamba1", inner=2 * width, state=state, dt_rank=width // 16, conv_taps=taps),
+             "attention": lambda: LayerSpec("attention", heads, kv_heads, dim, dim, scale=dim ** -0.5, softcap=30.0, chunk=chunk)}
+    layers = [kinds[("delta", "mamba1", "delta", "attention")[i % 4]]() for i in range(n_layers)]
     for s in layers:
         s.moe = moe
     return ModelConfig(architecture="noridra", hidden_size=width, num_layers=n_layers, num_heads=heads, num_kv_heads=kv_heads, head_dim=dim,
@@ -564,7 +564,7 @@ def noridra_lite() -> ModelConfig:
 
 
 def tiny_noridra() -> ModelConfig:
-    return noridra(256, 4, 4, 2, 64, 1024, 8, 2, 128, 48, positions=2048)
+    return noridra(192, 4, 3, 1, 64, 1024, 6, 2, 112, 48, state=8, groups=3, taps=3, positions=1024)
 
 
 PRESETS = {
